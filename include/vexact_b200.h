@@ -25,7 +25,7 @@
 extern "C" {
 #endif
 
-/* Changes whenever an exported signature changes or an entry point is added (currently 4). */
+/* Changes whenever an exported signature changes or an entry point is added (currently 5). */
 int b200_abi_version(void);
 
 /* Hash of the sources and compiler flags the binary was built from: the Python loader compares it with
@@ -379,6 +379,75 @@ int b200_moe_grouped_wgrad(const void* a, const void* b, void* c, const void* cu
 int b200_moe_unpermute_add_rmsnorm(const void* y, const void* scatter_index, const void* addend,
                                    const void* residual, const void* weight, void* sum_out, void* out,
                                    long long T, int topk, int H, float eps, int mode, void* stream);
+
+/* ---- Operators of the hybrid decoder family (state-space + latent-attention layers, hyper-connections).  No
+ *      counterpart in the reference.  dtype: 0 = bf16, 1 = fp32 ("the model dtype"); *_f32 arguments are always fp32.
+ *      Sequences: query_start_loc [S + 1], context_lens [S] (tokens after the step), state_slots [S] (-1 = none), i32. */
+
+/* b200_gemm_bf16 with an activation in the epilogue, as one product or a batch of them:
+ *   out[g][t, n] = act(sum_k x[g][t, k] * w[g][n, k] + bias[n]).
+ * act: 0 none, 1 the tanh form of gelu, 2 times sigmoid(gate[g][t, n]).  bias only with batch = 1.  w_batch_stride is
+ * a multiple of w_row_stride (at least N rows); strides of x and w are multiples of 8.  out_dtype 0 = bf16, 1 = f32. */
+int b200_gemm_bf16_ex(const void* x, const void* w, const void* bias, const void* gate, void* out, long long T, int N,
+                      int K, int batch, long long x_row_stride, long long x_batch_stride, long long w_row_stride,
+                      long long w_batch_stride, long long out_row_stride, long long out_batch_stride,
+                      long long gate_row_stride, long long gate_batch_stride, int act, int out_dtype, void* stream);
+/* The same in true fp32, every tensor fp32, any strides. */
+int b200_gemm_f32_ex(const void* x, const void* w, const void* bias, const void* gate, void* out, long long T, int N,
+                     int K, int batch, long long x_row_stride, long long x_batch_stride, long long w_row_stride,
+                     long long w_batch_stride, long long out_row_stride, long long out_batch_stride,
+                     long long gate_row_stride, long long gate_batch_stride, int act, void* stream);
+
+/* One sublayer boundary of a hyper-connected residual (streams [num_tokens, num_streams, W] fp32, in place):
+ *   x_t <- sum_s mix[s, t] x_s + m * out[t] * y   (y given), or the streams start as copies of embed[ids] (ids given);
+ *   xn = rms_norm(sum_s in[s] x_s) * (1 + norm_w)  (in NULL = ones; norm_w NULL = no xn), columns W .. xn_cols zero.
+ * rows_i32 (with write_back = 0): only these tokens, num_rows of them; otherwise num_rows = num_tokens.
+ * num_streams 1 .. 8. */
+int b200_hyper_step(void* streams_f32, const void* y, long long y_row_stride, const void* embed, const void* ids_i64,
+                    long long vocab, const void* rows_i32, long long num_tokens, long long num_rows, int num_streams,
+                    int W, const void* mix_f32, const void* out_f32, float m, const void* in_f32,
+                    const void* norm_w_f32, float eps, void* xn, long long xn_row_stride, int xn_cols, int write_back,
+                    int dtype, void* stream);
+
+/* State-space mixer, first step: causal convolution + silu of `channels` columns from conv_off of the projection rows
+ * (act [T, channels]) and dt = softplus(. + dt_bias) of `heads` columns from dt_off.  conv_state [slots, taps - 1,
+ * channels] is read and moved on.  tiled: 0 short portions (one launch), 1 long ones (two launches). */
+int b200_ssm_conv(const void* proj, long long proj_row_stride, int conv_off, int dt_off, int channels, int heads,
+                  int taps, const void* w_f32, const void* bias_f32, const void* dt_bias_f32, void* conv_state,
+                  void* act, void* dt_f32, const void* query_start_loc, const void* context_lens,
+                  const void* state_slots, int num_seqs, int num_slots, long long num_tokens, int tiled, int dtype,
+                  void* stream);
+/* Token-by-token recurrence over act rows [x: heads * P | B: groups * N | C: groups * N]:
+ *   S = exp(-exp(A_log) dt) S + dt B x^T,  y = S^T C + D x;  state [slots, heads, N, P] fp32, y [T, heads * P].
+ * Only sequences with min_len .. max_len tokens in this step.  P a multiple of 8, N <= 512. */
+int b200_ssm_scan(const void* act, long long act_row_stride, const void* dt_f32, const void* A_log_f32,
+                  const void* D_f32, void* state_f32, void* y, const void* query_start_loc, const void* context_lens,
+                  const void* state_slots, int num_seqs, int num_slots, int heads, int groups, int N, int P,
+                  int min_len, int max_len, int dtype, void* stream);
+/* out = rms_norm(y * silu(z)) * w in `parts` equal parts of the heads * p_true true columns; heads are P wide. */
+int b200_ssm_gate_norm(const void* y, long long y_row_stride, const void* z, long long z_row_stride, const void* w_f32,
+                       void* out, long long out_row_stride, long long T, int heads, int P, int p_true, int parts,
+                       float eps, int dtype, void* stream);
+
+/* Latent attention, before the attention call.  proj rows: [q: heads * (DN + DR) | c: R | k_rot: DR | ...].  Stores
+ * rms_norm(c) * c_norm and the rotated k_rot as cache row slot_mapping[t] ([num_slots, R + DR]), rotates the queries in
+ * place (interleaved pairs, the first rot_dims of the DR columns, angle position * inv_freq) and copies their rotated
+ * part into columns R .. of q_lat [T, heads, R + DR] (NULL = not wanted).  DN, DR, R multiples of 8; r_true: columns of
+ * c that are not padding. */
+int b200_latent_prep(void* proj, long long proj_row_stride, const void* positions_i64, const void* slot_mapping_i32,
+                     const void* inv_freq_f32, const void* c_norm_f32, void* cache, void* q_lat, long long T, int heads,
+                     int DN, int DR, int R, int r_true, int rot_dims, float eps, long long num_slots, int dtype,
+                     void* stream);
+/* Absorbed causal attention on CUDA cores: out[t, h] = sum_j softmax(scale * q_lat[t, h] . row_j) row_j[:R] over the
+ * cache rows of the sequence's positions 0 .. own.  Only sequences with min_len .. max_len tokens in this step. */
+int b200_latent_attn_simt(const void* q_lat, const void* cache, void* out, const void* query_start_loc,
+                          const void* context_lens, const void* page_table, long long page_table_stride, int max_pages,
+                          int page_size, int num_blocks, int num_seqs, int min_len, int max_len, long long T, int heads,
+                          int R, int DR, float scale, int dtype, void* stream);
+/* dst row r = cache row of key r - key_start[i] of sequence seq_ids[i], key_start[i] <= r < key_start[i + 1]. */
+int b200_latent_gather(const void* cache, void* dst, const void* seq_ids_i32, const void* key_start_i32, int n,
+                       long long rows, int row_bytes, const void* page_table, long long page_table_stride,
+                       int max_pages, int page_size, int num_blocks, int num_seqs, void* stream);
 
 #ifdef __cplusplus
 }

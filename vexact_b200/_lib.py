@@ -22,6 +22,15 @@ SIGNATURES = {
     "b200_status_read": [C.POINTER(C.c_int), P],
     "b200_gemm_bf16": [P, P, P, P, LL, I, I, LL, LL, LL, I, P],
     "b200_gemm_f16": [P, P, P, P, LL, I, I, LL, LL, LL, I, P],
+    "b200_gemm_bf16_ex": [P, P, P, P, P, LL, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, I, I, P],
+    "b200_gemm_f32_ex": [P, P, P, P, P, LL, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, I, P],
+    "b200_hyper_step": [P, P, LL, P, P, LL, P, LL, LL, I, I, P, P, F, P, P, F, P, LL, I, I, I, P],
+    "b200_ssm_conv": [P, LL, I, I, I, I, I, P, P, P, P, P, P, P, P, P, I, I, LL, I, I, P],
+    "b200_ssm_scan": [P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P],
+    "b200_ssm_gate_norm": [P, LL, P, LL, P, P, LL, LL, I, I, I, I, F, I, P],
+    "b200_latent_prep": [P, LL, P, P, P, P, P, P, LL, I, I, I, I, I, I, F, LL, I, P],
+    "b200_latent_attn_simt": [P, P, P, P, P, P, LL, I, I, I, I, I, I, LL, I, I, I, F, I, P],
+    "b200_latent_gather": [P, P, P, P, I, LL, I, P, LL, I, I, I, I, P],
     "b200_gemm_f32": [P, P, P, P, LL, I, I, LL, LL, LL, P],
     "b200_gemm_f32_from_bf16": [P, P, P, LL, I, I, LL, LL, LL, P],
     "b200_rmsnorm": [P, P, P, LL, I, LL, LL, F, I, P],
@@ -78,7 +87,7 @@ class B200Error(RuntimeError):
     pass
 
 
-ABI_VERSION = 4
+ABI_VERSION = 5
 
 
 def _check_fresh(lib) -> None:
@@ -130,7 +139,7 @@ def load() -> C.CDLL:
 
 
 # Kernels launched by one successful call of each entry point (for launch accounting).
-_KERNELS_PER_CALL = {"b200_moe_permute": 2, "b200_lm_head_greedy": 2, "b200_rmsnorm_backward": 3, "b200_status_read": 0, "b200_abi_version": 0}
+_KERNELS_PER_CALL = {"b200_moe_permute": 2, "b200_lm_head_greedy": 2, "b200_rmsnorm_backward": 3, "b200_ssm_conv2": 2, "b200_status_read": 0, "b200_abi_version": 0}
 _launches = 0
 
 

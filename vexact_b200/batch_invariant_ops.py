@@ -95,6 +95,55 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = No
     return out.reshape(*x.shape[:-1], N)
 
 
+GEMM_ACTS = {None: 0, "gelu_tanh": 1, "sigmoid_gate": 2}
+
+
+def gemm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = None, act: str | None = None,
+         gate: torch.Tensor | None = None, out: torch.Tensor | None = None,
+         out_dtype: torch.dtype | None = None) -> torch.Tensor:
+    """act(x @ weight^T + bias) for bf16 (tcgen05) or fp32 (true fp32) tensors, one product or a batch.
+
+    One product: x [T, K], weight [N, K] -> [T, N].  Batch (3-D weight [B, N, K]): x [T, B, K] -> [T, B, N]; x, `out`
+    and `gate` may be views with any row and batch stride.  act: None, "gelu_tanh", "sigmoid_gate" (times
+    sigmoid(gate), gate shaped like the output)."""
+    _require_cuda("x", x)
+    _require_cuda("weight", weight)
+    assert x.dtype == weight.dtype, "Incompatible dtypes"
+    if x.dtype not in (torch.bfloat16, torch.float32):
+        raise NotImplementedError(f"gemm on {x.dtype}")
+    batched = weight.dim() == 3
+    assert x.dim() == weight.dim() and x.shape[-1] == weight.shape[-1], "Incompatible dimensions"
+    if x.stride(-1) != 1 or weight.stride(-1) != 1 or (bias is not None and (batched or bias.dtype != x.dtype)):
+        raise ValueError("gemm: operands need contiguous rows, a bias needs a single product and the operand dtype")
+    T, K = x.shape[0], x.shape[-1]
+    B, N = (weight.shape[0], weight.shape[1]) if batched else (1, weight.shape[0])
+    out_dtype = out_dtype or x.dtype
+    if out is None:
+        out = torch.empty((T, B, N) if batched else (T, N), device=x.device, dtype=out_dtype)
+    for name, t in (("out", out), ("gate", gate)):
+        if t is not None and (tuple(t.shape) != ((T, B, N) if batched else (T, N)) or t.stride(-1) != 1):
+            raise ValueError(f"gemm: bad {name} shape {tuple(t.shape)}")
+    if gate is not None and gate.dtype != x.dtype:
+        raise ValueError("gemm: the gate has the operand dtype")
+
+    def strides(t):
+        return (0, 0) if t is None else (t.stride(0), t.stride(1) if batched else 0)
+
+    xs, os_, gs = strides(x), strides(out), strides(gate)
+    ws = (weight.stride(-2), weight.stride(0) if batched else 0)
+    args = [x.data_ptr(), weight.data_ptr(), _lib.ptr(bias), _lib.ptr(gate), out.data_ptr(), T, N, K, B, *xs, *ws, *os_,
+            *gs, GEMM_ACTS[act]]
+    if x.dtype == torch.bfloat16:
+        if out.dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError(f"unsupported output dtype {out.dtype}")
+        _lib.check(_lib.load().b200_gemm_bf16_ex(*args, 0 if out.dtype == torch.bfloat16 else 1,
+                                                 _lib.current_stream()), "b200_gemm_bf16_ex")
+    else:
+        assert out.dtype == torch.float32
+        _lib.check(_lib.load().b200_gemm_f32_ex(*args, _lib.current_stream()), "b200_gemm_f32_ex")
+    return out
+
+
 def linear_f32_from_bf16(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
     """`F.linear(x.float(), weight.float())` for bf16 tensors without the fp32 copies (same bits): the
     DeepSeek-V3 router projection (modeling_deepseek_v3.py:97-100)."""

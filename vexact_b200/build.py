@@ -69,15 +69,17 @@ def build(force: bool = False, verbose: bool = False) -> Path:
     want = _source_hash()
     if not force and built_hash() == want:
         return LIB_PATH
-    cmd = [_nvcc(), *NVCC_FLAGS, f'-DB200_SOURCE_HASH="{want}"', "-I", str(CSRC), str(CSRC / "lib.cu"), "-o",
-           str(LIB_PATH)]
+    part = OUT_DIR / f"{LIB_PATH.stem}.{os.getpid()}.part.so"
+    cmd = [_nvcc(), *NVCC_FLAGS, f'-DB200_SOURCE_HASH="{want}"', "-I", str(CSRC), str(CSRC / "lib.cu"), "-o", str(part)]
     if verbose:
         cmd.insert(1, "-Xptxas")
         cmd.insert(2, "-v")
         print(" ".join(cmd), file=sys.stderr)
     res = subprocess.run(cmd, capture_output=True, text=True)
     if res.returncode != 0:
+        part.unlink(missing_ok=True)
         raise RuntimeError(f"nvcc failed:\n{res.stdout}\n{res.stderr}")
+    os.replace(part, LIB_PATH)   # a process that loads the library meanwhile sees the old file or the new one
     if verbose:
         print(res.stderr, file=sys.stderr)
     return LIB_PATH

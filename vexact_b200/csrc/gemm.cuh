@@ -75,6 +75,14 @@ struct GemmParams {
   const __nv_bfloat16* bias;       // [n_w] or null (plain mode)
   const __nv_bfloat16* row_scale;  // [rows] or null (SwiGLU mode: routing weight of each permuted row)
   float4* head_part;               // head mode: [t_rows, w_tiles] per-tile {max, sum exp(x - max), argmax, 0}
+  // Batched plain mode: batch_extra + 1 independent products of one shape.  Product g reads the slice at index g
+  // of a 3-D activation map and weight rows from g * w_rows_per_group, and writes out + g * out_batch_stride.
+  int batch_extra;
+  long long out_batch_stride;
+  // Plain-mode activation of the fp32 accumulator (after the bias), see GEMM_ACT_*.
+  int act;
+  const __nv_bfloat16* gate;       // GEMM_ACT_SIGMOID_GATE: gate[row * gate_stride + g * gate_batch_stride + feature]
+  long long gate_stride, gate_batch_stride;
   uint64_t w_policy;
 };
 
@@ -84,6 +92,20 @@ constexpr int GEMM_SWIGLU = 1;  // gate / up rows stacked on M, out = silu(gate)
 constexpr int GEMM_HEAD = 2;    // lm_head: no logits are stored; per (token, weight tile) the maximum, the sum of
                                 // exp(x - max) and the arg-max of the tile's 128 bf16-rounded logits
 constexpr float kLog2e = 1.4426950408889634f;
+
+// Activations of the plain epilogue, applied in fp32 before the one rounding to the output type.
+constexpr int GEMM_ACT_NONE = 0;
+constexpr int GEMM_ACT_GELU_TANH = 1;     // z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3): the tanh form of gelu
+constexpr int GEMM_ACT_SIGMOID_GATE = 2;  // z * sigmoid(gate)
+
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+  const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return __fdividef(z, 1.f + __expf(fminf(-2.f * u, 80.f)));
+}
+__device__ __forceinline__ float gelu_tanh_exact(float z) {
+  const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return 0.5f * z * (1.f + tanhf(u));
+}
 
 // 2^x on the special-function unit (relative error below 2^-22; results below the normal range flush to zero).
 __device__ __forceinline__ float gemm_ex2(float x) {
@@ -111,7 +133,13 @@ struct GemmTile {
 };
 
 __device__ __forceinline__ bool gemm_tile(const GemmParams& p, int t_tiles, long long linear, GemmTile& t) {
-  if (linear >= (long long)t_tiles * p.w_tiles) return false;
+  const long long per_product = (long long)t_tiles * p.w_tiles;
+  if (linear >= per_product * (1 + p.batch_extra)) return false;
+  int product = 0;
+  if (p.batch_extra) {
+    product = (int)(linear / per_product);
+    linear -= product * per_product;
+  }
   t.wt = (int)(linear / t_tiles);
   const int tt = (int)(linear % t_tiles);
   if (p.tile_table) {
@@ -120,7 +148,7 @@ __device__ __forceinline__ bool gemm_tile(const GemmParams& p, int t_tiles, long
     t.row0 = e.y;
     t.n = e.z;
   } else {
-    t.group = 0;
+    t.group = product;
     t.row0 = tt * p.rows_per_tile;
     t.n = min(p.rows_per_tile, p.t_rows - t.row0);
   }
@@ -192,7 +220,7 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
       if (ptx::elect_one()) {
         const int nbox = (t.n + p.xbox - 1) / p.xbox;
         const uint32_t tx = GEMM_WBYTES + (uint32_t)nbox * p.xbox * (GEMM_BK * 2);
-        const int wrow = t.wt * GEMM_WTILE;
+        const int wrow = t.group * p.w_rows_per_group + t.wt * GEMM_WTILE;
         for (int kb = 0; kb < prefetched; ++kb) {
           ptx::mbar_expect_tx(full_bar(kb), tx * KA);
           for (int a = 0; a < KA; ++a)
@@ -290,9 +318,14 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             } else {
               ptx::tma_load_2d(sw, &tm_w, full_bar(s), kcol, wrow, p.w_policy);
             }
-            for (int b = 0; b < nbox; ++b)
-              ptx::tma_load_2d(sx + (uint32_t)b * p.xbox * (GEMM_BK * 2), &tm_x, full_bar(s), kcol,
-                               t.row0 + b * p.xbox, ptx::kEvictLast);
+            for (int b = 0; b < nbox; ++b) {
+              if (p.batch_extra)
+                ptx::tma_load_3d(sx + (uint32_t)b * p.xbox * (GEMM_BK * 2), &tm_x, full_bar(s), kcol,
+                                 t.row0 + b * p.xbox, t.group, ptx::kEvictLast);
+              else
+                ptx::tma_load_2d(sx + (uint32_t)b * p.xbox * (GEMM_BK * 2), &tm_x, full_bar(s), kcol,
+                                 t.row0 + b * p.xbox, ptx::kEvictLast);
+            }
           }
         }
       }
@@ -448,11 +481,22 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           if (p.fp16) return __half_as_ushort(__float2half_rn(v));
           return __bfloat16_as_ushort(f2bf(v));
         };
+        // activation of one accumulator element of tile column c (row t.row0 + c of the product)
+        const __nv_bfloat16* gate =
+            p.act == GEMM_ACT_SIGMOID_GATE ? p.gate + (long long)t.group * p.gate_batch_stride + f : nullptr;
+        const long long out_base = (long long)t.group * p.out_batch_stride;
+        auto finish = [&](float v, int c) -> float {
+          v += bias;
+          if (p.act == GEMM_ACT_GELU_TANH) v = gelu_tanh_fast(v);
+          if (gate && fvalid && c < t.n)
+            v = __fdividef(v, 1.f + __expf(-bf2f(gate[(long long)(t.row0 + c) * p.gate_stride])));
+          return v;
+        };
         // bf16 output whose rows allow 16-byte stores: each warp turns its 32 features x 16 tokens around in
         // shared memory, so that a lane stores eight consecutive features of one token (16 bytes) and one
         // instruction covers eight token rows, instead of one 2-byte store per (feature, token).
         const bool vec_out = !p.scalar_epilogue && !p.out_f32 && (p.ldo & 7) == 0 && (p.n_w & 7) == 0 &&
-                             (reinterpret_cast<uintptr_t>(p.out) & 15) == 0;
+                             (p.out_batch_stride & 7) == 0 && (reinterpret_cast<uintptr_t>(p.out) & 15) == 0;
         if (vec_out) {
           __nv_bfloat16* stg = exch + q * (16 * 32);      // [16 tokens][32 features] per warp
           const int part = lane & 3, rsub = lane >> 2;
@@ -463,14 +507,14 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             ptx::tmem_ld_wait();
 #pragma unroll
             for (int j = 0; j < 16; ++j)
-              reinterpret_cast<unsigned short*>(stg)[j * 32 + lane] = cvt16(__uint_as_float(r[j]) + bias);
+              reinterpret_cast<unsigned short*>(stg)[j * 32 + lane] = cvt16(finish(__uint_as_float(r[j]), c0 + j));
             __syncwarp();
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
               const int row = h * 8 + rsub, c = c0 + row;
               const uint4 v = *reinterpret_cast<const uint4*>(stg + row * 32 + part * 8);
               if (c < t.n && f8 < p.n_w)
-                *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(p.out) + (long long)(t.row0 + c) * p.ldo + f8) = v;
+                *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(p.out) + out_base + (long long)(t.row0 + c) * p.ldo + f8) = v;
             }
             __syncwarp();
           }
@@ -484,8 +528,8 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             for (int j = 0; j < 16; ++j) {
               const int c = c0 + j;
               if (c < t.n) {
-                const float v = __uint_as_float(r[j]) + bias;
-                const long long o = (long long)(t.row0 + c) * p.ldo + f;
+                const float v = finish(__uint_as_float(r[j]), c);
+                const long long o = out_base + (long long)(t.row0 + c) * p.ldo + f;
                 if (p.out_f32)
                   reinterpret_cast<float*>(p.out)[o] = v;
                 else
@@ -574,6 +618,24 @@ inline int make_tmap_2d(CUtensorMap* m, const void* base, uint64_t rows, uint64_
   return r == CUDA_SUCCESS ? B200_OK : B200_ERR_DRIVER;
 }
 
+// 3-D bf16 tensor [batch, rows, cols]; box = 64 cols x box_rows of one batch entry, 128-byte swizzle.
+inline int make_tmap_3d(CUtensorMap* m, const void* base, uint64_t batch, uint64_t rows, uint64_t cols,
+                        uint64_t batch_stride, uint64_t row_stride, uint32_t box_rows) {
+  EncodeTiledFn enc = tensor_map_encoder();
+  if (!enc) return B200_ERR_DRIVER;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || (row_stride * 2) % 16 || (batch_stride * 2) % 16 || box_rows == 0 ||
+      box_rows > 256)
+    return B200_ERR_ARG;
+  cuuint64_t dims[3] = {cols, rows, batch};
+  cuuint64_t strides[2] = {row_stride * 2, batch_stride * 2};
+  cuuint32_t box[3] = {(cuuint32_t)GEMM_BK, box_rows, 1};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
+                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? B200_OK : B200_ERR_DRIVER;
+}
+
 inline int round_up(int v, int m) { return (v + m - 1) / m * m; }
 
 // Development knobs (unset in normal use): B200_GEMM_XBOX = rows per activation box of the grouped
@@ -654,6 +716,83 @@ gemm_f32_kernel(const TIn* __restrict__ x, const TIn* __restrict__ w, const floa
 }
 }  // namespace b200
 
+namespace b200 {
+// True-fp32 GEMM for models that run in fp32: 64 x 64 output tile per CTA, 4 x 4 outputs per thread, K walked in
+// ascending steps of 16 through shared memory, plain fp32 FMA (no tensor cores, no reduced-precision mode).
+// blockIdx.z picks one product of the batch.
+__global__ void __launch_bounds__(256)
+gemm_f32_tiled_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias,
+                      const float* __restrict__ gate, float* __restrict__ out, long long T, int N, int K,
+                      long long x_row, long long x_batch, long long w_row, long long w_batch, long long out_row,
+                      long long out_batch, long long gate_row, long long gate_batch, int act) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float sx[16][68], sw[16][68];
+  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  const long long t0 = (long long)blockIdx.x * 64;
+  const int n0 = blockIdx.y * 64;
+  x += (long long)blockIdx.z * x_batch;
+  w += (long long)blockIdx.z * w_batch;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += 16) {
+    for (int e = tid; e < 64 * 16; e += 256) {
+      const int r = e >> 4, k = e & 15;
+      sx[k][r] = t0 + r < T && k0 + k < K ? x[(t0 + r) * x_row + k0 + k] : 0.f;
+      sw[k][r] = n0 + r < N && k0 + k < K ? w[(long long)(n0 + r) * w_row + k0 + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      float a[4], b[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        a[i] = sx[k][ty * 4 + i];
+        b[i] = sw[k][tx + 16 * i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const long long t = t0 + ty * 4 + i;
+    if (t >= T) break;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx + 16 * j;
+      if (n >= N) continue;
+      float v = acc[i][j] + (bias ? bias[n] : 0.f);
+      if (act == GEMM_ACT_GELU_TANH) v = gelu_tanh_exact(v);
+      if (act == GEMM_ACT_SIGMOID_GATE)
+        v = v / (1.f + expf(-gate[t * gate_row + (long long)blockIdx.z * gate_batch + n]));
+      out[t * out_row + (long long)blockIdx.z * out_batch + n] = v;
+    }
+  }
+}
+}  // namespace b200
+
+// b200_gemm_bf16_ex in true fp32 (all tensors fp32).
+extern "C" int b200_gemm_f32_ex(const void* x, const void* w, const void* bias, const void* gate, void* out,
+                                long long T, int N, int K, int batch, long long x_row_stride,
+                                long long x_batch_stride, long long w_row_stride, long long w_batch_stride,
+                                long long out_row_stride, long long out_batch_stride, long long gate_row_stride,
+                                long long gate_batch_stride, int act, void* stream) {
+  using namespace b200;
+  if (!x || !w || !out || T < 0 || N <= 0 || K <= 0 || batch < 1) return B200_ERR_ARG;
+  if (act < GEMM_ACT_NONE || act > GEMM_ACT_SIGMOID_GATE) return B200_ERR_ARG;
+  if ((act == GEMM_ACT_SIGMOID_GATE) != (gate != nullptr) || (batch > 1 && bias)) return B200_ERR_ARG;
+  if (T == 0) return B200_OK;
+  if ((T + 63) / 64 > 0x7fffffffLL || (N + 63) / 64 > 65535 || batch > 65535) return B200_ERR_SHAPE;
+  launch_k(gemm_f32_tiled_kernel, dim3((unsigned)((T + 63) / 64), (unsigned)((N + 63) / 64), (unsigned)batch), dim3(256),
+           0, (cudaStream_t)stream, (const float*)x, (const float*)w, (const float*)bias, (const float*)gate,
+           (float*)out, T, N, K, x_row_stride, x_batch_stride, w_row_stride, w_batch_stride, out_row_stride,
+           out_batch_stride, gate_row_stride, gate_batch_stride, act);
+  return launch_status();
+}
+
 extern "C" int b200_gemm_f32(const void* x, const void* w, const void* bias, void* out, long long T, int N,
                              int K, long long x_row_stride, long long w_row_stride, long long out_row_stride,
                              void* stream) {
@@ -686,9 +825,18 @@ extern "C" int b200_gemm_f32_from_bf16(const void* x, const void* w, void* out, 
 // out[T, N] = x[T, K] @ w[N, K]^T (+ bias[N], added in fp32 before the cast).
 // x rows are `x_row_stride` elements apart, w rows `w_row_stride`, out rows `out_row_stride`.
 namespace b200 {
+// What the plain dense form can do beyond one product: an activation, a batch of products.
+struct GemmExtra {
+  int act = GEMM_ACT_NONE;
+  const void* gate = nullptr;
+  long long gate_row_stride = 0, gate_batch_stride = 0;
+  int batch = 1;
+  long long x_batch_stride = 0, w_batch_stride = 0, out_batch_stride = 0;
+};
+
 inline int gemm_dense_16bit(const void* x, const void* w, const void* bias, void* out, long long T, int N, int K,
                             long long x_row_stride, long long w_row_stride, long long out_row_stride, int out_dtype,
-                            bool fp16, void* stream) {
+                            bool fp16, void* stream, const GemmExtra& ex = GemmExtra()) {
   if (!x || !w || !out || T < 0 || N <= 0 || K <= 0 || (out_dtype != 0 && out_dtype != 1)) return B200_ERR_ARG;
   if (K % 8 != 0 || x_row_stride % 8 != 0 || w_row_stride % 8 != 0) return B200_ERR_SHAPE;
   if (T == 0) return B200_OK;
@@ -712,7 +860,7 @@ inline int gemm_dense_16bit(const void* x, const void* w, const void* bias, void
     for (int tt = min_tiles; tt <= max_tiles; ++tt) {
       const int rows = round_up((int)((T + tt - 1) / tt), 16);
       const int tiles_t = (int)((T + rows - 1) / rows);
-      const long long rounds = ((long long)tiles_t * p.w_tiles + sms - 1) / sms;
+      const long long rounds = ((long long)tiles_t * p.w_tiles * ex.batch + sms - 1) / sms;
       const long long cost = rounds * (GEMM_WBYTES + rows * GEMM_BK * 2);
       if (best_cost < 0 || cost < best_cost) {
         best_cost = cost;
@@ -732,12 +880,31 @@ inline int gemm_dense_16bit(const void* x, const void* w, const void* bias, void
   p.row_scale = nullptr;
   p.w_policy = p.dense_t_tiles == 1 ? ptx::kEvictFirst : ptx::kEvictNormal;
   p.fp16 = fp16 ? 1 : 0;
+  p.act = ex.act;
+  p.gate = (const __nv_bfloat16*)ex.gate;
+  p.gate_stride = ex.gate_row_stride;
+  p.gate_batch_stride = ex.gate_batch_stride;
   CUtensorMap tw, tx;
-  int rc = make_tmap_2d(&tw, w, (uint64_t)N, (uint64_t)K, (uint64_t)w_row_stride, GEMM_WTILE, fp16);
+  int rc;
+  if (ex.batch > 1) {
+    // the weights of all products form one 2-D view of whole rows, the activations a 3-D view [batch, T, K]
+    if (ex.w_batch_stride % w_row_stride != 0 || ex.x_batch_stride % 8 != 0 || ex.w_batch_stride < w_row_stride * N)
+      return B200_ERR_SHAPE;
+    p.batch_extra = ex.batch - 1;
+    p.out_batch_stride = ex.out_batch_stride;
+    p.w_rows_per_group = (int)(ex.w_batch_stride / w_row_stride);
+    rc = make_tmap_2d(&tw, w, (uint64_t)p.w_rows_per_group * (ex.batch - 1) + N, (uint64_t)K, (uint64_t)w_row_stride,
+                      GEMM_WTILE);
+    if (rc) return rc;
+    rc = make_tmap_3d(&tx, x, (uint64_t)ex.batch, (uint64_t)T, (uint64_t)K, (uint64_t)ex.x_batch_stride,
+                      (uint64_t)x_row_stride, (uint32_t)p.xbox);
+  } else {
+    rc = make_tmap_2d(&tw, w, (uint64_t)N, (uint64_t)K, (uint64_t)w_row_stride, GEMM_WTILE, fp16);
+    if (rc) return rc;
+    rc = make_tmap_2d(&tx, x, (uint64_t)T, (uint64_t)K, (uint64_t)x_row_stride, (uint32_t)p.xbox, fp16);
+  }
   if (rc) return rc;
-  rc = make_tmap_2d(&tx, x, (uint64_t)T, (uint64_t)K, (uint64_t)x_row_stride, (uint32_t)p.xbox, fp16);
-  if (rc) return rc;
-  return gemm_launch<GEMM_PLAIN>(tw, tx, p, (long long)p.w_tiles * p.dense_t_tiles, (cudaStream_t)stream);
+  return gemm_launch<GEMM_PLAIN>(tw, tx, p, (long long)p.w_tiles * p.dense_t_tiles * ex.batch, (cudaStream_t)stream);
 }
 }  // namespace b200
 
@@ -746,6 +913,30 @@ extern "C" int b200_gemm_bf16(const void* x, const void* w, const void* bias, vo
                               int out_dtype /*0 = bf16, 1 = f32*/, void* stream) {
   return b200::gemm_dense_16bit(x, w, bias, out, T, N, K, x_row_stride, w_row_stride, out_row_stride, out_dtype, false,
                                 stream);
+}
+
+// The bf16 GEMM with an activation in its epilogue and / or as a batch of products (no bias then):
+//   out[g][t, n] = act(sum_k x[g][t, k] * w[g][n, k] + bias[n]),  g < batch
+// A product's arithmetic is that of b200_gemm_bf16 on its slices.
+extern "C" int b200_gemm_bf16_ex(const void* x, const void* w, const void* bias, const void* gate, void* out,
+                                 long long T, int N, int K, int batch, long long x_row_stride,
+                                 long long x_batch_stride, long long w_row_stride, long long w_batch_stride,
+                                 long long out_row_stride, long long out_batch_stride, long long gate_row_stride,
+                                 long long gate_batch_stride, int act, int out_dtype, void* stream) {
+  using namespace b200;
+  if (batch < 1 || act < GEMM_ACT_NONE || act > GEMM_ACT_SIGMOID_GATE) return B200_ERR_ARG;
+  if ((act == GEMM_ACT_SIGMOID_GATE) != (gate != nullptr) || (batch > 1 && bias)) return B200_ERR_ARG;
+  GemmExtra ex;
+  ex.act = act;
+  ex.gate = gate;
+  ex.gate_row_stride = gate_row_stride;
+  ex.gate_batch_stride = gate_batch_stride;
+  ex.batch = batch;
+  ex.x_batch_stride = x_batch_stride;
+  ex.w_batch_stride = w_batch_stride;
+  ex.out_batch_stride = out_batch_stride;
+  return gemm_dense_16bit(x, w, bias, out, T, N, K, x_row_stride, w_row_stride, out_row_stride, out_dtype, false,
+                          stream, ex);
 }
 
 // The same GEMM on fp16 tensors (the reference's matmul_persistent serves bf16, fp16 and fp32,

@@ -1,0 +1,302 @@
+// Latent attention over a paged cache that holds, per token, only the normed latent c and one rotated key part shared
+// by all heads: cache row = [c: R | k_rot: DR].
+//
+// A head's unrotated key is W_uk c and its value W_uv c, so with q' = W_uk^T q (one small product per head)
+//     score = (q' . c + q_rot . k_rot) * scale,      head output = W_uv (sum_j p_j c_j),
+// and attention runs as one KV head of width R + DR whose value is the first R columns of the key ("absorbed" form).
+//
+//   latent_prep_kernel    between the in-projection and attention: norms and stores c, rotates and stores k_rot,
+//                         rotates q in place and copies its rotated part behind q'.
+//   latent_attn_simt_kernel   absorbed attention on CUDA cores, any dims, fp32 or bf16 storage: the fp32 path and the
+//                         cross-check of the tensor-core kernels (latent_mma.cuh).
+//   latent_gather_kernel  the latents of whole sequences, gathered from their pages into packed rows (what the
+//                         expanded form of long prompts projects up).
+#pragma once
+#include "hyper.cuh"   // load4 / store4 / to_f32 / from_f32
+
+namespace b200 {
+
+struct LatentPrepParams {
+  void* proj;                // [T, proj_stride]: [q: H * (DN + DR) | c: R | k_rot: DR | ...]; q is rotated in place
+  long long proj_stride;
+  const long long* positions;
+  const int* slot_mapping;   // -1 = do not store
+  const float* inv_freq;     // [rot_dims / 2]
+  const float* c_norm;       // [R], plain weight (zero in padding columns)
+  void* cache;               // [num_slots, R + DR]
+  void* q_lat;               // [T, H, R + DR]: columns R .. R + DR are written here, or null
+  int heads, DN, DR, R;
+  int r_true;                // columns of c that exist (the rest is padding and zero)
+  int rot_dims;
+  float eps;
+  long long num_slots;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams p) {
+  __shared__ float red[32];
+  __shared__ float s_cos[128], s_sin[128];
+  pdl_trigger();
+  pdl_wait();
+  const long long t = blockIdx.x;
+  const int tid = threadIdx.x;
+  const float pos = (float)p.positions[t];
+  const int half = p.rot_dims >> 1;
+  for (int i = tid; i < half; i += 128) sincosf(pos * p.inv_freq[i], &s_sin[i], &s_cos[i]);
+  T* row = reinterpret_cast<T*>(p.proj) + t * p.proj_stride;
+  const int dq = p.DN + p.DR, dc = p.R + p.DR;
+  const T* c = row + p.heads * dq;
+  float ss = 0.f;
+  for (int i = tid * 4; i < p.R; i += 512) {
+    float v[4];
+    load4(c + i, v);   // padding columns hold zeros
+#pragma unroll
+    for (int k = 0; k < 4; ++k) ss = fmaf(v[k], v[k], ss);
+  }
+  ss = block_sum(ss, red);   // (its barriers also publish the sine table)
+  const float inv = 1.f / sqrtf(ss / (float)p.r_true + p.eps);
+  const long long slot = p.slot_mapping[t];
+  if (slot >= p.num_slots && tid == 0) report_status(B200_STATUS_BAD_INDEX, (int)slot);
+  if (slot >= 0 && slot < p.num_slots) {
+    T* dst = reinterpret_cast<T*>(p.cache) + slot * dc;
+    for (int i = tid * 4; i < p.R; i += 512) {
+      float v[4], w[4];
+      load4(c + i, v);
+      load4(p.c_norm + i, w);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[k] = v[k] * inv * w[k];
+      store4(dst + i, v);
+    }
+    const T* kr = c + p.R;
+    for (int i = tid; i < (p.DR >> 1); i += 128) {
+      float u = to_f32(kr[2 * i]), v = to_f32(kr[2 * i + 1]);
+      if (i < half) {
+        const float a = u * s_cos[i] - v * s_sin[i];
+        v = v * s_cos[i] + u * s_sin[i];
+        u = a;
+      }
+      dst[p.R + 2 * i] = from_f32<T>(u);
+      dst[p.R + 2 * i + 1] = from_f32<T>(v);
+    }
+  }
+  const int pairs = p.DR >> 1;
+  for (int e = tid; e < p.heads * pairs; e += 128) {
+    const int h = e / pairs, i = e - h * pairs;
+    T* q = row + h * dq + p.DN + 2 * i;
+    float u = to_f32(q[0]), v = to_f32(q[1]);
+    if (i < half) {
+      const float a = u * s_cos[i] - v * s_sin[i];
+      v = v * s_cos[i] + u * s_sin[i];
+      u = a;
+      q[0] = from_f32<T>(u);
+      q[1] = from_f32<T>(v);
+    }
+    if (p.q_lat) {
+      T* d = reinterpret_cast<T*>(p.q_lat) + (t * p.heads + h) * dc + p.R + 2 * i;
+      d[0] = from_f32<T>(u);
+      d[1] = from_f32<T>(v);
+    }
+  }
+}
+
+// Sequences and pages of a step, as every latent kernel reads them.
+struct LatentSeqs {
+  const int* query_start_loc;   // [S + 1]
+  const int* context_lens;      // [S]
+  const int* page_table;        // [S, page_table_stride]
+  long long page_table_stride;
+  int max_pages, page_size, num_blocks, num_seqs;
+  int min_len, max_len;         // only sequences whose step brings min_len .. max_len tokens
+};
+
+// Row of key j of sequence s in the cache, or -1 (reported) for a page id out of range.
+__device__ __forceinline__ long long latent_key_row(const LatentSeqs& q, int s, int j) {
+  const int pg = j / q.page_size;
+  const int blk = pg < q.max_pages ? q.page_table[(long long)s * q.page_table_stride + pg] : -1;
+  if (blk < 0 || blk >= q.num_blocks) {
+    report_status(B200_STATUS_BAD_INDEX, blk);
+    return -1;
+  }
+  return (long long)blk * q.page_size + (j - pg * q.page_size);
+}
+
+// Index of the sequence that packed token t belongs to.
+__device__ __forceinline__ int latent_seq_of(const int* query_start_loc, int num_seqs, long long t) {
+  int lo = 0, hi = num_seqs - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (query_start_loc[mid] <= t) lo = mid;
+    else hi = mid - 1;
+  }
+  return lo;
+}
+
+struct LatentAttnParams {
+  LatentSeqs seqs;
+  const void* q_lat;   // [T, H, R + DR]
+  const void* cache;   // [num_blocks * page_size, R + DR]
+  void* out;           // [T, H, R]
+  int heads, R, DR;
+  float scale;
+};
+
+constexpr int LATENT_SIMT_THREADS = 128;
+constexpr int LATENT_SIMT_VPT = 8;   // value columns per thread: R <= 1024
+
+template <typename T>
+__global__ void __launch_bounds__(LATENT_SIMT_THREADS) latent_attn_simt_kernel(const LatentAttnParams p) {
+  extern __shared__ float lat_smem[];   // q [R + DR]
+  __shared__ float red[32];
+  __shared__ float s_p[LATENT_SIMT_THREADS];
+  __shared__ long long s_row[LATENT_SIMT_THREADS];
+  __shared__ int s_seq;
+  pdl_trigger();
+  pdl_wait();
+  const int h = blockIdx.y, tid = threadIdx.x;
+  const long long t = blockIdx.x;
+  if (tid == 0) s_seq = latent_seq_of(p.seqs.query_start_loc, p.seqs.num_seqs, t);
+  __syncthreads();
+  const int s = s_seq;
+  const int t0 = p.seqs.query_start_loc[s], len = p.seqs.query_start_loc[s + 1] - t0;
+  if (t < t0 || t >= t0 + len || len < p.seqs.min_len || len > p.seqs.max_len) return;
+  const int keys = p.seqs.context_lens[s] - len + (int)(t - t0) + 1;   // visible keys: positions 0 .. own
+  const int dc = p.R + p.DR;
+  const T* q = reinterpret_cast<const T*>(p.q_lat) + (t * p.heads + h) * dc;
+  for (int i = tid; i < dc; i += LATENT_SIMT_THREADS) lat_smem[i] = to_f32(q[i]) * p.scale;
+  float acc[LATENT_SIMT_VPT];
+#pragma unroll
+  for (int v = 0; v < LATENT_SIMT_VPT; ++v) acc[v] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  const T* cache = reinterpret_cast<const T*>(p.cache);
+  for (int b = 0; b < keys; b += LATENT_SIMT_THREADS) {
+    const int n = min(LATENT_SIMT_THREADS, keys - b);
+    __syncthreads();
+    long long row = tid < n ? latent_key_row(p.seqs, s, b + tid) : -1;
+    s_row[tid] = row;
+    float sc = -INFINITY;
+    if (row >= 0) {
+      const T* k = cache + row * dc;
+      float a = 0.f;
+      for (int i = 0; i < dc; i += 4) {
+        float v[4];
+        load4(k + i, v);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) a = fmaf(lat_smem[i + u], v[u], a);
+      }
+      sc = a;
+    }
+    const float bm = fmaxf(m, block_max(sc, red));
+    const float e = sc == -INFINITY ? 0.f : expf(sc - bm);
+    s_p[tid] = e;
+    const float alpha = m == -INFINITY ? 0.f : expf(m - bm);
+    l = l * alpha + block_sum(e, red);
+    m = bm;
+    __syncthreads();
+#pragma unroll
+    for (int v = 0; v < LATENT_SIMT_VPT; ++v) {
+      const int c = v * LATENT_SIMT_THREADS + tid;
+      if (c < p.R) {
+        float a = acc[v] * alpha;
+        for (int j = 0; j < n; ++j)
+          if (s_row[j] >= 0) a = fmaf(s_p[j], to_f32(cache[s_row[j] * dc + c]), a);
+        acc[v] = a;
+      }
+    }
+  }
+  T* out = reinterpret_cast<T*>(p.out) + (t * p.heads + h) * (long long)p.R;
+#pragma unroll
+  for (int v = 0; v < LATENT_SIMT_VPT; ++v) {
+    const int c = v * LATENT_SIMT_THREADS + tid;
+    if (c < p.R) out[c] = from_f32<T>(l > 0.f ? acc[v] / l : 0.f);
+  }
+}
+
+// dst row r = cache row of key (r - key_start[i]) of sequence seq_ids[i], for the i that key_start brackets.
+struct LatentGatherParams {
+  LatentSeqs seqs;
+  const uint4* cache;
+  uint4* dst;
+  const int* seq_ids;     // [n]
+  const int* key_start;   // [n + 1] packed start of each gathered sequence
+  int n, vecs;            // 16-byte vectors per row
+};
+
+__global__ void __launch_bounds__(256) latent_gather_kernel(const LatentGatherParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long r = (long long)blockIdx.x * 8 + warp;
+  if (r >= p.key_start[p.n]) return;
+  const int i = latent_seq_of(p.key_start, p.n, r);
+  const long long row = latent_key_row(p.seqs, p.seq_ids[i], (int)(r - p.key_start[i]));
+  for (int v = lane; v < p.vecs; v += 32)
+    p.dst[r * p.vecs + v] = row >= 0 ? p.cache[row * p.vecs + v] : make_uint4(0, 0, 0, 0);
+}
+
+}  // namespace b200
+
+extern "C" int b200_latent_prep(void* proj, long long proj_row_stride, const void* positions_i64,
+                                const void* slot_mapping_i32, const void* inv_freq_f32, const void* c_norm_f32,
+                                void* cache, void* q_lat, long long T, int heads, int DN, int DR, int R, int r_true,
+                                int rot_dims, float eps, long long num_slots, int dtype, void* stream) {
+  using namespace b200;
+  if (!proj || !positions_i64 || !slot_mapping_i32 || !inv_freq_f32 || !c_norm_f32 || !cache || T < 0 || heads <= 0 ||
+      DN < 0 || DR < 0 || R <= 0 || r_true <= 0 || r_true > R || rot_dims < 0 || rot_dims > DR || (dtype != 0 && dtype != 1))
+    return B200_ERR_ARG;
+  if (DN % 8 || DR % 8 || R % 8 || proj_row_stride % 8 || rot_dims % 2 || rot_dims > 256 || T > 0x7fffffffLL)
+    return B200_ERR_SHAPE;
+  if (T == 0) return B200_OK;
+  LatentPrepParams p{proj, proj_row_stride, (const long long*)positions_i64, (const int*)slot_mapping_i32,
+                     (const float*)inv_freq_f32, (const float*)c_norm_f32, cache, q_lat, heads, DN, DR, R, r_true,
+                     rot_dims, eps, num_slots};
+  if (dtype == 0) launch_k(latent_prep_kernel<__nv_bfloat16>, dim3((unsigned)T), dim3(128), 0, (cudaStream_t)stream, p);
+  else launch_k(latent_prep_kernel<float>, dim3((unsigned)T), dim3(128), 0, (cudaStream_t)stream, p);
+  return launch_status();
+}
+
+namespace b200 {
+inline bool latent_seqs_ok(const LatentSeqs& q) {
+  return q.query_start_loc && q.context_lens && q.page_table && q.num_seqs > 0 && q.page_size > 0 && q.max_pages > 0 &&
+         q.num_blocks > 0;
+}
+}  // namespace b200
+
+extern "C" int b200_latent_attn_simt(const void* q_lat, const void* cache, void* out, const void* query_start_loc,
+                                     const void* context_lens, const void* page_table, long long page_table_stride,
+                                     int max_pages, int page_size, int num_blocks, int num_seqs, int min_len,
+                                     int max_len, long long T, int heads, int R, int DR, float scale, int dtype,
+                                     void* stream) {
+  using namespace b200;
+  LatentAttnParams p{{(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride,
+                      max_pages, page_size, num_blocks, num_seqs, min_len, max_len},
+                     q_lat, cache, out, heads, R, DR, scale};
+  if (!latent_seqs_ok(p.seqs) || !q_lat || !cache || !out || T < 0 || heads <= 0 || R <= 0 || DR < 0 ||
+      (dtype != 0 && dtype != 1))
+    return B200_ERR_ARG;
+  if (R % 8 || DR % 8 || R > LATENT_SIMT_THREADS * LATENT_SIMT_VPT || R + DR > 8192 || T > 0x7fffffffLL) return B200_ERR_SHAPE;
+  if (T == 0) return B200_OK;
+  const size_t smem = (size_t)(R + DR) * sizeof(float);
+  const dim3 grid((unsigned)T, (unsigned)heads);
+  if (dtype == 0)
+    launch_k(latent_attn_simt_kernel<__nv_bfloat16>, grid, dim3(LATENT_SIMT_THREADS), smem, (cudaStream_t)stream, p);
+  else
+    launch_k(latent_attn_simt_kernel<float>, grid, dim3(LATENT_SIMT_THREADS), smem, (cudaStream_t)stream, p);
+  return launch_status();
+}
+
+extern "C" int b200_latent_gather(const void* cache, void* dst, const void* seq_ids_i32, const void* key_start_i32, int n,
+                                  long long rows, int row_bytes, const void* page_table, long long page_table_stride,
+                                  int max_pages, int page_size, int num_blocks, int num_seqs, void* stream) {
+  using namespace b200;
+  if (!cache || !dst || !seq_ids_i32 || !key_start_i32 || !page_table || n <= 0 || rows < 0 || page_size <= 0 ||
+      max_pages <= 0 || num_blocks <= 0 || num_seqs <= 0)
+    return B200_ERR_ARG;
+  if (row_bytes % 16 || row_bytes <= 0 || rows > 0x7fffffffLL) return B200_ERR_SHAPE;
+  if (rows == 0) return B200_OK;
+  LatentGatherParams p{{nullptr, nullptr, (const int*)page_table, page_table_stride, max_pages, page_size, num_blocks,
+                        num_seqs, 0, 0},
+                       (const uint4*)cache, (uint4*)dst, (const int*)seq_ids_i32, (const int*)key_start_i32, n,
+                       row_bytes / 16};
+  launch_k(latent_gather_kernel, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, p);
+  return launch_status();
+}

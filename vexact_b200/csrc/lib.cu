@@ -12,6 +12,9 @@
 #include "noalloc.cuh"
 #include "step.cuh"
 #include "sample.cuh"
+#include "hyper.cuh"
+#include "ssm.cuh"
+#include "latent.cuh"
 
 // Self-test of the bounded wait every kernel here relies on: one CTA waits, with a limit of
 // `limit_us` microseconds, on an mbarrier that nothing ever completes.  The wait must give up, record
@@ -58,7 +61,7 @@ extern "C" int b200_status_read(int* host_out4, void* stream) {
 }
 
 // Bumped whenever an exported signature changes.
-extern "C" int b200_abi_version(void) { return 4; }
+extern "C" int b200_abi_version(void) { return 5; }
 
 // Hash of the sources and compiler flags this binary was built from (set by the build script);
 // the loader compares it with the sources beside it and refuses a stale library.

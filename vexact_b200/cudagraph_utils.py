@@ -39,7 +39,9 @@ class BatchExecutionDescriptor:
 
 class CudaGraphManager:
     def __init__(self, model: Callable, device, input_buffers: InputBuffers, cache_config, cache_store: KVCacheStore,
-                 max_size: int, pool: Any = None, forward_kwargs: Optional[dict] = None):
+                 max_size: int, pool: Any = None, forward_kwargs: Optional[dict] = None, decode_only: bool = False):
+        """decode_only: capture the pure-decode graphs alone (a model whose prompt steps are shaped by host-side
+        lengths runs those eagerly; `dispatch` then returns None for them)."""
         self.model = model
         self.device = torch.device(device)
         self.cache_config = cache_config
@@ -51,7 +53,7 @@ class CudaGraphManager:
         self.forward_kwargs = forward_kwargs or {}
         self.input_buffers = input_buffers
         self._descriptors = [BatchExecutionDescriptor(num_tokens=n, num_seqs=min(n, input_buffers.max_num_seqs))
-                             for n in self.capture_sizes]
+                             for n in self.capture_sizes] if not decode_only else []
         self._decode_descriptors = [BatchExecutionDescriptor(num_tokens=n, num_seqs=n, decode=True)
                                     for n in self.capture_sizes if n <= input_buffers.max_num_seqs]
 
@@ -117,10 +119,14 @@ class CudaGraphManager:
         query_start_loc[0].zero_()
         query_start_loc[1:].copy_(per_seq.cumsum(0))
         context_lens.copy_(per_seq)
+        recurrent = {}
+        if hasattr(self.cache_store, "num_state_slots"):
+            buf.state_slots.gpu.fill_(-1)          # nor any recurrent state
+            recurrent = dict(cache_store=self.cache_store, state_slots=buf.state_slots.gpu[:num_seqs])
         set_kv_cache_context(is_paged_attn=True, key_cache=self.cache_store.key_cache,
                              value_cache=self.cache_store.value_cache, block_tables=block_tables,
                              context_lens=context_lens, slot_mapping=slot_mapping, query_start_loc=query_start_loc,
-                             max_seqlen_q=1 if desc.decode else tokens)
+                             max_seqlen_q=1 if desc.decode else tokens, **recurrent)
         # warm-up outside the capture (lazy one-time set-up: attributes, tensor-map encoder lookup)
         self.model(**static_inputs, **self.forward_kwargs)
         graph = torch.cuda.CUDAGraph()

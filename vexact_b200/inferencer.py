@@ -675,8 +675,12 @@ class Inferencer:
         self.use_fp32_logits = bool(getattr(config.model, "use_fp32_logits", False))
         self.page_size = self.cache_config.page_size
         hf_config = config.model.hf_config
-        self.cache_store = KVCacheStore(hf_config, self.cache_config, self.device,
-                                        layer_ids=getattr(model, "layer_ids", None))
+        make_store = getattr(model, "make_cache_store", None)   # models whose caches are not per-head K / V pages
+        if make_store is not None:
+            self.cache_store = make_store(self.cache_config, config.scheduler.max_num_seqs, self.device)
+        else:
+            self.cache_store = KVCacheStore(hf_config, self.cache_config, self.device,
+                                            layer_ids=getattr(model, "layer_ids", None))
         if enable_batch_invariant and not is_batch_invariant_mode_enabled():
             enable_batch_invariant_mode()
         self.input_buffers = InputBuffers(
@@ -693,13 +697,18 @@ class Inferencer:
                                              buffers=self.input_buffers)
         self._rows: list = []          # per batch row: (request_id, blocks uploaded so far)
         self._cudagraph_mgr: Optional[CudaGraphManager] = None
+        # such a model runs its prompt steps eagerly (their launches are shaped by host-side lengths)
+        self._decode_graphs_only = bool(getattr(model, "decode_graphs_only", False))
+        self._recurrent = hasattr(self.cache_store, "num_state_slots")
+        self._logit_rows = None        # packed rows whose logits this step returns (None: each request's last token)
         if not getattr(config.model, "enforce_eager", False):
             if getattr(config.model, "attn_impl", "fa-invariant") == "flex":
                 raise RuntimeError("Cuda graph is enabled but flex attention is not supported for CUDA graph replay.")
             self._cudagraph_mgr = CudaGraphManager(
                 model=self.model, device=self.device, cache_store=self.cache_store,
                 max_size=config.scheduler.max_num_batched_tokens, cache_config=self.cache_config,
-                forward_kwargs=self.forward_kwargs, input_buffers=self.input_buffers)
+                forward_kwargs=self.forward_kwargs, input_buffers=self.input_buffers,
+                decode_only=self._decode_graphs_only)
             self._cudagraph_mgr.capture_graphs()
 
     # ------------------------------------------------------------------ one scheduler step
@@ -743,6 +752,29 @@ class Inferencer:
                 slot_mapping=gen_ctx.slot_mapping, max_seqlen_q=gen_ctx.max_seqlen_q,
                 generation_configs=gen_ctx.generation_configs, tokens_generated=gen_ctx.tokens_generated))
         return final_output
+
+    def infer_logits(self, requests, positions) -> Optional[torch.Tensor]:
+        """One step of the same forward that returns logits instead of tokens: `positions[i]` lists the places, among
+        request i's tokens of this step, whose logits are wanted.  [wanted, vocab] in the order of the requests, or
+        None when nothing is wanted.  Single-stage models only."""
+        if not (self._pp_info.is_first_rank and self._pp_info.is_last_rank):
+            raise NotImplementedError("infer_logits runs on a single pipeline stage")
+        rows, start = [], 0
+        for req, want in zip(requests, positions):
+            rows += [start + w for w in want]
+            start += req.tokens_this_step
+        one_each = start == len(requests)
+        # a decode step's logits are those of its rows (a captured graph computes them all)
+        self._logit_rows = None if one_each else torch.tensor(rows, dtype=torch.int32).to(self.device)
+        try:
+            outputs = self._forward(self._prepare_gen_ctx(requests))
+        finally:
+            self._logit_rows = None
+        if not rows:
+            return None
+        if not one_each:
+            return outputs.last_logits
+        return outputs.last_logits[torch.tensor(rows).to(self.device)]
 
     # ------------------------------------------------------------------ first rank: requests -> buffers
     def _upload_block_lists(self, requests) -> None:
@@ -790,17 +822,22 @@ class Inferencer:
         self._upload_block_lists(requests)
         max_q = max(this_step) if this_step else 0
         desc = self._cudagraph_mgr.dispatch(num_seqs, total, max_q) if self._cudagraph_mgr else None
-        if self._cudagraph_mgr and desc is None:
+        if self._cudagraph_mgr and desc is None and not self._decode_graphs_only:
             raise RuntimeError(f"Cuda graph is enabled but no captured descriptor can cover {num_seqs} sequences "
                                f"and {total} tokens. Available descriptors: {list(self._cudagraph_mgr.graphs)}")
         self._graph_desc = desc
         graph_seqs, cap_tokens = (desc.num_seqs, desc.num_tokens) if desc else (num_seqs, total)
-        inp = sb.prepare(computed, this_step, chunks, graph_seqs, cap_tokens)
+        inp = sb.prepare(computed, this_step, chunks, graph_seqs, cap_tokens,
+                         [r.state_slot for r in requests] if self._recurrent else None)
+        recurrent = {}
+        if self._recurrent:
+            recurrent = dict(cache_store=self.cache_store, state_slots=self.input_buffers.state_slots.gpu[:graph_seqs],
+                             seq_lens=list(zip(this_step, computed)), logit_rows=self._logit_rows)
         # the (padded) static views are what the forward reads; the context handed on holds the real sizes
         set_kv_cache_context(is_paged_attn=True, key_cache=self.cache_store.key_cache,
                              value_cache=self.cache_store.value_cache, block_tables=inp.block_tables,
                              context_lens=inp.context_lens, slot_mapping=inp.slot_mapping,
-                             query_start_loc=inp.query_start_loc, max_seqlen_q=max_q)
+                             query_start_loc=inp.query_start_loc, max_seqlen_q=max_q, **recurrent)
         return GenerationContext(
             batch_input_ids=sb.input_ids[:, :total], intermediate_tensors=None,
             query_start_loc=sb.query_start_loc[: num_seqs + 1], batch_position_ids=sb.position_ids[:, :total],
@@ -853,8 +890,10 @@ class Inferencer:
                      else gen_ctx.intermediate_tensors).size(1)
             num_seqs = gen_ctx.context_lens.size(0)
             desc = getattr(self, "_graph_desc", None) if self._pp_info.is_first_rank else None
-            if desc is None:
+            if desc is None and not self._decode_graphs_only:
                 desc = self._cudagraph_mgr.dispatch(num_seqs, total, gen_ctx.max_seqlen_q)
+            if desc is None and self._decode_graphs_only:
+                return self._forward_eager(gen_ctx)
             if desc is None:
                 raise RuntimeError(f"Cuda graph is enabled but no captured descriptor can cover {num_seqs} sequences "
                                    f"and {total} tokens. Available descriptors: {list(self._cudagraph_mgr.graphs)}")

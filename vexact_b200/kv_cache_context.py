@@ -30,6 +30,12 @@ class KVCacheContext:
     context_lens: Optional[torch.Tensor] = None   # [num_seqs] int32: past + new tokens
     query_start_loc: Optional[torch.Tensor] = None  # [num_seqs + 1] int32
     max_seqlen_q: Optional[int] = None
+    # models with recurrent layers: the store that owns their state, each sequence's slot in it (-1 = none)
+    cache_store: Optional[object] = None
+    state_slots: Optional[torch.Tensor] = None    # [num_seqs] int32
+    # (new tokens, past + new tokens) of every sequence as host integers, when the host knows them (eager steps)
+    seq_lens: Optional[list] = None
+    logit_rows: Optional[torch.Tensor] = None     # packed token rows whose logits are wanted; None: each last token
 
     def __post_init__(self):
         if self.is_paged_attn:
@@ -51,7 +57,9 @@ def set_kv_cache_context(
     slot_mapping: Optional[torch.Tensor] = None,
     query_start_loc: Optional[torch.Tensor] = None,
     max_seqlen_q: Optional[int] = None,
+    **recurrent,
 ):
+    """`recurrent`: the KVCacheContext fields of models with recurrent layers."""
     _context_storage.kv_cache_context = KVCacheContext(
         is_paged_attn=is_paged_attn,
         key_cache=key_cache,
@@ -61,6 +69,7 @@ def set_kv_cache_context(
         slot_mapping=slot_mapping,
         query_start_loc=query_start_loc,
         max_seqlen_q=max_seqlen_q,
+        **recurrent,
     )
 
 
@@ -133,6 +142,61 @@ class KVCacheManager:
             if b in self.allocated_blocks:
                 self.allocated_blocks.remove(b)
                 self.free_blocks_set.add(b)
+
+
+class StateSlotManager:
+    """Host-side allocator of recurrent-state slots, one per live request; lowest free slot first."""
+
+    def __init__(self, num_slots: int):
+        if num_slots <= 0:
+            raise ValueError(f"num_slots must be positive, got {num_slots}")
+        self.num_slots = num_slots
+        self._free = set(range(num_slots))
+
+    def allocate(self) -> Optional[int]:
+        """A slot, or None when every slot is held.  Its old contents need no clearing: a sequence that starts at
+        position 0 starts from zeros."""
+        if not self._free:
+            return None
+        slot = min(self._free)
+        self._free.remove(slot)
+        return slot
+
+    def free(self, slot: int) -> None:
+        if not 0 <= slot < self.num_slots or slot in self._free:
+            raise ValueError(f"state slot {slot} is not held")
+        self._free.add(slot)
+
+    def num_free(self) -> int:
+        return len(self._free)
+
+
+class HybridCacheStore:
+    """Caches of a model that mixes latent-attention and state-space layers, one entry per layer that needs it.
+
+    latent layer: `key_cache[layer]` [blocks, page, R + DR] (normed latent, rotated shared key part), paged like any KV
+    cache; `value_cache` is empty (the value is the latent itself).
+    state-space layer: `conv_state[layer]` [slots, taps - 1, channels] in the model dtype and `ssm_state[layer]`
+    [slots, heads, N, P] fp32."""
+
+    def __init__(self, latent_widths: dict, ssm_dims: dict, cache_config, num_slots: int, device,
+                 dtype=torch.bfloat16):
+        self.cache_config = cache_config
+        self.device = torch.device(device)
+        self.page_size = cache_config.page_size
+        self.max_blocks = cache_config.max_cache_blocks
+        self.num_state_slots = num_slots
+        self.key_cache = {li: torch.zeros((self.max_blocks, self.page_size, w), device=self.device, dtype=dtype)
+                          for li, w in latent_widths.items()}
+        self.value_cache: dict[int, torch.Tensor] = {}
+        self.conv_state, self.ssm_state = {}, {}
+        for li, (channels, taps, heads, n, p) in ssm_dims.items():
+            self.conv_state[li] = torch.zeros((num_slots, taps - 1, channels), device=self.device, dtype=dtype)
+            self.ssm_state[li] = torch.zeros((num_slots, heads, n, p), device=self.device, dtype=torch.float32)
+
+    def num_bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for d in (self.key_cache, self.conv_state, self.ssm_state)
+                   for t in d.values())
 
 
 class KVCacheStore:

@@ -265,3 +265,50 @@ def stage_weights_from_hf(source: Union[torch.nn.Module, Mapping[str, torch.Tens
         w.lm_head = get("model.embed_tokens.weight") if tie else get("lm_head.weight")
     w.inv_freq = _inv_freq(shape, device)
     return w
+
+
+# ----------------------------------------------------------------------------- model folders
+def _load_hybrid(cfg, folder, dtype, device):
+    from .checkpoint import read_tensors
+    from .hybrid import HybridModel, HybridShape, HybridWeights
+
+    shape = HybridShape.from_config(cfg)
+    return HybridModel(HybridWeights.from_tensors(shape, read_tensors(folder), dtype, device))
+
+
+def _load_stage(cfg, folder, dtype, device):
+    from types import SimpleNamespace
+
+    from .checkpoint import read_tensors
+    from .inferencer import StageModel
+
+    if dtype != torch.bfloat16:
+        raise NotImplementedError(f"{cfg['model_type']} runs in bfloat16")
+    hf = SimpleNamespace(**cfg)
+    if cfg["model_type"] == "deepseek_v3":
+        hf.qk_head_dim = hf.qk_nope_head_dim + hf.qk_rope_head_dim
+    shape = shape_from_hf_config(hf)
+    model = StageModel(stage_weights_from_hf(read_tensors(folder), shape, device=device))
+    model.config = hf
+    return model
+
+
+# config.json "architecture" (own designs) or "model_type" (HF checkpoints) -> loader(config, folder, dtype, device)
+MODEL_LOADERS = {
+    "Nurazen": _load_hybrid,
+    "qwen2": _load_stage,
+    "qwen3": _load_stage,
+    "qwen3_moe": _load_stage,
+    "deepseek_v3": _load_stage,
+}
+
+
+def load_model(folder, dtype=torch.bfloat16, device="cuda"):
+    """The model of a folder (config.json + *.safetensors), as the `Inferencer` drives it."""
+    from .checkpoint import read_config
+
+    cfg = read_config(folder)
+    name = cfg.get("architecture") or cfg.get("model_type")
+    if name not in MODEL_LOADERS:
+        raise NotImplementedError(f"no model for architecture {name!r} (known: {sorted(MODEL_LOADERS)})")
+    return MODEL_LOADERS[name](cfg, folder, dtype, device)

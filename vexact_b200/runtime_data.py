@@ -52,6 +52,7 @@ class InputBuffers:
         self.context_lens = mk(max_num_seqs, dtype=torch.int32, device=device)
         self.query_start_loc = mk(max_num_seqs + 1, dtype=torch.int32, device=device)
         self.block_tables = mk(max_num_seqs, max_blocks_per_req, dtype=torch.int32, device=device, fill_value=-1)
+        self.state_slots = mk(max_num_seqs, dtype=torch.int32, device=device, fill_value=-1)   # recurrent layers
         # the batch is always packed, so the batch dimension is 1
         self.input_ids = mk(1, max_num_batched_tokens, dtype=torch.long, device=device, fill_value=0)
         self.intermediate_tensors = mk(1, max_num_batched_tokens, hidden_size, dtype=torch.bfloat16, device=device,

@@ -63,6 +63,19 @@ class StepBuffers:
         self._prefill_dev = torch.empty(T, dtype=torch.long, device=dev)
         self._delta_host = torch.empty(3, S * 2, dtype=torch.int64, pin_memory=pin)
         self.h2d_bytes_last_step = 0
+        # recorded behind the last copy out of the pinned staging, waited on before the host writes it again
+        self._staged = torch.cuda.Event() if pin else None
+        self._state_slots = buffers.state_slots if buffers is not None else None
+
+    def _wait_staging(self) -> None:
+        """A caller that never reads a step's result may be a step ahead of the GPU: the staging buffers are rewritten
+        only after the copies out of them are done."""
+        if self._staged is not None:
+            self._staged.synchronize()
+
+    def _mark_staging(self) -> None:
+        if self._staged is not None:
+            self._staged.record()
 
     # ------------------------------------------------------------------ block-table deltas
     def set_request_blocks(self, row: int, block_ids: Sequence[int]) -> None:
@@ -80,20 +93,23 @@ class StepBuffers:
             return 0
         if n > self._delta_host.shape[1]:
             raise ValueError("too many block-table updates in one step")
+        self._wait_staging()
         d = self._delta_host[:, :n]
         d[0] = torch.as_tensor(list(rows), dtype=torch.int64)
         d[1] = torch.as_tensor(list(cols), dtype=torch.int64)
         d[2] = torch.as_tensor(list(block_ids), dtype=torch.int64)
         dd = d.to(self.device, non_blocking=True)
+        self._mark_staging()
         self.request_blocks.index_put_((dd[0], dd[1]), dd[2].to(torch.int32))
         return int(d.numel() * d.element_size())
 
     # ------------------------------------------------------------------ one step
     def prepare(self, num_computed_tokens: Sequence[int], tokens_this_step: Sequence[int],
                 prefill_chunks: Optional[dict] = None, graph_num_seqs: Optional[int] = None,
-                capture_tokens: Optional[int] = None) -> StepInputs:
+                capture_tokens: Optional[int] = None, state_slots: Optional[Sequence[int]] = None) -> StepInputs:
         """Build the step's buffers.  prefill_chunks: {request row: prompt tokens fed this step};
-        rows not in it are decode requests and read `last_tokens[row]` on the device."""
+        rows not in it are decode requests and read `last_tokens[row]` on the device.  state_slots: each request's
+        recurrent-state slot (padded requests get -1), into the InputBuffers' `state_slots`."""
         num_seqs = len(num_computed_tokens)
         total = int(sum(tokens_this_step))
         graph_num_seqs = num_seqs if graph_num_seqs is None else graph_num_seqs
@@ -104,6 +120,7 @@ class StepBuffers:
             raise ValueError(f"graph_num_seqs cannot be smaller than num_seqs: {graph_num_seqs} < {num_seqs}")
         if graph_num_seqs > self.max_num_seqs or capture_tokens > self.max_num_batched_tokens:
             raise ValueError("step exceeds the static buffers")
+        self._wait_staging()
         c = self._counters_host
         c[0, :num_seqs] = torch.as_tensor(list(num_computed_tokens), dtype=torch.int32)
         c[1, :num_seqs] = torch.as_tensor(list(tokens_this_step), dtype=torch.int32)
@@ -127,6 +144,12 @@ class StepBuffers:
             self._order_host[num_seqs:graph_num_seqs] = torch.arange(num_seqs, graph_num_seqs, dtype=torch.int32)
         self.seq_order[:graph_num_seqs].copy_(self._order_host[:graph_num_seqs], non_blocking=True)
         self.h2d_bytes_last_step = 3 * num_seqs * 4 + graph_num_seqs * 4 + n_prefill * 8
+        if state_slots is not None:
+            self._state_slots.cpu[:num_seqs] = torch.as_tensor(list(state_slots), dtype=torch.int32)
+            self._state_slots.cpu[num_seqs:graph_num_seqs] = -1
+            self._state_slots.to_device(slice(0, graph_num_seqs))
+            self.h2d_bytes_last_step += graph_num_seqs * 4
+        self._mark_staging()
         self.launch(num_seqs, graph_num_seqs, capture_tokens, n_prefill > 0)
         max_q = max((int(t) for t in tokens_this_step), default=0)
         return StepInputs(
