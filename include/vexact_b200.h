@@ -444,6 +444,22 @@ int b200_latent_attn_simt(const void* q_lat, const void* cache, void* out, const
                           const void* context_lens, const void* page_table, long long page_table_stride, int max_pages,
                           int page_size, int num_blocks, int num_seqs, int min_len, int max_len, long long T, int heads,
                           int R, int DR, float scale, int dtype, void* stream);
+/* The recurrence of b200_ssm_scan in chunks of 128 tokens on tensor cores (bf16), for the sequences that bring at least
+ * min_len tokens.  P and N multiples of 8, N <= 256.  slice: state columns per CTA, 16 or 32 (speed only). */
+int b200_ssm_chunk_scan(const void* act, long long act_row_stride, const void* dt_f32, const void* A_log_f32,
+                        const void* D_f32, void* state_f32, void* y, const void* query_start_loc,
+                        const void* context_lens, const void* state_slots, int num_seqs, int num_slots, int heads,
+                        int groups, int N, int P, int min_len, int slice, void* stream);
+/* Causal attention of n sequences over keys and values projected up from their gathered latents (bf16):
+ * kv rows [keys: heads * DN | values: heads * DV], the shared rotated key part at column rot_off of the lat rows, rows
+ * key_start[i] .. key_start[i + 1] belonging to sequence seq_ids[i]; q rows hold DN + DR columns per head.
+ * out = sigmoid(gate) * attention, [T, heads * DV].  DN, DR, DV multiples of 8, DN + DR and DV <= 256. */
+int b200_latent_attn_expanded(const void* q, long long q_row_stride, const void* kv, long long kv_row_stride,
+                              const void* lat, long long lat_row_stride, int rot_off, const void* gate,
+                              long long gate_row_stride, void* out, long long out_row_stride,
+                              const void* query_start_loc, const void* context_lens, const void* seq_ids_i32,
+                              const void* key_start_i32, int n, int max_len, int heads, int DN, int DR, int DV,
+                              float scale, void* stream);
 /* dst row r = cache row of key r - key_start[i] of sequence seq_ids[i], key_start[i] <= r < key_start[i + 1]. */
 int b200_latent_gather(const void* cache, void* dst, const void* seq_ids_i32, const void* key_start_i32, int n,
                        long long rows, int row_bytes, const void* page_table, long long page_table_stride,

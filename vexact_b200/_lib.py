@@ -30,6 +30,8 @@ SIGNATURES = {
     "b200_ssm_gate_norm": [P, LL, P, LL, P, P, LL, LL, I, I, I, I, F, I, P],
     "b200_latent_prep": [P, LL, P, P, P, P, P, P, LL, I, I, I, I, I, I, F, LL, I, P],
     "b200_latent_attn_simt": [P, P, P, P, P, P, LL, I, I, I, I, I, I, LL, I, I, I, F, I, P],
+    "b200_ssm_chunk_scan": [P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
+    "b200_latent_attn_expanded": [P, LL, P, LL, P, LL, I, P, LL, P, LL, P, P, P, P, I, I, I, I, I, I, F, P],
     "b200_latent_gather": [P, P, P, P, I, LL, I, P, LL, I, I, I, I, P],
     "b200_gemm_f32": [P, P, P, P, LL, I, I, LL, LL, LL, P],
     "b200_gemm_f32_from_bf16": [P, P, P, LL, I, I, LL, LL, LL, P],

@@ -256,6 +256,7 @@ class HybridWeights:
             uv = _pad_cols(_pad_rows(get("uv"), H, V), 1, R).reshape(H, V, R)
             i = torch.arange(0, m.rot_dims, 2, dtype=torch.float64)
             return LatentWeights(w_in=mat(_pad_cols(w_in, 1, W8)), w_uk_t=mat(uk.transpose(1, 2)), w_uv=mat(uv),
+                                 w_kv=mat(torch.cat([uk.reshape(H * DN, R), uv.reshape(H * V, R)])),
                                  w_out=mat(_pad_cols(get("o"), H, V)), c_norm=vec(_pad_rows(get("dkv.norm"), 1, R)),
                                  inv_freq=vec(m.rot_base ** (-i / max(m.rot_dims, 1))), heads=H, DN=DN, DR=DR, R=R,
                                  V=V, r_true=m.kv_rank, rot_dims=m.rot_dims, scale=m.scale)

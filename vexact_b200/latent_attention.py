@@ -3,7 +3,11 @@
 The cache holds the normed latent and the shared rotated key part of every token.  Attention runs in the absorbed
 form: the query's unrotated part goes through W_uk (one small product per head), attention is one KV head of width
 R + DR whose value is the latent, and W_uv turns a head's latent output into its value (the output gate rides on that
-product's epilogue)."""
+product's epilogue).
+
+Sequences that bring many tokens take the expanded form instead (bf16): their whole context's latents are gathered from
+the pages and projected up to per-head keys and values once, and ordinary causal attention runs over those
+(`csrc/latent_expand.cuh`); that is several times fewer products per (query, key) pair."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -21,6 +25,7 @@ class LatentWeights:
     w_in: torch.Tensor      # [q: H*(DN+DR) | c: R | k_rot: DR | gate: H*V][width]
     w_uk_t: torch.Tensor    # [H, R, DN]
     w_uv: torch.Tensor      # [H, V, R]
+    w_kv: torch.Tensor      # [H*DN + H*V, R]: W_uk over W_uv
     w_out: torch.Tensor     # [width, H*V]
     c_norm: torch.Tensor    # [R] fp32
     inv_freq: torch.Tensor  # [rot_dims / 2] fp32
@@ -68,16 +73,77 @@ def latent_attn_simt(w: LatentWeights, q_lat: torch.Tensor, cache: torch.Tensor,
         "b200_latent_attn_simt")
 
 
+# Portions of at most this many tokens attend in the absorbed form.
+ABSORBED_MAX_TOKENS = 16
+EXPANDED_MAX_DIM = 256       # widest query / key and value head the expanded kernel tiles
+
+
+def _split_plan(step, device):
+    """(runs, longs): token ranges [lo, hi) of neighbouring short sequences, and for the long ones (seq ids, first
+    gathered row of each and the end, most new tokens, rows in all).  Built once per step and kept on it."""
+    plan = getattr(step, "_latent_plan", None)
+    if plan is not None:
+        return plan
+    runs, ids, starts, most, at = [], [], [0], 0, 0
+    for i, (new, total) in enumerate(step.seq_lens):
+        if new > ABSORBED_MAX_TOKENS:
+            ids.append(i)
+            starts.append(starts[-1] + total)
+            most = max(most, new)
+        elif new:
+            if runs and runs[-1][1] == at:
+                runs[-1][1] = at + new
+            else:
+                runs.append([at, at + new])
+        at += new
+    both = torch.tensor(ids + starts, dtype=torch.int32).to(device)
+    plan = runs, (both[:len(ids)], both[len(ids):], most, starts[-1])
+    step._latent_plan = plan
+    return plan
+
+
+def latent_expanded(w: LatentWeights, q: torch.Tensor, gate: torch.Tensor, cache: torch.Tensor, heads: torch.Tensor,
+                    step, longs) -> None:
+    """Expanded attention of the long sequences; writes their rows of `heads` [T, H, V], output gate included."""
+    ids, starts, most, rows = longs
+    n, bt = ids.numel(), step.block_tables
+    lat = torch.empty((rows, w.row_width), device=cache.device, dtype=cache.dtype)
+    lib = _lib.load()
+    _lib.check(
+        lib.b200_latent_gather(cache.data_ptr(), lat.data_ptr(), ids.data_ptr(), starts.data_ptr(), n, rows,
+                               w.row_width * 2, bt.data_ptr(), bt.stride(0), bt.shape[1], cache.shape[1],
+                               cache.shape[0], step.context_lens.numel(), _lib.current_stream()),
+        "b200_latent_gather")
+    kv = gemm(lat[:, :w.R], w.w_kv)
+    _lib.check(
+        lib.b200_latent_attn_expanded(
+            q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), lat.data_ptr(), lat.stride(0), w.R,
+            gate.data_ptr(), gate.stride(0), heads.data_ptr(), heads.stride(0), step.query_start_loc.data_ptr(),
+            step.context_lens.data_ptr(), ids.data_ptr(), starts.data_ptr(), n, most, w.heads, w.DN, w.DR, w.V,
+            float(w.scale), _lib.current_stream()),
+        "b200_latent_attn_expanded")
+
+
 def latent_mixer(w: LatentWeights, xn: torch.Tensor, cache: torch.Tensor, step, eps: float) -> torch.Tensor:
     T, H = xn.shape[0], w.heads
     proj = gemm(xn, w.w_in)
     dq = w.DN + w.DR
     q = proj[:, :H * dq].view(T, H, dq)
     gate = proj[:, H * dq + w.row_width:].view(T, H, w.V)
-    q_lat = torch.empty((T, H, w.row_width), device=xn.device, dtype=xn.dtype)
+    heads = torch.empty((T, H, w.V), device=xn.device, dtype=xn.dtype)
+    runs, longs = [(0, T)], None
+    if (step.max_seqlen_q > ABSORBED_MAX_TOKENS and xn.dtype == torch.bfloat16
+            and max(dq, w.V) <= EXPANDED_MAX_DIM):
+        runs, longs = _split_plan(step, xn.device)
+    q_lat = torch.empty((T, H, w.row_width), device=xn.device, dtype=xn.dtype) if runs else None
     latent_prep(w, proj, cache, step, eps, q_lat)
-    gemm(q[:, :, :w.DN], w.w_uk_t, out=q_lat[:, :, :w.R])
-    o_lat = torch.empty((T, H, w.R), device=xn.device, dtype=xn.dtype)
-    latent_attn_simt(w, q_lat, cache, o_lat, step)
-    heads = gemm(o_lat, w.w_uv, act="sigmoid_gate", gate=gate)
+    if longs is not None:
+        latent_expanded(w, q, gate, cache, heads, step, longs)
+    if runs:
+        o_lat = torch.empty((T, H, w.R), device=xn.device, dtype=xn.dtype)
+        for lo, hi in runs:
+            gemm(q[lo:hi, :, :w.DN], w.w_uk_t, out=q_lat[lo:hi, :, :w.R])
+        latent_attn_simt(w, q_lat, cache, o_lat, step, 1, ABSORBED_MAX_TOKENS if longs is not None else 1 << 30)
+        for lo, hi in runs:
+            gemm(o_lat[lo:hi], w.w_uv, act="sigmoid_gate", gate=gate[lo:hi], out=heads[lo:hi])
     return gemm(heads.view(T, H * w.V), w.w_out)

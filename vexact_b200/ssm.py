@@ -81,6 +81,24 @@ def ssm_scan(w: SSMWeights, act: torch.Tensor, dt: torch.Tensor, state: torch.Te
         "b200_ssm_scan")
 
 
+CHUNK_MAX_STATE = 256     # widest state the chunked kernel tiles
+
+
+def ssm_chunk_scan(w: SSMWeights, act: torch.Tensor, dt: torch.Tensor, state: torch.Tensor, y: torch.Tensor, step,
+                   min_len: int, num_long: int, slice_cols: int | None = None) -> None:
+    """The same recurrence in chunks on tensor cores (bf16), for the sequences that bring at least min_len tokens.
+    `num_long`: how many those are; with few of them the state is cut finer, so that every SM has a slice."""
+    if slice_cols is None:
+        slice_cols = 32 if num_long * w.heads * ((w.P + 31) // 32) >= 148 else 16
+    _lib.check(
+        _lib.load().b200_ssm_chunk_scan(
+            act.data_ptr(), act.stride(0), dt.data_ptr(), w.A_log.data_ptr(), w.D.data_ptr(), state.data_ptr(),
+            y.data_ptr(), step.query_start_loc.data_ptr(), step.context_lens.data_ptr(), step.state_slots.data_ptr(),
+            step.state_slots.numel(), state.shape[0], w.heads, w.groups, w.N, w.P, min_len, slice_cols,
+            _lib.current_stream()),
+        "b200_ssm_chunk_scan")
+
+
 def ssm_gate_norm(w: SSMWeights, y: torch.Tensor, proj: torch.Tensor, eps: float) -> torch.Tensor:
     """rms_norm_by_part(y * silu(z)) * norm; z is the first block of the in-projection rows."""
     out = torch.empty((y.shape[0], w.inner), device=y.device, dtype=y.dtype)
@@ -98,5 +116,11 @@ def ssm_mixer(w: SSMWeights, xn: torch.Tensor, conv_state: torch.Tensor, state: 
     proj = gemm(xn, w.w_in)
     act, dt = ssm_conv(w, proj, conv_state, step)
     y = torch.empty((xn.shape[0], w.inner), device=xn.device, dtype=xn.dtype)
-    ssm_scan(w, act, dt, state, y, step)
+    if step.max_seqlen_q <= SCAN_MAX_TOKENS or xn.dtype != torch.bfloat16 or w.N > CHUNK_MAX_STATE:
+        ssm_scan(w, act, dt, state, y, step)
+    else:
+        num_long = sum(n > SCAN_MAX_TOKENS for n, _ in step.seq_lens)
+        ssm_chunk_scan(w, act, dt, state, y, step, SCAN_MAX_TOKENS + 1, num_long)
+        if num_long < len(step.seq_lens):
+            ssm_scan(w, act, dt, state, y, step, 1, SCAN_MAX_TOKENS)
     return gemm(ssm_gate_norm(w, y, proj, eps), w.w_out)
