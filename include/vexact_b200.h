@@ -450,6 +450,18 @@ int b200_ssm_chunk_scan(const void* act, long long act_row_stride, const void* d
                         const void* D_f32, void* state_f32, void* y, const void* query_start_loc,
                         const void* context_lens, const void* state_slots, int num_seqs, int num_slots, int heads,
                         int groups, int N, int P, int min_len, int slice, void* stream);
+/* b200_latent_attn_simt on tcgen05 tensor cores (bf16).  b200_latent_plan lists the work of a step once for all layers
+ * with `heads` heads: items [max_items][4], item_count [1], first_item [num_seqs], i32; at most max_items =
+ * sum over sequences of ceil(new tokens * heads / 16) * ceil(context / 512).  R <= 512, DR <= 128, multiples of 8;
+ * page_size a power of two of at least 8 or a multiple of 128.  part_o [max_items, 16, R], part_ml [max_items, 16, 2]
+ * fp32 scratch, NULL when no context exceeds 512 tokens. */
+int b200_latent_plan(const void* query_start_loc, const void* context_lens, int num_seqs, int min_len, int max_len,
+                     int heads, int max_items, void* items, void* item_count, void* first_item, void* stream);
+int b200_latent_attn_tc(const void* q_lat, const void* cache, void* out, const void* query_start_loc,
+                        const void* context_lens, const void* page_table, long long page_table_stride, int max_pages,
+                        int page_size, int num_blocks, int num_seqs, int min_len, int max_len, long long T, int heads,
+                        int R, int DR, float scale, const void* items, const void* item_count, const void* first_item,
+                        int max_items, void* part_o, void* part_ml, void* stream);
 /* Causal attention of n sequences over keys and values projected up from their gathered latents (bf16):
  * kv rows [keys: heads * DN | values: heads * DV], the shared rotated key part at column rot_off of the lat rows, rows
  * key_start[i] .. key_start[i + 1] belonging to sequence seq_ids[i]; q rows hold DN + DR columns per head.

@@ -32,6 +32,8 @@ SIGNATURES = {
     "b200_latent_attn_simt": [P, P, P, P, P, P, LL, I, I, I, I, I, I, LL, I, I, I, F, I, P],
     "b200_ssm_chunk_scan": [P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
     "b200_latent_attn_expanded": [P, LL, P, LL, P, LL, I, P, LL, P, LL, P, P, P, P, I, I, I, I, I, I, F, P],
+    "b200_latent_plan": [P, P, I, I, I, I, I, P, P, P, P],
+    "b200_latent_attn_tc": [P, P, P, P, P, P, LL, I, I, I, I, I, I, LL, I, I, I, F, P, P, P, I, P, P, P],
     "b200_latent_gather": [P, P, P, P, I, LL, I, P, LL, I, I, I, I, P],
     "b200_gemm_f32": [P, P, P, P, LL, I, I, LL, LL, LL, P],
     "b200_gemm_f32_from_bf16": [P, P, P, LL, I, I, LL, LL, LL, P],
@@ -141,7 +143,7 @@ def load() -> C.CDLL:
 
 
 # Kernels launched by one successful call of each entry point (for launch accounting).
-_KERNELS_PER_CALL = {"b200_moe_permute": 2, "b200_lm_head_greedy": 2, "b200_rmsnorm_backward": 3, "b200_ssm_conv2": 2, "b200_status_read": 0, "b200_abi_version": 0}
+_KERNELS_PER_CALL = {"b200_moe_permute": 2, "b200_lm_head_greedy": 2, "b200_rmsnorm_backward": 3, "b200_ssm_conv2": 2, "b200_latent_attn_tc2": 2, "b200_status_read": 0, "b200_abi_version": 0}
 _launches = 0
 
 

@@ -17,6 +17,7 @@
 #include "ssm_chunk.cuh"
 #include "latent.cuh"
 #include "latent_expand.cuh"
+#include "latent_tc.cuh"
 
 // Self-test of the bounded wait every kernel here relies on: one CTA waits, with a limit of
 // `limit_us` microseconds, on an mbarrier that nothing ever completes.  The wait must give up, record

@@ -333,6 +333,7 @@ class HybridStep:
     block_tables: torch.Tensor
     max_seqlen_q: int
     state_slots: torch.Tensor
+    page_size: int = 64
     seq_lens: Optional[list] = None      # host (new, total) tokens per sequence; None inside a captured graph
 
 
@@ -414,7 +415,8 @@ class HybridModel:
         step = HybridStep(input_ids=input_ids.reshape(-1), positions=position_ids.reshape(-1),
                           slot_mapping=ctx.slot_mapping, query_start_loc=ctx.query_start_loc,
                           context_lens=ctx.context_lens, block_tables=ctx.block_tables,
-                          max_seqlen_q=int(ctx.max_seqlen_q), state_slots=ctx.state_slots, seq_lens=ctx.seq_lens)
+                          max_seqlen_q=int(ctx.max_seqlen_q), state_slots=ctx.state_slots,
+                          page_size=ctx.cache_store.page_size, seq_lens=ctx.seq_lens)
         rows = ctx.logit_rows
         if rows is None:      # each sequence's last token; a padded, empty sequence reads row 0
             rows = (ctx.query_start_loc[1:] - 1).clamp(min=0)

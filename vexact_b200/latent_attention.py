@@ -73,6 +73,62 @@ def latent_attn_simt(w: LatentWeights, q_lat: torch.Tensor, cache: torch.Tensor,
         "b200_latent_attn_simt")
 
 
+TC_SPLIT, TC_COLUMNS = 512, 16     # keys of a split and columns of a tile of the tensor-core kernel
+
+
+def tc_supported(w: LatentWeights, dtype, page_size: int) -> bool:
+    """Whether the tensor-core kernel takes these dims (the CUDA-core kernel takes every one)."""
+    pages = page_size % 128 == 0 or (page_size >= 8 and 128 % page_size == 0)
+    return dtype == torch.bfloat16 and pages and w.R <= 512 and 0 < w.DR <= 128
+
+
+def _tc_plan(step, heads: int, pool_tokens: int, min_len: int, max_len: int, device):
+    """(items, count, first item of each sequence, capacity, whether a context has several splits), made once per step
+    for every layer with this many heads."""
+    plans = step.__dict__.setdefault("_tc_plans", {})
+    plan = plans.get((heads, min_len, max_len))
+    if plan is not None:
+        return plan
+    S = step.context_lens.numel()
+    if step.seq_lens is not None:
+        live = [(n, t) for n, t in step.seq_lens if min_len <= n <= max_len]
+        cap = sum(-(-n * heads // TC_COLUMNS) * -(-t // TC_SPLIT) for n, t in live)
+        several = any(t > TC_SPLIT for _, t in live)
+    else:     # a captured decode graph: every token of the pool could be live
+        cap = -(-min(step.max_seqlen_q, max_len) * heads // TC_COLUMNS) * (S + pool_tokens // TC_SPLIT)
+        several = step.block_tables.shape[1] * step.page_size > TC_SPLIT
+    cap = max(cap, 1)
+    items = torch.empty((cap, 4), device=device, dtype=torch.int32)
+    meta = torch.empty(S + 4, device=device, dtype=torch.int32)
+    _lib.check(
+        _lib.load().b200_latent_plan(step.query_start_loc.data_ptr(), step.context_lens.data_ptr(), S, min_len, max_len,
+                                     heads, cap, items.data_ptr(), meta.data_ptr(), meta[4:].data_ptr(),
+                                     _lib.current_stream()),
+        "b200_latent_plan")
+    plan = plans[(heads, min_len, max_len)] = items, meta[:1], meta[4:], cap, several
+    return plan
+
+
+def latent_attn_tc(w: LatentWeights, q_lat: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, step,
+                   min_len: int = 1, max_len: int = 1 << 30) -> None:
+    """Absorbed attention on tensor cores (bf16) for the sequences that bring min_len .. max_len tokens."""
+    bt = step.block_tables
+    items, count, first, cap, several = _tc_plan(step, w.heads, cache.shape[0] * cache.shape[1], min_len, max_len,
+                                                 cache.device)
+    part_o = part_ml = None
+    if several:
+        part_o = torch.empty((cap, TC_COLUMNS, w.R), device=cache.device, dtype=torch.float32)
+        part_ml = torch.empty((cap, TC_COLUMNS, 2), device=cache.device, dtype=torch.float32)
+    _lib.check(
+        _lib.load().b200_latent_attn_tc(
+            q_lat.data_ptr(), cache.data_ptr(), out.data_ptr(), step.query_start_loc.data_ptr(),
+            step.context_lens.data_ptr(), bt.data_ptr(), bt.stride(0), bt.shape[1], cache.shape[1], cache.shape[0],
+            step.context_lens.numel(), min_len, max_len, q_lat.shape[0], w.heads, w.R, w.DR, float(w.scale),
+            items.data_ptr(), count.data_ptr(), first.data_ptr(), cap, _lib.ptr(part_o), _lib.ptr(part_ml),
+            _lib.current_stream()),
+        "b200_latent_attn_tc2" if several else "b200_latent_attn_tc")
+
+
 # Portions of at most this many tokens attend in the absorbed form.
 ABSORBED_MAX_TOKENS = 16
 EXPANDED_MAX_DIM = 256       # widest query / key and value head the expanded kernel tiles
@@ -143,7 +199,8 @@ def latent_mixer(w: LatentWeights, xn: torch.Tensor, cache: torch.Tensor, step, 
         o_lat = torch.empty((T, H, w.R), device=xn.device, dtype=xn.dtype)
         for lo, hi in runs:
             gemm(q[lo:hi, :, :w.DN], w.w_uk_t, out=q_lat[lo:hi, :, :w.R])
-        latent_attn_simt(w, q_lat, cache, o_lat, step, 1, ABSORBED_MAX_TOKENS if longs is not None else 1 << 30)
+        attend = latent_attn_tc if tc_supported(w, xn.dtype, cache.shape[1]) else latent_attn_simt
+        attend(w, q_lat, cache, o_lat, step, 1, ABSORBED_MAX_TOKENS if longs is not None else 1 << 30)
         for lo, hi in runs:
             gemm(o_lat[lo:hi], w.w_uv, act="sigmoid_gate", gate=gate[lo:hi], out=heads[lo:hi])
     return gemm(heads.view(T, H * w.V), w.w_out)
