@@ -74,6 +74,9 @@ def parse_args():
     ap.add_argument("--train-kernels", action="store_true",
                     help="side measurement: forward + backward of the packed attention call and of one fused-MoE "
                          "layer at the model's widths (the training-side operators; correctness-first kernels)")
+    ap.add_argument("--hybrid", action="store_true",
+                    help="side measurement: prefill and decode steps of the hybrid decoder family (state-space + latent "
+                         "attention) beside an MLA + dense model of equal size, and its kernels beside that model's")
     ap.add_argument("--prefill-attention", type=int, default=0, metavar="QLEN",
                     help="side measurement: time one causal prefill attention call of QLEN queries on the "
                          "model's head shape (context --ctx if larger) and print its own JSON line")
@@ -667,6 +670,298 @@ def run_prefill_attention(args, shape):
                       "eager_call_tflops": flops / eager / 1e9}))
 
 
+# --------------------------------------------------------------------------- hybrid decoders
+def hybrid_shapes():
+    """(hybrid of 6 state-space + 2 latent layers, 8 latent layers, the closest other model: MLA + dense FFN) at equal
+    width, heads, head dims and parameters per feed-forward."""
+    from vexact_b200.hybrid import HybridLayer, HybridShape, LatentSpec, SSMSpec
+    from vexact_b200.inferencer import MLAShape, ModelShape
+
+    W, V, FF = 2048, 32768, 8192
+    ssm = SSMSpec(heads=64, vdim=64, state=128, groups=8, conv=4, norm_groups=8)
+    lat = LatentSpec(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot_base=50000.0, rot_dims=64)
+
+    def make(name, kinds):
+        return HybridShape(name, tuple(HybridLayer(m, FF, i) for i, m in enumerate(kinds)), W, V, 4, 0.3, 1e-5)
+
+    return (make("hybrid-6ssm-2latent", [ssm, ssm, lat, ssm, ssm, ssm, lat, ssm]),
+            make("hybrid-8latent", [lat] * 8),
+            ModelShape("mla-dense", 8, W, 16, 16, 192, V, ffn=5504, qk_norm=False, rope_theta=50000.0, rms_eps=1e-5,
+                       mla=MLAShape(), norm_single_round=True))
+
+
+def hybrid_step(lens, page, device, seed=0):
+    """Packed-step metadata for sequences of (new, total) tokens on randomly dealt pages, and the page count."""
+    from vexact_b200.hybrid import HybridStep
+
+    g = torch.Generator().manual_seed(seed)
+    pages = [(t + page - 1) // page for _, t in lens]
+    order = torch.randperm(sum(pages), generator=g).to(torch.int32)
+    table = torch.full((len(lens), max(pages)), -1, dtype=torch.int32)
+    pos, slots, at = [], [], 0
+    for i, (n, t) in enumerate(lens):
+        table[i, :pages[i]] = order[at:at + pages[i]]
+        at += pages[i]
+        p = torch.arange(t - n, t)
+        pos.append(p)
+        slots.append((table[i, p // page].long() * page + p % page).to(torch.int32))
+    T = sum(n for n, _ in lens)
+    dev = lambda t: t.to(device)   # noqa: E731
+    cu = torch.tensor([0] + [n for n, _ in lens]).cumsum(0).to(torch.int32)
+    step = HybridStep(input_ids=dev(torch.randint(0, 32768, (T,), generator=g)), positions=dev(torch.cat(pos)),
+                      slot_mapping=dev(torch.cat(slots)), query_start_loc=dev(cu),
+                      context_lens=dev(torch.tensor([t for _, t in lens], dtype=torch.int32)), block_tables=dev(table),
+                      max_seqlen_q=max(n for n, _ in lens), page_size=page, seq_lens=list(lens),
+                      state_slots=dev(torch.arange(len(lens), dtype=torch.int32)))
+    return step, sum(pages)
+
+
+def graph_ms(calls, reps=10):
+    """Device time of one call: `calls` (closures over their own buffers, together larger than L2) captured in one CUDA
+    graph; the best of `reps` replays, per call."""
+    side = torch.cuda.Stream()
+    side.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(side):
+        for c in calls:
+            c()
+    torch.cuda.current_stream().wait_stream(side)
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for c in calls:
+            c()
+    best = float("inf")
+    for i in range(reps + 3):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        graph.replay()
+        b.record()
+        torch.cuda.synchronize()
+        if i >= 3:
+            best = min(best, a.elapsed_time(b) / len(calls))
+    return best
+
+
+def run_hybrid(args):
+    """Side measurement (not the contract line): prefill and decode steps of the hybrid decoder family and of the closest
+    other model at equal size (random weights), then its kernels beside the like kernels of that model."""
+    from vexact_b200 import _lib
+
+    device = torch.device("cuda", 0)
+    torch.cuda.set_device(device)
+    page = 64
+    cases = [("decode", 64, 1, 4096), ("decode", 256, 1, 1024), ("prefill", 4, 2048, 2048), ("prefill", 1, 2048, 8192)]
+    hyb, lat, mla = hybrid_shapes()
+    clocks = ClockSampler(0)
+    clocks.start()
+    clocks.wait_first_sample()
+    for shape in (hyb, lat, mla):
+        for kind, S, new, total in cases:
+            print(json.dumps(hybrid_model_case(args, shape, kind, S, new, total, page, device)), flush=True)
+            torch.cuda.empty_cache()
+    for line in hybrid_kernels(args, page, device):
+        print(json.dumps(line), flush=True)
+    print(json.dumps({"measurement": "hybrid", "clocks": clocks.stop(), "status": list(_lib.read_status())}))
+
+
+def hybrid_model_case(args, shape, kind, S, new, total, page, device):
+    from vexact_b200 import _lib
+    from vexact_b200.hybrid import HybridModel, HybridShape, HybridWeights
+    from vexact_b200.config import CacheConfig
+    from vexact_b200.inferencer import StageRunner, StageWeights, StepInputs, allocate_kv_cache
+
+    step, blocks = hybrid_step([(new, total)] * S, page, device)
+    if isinstance(shape, HybridShape):
+        model = HybridModel(HybridWeights.random_init(shape, device=device))
+        runner, w = model.runner, model.runner.w
+        runner.store = model.make_cache_store(CacheConfig(page, blocks), S, device)
+        for t in runner.store.key_cache.values():
+            t.normal_()
+        rows = (step.query_start_loc[1:] - 1).contiguous()
+        if kind == "decode":
+            step.seq_lens = None
+
+        def run():
+            for k in ("_latent_plan", "_tc_plans"):      # what belongs to one step is made in every step
+                step.__dict__.pop(k, None)
+            return runner.logits(runner.forward(step, rows))
+
+        cache_bytes = sum(S * total * t.shape[-1] * 2 for t in runner.store.key_cache.values())
+        cache_bytes += 2 * sum(t.numel() * t.element_size() for d in (runner.store.conv_state, runner.store.ssm_state)
+                               for t in d.values())
+        vocab, width = shape.vocab, shape.width
+    else:
+        w = StageWeights.random_init(shape, device=device)
+        kc, vc = allocate_kv_cache(shape, 0, shape.num_layers, blocks, page, device=device, fill_std=1.0)
+        stage = StageRunner(w, kc, vc)
+        inp = StepInputs(step.input_ids, None, step.positions, step.slot_mapping, step.query_start_loc, step.context_lens,
+                         step.block_tables, step.max_seqlen_q)
+        stage.prepare(step.input_ids.numel())
+        run = lambda: stage.last_token_logits(stage.forward(inp), inp)   # noqa: E731
+        cache_bytes = S * total * shape.num_kv_heads * (shape.k_dim + shape.v_dim) * 2 * shape.num_layers
+        vocab, width = shape.vocab, shape.hidden
+    _lib.reset_launch_count()
+    run()
+    torch.cuda.synchronize()
+    launches = _lib.launch_count()
+    if kind == "decode":
+        ms = graph_ms([run], max(args.steps, 5))
+    else:
+        for _ in range(max(args.warmup, 3)):
+            run()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record()
+        for _ in range(args.steps):
+            run()
+        b.record()
+        torch.cuda.synchronize()
+        ms = a.elapsed_time(b) / args.steps
+    out = {"measurement": f"hybrid_{kind}", "model": shape.name, "sequences": S, "new_tokens": new, "context": total,
+           "ms_per_step": round(ms, 4), "tokens_per_s": round(S * new / ms * 1e3), "launches": launches}
+    if kind == "decode":
+        nbytes = w.num_bytes() - vocab * width * 2 + cache_bytes
+        out.update(weights_and_state_gb=round(nbytes / 1e9, 3),
+                   frac_of_hbm=round(nbytes / ms / 1e6 / float(measured_peaks().get("hbm_gbs", 6650.0)), 3))
+    return out
+
+
+def hybrid_kernels(args, page, device):
+    """Per kernel of the hybrid family (and the like kernel of the MLA model): device time, achieved bytes or flops over
+    the measured peak.  Several buffers per kernel, together larger than L2."""
+    import vexact_b200 as vb
+    from vexact_b200 import _lib
+    from vexact_b200.batch_invariant_ops import gemm
+    from vexact_b200.hybrid import HybridWeights, HybridShape
+    from vexact_b200.hyper import hyper_step
+    from vexact_b200 import latent_attention as la, ssm
+
+    peaks = measured_peaks()
+    hbm, tc = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    BF = torch.bfloat16
+    hyb, _, mla = hybrid_shapes()
+    two = HybridShape("pair", (hyb.layers[0], hyb.layers[2].__class__(hyb.layers[2].mixer, 8192, 1)), hyb.width, hyb.vocab,
+                      hyb.streams, hyb.residual_mult, hyb.eps)
+    w = HybridWeights.random_init(two, device=device)
+    sw, lw, mw, hc = w.layers[0].mixer, w.layers[1].mixer, w.layers[0].mlp, w.layers[0].hc
+    W, n = hyb.width, hyb.streams
+    rn = lambda *s: torch.randn(s, device=device).to(BF)   # noqa: E731
+
+    def line(name, ms, nbytes=None, flops=None, like=None):
+        out = {"measurement": "hybrid_kernel", "kernel": name, "us": round(ms * 1e3, 2)}
+        fr = []
+        if nbytes:
+            out["gb_s"] = round(nbytes / ms / 1e6)
+            fr.append(nbytes / ms / 1e6 / hbm)
+        if flops:
+            out["tflop_s"] = round(flops / ms / 1e9, 1)
+            fr.append(flops / ms / 1e9 / tc)
+        out["of_measured_roofline"] = round(max(fr), 3)
+        if like:
+            out["like"] = like
+        return out
+
+    for T in (64, 8192):
+        k = 24 if T == 64 else 3
+        sets = [(torch.randn(T, n, W, device=device), rn(T, W)) for _ in range(k)]
+        ms = graph_ms([lambda s=s, y=y: hyper_step(s, done=hc[0], y=y, residual_mult=0.3, read=hc[1].read, norm=hc[1].norm,
+                                                   eps=1e-5, xn_cols=W) for s, y in sets])
+        yield line(f"hyper_step T={T}", ms, T * W * (8 * n + 4))
+        sets = [(rn(T, W), rn(T, W)) for _ in range(k)]
+        nw = rn(W)
+        ms = graph_ms([lambda x=x, r=r: vb.add_rms_norm(x, r, nw, 1e-5, hf=False) for x, r in sets])
+        yield line(f"add_rmsnorm T={T}", ms, T * W * 8, like=f"hyper_step T={T}")
+        xs, up = [rn(T, W) for _ in range(k)], mw.up
+        ms = graph_ms([lambda x=x: gemm(x, up, mw.up_b, act="gelu_tanh") for x in xs])
+        yield line(f"gemm+gelu T={T}", ms, 2 * (up.numel() + T * W + T * up.shape[0]), 2.0 * T * up.numel())
+        ms = graph_ms([lambda x=x: vb.linear(x, up) for x in xs])
+        yield line(f"gemm T={T}", ms, 2 * (up.numel() + T * W + T * up.shape[0]), 2.0 * T * up.numel(), like=f"gemm+gelu T={T}")
+        # state-space kernels: T sequences of one token, or 4 of T / 4
+        st, _ = hybrid_step([(1, 100)] * T if T == 64 else [(T // 4, T // 4)] * 4, page, device)
+        S = st.state_slots.numel()
+        proj = [rn(T, sw.w_in.shape[0]) for _ in range(k)]
+        conv = [torch.zeros(S, sw.taps - 1, sw.channels, device=device, dtype=BF) for _ in range(k)]
+        ms = graph_ms([lambda p=p, c=c: ssm.ssm_conv(sw, p, c, st) for p, c in zip(proj, conv)])
+        state_b = 4 * S * (sw.taps - 1) * sw.channels
+        yield line(f"ssm_conv T={T}", ms, T * (sw.channels * 4 + sw.heads * 6) + state_b)
+        act = [(rn(T, sw.channels), torch.rand(T, sw.heads, device=device) * 0.1,
+                torch.zeros(S, sw.heads, sw.N, sw.P, device=device), rn(T, sw.inner)) for _ in range(k)]
+        scan_b = T * (sw.channels + sw.inner) * 2 + T * sw.heads * 4 + 8 * S * sw.heads * sw.N * sw.P
+        if T == 64:
+            ms = graph_ms([lambda a=a: ssm.ssm_scan(sw, *a, st) for a in act])
+            yield line("ssm_scan (decode) S=64", ms, scan_b)
+        else:
+            for cols in (16, 32):
+                ms = graph_ms([lambda a=a: ssm.ssm_chunk_scan(sw, *a, st, 17, 4, cols) for a in act])
+                flops = T * sw.heads * (2.0 * 64 * sw.N + 2.0 * 64 * sw.P + 4.0 * sw.N * sw.P)
+                yield line(f"ssm_chunk T={T} slice={cols}", ms, scan_b, flops)
+        ms = graph_ms([lambda a=a, p=p: ssm.ssm_gate_norm(sw, a[3], p, 1e-5) for a, p in zip(act, proj)])
+        yield line(f"ssm_gate_norm T={T}", ms, T * sw.inner * 6)
+        del proj, conv, act, sets, xs
+        torch.cuda.empty_cache()
+        # latent attention preparation beside the MLA model's
+        st, blocks = hybrid_step([(1, 100)] * T if T == 64 else [(T // 4, T // 4)] * 4, page, device)
+        proj = [rn(T, lw.w_in.shape[0]) for _ in range(k)]
+        cache = torch.zeros(blocks, page, lw.row_width, device=device, dtype=BF)
+        qlat = [torch.empty(T, 16, lw.row_width, device=device, dtype=BF) for _ in range(k)] if T == 64 else [None] * k
+        ms = graph_ms([lambda p=p, q=q: la.latent_prep(lw, p, cache, st, 1e-5, q) for p, q in zip(proj, qlat)])
+        yield line(f"latent_prep T={T}", ms, T * (lw.row_width * 4 + 16 * 64 * (4 if T > 64 else 6)))
+        lib, inv = _lib.load(), lw.inv_freq
+        sets = [(rn(T, 16 * 192), rn(T, 16 * 256), rn(T, 576)) for _ in range(k)]
+        kc, vc = (torch.zeros(blocks, page, 16, d, device=device, dtype=BF) for d in (192, 128))
+
+        def mla_store(q, kvb, kr):
+            out = torch.empty_like(q)
+            _lib.check(lib.b200_mla_rope_store(q.data_ptr(), q.stride(0), kvb.data_ptr(), kvb.stride(0), kr[:, 512:].data_ptr(),
+                                               kr.stride(0), st.positions.data_ptr(), st.slot_mapping.data_ptr(),
+                                               inv.data_ptr(), out.data_ptr(), kc.data_ptr(), vc.data_ptr(), T, 16, 128, 64,
+                                               128, blocks * page, _lib.current_stream()), "b200_mla_rope_store")
+
+        ms = graph_ms([lambda s=s: mla_store(*s) for s in sets])
+        yield line(f"mla_rope_store T={T}", ms, T * 2 * (2 * 16 * 192 + 16 * 256 + 64 + 16 * 320), like=f"latent_prep T={T}")
+        del proj, qlat, sets, kc, vc
+        torch.cuda.empty_cache()
+    for S, ctx in ((64, 4096), (256, 1024)):
+        st, blocks = hybrid_step([(1, ctx)] * S, page, device)
+        sets = [(rn(S, 16, lw.row_width), rn(blocks, page, lw.row_width), torch.empty(S, 16, lw.R, device=device, dtype=BF))
+                for _ in range(2)]
+        ms = graph_ms([lambda s=s: la.latent_attn_tc(lw, *s, st) for s in sets])
+        yield line(f"latent_tc decode {S}x{ctx}", ms, S * ctx * lw.row_width * 2, 2.0 * S * ctx * 16 * (lw.row_width + lw.R))
+        kc, vc, q = rn(blocks, page, 16, 192), rn(blocks, page, 16, 128), rn(S, 16, 192)
+        ms = graph_ms([lambda: vb.paged_attention(q, kc, vc, st.query_start_loc, st.context_lens, st.block_tables,
+                                                  192 ** -0.5, 1)])
+        yield line(f"paged_attn 192/128 decode {S}x{ctx}", ms, S * ctx * 16 * 320 * 2, like=f"latent_tc decode {S}x{ctx}")
+        del kc, vc, sets
+        torch.cuda.empty_cache()
+    for S, new, total in ((4, 2048, 2048), (1, 2048, 8192)):
+        st, blocks = hybrid_step([(new, total)] * S, page, device)
+        T = S * new
+        q, gate, cache = rn(T, 16, 192), rn(T, 16, 128), rn(blocks, page, lw.row_width)
+        heads, plan = torch.empty(T, 16, 128, device=device, dtype=BF), la._split_plan(st, device)[1]
+        pairs = S * sum(range(total - new + 1, total + 1))
+        flops = 2.0 * pairs * 16 * 320
+        ms = graph_ms([lambda: la.latent_expanded(lw, q, gate, cache, heads, st, plan)])
+        yield line(f"latent gather + up-projection + expanded attention {S}x{new}/{total}", ms, None,
+                   flops + 2.0 * S * total * lw.w_kv.numel())
+        lat, kv = rn(S * total, lw.row_width), rn(S * total, lw.w_kv.shape[0])
+        ids, starts, most, _ = plan
+
+        def attn():
+            _lib.check(_lib.load().b200_latent_attn_expanded(
+                q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), lat.data_ptr(), lat.stride(0), lw.R, gate.data_ptr(),
+                gate.stride(0), heads.data_ptr(), heads.stride(0), st.query_start_loc.data_ptr(), st.context_lens.data_ptr(),
+                ids.data_ptr(), starts.data_ptr(), ids.numel(), most, 16, 128, 64, 128, float(lw.scale),
+                _lib.current_stream()), "b200_latent_attn_expanded")
+
+        yield line(f"latent_expand {S}x{new}/{total}", graph_ms([attn]), None, flops)
+        kc, vc = rn(blocks, page, 16, 192), rn(blocks, page, 16, 128)
+        ms = graph_ms([lambda: vb.paged_attention(q, kc, vc, st.query_start_loc, st.context_lens, st.block_tables,
+                                                  192 ** -0.5, new)])
+        yield line(f"paged_attn 192/128 prefill {S}x{new}/{total}", ms, None, flops, like=f"latent_expand {S}x{new}/{total}")
+        del kc, vc, lat, kv
+        torch.cuda.empty_cache()
+
+
 def main():
     args = parse_args()
     rank = int(os.environ.get("RANK", "0"))
@@ -680,6 +975,9 @@ def main():
         shape = ModelShape(**{**shape.__dict__, "num_layers": args.layers})
     if args.impl == "reference":
         run_reference(args, shape, rank)
+        return
+    if args.hybrid:
+        run_hybrid(args)
         return
     if args.skew:
         run_skew(args, shape)
