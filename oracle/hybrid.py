@@ -146,7 +146,10 @@ def forward(config, weights, tokens, want_layers=False):
     xs = streams_start(weights["embed"][torch.as_tensor(tokens, dtype=torch.long)], n)
     after = []
     for i, layer in enumerate(config["layers"]):
-        p = f"l{layer.get('weights_of', i)}."
+        owner = i
+        while config["layers"][owner].get("weights_of") is not None:
+            owner = config["layers"][owner]["weights_of"]
+        p = f"l{owner}."
 
         def sublayer(xs, q, fn):
             hc = _sub(weights, f"{p}hc{q}.")
