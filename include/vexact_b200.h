@@ -444,7 +444,7 @@ int b200_latent_attn_simt(const void* q_lat, const void* cache, void* out, const
                           const void* context_lens, const void* page_table, long long page_table_stride, int max_pages,
                           int page_size, int num_blocks, int num_seqs, int min_len, int max_len, long long T, int heads,
                           int R, int DR, float scale, int dtype, void* stream);
-/* The recurrence of b200_ssm_scan in chunks of 128 tokens on tensor cores (bf16), for the sequences that bring at least
+/* The recurrence of b200_ssm_scan in chunks of 64 tokens on tensor cores (bf16), for the sequences that bring at least
  * min_len tokens.  P and N multiples of 8, N <= 256.  slice: state columns per CTA, 16 or 32 (speed only). */
 int b200_ssm_chunk_scan(const void* act, long long act_row_stride, const void* dt_f32, const void* A_log_f32,
                         const void* D_f32, void* state_f32, void* y, const void* query_start_loc,

@@ -485,12 +485,21 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
         const __nv_bfloat16* gate =
             p.act == GEMM_ACT_SIGMOID_GATE ? p.gate + (long long)t.group * p.gate_batch_stride + f : nullptr;
         const long long out_base = (long long)t.group * p.out_batch_stride;
-        auto finish = [&](float v, int c) -> float {
-          v += bias;
-          if (p.act == GEMM_ACT_GELU_TANH) v = gelu_tanh_fast(v);
-          if (gate && fvalid && c < t.n)
-            v = __fdividef(v, 1.f + __expf(-bf2f(gate[(long long)(t.row0 + c) * p.gate_stride])));
-          return v;
+        // one branch around sixteen independent chains, not one inside each: the chains then overlap
+        auto finish = [&](const uint32_t (&r)[16], float (&v)[16], int c0) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]) + bias;
+          if (p.act == GEMM_ACT_GELU_TANH) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = gelu_tanh_fast(v[j]);
+          } else if (gate && fvalid) {
+            float e[16];
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              e[j] = c0 + j < t.n ? bf2f(gate[(long long)(t.row0 + c0 + j) * p.gate_stride]) : 0.f;
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = __fdividef(v[j], 1.f + __expf(-e[j]));
+          }
         };
         // bf16 output whose rows allow 16-byte stores: each warp turns its 32 features x 16 tokens around in
         // shared memory, so that a lane stores eight consecutive features of one token (16 bytes) and one
@@ -505,9 +514,10 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             uint32_t r[16];
             ptx::tmem_ld16(taddr + c0, r);
             ptx::tmem_ld_wait();
+            float v[16];
+            finish(r, v, c0);
 #pragma unroll
-            for (int j = 0; j < 16; ++j)
-              reinterpret_cast<unsigned short*>(stg)[j * 32 + lane] = cvt16(finish(__uint_as_float(r[j]), c0 + j));
+            for (int j = 0; j < 16; ++j) reinterpret_cast<unsigned short*>(stg)[j * 32 + lane] = cvt16(v[j]);
             __syncwarp();
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
@@ -524,11 +534,13 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           ptx::tmem_ld16(taddr + c0, r);
           ptx::tmem_ld_wait();
           if (fvalid) {
+            float act[16];
+            finish(r, act, c0);
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const int c = c0 + j;
               if (c < t.n) {
-                const float v = finish(__uint_as_float(r[j]), c);
+                const float v = act[j];
                 const long long o = out_base + (long long)(t.row0 + c) * p.ldo + f;
                 if (p.out_f32)
                   reinterpret_cast<float*>(p.out)[o] = v;

@@ -39,6 +39,11 @@ __device__ __forceinline__ bool ssm_seq(const SsmSeqs& q, int s, int& t0, int& l
 }
 
 __device__ __forceinline__ float silu_f32(float v) { return v / (1.f + expf(-v)); }
+// silu of an activation that is stored in T.
+template <typename T>
+__device__ __forceinline__ float silu_as(float v) { return silu_f32(v); }
+template <>
+__device__ __forceinline__ float silu_as<__nv_bfloat16>(float v) { return __fdividef(v, 1.f + __expf(-v)); }
 __device__ __forceinline__ float softplus_f32(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
 struct SsmConvParams {
@@ -68,7 +73,7 @@ __device__ __forceinline__ float ssm_conv_at(const SsmConvParams& p, const T* pr
     else if (st) v = to_f32(st[(long long)(i + p.taps - 1) * p.channels + c]);
     a = fmaf(p.w[c * p.taps + k], v, a);
   }
-  return silu_f32(a);
+  return silu_as<T>(a);
 }
 
 // The last taps - 1 inputs of (old state, this step's inputs) become the state.  Ascending k reads only entries at or
@@ -136,6 +141,45 @@ __global__ void __launch_bounds__(128) ssm_conv_tile_kernel(const SsmConvParams 
   int s = s_seq, len, slot, t0;
   bool fresh;
   ssm_seq(p.seqs, s, t0, len, fresh, slot);
+  if (sizeof(T) == 2 && p.taps <= 4 && p.channels % 256 == 0 && (int)blockIdx.x * 128 < p.channels && tile0 >= t0 &&
+      tile0 + SSM_CONV_TILE <= t0 + len) {
+    if ((int)blockIdx.x * 256 >= p.channels) return;
+    // a tile inside one sequence: two channels per thread, every input loaded up front
+    const int c2 = (blockIdx.x * 128 + threadIdx.x) * 2;
+    float2 w[4], in[SSM_CONV_TILE + 3];
+    const int j0 = (int)(tile0 - t0);
+#pragma unroll
+    for (int i = 0; i < SSM_CONV_TILE + 3; ++i) {
+      const int q = j0 - 3 + i;
+      in[i] = make_float2(0.f, 0.f);
+      if (q >= 0) {
+        unpack_bf2(*reinterpret_cast<const uint32_t*>(proj + (t0 + (long long)q) * p.proj_stride + p.conv_off + c2), in[i].x,
+                   in[i].y);
+      } else if (!fresh && slot >= 0 && q + p.taps - 1 >= 0) {
+        unpack_bf2(*reinterpret_cast<const uint32_t*>(reinterpret_cast<const T*>(p.conv_state) +
+                                                      ((long long)slot * (p.taps - 1) + q + p.taps - 1) * p.channels + c2),
+                   in[i].x, in[i].y);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int kk = k - (4 - p.taps);
+      w[k] = kk >= 0 ? make_float2(p.w[c2 * p.taps + kk], p.w[(c2 + 1) * p.taps + kk]) : make_float2(0.f, 0.f);
+    }
+    const float2 bias = *reinterpret_cast<const float2*>(p.bias + c2);
+    T* out = reinterpret_cast<T*>(p.act) + tile0 * p.channels + c2;
+#pragma unroll
+    for (int i = 0; i < SSM_CONV_TILE; ++i) {
+      float a = bias.x, b = bias.y;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        a = fmaf(w[k].x, in[i + k].x, a);
+        b = fmaf(w[k].y, in[i + k].y, b);
+      }
+      *reinterpret_cast<uint32_t*>(out + (long long)i * p.channels) = pack_bf2(silu_as<T>(a), silu_as<T>(b));
+    }
+    return;
+  }
   const bool is_dt = c >= p.channels;
   if (c >= p.channels + p.heads) return;
   if (!is_dt && p.taps <= 4) {
@@ -177,7 +221,7 @@ __global__ void __launch_bounds__(128) ssm_conv_tile_kernel(const SsmConvParams 
       float a = bias;
 #pragma unroll
       for (int k = 0; k < 4; ++k) a = fmaf(w[k], win[k], a);
-      reinterpret_cast<T*>(p.act)[t * p.channels + c] = from_f32<T>(silu_f32(a));
+      reinterpret_cast<T*>(p.act)[t * p.channels + c] = from_f32<T>(silu_as<T>(a));
     }
     return;
   }
@@ -344,6 +388,62 @@ struct SsmGateNormParams {
   float eps;
 };
 
+// The common case (heads unpadded, parts of a multiple of 8 up to 2048 columns, bf16): one warp per (token, part), its
+// gated values in registers.
+__global__ void __launch_bounds__(256) ssm_gate_norm_warp_kernel(const SsmGateNormParams p, long long pairs) {
+  pdl_trigger();
+  pdl_wait();
+  const long long id = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (id >= pairs) return;
+  const int lane = threadIdx.x & 31, n = p.heads * p.P / p.parts;
+  const long long t = id / p.parts;
+  const int j0 = (int)(id - t * p.parts) * n;
+  const __nv_bfloat16* y = reinterpret_cast<const __nv_bfloat16*>(p.y) + t * p.y_stride + j0;
+  const __nv_bfloat16* z = reinterpret_cast<const __nv_bfloat16*>(p.z) + t * p.z_stride + j0;
+  __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.out) + t * p.out_stride + j0;
+  uint4 a[8], b[8];
+#pragma unroll
+  for (int c = 0; c < 8; ++c) {
+    const int i = (c * 32 + lane) * 8;
+    if (i < n) {
+      a[c] = *reinterpret_cast<const uint4*>(y + i);
+      b[c] = *reinterpret_cast<const uint4*>(z + i);
+    }
+  }
+  float g[8][8], ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < 8; ++c) {
+    const int i = (c * 32 + lane) * 8;
+    if (i < n) {
+      const uint32_t av[4] = {a[c].x, a[c].y, a[c].z, a[c].w}, bv[4] = {b[c].x, b[c].y, b[c].z, b[c].w};
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        float y0, y1, z0, z1;
+        unpack_bf2(av[k], y0, y1);
+        unpack_bf2(bv[k], z0, z1);
+        g[c][2 * k] = y0 * silu_as<__nv_bfloat16>(z0);
+        g[c][2 * k + 1] = y1 * silu_as<__nv_bfloat16>(z1);
+        ss = fmaf(g[c][2 * k], g[c][2 * k], ss);
+        ss = fmaf(g[c][2 * k + 1], g[c][2 * k + 1], ss);
+      }
+    }
+  }
+  const float inv = 1.f / sqrtf(warp_sum(ss) / (float)n + p.eps);
+#pragma unroll
+  for (int c = 0; c < 8; ++c) {
+    const int i = (c * 32 + lane) * 8;
+    if (i < n) {
+      float w[8];
+      load4(p.w + j0 + i, *reinterpret_cast<float(*)[4]>(w));
+      load4(p.w + j0 + i + 4, *reinterpret_cast<float(*)[4]>(w + 4));
+      uint32_t o[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) o[k] = pack_bf2(g[c][2 * k] * inv * w[2 * k], g[c][2 * k + 1] * inv * w[2 * k + 1]);
+      *reinterpret_cast<uint4*>(out + i) = make_uint4(o[0], o[1], o[2], o[3]);
+    }
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) ssm_gate_norm_kernel(const SsmGateNormParams p) {
   __shared__ float red[32];
@@ -497,6 +597,12 @@ extern "C" int b200_ssm_gate_norm(const void* y, long long y_row_stride, const v
   SsmGateNormParams p{y, z, y_row_stride, z_row_stride, out_row_stride, (const float*)w_f32, out, heads, P, p_true,
                       parts, eps};
   const int n = heads * p_true / parts;
+  auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  if (dtype == 0 && p_true == P && n % 8 == 0 && n <= 2048 && aligned(y) && aligned(z) && aligned(out) && aligned(w_f32)) {
+    const long long pairs = T * parts;
+    launch_k(ssm_gate_norm_warp_kernel, dim3((unsigned)((pairs + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, p, pairs);
+    return launch_status();
+  }
   const int threads = n <= 512 ? 64 : (n <= 2048 ? 128 : 256);
   if (dtype == 0)
     launch_k(ssm_gate_norm_kernel<__nv_bfloat16>, dim3((unsigned)T, (unsigned)parts), dim3(threads), 0,

@@ -9,15 +9,16 @@
 // decay-weighted x) enters its product as a bf16 pair hi + lo with both products accumulated in fp32, which keeps
 // 16 bits of it.  Tiles of the next chunk arrive by cp.async while this one is computed.
 //
-// Warp w of 8 owns token rows 16 w .. 16 w + 15 of the chunk for y and state rows 16 w .. (then every 128) for S.
+// Warp w of 4 owns token rows 16 w .. 16 w + 15 of the chunk for y and state rows 16 w .. (then every 64) for S.  Two or
+// more CTAs share an SM, so that one's matrix products run under another's copies, exponentials and barriers.
 #pragma once
 #include "attn_bwd_mma.cuh"   // abm_frag_a, abm_frag_b_rows, abm_frag_b_cols (ldmatrix fragment loads)
 #include "ssm.cuh"
 
 namespace b200 {
 
-constexpr int SSC_L = 128;
-constexpr int SSC_THREADS = 256;
+constexpr int SSC_L = 64;
+constexpr int SSC_THREADS = 128;
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
   const int n = valid ? 16 : 0;   // 0 source bytes: the 16 destination bytes are zeroed
@@ -74,7 +75,8 @@ struct SscLayout {
 template <int NMAX, int PS>
 __global__ void __launch_bounds__(SSC_THREADS) ssm_chunk_kernel(const SsmChunkParams p) {
   using L = SscLayout<NMAX, PS>;
-  constexpr int NT = NMAX <= 128 ? 1 : NMAX / 128;   // state row tiles per warp
+  constexpr int NT = NMAX / 64;                      // state row tiles per warp
+  constexpr bool KEEP_C = NMAX <= 128;               // the warp's rows of C stay in registers
   constexpr int PT = PS / 8;
   extern __shared__ __align__(16) uint8_t ssc_smem[];
   pdl_trigger();
@@ -119,7 +121,7 @@ __global__ void __launch_bounds__(SSC_THREADS) ssm_chunk_kernel(const SsmChunkPa
   };
   load(0);
 
-  float S[NT][PT][4];   // rows 16 (warp + 8 i) + g4 (+ 8), columns 8 j + 2 t4 (+ 1)
+  float S[NT][PT][4];   // rows 16 (warp + 4 i) + g4 (+ 8), columns 8 j + 2 t4 (+ 1)
   float* st = slot < 0 ? nullptr : p.state + ((long long)slot * p.heads + h) * N * P;
 #pragma unroll
   for (int i = 0; i < NT; ++i)
@@ -127,14 +129,13 @@ __global__ void __launch_bounds__(SSC_THREADS) ssm_chunk_kernel(const SsmChunkPa
     for (int j = 0; j < PT; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int n = 16 * (warp + 8 * i) + g4 + (e >> 1) * 8, c = p0 + 8 * j + 2 * t4 + (e & 1);
+        const int n = 16 * (warp + 4 * i) + g4 + (e >> 1) * 8, c = p0 + 8 * j + 2 * t4 + (e & 1);
         S[i][j][e] = st && !fresh && n < N && c < P ? st[(long long)n * P + c] : 0.f;
       }
   auto publish_state = [&]() {
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
-      const int n0 = 16 * (warp + 8 * i);
-      if (n0 >= NMAX) break;
+      const int n0 = 16 * (warp + 4 * i);
 #pragma unroll
       for (int j = 0; j < PT; ++j)
 #pragma unroll
@@ -157,19 +158,17 @@ __global__ void __launch_bounds__(SSC_THREADS) ssm_chunk_kernel(const SsmChunkPa
     cp_async_wait<0>();
     __syncthreads();          // the tiles and the state are in place, everyone has left chunk c - 1
     if (L::STAGES == 2 && c + 1 < chunks) load(c + 1);
-    if (warp == 0) {          // inclusive sums of -exp(A_log) dt: four tokens per lane, then across the warp
-      float v[4], run = 0.f;
-#pragma unroll
-      for (int k = 0; k < 4; ++k) v[k] = run += a_head * s_dt[lane * 4 + k];
-      float before = run;
+    if (warp == 0) {          // inclusive sums of -exp(A_log) dt: two tokens per lane, then across the warp
+      const float v0 = a_head * s_dt[2 * lane], v1 = v0 + a_head * s_dt[2 * lane + 1];
+      float before = v1;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const float q = __shfl_up_sync(0xffffffffu, before, o);
         if (lane >= o) before += q;
       }
-      before -= run;
-#pragma unroll
-      for (int k = 0; k < 4; ++k) s_cum[lane * 4 + k] = before + v[k];
+      before -= v1;
+      s_cum[2 * lane] = before + v0;
+      s_cum[2 * lane + 1] = before + v1;
     }
     __syncthreads();
     const float last = s_cum[SSC_L - 1];
@@ -191,10 +190,23 @@ __global__ void __launch_bounds__(SSC_THREADS) ssm_chunk_kernel(const SsmChunkPa
       float y[PT][4];
 #pragma unroll
       for (int j = 0; j < PT; ++j) y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+      uint32_t cf[KEEP_C ? NMAX / 16 : 1][4];
+      if constexpr (KEEP_C) {
+#pragma unroll
+        for (int kk = 0; kk < NMAX / 16; ++kk)
+          if (kk < n16) abm_frag_a(sC, L::LDN, r0, kk * 16, lane, cf[kk]);
+      }
       // exp(cum_i) C_i . S
-      for (int kk = 0; kk < n16; ++kk) {
+#pragma unroll
+      for (int kk = 0; kk < NMAX / 16; ++kk) {
+        if (kk >= n16) break;
         uint32_t a[4];
-        abm_frag_a(sC, L::LDN, r0, kk * 16, lane, a);
+        if constexpr (KEEP_C) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) a[e] = cf[kk][e];
+        } else {
+          abm_frag_a(sC, L::LDN, r0, kk * 16, lane, a);
+        }
 #pragma unroll
         for (int j = 0; j < PT; j += 2) {
           uint32_t b[4];
@@ -215,37 +227,52 @@ __global__ void __launch_bounds__(SSC_THREADS) ssm_chunk_kernel(const SsmChunkPa
         y[j][2] *= e1;
         y[j][3] *= e1;
       }
-      // keys 16 at a time up to the diagonal tile
-      for (int kt = 0; kt <= warp; ++kt) {
-        float gacc[2][4] = {};
-        for (int kk = 0; kk < n16; ++kk) {
-          uint32_t a[4], b[4];
-          abm_frag_a(sC, L::LDN, r0, kk * 16, lane, a);
+      // keys 32 at a time up to the diagonal tile
+      for (int kt = 0; kt <= warp; kt += 2) {
+        float gacc[4][4] = {};
+#pragma unroll
+        for (int kk = 0; kk < NMAX / 16; ++kk) {
+          if (kk >= n16) break;
+          uint32_t a[4], b[4], b2[4];
+          if constexpr (KEEP_C) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) a[e] = cf[kk][e];
+          } else {
+            abm_frag_a(sC, L::LDN, r0, kk * 16, lane, a);
+          }
           abm_frag_b_rows(sB, L::LDN, kt * 16, kk * 16, lane, b);
+          abm_frag_b_rows(sB, L::LDN, kt * 16 + 16, kk * 16, lane, b2);
           mma_bf16_16816(gacc[0], a[0], a[1], a[2], a[3], b[0], b[1]);
           mma_bf16_16816(gacc[1], a[0], a[1], a[2], a[3], b[2], b[3]);
-        }
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          const int j0 = kt * 16 + q * 8 + 2 * t4;
-          const float c0 = s_cum[j0], c1 = s_cum[j0 + 1], d0 = s_dt[j0], d1 = s_dt[j0 + 1];
-          const int i0 = r0 + g4, i1 = i0 + 8;
-          const float w00 = j0 <= i0 ? gacc[q][0] * (expf(cum0 - c0) * d0) : 0.f;
-          const float w01 = j0 + 1 <= i0 ? gacc[q][1] * (expf(cum0 - c1) * d1) : 0.f;
-          const float w10 = j0 <= i1 ? gacc[q][2] * (expf(cum1 - c0) * d0) : 0.f;
-          const float w11 = j0 + 1 <= i1 ? gacc[q][3] * (expf(cum1 - c1) * d1) : 0.f;
-          split_bf2(w00, w01, hi[2 * q], lo[2 * q]);
-          split_bf2(w10, w11, hi[2 * q + 1], lo[2 * q + 1]);
+          mma_bf16_16816(gacc[2], a[0], a[1], a[2], a[3], b2[0], b2[1]);
+          mma_bf16_16816(gacc[3], a[0], a[1], a[2], a[3], b2[2], b2[3]);
         }
 #pragma unroll
-        for (int j = 0; j < PT; j += 2) {
-          uint32_t b[4];
-          abm_frag_b_cols(sX, L::LDP, kt * 16, j * 8, lane, b);
-          mma_bf16_16816(y[j], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
-          mma_bf16_16816(y[j], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
-          mma_bf16_16816(y[j + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
-          mma_bf16_16816(y[j + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
+        for (int half = 0; half < 2; ++half) {
+          if (kt + half > warp) break;
+          uint32_t hi[4], lo[4];
+#pragma unroll
+          for (int q = 0; q < 2; ++q) {
+            const float(&gv)[4] = gacc[2 * half + q];
+            const int j0 = (kt + half) * 16 + q * 8 + 2 * t4;
+            const float c0 = s_cum[j0], c1 = s_cum[j0 + 1], d0 = s_dt[j0], d1 = s_dt[j0 + 1];
+            const int i0 = r0 + g4, i1 = i0 + 8;
+            const float w00 = j0 <= i0 ? gv[0] * (__expf(cum0 - c0) * d0) : 0.f;
+            const float w01 = j0 + 1 <= i0 ? gv[1] * (__expf(cum0 - c1) * d1) : 0.f;
+            const float w10 = j0 <= i1 ? gv[2] * (__expf(cum1 - c0) * d0) : 0.f;
+            const float w11 = j0 + 1 <= i1 ? gv[3] * (__expf(cum1 - c1) * d1) : 0.f;
+            split_bf2(w00, w01, hi[2 * q], lo[2 * q]);
+            split_bf2(w10, w11, hi[2 * q + 1], lo[2 * q + 1]);
+          }
+#pragma unroll
+          for (int j = 0; j < PT; j += 2) {
+            uint32_t b[4];
+            abm_frag_b_cols(sX, L::LDP, (kt + half) * 16, j * 8, lane, b);
+            mma_bf16_16816(y[j], hi[0], hi[1], hi[2], hi[3], b[0], b[1]);
+            mma_bf16_16816(y[j + 1], hi[0], hi[1], hi[2], hi[3], b[2], b[3]);
+            mma_bf16_16816(y[j], lo[0], lo[1], lo[2], lo[3], b[0], b[1]);
+            mma_bf16_16816(y[j + 1], lo[0], lo[1], lo[2], lo[3], b[2], b[3]);
+          }
         }
       }
 #pragma unroll
@@ -266,13 +293,15 @@ __global__ void __launch_bounds__(SSC_THREADS) ssm_chunk_kernel(const SsmChunkPa
     const int ktiles = (min(SSC_L, len - base) + 15) / 16;
 #pragma unroll
     for (int i = 0; i < NT; ++i) {
-      const int n0 = 16 * (warp + 8 * i);
+      const int n0 = 16 * (warp + 4 * i);
 #pragma unroll
       for (int j = 0; j < PT; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) S[i][j][e] *= keep;
       if (n0 < N) {
-        for (int kt = 0; kt < ktiles; ++kt) {
+#pragma unroll
+        for (int kt = 0; kt < SSC_L / 16; ++kt) {
+          if (kt >= ktiles) break;
           uint32_t a[4], b[4];
           frag_a_trans(sB, L::LDN, n0, kt * 16, lane, a);
 #pragma unroll
@@ -297,7 +326,7 @@ __global__ void __launch_bounds__(SSC_THREADS) ssm_chunk_kernel(const SsmChunkPa
       for (int j = 0; j < PT; ++j)
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-          const int n = 16 * (warp + 8 * i) + g4 + 8 * half, c = p0 + 8 * j + 2 * t4;
+          const int n = 16 * (warp + 4 * i) + g4 + 8 * half, c = p0 + 8 * j + 2 * t4;
           if (n < N && c < P)
             *reinterpret_cast<float2*>(st + (long long)n * P + c) = make_float2(S[i][j][2 * half], S[i][j][2 * half + 1]);
         }
