@@ -104,6 +104,21 @@ __global__ void __launch_bounds__(128) ssm_conv_seq_kernel(const SsmConvParams p
     T* st = slot < 0 ? nullptr
                      : reinterpret_cast<T*>(p.conv_state) + (long long)slot * (p.taps - 1) * p.channels;
     T* act = reinterpret_cast<T*>(p.act);
+    if (len == 1 && p.taps == 4 && st) {   // a decoded token: every load at once, then the shift from registers
+      const float4 w = *reinterpret_cast<const float4*>(p.w + (long long)c * 4);
+      const T zero = from_f32<T>(0.f), x = proj[(long long)t0 * p.proj_stride + p.conv_off + c];
+      const T s0 = fresh ? zero : st[c], s1 = fresh ? zero : st[p.channels + c], s2 = fresh ? zero : st[2 * p.channels + c];
+      float a = p.bias[c];
+      a = fmaf(w.x, to_f32(s0), a);
+      a = fmaf(w.y, to_f32(s1), a);
+      a = fmaf(w.z, to_f32(s2), a);
+      a = fmaf(w.w, to_f32(x), a);
+      act[(long long)t0 * p.channels + c] = from_f32<T>(silu_as<T>(a));
+      st[c] = s1;
+      st[p.channels + c] = s2;
+      st[2 * p.channels + c] = x;
+      return;
+    }
     for (int j = 0; j < len; ++j)
       act[(long long)(t0 + j) * p.channels + c] =
           from_f32<T>(ssm_conv_at<T>(p, proj, fresh ? nullptr : st, c, t0, j));
