@@ -377,16 +377,17 @@ def test_absorbed_attention_leaves_other_lengths_alone_and_does_not_depend_on_th
         at += n
 
 
+@pytest.mark.parametrize("longest", [130, 100])       # two and one row tiles per warp
 @pytest.mark.parametrize("H,DN,DR,R,V,page", [(2, 24, 16, 40, 40, 16), (3, 64, 64, 64, 64, 64), (1, 128, 64, 136, 128, 64),
                                               (2, 160, 96, 64, 256, 32), (4, 8, 8, 8, 8, 16)])
-def test_expanded_attention(H, DN, DR, R, V, page):
+def test_expanded_attention(H, DN, DR, R, V, page, longest):
     """Long portions at the start, after a cached context and in the middle of pages, beside a decoded token."""
     from vexact_b200 import latent_attention as la
 
     dq = DN + DR
     w = _lat_weights(H, DN, DR, R, V, dq ** -0.5)
     w.w_kv = _rand(H * (DN + V), R, seed=7, std=R ** -0.5, dtype=BF).cuda()
-    lens = [(17, 17), (1, 33), (130, 130), (64, 331), (100, 165), (18, 500)]
+    lens = [(17, 17), (1, 33), (longest, longest), (64, 331), (100, 165), (18, 500)]
     st = hu.step(lens, page=page)
     T = sum(n for n, _ in lens)
     q = _rand(T, H * dq + 16, seed=1, dtype=BF)

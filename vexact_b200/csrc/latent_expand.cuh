@@ -7,8 +7,9 @@
 //   q         [T, q_stride]: per head DN unrotated, then DR rotated columns
 //   out[t, h] = sigmoid(gate[t, h]) * sum_j softmax(scale q.k_j) v_j
 //
-// One CTA per (128 queries, head, sequence); warp w owns query rows 16 w .. 16 w + 15; 64 keys per block, double
-// buffered with cp.async.  Scores and weights stay fp32: a weight enters the value product as a bf16 pair hi + lo.
+// One CTA per (128 MT queries, head, sequence); warp w of 8 owns query rows 16 MT w .. 16 MT (w + 1) - 1 (MT = 2 for long
+// portions: every key and value fragment read from shared memory then serves two products); 64 keys per block, double
+// buffered with cp.async, 32 per softmax step.  Scores and weights stay fp32: a weight enters the value product as a bf16 pair hi + lo.
 // Query tiles are dealt from a sequence's last (longest) to its first.
 #pragma once
 #include "attn_tc.cuh"     // fast_exp2
@@ -17,7 +18,7 @@
 
 namespace b200 {
 
-constexpr int LEX_BM = 128, LEX_BN = 64, LEX_THREADS = 256;
+constexpr int LEX_BN = 64, LEX_SUB = 32, LEX_THREADS = 256;
 
 struct LatentExpandParams {
   const int* query_start_loc;
@@ -34,16 +35,18 @@ struct LatentExpandParams {
   float scale_log2;
 };
 
-template <int DK, int DV>
+template <int DK, int DV, int MT>
 struct LexLayout {
+  static constexpr int BM = 128 * MT;
   static constexpr int LDK = DK + 8, LDV = DV + 8;
-  static constexpr int Q = LEX_BM * LDK * 2, K = LEX_BN * LDK * 2, V = LEX_BN * LDV * 2;
+  static constexpr int Q = BM * LDK * 2, K = LEX_BN * LDK * 2, V = LEX_BN * LDV * 2;
   static constexpr int BYTES = Q + 2 * (K + V);
 };
 
-template <int DK, int DV>
-__global__ void __launch_bounds__(LEX_THREADS) latent_expand_kernel(const LatentExpandParams p) {
-  using L = LexLayout<DK, DV>;
+template <int DK, int DV, int MT>
+__global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const LatentExpandParams p) {
+  using L = LexLayout<DK, DV, MT>;
+  constexpr int LEX_BM = L::BM, NS = LEX_SUB / 8;
   extern __shared__ __align__(16) uint8_t lex_smem[];
   pdl_trigger();
   pdl_wait();
@@ -91,12 +94,19 @@ __global__ void __launch_bounds__(LEX_THREADS) latent_expand_kernel(const Latent
   };
   load(0);
 
-  float o[DV / 8][4];
+  float o[MT][DV / 8][4];
 #pragma unroll
-  for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-  float m[2] = {-3.0e38f, -3.0e38f}, l[2] = {0.f, 0.f};
-  const int r0 = 16 * warp;
-  const int pos0 = past + row_base + r0 + g4;                    // position of row g4 of the warp (and + 8)
+  for (int t = 0; t < MT; ++t)
+#pragma unroll
+    for (int j = 0; j < DV / 8; ++j) o[t][j][0] = o[t][j][1] = o[t][j][2] = o[t][j][3] = 0.f;
+  float m[MT][2], l[MT][2];
+#pragma unroll
+  for (int t = 0; t < MT; ++t) {
+    m[t][0] = m[t][1] = -3.0e38f;
+    l[t][0] = l[t][1] = 0.f;
+  }
+  const int r0 = 16 * MT * warp;
+  const int first_pos = past + row_base + r0;                    // position of the warp's first row
   for (int b = 0; b < blocks; ++b) {
     if (b + 1 < blocks) {
       load(b + 1);
@@ -105,106 +115,133 @@ __global__ void __launch_bounds__(LEX_THREADS) latent_expand_kernel(const Latent
       cp_async_wait<0>();
     }
     __syncthreads();
-    const int base = b * LEX_BN;
     const uint32_t sk = smem + L::Q + (b & 1) * (L::K + L::V), sv = sk + L::K;
-    if (r0 < rows && base <= past + row_base + r0 + 15) {
-      float s[LEX_BN / 8][4];
+#pragma unroll 1
+    for (int sub = 0; sub < LEX_BN / LEX_SUB; ++sub) {
+      const int base = b * LEX_BN + sub * LEX_SUB;
+      if (r0 >= rows || base > first_pos + 16 * MT - 1) break;   // no row of this warp sees these keys
+      float s[MT][NS][4];
 #pragma unroll
-      for (int j = 0; j < LEX_BN / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+      for (int t = 0; t < MT; ++t)
+#pragma unroll
+        for (int j = 0; j < NS; ++j) s[t][j][0] = s[t][j][1] = s[t][j][2] = s[t][j][3] = 0.f;
 #pragma unroll 4
       for (int kk = 0; kk < dk16; ++kk) {
-        uint32_t a[4], kb[4];
-        abm_frag_a(smem, L::LDK, r0, kk * 16, lane, a);
+        uint32_t a[MT][4], kb[4];
 #pragma unroll
-        for (int j = 0; j < LEX_BN / 8; j += 2) {
-          abm_frag_b_rows(sk, L::LDK, j * 8, kk * 16, lane, kb);
-          mma_bf16_16816(s[j], a[0], a[1], a[2], a[3], kb[0], kb[1]);
-          mma_bf16_16816(s[j + 1], a[0], a[1], a[2], a[3], kb[2], kb[3]);
+        for (int t = 0; t < MT; ++t) abm_frag_a(smem, L::LDK, r0 + 16 * t, kk * 16, lane, a[t]);
+#pragma unroll
+        for (int j = 0; j < NS; j += 2) {
+          abm_frag_b_rows(sk, L::LDK, sub * LEX_SUB + j * 8, kk * 16, lane, kb);
+#pragma unroll
+          for (int t = 0; t < MT; ++t) {
+            mma_bf16_16816(s[t][j], a[t][0], a[t][1], a[t][2], a[t][3], kb[0], kb[1]);
+            mma_bf16_16816(s[t][j + 1], a[t][0], a[t][1], a[t][2], a[t][3], kb[2], kb[3]);
+          }
         }
       }
-      float mb[2] = {m[0], m[1]};
-      const bool edge = base + LEX_BN - 1 > past + row_base + r0;   // some (row, key) of this block is masked
+      const bool edge = base + LEX_SUB - 1 > first_pos;           // some (row, key) of these is masked
 #pragma unroll
-      for (int j = 0; j < LEX_BN / 8; ++j)
+      for (int t = 0; t < MT; ++t) {
+        const int pos0 = first_pos + 16 * t + g4;                 // position of row g4 of the tile (and + 8)
+        float mb[2] = {m[t][0], m[t][1]};
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          float v = s[j][e] * p.scale_log2;
-          if (edge && base + 8 * j + 2 * t4 + (e & 1) > pos0 + 8 * (e >> 1)) v = -INFINITY;
-          s[j][e] = v;
-          mb[e >> 1] = fmaxf(mb[e >> 1], v);
+        for (int j = 0; j < NS; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            float v = s[t][j][e] * p.scale_log2;
+            if (edge && base + 8 * j + 2 * t4 + (e & 1) > pos0 + 8 * (e >> 1)) v = -INFINITY;
+            s[t][j][e] = v;
+            mb[e >> 1] = fmaxf(mb[e >> 1], v);
+          }
+        float alpha[2], sum[2] = {0.f, 0.f};
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          mb[e] = abm_quad_max(mb[e]);
+          alpha[e] = fast_exp2(m[t][e] - mb[e]);
         }
-      float alpha[2], sum[2] = {0.f, 0.f};
+        const bool moved = mb[0] > m[t][0] || mb[1] > m[t][1];
+        m[t][0] = mb[0];
+        m[t][1] = mb[1];
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        mb[e] = abm_quad_max(mb[e]);
-        alpha[e] = fast_exp2(m[e] - mb[e]);
-        m[e] = mb[e];
+        for (int j = 0; j < NS; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            s[t][j][e] = fast_exp2(s[t][j][e] - m[t][e >> 1]);
+            sum[e >> 1] += s[t][j][e];
+          }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) l[t][e] = l[t][e] * alpha[e] + sum[e];   // the quad's four shares meet at the end
+        if (__any_sync(0xffffffffu, moved)) {                     // otherwise every factor is exactly 1
+#pragma unroll
+          for (int j = 0; j < DV / 8; ++j) {
+            o[t][j][0] *= alpha[0];
+            o[t][j][1] *= alpha[0];
+            o[t][j][2] *= alpha[1];
+            o[t][j][3] *= alpha[1];
+          }
+        }
       }
 #pragma unroll
-      for (int j = 0; j < LEX_BN / 8; ++j)
+      for (int kt = 0; kt < LEX_SUB / 16; ++kt) {
+        uint32_t hi[MT][4], lo[MT][4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          s[j][e] = fast_exp2(s[j][e] - m[e >> 1]);
-          sum[e >> 1] += s[j][e];
-        }
+        for (int t = 0; t < MT; ++t)
 #pragma unroll
-      for (int e = 0; e < 2; ++e) l[e] = l[e] * alpha[e] + sum[e];   // the quad's four shares meet at the end
-#pragma unroll
-      for (int j = 0; j < DV / 8; ++j) {
-        o[j][0] *= alpha[0];
-        o[j][1] *= alpha[0];
-        o[j][2] *= alpha[1];
-        o[j][3] *= alpha[1];
-      }
-#pragma unroll
-      for (int kt = 0; kt < LEX_BN / 16; ++kt) {
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          split_bf2(s[2 * kt + q][0], s[2 * kt + q][1], hi[2 * q], lo[2 * q]);
-          split_bf2(s[2 * kt + q][2], s[2 * kt + q][3], hi[2 * q + 1], lo[2 * q + 1]);
-        }
+          for (int q = 0; q < 2; ++q) {
+            const float(&w)[4] = s[t][2 * kt + q];
+            split_bf2(w[0], w[1], hi[t][2 * q], lo[t][2 * q]);
+            split_bf2(w[2], w[3], hi[t][2 * q + 1], lo[t][2 * q + 1]);
+          }
 #pragma unroll
         for (int j = 0; j < DV / 8; j += 2) {
           if (j * 8 >= p.DV) break;
           uint32_t vb[4];
-          abm_frag_b_cols(sv, L::LDV, kt * 16, j * 8, lane, vb);
-          mma_bf16_16816(o[j], hi[0], hi[1], hi[2], hi[3], vb[0], vb[1]);
-          mma_bf16_16816(o[j + 1], hi[0], hi[1], hi[2], hi[3], vb[2], vb[3]);
-          mma_bf16_16816(o[j], lo[0], lo[1], lo[2], lo[3], vb[0], vb[1]);
-          mma_bf16_16816(o[j + 1], lo[0], lo[1], lo[2], lo[3], vb[2], vb[3]);
+          abm_frag_b_cols(sv, L::LDV, sub * LEX_SUB + kt * 16, j * 8, lane, vb);
+#pragma unroll
+          for (int t = 0; t < MT; ++t) {
+            mma_bf16_16816(o[t][j], hi[t][0], hi[t][1], hi[t][2], hi[t][3], vb[0], vb[1]);
+            mma_bf16_16816(o[t][j + 1], hi[t][0], hi[t][1], hi[t][2], hi[t][3], vb[2], vb[3]);
+          }
+#pragma unroll
+          for (int t = 0; t < MT; ++t) {
+            mma_bf16_16816(o[t][j], lo[t][0], lo[t][1], lo[t][2], lo[t][3], vb[0], vb[1]);
+            mma_bf16_16816(o[t][j + 1], lo[t][0], lo[t][1], lo[t][2], lo[t][3], vb[2], vb[3]);
+          }
         }
       }
     }
     __syncthreads();
   }
 #pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    const float inv = 1.f / abm_quad_sum(l[e]);
-    const int r = r0 + g4 + 8 * e;
-    if (r >= rows) continue;
-    const long long t = t0 + row_base + r;
+  for (int tt = 0; tt < MT; ++tt)
 #pragma unroll
-    for (int j = 0; j < DV / 8; ++j) {
-      const int c = 8 * j + 2 * t4;
-      if (c < p.DV) {
-        float ga, gb;
-        unpack_bf2(*reinterpret_cast<const uint32_t*>(p.gate + t * p.gate_stride + (long long)h * p.DV + c), ga, gb);
-        *reinterpret_cast<uint32_t*>(p.out + t * p.out_stride + (long long)h * p.DV + c) =
-            pack_bf2(o[j][2 * e] * inv * __fdividef(1.f, 1.f + __expf(-ga)),
-                     o[j][2 * e + 1] * inv * __fdividef(1.f, 1.f + __expf(-gb)));
+    for (int e = 0; e < 2; ++e) {
+      const float inv = 1.f / abm_quad_sum(l[tt][e]);
+      const int r = r0 + 16 * tt + g4 + 8 * e;
+      if (r >= rows) continue;
+      const long long t = t0 + row_base + r;
+#pragma unroll
+      for (int j = 0; j < DV / 8; ++j) {
+        const int c = 8 * j + 2 * t4;
+        if (c < p.DV) {
+          float ga, gb;
+          unpack_bf2(*reinterpret_cast<const uint32_t*>(p.gate + t * p.gate_stride + (long long)h * p.DV + c), ga, gb);
+          *reinterpret_cast<uint32_t*>(p.out + t * p.out_stride + (long long)h * p.DV + c) =
+              pack_bf2(o[tt][j][2 * e] * inv * __fdividef(1.f, 1.f + __expf(-ga)),
+                       o[tt][j][2 * e + 1] * inv * __fdividef(1.f, 1.f + __expf(-gb)));
+        }
       }
     }
-  }
 }
 
-template <int DK, int DV>
+template <int DK, int DV, int MT>
 inline int latent_expand_launch(const LatentExpandParams& p, int max_len, int n, cudaStream_t st) {
-  constexpr int smem = LexLayout<DK, DV>::BYTES;
+  constexpr int smem = LexLayout<DK, DV, MT>::BYTES, LEX_BM = LexLayout<DK, DV, MT>::BM;
   static_assert(smem <= 227 * 1024, "shared memory budget");
   static PerDeviceFlags attr_set;
-  if (int rc = set_max_dyn_smem_once(attr_set, latent_expand_kernel<DK, DV>, smem)) return rc;
-  launch_k(latent_expand_kernel<DK, DV>, dim3((unsigned)((max_len + LEX_BM - 1) / LEX_BM), (unsigned)p.heads, (unsigned)n),
+  if (int rc = set_max_dyn_smem_once(attr_set, latent_expand_kernel<DK, DV, MT>, smem)) return rc;
+  launch_k(latent_expand_kernel<DK, DV, MT>, dim3((unsigned)((max_len + LEX_BM - 1) / LEX_BM), (unsigned)p.heads, (unsigned)n),
            dim3(LEX_THREADS), (size_t)smem, st, p);
   return launch_status();
 }
@@ -233,8 +270,11 @@ extern "C" int b200_latent_attn_expanded(const void* q, long long q_row_stride, 
                        scale * kLog2e};
   const int dk = DN + DR;
   const cudaStream_t st = (cudaStream_t)stream;
-  if (dk <= 64 && DV <= 64) return latent_expand_launch<64, 64>(p, max_len, n, st);
-  if (dk <= 128 && DV <= 128) return latent_expand_launch<128, 128>(p, max_len, n, st);
-  if (dk <= 192 && DV <= 128) return latent_expand_launch<192, 128>(p, max_len, n, st);
-  return latent_expand_launch<256, 256>(p, max_len, n, st);
+  const bool two = max_len > 128;
+  if (dk <= 64 && DV <= 64) return two ? latent_expand_launch<64, 64, 2>(p, max_len, n, st) : latent_expand_launch<64, 64, 1>(p, max_len, n, st);
+  if (dk <= 128 && DV <= 128)
+    return two ? latent_expand_launch<128, 128, 2>(p, max_len, n, st) : latent_expand_launch<128, 128, 1>(p, max_len, n, st);
+  if (dk <= 192 && DV <= 128)
+    return two ? latent_expand_launch<192, 128, 2>(p, max_len, n, st) : latent_expand_launch<192, 128, 1>(p, max_len, n, st);
+  return latent_expand_launch<256, 256, 1>(p, max_len, n, st);
 }
