@@ -451,7 +451,7 @@ int b200_ssm_chunk_scan(const void* act, long long act_row_stride, const void* d
                         const void* context_lens, const void* state_slots, int num_seqs, int num_slots, int heads,
                         int groups, int N, int P, int min_len, int slice, void* stream);
 /* b200_latent_attn_simt on tcgen05 tensor cores (bf16).  b200_latent_plan lists the work of a step once for all layers
- * with `heads` heads: items [max_items][4], item_count [1], first_item [num_seqs], i32; at most max_items =
+ * with `heads` heads: items [max_items][8], item_count [1], first_item [num_seqs], i32; at most max_items =
  * sum over sequences of ceil(new tokens * heads / 16) * ceil(context / 512).  R <= 512, DR <= 128, multiples of 8;
  * page_size a power of two of at least 8 or a multiple of 128.  part_o [max_items, 16, R], part_ml [max_items, 16, 2]
  * fp32 scratch, NULL when no context exceeds 512 tokens. */

@@ -15,6 +15,10 @@
 // Boxes of c travel in pairs (128 dims, one UMMA M block) through a ring of slots that are given back one by one as the
 // value product has read them; the boxes of k_rot have slots of their own, free again after QK^T.
 //
+// O^T stays in tensor memory across blocks.  A column's reference maximum moves only when a block's maximum exceeds it by
+// more than 2^8 (weights up to 2^8 are as exact as weights up to 1); then the sums so far are taken into registers and
+// rescaled, and O^T starts anew.
+//
 // Persistent CTAs take items (sequence, column tile, split) from a list made once per step (latent_plan_kernel).
 // Warps: 0 = TMA producer, 1 = UMMA issuer and TMEM owner, 2..9 = softmax and accumulation (thread = TMEM lane, half of
 // the columns), 10 = query loader.  A row whose sequence has one split is finished here, otherwise
@@ -31,13 +35,14 @@ namespace b200 {
 constexpr int LTC_BN = 128, LTC_NC = 16, LTC_SPLIT = 512, LTC_THREADS = 352;
 constexpr int LTC_BOX = LTC_BN * 128;             // bytes of a 128-key x 64-column box
 constexpr int LTC_MAX_PAIRS = 6;
+constexpr float LTC_SLACK = 8.f;                  // log2 of how far a weight may exceed 1 before the rescale
 constexpr int LTC_SMEM = 225 * 1024;          // always this much: one CTA per SM (the static arrays are beside it)
 
 struct LatentTcParams {
   LatentSeqs seqs;
   const __nv_bfloat16* q_lat;   // [T, H, R + DR]
   __nv_bfloat16* out;           // [T, H, R]
-  const int4* items;            // {sequence, column tile, split, splits of the sequence}
+  const int4* items;            // pairs {sequence, first token, new tokens, context}, {column tile, split, splits, 0}
   const int* item_count;
   int max_items;
   float* part_o;                // [items, 16, R]
@@ -66,12 +71,14 @@ __global__ void __launch_bounds__(1024) latent_plan_kernel(const LatentPlanParam
   __syncthreads();
   for (int s0 = 0; s0 < p.seqs.num_seqs; s0 += 1024) {
     const int s = s0 + tid;
-    int tiles = 0, splits = 0;
+    int tiles = 0, splits = 0, t0 = 0, len = 0, ctx = 0;
     if (s < p.seqs.num_seqs) {
-      const int len = p.seqs.query_start_loc[s + 1] - p.seqs.query_start_loc[s];
+      t0 = p.seqs.query_start_loc[s];
+      len = p.seqs.query_start_loc[s + 1] - t0;
+      ctx = p.seqs.context_lens[s];
       if (len >= p.seqs.min_len && len <= p.seqs.max_len && len > 0) {
         tiles = (len * p.heads + LTC_NC - 1) / LTC_NC;
-        splits = (p.seqs.context_lens[s] + LTC_SPLIT - 1) / LTC_SPLIT;
+        splits = (ctx + LTC_SPLIT - 1) / LTC_SPLIT;
       }
     }
     const int n = tiles * splits;
@@ -88,8 +95,10 @@ __global__ void __launch_bounds__(1024) latent_plan_kernel(const LatentPlanParam
     const int first = before + inc - n;
     if (s < p.seqs.num_seqs) p.first_item[s] = first;
     for (int i = 0; i < n; ++i) {
-      if (first + i < p.max_items) p.items[first + i] = make_int4(s, i / splits, i % splits, splits);
-      else report_status(B200_STATUS_BAD_INDEX, first + i);
+      if (first + i < p.max_items) {
+        p.items[2 * (first + i)] = make_int4(s, t0, len, ctx);
+        p.items[2 * (first + i) + 1] = make_int4(i / splits, i % splits, splits, 0);
+      } else report_status(B200_STATUS_BAD_INDEX, first + i);
     }
     __syncthreads();
     if (tid == 1023) s_base = before + inc;
@@ -145,26 +154,46 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentCombine
   }
 }
 
-// One item's extent.
+// One item's extent.  The two words of its description are read an item ahead (LtcRaw), so that nobody waits for them.
+struct LtcRaw {
+  int4 a, b;
+};
 struct LtcItem {
-  int seq, tile, split, splits, t0, len, ctx, key0, key_end, nblk, rows;
+  int seq, tile, splits, t0, len, ctx, key0, nblk, rows;
 };
 
-__device__ __forceinline__ LtcItem ltc_item(const LatentTcParams& p, int idx) {
-  const int4 e = p.items[idx];
+__device__ __forceinline__ LtcRaw ltc_raw(const LatentTcParams& p, int idx, int count) {
+  const int i = min(idx, count - 1);
+  return LtcRaw{p.items[2 * i], p.items[2 * i + 1]};
+}
+__device__ __forceinline__ LtcItem ltc_item(const LatentTcParams& p, const LtcRaw& r) {
   LtcItem t;
-  t.seq = e.x;
-  t.tile = e.y;
-  t.split = e.z;
-  t.splits = e.w;
-  t.t0 = p.seqs.query_start_loc[e.x];
-  t.len = p.seqs.query_start_loc[e.x + 1] - t.t0;
-  t.ctx = p.seqs.context_lens[e.x];
-  t.key0 = e.z * LTC_SPLIT;
-  t.key_end = min(t.ctx, t.key0 + LTC_SPLIT);
-  t.nblk = (t.key_end - t.key0 + LTC_BN - 1) / LTC_BN;
-  t.rows = min(LTC_NC, t.len * p.heads - e.y * LTC_NC);
+  t.seq = r.a.x;
+  t.t0 = r.a.y;
+  t.len = r.a.z;
+  t.ctx = r.a.w;
+  t.tile = r.b.x;
+  t.splits = r.b.z;
+  t.key0 = r.b.y * LTC_SPLIT;
+  t.nblk = (min(t.ctx, t.key0 + LTC_SPLIT) - t.key0 + LTC_BN - 1) / LTC_BN;
+  t.rows = min(LTC_NC, t.len * p.heads - t.tile * LTC_NC);
   return t;
+}
+
+// Named barrier 3 of the compute warps with a vote: true when any of the n threads brings true.
+__device__ __forceinline__ bool barrier_any(bool mine, int n) {
+  uint32_t any;
+  asm volatile(
+      "{\n"
+      ".reg .pred p, q;\n"
+      "setp.ne.u32 q, %1, 0;\n"
+      "barrier.cta.red.or.pred p, 3, %2, q;\n"
+      "selp.u32 %0, 1, 0, p;\n"
+      "}\n"
+      : "=r"(any)
+      : "r"((uint32_t)mine), "r"(n)
+      : "memory");
+  return any != 0;
 }
 
 __device__ __forceinline__ void tmem_ld8(uint32_t taddr, uint32_t* r) {
@@ -179,10 +208,9 @@ __global__ void __launch_bounds__(LTC_THREADS, 1)
 latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p) {
   constexpr int NC = LTC_NC, NH = NC / 2;
   constexpr int TMEM_COLS = 2 * NC + CP * 2 * NC <= 64 ? 64 : 2 * NC + CP * 2 * NC <= 128 ? 128 : 256;
-  constexpr int P_BYTES = 2 * 2 * NC * 128;
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t bars[2 * LTC_MAX_PAIRS + 4 + 4 + 3 + 4];
-  __shared__ int abort_mem;
+  __shared__ int abort_mem, s_fresh;
   __shared__ uint32_t tmem_slot;
   __shared__ __align__(16) float s_wmax[2][NC][4];
   __shared__ __align__(16) float s_lred[NC][4];
@@ -201,8 +229,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
   auto rempty = [&](int s) { return bar(2 * LTC_MAX_PAIRS + 2 + s); };
   auto sfull = [&](int b) { return bar(2 * LTC_MAX_PAIRS + 4 + b); };
   auto sfree = [&](int b) { return bar(2 * LTC_MAX_PAIRS + 6 + b); };
-  const uint32_t pready = bar(2 * LTC_MAX_PAIRS + 8), ofull = bar(2 * LTC_MAX_PAIRS + 9),
-                 ofree = bar(2 * LTC_MAX_PAIRS + 10);
+  const uint32_t pready = bar(2 * LTC_MAX_PAIRS + 8), ofull = bar(2 * LTC_MAX_PAIRS + 9);
   auto qfull = [&](int b) { return bar(2 * LTC_MAX_PAIRS + 11 + b); };
   auto qfree = [&](int b) { return bar(2 * LTC_MAX_PAIRS + 13 + b); };
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -223,7 +250,6 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
     }
     ptx::mbar_init(pready, 8);
     ptx::mbar_init(ofull, 1);
-    ptx::mbar_init(ofree, 8);
     ptx::fence_barrier_init();
     ptx::prefetch_tensormap(&tm);
   }
@@ -239,22 +265,32 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
   pdl_wait();
   const int count = *p.item_count;
 
-  if (warp == 0) {
+  if (count == 0) {
+    // nothing to do: straight to the teardown
+  } else if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer (whole warp)
     const int subs = LTC_BN / p.box_tokens;      // boxes of one page's tokens per 128 keys
     const long long none = (long long)p.seqs.num_blocks * p.seqs.page_size;   // past the tensor: zeros arrive
+    auto row_of = [&](const LtcItem& t, int j) -> int {      // first cache row of this lane's box of block j
+      const int key = t.key0 + j * LTC_BN + lane * p.box_tokens;
+      if (lane >= subs || key >= t.ctx) return (int)none;
+      const long long row = latent_key_row(p.seqs, t.seq, key);
+      return row < 0 ? (int)none : (int)row;
+    };
     uint32_t pc = 0, rc = 0;
     bool ok = true;
+    LtcItem t = ltc_item(p, ltc_raw(p, blockIdx.x, count));
+    int row_next = (int)blockIdx.x < count ? row_of(t, 0) : (int)none;
     for (int idx = blockIdx.x; idx < count && ok; idx += gridDim.x) {
-      const LtcItem t = ltc_item(p, idx);
-      for (int j = 0; j < t.nblk && ok; ++j) {
-        long long row = none;
-        if (lane < subs) {
-          const int key = t.key0 + j * LTC_BN + lane * p.box_tokens;
-          if (key < t.ctx) {
-            row = latent_key_row(p.seqs, t.seq, key);
-            if (row < 0) row = none;
-          }
+      const LtcRaw raw_next = ltc_raw(p, idx + gridDim.x, count);
+      const int nblk = t.nblk;
+      for (int j = 0; j < nblk && ok; ++j) {
+        const int row = row_next;       // the look-up of the next block runs under this block's waits
+        if (j + 1 < nblk) {
+          row_next = row_of(t, j + 1);
+        } else {
+          t = ltc_item(p, raw_next);
+          row_next = row_of(t, 0);
         }
         {
           const int s = rc % NR;
@@ -265,7 +301,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
           if (lane < subs)
             for (int b = 0; b < RB; ++b)
               ptx::tma_load_2d(base + rot_off + (uint32_t)(s * RB + b) * LTC_BOX + (uint32_t)(lane * p.box_tokens) * 128,
-                               &tm, rfull(s), R + b * 64, (int)row, ptx::kEvictFirst);
+                               &tm, rfull(s), R + b * 64, row, ptx::kEvictFirst);
           ++rc;
         }
         for (int i = 0; i < CP; ++i, ++pc) {
@@ -277,7 +313,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
           if (lane < subs)
             for (int b = 0; b < nb; ++b)
               ptx::tma_load_2d(base + (uint32_t)(2 * s + b) * LTC_BOX + (uint32_t)(lane * p.box_tokens) * 128, &tm,
-                               pfull(s), (2 * i + b) * 64, (int)row, ptx::kEvictFirst);
+                               pfull(s), (2 * i + b) * 64, row, ptx::kEvictFirst);
         }
       }
     }
@@ -288,32 +324,48 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
       const uint64_t hi_k = ptx::umma_desc_k_sw128(0) & 0xFFFFFFFF00000000ull;
       auto kdesc = [&](uint32_t a) { return hi_k | (uint64_t)(((a & 0x3FFFFu) >> 4) | (1u << 16)); };
       const bool ahead = NP >= 2 * CP;   // QK^T of the next block may be issued before this block's value product
-      uint32_t gs = 0, gp = 0, it = 0;
+      uint32_t gs = 0, gp = 0, it = 0, sph = 0;
+      int ss = 0, sp = 0;                // ring slot of the next pair of QK^T (sph: parity of its use) / of the value product
       int idx = blockIdx.x, j = 0, nblk = 0;
-      if (idx < count) nblk = ltc_item(p, idx).nblk;
+      LtcRaw raw_next = ltc_raw(p, idx, count);
+      if (idx < count) {
+        nblk = ltc_item(p, raw_next).nblk;
+        raw_next = ltc_raw(p, idx + gridDim.x, count);
+      }
       auto issue_s = [&]() {
-        const int qb = it & 1, b = gs & 1, rs = gs % NR;
+        const int qb = it & 1, b = gs & 1, rs = NR == 2 ? gs & 1 : 0;
         if (j == 0 && !ptx::mbar_wait(qfull(qb), (it >> 1) & 1, abort_flag, 720 + qb)) return false;
         if (!ptx::mbar_wait(sfree(b), ((gs >> 1) & 1) ^ 1, abort_flag, 722 + b)) return false;
-        if (!ptx::mbar_wait(rfull(rs), (gs / NR) & 1, abort_flag, 724 + rs)) return false;
+        if (!ptx::mbar_wait(rfull(rs), (NR == 2 ? gs >> 1 : gs) & 1, abort_flag, 724 + rs)) return false;
         ptx::tc_fence_after();
-        const uint32_t q0 = base + q_off + qb * q_bytes;
-        uint32_t acc = 0;
-        auto box = [&](uint32_t a, int bx, int cols) {   // one 64-column box of the contraction
-          for (int kk = 0; kk < (cols + 15) / 16; ++kk) {
-            ptx::umma_bf16(tm_s + b * NC, kdesc(a + kk * 32), kdesc(q0 + bx * (NC * 128) + kk * 32), idesc_s, acc);
-            acc = 1;
+        const uint32_t q0 = base + q_off + qb * q_bytes, d = tm_s + b * NC;
+        // one 64-column box of the contraction; descriptors step by 32 bytes (2 units) per 16 columns
+        auto box = [&](uint32_t a, int bx, int cols, uint32_t acc) {
+          const uint64_t da = kdesc(a), db = kdesc(q0 + bx * (NC * 128));
+          ptx::umma_bf16(d, da, db, idesc_s, acc);
+          if (cols > 48) {
+            ptx::umma_bf16_acc(d, da + 2, db + 2, idesc_s);
+            ptx::umma_bf16_acc(d, da + 4, db + 4, idesc_s);
+            ptx::umma_bf16_acc(d, da + 6, db + 6, idesc_s);
+          } else {
+            if (cols > 16) ptx::umma_bf16_acc(d, da + 2, db + 2, idesc_s);
+            if (cols > 32) ptx::umma_bf16_acc(d, da + 4, db + 4, idesc_s);
           }
         };
-        for (int r = 0; r < RB; ++r) box(base + rot_off + (uint32_t)(rs * RB + r) * LTC_BOX, r, min(64, DR - 64 * r));
+        for (int r = 0; r < RB; ++r)
+          box(base + rot_off + (uint32_t)(rs * RB + r) * LTC_BOX, r, min(64, DR - 64 * r), r != 0 ? 1u : 0u);
         ptx::umma_commit(rempty(rs));
+#pragma unroll
         for (int i = 0; i < CP; ++i) {
-          const uint32_t n = gs * CP + i;
-          const int s = n % NP;
-          if (!ptx::mbar_wait(pfull(s), (n / NP) & 1, abort_flag, 730 + s)) return false;
+          if (!ptx::mbar_wait(pfull(ss), sph, abort_flag, 730 + ss)) return false;
           ptx::tc_fence_after();
-          for (int h = 0; h < 2 && 2 * i + h < CB; ++h)
-            box(base + (uint32_t)(2 * s + h) * LTC_BOX, RB + 2 * i + h, min(64, R - 64 * (2 * i + h)));
+          const uint32_t a = base + (uint32_t)(2 * ss) * LTC_BOX;
+          box(a, RB + 2 * i, min(64, R - 128 * i), 1u);
+          if (2 * i + 1 < CB) box(a + LTC_BOX, RB + 2 * i + 1, min(64, R - 128 * i - 64), 1u);
+          if (++ss == NP) {
+            ss = 0;
+            sph ^= 1;
+          }
         }
         ptx::umma_commit(sfull(b));
         ++gs;
@@ -322,7 +374,8 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
           j = 0;
           ++it;
           idx += gridDim.x;
-          if (idx < count) nblk = ltc_item(p, idx).nblk;
+          nblk = ltc_item(p, raw_next).nblk;
+          raw_next = ltc_raw(p, idx + gridDim.x, count);
         }
         return true;
       };
@@ -330,16 +383,19 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
       while (ok && gp < gs) {
         if (ahead && idx < count && !issue_s()) break;
         if (!ptx::mbar_wait(pready, gp & 1, abort_flag, 740)) break;
-        if (!ptx::mbar_wait(ofree, (gp & 1) ^ 1, abort_flag, 741)) break;
         ptx::tc_fence_after();
-        for (int i = 0; i < CP; ++i) {
-          const int s = (gp * CP + i) % NP;
-          const uint32_t a = base + (uint32_t)(2 * s) * LTC_BOX;
+        const uint32_t keep = *(volatile int*)&s_fresh ? 0u : 1u;
+        const uint64_t db = kdesc(base + p_off);
 #pragma unroll
-          for (int kk = 0; kk < LTC_BN / 16; ++kk)
-            ptx::umma_bf16(tm_o + i * 2 * NC, umma_desc_mn_sw128(a + kk * 16 * 128, LTC_BOX),
-                           kdesc(base + p_off + (kk >> 2) * (2 * NC * 128) + (kk & 3) * 32), idesc_o, kk != 0 ? 1u : 0u);
-          ptx::umma_commit(pempty(s));
+        for (int i = 0; i < CP; ++i) {
+          const uint64_t da = umma_desc_mn_sw128(base + (uint32_t)(2 * sp) * LTC_BOX, LTC_BOX);   // + 16 keys: 2 KB
+          const uint32_t d = tm_o + i * 2 * NC;
+          ptx::umma_bf16(d, da, db, idesc_o, keep);
+#pragma unroll
+          for (int kk = 1; kk < LTC_BN / 16; ++kk)
+            ptx::umma_bf16_acc(d, da + 128 * kk, db + (kk >> 2) * (2 * NC * 128 >> 4) + (kk & 3) * 2, idesc_o);
+          ptx::umma_commit(pempty(sp));
+          if (++sp == NP) sp = 0;
         }
         ptx::umma_commit(ofull);
         ++gp;
@@ -349,10 +405,12 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
   } else if (warp == 10) {
     // ------------------------------------------------------------------ query loader (whole warp), one item ahead
     uint32_t it = 0;
+    LtcRaw raw_next = ltc_raw(p, blockIdx.x, count);
     for (int idx = blockIdx.x; idx < count; idx += gridDim.x, ++it) {
-      const LtcItem t = ltc_item(p, idx);
+      const LtcItem t = ltc_item(p, raw_next);
+      raw_next = ltc_raw(p, idx + gridDim.x, count);
       const int qb = it & 1;
-      if (!ptx::mbar_wait_warp(qfree(qb), ((it >> 1) & 1) ^ 1, abort_flag, 750 + qb)) break;
+      if (!ptx::mbar_wait_warp(qfree(qb), ((it >> 1) & 1) ^ 1, abort_flag, 760 + qb)) break;
       uint8_t* qd = base_ptr + q_off + qb * q_bytes;
       const __nv_bfloat16* q = p.q_lat + ((long long)t.t0 * p.heads + t.tile * NC) * (R + DR);
 #pragma unroll 4
@@ -378,8 +436,10 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
     uint8_t* p_mine = base_ptr + p_off + (tl >> 6) * (2 * NC * 128) + (tl & 7) * 2;
     const int p_ch = (tl & 63) >> 3;
     uint32_t g = 0;
+    LtcRaw raw_next = ltc_raw(p, blockIdx.x, count);
     for (int idx = blockIdx.x; idx < count; idx += gridDim.x) {
-      const LtcItem t = ltc_item(p, idx);
+      const LtcItem t = ltc_item(p, raw_next);
+      raw_next = ltc_raw(p, idx + gridDim.x, count);
       int cpos[NH];
 #pragma unroll
       for (int i = 0; i < NH; ++i)
@@ -391,7 +451,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
 #pragma unroll
         for (int k = 0; k < CP; ++k) o[k][i] = 0.f;
       }
-      auto fold = [&](const float (&f)[NH], bool have) {   // o = (o + O^T of the last block) * f
+      auto fold = [&](const float (&f)[NH]) {   // o = (o + O^T) * f
 #pragma unroll
         for (int k = 0; k < CP; ++k) {
           uint32_t hi[NH], lo[NH];
@@ -400,27 +460,25 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
           ptx::tmem_ld_wait();
 #pragma unroll
           for (int i = 0; i < NH; ++i)
-            o[k][i] = (o[k][i] + (have ? __uint_as_float(hi[i]) + __uint_as_float(lo[i]) : 0.f)) * f[i];
+            o[k][i] = (o[k][i] + (__uint_as_float(hi[i]) + __uint_as_float(lo[i]))) * f[i];
         }
       };
       for (int j = 0; j < t.nblk; ++j, ++g) {
-        const int b = g & 1, kb = t.key0 + j * LTC_BN, key = kb + tl;
+        const int b = g & 1, key = t.key0 + j * LTC_BN + tl;
         float v[NH];
-        if (__all_sync(0xffffffffu, ptx::mbar_wait(sfull(b), (g >> 1) & 1, abort_flag, 760 + b))) {
+        bool over = j == 0;            // some weight would exceed the slack: the reference maxima have to move
+        if (__all_sync(0xffffffffu, ptx::mbar_wait(sfull(b), (g >> 1) & 1, abort_flag, 770 + b))) {
           ptx::tc_fence_after();
           uint32_t r[NH];
           tmem_ld8(tm_s + lane_addr + b * NC + c0, r);
           ptx::tmem_ld_wait();
-          float mine = -INFINITY;
 #pragma unroll
           for (int i = 0; i < NH; ++i) {
             v[i] = key > cpos[i] ? -INFINITY : __uint_as_float(r[i]) * p.scale_log2;
-            float w;
-            asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(w) : "f"(v[i]));
-            if ((lane & 7) == i) mine = w;
+            over |= v[i] > m[i] + LTC_SLACK;
           }
-          if (lane < 8) s_wmax[b][c0 + lane][q4] = mine;
           // keys past the context may hold anything: clear their rows of c so that 0 * value stays 0
+          const int kb = t.key0 + j * LTC_BN;
           if (kb + LTC_BN > t.ctx) {
             for (int k = 0; k < CP; ++k) {
               uint8_t* slot = base_ptr + (size_t)(2 * ((g * CP + k) % NP)) * LTC_BOX;
@@ -431,22 +489,47 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
             }
           }
         }
-        ptx::named_barrier_sync(3, NCT);
+        const bool rescale = barrier_any(over, NCT);
         if (*abort_flag) break;
-        bool go = true;
-        if (j > 0) go = __all_sync(0xffffffffu, ptx::mbar_wait(ofull, (g - 1) & 1, abort_flag, 762));
-        if (go) {
-          ptx::tc_fence_after();
-          float alpha[NH], e[NH], a_mine = 0.f;
+        float alpha[NH];
+#pragma unroll
+        for (int i = 0; i < NH; ++i) alpha[i] = 1.f;
+        if (rescale) {                 // uniform over the compute threads
+          float mine = -INFINITY;
+#pragma unroll
+          for (int i = 0; i < NH; ++i) {
+            float w;
+            asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(w) : "f"(v[i]));
+            if ((lane & 7) == i) mine = w;
+          }
+          if (lane < 8) s_wmax[b][c0 + lane][q4] = mine;
+          ptx::named_barrier_sync(3, NCT);
+          if (*abort_flag) break;
 #pragma unroll
           for (int i = 0; i < NH; ++i) {
             const float4 w = *reinterpret_cast<const float4*>(s_wmax[b][c0 + i]);
-            const float mn = fmaxf(m[i], fmaxf(fmaxf(w.x, w.y), fmaxf(w.z, w.w)));
-            alpha[i] = fast_exp2(m[i] - mn);
-            m[i] = mn;
-            e[i] = fast_exp2(v[i] - mn);
-            if (i == mycol) a_mine = alpha[i];
+            const float cand = fmaxf(fmaxf(w.x, w.y), fmaxf(w.z, w.w));
+            if (cand > m[i] + LTC_SLACK) {
+              alpha[i] = fast_exp2(m[i] - cand);
+              m[i] = cand;
+            }
           }
+        }
+        float e[NH], a_mine = 1.f;
+#pragma unroll
+        for (int i = 0; i < NH; ++i) {
+          e[i] = fast_exp2(v[i] - m[i]);
+          if (i == mycol) a_mine = alpha[i];
+        }
+        // every value product so far has read its P^T tile and left its sums in tensor memory
+        bool go = true;
+        if (g > 0) go = __all_sync(0xffffffffu, ptx::mbar_wait(ofull, (g - 1) & 1, abort_flag, 772));
+        if (go) {
+          if (rescale && j > 0) {
+            ptx::tc_fence_after();
+            fold(alpha);
+          }
+          if (ct == 0) s_fresh = rescale;
 #pragma unroll
           for (int i = 0; i < NH; ++i) {
             const int c = c0 + i;
@@ -455,30 +538,27 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
             *reinterpret_cast<__nv_bfloat16*>(d) = hi;
             *reinterpret_cast<__nv_bfloat16*>(d + NC * 128) = f2bf(e[i] - bf2f(hi));   // row 16 + c swizzles as row c
           }
-          fold(alpha, j > 0);
-          halving_warp_sum<NH>(e, lane);
-          l_w = l_w * a_mine + e[0];
           ptx::tc_fence_before();
           ptx::fence_proxy_async_smem();
           __syncwarp();
           if (lane == 0) {
             ptx::mbar_arrive(sfree(b));
-            if (j > 0) ptx::mbar_arrive(ofree);
             ptx::mbar_arrive(pready);
           }
+          // the row sums, while the value product runs
+          halving_warp_sum<NH>(e, lane);
+          l_w = l_w * a_mine + e[0];
         }
       }
       bool go = !*abort_flag;
-      if (go) go = __all_sync(0xffffffffu, ptx::mbar_wait(ofull, (g - 1) & 1, abort_flag, 763));
+      if (go) go = __all_sync(0xffffffffu, ptx::mbar_wait(ofull, (g - 1) & 1, abort_flag, 773));
       if (go) {
         ptx::tc_fence_after();
         float one[NH];
 #pragma unroll
         for (int i = 0; i < NH; ++i) one[i] = 1.f;
-        fold(one, true);
+        fold(one);
         ptx::tc_fence_before();
-        __syncwarp();
-        if (lane == 0) ptx::mbar_arrive(ofree);
         s_lred[c0 + mycol][q4] = l_w;
       }
       ptx::named_barrier_sync(3, NCT);
@@ -529,7 +609,7 @@ inline int latent_tc_launch(const CUtensorMap& tm, const LatentTcParams& p, int 
 
 }  // namespace b200
 
-// Work items of a step for b200_latent_attn_tc: items [max_items] int4, item_count [1], first_item [num_seqs] (i32).
+// Work items of a step for b200_latent_attn_tc: items [max_items] pairs of int4, item_count [1], first_item [num_seqs] (i32).
 // The list depends on the sequences and the head count only, so one list serves every layer with `heads` heads.
 extern "C" int b200_latent_plan(const void* query_start_loc, const void* context_lens, int num_seqs, int min_len,
                                 int max_len, int heads, int max_items, void* items, void* item_count, void* first_item,

@@ -98,7 +98,7 @@ def _tc_plan(step, heads: int, pool_tokens: int, min_len: int, max_len: int, dev
         cap = -(-min(step.max_seqlen_q, max_len) * heads // TC_COLUMNS) * (S + pool_tokens // TC_SPLIT)
         several = step.block_tables.shape[1] * step.page_size > TC_SPLIT
     cap = max(cap, 1)
-    items = torch.empty((cap, 4), device=device, dtype=torch.int32)
+    items = torch.empty((cap, 2, 4), device=device, dtype=torch.int32)
     meta = torch.empty(S + 4, device=device, dtype=torch.int32)
     _lib.check(
         _lib.load().b200_latent_plan(step.query_start_loc.data_ptr(), step.context_lens.data_ptr(), S, min_len, max_len,
