@@ -743,7 +743,7 @@ def graph_ms(calls, reps=10):
 
 
 def run_hybrid(args):
-    """Side measurement (not the contract line): prefill and decode steps of the hybrid decoder family and of the closest
+    """Side measurement: prefill and decode steps of the hybrid decoder family and of the closest
     other model at equal size (random weights), then its kernels beside the like kernels of that model."""
     from vexact_b200 import _lib
 
