@@ -325,7 +325,8 @@ def _absorbed_reference(w, q_lat, rows, new, total):
 
 
 @pytest.mark.parametrize("form,dtype", [("simt", F32), ("simt", BF), ("tc", BF)])
-@pytest.mark.parametrize("H,R,DR,page", [(3, 40, 16, 16), (1, 8, 8, 64), (16, 512, 64, 64), (5, 136, 24, 32), (20, 128, 32, 128)])
+@pytest.mark.parametrize("H,R,DR,page", [(3, 40, 16, 16), (1, 8, 8, 64), (16, 512, 64, 64), (5, 136, 24, 32), (20, 128, 32, 128),
+                                            (2, 320, 128, 16), (2, 400, 72, 64)])
 def test_absorbed_attention(form, dtype, H, R, DR, page):
     """Decoded tokens and short portions beside each other; contexts around page, block and split borders; one
     sequence's keys poisoned beyond its context; a key that stands out at a border."""
