@@ -674,7 +674,7 @@ def run_prefill_attention(args, shape):
 def hybrid_shapes():
     """(hybrid of 6 state-space + 2 latent layers, 8 latent layers, the closest other model: MLA + dense FFN) at equal
     width, heads, head dims and parameters per feed-forward."""
-    from vexact_b200.hybrid import HybridLayer, HybridShape, LatentSpec, SSMSpec
+    from vexact_b200.hybrid import DenseSpec, HybridLayer, HybridShape, LatentSpec, SSMSpec
     from vexact_b200.inferencer import MLAShape, ModelShape
 
     W, V, FF = 2048, 32768, 8192
@@ -682,7 +682,7 @@ def hybrid_shapes():
     lat = LatentSpec(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot_base=50000.0, rot_dims=64)
 
     def make(name, kinds):
-        return HybridShape(name, tuple(HybridLayer(m, FF, i) for i, m in enumerate(kinds)), W, V, 4, 0.3, 1e-5)
+        return HybridShape(name, tuple(HybridLayer(m, DenseSpec(FF), i) for i, m in enumerate(kinds)), W, V, 4, 0.3, 1e-5)
 
     return (make("hybrid-6ssm-2latent", [ssm, ssm, lat, ssm, ssm, ssm, lat, ssm]),
             make("hybrid-8latent", [lat] * 8),
@@ -782,7 +782,7 @@ def hybrid_model_case(args, shape, kind, S, new, total, page, device):
             step.seq_lens = None
 
         def run():
-            for k in ("_latent_plan", "_tc_plans"):      # what belongs to one step is made in every step
+            for k in ("_latent_plans", "_long_plan", "_tc_plans"):      # what belongs to one step is made in every step
                 step.__dict__.pop(k, None)
             return runner.logits(runner.forward(step, rows))
 
@@ -840,7 +840,7 @@ def hybrid_kernels(args, page, device):
     hbm, tc = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
     BF = torch.bfloat16
     hyb, _, mla = hybrid_shapes()
-    two = HybridShape("pair", (hyb.layers[0], hyb.layers[2].__class__(hyb.layers[2].mixer, 8192, 1)), hyb.width, hyb.vocab,
+    two = HybridShape("pair", (hyb.layers[0], hyb.layers[2].__class__(hyb.layers[2].mixer, hyb.layers[2].ff, 1)), hyb.width, hyb.vocab,
                       hyb.streams, hyb.residual_mult, hyb.eps)
     w = HybridWeights.random_init(two, device=device)
     sw, lw, mw, hc = w.layers[0].mixer, w.layers[1].mixer, w.layers[0].mlp, w.layers[0].hc
@@ -881,7 +881,7 @@ def hybrid_kernels(args, page, device):
         S = st.state_slots.numel()
         proj = [rn(T, sw.w_in.shape[0]) for _ in range(k)]
         conv = [torch.zeros(S, sw.taps - 1, sw.channels, device=device, dtype=BF) for _ in range(k)]
-        ms = graph_ms([lambda p=p, c=c: ssm.ssm_conv(sw, p, c, st) for p, c in zip(proj, conv)])
+        ms = graph_ms([lambda p=p, c=c: ssm.short_conv(sw, p, c, st) for p, c in zip(proj, conv)])
         state_b = 4 * S * (sw.taps - 1) * sw.channels
         yield line(f"ssm_conv T={T}", ms, T * (sw.channels * 4 + sw.heads * 6) + state_b)
         act = [(rn(T, sw.channels), torch.rand(T, sw.heads, device=device) * 0.1,
@@ -904,7 +904,8 @@ def hybrid_kernels(args, page, device):
         proj = [rn(T, lw.w_in.shape[0]) for _ in range(k)]
         cache = torch.zeros(blocks, page, lw.row_width, device=device, dtype=BF)
         qlat = [torch.empty(T, 16, lw.row_width, device=device, dtype=BF) for _ in range(k)] if T == 64 else [None] * k
-        ms = graph_ms([lambda p=p, q=q: la.latent_prep(lw, p, cache, st, 1e-5, q) for p, q in zip(proj, qlat)])
+        ms = graph_ms([lambda p=p, q=q: la.latent_prep(lw, cache, st, 1e-5, q=p[:, :lw.q_cols], kv=p[:, lw.q_cols:lw.q_cols + lw.row_width],
+                                               q_lat=q) for p, q in zip(proj, qlat)])
         yield line(f"latent_prep T={T}", ms, T * (lw.row_width * 4 + 16 * 64 * (4 if T > 64 else 6)))
         lib, inv = _lib.load(), lw.inv_freq
         sets = [(rn(T, 16 * 192), rn(T, 16 * 256), rn(T, 576)) for _ in range(k)]
@@ -937,20 +938,20 @@ def hybrid_kernels(args, page, device):
         st, blocks = hybrid_step([(new, total)] * S, page, device)
         T = S * new
         q, gate, cache = rn(T, 16, 192), rn(T, 16, 128), rn(blocks, page, lw.row_width)
-        heads, plan = torch.empty(T, 16, 128, device=device, dtype=BF), la._split_plan(st, device)[1]
+        heads, plan = torch.empty(T, 16, 128, device=device, dtype=BF), la._split_plan(st, None, device)[1]
         pairs = S * sum(range(total - new + 1, total + 1))
         flops = 2.0 * pairs * 16 * 320
         ms = graph_ms([lambda: la.latent_expanded(lw, q, gate, cache, heads, st, plan)])
         yield line(f"latent gather + up-projection + expanded attention {S}x{new}/{total}", ms, None,
                    flops + 2.0 * S * total * lw.w_kv.numel())
         lat, kv = rn(S * total, lw.row_width), rn(S * total, lw.w_kv.shape[0])
-        ids, starts, most, _ = plan
+        ids, starts, bases, most, _ = plan
 
         def attn():
             _lib.check(_lib.load().b200_latent_attn_expanded(
                 q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), lat.data_ptr(), lat.stride(0), lw.R, gate.data_ptr(),
                 gate.stride(0), heads.data_ptr(), heads.stride(0), st.query_start_loc.data_ptr(), st.context_lens.data_ptr(),
-                ids.data_ptr(), starts.data_ptr(), ids.numel(), most, 16, 128, 64, 128, float(lw.scale),
+                ids.data_ptr(), starts.data_ptr(), bases.data_ptr(), ids.numel(), most, 0, 16, 128, 64, 128, float(lw.scale),
                 _lib.current_stream()), "b200_latent_attn_expanded")
 
         yield line(f"latent_expand {S}x{new}/{total}", graph_ms([attn]), None, flops)

@@ -380,7 +380,7 @@ int b200_moe_unpermute_add_rmsnorm(const void* y, const void* scatter_index, con
                                    const void* residual, const void* weight, void* sum_out, void* out,
                                    long long T, int topk, int H, float eps, int mode, void* stream);
 
-/* ---- Operators of the hybrid decoder family (state-space + latent-attention layers, hyper-connections).  No
+/* ---- Operators of the hybrid decoder families.  No
  *      counterpart in the reference.  dtype: 0 = bf16, 1 = fp32 ("the model dtype"); *_f32 arguments are always fp32.
  *      Sequences: query_start_loc [S + 1], context_lens [S] (tokens after the step), state_slots [S] (-1 = none), i32. */
 
@@ -424,26 +424,29 @@ int b200_ssm_scan(const void* act, long long act_row_stride, const void* dt_f32,
                   const void* D_f32, void* state_f32, void* y, const void* query_start_loc, const void* context_lens,
                   const void* state_slots, int num_seqs, int num_slots, int heads, int groups, int N, int P,
                   int min_len, int max_len, int dtype, void* stream);
-/* out = rms_norm(y * silu(z)) * w in `parts` equal parts of the heads * p_true true columns; heads are P wide. */
-int b200_ssm_gate_norm(const void* y, long long y_row_stride, const void* z, long long z_row_stride, const void* w_f32,
-                       void* out, long long out_row_stride, long long T, int heads, int P, int p_true, int parts,
-                       float eps, int dtype, void* stream);
+/* out = rms_norm(y * silu(z)) * w in `parts` equal parts of the heads * p_true true columns; heads are P wide.
+ * norm_first: rms_norm(y) * w * silu(z) instead. */
+int b200_ssm_gate_norm(const void* y, long long y_row_stride, const void* z, long long z_row_stride, const void*
+                       w_f32, void* out, long long out_row_stride, long long T, int heads, int P, int p_true, int
+                       parts, float eps, int norm_first, int dtype, void* stream);
 
-/* Latent attention, before the attention call.  proj rows: [q: heads * (DN + DR) | c: R | k_rot: DR | ...].  Stores
- * rms_norm(c) * c_norm and the rotated k_rot as cache row slot_mapping[t] ([num_slots, R + DR]), rotates the queries in
- * place (interleaved pairs, the first rot_dims of the DR columns, angle position * inv_freq) and copies their rotated
- * part into columns R .. of q_lat [T, heads, R + DR] (NULL = not wanted).  DN, DR, R multiples of 8; r_true: columns of
- * c that are not padding. */
-int b200_latent_prep(void* proj, long long proj_row_stride, const void* positions_i64, const void* slot_mapping_i32,
-                     const void* inv_freq_f32, const void* c_norm_f32, void* cache, void* q_lat, long long T, int heads,
-                     int DN, int DR, int R, int r_true, int rot_dims, float eps, long long num_slots, int dtype,
-                     void* stream);
+/* Latent attention, between the projections and the attention call; every part may be NULL.  kv rows [c: R | k_rot: DR]:
+ * stores rms_norm(c) * c_norm and the rotated k_rot as cache row slot_mapping[t] ([num_slots, R + DR]).  q_latent rows
+ * [QL]: rms_norm(.) * q_norm in place (the latent queries come from).  q rows [heads * (DN + DR)]: rotates the first
+ * rot_dims of every head's DR columns in place (pairs (2i, 2i + 1), or with rot_half (i, i + rot_dims / 2); angle position *
+ * inv_freq) and copies the DR columns into columns R .. of q_lat [T, heads, R + DR].  DN, DR, R, QL multiples of 8; r_true /
+ * ql_true: columns that are not padding. */
+int b200_latent_prep(void* q, long long q_row_stride, const void* kv, long long kv_row_stride, void* q_latent,
+                     long long q_latent_row_stride, const void* q_norm_f32, int QL, int ql_true, const void* positions_i64,
+                     const void* slot_mapping_i32, const void* inv_freq_f32, const void* c_norm_f32, void* cache,
+                     void* q_lat, long long T, int heads, int DN, int DR, int R, int r_true, int rot_dims, int
+                     rot_half, float eps, long long num_slots, int dtype, void* stream);
 /* Absorbed causal attention on CUDA cores: out[t, h] = sum_j softmax(scale * q_lat[t, h] . row_j) row_j[:R] over the
- * cache rows of the sequence's positions 0 .. own.  Only sequences with min_len .. max_len tokens in this step. */
-int b200_latent_attn_simt(const void* q_lat, const void* cache, void* out, const void* query_start_loc,
-                          const void* context_lens, const void* page_table, long long page_table_stride, int max_pages,
-                          int page_size, int num_blocks, int num_seqs, int min_len, int max_len, long long T, int heads,
-                          int R, int DR, float scale, int dtype, void* stream);
+ * cache rows of the sequence's positions 0 .. own (window > 0: own - window + 1 .. own).  Only sequences with min_len .. max_len tokens in this step. */
+int b200_latent_attn_simt(const void* q_lat, const void* cache, void* out, const void* query_start_loc, const void*
+                          context_lens, const void* page_table, long long page_table_stride, int max_pages, int
+                          page_size, int num_blocks, int num_seqs, int min_len, int max_len, int window, long long T,
+                          int heads, int R, int DR, float scale, int dtype, void* stream);
 /* The recurrence of b200_ssm_scan in chunks of 64 tokens on tensor cores (bf16), for the sequences that bring at least
  * min_len tokens.  P and N multiples of 8, N <= 256.  slice: state columns per CTA, 16 or 32 (speed only). */
 int b200_ssm_chunk_scan(const void* act, long long act_row_stride, const void* dt_f32, const void* A_log_f32,
@@ -451,31 +454,103 @@ int b200_ssm_chunk_scan(const void* act, long long act_row_stride, const void* d
                         const void* context_lens, const void* state_slots, int num_seqs, int num_slots, int heads,
                         int groups, int N, int P, int min_len, int slice, void* stream);
 /* b200_latent_attn_simt on tcgen05 tensor cores (bf16).  b200_latent_plan lists the work of a step once for all layers
- * with `heads` heads: items [max_items][8], item_count [1], first_item [num_seqs], i32; at most max_items =
+ * with `heads` heads and one window (0: none): items [max_items][8], item_count [1], first_item [num_seqs], i32; at most max_items =
  * sum over sequences of ceil(new tokens * heads / 16) * ceil(context / 512).  R <= 512, DR <= 128, multiples of 8;
  * page_size a power of two of at least 8 or a multiple of 128.  part_o [max_items, 16, R], part_ml [max_items, 16, 2]
- * fp32 scratch, NULL when no context exceeds 512 tokens. */
+ * fp32 scratch, NULL when no sequence has keys in several splits of 512. */
 int b200_latent_plan(const void* query_start_loc, const void* context_lens, int num_seqs, int min_len, int max_len,
-                     int heads, int max_items, void* items, void* item_count, void* first_item, void* stream);
-int b200_latent_attn_tc(const void* q_lat, const void* cache, void* out, const void* query_start_loc,
-                        const void* context_lens, const void* page_table, long long page_table_stride, int max_pages,
-                        int page_size, int num_blocks, int num_seqs, int min_len, int max_len, long long T, int heads,
-                        int R, int DR, float scale, const void* items, const void* item_count, const void* first_item,
-                        int max_items, void* part_o, void* part_ml, void* stream);
+                     int window, int heads, int max_items, void* items, void* item_count, void* first_item, void*
+                     stream);
+int b200_latent_attn_tc(const void* q_lat, const void* cache, void* out, const void* query_start_loc, const void*
+                        context_lens, const void* page_table, long long page_table_stride, int max_pages, int
+                        page_size, int num_blocks, int num_seqs, int min_len, int max_len, int window, long long T,
+                        int heads, int R, int DR, float scale, const void* items, const void* item_count, const void*
+                        first_item, int max_items, void* part_o, void* part_ml, void* stream);
 /* Causal attention of n sequences over keys and values projected up from their gathered latents (bf16):
  * kv rows [keys: heads * DN | values: heads * DV], the shared rotated key part at column rot_off of the lat rows, rows
  * key_start[i] .. key_start[i + 1] belonging to sequence seq_ids[i]; q rows hold DN + DR columns per head.
- * out = sigmoid(gate) * attention, [T, heads * DV].  DN, DR, DV multiples of 8, DN + DR and DV <= 256. */
-int b200_latent_attn_expanded(const void* q, long long q_row_stride, const void* kv, long long kv_row_stride,
-                              const void* lat, long long lat_row_stride, int rot_off, const void* gate,
-                              long long gate_row_stride, void* out, long long out_row_stride,
-                              const void* query_start_loc, const void* context_lens, const void* seq_ids_i32,
-                              const void* key_start_i32, int n, int max_len, int heads, int DN, int DR, int DV,
-                              float scale, void* stream);
-/* dst row r = cache row of key r - key_start[i] of sequence seq_ids[i], key_start[i] <= r < key_start[i + 1]. */
-int b200_latent_gather(const void* cache, void* dst, const void* seq_ids_i32, const void* key_start_i32, int n,
-                       long long rows, int row_bytes, const void* page_table, long long page_table_stride,
-                       int max_pages, int page_size, int num_blocks, int num_seqs, void* stream);
+ * key_base[i] the position of the first of them.  out = sigmoid(gate) * attention (gate NULL: 1), [T, heads * DV].  DN, DR, DV multiples of 8, DN + DR and DV <= 256. */
+int b200_latent_attn_expanded(const void* q, long long q_row_stride, const void* kv, long long kv_row_stride, const
+                              void* lat, long long lat_row_stride, int rot_off, const void* gate, long long
+                              gate_row_stride, void* out, long long out_row_stride, const void* query_start_loc, const
+                              void* context_lens, const void* seq_ids_i32, const void* key_start_i32, const void*
+                              key_base_i32, int n, int max_len, int window, int heads, int DN, int DR, int DV, float
+                              scale, void* stream);
+/* dst row r = cache row of key key_base[i] + r - key_start[i] of sequence seq_ids[i], key_start[i] <= r < key_start[i + 1]. */
+int b200_latent_gather(const void* cache, void* dst, const void* seq_ids_i32, const void* key_start_i32, const void*
+                       key_base_i32, int n, long long rows, int row_bytes, const void* page_table, long long
+                       page_table_stride, int max_pages, int page_size, int num_blocks, int num_seqs, void* stream);
+
+/* Grouped-query attention over paged per-head keys and values [blocks, page, kv_heads, DK | DV], no positions in the
+ * scores, inside a window (0: none), fp32 weights.  _decode: bf16, tensor cores, sequences with min_len .. max_len new
+ * tokens (most_new: the most any brings); DK, DV <= 256, page_size a multiple of 8 that divides 32 or is a multiple of it.
+ * _prefill: bf16, tensor cores, the n sequences named.  _simt: any dims, both dtypes.  q and out rows hold the heads. */
+int b200_window_attn_decode(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void*
+                            out, long long out_row_stride, const void* query_start_loc, const void* context_lens,
+                            const void* page_table, long long page_table_stride, int max_pages, int page_size, int
+                            num_blocks, int num_seqs, int min_len, int max_len, int most_new, int window, int heads,
+                            int kv_heads, int DK, int DV, float scale, void* stream);
+int b200_window_attn_prefill(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void*
+                             out, long long out_row_stride, const void* query_start_loc, const void* context_lens,
+                             const void* page_table, long long page_table_stride, int max_pages, int page_size, int
+                             num_blocks, int num_seqs, const void* seq_ids_i32, int n, int max_len, int window, int
+                             heads, int kv_heads, int DK, int DV, float scale, void* stream);
+int b200_window_attn_simt(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void* out,
+                          const void* query_start_loc, const void* context_lens, const void* page_table, long long
+                          page_table_stride, int max_pages, int page_size, int num_blocks, int num_seqs, int min_len,
+                          int max_len, int window, long long T, int heads, int kv_heads, int DK, int DV, float scale,
+                          int dtype, void* stream);
+
+/* Gated delta rule over act rows [q: groups * N | k: groups * N | v: heads * P] (convolved, not yet unit vectors):
+ *   S = g S; u = beta (v - S^T k); S += k u^T; o = S^T q,   g = exp(-exp(A_log) dt), beta = sigmoid(b), k and q divided by
+ * their lengths (q times scale).  state [slots, heads, N, P] fp32, o [T, heads * P].  _scan: token by token, sequences with
+ * min_len .. max_len new tokens, N <= 512.  _chunk_scan: bf16, chunks of 64 tokens on tensor cores, sequences with at least
+ * min_len new tokens (max_new: the most any brings), N <= 256; scratch for T / 64 + num_seqs chunks, mats 32 KB and vecs
+ * 768 bytes per chunk and head; slice: state columns per CTA, 16 or 32 (speed only). */
+int b200_delta_scan(const void* act, long long act_row_stride, const void* dt_f32, const void* b, long long
+                    b_row_stride, const void* A_log_f32, void* state_f32, void* o, const void* query_start_loc, const
+                    void* context_lens, const void* state_slots, int num_seqs, int num_slots, int heads, int groups,
+                    int N, int P, float scale, int min_len, int max_len, int dtype, void* stream);
+int b200_delta_chunk_scan(const void* act, long long act_row_stride, const void* dt_f32, const void* b, long long
+                          b_row_stride, const void* A_log_f32, void* state_f32, void* o, void* mats, void* vecs_f32,
+                          const void* query_start_loc, const void* context_lens, const void* state_slots, int
+                          num_seqs, int num_slots, int heads, int groups, int N, int P, float scale, int min_len, int
+                          max_new, int slice, void* stream);
+
+/* One boundary of a residual with a norm on both sides of every sublayer (x [num_tokens, W] fp32, in place):
+ *   x <- x + rms_norm(y) * post (+ add);  xn = rms_norm(x) * norm_w (NULL = no xn), columns W .. xn_cols zero.
+ * y: rows, or with scatter_index the sum of the token's topk rows of y [y_rows]; extra (or NULL) is added to it.  ids given
+ * instead of y: the model starts, x = rms_norm(embed[ids]) * post (+ add).  rows_i32 (with write_back = 0): only these. */
+int b200_residual_step(void* x_f32, const void* y, long long y_row_stride, long long y_rows, const void*
+                       scatter_index_i32, int topk, const void* extra, long long extra_row_stride, const void* embed,
+                       const void* ids_i64, long long vocab, const void* rows_i32, long long num_tokens, long long
+                       num_rows, int W, const void* post_f32, const void* add_f32, const void* norm_w_f32, float eps,
+                       void* xn, long long xn_row_stride, int xn_cols, int write_back, int dtype, void* stream);
+
+/* Gated feed-forwards: act(s g) * (s u) * o with fp32 row factors s = scale_in, o = scale_out (NULL: 1); act 1 silu, 2 the
+ * tanh form of gelu.  _gemm_glu: one product, w [2 * n_out, K] gate rows first; _moe_grouped_gemm_glu: expert-sorted rows,
+ * w [groups, 2 * n_out, K]; _glu: over rows [gate: F | up: F] of a plain product, both dtypes. */
+int b200_gemm_glu(const void* x, const void* w, const void* scale_out_f32, void* out, long long T, int n_out, int K,
+                  long long x_row_stride, long long out_row_stride, int act, void* stream);
+int b200_moe_grouped_gemm_glu(const void* x, const void* w, const void* scale_in_f32, const void* scale_out_f32, void*
+                              out, const void* tile_table, const void* tile_count, long long x_rows, int num_groups,
+                              int n_out, int K, long long out_row_stride, int max_tiles, int tile_rows_max, int act,
+                              void* stream);
+int b200_glu(const void* gu, long long gu_row_stride, const void* scale_in_f32, const void* scale_out_f32, void* out,
+             long long rows, int F, int act, int dtype, void* stream);
+/* Expert-sorted rows in true fp32: out[r] = w[group] x[r]; tile table entries of at most 64 rows. */
+int b200_moe_grouped_gemm_f32(const void* x, const void* w, void* out, const void* tile_table, const void* tile_count,
+                              long long x_rows, int num_groups, int n_out, int K, int max_tiles, void* stream);
+/* b200_moe_route_plan_softmax_topk / b200_moe_scatter_ranked for sigmoid scores and fp32 weights: weights = the chosen
+ * scores (renorm: over their sum); gate_f32 [T] or NULL = sigmoid of the logit in column E; rows of row_bytes bytes. */
+int b200_moe_route_plan_sigmoid_topk(const void* logits_f32, long long row_stride, void* weights_f32, void* gate_f32,
+                                     void* experts_i64, void* rank_i32, void* counters_i32, void* cu_seqlens, void*
+                                     tile_table, void* tile_count, long long T, int E, int topk, int renorm, int
+                                     tile_rows, int max_tiles, void* stream);
+int b200_moe_scatter_ranked_f32(const void* x, long long x_row_bytes, const void* experts_i64, const void*
+                                weights_f32, const void* rank_i32, const void* cu_seqlens, void* scatter_index, void*
+                                x_perm, void* row_scale_f32, long long T, int topk, int E, int row_bytes, void*
+                                stream);
 
 #ifdef __cplusplus
 }

@@ -140,7 +140,7 @@ def _scan_reference(w, act, dt):
 @pytest.mark.parametrize("taps", [1, 2, 4, 6])
 def test_conv_in_portions_of_unequal_sequences(dtype, taps):
     """Portions down to one and two tokens, both forms, sequences that come and go beside each other."""
-    from vexact_b200.ssm import ssm_conv
+    from vexact_b200.ssm import short_conv
 
     w = _ssm_weights(3, 8, 16, 1, taps, seed=taps)
     lengths, slots = [70, 45, 23], [5, 0, 2]
@@ -152,7 +152,7 @@ def test_conv_in_portions_of_unequal_sequences(dtype, taps):
         live = [i for i in range(3) if cut[i]]
         rows = torch.cat([proj[i][done[i]:done[i] + cut[i]] for i in live])
         st = hu.step([(cut[i], done[i] + cut[i]) for i in live], slots=[slots[i] for i in live])
-        act, dt = ssm_conv(w, rows, state, st)
+        act, dt = short_conv(w, rows, state, st)
         at = 0
         for i in live:
             _close(act[at:at + cut[i]], ref[i][0][done[i]:done[i] + cut[i]], dtype)
@@ -287,7 +287,7 @@ def test_latent_prep_norms_rotates_and_stores(dtype, rot_dims, r_true):
     q_lat = torch.zeros(T, H, R + DR, dtype=dtype, device=DEV)
     st.slot_mapping[6] = -1                        # a padded token stores nothing
     work = proj.cuda()
-    latent_prep(w, work, cache, st, eps, q_lat)
+    latent_prep(w, cache, st, eps, q=work[:, :H * dq], kv=work[:, H * dq:H * dq + R + DR], q_lat=q_lat)
     pos = st.positions.cpu()
     p = proj.double()
     q = p[:, :H * dq].view(T, H, dq)
@@ -400,7 +400,7 @@ def test_expanded_attention(H, DN, DR, R, V, page, longest):
         r = _rand(total, R + DR, seed=50 + i, dtype=BF)
         rows.append(r)
         cache[st.rows(i)] = r
-    runs, longs = la._split_plan(st, DEV)
+    runs, longs = la._split_plan(st, w.window, DEV)
     assert runs == [[17, 18]] and longs[0].tolist() == [0, 2, 3, 4, 5]
     heads = torch.full((T, H, V), 9.0, dtype=BF, device=DEV)
     la.latent_expanded(w, q.cuda()[:, :H * dq].view(T, H, dq), gate.cuda()[:, 8:].unflatten(1, (H, V)),

@@ -74,6 +74,11 @@ struct GemmParams {
   int out_f32;
   const __nv_bfloat16* bias;       // [n_w] or null (plain mode)
   const __nv_bfloat16* row_scale;  // [rows] or null (SwiGLU mode: routing weight of each permuted row)
+  // SwiGLU mode with GLU_SILU / GLU_GELU_TANH: out = act(s g) * (s u) * o in fp32 with one rounding, s = scale_in[row],
+  // o = scale_out[row] (null: 1).  GLU_REFERENCE: the rounding points of the fused MoE and row_scale.
+  int glu;
+  const float* scale_in;
+  const float* scale_out;
   float4* head_part;               // head mode: [t_rows, w_tiles] per-tile {max, sum exp(x - max), argmax, 0}
   // Batched plain mode: batch_extra + 1 independent products of one shape.  Product g reads the slice at index g
   // of a 3-D activation map and weight rows from g * w_rows_per_group, and writes out + g * out_batch_stride.
@@ -98,6 +103,11 @@ constexpr int GEMM_ACT_NONE = 0;
 constexpr int GEMM_ACT_GELU_TANH = 1;     // z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3): the tanh form of gelu
 constexpr int GEMM_ACT_SIGMOID_GATE = 2;  // z * sigmoid(gate)
 
+// Activations of the gated forms (SwiGLU mode of the GEMM and glu_kernel).
+constexpr int GLU_REFERENCE = 0;
+constexpr int GLU_SILU = 1;
+constexpr int GLU_GELU_TANH = 2;
+
 __device__ __forceinline__ float gelu_tanh_fast(float z) {
   const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
   return __fdividef(z, 1.f + __expf(fminf(-2.f * u, 80.f)));
@@ -105,6 +115,13 @@ __device__ __forceinline__ float gelu_tanh_fast(float z) {
 __device__ __forceinline__ float gelu_tanh_exact(float z) {
   const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
   return 0.5f * z * (1.f + tanhf(u));
+}
+
+// act(g) * u for an output stored in T.
+template <typename T>
+__device__ __forceinline__ float glu_value(int act, float g, float u) {
+  if (sizeof(T) == 2) return (act == GLU_SILU ? __fdividef(g, 1.f + __expf(-g)) : gelu_tanh_fast(g)) * u;
+  return (act == GLU_SILU ? g / (1.f + expf(-g)) : gelu_tanh_exact(g)) * u;
 }
 
 // 2^x on the special-function unit (relative error below 2^-22; results below the normal range flush to zero).
@@ -570,7 +587,19 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
             uint32_t r[16];
             ptx::tmem_ld16(taddr + c0, r);
             ptx::tmem_ld_wait();
-            if (fvalid) {
+            if (fvalid && p.glu != GLU_REFERENCE) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) {
+                const int c = c0 + j;
+                if (c < t.n) {
+                  const float si = p.scale_in ? p.scale_in[t.row0 + c] : 1.f;
+                  const float so = p.scale_out ? p.scale_out[t.row0 + c] : 1.f;
+                  const float u = bf2f(exch[fi * exch_pitch + c]);
+                  reinterpret_cast<__nv_bfloat16*>(p.out)[(long long)(t.row0 + c) * p.ldo + f] =
+                      f2bf(so * glu_value<__nv_bfloat16>(p.glu, si * __uint_as_float(r[j]), si * u));
+                }
+              }
+            } else if (fvalid) {
 #pragma unroll
               for (int j = 0; j < 16; ++j) {
                 const int c = c0 + j;
@@ -731,18 +760,27 @@ gemm_f32_kernel(const TIn* __restrict__ x, const TIn* __restrict__ w, const floa
 namespace b200 {
 // True-fp32 GEMM for models that run in fp32: 64 x 64 output tile per CTA, 4 x 4 outputs per thread, K walked in
 // ascending steps of 16 through shared memory, plain fp32 FMA (no tensor cores, no reduced-precision mode).
-// blockIdx.z picks one product of the batch.
+// blockIdx.z picks one product of the batch.  With a tile table (at most 64 rows of one group per entry, as the MoE plans
+// make it) blockIdx.x is an entry and the group picks the weights.
 __global__ void __launch_bounds__(256)
 gemm_f32_tiled_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias,
                       const float* __restrict__ gate, float* __restrict__ out, long long T, int N, int K,
                       long long x_row, long long x_batch, long long w_row, long long w_batch, long long out_row,
-                      long long out_batch, long long gate_row, long long gate_batch, int act) {
+                      long long out_batch, long long gate_row, long long gate_batch, int act,
+                      const int4* __restrict__ tile_table = nullptr, const int* __restrict__ tile_count = nullptr) {
   pdl_trigger();
   pdl_wait();
   __shared__ float sx[16][68], sw[16][68];
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-  const long long t0 = (long long)blockIdx.x * 64;
+  long long t0 = (long long)blockIdx.x * 64;
   const int n0 = blockIdx.y * 64;
+  if (tile_table) {
+    if ((int)blockIdx.x >= *tile_count) return;
+    const int4 e = tile_table[blockIdx.x];
+    t0 = e.y;
+    T = min(T, (long long)e.y + min(e.z, 64));
+    w += (long long)e.x * w_batch;
+  }
   x += (long long)blockIdx.z * x_batch;
   w += (long long)blockIdx.z * w_batch;
   float acc[4][4] = {};
@@ -801,7 +839,7 @@ extern "C" int b200_gemm_f32_ex(const void* x, const void* w, const void* bias, 
   launch_k(gemm_f32_tiled_kernel, dim3((unsigned)((T + 63) / 64), (unsigned)((N + 63) / 64), (unsigned)batch), dim3(256),
            0, (cudaStream_t)stream, (const float*)x, (const float*)w, (const float*)bias, (const float*)gate,
            (float*)out, T, N, K, x_row_stride, x_batch_stride, w_row_stride, w_batch_stride, out_row_stride,
-           out_batch_stride, gate_row_stride, gate_batch_stride, act);
+           out_batch_stride, gate_row_stride, gate_batch_stride, act, (const int4*)nullptr, (const int*)nullptr);
   return launch_status();
 }
 
@@ -1067,7 +1105,8 @@ namespace b200 {
 inline int moe_grouped_gemm_impl(const void* x, long long x_rows, long long x_row_stride, const void* gather_index,
                                  const void* w, const void* row_scale, void* out, const void* tile_table,
                                  const void* tile_count, int num_groups, int n_out, int K, long long out_row_stride,
-                                 int max_tiles, int tile_rows_max, int mode, void* stream) {
+                                 int max_tiles, int tile_rows_max, int mode, void* stream, int glu = GLU_REFERENCE,
+                                 const void* scale_in = nullptr, const void* scale_out = nullptr) {
   if (!x || !w || !out || !tile_table || !tile_count || x_rows < 0 || num_groups <= 0 || n_out <= 0 || K <= 0 ||
       max_tiles < 0 || (mode != 0 && mode != 1))
     return B200_ERR_ARG;
@@ -1095,6 +1134,9 @@ inline int moe_grouped_gemm_impl(const void* x, long long x_rows, long long x_ro
   p.out_f32 = 0;
   p.bias = nullptr;
   p.row_scale = (const __nv_bfloat16*)row_scale;
+  p.glu = glu;
+  p.scale_in = (const float*)scale_in;
+  p.scale_out = (const float*)scale_out;
   p.w_policy = ptx::kEvictFirst;
   CUtensorMap tw, tx;
   int rc = make_tmap_2d(&tw, w, (uint64_t)num_groups * p.w_rows_per_group, (uint64_t)K, (uint64_t)K,
@@ -1129,6 +1171,127 @@ extern "C" int b200_moe_grouped_gemm_gather(const void* x, long long T, long lon
   if (!gather_index) return B200_ERR_ARG;
   return b200::moe_grouped_gemm_impl(x, T, x_row_stride, gather_index, w, row_scale, out, tile_table, tile_count,
                                      num_groups, n_out, K, out_row_stride, max_tiles, tile_rows_max, mode, stream);
+}
+
+// The grouped GEMM with a gated activation: out[r, i] = act(s g) * (s u) * o with g = x[r] . w[group, i],
+// u = x[r] . w[group, I + i], s = scale_in[r], o = scale_out[r] (NULL: 1); act: 1 silu, 2 the tanh form of gelu.
+// w [groups, 2 * n_out, K].
+extern "C" int b200_moe_grouped_gemm_glu(const void* x, const void* w, const void* scale_in_f32, const void* scale_out_f32,
+                                         void* out, const void* tile_table, const void* tile_count, long long x_rows,
+                                         int num_groups, int n_out, int K, long long out_row_stride, int max_tiles,
+                                         int tile_rows_max, int act, void* stream) {
+  if (act != b200::GLU_SILU && act != b200::GLU_GELU_TANH) return B200_ERR_ARG;
+  return b200::moe_grouped_gemm_impl(x, x_rows, K, nullptr, w, nullptr, out, tile_table, tile_count, num_groups, n_out, K,
+                                     out_row_stride, max_tiles, tile_rows_max, 1, stream, act, scale_in_f32, scale_out_f32);
+}
+
+// One product of the same form over T rows as they lie (no tile table): w [2 * n_out, K].
+extern "C" int b200_gemm_glu(const void* x, const void* w, const void* scale_out_f32, void* out, long long T, int n_out,
+                             int K, long long x_row_stride, long long out_row_stride, int act, void* stream) {
+  using namespace b200;
+  if (!x || !w || !out || T < 0 || n_out <= 0 || K <= 0 || (act != GLU_SILU && act != GLU_GELU_TANH)) return B200_ERR_ARG;
+  if (K % 8 != 0 || x_row_stride % 8 != 0 || T > 0x7fffffffLL) return B200_ERR_SHAPE;
+  if (T == 0) return B200_OK;
+  GemmParams p{};
+  p.n_w = n_out;
+  p.k = K;
+  p.w_tiles = (n_out + 63) / 64;
+  p.w_rows_per_group = 2 * n_out;
+  p.up_offset = n_out;
+  p.t_rows = (int)T;
+  p.rows_per_tile = T <= 64 ? round_up((int)T, 16) : 64;
+  p.dense_t_tiles = (int)((T + p.rows_per_tile - 1) / p.rows_per_tile);
+  p.xbox = p.rows_per_tile;
+  p.xrows_max = p.rows_per_tile;
+  p.out = out;
+  p.ldo = out_row_stride;
+  p.glu = act;
+  p.scale_out = (const float*)scale_out_f32;
+  p.w_policy = p.dense_t_tiles == 1 ? ptx::kEvictFirst : ptx::kEvictNormal;
+  CUtensorMap tw, tx;
+  int rc = make_tmap_2d(&tw, w, (uint64_t)2 * n_out, (uint64_t)K, (uint64_t)K, 64);
+  if (rc) return rc;
+  rc = make_tmap_2d(&tx, x, (uint64_t)T, (uint64_t)K, (uint64_t)x_row_stride, (uint32_t)p.xbox);
+  if (rc) return rc;
+  return gemm_launch<GEMM_SWIGLU>(tw, tx, p, (long long)p.w_tiles * p.dense_t_tiles, (cudaStream_t)stream);
+}
+
+// The grouped GEMM in true fp32: out[r, n] = x[r] . w[group, n]; tile table entries of at most 64 rows.
+extern "C" int b200_moe_grouped_gemm_f32(const void* x, const void* w, void* out, const void* tile_table,
+                                         const void* tile_count, long long x_rows, int num_groups, int n_out, int K,
+                                         int max_tiles, void* stream) {
+  using namespace b200;
+  if (!x || !w || !out || !tile_table || !tile_count || x_rows < 0 || num_groups <= 0 || n_out <= 0 || K <= 0 || max_tiles < 0)
+    return B200_ERR_ARG;
+  if (x_rows == 0 || max_tiles == 0) return B200_OK;
+  if ((n_out + 63) / 64 > 65535) return B200_ERR_SHAPE;
+  launch_k(gemm_f32_tiled_kernel, dim3((unsigned)max_tiles, (unsigned)((n_out + 63) / 64), 1u), dim3(256), 0,
+           (cudaStream_t)stream, (const float*)x, (const float*)w, (const float*)nullptr, (const float*)nullptr,
+           (float*)out, x_rows, n_out, K, (long long)K, 0LL, (long long)K, (long long)n_out * K, (long long)n_out, 0LL, 0LL,
+           0LL, GEMM_ACT_NONE, (const int4*)tile_table, (const int*)tile_count);
+  return launch_status();
+}
+
+namespace b200 {
+// out[r, i] = act(s g) * (s u) * o over rows [gate: F | up: F]: the gated activation after a plain GEMM.  Eight columns
+// per thread.
+template <typename T>
+__global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ gu, long long gu_stride,
+                                                  const float* __restrict__ scale_in, const float* __restrict__ scale_out,
+                                                  T* __restrict__ out, int F, int act) {
+  pdl_trigger();
+  pdl_wait();
+  const long long r = blockIdx.x;
+  const float si = scale_in ? scale_in[r] : 1.f, so = scale_out ? scale_out[r] : 1.f;
+  const T* g = gu + r * gu_stride;
+  for (int i = threadIdx.x * 8; i < F; i += 256 * 8) {
+    float a[8], b[8];
+    if constexpr (sizeof(T) == 2) {
+      const uint4 av = *reinterpret_cast<const uint4*>(g + i), bv = *reinterpret_cast<const uint4*>(g + F + i);
+      const uint32_t ap[4] = {av.x, av.y, av.z, av.w}, bp[4] = {bv.x, bv.y, bv.z, bv.w};
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        unpack_bf2(ap[k], a[2 * k], a[2 * k + 1]);
+        unpack_bf2(bp[k], b[2 * k], b[2 * k + 1]);
+      }
+    } else {
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        a[k] = g[i + k];
+        b[k] = g[F + i + k];
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < 8; ++k) a[k] = so * glu_value<T>(act, si * a[k], si * b[k]);
+    if constexpr (sizeof(T) == 2) {
+      *reinterpret_cast<uint4*>(out + r * F + i) =
+          make_uint4(pack_bf2(a[0], a[1]), pack_bf2(a[2], a[3]), pack_bf2(a[4], a[5]), pack_bf2(a[6], a[7]));
+    } else {
+#pragma unroll
+      for (int k = 0; k < 8; ++k) out[r * F + i + k] = a[k];
+    }
+  }
+}
+}  // namespace b200
+
+// gu rows [gate: F | up: F], gu_row_stride apart; out [rows, F] contiguous.  F a multiple of 8.
+extern "C" int b200_glu(const void* gu, long long gu_row_stride, const void* scale_in_f32, const void* scale_out_f32,
+                        void* out, long long rows, int F, int act, int dtype, void* stream) {
+  using namespace b200;
+  if (!gu || !out || rows < 0 || F <= 0 || gu_row_stride < 2 * F || (act != GLU_SILU && act != GLU_GELU_TANH) ||
+      (dtype != 0 && dtype != 1))
+    return B200_ERR_ARG;
+  if (F % 8 != 0 || gu_row_stride % 8 != 0 || rows > 0x7fffffffLL || (reinterpret_cast<uintptr_t>(gu) & 15) ||
+      (reinterpret_cast<uintptr_t>(out) & 15))
+    return B200_ERR_SHAPE;
+  if (rows == 0) return B200_OK;
+  if (dtype == 0)
+    launch_k(glu_kernel<__nv_bfloat16>, dim3((unsigned)rows), dim3(256), 0, (cudaStream_t)stream, (const __nv_bfloat16*)gu,
+             gu_row_stride, (const float*)scale_in_f32, (const float*)scale_out_f32, (__nv_bfloat16*)out, F, act);
+  else
+    launch_k(glu_kernel<float>, dim3((unsigned)rows), dim3(256), 0, (cudaStream_t)stream, (const float*)gu, gu_row_stride,
+             (const float*)scale_in_f32, (const float*)scale_out_f32, (float*)out, F, act);
+  return launch_status();
 }
 
 #ifdef B200_GEMM_TRACE

@@ -1,16 +1,18 @@
-// Expanded form of latent attention for long portions of prompts (bf16): the latents of a sequence's whole context have
-// been gathered from their pages and projected up to per-head keys and values, and this kernel runs ordinary causal
-// attention over them.
+// Causal attention of long portions of prompts over per-head keys and values (bf16), optionally inside a window.  Two
+// sources of keys:
 //
-//   kv rows   [keys: H * DN | values: H * DV]  (one row per key of the gathered sequences)
-//   lat rows  [c: R | k_rot: DR]               (the rotated key part shared by the heads is read from here)
-//   q         [T, q_stride]: per head DN unrotated, then DR rotated columns
-//   out[t, h] = sigmoid(gate[t, h]) * sum_j softmax(scale q.k_j) v_j
+//   expanded latents   the latents of a sequence's context (from the first key the window reaches) have been gathered from
+//                      their pages and projected up: packed kv rows [keys: G * DN | values: G * DV], and lat rows
+//                      [c: R | k_rot: DR] from which the rotated key part shared by the heads is read
+//   paged heads        k and v rows of a paged cache, [G * DN] and [G * DV] (DR = 0)
+//
+//   q         [T, q_stride]: per head DN unrotated, then DR rotated columns; head h uses key / value head h / group
+//   out[t, h] = sum_j softmax(scale q.k_j) v_j, times sigmoid(gate[t, h]) when there is a gate
 //
 // One CTA per (128 MT queries, head, sequence); warp w of 8 owns query rows 16 MT w .. 16 MT (w + 1) - 1 (MT = 2 for long
 // portions: every key and value fragment read from shared memory then serves two products); 64 keys per block, double
-// buffered with cp.async, 32 per softmax step.  Scores and weights stay fp32: a weight enters the value product as a bf16 pair hi + lo.
-// Query tiles are dealt from a sequence's last (longest) to its first.
+// buffered with cp.async, 32 per softmax step.  Scores and weights stay fp32: a weight enters the value product as a bf16
+// pair hi + lo.  Query tiles are dealt from a sequence's last (longest) to its first.
 #pragma once
 #include "attn_tc.cuh"     // fast_exp2
 #include "latent.cuh"
@@ -21,17 +23,18 @@ namespace b200 {
 constexpr int LEX_BN = 64, LEX_SUB = 32, LEX_THREADS = 256;
 
 struct LatentExpandParams {
-  const int* query_start_loc;
-  const int* context_lens;
-  const int* seq_ids;      // [n] gathered sequences
-  const int* key_start;    // [n + 1] first kv / lat row of each
+  LatentSeqs seqs;
+  const int* seq_ids;      // [n] sequences with long portions
+  const int* key_start;    // [n + 1] first packed row of each (packed sources)
+  const int* key_base;     // [n] position of that row's key (packed sources)
   const __nv_bfloat16* q;
-  const __nv_bfloat16* kv;
-  const __nv_bfloat16* lat;
-  const __nv_bfloat16* gate;
+  const __nv_bfloat16* k;      // rows k_stride apart, head g at column g * DN
+  const __nv_bfloat16* v;      // rows v_stride apart, head g at column g * DV
+  const __nv_bfloat16* rot;    // rows rot_stride apart: the shared rotated part (DR > 0)
+  const __nv_bfloat16* gate;   // or null
   __nv_bfloat16* out;
-  long long q_stride, kv_stride, lat_stride, gate_stride, out_stride;
-  int heads, DN, DR, DV, rot_off;   // rot_off: column of k_rot in a lat row
+  long long q_stride, k_stride, v_stride, rot_stride, gate_stride, out_stride;
+  int heads, group, DN, DR, DV;
   float scale_log2;
 };
 
@@ -43,26 +46,28 @@ struct LexLayout {
   static constexpr int BYTES = Q + 2 * (K + V);
 };
 
-template <int DK, int DV, int MT>
+template <int DK, int DV, int MT, bool PAGED>
 __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const LatentExpandParams p) {
   using L = LexLayout<DK, DV, MT>;
   constexpr int LEX_BM = L::BM, NS = LEX_SUB / 8;
   extern __shared__ __align__(16) uint8_t lex_smem[];
   pdl_trigger();
   pdl_wait();
-  const int i = blockIdx.z, h = blockIdx.y, seq = p.seq_ids[i];
-  const int t0 = p.query_start_loc[seq], len = p.query_start_loc[seq + 1] - t0;
+  const int i = blockIdx.z, h = blockIdx.y, kvh = h / p.group, seq = p.seq_ids[i];
+  const int t0 = p.seqs.query_start_loc[seq], len = p.seqs.query_start_loc[seq + 1] - t0;
   const int tiles = (len + LEX_BM - 1) / LEX_BM;
   if ((int)blockIdx.x >= tiles) return;
   const int row_base = (tiles - 1 - (int)blockIdx.x) * LEX_BM;
-  const int keys = p.key_start[i + 1] - p.key_start[i], past = keys - len;
-  const long long key0 = p.key_start[i];
+  const int keys = p.seqs.context_lens[seq], past = keys - len, window = p.seqs.window;
+  const int key_base = PAGED ? 0 : p.key_base[i];
+  const long long key0 = PAGED ? 0 : p.key_start[i] - key_base;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
   const uint32_t smem = ptx::smem_u32(lex_smem);
   const int dk16 = (p.DN + p.DR + 15) / 16;
   const int rows = min(LEX_BM, len - row_base);
   const int last_key = min(keys, past + row_base + rows);       // keys any row of the tile sees
-  const int blocks = (last_key + LEX_BN - 1) / LEX_BN;
+  const int first_key = window_first(window, past + row_base);
+  const int block0 = first_key / LEX_BN, blocks = (last_key + LEX_BN - 1) / LEX_BN;
 
   for (int e = tid; e < LEX_BM * (DK / 8); e += LEX_THREADS) {
     const int r = e / (DK / 8), v = e % (DK / 8);
@@ -76,23 +81,23 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
     const int base = b * LEX_BN;
     for (int e = tid; e < LEX_BN * (DK / 8); e += LEX_THREADS) {
       const int r = e / (DK / 8), col = (e % (DK / 8)) * 8;
-      const bool in = base + r < last_key && col < p.DN + p.DR;
-      const long long row = key0 + (in ? base + r : 0);
-      const __nv_bfloat16* src = col < p.DN || !in ? p.kv + row * p.kv_stride + (long long)h * p.DN + (in ? col : 0)
-                                                   : p.lat + row * p.lat_stride + p.rot_off + (col - p.DN);
+      const bool seen = base + r >= first_key && base + r < last_key;
+      const long long row = seen ? (PAGED ? latent_key_row(p.seqs, seq, base + r) : key0 + base + r) : -1;
+      const bool in = row >= 0 && col < p.DN + p.DR;
+      const __nv_bfloat16* src = p.k;
+      if (in) src = col < p.DN ? p.k + row * p.k_stride + (long long)kvh * p.DN + col : p.rot + row * p.rot_stride + (col - p.DN);
       cp_async16(k + (uint32_t)(r * L::LDK + col) * 2, src, in);
     }
     for (int e = tid; e < LEX_BN * (DV / 8); e += LEX_THREADS) {
       const int r = e / (DV / 8), col = (e % (DV / 8)) * 8;
-      const bool in = base + r < last_key && col < p.DV;
-      cp_async16(vt + (uint32_t)(r * L::LDV + col) * 2,
-                 p.kv + (key0 + (in ? base + r : 0)) * p.kv_stride + (long long)p.heads * p.DN + (long long)h * p.DV +
-                     (in ? col : 0),
-                 in);
+      const bool seen = base + r >= first_key && base + r < last_key;
+      const long long row = seen ? (PAGED ? latent_key_row(p.seqs, seq, base + r) : key0 + base + r) : -1;
+      const bool in = row >= 0 && col < p.DV;
+      cp_async16(vt + (uint32_t)(r * L::LDV + col) * 2, in ? p.v + row * p.v_stride + (long long)kvh * p.DV + col : p.v, in);
     }
     cp_async_commit();
   };
-  load(0);
+  load(block0);
 
   float o[MT][DV / 8][4];
 #pragma unroll
@@ -107,7 +112,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   }
   const int r0 = 16 * MT * warp;
   const int first_pos = past + row_base + r0;                    // position of the warp's first row
-  for (int b = 0; b < blocks; ++b) {
+  for (int b = block0; b < blocks; ++b) {
     if (b + 1 < blocks) {
       load(b + 1);
       cp_async_wait<1>();
@@ -120,6 +125,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
     for (int sub = 0; sub < LEX_BN / LEX_SUB; ++sub) {
       const int base = b * LEX_BN + sub * LEX_SUB;
       if (r0 >= rows || base > first_pos + 16 * MT - 1) break;   // no row of this warp sees these keys
+      if (window > 0 && base + LEX_SUB - 1 <= first_pos - window) continue;   // nor these, before every row's window
       float s[MT][NS][4];
 #pragma unroll
       for (int t = 0; t < MT; ++t)
@@ -140,7 +146,9 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
           }
         }
       }
-      const bool edge = base + LEX_SUB - 1 > first_pos;           // some (row, key) of these is masked
+      // some (row, key) of these is masked
+      const bool edge = base + LEX_SUB - 1 > first_pos || (window > 0 && base <= first_pos + 16 * MT - 1 - window);
+      const uint32_t reach = window > 0 ? (uint32_t)window : 0x80000000u;     // a row sees 0 <= its position - key < reach
 #pragma unroll
       for (int t = 0; t < MT; ++t) {
         const int pos0 = first_pos + 16 * t + g4;                 // position of row g4 of the tile (and + 8)
@@ -150,7 +158,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             float v = s[t][j][e] * p.scale_log2;
-            if (edge && base + 8 * j + 2 * t4 + (e & 1) > pos0 + 8 * (e >> 1)) v = -INFINITY;
+            if (edge && (uint32_t)(pos0 + 8 * (e >> 1) - (base + 8 * j + 2 * t4 + (e & 1))) >= reach) v = -INFINITY;
             s[t][j][e] = v;
             mb[e >> 1] = fmaxf(mb[e >> 1], v);
           }
@@ -225,56 +233,118 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
       for (int j = 0; j < DV / 8; ++j) {
         const int c = 8 * j + 2 * t4;
         if (c < p.DV) {
-          float ga, gb;
-          unpack_bf2(*reinterpret_cast<const uint32_t*>(p.gate + t * p.gate_stride + (long long)h * p.DV + c), ga, gb);
-          *reinterpret_cast<uint32_t*>(p.out + t * p.out_stride + (long long)h * p.DV + c) =
-              pack_bf2(o[tt][j][2 * e] * inv * __fdividef(1.f, 1.f + __expf(-ga)),
-                       o[tt][j][2 * e + 1] * inv * __fdividef(1.f, 1.f + __expf(-gb)));
+          float a = o[tt][j][2 * e] * inv, b = o[tt][j][2 * e + 1] * inv;
+          if (p.gate) {
+            float ga, gb;
+            unpack_bf2(*reinterpret_cast<const uint32_t*>(p.gate + t * p.gate_stride + (long long)h * p.DV + c), ga, gb);
+            a *= __fdividef(1.f, 1.f + __expf(-ga));
+            b *= __fdividef(1.f, 1.f + __expf(-gb));
+          }
+          *reinterpret_cast<uint32_t*>(p.out + t * p.out_stride + (long long)h * p.DV + c) = pack_bf2(a, b);
         }
       }
     }
 }
 
-template <int DK, int DV, int MT>
+template <int DK, int DV, int MT, bool PAGED>
 inline int latent_expand_launch(const LatentExpandParams& p, int max_len, int n, cudaStream_t st) {
   constexpr int smem = LexLayout<DK, DV, MT>::BYTES, LEX_BM = LexLayout<DK, DV, MT>::BM;
   static_assert(smem <= 227 * 1024, "shared memory budget");
   static PerDeviceFlags attr_set;
-  if (int rc = set_max_dyn_smem_once(attr_set, latent_expand_kernel<DK, DV, MT>, smem)) return rc;
-  launch_k(latent_expand_kernel<DK, DV, MT>, dim3((unsigned)((max_len + LEX_BM - 1) / LEX_BM), (unsigned)p.heads, (unsigned)n),
-           dim3(LEX_THREADS), (size_t)smem, st, p);
+  if (int rc = set_max_dyn_smem_once(attr_set, latent_expand_kernel<DK, DV, MT, PAGED>, smem)) return rc;
+  launch_k(latent_expand_kernel<DK, DV, MT, PAGED>,
+           dim3((unsigned)((max_len + LEX_BM - 1) / LEX_BM), (unsigned)p.heads, (unsigned)n), dim3(LEX_THREADS), (size_t)smem,
+           st, p);
   return launch_status();
+}
+
+template <bool PAGED>
+inline int latent_expand_dispatch(const LatentExpandParams& p, int max_len, int n, cudaStream_t st) {
+  const int dk = p.DN + p.DR;
+  const bool two = max_len > 128;
+  if (dk <= 64 && p.DV <= 64)
+    return two ? latent_expand_launch<64, 64, 2, PAGED>(p, max_len, n, st) : latent_expand_launch<64, 64, 1, PAGED>(p, max_len, n, st);
+  if (dk <= 128 && p.DV <= 128)
+    return two ? latent_expand_launch<128, 128, 2, PAGED>(p, max_len, n, st) : latent_expand_launch<128, 128, 1, PAGED>(p, max_len, n, st);
+  if (dk <= 192 && p.DV <= 128)
+    return two ? latent_expand_launch<192, 128, 2, PAGED>(p, max_len, n, st) : latent_expand_launch<192, 128, 1, PAGED>(p, max_len, n, st);
+  return latent_expand_launch<256, 256, 1, PAGED>(p, max_len, n, st);
 }
 
 }  // namespace b200
 
-// Causal attention of n gathered sequences (bf16; see the head of this file).  DN, DR, DV multiples of 8,
+// Causal attention of n gathered sequences (bf16; see the head of this file): packed row r of sequence i holds the key at
+// position key_base[i] + r - key_start[i], up to its last.  gate NULL: no output gate.  DN, DR, DV multiples of 8,
 // DN + DR and DV <= 256; max_len: the most tokens any of them brings in this step.
 extern "C" int b200_latent_attn_expanded(const void* q, long long q_row_stride, const void* kv, long long kv_row_stride,
                                          const void* lat, long long lat_row_stride, int rot_off, const void* gate,
                                          long long gate_row_stride, void* out, long long out_row_stride,
                                          const void* query_start_loc, const void* context_lens, const void* seq_ids_i32,
-                                         const void* key_start_i32, int n, int max_len, int heads, int DN, int DR, int DV,
-                                         float scale, void* stream) {
+                                         const void* key_start_i32, const void* key_base_i32, int n, int max_len, int window,
+                                         int heads, int DN, int DR, int DV, float scale, void* stream) {
   using namespace b200;
-  if (!q || !kv || !lat || !gate || !out || !query_start_loc || !context_lens || !seq_ids_i32 || !key_start_i32 || n <= 0 ||
-      max_len <= 0 || heads <= 0 || DN <= 0 || DR < 0 || DV <= 0)
+  if (!q || !kv || !lat || !out || !query_start_loc || !context_lens || !seq_ids_i32 || !key_start_i32 || !key_base_i32 ||
+      n <= 0 || max_len <= 0 || heads <= 0 || DN <= 0 || DR < 0 || DV <= 0 || window < 0)
     return B200_ERR_ARG;
   if (DN % 8 || DR % 8 || DV % 8 || rot_off % 8 || q_row_stride % 8 || kv_row_stride % 8 || lat_row_stride % 8 ||
       gate_row_stride % 8 || out_row_stride % 8 || DN + DR > 256 || DV > 256 || heads > 65535 || n > 65535)
     return B200_ERR_SHAPE;
-  LatentExpandParams p{(const int*)query_start_loc, (const int*)context_lens, (const int*)seq_ids_i32,
-                       (const int*)key_start_i32, (const __nv_bfloat16*)q, (const __nv_bfloat16*)kv,
-                       (const __nv_bfloat16*)lat, (const __nv_bfloat16*)gate, (__nv_bfloat16*)out, q_row_stride,
-                       kv_row_stride, lat_row_stride, gate_row_stride, out_row_stride, heads, DN, DR, DV, rot_off,
-                       scale * kLog2e};
-  const int dk = DN + DR;
-  const cudaStream_t st = (cudaStream_t)stream;
-  const bool two = max_len > 128;
-  if (dk <= 64 && DV <= 64) return two ? latent_expand_launch<64, 64, 2>(p, max_len, n, st) : latent_expand_launch<64, 64, 1>(p, max_len, n, st);
-  if (dk <= 128 && DV <= 128)
-    return two ? latent_expand_launch<128, 128, 2>(p, max_len, n, st) : latent_expand_launch<128, 128, 1>(p, max_len, n, st);
-  if (dk <= 192 && DV <= 128)
-    return two ? latent_expand_launch<192, 128, 2>(p, max_len, n, st) : latent_expand_launch<192, 128, 1>(p, max_len, n, st);
-  return latent_expand_launch<256, 256, 1>(p, max_len, n, st);
+  LatentExpandParams p{};
+  p.seqs.query_start_loc = (const int*)query_start_loc;
+  p.seqs.context_lens = (const int*)context_lens;
+  p.seqs.window = window;
+  p.seq_ids = (const int*)seq_ids_i32;
+  p.key_start = (const int*)key_start_i32;
+  p.key_base = (const int*)key_base_i32;
+  p.q = (const __nv_bfloat16*)q;
+  p.k = (const __nv_bfloat16*)kv;
+  p.v = (const __nv_bfloat16*)kv + (long long)heads * DN;
+  p.rot = (const __nv_bfloat16*)lat + rot_off;
+  p.gate = (const __nv_bfloat16*)gate;
+  p.out = (__nv_bfloat16*)out;
+  p.q_stride = q_row_stride;
+  p.k_stride = p.v_stride = kv_row_stride;
+  p.rot_stride = lat_row_stride;
+  p.gate_stride = gate_row_stride;
+  p.out_stride = out_row_stride;
+  p.heads = heads;
+  p.group = 1;
+  p.DN = DN;
+  p.DR = DR;
+  p.DV = DV;
+  p.scale_log2 = scale * kLog2e;
+  return latent_expand_dispatch<false>(p, max_len, n, (cudaStream_t)stream);
+}
+
+// The same kernel over the pages of a per-head cache: k_cache [blocks, page, kv_heads, DK], v_cache [.., DV], contiguous.
+extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache,
+                                        void* out, long long out_row_stride, const void* query_start_loc,
+                                        const void* context_lens, const void* page_table, long long page_table_stride,
+                                        int max_pages, int page_size, int num_blocks, int num_seqs, const void* seq_ids_i32,
+                                        int n, int max_len, int window, int heads, int kv_heads, int DK, int DV, float scale,
+                                        void* stream) {
+  using namespace b200;
+  LatentExpandParams p{};
+  p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
+            page_size, num_blocks, num_seqs, 0, 0, window};
+  if (!latent_seqs_ok(p.seqs) || !q || !k_cache || !v_cache || !out || !seq_ids_i32 || n <= 0 || max_len <= 0 || heads <= 0 ||
+      kv_heads <= 0 || heads % kv_heads || DK <= 0 || DV <= 0 || window < 0)
+    return B200_ERR_ARG;
+  if (DK % 8 || DV % 8 || q_row_stride % 8 || out_row_stride % 8 || DK > 256 || DV > 256 || heads > 65535 || n > 65535)
+    return B200_ERR_SHAPE;
+  p.seq_ids = (const int*)seq_ids_i32;
+  p.q = (const __nv_bfloat16*)q;
+  p.k = (const __nv_bfloat16*)k_cache;
+  p.v = (const __nv_bfloat16*)v_cache;
+  p.out = (__nv_bfloat16*)out;
+  p.q_stride = q_row_stride;
+  p.k_stride = (long long)kv_heads * DK;
+  p.v_stride = (long long)kv_heads * DV;
+  p.out_stride = out_row_stride;
+  p.heads = heads;
+  p.group = heads / kv_heads;
+  p.DN = DK;
+  p.DV = DV;
+  p.scale_log2 = scale * kLog2e;
+  return latent_expand_dispatch<true>(p, max_len, n, (cudaStream_t)stream);
 }

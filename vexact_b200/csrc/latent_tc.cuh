@@ -19,6 +19,9 @@
 // more than 2^8 (weights up to 2^8 are as exact as weights up to 1); then the sums so far are taken into registers and
 // rescaled, and O^T starts anew.
 //
+// With a window the walk starts at the block (of 128) that holds the first key any of the sequence's new tokens sees, and
+// the splits before it do not exist; blocks and splits lie at the same keys either way.
+//
 // Persistent CTAs take items (sequence, column tile, split) from a list made once per step (latent_plan_kernel).
 // Warps: 0 = TMA producer, 1 = UMMA issuer and TMEM owner, 2..9 = softmax and accumulation (thread = TMEM lane, half of
 // the columns), 10 = query loader.  A row whose sequence has one split is finished here, otherwise
@@ -42,7 +45,7 @@ struct LatentTcParams {
   LatentSeqs seqs;
   const __nv_bfloat16* q_lat;   // [T, H, R + DR]
   __nv_bfloat16* out;           // [T, H, R]
-  const int4* items;            // pairs {sequence, first token, new tokens, context}, {column tile, split, splits, 0}
+  const int4* items;            // pairs {sequence, first token, new tokens, context}, {column tile, split, splits, first key}
   const int* item_count;
   int max_items;
   float* part_o;                // [items, 16, R]
@@ -61,6 +64,14 @@ struct LatentPlanParams {
   int* first_item;   // [S]
 };
 
+// First key walked for a sequence, and how many splits there are from the one that holds it.
+__device__ __forceinline__ int ltc_first_key(int window, int ctx, int len) {
+  return window_first(window, ctx - len) / LTC_BN * LTC_BN;
+}
+__device__ __forceinline__ int ltc_splits(int first_key, int ctx) {
+  return (ctx + LTC_SPLIT - 1) / LTC_SPLIT - first_key / LTC_SPLIT;
+}
+
 __global__ void __launch_bounds__(1024) latent_plan_kernel(const LatentPlanParams p) {
   __shared__ int s_warp[32];
   __shared__ int s_base;
@@ -71,14 +82,15 @@ __global__ void __launch_bounds__(1024) latent_plan_kernel(const LatentPlanParam
   __syncthreads();
   for (int s0 = 0; s0 < p.seqs.num_seqs; s0 += 1024) {
     const int s = s0 + tid;
-    int tiles = 0, splits = 0, t0 = 0, len = 0, ctx = 0;
+    int tiles = 0, splits = 0, t0 = 0, len = 0, ctx = 0, key = 0;
     if (s < p.seqs.num_seqs) {
       t0 = p.seqs.query_start_loc[s];
       len = p.seqs.query_start_loc[s + 1] - t0;
       ctx = p.seqs.context_lens[s];
       if (len >= p.seqs.min_len && len <= p.seqs.max_len && len > 0) {
         tiles = (len * p.heads + LTC_NC - 1) / LTC_NC;
-        splits = (ctx + LTC_SPLIT - 1) / LTC_SPLIT;
+        key = ltc_first_key(p.seqs.window, ctx, len);
+        splits = ltc_splits(key, ctx);
       }
     }
     const int n = tiles * splits;
@@ -97,7 +109,7 @@ __global__ void __launch_bounds__(1024) latent_plan_kernel(const LatentPlanParam
     for (int i = 0; i < n; ++i) {
       if (first + i < p.max_items) {
         p.items[2 * (first + i)] = make_int4(s, t0, len, ctx);
-        p.items[2 * (first + i) + 1] = make_int4(i / splits, i % splits, splits, 0);
+        p.items[2 * (first + i) + 1] = make_int4(i / splits, key / LTC_SPLIT + i % splits, splits, key);
       } else report_status(B200_STATUS_BAD_INDEX, first + i);
     }
     __syncthreads();
@@ -126,7 +138,8 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentCombine
   const int s = latent_seq_of(p.seqs.query_start_loc, p.seqs.num_seqs, t);
   const int t0 = p.seqs.query_start_loc[s], len = p.seqs.query_start_loc[s + 1] - t0;
   if (t < t0 || t >= t0 + len || len < p.seqs.min_len || len > p.seqs.max_len) return;
-  const int splits = (p.seqs.context_lens[s] + LTC_SPLIT - 1) / LTC_SPLIT;
+  const int ctx = p.seqs.context_lens[s];
+  const int splits = ltc_splits(ltc_first_key(p.seqs.window, ctx, len), ctx);
   if (splits <= 1) return;
   const int row = (int)(t - t0) * p.heads + h;
   const long long item = p.first_item[s] + (long long)(row / LTC_NC) * splits;
@@ -174,8 +187,8 @@ __device__ __forceinline__ LtcItem ltc_item(const LatentTcParams& p, const LtcRa
   t.ctx = r.a.w;
   t.tile = r.b.x;
   t.splits = r.b.z;
-  t.key0 = r.b.y * LTC_SPLIT;
-  t.nblk = (min(t.ctx, t.key0 + LTC_SPLIT) - t.key0 + LTC_BN - 1) / LTC_BN;
+  t.key0 = max(r.b.y * LTC_SPLIT, r.b.w);
+  t.nblk = (min(t.ctx, (r.b.y + 1) * LTC_SPLIT) - t.key0 + LTC_BN - 1) / LTC_BN;
   t.rows = min(LTC_NC, t.len * p.heads - t.tile * LTC_NC);
   return t;
 }
@@ -435,6 +448,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
     const int mycol = halving_col<NH>(lane);
     uint8_t* p_mine = base_ptr + p_off + (tl >> 6) * (2 * NC * 128) + (tl & 7) * 2;
     const int p_ch = (tl & 63) >> 3;
+    const uint32_t reach = p.seqs.window > 0 ? (uint32_t)p.seqs.window : 0x80000000u;   // keys a column sees: 0 <= cpos - key < reach
     uint32_t g = 0;
     LtcRaw raw_next = ltc_raw(p, blockIdx.x, count);
     for (int idx = blockIdx.x; idx < count; idx += gridDim.x) {
@@ -474,7 +488,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
           ptx::tmem_ld_wait();
 #pragma unroll
           for (int i = 0; i < NH; ++i) {
-            v[i] = key > cpos[i] ? -INFINITY : __uint_as_float(r[i]) * p.scale_log2;
+            v[i] = (uint32_t)(cpos[i] - key) >= reach ? -INFINITY : __uint_as_float(r[i]) * p.scale_log2;
             over |= v[i] > m[i] + LTC_SLACK;
           }
           // keys past the context may hold anything: clear their rows of c so that 0 * value stays 0
@@ -610,15 +624,16 @@ inline int latent_tc_launch(const CUtensorMap& tm, const LatentTcParams& p, int 
 }  // namespace b200
 
 // Work items of a step for b200_latent_attn_tc: items [max_items] pairs of int4, item_count [1], first_item [num_seqs] (i32).
-// The list depends on the sequences and the head count only, so one list serves every layer with `heads` heads.
+// The list depends on the sequences, the head count and the window only, so one list serves every layer that shares them.
 extern "C" int b200_latent_plan(const void* query_start_loc, const void* context_lens, int num_seqs, int min_len,
-                                int max_len, int heads, int max_items, void* items, void* item_count, void* first_item,
+                                int max_len, int window, int heads, int max_items, void* items, void* item_count, void* first_item,
                                 void* stream) {
   using namespace b200;
   if (!query_start_loc || !context_lens || !items || !item_count || !first_item || num_seqs <= 0 || heads <= 0 ||
-      max_items <= 0)
+      max_items <= 0 || window < 0)
     return B200_ERR_ARG;
-  LatentPlanParams p{{(const int*)query_start_loc, (const int*)context_lens, nullptr, 0, 0, 0, 0, num_seqs, min_len, max_len},
+  LatentPlanParams p{{(const int*)query_start_loc, (const int*)context_lens, nullptr, 0, 0, 0, 0, num_seqs, min_len, max_len,
+                      window},
                      heads, max_items, (int4*)items, (int*)item_count, (int*)first_item};
   launch_k(latent_plan_kernel, dim3(1), dim3(1024), 0, (cudaStream_t)stream, p);
   return launch_status();
@@ -626,18 +641,19 @@ extern "C" int b200_latent_plan(const void* query_start_loc, const void* context
 
 // b200_latent_attn_simt on tensor cores (bf16) for the sequences of a plan; min_len / max_len as the plan was made with.
 // R <= 512, DR <= 128, multiples of 8; page_size a power of two of at least 8, or a multiple of 128.
-// part_o [max_items, 16, R] and part_ml [max_items, 16, 2] fp32: scratch, NULL when no context exceeds 512 tokens.
+// part_o [max_items, 16, R] and part_ml [max_items, 16, 2] fp32: scratch, NULL when no sequence has several splits (of 512
+// keys, at multiples of 512).
 extern "C" int b200_latent_attn_tc(const void* q_lat, const void* cache, void* out, const void* query_start_loc,
                                    const void* context_lens, const void* page_table, long long page_table_stride,
                                    int max_pages, int page_size, int num_blocks, int num_seqs, int min_len, int max_len,
-                                   long long T, int heads, int R, int DR, float scale, const void* items,
+                                   int window, long long T, int heads, int R, int DR, float scale, const void* items,
                                    const void* item_count, const void* first_item, int max_items, void* part_o,
                                    void* part_ml, void* stream) {
   using namespace b200;
   LatentTcParams p{};
   p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
-            page_size, num_blocks, num_seqs, min_len, max_len};
-  if (!latent_seqs_ok(p.seqs) || !q_lat || !cache || !out || !items || !item_count || !first_item || T < 0 || heads <= 0 ||
+            page_size, num_blocks, num_seqs, min_len, max_len, window};
+  if (!latent_seqs_ok(p.seqs) || window < 0 || !q_lat || !cache || !out || !items || !item_count || !first_item || T < 0 || heads <= 0 ||
       R <= 0 || DR <= 0 || max_items <= 0 || (part_o != nullptr) != (part_ml != nullptr))
     return B200_ERR_ARG;
   const bool pages_ok = page_size % LTC_BN == 0 || (page_size >= 8 && LTC_BN % page_size == 0);

@@ -13,11 +13,15 @@
 #include "step.cuh"
 #include "sample.cuh"
 #include "hyper.cuh"
+#include "residual.cuh"
 #include "ssm.cuh"
 #include "ssm_chunk.cuh"
+#include "delta.cuh"
+#include "delta_chunk.cuh"
 #include "latent.cuh"
 #include "latent_expand.cuh"
 #include "latent_tc.cuh"
+#include "window_attn.cuh"
 
 // Self-test of the bounded wait every kernel here relies on: one CTA waits, with a limit of
 // `limit_us` microseconds, on an mbarrier that nothing ever completes.  The wait must give up, record
@@ -64,7 +68,7 @@ extern "C" int b200_status_read(int* host_out4, void* stream) {
 }
 
 // Bumped whenever an exported signature changes.
-extern "C" int b200_abi_version(void) { return 5; }
+extern "C" int b200_abi_version(void) { return 6; }
 
 // Hash of the sources and compiler flags this binary was built from (set by the build script);
 // the loader compares it with the sources beside it and refuses a stale library.

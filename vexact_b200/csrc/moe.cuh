@@ -23,9 +23,9 @@ namespace b200 {
 constexpr int MOE_MAX_EXPERTS = 256;
 constexpr int MOE_MAX_TOPK = 16;
 
-// Softmax -> top-k -> renorm of one token's logits by one warp.  Each lane owns experts lane,
-// lane + 32, ... (up to 8).
-template <typename TIn>
+// Scores -> top-k -> renorm of one token's logits by one warp.  Each lane owns experts lane,
+// lane + 32, ... (up to 8).  Scores: softmax over the experts, or (SIGMOID) each expert's sigmoid.
+template <typename TIn, bool SIGMOID = false>
 __device__ __forceinline__ void route_softmax_topk_token(const TIn* __restrict__ row, long long tok,
                                                          __nv_bfloat16* __restrict__ w_bf16,
                                                          float* __restrict__ w_f32, int* __restrict__ idx_i32,
@@ -40,18 +40,20 @@ __device__ __forceinline__ void route_softmax_topk_token(const TIn* __restrict__
     v[i] = e < E ? (float)row[e] : -INFINITY;
     mx = fmaxf(mx, v[i]);
   }
-  mx = warp_max(mx);
   float sum = 0.f;
+  if constexpr (!SIGMOID) {
+    mx = warp_max(mx);
 #pragma unroll
-  for (int i = 0; i < PER; ++i) {
-    const int e = lane + 32 * i;
-    v[i] = e < E ? expf(v[i] - mx) : 0.f;
-    sum += v[i];
+    for (int i = 0; i < PER; ++i) {
+      const int e = lane + 32 * i;
+      v[i] = e < E ? expf(v[i] - mx) : 0.f;
+      sum += v[i];
+    }
+    sum = warp_sum(sum);
   }
-  sum = warp_sum(sum);
 #pragma unroll
   for (int i = 0; i < PER; ++i) {
-    v[i] = v[i] / sum;  // softmax probabilities (fp32)
+    v[i] = SIGMOID ? 1.f / (1.f + expf(-v[i])) : v[i] / sum;  // softmax probabilities (fp32)
     // A row of NaN logits (a padded token of a captured batch: its hidden state is never defined) must
     // still select experts inside [0, E): NaN compares false with everything, so it counts as 0 here.
     if (!(v[i] == v[i])) v[i] = 0.f;
@@ -837,10 +839,11 @@ extern "C" int b200_moe_route_softmax_topk(const void* logits, int logits_dtype 
 // (it is what reproduces the reference's index arrays).
 namespace b200 {
 
-template <typename TIn>
+// gate_f32: sigmoid of the logit in column E (a gate that shares the router's product), or null.
+template <typename TIn, bool SIGMOID = false>
 __global__ void __launch_bounds__(256)
 moe_route_plan_kernel(const TIn* __restrict__ logits, long long row_stride, __nv_bfloat16* __restrict__ w_bf16,
-                      long long* __restrict__ idx_i64, int* __restrict__ rank_out, int* __restrict__ counters,
+                      float* __restrict__ w_f32, float* __restrict__ gate_f32, long long* __restrict__ idx_i64, int* __restrict__ rank_out, int* __restrict__ counters,
                       int* __restrict__ cu_seqlens, int4* __restrict__ tile_table, int* __restrict__ tile_count,
                       long long T, int E, int topk, int renorm, int tile_rows, int max_tiles) {
   pdl_trigger();
@@ -850,8 +853,9 @@ moe_route_plan_kernel(const TIn* __restrict__ logits, long long row_stride, __nv
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const long long tok = (long long)blockIdx.x * 8 + warp;
   if (tok < T) {
-    route_softmax_topk_token<TIn>(logits + tok * row_stride, tok, w_bf16, nullptr, nullptr, idx_i64, E, topk, renorm,
-                                  lane);
+    route_softmax_topk_token<TIn, SIGMOID>(logits + tok * row_stride, tok, w_bf16, w_f32, nullptr, idx_i64, E, topk,
+                                           renorm, lane);
+    if (gate_f32 && lane == 0) gate_f32[tok] = 1.f / (1.f + expf(-(float)logits[tok * row_stride + E]));
     __syncwarp();
     // the expert ids were just written by lane 0: lane k takes entry k's rank in its expert's group
     if (lane < topk) {
@@ -906,12 +910,13 @@ moe_route_plan_kernel(const TIn* __restrict__ logits, long long row_stride, __nv
 }
 
 // Row f = (token f / topk, choice f % topk) goes to sorted row cu_seqlens[expert] + rank[f].
+template <typename TW>
 __global__ void __launch_bounds__(128)
 moe_scatter_ranked_kernel(const __nv_bfloat16* __restrict__ x, long long x_stride,
-                          const long long* __restrict__ experts, const __nv_bfloat16* __restrict__ weights,
+                          const long long* __restrict__ experts, const TW* __restrict__ weights,
                           const int* __restrict__ rank, const int* __restrict__ cu_seqlens,
                           int* __restrict__ scatter_index, __nv_bfloat16* __restrict__ x_perm,
-                          __nv_bfloat16* __restrict__ row_scale, int H, int topk, int E, long long n) {
+                          TW* __restrict__ row_scale, int H, int topk, int E, long long n) {
   pdl_trigger();
   pdl_wait();
   const long long f = blockIdx.x;
@@ -962,12 +967,13 @@ extern "C" int b200_moe_route_plan_softmax_topk(const void* logits, int logits_d
   const unsigned grid = (unsigned)((T + 7) / 8);
   if (logits_dtype == 0)
     launch_k(moe_route_plan_kernel<float>, dim3(grid), dim3(256), 0, st, (const float*)logits, row_stride,
-             (__nv_bfloat16*)weights_bf16, (long long*)experts_i64, (int*)rank_i32, (int*)counters_i32,
+             (__nv_bfloat16*)weights_bf16, (float*)nullptr, (float*)nullptr, (long long*)experts_i64, (int*)rank_i32,
+             (int*)counters_i32,
              (int*)cu_seqlens, (int4*)tile_table, (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles);
   else if (logits_dtype == 1)
     launch_k(moe_route_plan_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, st, (const __nv_bfloat16*)logits,
-             row_stride, (__nv_bfloat16*)weights_bf16, (long long*)experts_i64, (int*)rank_i32, (int*)counters_i32,
-             (int*)cu_seqlens, (int4*)tile_table, (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles);
+             row_stride, (__nv_bfloat16*)weights_bf16, (float*)nullptr, (float*)nullptr, (long long*)experts_i64,
+             (int*)rank_i32, (int*)counters_i32, (int*)cu_seqlens, (int4*)tile_table, (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles);
   else
     return B200_ERR_ARG;
   return launch_status();
@@ -986,9 +992,48 @@ extern "C" int b200_moe_scatter_ranked(const void* x, long long x_row_stride, co
   const long long n = T * topk;
   if (n == 0) return B200_OK;
   if (n > 0x7fffffffLL) return B200_ERR_SHAPE;
-  launch_k(moe_scatter_ranked_kernel, dim3((unsigned)n), dim3(128), 0, (cudaStream_t)stream, (const __nv_bfloat16*)x,
-           x_row_stride, (const long long*)experts_i64, (const __nv_bfloat16*)weights_bf16, (const int*)rank_i32,
-           (const int*)cu_seqlens, (int*)scatter_index, (__nv_bfloat16*)x_perm, (__nv_bfloat16*)row_scale, H, topk, E, n);
+  launch_k(moe_scatter_ranked_kernel<__nv_bfloat16>, dim3((unsigned)n), dim3(128), 0, (cudaStream_t)stream,
+           (const __nv_bfloat16*)x, x_row_stride, (const long long*)experts_i64, (const __nv_bfloat16*)weights_bf16,
+           (const int*)rank_i32, (const int*)cu_seqlens, (int*)scatter_index, (__nv_bfloat16*)x_perm,
+           (__nv_bfloat16*)row_scale, H, topk, E, n);
+  return launch_status();
+}
+
+// The same pair for routers that score experts by their sigmoid and keep fp32 weights: weights = the chosen scores as they
+// are (renorm 0) or over their sum; gate_f32 [T] (or NULL) = sigmoid of the logit in column E, a gate whose projection is
+// stacked under the router's.
+extern "C" int b200_moe_route_plan_sigmoid_topk(const void* logits_f32, long long row_stride, void* weights_f32,
+                                                void* gate_f32, void* experts_i64, void* rank_i32, void* counters_i32,
+                                                void* cu_seqlens, void* tile_table, void* tile_count, long long T, int E,
+                                                int topk, int renorm, int tile_rows, int max_tiles, void* stream) {
+  using namespace b200;
+  if (!logits_f32 || !weights_f32 || !experts_i64 || !rank_i32 || !counters_i32 || !cu_seqlens || !tile_table ||
+      !tile_count || T <= 0 || E <= 0 || topk <= 0 || tile_rows <= 0 || max_tiles <= 0)
+    return B200_ERR_ARG;
+  if (E > MOE_MAX_EXPERTS || topk > MOE_MAX_TOPK || topk > E || row_stride < E + (gate_f32 ? 1 : 0)) return B200_ERR_SHAPE;
+  launch_k(moe_route_plan_kernel<float, true>, dim3((unsigned)((T + 7) / 8)), dim3(256), 0, (cudaStream_t)stream,
+           (const float*)logits_f32, row_stride, (__nv_bfloat16*)nullptr, (float*)weights_f32, (float*)gate_f32,
+           (long long*)experts_i64, (int*)rank_i32, (int*)counters_i32, (int*)cu_seqlens, (int4*)tile_table,
+           (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles);
+  return launch_status();
+}
+
+// b200_moe_scatter_ranked with fp32 weights and rows of either model dtype: row_bytes a multiple of 16.
+extern "C" int b200_moe_scatter_ranked_f32(const void* x, long long x_row_bytes, const void* experts_i64,
+                                           const void* weights_f32, const void* rank_i32, const void* cu_seqlens,
+                                           void* scatter_index, void* x_perm, void* row_scale_f32, long long T, int topk,
+                                           int E, int row_bytes, void* stream) {
+  using namespace b200;
+  if (!x || !experts_i64 || !weights_f32 || !rank_i32 || !cu_seqlens || !scatter_index || !x_perm || !row_scale_f32 ||
+      T < 0 || topk <= 0 || E <= 0 || row_bytes <= 0)
+    return B200_ERR_ARG;
+  const long long n = T * topk;
+  if (row_bytes % 16 != 0 || x_row_bytes % 16 != 0 || n > 0x7fffffffLL) return B200_ERR_SHAPE;
+  if (n == 0) return B200_OK;
+  launch_k(moe_scatter_ranked_kernel<float>, dim3((unsigned)n), dim3(128), 0, (cudaStream_t)stream, (const __nv_bfloat16*)x,
+           x_row_bytes / 2, (const long long*)experts_i64, (const float*)weights_f32, (const int*)rank_i32,
+           (const int*)cu_seqlens, (int*)scatter_index, (__nv_bfloat16*)x_perm, (float*)row_scale_f32, row_bytes / 2, topk, E,
+           n);
   return launch_status();
 }
 

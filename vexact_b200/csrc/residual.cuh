@@ -1,0 +1,188 @@
+// One residual stream (fp32) with a norm on both sides of every sublayer, fused across the boundary of two sublayers.
+//
+// For every token, with y the output of the sublayer just done:
+//     x  <- x + y / sqrt(mean(y^2) + eps) * post            (start of the model: x = 0 and y the embedding row)
+//     x  <- x + add                                         (optional vector, the same for every token)
+//     xn  = x / sqrt(mean(x^2) + eps) * norm                (the next sublayer's input)
+// y comes as rows, or as what a mixture of experts leaves: expert-sorted rows of which a token sums `topk` (found through
+// scatter_index), plus a row of the shared expert; that sum is then never a tensor of its own.
+//
+// One CTA per token, everything in registers between the two reductions.  `rows` picks tokens at the end of a model;
+// nothing is written back then.
+// Algorithmic bytes per token: 8 W (x) + b W (topk + shared rows of y) + b W (xn), b = 2 or 4: HBM bandwidth.
+#pragma once
+#include "hyper.cuh"   // load4 / store4 / to_f32 / from_f32
+
+namespace b200 {
+
+constexpr int RES_CHUNKS = 4;   // register chunks per thread: W <= threads * RES_CHUNKS * 4
+
+struct ResidualParams {
+  float* x;                   // [T, W]
+  const void* y;              // [T or y_rows, y_stride], or null (then `extra` or ids)
+  long long y_stride, y_rows;
+  const int* scatter_index;   // [T, topk] rows of y to sum, or null (row t)
+  int topk;
+  const void* extra;          // [T, extra_stride] added to y, or null
+  long long extra_stride;
+  const void* embed;          // [vocab, W] or null
+  const long long* ids;       // [T]
+  long long vocab;
+  const int* rows;            // [R] source token of each output row, or null (row r is token r)
+  long long num_tokens;
+  const float* post;          // [W]
+  const float* add;           // [W] or null
+  const float* norm_w;        // [W] or null (no xn)
+  float eps;
+  void* xn;                   // [R, xn_stride]; columns W .. xn_cols are zeroed
+  long long xn_stride;
+  int xn_cols;
+  int W;
+  int write_back;
+};
+
+template <typename T>
+__device__ __forceinline__ void load4_tail(const T* p, int left, float (&v)[4]) {
+#pragma unroll
+  for (int k = 0; k < 4; ++k) v[k] = k < left ? to_f32(p[k]) : 0.f;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualParams p) {
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const long long r = blockIdx.x;
+  long long t = p.rows ? p.rows[r] : r;
+  if (t < 0 || t >= p.num_tokens) {
+    if (threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, (int)t);
+    t = 0;
+  }
+  const int W = p.W;
+  const bool vec = W % 4 == 0;
+  auto get = [&](const auto* row, int i, float (&v)[4]) {
+    if (vec) load4(row + i, v);
+    else load4_tail(row + i, W - i, v);
+  };
+  const T* src = nullptr;      // the one row of y, or of the embedding
+  if (p.ids) {
+    long long id = p.ids[t];
+    if (id < 0 || id >= p.vocab) {
+      if (threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, (int)id);
+      id = 0;
+    }
+    src = reinterpret_cast<const T*>(p.embed) + id * W;
+  } else if (p.y && !p.scatter_index) {
+    src = reinterpret_cast<const T*>(p.y) + t * p.y_stride;
+  }
+  const T* extra = p.extra ? reinterpret_cast<const T*>(p.extra) + t * p.extra_stride : nullptr;
+  const int* pick = p.scatter_index ? p.scatter_index + t * p.topk : nullptr;
+  float* xrow = p.x + t * (long long)W;
+  float v[RES_CHUNKS][4], x[RES_CHUNKS][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < RES_CHUNKS; ++c) {
+    const int i = (c * blockDim.x + threadIdx.x) * 4;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) v[c][k] = x[c][k] = 0.f;
+    if (i >= W) continue;
+    if (src) get(src, i, v[c]);
+    if (!p.ids) get(xrow, i, x[c]);
+    if (pick) {
+      int row = p.topk > 0 ? pick[0] : -1;
+      for (int k = 0; k < p.topk; ++k) {
+        const int next = k + 1 < p.topk ? pick[k + 1] : -1;
+        if (row >= 0 && row < p.y_rows) {
+          float e[4];
+          get(reinterpret_cast<const T*>(p.y) + row * p.y_stride, i, e);
+#pragma unroll
+          for (int q = 0; q < 4; ++q) v[c][q] += e[q];
+        } else if (threadIdx.x == 0 && c == 0) {
+          report_status(B200_STATUS_BAD_INDEX, row);
+        }
+        row = next;
+      }
+    }
+    if (extra) {
+      float e[4];
+      get(extra, i, e);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) v[c][q] += e[q];
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) ss = fmaf(v[c][k], v[c][k], ss);
+  }
+  ss = block_sum(ss, red);
+  const float inv_y = 1.f / sqrtf(ss / (float)W + p.eps);
+  ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < RES_CHUNKS; ++c) {
+    const int i = (c * blockDim.x + threadIdx.x) * 4;
+    if (i >= W) continue;
+    float w[4], a[4] = {0.f, 0.f, 0.f, 0.f};
+    get(p.post, i, w);
+    if (p.add) get(p.add, i, a);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      x[c][k] = x[c][k] + v[c][k] * inv_y * w[k] + a[k];
+      ss = fmaf(x[c][k], x[c][k], ss);      // columns past W are zero in every term
+    }
+    if (p.write_back) {
+      if (vec) store4(xrow + i, x[c]);
+      else
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (i + k < W) xrow[i + k] = x[c][k];
+    }
+  }
+  if (!p.norm_w) return;
+  ss = block_sum(ss, red);
+  const float inv = 1.f / sqrtf(ss / (float)W + p.eps);
+  T* orow = reinterpret_cast<T*>(p.xn) + r * p.xn_stride;
+#pragma unroll
+  for (int c = 0; c < RES_CHUNKS; ++c) {
+    const int i = (c * blockDim.x + threadIdx.x) * 4;
+    if (i >= W) continue;
+    float w[4];
+    get(p.norm_w, i, w);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) w[k] *= x[c][k] * inv;
+    if (vec) store4(orow + i, w);
+    else
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        if (i + k < W) orow[i + k] = from_f32<T>(w[k]);
+  }
+  for (int i = W + threadIdx.x; i < p.xn_cols; i += blockDim.x) orow[i] = from_f32<T>(0.f);
+}
+
+}  // namespace b200
+
+// dtype: 0 = bf16, 1 = fp32 (embed, y, extra and xn; the residual and the norm weights are always fp32).
+extern "C" int b200_residual_step(void* x_f32, const void* y, long long y_row_stride, long long y_rows,
+                                  const void* scatter_index_i32, int topk, const void* extra, long long extra_row_stride,
+                                  const void* embed, const void* ids_i64, long long vocab, const void* rows_i32,
+                                  long long num_tokens, long long num_rows, int W, const void* post_f32,
+                                  const void* add_f32, const void* norm_w_f32, float eps, void* xn,
+                                  long long xn_row_stride, int xn_cols, int write_back, int dtype, void* stream) {
+  using namespace b200;
+  if (!x_f32 || !post_f32 || num_tokens < 0 || num_rows < 0 || W <= 0 || (dtype != 0 && dtype != 1)) return B200_ERR_ARG;
+  if ((y != nullptr) == (ids_i64 != nullptr) || (ids_i64 && (!embed || extra)) || (scatter_index_i32 && (!y || topk < 1)))
+    return B200_ERR_ARG;
+  if ((norm_w_f32 && (!xn || xn_cols < W)) || (rows_i32 && write_back)) return B200_ERR_ARG;
+  if (num_rows > 0x7fffffffLL) return B200_ERR_SHAPE;
+  if (num_rows == 0) return B200_OK;
+  if (W % 4 == 0 && (y_row_stride % 4 || xn_row_stride % 4 || extra_row_stride % 4)) return B200_ERR_SHAPE;
+  const int chunks = (W + 3) / 4;
+  int threads = 64;
+  while (threads < 512 && chunks > threads) threads <<= 1;
+  while (threads < 1024 && chunks > threads * RES_CHUNKS) threads <<= 1;
+  if (chunks > threads * RES_CHUNKS) return B200_ERR_SHAPE;
+  ResidualParams p{(float*)x_f32, y, y_row_stride, y_rows, (const int*)scatter_index_i32, topk, extra, extra_row_stride,
+                   embed, (const long long*)ids_i64, vocab, (const int*)rows_i32, num_tokens, (const float*)post_f32,
+                   (const float*)add_f32, (const float*)norm_w_f32, eps, xn, xn_row_stride, xn_cols, W, write_back};
+  const dim3 g((unsigned)num_rows), b((unsigned)threads);
+  if (dtype == 0) launch_k(residual_step_kernel<__nv_bfloat16>, g, b, 0, (cudaStream_t)stream, p);
+  else launch_k(residual_step_kernel<float>, g, b, 0, (cudaStream_t)stream, p);
+  return launch_status();
+}

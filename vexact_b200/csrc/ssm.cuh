@@ -401,10 +401,12 @@ struct SsmGateNormParams {
   void* out;
   int heads, P, p_true, parts;
   float eps;
+  int norm_first;   // 1: the norm is of y alone and the gate multiplies its result; 0: the norm is of y * silu(z)
 };
 
 // The common case (heads unpadded, parts of a multiple of 8 up to 2048 columns, bf16): one warp per (token, part), its
 // gated values in registers.
+template <bool NORM_FIRST>
 __global__ void __launch_bounds__(256) ssm_gate_norm_warp_kernel(const SsmGateNormParams p, long long pairs) {
   pdl_trigger();
   pdl_wait();
@@ -436,8 +438,8 @@ __global__ void __launch_bounds__(256) ssm_gate_norm_warp_kernel(const SsmGateNo
         float y0, y1, z0, z1;
         unpack_bf2(av[k], y0, y1);
         unpack_bf2(bv[k], z0, z1);
-        g[c][2 * k] = y0 * silu_as<__nv_bfloat16>(z0);
-        g[c][2 * k + 1] = y1 * silu_as<__nv_bfloat16>(z1);
+        g[c][2 * k] = NORM_FIRST ? y0 : y0 * silu_as<__nv_bfloat16>(z0);
+        g[c][2 * k + 1] = NORM_FIRST ? y1 : y1 * silu_as<__nv_bfloat16>(z1);
         ss = fmaf(g[c][2 * k], g[c][2 * k], ss);
         ss = fmaf(g[c][2 * k + 1], g[c][2 * k + 1], ss);
       }
@@ -452,8 +454,17 @@ __global__ void __launch_bounds__(256) ssm_gate_norm_warp_kernel(const SsmGateNo
       load4(p.w + j0 + i, *reinterpret_cast<float(*)[4]>(w));
       load4(p.w + j0 + i + 4, *reinterpret_cast<float(*)[4]>(w + 4));
       uint32_t o[4];
+      const uint32_t bv[4] = {b[c].x, b[c].y, b[c].z, b[c].w};
 #pragma unroll
-      for (int k = 0; k < 4; ++k) o[k] = pack_bf2(g[c][2 * k] * inv * w[2 * k], g[c][2 * k + 1] * inv * w[2 * k + 1]);
+      for (int k = 0; k < 4; ++k) {
+        float z0 = 1.f, z1 = 1.f;
+        if constexpr (NORM_FIRST) {
+          unpack_bf2(bv[k], z0, z1);
+          z0 = silu_as<__nv_bfloat16>(z0);
+          z1 = silu_as<__nv_bfloat16>(z1);
+        }
+        o[k] = pack_bf2(g[c][2 * k] * inv * w[2 * k] * z0, g[c][2 * k + 1] * inv * w[2 * k + 1] * z1);
+      }
       *reinterpret_cast<uint4*>(out + i) = make_uint4(o[0], o[1], o[2], o[3]);
     }
   }
@@ -470,6 +481,9 @@ __global__ void __launch_bounds__(256) ssm_gate_norm_kernel(const SsmGateNormPar
   const T* z = reinterpret_cast<const T*>(p.z) + t * p.z_stride;
   T* out = reinterpret_cast<T*>(p.out) + t * p.out_stride;
   const bool plain = p.p_true == p.P;
+  // factor of y inside the norm, and of the normed value after it
+  auto inner_gate = [&](float v) { return p.norm_first ? 1.f : silu_f32(v); };
+  auto outer_gate = [&](float v) { return p.norm_first ? silu_f32(v) : 1.f; };
   auto column = [&](int j) { return plain ? j : (j / p.p_true) * p.P + j % p.p_true; };
   constexpr int KEEP = 8;
   float keep[KEEP][4];
@@ -486,7 +500,7 @@ __global__ void __launch_bounds__(256) ssm_gate_norm_kernel(const SsmGateNormPar
         load4(z + j0 + i * 4, b);
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
-          keep[c][k] = a[k] * silu_f32(b[k]);
+          keep[c][k] = a[k] * inner_gate(b[k]);
           ss = fmaf(keep[c][k], keep[c][k], ss);
         }
       }
@@ -497,7 +511,7 @@ __global__ void __launch_bounds__(256) ssm_gate_norm_kernel(const SsmGateNormPar
       load4(z + j0 + i * 4, b);
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        const float v = a[k] * silu_f32(b[k]);
+        const float v = a[k] * inner_gate(b[k]);
         ss = fmaf(v, v, ss);
       }
     }
@@ -509,8 +523,10 @@ __global__ void __launch_bounds__(256) ssm_gate_norm_kernel(const SsmGateNormPar
       if (i < chunks) {
         float w[4], o[4];
         load4(p.w + j0 + i * 4, w);
+        float b[4];
+        if (p.norm_first) load4(z + j0 + i * 4, b);
 #pragma unroll
-        for (int k = 0; k < 4; ++k) o[k] = keep[c][k] * inv * w[k];
+        for (int k = 0; k < 4; ++k) o[k] = keep[c][k] * inv * w[k] * (p.norm_first ? silu_f32(b[k]) : 1.f);
         store4(out + j0 + i * 4, o);
       }
     }
@@ -520,21 +536,21 @@ __global__ void __launch_bounds__(256) ssm_gate_norm_kernel(const SsmGateNormPar
       load4(z + j0 + i * 4, b);
       load4(p.w + j0 + i * 4, w);
 #pragma unroll
-      for (int k = 0; k < 4; ++k) o[k] = a[k] * silu_f32(b[k]) * inv * w[k];
+      for (int k = 0; k < 4; ++k) o[k] = a[k] * inner_gate(b[k]) * inv * w[k] * outer_gate(b[k]);
       store4(out + j0 + i * 4, o);
     }
     return;
   }
   for (int j = threadIdx.x; j < n; j += blockDim.x) {
     const int c = column(j0 + j);
-    const float v = to_f32(y[c]) * silu_f32(to_f32(z[c]));
+    const float v = to_f32(y[c]) * inner_gate(to_f32(z[c]));
     ss = fmaf(v, v, ss);
   }
   ss = block_sum(ss, red);
   const float inv = 1.f / sqrtf(ss / (float)n + p.eps);
   for (int j = threadIdx.x; j < n; j += blockDim.x) {
     const int c = column(j0 + j);
-    out[c] = from_f32<T>(to_f32(y[c]) * silu_f32(to_f32(z[c])) * inv * p.w[c]);
+    out[c] = from_f32<T>(to_f32(y[c]) * inner_gate(to_f32(z[c])) * inv * p.w[c] * outer_gate(to_f32(z[c])));
   }
   if (!plain && blockIdx.y == 0)
     for (int h = threadIdx.x; h < p.heads; h += blockDim.x)
@@ -600,7 +616,7 @@ extern "C" int b200_ssm_scan(const void* act, long long act_row_stride, const vo
 
 extern "C" int b200_ssm_gate_norm(const void* y, long long y_row_stride, const void* z, long long z_row_stride,
                                   const void* w_f32, void* out, long long out_row_stride, long long T, int heads, int P,
-                                  int p_true, int parts, float eps, int dtype, void* stream) {
+                                  int p_true, int parts, float eps, int norm_first, int dtype, void* stream) {
   using namespace b200;
   if (!y || !z || !w_f32 || !out || T < 0 || heads <= 0 || P <= 0 || p_true <= 0 || p_true > P || parts <= 0 ||
       (dtype != 0 && dtype != 1))
@@ -610,12 +626,13 @@ extern "C" int b200_ssm_gate_norm(const void* y, long long y_row_stride, const v
     return B200_ERR_SHAPE;
   if (T == 0) return B200_OK;
   SsmGateNormParams p{y, z, y_row_stride, z_row_stride, out_row_stride, (const float*)w_f32, out, heads, P, p_true,
-                      parts, eps};
+                      parts, eps, norm_first};
   const int n = heads * p_true / parts;
   auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   if (dtype == 0 && p_true == P && n % 8 == 0 && n <= 2048 && aligned(y) && aligned(z) && aligned(out) && aligned(w_f32)) {
     const long long pairs = T * parts;
-    launch_k(ssm_gate_norm_warp_kernel, dim3((unsigned)((pairs + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, p, pairs);
+    launch_k(norm_first ? ssm_gate_norm_warp_kernel<true> : ssm_gate_norm_warp_kernel<false>,
+             dim3((unsigned)((pairs + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, p, pairs);
     return launch_status();
   }
   const int threads = n <= 512 ? 64 : (n <= 2048 ? 128 : 256);

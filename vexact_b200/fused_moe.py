@@ -15,11 +15,14 @@ Pipeline (all on the caller's stream, scratch from torch's caching allocator):
 from __future__ import annotations
 
 import os
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
 
 from . import _lib
+from .batch_invariant_ops import gemm
+from .feed_forward import GLU_ACTS, GLUWeights, glu, glu_forward
 
 TILE_ROWS = 64  # largest token tile of the grouped GEMM (rows of one expert per tile)
 FUSED_SWIGLU_MAX_ROWS_PER_EXPERT = 64  # mean rows per expert up to which fc1 keeps its fused SwiGLU epilogue
@@ -61,6 +64,16 @@ def route_softmax_topk(router_logits: torch.Tensor, top_k: int, norm_topk_prob: 
 _PLAN_COUNTERS: dict = {}      # device index -> the 257 zeroed int32 counters of the routing-plan kernel
 
 
+def _plan_counters(dev) -> torch.Tensor:
+    counters = _PLAN_COUNTERS.get(dev.index)
+    if counters is None:
+        if torch.cuda.is_current_stream_capturing():
+            raise RuntimeError("make the first routing-plan call on a device outside graph capture")
+        counters = torch.zeros(257, device=dev, dtype=torch.int32)
+        _PLAN_COUNTERS[dev.index] = counters
+    return counters
+
+
 def route_plan_softmax_topk(router_logits: torch.Tensor, top_k: int, norm_topk_prob: bool, num_experts: int):
     """`route_softmax_topk` that also plans the expert permutation in the same launch.
 
@@ -77,12 +90,7 @@ def route_plan_softmax_topk(router_logits: torch.Tensor, top_k: int, norm_topk_p
     if x.dtype not in (torch.float32, torch.bfloat16):
         raise NotImplementedError(f"router logits dtype {x.dtype}")
     dev = x.device
-    counters = _PLAN_COUNTERS.get(dev.index)
-    if counters is None:
-        if torch.cuda.is_current_stream_capturing():
-            raise RuntimeError("make the first routing-plan call on a device outside graph capture")
-        counters = torch.zeros(257, device=dev, dtype=torch.int32)
-        _PLAN_COUNTERS[dev.index] = counters
+    counters = _plan_counters(dev)
     n = T * top_k
     max_tiles = max(1, max_token_tiles(n, num_experts))
     w = torch.empty((T, top_k), device=dev, dtype=torch.bfloat16)
@@ -378,6 +386,102 @@ def fused_moe_forward(
         addend = addend.to(torch.bfloat16).reshape(T, H).contiguous()
     pending = PendingMoE(y, plan["scatter_index"], addend, T, k, H, orig_shape)
     return pending if defer_reduce else pending.finish()
+
+
+# ------------------------------------------------------------------ mixtures of the hybrid decoders
+@dataclass
+class MixtureWeights:
+    """Sigmoid-scored experts whose score multiplies their input, and a gated shared expert."""
+
+    router: torch.Tensor             # [experts (+ 1: the shared expert's gate), width]
+    gate_up: torch.Tensor            # [experts, 2 * F, width], gate rows first
+    down: torch.Tensor               # [experts, width (padded), F]
+    experts: int
+    top: int
+    shared: Optional[GLUWeights] = None
+
+
+@dataclass
+class PendingMixture:
+    """Expert outputs in expert-sorted order plus the shared expert's rows; the sum over a token's `top` rows (found
+    through scatter_index [T * top]) and its shared row runs in the residual step that follows."""
+
+    rows: torch.Tensor
+    scatter_index: torch.Tensor
+    top: int
+    shared: Optional[torch.Tensor]
+
+
+def route_plan_sigmoid_topk(router_logits: torch.Tensor, top_k: int, num_experts: int, gate: bool, renorm: bool = False):
+    """Top-k by sigmoid scores with the expert permutation planned in the same launch (fp32 logits).
+
+    Returns (scores [T, k] fp32, experts [T, k] int64, gate [T] fp32 or None: the sigmoid of column `num_experts`, plan);
+    the order of rows inside an expert's group is that of arrival, on which no output depends."""
+    T, dev = router_logits.shape[0], router_logits.device
+    n = T * top_k
+    max_tiles = max(1, max_token_tiles(n, num_experts))
+    w = torch.empty((T, top_k), device=dev, dtype=torch.float32)
+    g = torch.empty(T, device=dev, dtype=torch.float32) if gate else None
+    idx = torch.empty((T, top_k), device=dev, dtype=torch.int64)
+    ints = torch.empty(n + num_experts + 2, device=dev, dtype=torch.int32)
+    rank, cu_seqlens, tile_count = ints[:n], ints[n:n + num_experts + 1], ints[n + num_experts + 1:]
+    tile_table = torch.empty((max_tiles, 4), device=dev, dtype=torch.int32)
+    _lib.check(
+        _lib.load().b200_moe_route_plan_sigmoid_topk(
+            router_logits.data_ptr(), router_logits.stride(0), w.data_ptr(), _lib.ptr(g), idx.data_ptr(), rank.data_ptr(),
+            _plan_counters(dev).data_ptr(), cu_seqlens.data_ptr(), tile_table.data_ptr(), tile_count.data_ptr(), T,
+            num_experts, top_k, int(renorm), TILE_ROWS, max_tiles, _lib.current_stream()),
+        "b200_moe_route_plan_sigmoid_topk",
+    )
+    return w, idx, g, dict(rank=rank, cu_seqlens=cu_seqlens, tile_table=tile_table, tile_count=tile_count,
+                           max_tiles=max_tiles)
+
+
+def _grouped_rows(x: torch.Tensor, w: torch.Tensor, plan: dict) -> torch.Tensor:
+    """Grouped product of expert-sorted rows in the rows' dtype."""
+    if x.dtype == torch.bfloat16:
+        return _grouped_gemm(x, w, None, plan, w.shape[1], mode=0)
+    out = torch.empty((x.shape[0], w.shape[1]), device=x.device, dtype=x.dtype)
+    _lib.check(
+        _lib.load().b200_moe_grouped_gemm_f32(x.data_ptr(), w.data_ptr(), out.data_ptr(), plan["tile_table"].data_ptr(),
+                                              plan["tile_count"].data_ptr(), x.shape[0], w.shape[0], w.shape[1],
+                                              x.shape[1], plan["max_tiles"], _lib.current_stream()),
+        "b200_moe_grouped_gemm_f32",
+    )
+    return out
+
+
+def mixture_forward(w: MixtureWeights, x: torch.Tensor) -> PendingMixture:
+    """sum over the top experts e of expert_e(s_e x), s = sigmoid(router x), plus sigmoid(gate x) * shared(x)."""
+    T, K = x.shape
+    n, E = T * w.top, w.experts
+    logits = gemm(x, w.router, out_dtype=torch.float32)      # exact products, fp32 sums
+    scores, idx, gate, plan = route_plan_sigmoid_topk(logits, w.top, E, w.shared is not None)
+    x_perm = torch.empty((n, K), device=x.device, dtype=x.dtype)
+    row_scale = torch.empty(n, device=x.device, dtype=torch.float32)
+    scatter_index = torch.empty(n, device=x.device, dtype=torch.int32)
+    size = x.element_size()
+    _lib.check(
+        _lib.load().b200_moe_scatter_ranked_f32(
+            x.data_ptr(), x.stride(0) * size, idx.data_ptr(), scores.data_ptr(), plan["rank"].data_ptr(),
+            plan["cu_seqlens"].data_ptr(), scatter_index.data_ptr(), x_perm.data_ptr(), row_scale.data_ptr(), T, w.top, E,
+            K * size, _lib.current_stream()),
+        "b200_moe_scatter_ranked_f32",
+    )
+    F = w.gate_up.shape[1] // 2
+    if x.dtype == torch.bfloat16 and n <= FUSED_SWIGLU_MAX_ROWS_PER_EXPERT * E:
+        h = torch.empty((n, F), device=x.device, dtype=x.dtype)
+        _lib.check(
+            _lib.load().b200_moe_grouped_gemm_glu(
+                x_perm.data_ptr(), w.gate_up.data_ptr(), row_scale.data_ptr(), None, h.data_ptr(),
+                plan["tile_table"].data_ptr(), plan["tile_count"].data_ptr(), n, E, F, K, h.stride(0), plan["max_tiles"],
+                TILE_ROWS, GLU_ACTS["silu"], _lib.current_stream()),
+            "b200_moe_grouped_gemm_glu",
+        )
+    else:
+        h = glu(_grouped_rows(x_perm, w.gate_up, plan), "silu", scale_in=row_scale)
+    shared = None if w.shared is None else glu_forward(w.shared, x, scale_out=gate)
+    return PendingMixture(_grouped_rows(h, w.down, plan), scatter_index, w.top, shared)
 
 
 class FusedMoeExpertFunction(torch.autograd.Function):

@@ -1,0 +1,241 @@
+"""Device weights of the hybrid decoders: checkpoint tensors as the kernels take them.
+
+Every reduction length and per-head width is padded to a multiple of 8 with zeros (TMA rows are 16-byte multiples);
+projections that read the same input are stacked into one matrix."""
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+from typing import Mapping, Optional, Union
+
+import torch
+
+from .delta import DeltaWeights
+from .fused_moe import MixtureWeights
+from .feed_forward import GLUWeights, MLPWeights
+from .hybrid_config import AttentionSpec, DeltaSpec, DenseSpec, HybridShape, LatentSpec, random_tensors, tensor_shapes
+from .hyper import Connection
+from .latent_attention import LatentWeights
+from .ssm import SSMWeights
+from .window_attention import AttentionWeights
+
+MixerWeights = Union[LatentWeights, AttentionWeights, SSMWeights, DeltaWeights]
+FFWeights = Union[MLPWeights, GLUWeights, MixtureWeights]
+
+
+def _up8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+def _pad_rows(t: torch.Tensor, blocks: int, rows: int) -> torch.Tensor:
+    """[blocks * r, ...] -> [blocks * rows, ...]: each block of r rows grows to `rows` with zeros."""
+    r = t.shape[0] // blocks
+    if r == rows:
+        return t
+    v = t.reshape(blocks, r, *t.shape[1:])
+    out = v.new_zeros((blocks, rows) + tuple(t.shape[1:]))
+    out[:, :r] = v
+    return out.reshape(blocks * rows, *t.shape[1:])
+
+
+def _pad_cols(t: torch.Tensor, blocks: int, cols: int) -> torch.Tensor:
+    return _pad_rows(t.t(), blocks, cols).t()
+
+
+@dataclass
+class HybridLayerWeights:
+    mixer: MixerWeights
+    mlp: Optional[FFWeights]
+    hc: list = field(default_factory=list)      # hyper-connections: Connection of the mixer (and of the feed-forward)
+    norms: list = field(default_factory=list)   # norms on both sides: (before, after) of each, fp32
+
+
+@dataclass
+class HybridWeights:
+    """Layers that share tensors share the objects; aligned models are stored as they come."""
+
+    shape: HybridShape
+    dtype: torch.dtype
+    embed: torch.Tensor
+    layers: list = field(default_factory=list)
+    final_norm: Optional[torch.Tensor] = None
+    head: Optional[torch.Tensor] = None
+    embed_norm: Optional[torch.Tensor] = None
+    loop_step: Optional[torch.Tensor] = None     # [times, width] fp32
+
+    @property
+    def xn_cols(self) -> int:
+        return _up8(self.shape.width)
+
+    @staticmethod
+    def from_tensors(shape: HybridShape, tensors: Mapping[str, torch.Tensor], dtype=torch.bfloat16,
+                     device="cuda") -> "HybridWeights":
+        for name, dims in tensor_shapes(shape).items():
+            if name not in tensors:
+                raise KeyError(f"missing tensor {name}")
+            if tuple(tensors[name].shape) != dims:
+                raise ValueError(f"tensor {name} is {tuple(tensors[name].shape)}, the configuration says {dims}")
+        b = _Builder(tensors, shape.width, dtype, device)
+        out = HybridWeights(shape, dtype, embed=b.mat(tensors["embed"]), final_norm=b.vec(tensors["final.norm"]),
+                            head=b.mat(_pad_cols(tensors["head"], 1, b.W8)))
+        if shape.sandwich:
+            out.embed_norm = b.vec(tensors["embed.norm"])
+            if shape.loop is not None:
+                out.loop_step = b.vec(tensors["loop.step"])
+        for i, layer in enumerate(shape.layers):
+            if layer.weights_of != i:
+                out.layers.append(out.layers[layer.weights_of])
+                continue
+            p, spec = f"l{i}.", layer.ff
+            lw = HybridLayerWeights(b.mixer(p + "mix.", layer.mixer), None if spec is None else b.ff(p + "mlp.", spec))
+            for q in ([1] if spec is None else [1, 2]):
+                if shape.sandwich:
+                    lw.norms.append((b.vec(tensors[f"{p}norm{q}"]), b.vec(tensors[f"{p}norm{q}b"])))
+                else:
+                    hc = f"{p}hc{q}."
+                    lw.hc.append(Connection(read=b.vec(tensors[hc + "in"]), mix=b.vec(tensors[hc + "mix"]),
+                                            write=b.vec(tensors[hc + "out"]), norm=b.vec(tensors[f"{p}norm{q}"])))
+            out.layers.append(lw)
+        return out
+
+    @staticmethod
+    def random_init(shape: HybridShape, seed: int = 0, dtype=torch.bfloat16, device="cuda") -> "HybridWeights":
+        return HybridWeights.from_tensors(shape, random_tensors(shape, seed, device), dtype, device)
+
+    def num_bytes(self) -> int:
+        seen, n = set(), 0
+
+        def walk(o):
+            nonlocal n
+            if isinstance(o, torch.Tensor):
+                if o.data_ptr() not in seen:
+                    seen.add(o.data_ptr())
+                    n += o.numel() * o.element_size()
+            elif isinstance(o, (list, tuple)):
+                for v in o:
+                    walk(v)
+            elif hasattr(o, "__dataclass_fields__") and not isinstance(o, HybridShape):
+                for v in vars(o).values():
+                    walk(v)
+
+        walk(self)
+        return n
+
+
+class _Builder:
+    def __init__(self, tensors, width, dtype, device):
+        self.tensors, self.width, self.W8, self.dtype, self.device = tensors, width, _up8(width), dtype, device
+
+    def mat(self, t):
+        return t.to(device=self.device, dtype=self.dtype).contiguous()
+
+    def vec(self, t):
+        return t.to(device=self.device, dtype=torch.float32).contiguous()
+
+    def in_proj(self, parts):
+        """Row blocks that read the layer's input, stacked; rows up to a multiple of 8."""
+        t = torch.cat(parts)
+        return self.mat(_pad_cols(_pad_rows(t, 1, _up8(t.shape[0])), 1, self.W8))
+
+    # ------------------------------------------------------------------ mixers
+    def mixer(self, p, m):
+        if isinstance(m, LatentSpec):
+            return self.latent(p, m)
+        if isinstance(m, AttentionSpec):
+            return self.attention(p, m)
+        return self.delta(p, m) if isinstance(m, DeltaSpec) else self.ssm(p, m)
+
+    def latent(self, p, m):
+        H, DN, DR, R, V = m.heads, _up8(m.dim), _up8(m.rot_dim), _up8(m.kv_rank), _up8(m.vdim)
+        get = lambda n: self.tensors[p + n]   # noqa: E731
+        q = get("q" if m.q_rank is None else "uq").view(H, m.dim + m.rot_dim, -1)
+        qn, qr = _pad_rows(q[:, :m.dim].reshape(H * m.dim, -1), H, DN), _pad_rows(q[:, m.dim:].reshape(H * m.rot_dim, -1), H, DR)
+        q = torch.cat([qn.view(H, DN, -1), qr.view(H, DR, -1)], 1).reshape(H * (DN + DR), -1)
+        dkv, query = get("dkv"), {}
+        head = q
+        if m.q_rank is not None:
+            Q = _up8(m.q_rank)
+            head = _pad_rows(get("dq"), 1, Q)
+            query = dict(w_uq=self.mat(_pad_cols(q, 1, Q)), q_norm=self.vec(_pad_rows(get("dq.norm"), 1, Q)),
+                         q_true=m.q_rank)
+        gate = [_pad_rows(get("g"), H, V)] if m.gated else []
+        uk = _pad_cols(_pad_rows(get("uk"), H, DN), 1, R).reshape(H, DN, R)
+        uv = _pad_cols(_pad_rows(get("uv"), H, V), 1, R).reshape(H, V, R)
+        i = torch.arange(0, m.rot_dims, 2, dtype=torch.float64)
+        return LatentWeights(w_in=self.in_proj([head, _pad_rows(dkv[:m.kv_rank], 1, R), _pad_rows(dkv[m.kv_rank:], 1, DR)] + gate),
+                             w_uk_t=self.mat(uk.transpose(1, 2)), w_uv=self.mat(uv),
+                             w_kv=self.mat(torch.cat([uk.reshape(H * DN, R), uv.reshape(H * V, R)])),
+                             w_out=self.mat(_pad_cols(get("o"), H, V)), c_norm=self.vec(_pad_rows(get("dkv.norm"), 1, R)),
+                             inv_freq=self.vec(m.rot_base ** (-i / max(m.rot_dims, 1))), heads=H, DN=DN, DR=DR, R=R,
+                             V=V, r_true=m.kv_rank, rot_dims=m.rot_dims, scale=m.scale, rot_half=m.rot_half,
+                             window=m.window, gated=m.gated, **query)
+
+    def attention(self, p, m):
+        H, G, DK, DV = m.heads, m.kv_heads, _up8(m.dim), _up8(m.vdim)
+        get = lambda n: self.tensors[p + n]   # noqa: E731
+        return AttentionWeights(w_in=self.in_proj([_pad_rows(get("q"), H, DK), _pad_rows(get("k"), G, DK),
+                                                   _pad_rows(get("v"), G, DV)]),
+                                w_out=self.mat(_pad_cols(get("o"), H, DV)), heads=H, kv_heads=G, DK=DK, DV=DV,
+                                scale=m.scale, window=m.window)
+
+    def ssm(self, p, m):
+        H, P, G, N = m.heads, _up8(m.vdim), m.groups, _up8(m.state)
+        inner, bc = m.heads * m.vdim, m.groups * m.state
+        get = lambda n: self.tensors[p + n]   # noqa: E731
+        z, x, B, C, dt = torch.split(get("in"), [inner, inner, bc, bc, H])
+
+        def channels(t):
+            a, b, c = torch.split(t, [inner, bc, bc])
+            return torch.cat([_pad_rows(a, H, P), _pad_rows(b, G, N), _pad_rows(c, G, N)])
+
+        return SSMWeights(w_in=self.in_proj([_pad_rows(z, H, P), _pad_rows(x, H, P), _pad_rows(B, G, N),
+                                             _pad_rows(C, G, N), dt]),
+                          w_out=self.mat(_pad_cols(get("o"), H, P)), conv_w=self.vec(channels(get("conv"))),
+                          conv_b=self.vec(channels(get("conv.b"))), dt_bias=self.vec(get("dt_bias")),
+                          A_log=self.vec(get("A_log")), D=self.vec(get("D")), norm=self.vec(_pad_rows(get("norm"), H, P)),
+                          heads=H, groups=G, P=P, N=N, vdim=m.vdim, parts=m.norm_groups)
+
+    def delta(self, p, m):
+        H, G, N, P = m.heads, m.kv_heads, _up8(m.dim), _up8(m.vdim)
+        get = lambda n: self.tensors[p + n]   # noqa: E731
+        wide = {"q": (G, N), "k": (G, N), "v": (H, P)}
+        conv = torch.cat([_pad_rows(get(n + ".conv"), *wide[n]) for n in "qkv"])
+        return DeltaWeights(w_in=self.in_proj([_pad_rows(get(n), *wide[n]) for n in "qkv"] + [_pad_rows(get("g"), H, P),
+                                                                                               get("a"), get("b")]),
+                            w_out=self.mat(_pad_cols(get("o"), H, P)), conv_w=self.vec(conv),
+                            conv_b=torch.zeros(conv.shape[0], device=self.device), dt_bias=self.vec(get("dt_bias")),
+                            A_log=self.vec(get("A_log")),
+                            norm=self.vec(_pad_rows(get("norm"), 1, P)).repeat(H), heads=H, groups=G, P=P, N=N,
+                            vdim=m.vdim, dim=m.dim)
+
+    # ------------------------------------------------------------------ feed-forwards
+    def ff(self, p, spec):
+        if isinstance(spec, DenseSpec):
+            return self.glu(p, spec.ff, "gelu_tanh") if spec.gated else self.mlp(p, spec.ff)
+        return self.mixture(p, spec)
+
+    def mlp(self, p, ff):
+        F8, get = _up8(ff), lambda n: self.tensors[p + n]
+        return MLPWeights(up=self.mat(_pad_cols(_pad_rows(get("up"), 1, F8), 1, self.W8)),
+                          up_b=self.mat(_pad_rows(get("up.b"), 1, F8)), down=self.mat(_pad_cols(get("down"), 1, F8)),
+                          down_b=self.mat(get("down.b")))
+
+    def _gate_up(self, p, ff):
+        F8 = _up8(ff)
+        return self.mat(_pad_cols(torch.cat([_pad_rows(self.tensors[p + n], 1, F8) for n in ("gate", "up")]), 1, self.W8))
+
+    def glu(self, p, ff, act):
+        return GLUWeights(gate_up=self._gate_up(p, ff), down=self.mat(_pad_cols(self.tensors[p + "down"], 1, _up8(ff))),
+                          act=act)
+
+    def mixture(self, p, spec):
+        rows = [self.tensors[p + "router"]]
+        shared = None
+        if spec.shared_ff is not None:
+            shared = self.glu(p + "shared.", spec.shared_ff, "silu")
+            rows.append(self.tensors[p + "shared.sg"])
+        # the output rows of an expert are padded like the layer's input, so that its rows are 16-byte multiples
+        down = [self.mat(_pad_rows(_pad_cols(self.tensors[f"{p}e{e}.down"], 1, _up8(spec.ff)), 1, self.W8))
+                for e in range(spec.experts)]
+        return MixtureWeights(router=self.mat(_pad_cols(torch.cat(rows), 1, self.W8)),
+                              gate_up=torch.stack([self._gate_up(f"{p}e{e}.", spec.ff) for e in range(spec.experts)]),
+                              down=torch.stack(down), experts=spec.experts, top=spec.top, shared=shared)

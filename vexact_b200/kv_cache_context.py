@@ -172,15 +172,16 @@ class StateSlotManager:
 
 
 class HybridCacheStore:
-    """Caches of a model that mixes latent-attention and state-space layers, one entry per layer that needs it.
+    """Caches of a model that mixes attention and recurrent layers, one entry per layer run that needs it.
 
     latent layer: `key_cache[layer]` [blocks, page, R + DR] (normed latent, rotated shared key part), paged like any KV
-    cache; `value_cache` is empty (the value is the latent itself).
-    state-space layer: `conv_state[layer]` [slots, taps - 1, channels] in the model dtype and `ssm_state[layer]`
+    cache; no entry in `value_cache` (the value is the latent itself).
+    attention layer: `key_cache[layer]` [blocks, page, kv_heads, DK] and `value_cache[layer]` [blocks, page, kv_heads, DV].
+    recurrent layer: `conv_state[layer]` [slots, taps - 1, channels] in the model dtype and `ssm_state[layer]`
     [slots, heads, N, P] fp32."""
 
     def __init__(self, latent_widths: dict, ssm_dims: dict, cache_config, num_slots: int, device,
-                 dtype=torch.bfloat16):
+                 dtype=torch.bfloat16, head_dims: Optional[dict] = None):
         self.cache_config = cache_config
         self.device = torch.device(device)
         self.page_size = cache_config.page_size
@@ -189,14 +190,17 @@ class HybridCacheStore:
         self.key_cache = {li: torch.zeros((self.max_blocks, self.page_size, w), device=self.device, dtype=dtype)
                           for li, w in latent_widths.items()}
         self.value_cache: dict[int, torch.Tensor] = {}
+        for li, (kv_heads, dk, dv) in (head_dims or {}).items():
+            for cache, d in ((self.key_cache, dk), (self.value_cache, dv)):
+                cache[li] = torch.zeros((self.max_blocks, self.page_size, kv_heads, d), device=self.device, dtype=dtype)
         self.conv_state, self.ssm_state = {}, {}
         for li, (channels, taps, heads, n, p) in ssm_dims.items():
             self.conv_state[li] = torch.zeros((num_slots, taps - 1, channels), device=self.device, dtype=dtype)
             self.ssm_state[li] = torch.zeros((num_slots, heads, n, p), device=self.device, dtype=torch.float32)
 
     def num_bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for d in (self.key_cache, self.conv_state, self.ssm_state)
-                   for t in d.values())
+        return sum(t.numel() * t.element_size() for d in (self.key_cache, self.value_cache, self.conv_state,
+                                                                 self.ssm_state) for t in d.values())
 
 
 class KVCacheStore:
@@ -249,9 +253,10 @@ def store_kvcache(key: torch.Tensor, value: torch.Tensor, k_cache: torch.Tensor,
     if slot_mapping.dtype != torch.int32:
         slot_mapping = slot_mapping.to(torch.int32)
     num_slots = k_cache.shape[0] * k_cache.shape[1]
+    w = key.element_size() // 2      # the kernel moves 2-byte elements; an fp32 row is twice as many
     _lib.check(
         _lib.load().b200_kv_store(key.data_ptr(), value.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
-                                  slot_mapping.data_ptr(), N, heads, k_dim, v_dim, key.stride(0), value.stride(0),
-                                  num_slots, _lib.current_stream()),
+                                  slot_mapping.data_ptr(), N, heads, k_dim * w, v_dim * w, key.stride(0) * w,
+                                  value.stride(0) * w, num_slots, _lib.current_stream()),
         "b200_kv_store",
     )

@@ -296,6 +296,7 @@ def _load_stage(cfg, folder, dtype, device):
 # config.json "architecture" (own designs) or "model_type" (HF checkpoints) -> loader(config, folder, dtype, device)
 MODEL_LOADERS = {
     "Nurazen": _load_hybrid,
+    "Dekerax": _load_hybrid,
     "qwen2": _load_stage,
     "qwen3": _load_stage,
     "qwen3_moe": _load_stage,

@@ -45,6 +45,14 @@ class SSMWeights:
     def taps(self) -> int:
         return self.conv_w.shape[1]
 
+    @property
+    def conv_off(self) -> int:
+        return self.inner
+
+    @property
+    def dt_off(self) -> int:
+        return self.inner + self.channels
+
     def state_dims(self):
         return self.channels, self.taps, self.heads, self.N, self.P
 
@@ -53,15 +61,16 @@ def _dt(dtype) -> int:
     return 0 if dtype == torch.bfloat16 else 1
 
 
-def ssm_conv(w: SSMWeights, proj: torch.Tensor, conv_state: torch.Tensor, step):
-    """(act [T, channels], dt [T, heads] fp32) of the in-projection rows; moves the convolution state on."""
+def short_conv(w, proj: torch.Tensor, conv_state: torch.Tensor, step):
+    """(act [T, channels], dt [T, heads] fp32) of the in-projection rows: causal convolution + silu of `channels` columns
+    from w.conv_off, softplus(. + dt_bias) of `heads` columns from w.dt_off; moves the convolution state on."""
     T = proj.shape[0]
     act = torch.empty((T, w.channels), device=proj.device, dtype=proj.dtype)
     dt = torch.empty((T, w.heads), device=proj.device, dtype=torch.float32)
     tiled = int(step.max_seqlen_q > SCAN_MAX_TOKENS)
     _lib.check(
         _lib.load().b200_ssm_conv(
-            proj.data_ptr(), proj.stride(0), w.inner, w.inner + w.channels, w.channels, w.heads, w.taps,
+            proj.data_ptr(), proj.stride(0), w.conv_off, w.dt_off, w.channels, w.heads, w.taps,
             w.conv_w.data_ptr(), w.conv_b.data_ptr(), w.dt_bias.data_ptr(), conv_state.data_ptr(), act.data_ptr(),
             dt.data_ptr(), step.query_start_loc.data_ptr(), step.context_lens.data_ptr(), step.state_slots.data_ptr(),
             step.state_slots.numel(), conv_state.shape[0], T, tiled, _dt(proj.dtype), _lib.current_stream()),
@@ -99,22 +108,29 @@ def ssm_chunk_scan(w: SSMWeights, act: torch.Tensor, dt: torch.Tensor, state: to
         "b200_ssm_chunk_scan")
 
 
-def ssm_gate_norm(w: SSMWeights, y: torch.Tensor, proj: torch.Tensor, eps: float) -> torch.Tensor:
-    """rms_norm_by_part(y * silu(z)) * norm; z is the first block of the in-projection rows."""
-    out = torch.empty((y.shape[0], w.inner), device=y.device, dtype=y.dtype)
+def head_gate_norm(y: torch.Tensor, z: torch.Tensor, norm: torch.Tensor, heads: int, P: int, vdim: int, parts: int,
+                   eps: float, norm_first: bool = False) -> torch.Tensor:
+    """rms_norm_by_part(y * silu(z)) * norm, or with norm_first rms_norm_by_part(y) * norm * silu(z); `parts` equal parts
+    of the heads * vdim true columns (heads are P wide)."""
+    out = torch.empty((y.shape[0], heads * P), device=y.device, dtype=y.dtype)
     _lib.check(
         _lib.load().b200_ssm_gate_norm(
-            y.data_ptr(), y.stride(0), proj.data_ptr(), proj.stride(0), w.norm.data_ptr(), out.data_ptr(),
-            out.stride(0), y.shape[0], w.heads, w.P, w.vdim, w.parts, float(eps), _dt(y.dtype),
+            y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), norm.data_ptr(), out.data_ptr(),
+            out.stride(0), y.shape[0], heads, P, vdim, parts, float(eps), int(norm_first), _dt(y.dtype),
             _lib.current_stream()),
         "b200_ssm_gate_norm")
     return out
 
 
+def ssm_gate_norm(w: SSMWeights, y: torch.Tensor, proj: torch.Tensor, eps: float) -> torch.Tensor:
+    """rms_norm_by_part(y * silu(z)) * norm; z is the first block of the in-projection rows."""
+    return head_gate_norm(y, proj[:, :w.inner], w.norm, w.heads, w.P, w.vdim, w.parts, eps)
+
+
 def ssm_mixer(w: SSMWeights, xn: torch.Tensor, conv_state: torch.Tensor, state: torch.Tensor, step,
               eps: float) -> torch.Tensor:
     proj = gemm(xn, w.w_in)
-    act, dt = ssm_conv(w, proj, conv_state, step)
+    act, dt = short_conv(w, proj, conv_state, step)
     y = torch.empty((xn.shape[0], w.inner), device=xn.device, dtype=xn.dtype)
     if step.max_seqlen_q <= SCAN_MAX_TOKENS or xn.dtype != torch.bfloat16 or w.N > CHUNK_MAX_STATE:
         ssm_scan(w, act, dt, state, y, step)
