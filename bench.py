@@ -77,6 +77,10 @@ def parse_args():
     ap.add_argument("--hybrid", action="store_true",
                     help="side measurement: prefill and decode steps of the hybrid decoder family (state-space + latent "
                          "attention) beside an MLA + dense model of equal size, and its kernels beside that model's")
+    ap.add_argument("--dekerax", action="store_true",
+                    help="side measurement: prefill and decode steps of the Dekerax decoders (gated delta rule, windowed "
+                         "attention and latent attention, mixtures) beside a grouped-query MoE model and the state-space "
+                         "hybrid of equal width, and its kernels beside theirs")
     ap.add_argument("--prefill-attention", type=int, default=0, metavar="QLEN",
                     help="side measurement: time one causal prefill attention call of QLEN queries on the "
                          "model's head shape (context --ctx if larger) and print its own JSON line")
@@ -775,7 +779,7 @@ def hybrid_model_case(args, shape, kind, S, new, total, page, device):
         model = HybridModel(HybridWeights.random_init(shape, device=device))
         runner, w = model.runner, model.runner.w
         runner.store = model.make_cache_store(CacheConfig(page, blocks), S, device)
-        for t in runner.store.key_cache.values():
+        for t in [*runner.store.key_cache.values(), *runner.store.value_cache.values()]:
             t.normal_()
         rows = (step.query_start_loc[1:] - 1).contiguous()
         if kind == "decode":
@@ -786,7 +790,10 @@ def hybrid_model_case(args, shape, kind, S, new, total, page, device):
                 step.__dict__.pop(k, None)
             return runner.logits(runner.forward(step, rows))
 
-        cache_bytes = sum(S * total * t.shape[-1] * 2 for t in runner.store.key_cache.values())
+        seen = {run: min(total, (getattr(w.layers[i].mixer, "window", None) or total) + new - 1)
+                for run, (i, _) in enumerate(shape.runs)}
+        cache_bytes = sum(S * seen[run] * t[0, 0].numel() * 2 for d in (runner.store.key_cache, runner.store.value_cache)
+                          for run, t in d.items())
         cache_bytes += 2 * sum(t.numel() * t.element_size() for d in (runner.store.conv_state, runner.store.ssm_state)
                                for t in d.values())
         vocab, width = shape.vocab, shape.width
@@ -962,6 +969,259 @@ def hybrid_kernels(args, page, device):
         del kc, vc, lat, kv
         torch.cuda.empty_cache()
 
+# --------------------------------------------------------------------------- Dekerax decoders
+DK_WINDOW, DK_PAGE = 1024, 64
+
+
+def dekerax_shapes():
+    """(Dekerax: 5 delta + 2 latent + 1 attention layers, the grouped-query MoE model, the state-space hybrid), equal
+    width, heads and expert sizes, 8 layers each."""
+    from vexact_b200.hybrid import AttentionSpec, DeltaSpec, DenseSpec, HybridLayer, HybridShape, LatentSpec, MixtureSpec
+    from vexact_b200.inferencer import ModelShape, MoEShape
+
+    W, V, E, TOP, FF = 2048, 32768, 64, 4, 1024
+    delta = DeltaSpec(heads=32, kv_heads=16, dim=128, vdim=128, conv=4)
+    lat = LatentSpec(heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=192 ** -0.5, rot_base=50000.0, rot_dims=64,
+                     q_rank=768, window=DK_WINDOW, gated=False, rot_half=True)
+    att = AttentionSpec(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, window=DK_WINDOW)
+    mix = MixtureSpec(E, TOP, FF, FF)
+    kinds = [delta, delta, lat, delta, delta, att, delta, lat]
+    layers = tuple(HybridLayer(m, DenseSpec(5504, gated=True) if i == 0 else mix, i) for i, m in enumerate(kinds))
+    return (HybridShape("dekerax-5delta-2latent-1attention", layers, W, V, 1, 1.0, 1e-6, "Dekerax"),
+            ModelShape("gqa-moe", 8, W, 16, 4, 128, V, moe=MoEShape(E, TOP, FF), qk_norm=False, rms_eps=1e-6),
+            hybrid_shapes()[0])
+
+
+def run_dekerax(args):
+    """Side measurement: steps of the Dekerax decoders beside the closest other models (random weights), then its kernels
+    beside the like kernels of those."""
+    from vexact_b200 import _lib
+
+    device = torch.device("cuda", 0)
+    torch.cuda.set_device(device)
+    cases = [("decode", 64, 1, 4096), ("decode", 256, 1, 1024), ("prefill", 4, 2048, 2048), ("prefill", 1, 2048, 8192)]
+    clocks = ClockSampler(0)
+    clocks.start()
+    clocks.wait_first_sample()
+    for shape in dekerax_shapes():
+        for kind, S, new, total in cases:
+            print(json.dumps(hybrid_model_case(args, shape, kind, S, new, total, DK_PAGE, device)), flush=True)
+            torch.cuda.empty_cache()
+    for line in dekerax_kernels(device):
+        print(json.dumps(line), flush=True)
+    print(json.dumps({"measurement": "dekerax", "clocks": clocks.stop(), "status": list(_lib.read_status())}))
+
+
+def dekerax_kernels(device):
+    """Per kernel of the Dekerax decoders and the like kernel of the other models: device time, achieved bytes or flops
+    over the measured peak.  Several buffers per kernel, together larger than L2."""
+    import vexact_b200 as vb
+    from vexact_b200 import delta as dl, fused_moe as fm, latent_attention as la, ssm, window_attention as wa
+    from vexact_b200.batch_invariant_ops import gemm
+    from vexact_b200.feed_forward import glu, glu_forward
+    from vexact_b200.hybrid import HybridShape, HybridWeights
+    from vexact_b200.hyper import hyper_step
+    from vexact_b200.residual import residual_step
+
+    peaks = measured_peaks()
+    hbm, tc = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    BF = torch.bfloat16
+    dek, _, hyb = dekerax_shapes()
+    kinds = dict(zip(("dense", "delta", "latent", "attention"), (0, 1, 2, 5)))
+    few = HybridShape("few", tuple(dek.layers[i].__class__(dek.layers[i].mixer, dek.layers[i].ff, n)
+                                   for n, i in enumerate(kinds.values())), dek.width, 1024, 1, 1.0, 1e-6, "Dekerax")
+    w = HybridWeights.random_init(few, device=device)
+    dw, lw, aw = (w.layers[n].mixer for n in (1, 2, 3))
+    mixw, densew = w.layers[1].mlp, w.layers[0].mlp
+    pair = HybridShape("pair", tuple(hyb.layers[i].__class__(hyb.layers[i].mixer, None, n) for n, i in enumerate((0, 2))),
+                       hyb.width, 1024, 4, 0.3, 1e-5)
+    hw = HybridWeights.random_init(pair, device=device)
+    sw, hc = hw.layers[0].mixer, hw.layers[0].hc[0]
+    W = dek.width
+    rn = lambda *s: torch.randn(s, device=device).to(BF)   # noqa: E731
+    norm = torch.ones(W, device=device)
+
+    def line(name, ms, nbytes=None, flops=None, like=None):
+        out = {"measurement": "dekerax_kernel", "kernel": name, "us": round(ms * 1e3, 2)}
+        fr = []
+        if nbytes:
+            out["gb_s"] = round(nbytes / ms / 1e6)
+            fr.append(nbytes / ms / 1e6 / hbm)
+        if flops:
+            out["tflop_s"] = round(flops / ms / 1e9, 1)
+            fr.append(flops / ms / 1e9 / tc)
+        out["of_measured_roofline"] = round(max(fr), 3)
+        if like:
+            out["like"] = like
+        return out
+
+    for T in (64, 8192):
+        k = 24 if T == 64 else 3
+        st, blocks = hybrid_step([(1, 100)] * T if T == 64 else [(T // 4, T // 4)] * 4, DK_PAGE, device)
+        S = st.state_slots.numel()
+        # boundaries of sublayers
+        sets = [(torch.randn(T, W, device=device), rn(T, W)) for _ in range(k)]
+        ms = graph_ms([lambda x=x, y=y: residual_step(x, y=y, post=norm, norm=norm, eps=1e-6) for x, y in sets])
+        yield line(f"residual_step T={T}", ms, T * W * 12)
+        nw = rn(W)
+        pairs = [(y, rn(T, W)) for _, y in sets]
+        ms = graph_ms([lambda x=x, r=r: vb.add_rms_norm(x, r, nw, 1e-6) for x, r in pairs])
+        yield line(f"add_rmsnorm T={T}", ms, T * W * 8, like=f"residual_step T={T}")
+        top, E = mixw.top, mixw.experts
+        scatter = torch.randperm(T * top, device=device).to(torch.int32)
+        pend = [(x, fm.PendingMixture(rn(T * top, W), scatter, top, y)) for x, y in sets]
+        ms = graph_ms([lambda x=x, y=y: residual_step(x, y=y, post=norm, norm=norm, eps=1e-6) for x, y in pend])
+        yield line(f"residual_step of a mixture T={T}", ms, T * W * (10 + 2 * (top + 1)))
+        ms = graph_ms([lambda y=y: fm.PendingMoE(y.rows, scatter, None, T, top, W, (T, W)).add_norm(y.shared, nw, 1e-6)
+                       for _, y in pend])
+        yield line(f"moe_unpermute_add_rmsnorm T={T}", ms, T * W * (6 + 2 * top), like=f"residual_step of a mixture T={T}")
+        del pend, pairs
+        # mixture: route + permute + two grouped products, without the sum (in the boundary)
+        xs = [y for _, y in sets]
+        rows = T * top
+        live = min(E, rows)
+        F = mixw.gate_up.shape[1] // 2
+        nbytes = 2 * (live * 3 * F * W + rows * (2 * W + 2 * F) + T * W)
+        flops = 6.0 * rows * F * W
+        lone = fm.MixtureWeights(mixw.router[:E].contiguous(), mixw.gate_up, mixw.down, E, top, None)
+        ms = graph_ms([lambda x=x: fm.mixture_forward(lone, x) for x in xs])
+        yield line(f"mixture (router to second product) T={T}", ms, nbytes, flops)
+
+        def moe(x):
+            rw, sel, plan = fm.route_plan_softmax_topk(vb.linear(x, lone.router), top, True, E)
+            return fm.fused_moe_forward(E, rw, sel, x, fc2_weight=mixw.down, fc1_1_2_weight=mixw.gate_up, defer_reduce=True,
+                                        plan=plan)
+
+        ms = graph_ms([lambda x=x: moe(x) for x in xs])
+        yield line(f"fused_moe (router to second product) T={T}", ms, nbytes, flops, like=f"mixture (router to second product) T={T}")
+        # the weights of several copies rotate at the small size, so that they come from HBM
+        copies = [densew] + [densew.__class__(densew.gate_up.clone(), densew.down.clone(), densew.act) for _ in range(3)]
+        gu, dn = densew.gate_up, densew.down
+        ms = graph_ms([lambda x=x, c=c: glu_forward(c, x) for x, c in zip(xs, copies * 6)])
+        yield line(f"gated feed-forward T={T}", ms, 2 * (gu.numel() + dn.numel() + 2 * T * W), 2.0 * T * (gu.numel() + dn.numel()))
+        ms = graph_ms([lambda x=x, c=c: gemm(gemm(x, c.gate_up)[:, :dn.shape[1]], c.down) for x, c in zip(xs, copies * 6)])
+        yield line(f"its two products alone, plain gemm T={T}", ms, 2 * (gu.numel() + dn.numel() + 2 * T * W),
+                   2.0 * T * (gu.numel() + dn.numel()), like=f"gated feed-forward T={T}")
+        del copies
+        if T > 64:
+            big = [rn(rows, 2 * F) for _ in range(2)]
+            scale = torch.rand(rows, device=device)
+            ms = graph_ms([lambda g=g: glu(g, "silu", scale_in=scale) for g in big])
+            yield line(f"glu rows={rows}", ms, rows * F * 6)
+            del big
+        # gated delta rule beside the state-space scan
+        proj = [rn(T, dw.w_in.shape[0]) for _ in range(k)]
+        conv = [torch.zeros(S, dw.taps - 1, dw.channels, device=device, dtype=BF) for _ in range(k)]
+        state_b = 4 * S * (dw.taps - 1) * dw.channels
+        ms = graph_ms([lambda p=p, c=c: ssm.short_conv(dw, p, c, st) for p, c in zip(proj, conv)])
+        yield line(f"short_conv (delta) T={T}", ms, T * (dw.channels * 4 + dw.heads * 6) + state_b)
+        act = [(rn(T, dw.channels), torch.rand(T, dw.heads, device=device) * 0.1, p[:, dw.dt_off + dw.heads:dw.dt_off + 2 * dw.heads],
+                torch.zeros(S, dw.heads, dw.N, dw.P, device=device), rn(T, dw.inner)) for p in proj]
+        scan_b = T * (dw.channels + dw.inner) * 2 + T * dw.heads * 6 + 8 * S * dw.heads * dw.N * dw.P
+        if T == 64:
+            ms = graph_ms([lambda a=a: dl.delta_scan(dw, *a, st) for a in act])
+            yield line("delta_scan (decode) S=64", ms, scan_b)
+        else:
+            flops = T * dw.heads * (2.0 * 64 * dw.N * 2 + 2.0 * 64 * dw.P * 2 + 6.0 * dw.N * dw.P)
+            for cols in (16, 32):
+                ms = graph_ms([lambda a=a: dl.delta_chunk_scan(dw, *a, st, 17, 4, cols) for a in act])
+                yield line(f"delta prep + chunk T={T} slice={cols}", ms, scan_b, flops)
+        z = [p[:, dw.channels:dw.channels + dw.inner] for p in proj]
+        ms = graph_ms([lambda a=a, z=z: ssm.head_gate_norm(a[4], z, dw.norm, dw.heads, dw.P, dw.vdim, dw.heads, 1e-6, True)
+                       for a, z in zip(act, z)])
+        yield line(f"norm then gate T={T}", ms, T * dw.inner * 6)
+        del proj, conv, act, z
+        torch.cuda.empty_cache()
+        proj = [rn(T, sw.w_in.shape[0]) for _ in range(k)]
+        conv = [torch.zeros(S, sw.taps - 1, sw.channels, device=device, dtype=BF) for _ in range(k)]
+        ms = graph_ms([lambda p=p, c=c: ssm.short_conv(sw, p, c, st) for p, c in zip(proj, conv)])
+        yield line(f"short_conv (state space) T={T}", ms, T * (sw.channels * 4 + sw.heads * 6) + 4 * S * (sw.taps - 1) * sw.channels,
+                   like=f"short_conv (delta) T={T}")
+        act = [(rn(T, sw.channels), torch.rand(T, sw.heads, device=device) * 0.1,
+                torch.zeros(S, sw.heads, sw.N, sw.P, device=device), rn(T, sw.inner)) for _ in range(k)]
+        scan_b = T * (sw.channels + sw.inner) * 2 + T * sw.heads * 4 + 8 * S * sw.heads * sw.N * sw.P
+        if T == 64:
+            ms = graph_ms([lambda a=a: ssm.ssm_scan(sw, *a, st) for a in act])
+            yield line("ssm_scan (decode) S=64", ms, scan_b, like="delta_scan (decode) S=64")
+        else:
+            ms = graph_ms([lambda a=a: ssm.ssm_chunk_scan(sw, *a, st, 17, 4, 32) for a in act])
+            flops = T * sw.heads * (2.0 * 64 * sw.N + 2.0 * 64 * sw.P + 4.0 * sw.N * sw.P)
+            yield line(f"ssm_chunk T={T}", ms, scan_b, flops, like=f"delta prep + chunk T={T}")
+        ms = graph_ms([lambda a=a, p=p: ssm.ssm_gate_norm(sw, a[3], p, 1e-5) for a, p in zip(act, proj)])
+        yield line(f"ssm_gate_norm T={T}", ms, T * sw.inner * 6, like=f"norm then gate T={T}")
+        del proj, act, conv
+        streams = [(torch.randn(T, 4, W, device=device), y) for y in xs]
+        ms = graph_ms([lambda s=s, y=y: hyper_step(s, done=hc, y=y, read=hc.read, norm=hc.norm, eps=1e-5) for s, y in streams])
+        yield line(f"hyper_step T={T}", ms, T * W * 36, like=f"residual_step T={T}")
+        del streams, sets, xs
+        torch.cuda.empty_cache()
+        # what lies between the projections and latent attention
+        cache = torch.zeros(blocks, DK_PAGE, lw.row_width, device=device, dtype=BF)
+        first, second = [rn(T, lw.w_in.shape[0]) for _ in range(k)], [rn(T, 16 * 192) for _ in range(k)]
+        qc = lw.q_cols
+        ms = graph_ms([lambda p=p: la.latent_prep(lw, cache, st, 1e-6, kv=p[:, qc:qc + lw.row_width], q_latent=p[:, :qc]) for p in first])
+        yield line(f"latent_prep (latents) T={T}", ms, T * (lw.row_width * 4 + qc * 4))
+        ms = graph_ms([lambda q=q: la.latent_prep(lw, cache, st, 1e-6, q=q) for q in second])
+        yield line(f"latent_prep (queries) T={T}", ms, T * 16 * 64 * 4)
+        del first, second, cache
+        torch.cuda.empty_cache()
+    # attention of decoded tokens: a window of 1024 out of 4096 keys, beside a context of 1024
+    for S, ctx in ((64, 4096), (256, 1024), (64, 1024)):
+        st, blocks = hybrid_step([(1, ctx)] * S, DK_PAGE, device)
+        n = min(ctx, DK_WINDOW)
+        sets = [(rn(S, aw.heads * aw.DK), rn(blocks, DK_PAGE, 4, 128), rn(blocks, DK_PAGE, 4, 128),
+                 torch.empty(S, aw.heads * aw.DV, device=device, dtype=BF)) for _ in range(2 if ctx * S > 200000 else 4)]
+        ms = graph_ms([lambda s=s: wa.attend_decode(aw, *s, st) for s in sets])
+        yield line(f"window_attn decode {S}x{ctx}", ms, S * n * 4 * 256 * 2)
+        if ctx == n:
+            ms = graph_ms([lambda s=s: vb.paged_attention(s[0].view(S, 16, 128), s[1], s[2], st.query_start_loc, st.context_lens,
+                                                          st.block_tables, 128 ** -0.5, 1) for s in sets])
+            yield line(f"paged_attn 128/128 decode {S}x{ctx}", ms, S * n * 4 * 256 * 2, like=f"window_attn decode {S}x{ctx}")
+        del sets
+        torch.cuda.empty_cache()
+        sets = [(rn(S, 16, lw.row_width), rn(blocks, DK_PAGE, lw.row_width), torch.empty(S, 16, lw.R, device=device, dtype=BF))
+                for _ in range(4)]
+        ms = graph_ms([lambda s=s: la.latent_attn_tc(lw, *s, st) for s in sets])
+        yield line(f"latent_tc window {S}x{ctx}", ms, S * n * lw.row_width * 2)
+        del sets
+        torch.cuda.empty_cache()
+    open_lw = lw.__class__(**{**vars(lw), "window": None})
+    st, blocks = hybrid_step([(1, 1024)] * 64, DK_PAGE, device)
+    sets = [(rn(64, 16, lw.row_width), rn(blocks, DK_PAGE, lw.row_width), torch.empty(64, 16, lw.R, device=device, dtype=BF))
+            for _ in range(4)]
+    ms = graph_ms([lambda s=s: la.latent_attn_tc(open_lw, *s, st) for s in sets])
+    yield line("latent_tc without a window 64x1024", ms, 64 * 1024 * lw.row_width * 2, like="latent_tc window 64x4096")
+    del sets
+    # attention of prompts
+    for S, new, total in ((4, 2048, 2048), (1, 2048, 8192)):
+        st, blocks = hybrid_step([(new, total)] * S, DK_PAGE, device)
+        T = S * new
+        q, kc, vc = rn(T, 16 * 128), rn(blocks, DK_PAGE, 4, 128), rn(blocks, DK_PAGE, 4, 128)
+        out, longs = torch.empty(T, 16 * 128, device=device, dtype=BF), wa._long_sequences(st, device)[0]
+        pairs = lambda win: S * sum(min(t + 1, win) for t in range(total - new, total))   # noqa: E731
+        wide = wa.AttentionWeights(**{**vars(aw), "window": None})
+        for form, tag in ((0, "window_attn prefill"), (1, "window_attn prefill, mma.sync")):
+            ms = graph_ms([lambda: wa.attend_prefill(aw, q, kc, vc, out, st, longs, form)])
+            yield line(f"{tag} {S}x{new}/{total}", ms, None, 2.0 * pairs(DK_WINDOW) * 16 * 256)
+            ms = graph_ms([lambda: wa.attend_prefill(wide, q, kc, vc, out, st, longs, form)])
+            yield line(f"{tag} without a window {S}x{new}/{total}", ms, None, 2.0 * pairs(1 << 30) * 16 * 256)
+        ms = graph_ms([lambda: vb.paged_attention(q.view(T, 16, 128), kc, vc, st.query_start_loc, st.context_lens, st.block_tables,
+                                                  128 ** -0.5, new)])
+        yield line(f"paged_attn 128/128 prefill {S}x{new}/{total}", ms, None, 2.0 * pairs(1 << 30) * 16 * 256,
+                   like=f"window_attn prefill {S}x{new}/{total}")
+        q, cache, heads = rn(T, 16, 192), rn(blocks, DK_PAGE, lw.row_width), torch.empty(T, 16, 128, device=device, dtype=BF)
+        plan = la._split_plan(st, lw.window, device)[1]
+        ms = graph_ms([lambda: la.latent_expanded(lw, q, None, cache, heads, st, plan)])
+        yield line(f"latent gather + up-projection + windowed attention {S}x{new}/{total}", ms, None,
+                   2.0 * pairs(DK_WINDOW) * 16 * 320 + 2.0 * plan[4] * lw.w_kv.numel())
+        plan = la._split_plan(st, None, device)[1]
+        ms = graph_ms([lambda: la.latent_expanded(open_lw, q, None, cache, heads, st, plan)])
+        yield line(f"the same without a window {S}x{new}/{total}", ms, None,
+                   2.0 * pairs(1 << 30) * 16 * 320 + 2.0 * plan[4] * lw.w_kv.numel(),
+                   like=f"latent gather + up-projection + windowed attention {S}x{new}/{total}")
+        del q, kc, vc, cache, heads
+        torch.cuda.empty_cache()
+
 
 def main():
     args = parse_args()
@@ -979,6 +1239,9 @@ def main():
         return
     if args.hybrid:
         run_hybrid(args)
+        return
+    if args.dekerax:
+        run_dekerax(args)
         return
     if args.skew:
         run_skew(args, shape)

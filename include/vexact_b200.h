@@ -484,7 +484,8 @@ int b200_latent_gather(const void* cache, void* dst, const void* seq_ids_i32, co
 /* Grouped-query attention over paged per-head keys and values [blocks, page, kv_heads, DK | DV], no positions in the
  * scores, inside a window (0: none), fp32 weights.  _decode: bf16, tensor cores, sequences with min_len .. max_len new
  * tokens (most_new: the most any brings); DK, DV <= 256, page_size a multiple of 8 that divides 32 or is a multiple of it.
- * _prefill: bf16, tensor cores, the n sequences named.  _simt: any dims, both dtypes.  q and out rows hold the heads. */
+ * _prefill: bf16, tensor cores, the n sequences named, which are all those with at least min_len new tokens; form 0, or 1
+ * to keep off the tcgen05 kernel.  _simt: any dims, both dtypes.  q and out rows hold the heads. */
 int b200_window_attn_decode(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void*
                             out, long long out_row_stride, const void* query_start_loc, const void* context_lens,
                             const void* page_table, long long page_table_stride, int max_pages, int page_size, int
@@ -493,8 +494,9 @@ int b200_window_attn_decode(const void* q, long long q_row_stride, const void* k
 int b200_window_attn_prefill(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void*
                              out, long long out_row_stride, const void* query_start_loc, const void* context_lens,
                              const void* page_table, long long page_table_stride, int max_pages, int page_size, int
-                             num_blocks, int num_seqs, const void* seq_ids_i32, int n, int max_len, int window, int
-                             heads, int kv_heads, int DK, int DV, float scale, void* stream);
+                             num_blocks, int num_seqs, const void* seq_ids_i32, int n, int max_len, int min_len, int
+                             window, long long T, int heads, int kv_heads, int DK, int DV, float scale, int form,
+                             void* stream);
 int b200_window_attn_simt(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void* out,
                           const void* query_start_loc, const void* context_lens, const void* page_table, long long
                           page_table_stride, int max_pages, int page_size, int num_blocks, int num_seqs, int min_len,

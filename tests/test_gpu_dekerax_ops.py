@@ -157,9 +157,9 @@ def _attention_reference(w, q, k, v, new):
 def _attend(form, w, q, kc, vc, out, st, *lens):
     from vexact_b200 import window_attention as wa
 
-    if form == "prefill":
+    if form.startswith("prefill"):
         longs, _ = wa._long_sequences(st, DEV)
-        wa.attend_prefill(w, q, kc, vc, out, st, longs)
+        wa.attend_prefill(w, q, kc, vc, out, st, longs, int(form == "prefill_mma"))
     else:
         (wa.attend_simt if form == "simt" else wa.attend_decode)(w, q, kc, vc, out, st, *lens)
 
@@ -184,12 +184,14 @@ LONG = [(17, 17), (1, 33), (130, 130), (64, 331), (100, 165), (18, 500), (300, 4
     ("decode", BF, 6, 2, 40, 24, 16), ("decode", BF, 12, 1, 72, 128, 64), ("decode", BF, 3, 3, 192, 96, 32),
     ("decode", BF, 8, 4, 200, 256, 8), ("decode", BF, 5, 1, 64, 64, 128),
     ("prefill", BF, 6, 2, 40, 24, 16), ("prefill", BF, 4, 1, 72, 128, 64), ("prefill", BF, 2, 2, 192, 96, 8),
-    ("prefill", BF, 2, 1, 200, 256, 32), ("prefill", BF, 4, 4, 128, 80, 64)])
+    ("prefill", BF, 2, 1, 200, 256, 32), ("prefill", BF, 4, 4, 128, 80, 64), ("prefill", BF, 16, 1, 64, 72, 32),
+    ("prefill", BF, 5, 1, 104, 40, 16), ("prefill", BF, 3, 1, 128, 128, 8), ("prefill", BF, 12, 1, 96, 96, 128),
+    ("prefill_mma", BF, 4, 4, 128, 80, 64), ("prefill_mma", BF, 3, 1, 72, 128, 16)])
 def test_windowed_attention(form, dtype, H, G, DK, DV, page, window):
     """Decoded tokens, portions and prompts beside each other; the last token's first head points at one key: just inside
     the window, just outside it, the first of a page, the first of all, itself."""
     w = _attention_weights(H, G, DK, DV, window)
-    lens = LONG if form == "prefill" else SHORT
+    lens = LONG if form.startswith("prefill") else SHORT
     st = hu.step(lens, page=page, seed=H)
     T = sum(n for n, _ in lens)
     q = _rand(T, H * DK + 16, seed=1, dtype=dtype)
@@ -211,7 +213,7 @@ def test_windowed_attention(form, dtype, H, G, DK, DV, page, window):
         at = 0
         for i, (n, total) in enumerate(lens):
             got = out[at:at + n].double().cpu().view(n, H, DV)
-            if form != "prefill" or n > 16:
+            if not form.startswith("prefill") or n > 16:
                 want = _attention_reference(w, q[at:at + n, :H * DK].double().view(n, H, DK), ks[i].double(), vs[i].double(), n)
                 tol = 1e-5 if dtype == F32 else 2 ** -7
                 assert ((got - want).abs() <= tol * want.abs() + tol * 0.5).all(), (n, total, (got - want).abs().max())
@@ -220,43 +222,45 @@ def test_windowed_attention(form, dtype, H, G, DK, DV, page, window):
             at += n
 
 
-@pytest.mark.parametrize("form", ["simt", "decode", "prefill"])
-def test_windowed_attention_of_a_batch_equals_each_alone(form):
-    w = _attention_weights(6, 2, 40, 24, 50)
-    lens = [(20, 20), (40, 300), (17, 90)] if form == "prefill" else [(1, 700), (2, 300), (1, 5), (9, 60)]
+@pytest.mark.parametrize("DK,DV", [(40, 24), (88, 72)])
+@pytest.mark.parametrize("form", ["simt", "decode", "prefill", "prefill_mma"])
+def test_windowed_attention_of_a_batch_equals_each_alone(form, DK, DV):
+    w = _attention_weights(6, 2, DK, DV, 50)
+    lens = [(20, 20), (40, 300), (17, 90)] if form.startswith("prefill") else [(1, 700), (2, 300), (1, 5), (9, 60)]
     st = hu.step(lens, page=16)
     T = sum(n for n, _ in lens)
-    q = _rand(T, 240, seed=1, dtype=BF).cuda()
-    kc, vc = (_rand(st.num_blocks, 16, 2, d, seed=d, dtype=BF).cuda() for d in (40, 24))
-    out = torch.empty(T, 144, dtype=BF, device=DEV)
+    q = _rand(T, 6 * DK, seed=1, dtype=BF).cuda()
+    kc, vc = (_rand(st.num_blocks, 16, 2, d, seed=d, dtype=BF).cuda() for d in (DK, DV))
+    out = torch.empty(T, 6 * DV, dtype=BF, device=DEV)
     _attend(form, w, q, kc, vc, out, st)
     at = 0
     for i, (n, total) in enumerate(lens):
         one = hu.step([(n, total)], page=16)
         one.block_tables = st.block_tables[i:i + 1].contiguous()
-        alone = torch.empty(n, 144, dtype=BF, device=DEV)
+        alone = torch.empty(n, 6 * DV, dtype=BF, device=DEV)
         _attend(form, w, q[at:at + n].contiguous(), kc, vc, alone, one)
         assert torch.equal(alone, out[at:at + n])
         at += n
 
 
+@pytest.mark.parametrize("D", [8, 72])
 @pytest.mark.parametrize("form", ["simt", "decode", "prefill"])
-def test_attention_weights_are_not_rounded_to_sixteen_bits(form):
+def test_attention_weights_are_not_rounded_to_sixteen_bits(form, D):
     """Values that cancel under nearly equal weights: weights rounded to bf16 would miss the small result by 10 %."""
     n, new = 400, 20 if form == "prefill" else 1
-    w = _attention_weights(1, 1, 8, 8, None, 1.0)
+    w = _attention_weights(1, 1, D, D, None, 1.0)
     st = hu.step([(new, n)], page=16)
-    k, v = torch.zeros(n, 1, 8), torch.zeros(n, 1, 8)
+    k, v = torch.zeros(n, 1, D), torch.zeros(n, 1, D)
     v[:, 0, 3] = torch.tensor([1.0, -1.0]).repeat(n // 2)
     k[:, 0, 0] = torch.linspace(0, -0.9, n).to(BF).float()
-    q = torch.zeros(new, 1, 8)
+    q = torch.zeros(new, 1, D)
     q[:, 0, 0] = 1.0
     want = _attention_reference(w, q.double(), k.double(), v.double(), new)[-1, 0, 3].item()
     assert 1e-4 < want < 1e-2
-    kc, vc = torch.zeros(st.num_blocks * 16, 1, 8), torch.zeros(st.num_blocks * 16, 1, 8)
+    kc, vc = torch.zeros(st.num_blocks * 16, 1, D), torch.zeros(st.num_blocks * 16, 1, D)
     kc[st.rows(0)], vc[st.rows(0)] = k, v
-    out = torch.empty(new, 8, dtype=BF, device=DEV)
-    _attend(form, w, q.view(new, 8).to(BF).cuda(), kc.to(BF).view(-1, 16, 1, 8).cuda(), vc.to(BF).view(-1, 16, 1, 8).cuda(), out, st)
+    out = torch.empty(new, D, dtype=BF, device=DEV)
+    _attend(form, w, q.view(new, D).to(BF).cuda(), kc.to(BF).view(-1, 16, 1, D).cuda(), vc.to(BF).view(-1, 16, 1, D).cuda(), out, st)
     assert abs(out[-1, 3].item() - want) < 0.01 * abs(want)
 
 

@@ -35,7 +35,7 @@ SIGNATURES = {
     "b200_latent_attn_simt": [P, P, P, P, P, P, LL, I, I, I, I, I, I, I, LL, I, I, I, F, I, P],
     "b200_window_attn_simt": [P, LL, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, LL, I, I, I, I, F, I, P],
     "b200_window_attn_decode": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, I, I, I, I, I, I, I, I, F, P],
-    "b200_window_attn_prefill": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, P, I, I, I, I, I, I, I, F, P],
+    "b200_window_attn_prefill": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, P, I, I, I, I, LL, I, I, I, I, F, I, P],
     "b200_gemm_glu": [P, P, P, P, LL, I, I, LL, LL, I, P],
     "b200_glu": [P, LL, P, P, P, LL, I, I, I, P],
     "b200_moe_grouped_gemm_glu": [P, P, P, P, P, P, P, LL, I, I, I, LL, I, I, I, P],

@@ -63,6 +63,9 @@ struct AttnParams {
   int max_seqlen_q;      // the caller's bound on queries per sequence: it sized the tile grid
   int q_tma;             // rows-on-lanes kernel: the query tile comes by TMA (a 3-D box over [token, head, dim])
   int o_tma;             // rows-on-lanes kernel: a warp's 32 output rows leave by one asynchronous TMA store
+  int min_q;             // tcgen05 kernels: sequences with fewer queries are skipped (another kernel's)
+  int window;            // rows-on-lanes kernel, exact form: keys a query sees, its own included (0: every earlier one)
+  int dv;                // rows-on-lanes kernel, exact form: value columns of a head (at most 128)
   int scalar_out;        // development knob B200_ATTN_OUT_SCALAR=1: 2-byte output stores in the keys-on-lanes kernel
 };
 

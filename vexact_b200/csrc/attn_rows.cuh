@@ -21,6 +21,11 @@
 // block and l = (l_0 + l_1) + (l_2 + l_3) at the end, O folded block by block as o = (o + O_prev) * alpha.
 // A token therefore gets the same bits from a decode step, a chunk and a full prefill.
 //
+// Exact form (EXACT): the weights are not rounded.  P enters its product as a bf16 pair hi + lo in two tiles (two chains of
+// UMMAs into the same O), the row sum adds the fp32 weights, a query may be limited to a window of keys (blocks before it
+// are not walked), and heads may be narrower than 128 columns (the rest arrives as zeros and is not stored).  The second
+// P tile takes the place of the second Q buffer.
+//
 // Warps (12): 0 K producer, 1 UMMA issuer + TMEM owner, 2 V producer, 3 Q loader, 4-11 compute: a row is
 // shared by two threads (warps w and w + 4 of a lane quadrant), each taking 64 of the block's 128 keys for
 // the softmax and 64 of the 128 value dims for o, the fold and the final store.
@@ -78,7 +83,7 @@ __device__ __forceinline__ float butterfly_order_sum32(const float (&p)[32]) {
   return (c[0] + c[2]) + (c[1] + c[3]);
 }
 
-template <int DK>
+template <int DK, bool EXACT>
 __global__ void __launch_bounds__(ATR_THREADS, 1)
 paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                        const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_out,
@@ -87,8 +92,13 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   constexpr int KH = DK / 64, VH = DV / 64;
   constexpr int K_BYTES = ATC_BN * DK * 2, V_BYTES = ATC_BN * DV * 2;
   constexpr int KV_BYTES = KST * K_BYTES + VST * V_BYTES;
-  constexpr int Q_BYTES = KH * NC * 128;   // KH halves of [128 rows][128 B]; two such buffers
-  constexpr int P_BYTES = 2 * NC * 128;    // two 64-key halves of [128 rows][128 B]
+  constexpr int Q_BYTES = KH * NC * 128;   // KH halves of [128 rows][128 B]; QBUFS such buffers
+  constexpr int QBUFS = EXACT ? 1 : 2;
+  constexpr int P_TILE = 2 * NC * 128;     // two 64-key halves of [128 rows][128 B]
+  constexpr int P_BYTES = EXACT ? 2 * P_TILE : P_TILE;   // hi, lo
+  // Q buffer of a tile, and the parity of its use
+  auto q_buf = [](uint32_t it) { return EXACT ? 0u : it & 1u; };
+  auto q_par = [](uint32_t it) { return EXACT ? it & 1u : (it >> 1) & 1u; };
   constexpr int TMEM_COLS = 512;           // S0, S1 (128 each), O (128)
 
   // All shared memory is dynamic (the tiles take 224 of the 227 KB): the 1024-byte aligned tiles first,
@@ -99,14 +109,14 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   uint8_t* base_ptr = smem_raw + (base - raw);
   const uint32_t v_ring = base + KST * K_BYTES;
   const uint32_t q_smem = base + KV_BYTES;
-  const uint32_t p_smem = q_smem + 2 * Q_BYTES;
+  const uint32_t p_smem = q_smem + QBUFS * Q_BYTES;
   uint8_t* q_ptr = base_ptr + KV_BYTES;
-  uint8_t* p_ptr = q_ptr + 2 * Q_BYTES;
+  uint8_t* p_ptr = q_ptr + QBUFS * Q_BYTES;
   uint8_t* small = p_ptr + P_BYTES;
   {
     uint32_t granted;
     asm volatile("mov.u32 %0, %%dynamic_smem_size;" : "=r"(granted));
-    if ((base - raw) + KV_BYTES + 2 * Q_BYTES + P_BYTES + 256 + 4 * NC * 4 + 16 > granted) {
+    if ((base - raw) + KV_BYTES + QBUFS * Q_BYTES + P_BYTES + 256 + 4 * NC * 4 + 16 > granted) {
       // the aligned layout does not fit what the launch granted (only possible if something else put
       // static shared memory in front of the dynamic region): every thread leaves before any set-up
       if (threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, -(int)(base - raw));
@@ -190,7 +200,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       const int* ptab = p.page_table + (long long)t.seq * p.page_table_stride;
       const int valid_pages = (t.kv_len + p.page_size - 1) / p.page_size;
       auto page_of = [&](int j, int b, int& in_page) {
-        const int tok = j * ATC_BN + b * p.box_tokens;
+        const int tok = (EXACT ? t.blk0 + j : j) * ATC_BN + b * p.box_tokens;
         const int lpage = tok / p.page_size;
         in_page = tok - lpage * p.page_size;
         int phys = -1;
@@ -235,8 +245,8 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       uint32_t gs = 0, gp = 0, tile_it = 0;             // next QK^T block, next PV block, tile counter
       int j = 0;
       auto issue_next_s = [&]() {   // S of global block gs into S buffer gs & 1
-        const int qb = tile_it & 1;
-        if (j == 0 && !ptx::mbar_wait(qfull_bar(qb), (tile_it >> 1) & 1, abort_flag, 705 + qb)) return false;
+        const int qb = q_buf(tile_it);
+        if (j == 0 && !ptx::mbar_wait(qfull_bar(qb), q_par(tile_it), abort_flag, 705 + qb)) return false;
         const int s = gs % KST, b = gs & 1;
         if (!ptx::mbar_wait(kfull_bar(s), (gs / KST) & 1, abort_flag, 710 + s)) return false;
         if (!ptx::mbar_wait(sfree_bar(b), ((gs >> 1) & 1) ^ 1, abort_flag, 720 + b)) return false;
@@ -280,6 +290,12 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
           const uint64_t db = umma_desc_mn_sw128(sv + kk * 16 * 128, ATC_BN * 128);
           ptx::umma_bf16(tm_o, da, db, idesc_o, kk != 0 ? 1u : 0u);
         }
+        if constexpr (EXACT) {
+#pragma unroll
+          for (int kk = 0; kk < ATC_BN / 16; ++kk)
+            ptx::umma_bf16(tm_o, kdesc(p_smem + P_TILE + (kk >> 2) * (NC * 128) + (kk & 3) * 32),
+                           umma_desc_mn_sw128(sv + kk * 16 * 128, ATC_BN * 128), idesc_o, 1u);
+        }
         ptx::umma_commit(ofull_bar);
         ptx::umma_commit(vempty_bar(s));
         ATR_STAMP(0, g, 4);    // PV issued
@@ -292,9 +308,9 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
     uint32_t tile_it = 0;
     for (int lin = atc_next_tile<NC>(p, blockIdx.x, t); lin >= 0;
          lin = atc_next_tile<NC>(p, lin + (int)gridDim.x, t), ++tile_it) {
-      const int qb = tile_it & 1;
+      const int qb = q_buf(tile_it);
       bool w = true;
-      if (lane == 0) w = ptx::mbar_wait(qfree_bar(qb), ((tile_it >> 1) & 1) ^ 1, abort_flag, 760 + qb);
+      if (lane == 0) w = ptx::mbar_wait(qfree_bar(qb), q_par(tile_it) ^ 1, abort_flag, 760 + qb);
       if (!__all_sync(0xffffffffu, w)) break;
       uint8_t* qd = q_ptr + qb * Q_BYTES;
       if (p.q_tma) {
@@ -368,6 +384,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       const int npos = min(t.pos_per_tile, t.q_len - t.tile_pos0);
       const int pi = row / t.heads_here, hd = row - pi * t.heads_here;
       const int cpos = t.q_abs0 + t.tile_pos0 + (pi < npos ? pi : 0);   // padding rows borrow position 0's mask
+      const uint32_t reach = p.window > 0 ? (uint32_t)p.window : 0x80000000u;   // exact form: 0 <= cpos - key < reach
       float m_run = -INFINITY, l_a = 0.f, l_b = 0.f;   // l of my two key groups (2 half, 2 half + 1)
       float o[64];
 #pragma unroll
@@ -375,8 +392,9 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       for (int j = 0; j < t.nblk; ++j) {
         const uint32_t g = g0 + j;
         const int b = g & 1, s = g % VST;
-        const int key0 = j * ATC_BN + half * 64;          // first key of my half of the block
-        const bool masked = key0 + 63 > cpos;
+        const int blk = EXACT ? t.blk0 + j : j;
+        const int key0 = blk * ATC_BN + half * 64;        // first key of my half of the block
+        const bool masked = key0 + 63 > cpos || (EXACT && (uint32_t)(cpos - key0) >= reach);
         if (!ptx::mbar_wait_warp(sfull_bar(b), (g >> 1) & 1, abort_flag, 740 + b)) {
           alive = false;
           break;
@@ -403,7 +421,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         if (masked) {
 #pragma unroll
           for (int i = 0; i < 64; ++i)
-            if (key0 + i > cpos) v[i] = -INFINITY;
+            if (EXACT ? (uint32_t)(cpos - key0 - i) >= reach : key0 + i > cpos) v[i] = -INFINITY;
         }
         float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -444,7 +462,26 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         if (warp == 4) ATR_STAMP(1, g, 2);   // folded
         // p = bf16(2^(v - m)), group sums in butterfly order, P half row -> shared memory
         float sa, sb;
-        {
+        if constexpr (EXACT) {
+          float s4[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+          for (int q = 0; q < 8; ++q) {      // eight keys: sixteen bytes of either tile
+            uint32_t hi[4], lo[4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+              const float a = fast_exp2(v[q * 8 + 2 * k] - m_new), c = fast_exp2(v[q * 8 + 2 * k + 1] - m_new);
+              s4[k] += a + c;
+              hi[k] = pack_bf2(a, c);
+              float ha, hc;
+              unpack_bf2(hi[k], ha, hc);
+              lo[k] = pack_bf2(a - ha, c - hc);
+            }
+            *reinterpret_cast<uint4*>(p_half + sw128(row, q)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+            *reinterpret_cast<uint4*>(p_half + P_TILE + sw128(row, q)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          }
+          sa = (s4[0] + s4[1]) + (s4[2] + s4[3]);
+          sb = 0.f;
+        } else {
           float pf[32];
           uint32_t pk[16];
 #pragma unroll
@@ -474,13 +511,13 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         l_a = l_a * alpha + sa;
         l_b = l_b * alpha + sb;
         // keys at or beyond kv_len may hold anything: clear their V rows so that 0 * V stays 0
-        if (j * ATC_BN + ATC_BN > t.kv_len) {
+        if (blk * ATC_BN + ATC_BN > t.kv_len) {
           if (!ptx::mbar_wait_warp(vfull_bar(s), (g / VST) & 1, abort_flag, 745)) {
             alive = false;
             break;
           }
           uint8_t* vt = base_ptr + (size_t)KST * K_BYTES + (size_t)s * V_BYTES;
-          for (int r = t.kv_len - j * ATC_BN + (warp - 4); r < ATC_BN; r += 8)
+          for (int r = t.kv_len - blk * ATC_BN + (warp - 4); r < ATC_BN; r += 8)
 #pragma unroll
             for (int h = 0; h < VH; ++h) reinterpret_cast<uint32_t*>(vt + h * (ATC_BN * 128) + r * 128)[lane] = 0u;
         }
@@ -538,7 +575,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
             // every row of the warp is a real query: one asynchronous store of the warp's box
             ptx::fence_proxy_async_smem();
             __syncwarp();
-            if (lane == 0) {
+            if (lane == 0 && (!EXACT || half * 64 < p.dv)) {
               ptx::tma_store_3d(&tm_out, ptx::smem_u32(p_half + q4 * 32 * 128), half * 64,
                                 t.kvh * p.group + t.hchunk * 8, t.q_start + t.tile_pos0 + q4 * ppw);
               ptx::bulk_commit();
@@ -551,7 +588,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
             const int r = q4 * 32 + it * 4 + (lane >> 3);          // tile row whose chunk (lane & 7) I store
             // r / heads_here without an integer division: exact for r < 128 and at most 8 heads
             const int rpi = (int)(((float)r + 0.5f) * inv_heads), rhd = r - rpi * t.heads_here;
-            if (rpi < npos) {
+            if (rpi < npos && (!EXACT || half * 64 + (lane & 7) * 8 < p.dv)) {
               const uint4 v = *reinterpret_cast<const uint4*>(p_half + sw128(r, lane & 7));
               __nv_bfloat16* orow = p.out + (long long)(t.q_start + t.tile_pos0 + rpi) * p.o_tok_stride +
                                     (long long)(t.kvh * p.group + t.hchunk * 8 + rhd) * p.o_head_stride + half * 64;
@@ -564,7 +601,8 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
           __nv_bfloat16* orow = p.out + (long long)(t.q_start + t.tile_pos0 + pi) * p.o_tok_stride +
                                 (long long)(t.kvh * p.group + t.hchunk * 8 + hd) * p.o_head_stride + half * 64;
 #pragma unroll
-          for (int i = 0; i < 64; ++i) orow[i] = f2bf(o[i] * inv);
+          for (int i = 0; i < 64; ++i)
+            if (!EXACT || half * 64 + i < p.dv) orow[i] = f2bf(o[i] * inv);
         }
       }
       if (warp == 4) ATR_STAMP(2, g0 + t.nblk - 1, 3);   // tile stored
@@ -592,24 +630,25 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   }
 }
 
-template <int DK>
+template <int DK, bool EXACT>
 inline int attn_rows_launch(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq, const CUtensorMap& to,
                             const AttnParams& p, cudaStream_t st) {
-  // tiles (K ring, V ring, two Q buffers, P) + small arrays (barriers, alpha, l, TMEM slot, abort flag) + alignment
-  constexpr int tiles = ATC_BN * (2 * DK + 2 * 128) * 2 + 2 * (DK / 64) * ATR_ROWS * 128 + 2 * ATR_ROWS * 128;
+  // tiles (K ring, V ring, Q buffers, P) + small arrays (barriers, alpha, l, TMEM slot, abort flag) + alignment
+  constexpr int tiles = ATC_BN * (2 * DK + 2 * 128) * 2 + (EXACT ? 1 : 2) * (DK / 64) * ATR_ROWS * 128 +
+                        (EXACT ? 4 : 2) * ATR_ROWS * 128;
   constexpr int small = 256 + 4 * ATR_ROWS * 4 + 16;
   constexpr int smem = (tiles + small + 1023 <= 227 * 1024) ? tiles + small + 1023 : 227 * 1024;
   static_assert(tiles + small <= 227 * 1024, "shared memory budget");
   static PerDeviceFlags attr_set;
-  if (int rc = set_max_dyn_smem_once(attr_set, paged_attn_rows_kernel<DK>, smem)) return rc;
+  if (int rc = set_max_dyn_smem_once(attr_set, paged_attn_rows_kernel<DK, EXACT>, smem)) return rc;
   const int nctas = p.tc_tiles < sm_count() ? p.tc_tiles : sm_count();
-  launch_k(paged_attn_rows_kernel<DK>, dim3((unsigned)nctas), dim3(ATR_THREADS), (size_t)smem, st, tk, tv, tq, to, p);
+  launch_k(paged_attn_rows_kernel<DK, EXACT>, dim3((unsigned)nctas), dim3(ATR_THREADS), (size_t)smem, st, tk, tv, tq, to, p);
   return launch_status();
 }
 
 inline int attn_rows_dispatch(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq, const CUtensorMap& to,
                               const AttnParams& p, cudaStream_t st) {
-  return attn_rows_launch<128>(tk, tv, tq, to, p, st);
+  return attn_rows_launch<128, false>(tk, tv, tq, to, p, st);
 }
 
 }  // namespace b200

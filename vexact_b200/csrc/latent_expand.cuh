@@ -315,36 +315,3 @@ extern "C" int b200_latent_attn_expanded(const void* q, long long q_row_stride, 
   p.scale_log2 = scale * kLog2e;
   return latent_expand_dispatch<false>(p, max_len, n, (cudaStream_t)stream);
 }
-
-// The same kernel over the pages of a per-head cache: k_cache [blocks, page, kv_heads, DK], v_cache [.., DV], contiguous.
-extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache,
-                                        void* out, long long out_row_stride, const void* query_start_loc,
-                                        const void* context_lens, const void* page_table, long long page_table_stride,
-                                        int max_pages, int page_size, int num_blocks, int num_seqs, const void* seq_ids_i32,
-                                        int n, int max_len, int window, int heads, int kv_heads, int DK, int DV, float scale,
-                                        void* stream) {
-  using namespace b200;
-  LatentExpandParams p{};
-  p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
-            page_size, num_blocks, num_seqs, 0, 0, window};
-  if (!latent_seqs_ok(p.seqs) || !q || !k_cache || !v_cache || !out || !seq_ids_i32 || n <= 0 || max_len <= 0 || heads <= 0 ||
-      kv_heads <= 0 || heads % kv_heads || DK <= 0 || DV <= 0 || window < 0)
-    return B200_ERR_ARG;
-  if (DK % 8 || DV % 8 || q_row_stride % 8 || out_row_stride % 8 || DK > 256 || DV > 256 || heads > 65535 || n > 65535)
-    return B200_ERR_SHAPE;
-  p.seq_ids = (const int*)seq_ids_i32;
-  p.q = (const __nv_bfloat16*)q;
-  p.k = (const __nv_bfloat16*)k_cache;
-  p.v = (const __nv_bfloat16*)v_cache;
-  p.out = (__nv_bfloat16*)out;
-  p.q_stride = q_row_stride;
-  p.k_stride = (long long)kv_heads * DK;
-  p.v_stride = (long long)kv_heads * DV;
-  p.out_stride = out_row_stride;
-  p.heads = heads;
-  p.group = heads / kv_heads;
-  p.DN = DK;
-  p.DV = DV;
-  p.scale_log2 = scale * kLog2e;
-  return latent_expand_dispatch<true>(p, max_len, n, (cudaStream_t)stream);
-}

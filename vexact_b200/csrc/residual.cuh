@@ -15,8 +15,6 @@
 
 namespace b200 {
 
-constexpr int RES_CHUNKS = 4;   // register chunks per thread: W <= threads * RES_CHUNKS * 4
-
 struct ResidualParams {
   float* x;                   // [T, W]
   const void* y;              // [T or y_rows, y_stride], or null (then `extra` or ids)
@@ -47,8 +45,9 @@ __device__ __forceinline__ void load4_tail(const T* p, int left, float (&v)[4]) 
   for (int k = 0; k < 4; ++k) v[k] = k < left ? to_f32(p[k]) : 0.f;
 }
 
-template <typename T>
-__global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualParams p) {
+// CH: register chunks of four columns per thread (W <= threads * CH * 4); MAXT: threads at most.
+template <typename T, int CH, int MAXT>
+__global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParams p) {
   __shared__ float red[32];
   pdl_trigger();
   pdl_wait();
@@ -78,37 +77,44 @@ __global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualParam
   const T* extra = p.extra ? reinterpret_cast<const T*>(p.extra) + t * p.extra_stride : nullptr;
   const int* pick = p.scatter_index ? p.scatter_index + t * p.topk : nullptr;
   float* xrow = p.x + t * (long long)W;
-  float v[RES_CHUNKS][4], x[RES_CHUNKS][4];
+  int pos[8];                  // the token's rows of a mixture, looked up once
+  if (pick)
+#pragma unroll
+    for (int k = 0; k < 8; ++k) pos[k] = k < p.topk ? pick[k] : -1;
+  float v[CH][4], x[CH][4], w[CH][4], nw[CH][4];
   float ss = 0.f;
 #pragma unroll
-  for (int c = 0; c < RES_CHUNKS; ++c) {
+  for (int c = 0; c < CH; ++c) {   // every load that depends on nothing, ahead of the first use
     const int i = (c * blockDim.x + threadIdx.x) * 4;
 #pragma unroll
-    for (int k = 0; k < 4; ++k) v[c][k] = x[c][k] = 0.f;
+    for (int k = 0; k < 4; ++k) v[c][k] = x[c][k] = w[c][k] = nw[c][k] = 0.f;
     if (i >= W) continue;
     if (src) get(src, i, v[c]);
     if (!p.ids) get(xrow, i, x[c]);
+    get(p.post, i, w[c]);
+    if (p.norm_w) get(p.norm_w, i, nw[c]);
+  }
+  auto add_row = [&](const T* row, int i, float (&a)[4]) {
+    float e[4];
+    get(row, i, e);
+#pragma unroll
+    for (int q = 0; q < 4; ++q) a[q] += e[q];
+  };
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int i = (c * blockDim.x + threadIdx.x) * 4;
+    if (i >= W) continue;
     if (pick) {
-      int row = p.topk > 0 ? pick[0] : -1;
-      for (int k = 0; k < p.topk; ++k) {
-        const int next = k + 1 < p.topk ? pick[k + 1] : -1;
-        if (row >= 0 && row < p.y_rows) {
-          float e[4];
-          get(reinterpret_cast<const T*>(p.y) + row * p.y_stride, i, e);
+      auto one = [&](int row) {
+        if (row >= 0 && row < p.y_rows) add_row(reinterpret_cast<const T*>(p.y) + row * p.y_stride, i, v[c]);
+        else if (threadIdx.x == 0 && c == 0) report_status(B200_STATUS_BAD_INDEX, row);
+      };
 #pragma unroll
-          for (int q = 0; q < 4; ++q) v[c][q] += e[q];
-        } else if (threadIdx.x == 0 && c == 0) {
-          report_status(B200_STATUS_BAD_INDEX, row);
-        }
-        row = next;
-      }
+      for (int k = 0; k < 8; ++k)
+        if (k < p.topk) one(pos[k]);
+      for (int k = 8; k < p.topk; ++k) one(pick[k]);
     }
-    if (extra) {
-      float e[4];
-      get(extra, i, e);
-#pragma unroll
-      for (int q = 0; q < 4; ++q) v[c][q] += e[q];
-    }
+    if (extra) add_row(extra, i, v[c]);
 #pragma unroll
     for (int k = 0; k < 4; ++k) ss = fmaf(v[c][k], v[c][k], ss);
   }
@@ -116,15 +122,14 @@ __global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualParam
   const float inv_y = 1.f / sqrtf(ss / (float)W + p.eps);
   ss = 0.f;
 #pragma unroll
-  for (int c = 0; c < RES_CHUNKS; ++c) {
+  for (int c = 0; c < CH; ++c) {
     const int i = (c * blockDim.x + threadIdx.x) * 4;
     if (i >= W) continue;
-    float w[4], a[4] = {0.f, 0.f, 0.f, 0.f};
-    get(p.post, i, w);
+    float a[4] = {0.f, 0.f, 0.f, 0.f};
     if (p.add) get(p.add, i, a);
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
-      x[c][k] = x[c][k] + v[c][k] * inv_y * w[k] + a[k];
+      x[c][k] = x[c][k] + v[c][k] * inv_y * w[c][k] + a[k];
       ss = fmaf(x[c][k], x[c][k], ss);      // columns past W are zero in every term
     }
     if (p.write_back) {
@@ -140,20 +145,33 @@ __global__ void __launch_bounds__(1024) residual_step_kernel(const ResidualParam
   const float inv = 1.f / sqrtf(ss / (float)W + p.eps);
   T* orow = reinterpret_cast<T*>(p.xn) + r * p.xn_stride;
 #pragma unroll
-  for (int c = 0; c < RES_CHUNKS; ++c) {
+  for (int c = 0; c < CH; ++c) {
     const int i = (c * blockDim.x + threadIdx.x) * 4;
     if (i >= W) continue;
-    float w[4];
-    get(p.norm_w, i, w);
+    float o[4];
 #pragma unroll
-    for (int k = 0; k < 4; ++k) w[k] *= x[c][k] * inv;
-    if (vec) store4(orow + i, w);
+    for (int k = 0; k < 4; ++k) o[k] = x[c][k] * inv * nw[c][k];
+    if (vec) store4(orow + i, o);
     else
 #pragma unroll
       for (int k = 0; k < 4; ++k)
-        if (i + k < W) orow[i + k] = from_f32<T>(w[k]);
+        if (i + k < W) orow[i + k] = from_f32<T>(o[k]);
   }
   for (int i = W + threadIdx.x; i < p.xn_cols; i += blockDim.x) orow[i] = from_f32<T>(0.f);
+}
+
+template <typename T>
+inline int residual_launch(const ResidualParams& p, long long rows, cudaStream_t st) {
+  const int chunks = (p.W + 3) / 4;
+  const dim3 g((unsigned)rows);
+  int threads = 64;
+  while (threads < 256 && chunks > threads) threads <<= 1;
+  if (chunks <= threads) launch_k(residual_step_kernel<T, 1, 256>, g, dim3(threads), 0, st, p);
+  else if (chunks <= 512) launch_k(residual_step_kernel<T, 2, 256>, g, dim3(256), 0, st, p);
+  else if (chunks <= 1024) launch_k(residual_step_kernel<T, 2, 512>, g, dim3(512), 0, st, p);
+  else if (chunks <= 4096) launch_k(residual_step_kernel<T, 4, 1024>, g, dim3(1024), 0, st, p);
+  else return B200_ERR_SHAPE;
+  return launch_status();
 }
 
 }  // namespace b200
@@ -173,16 +191,9 @@ extern "C" int b200_residual_step(void* x_f32, const void* y, long long y_row_st
   if (num_rows > 0x7fffffffLL) return B200_ERR_SHAPE;
   if (num_rows == 0) return B200_OK;
   if (W % 4 == 0 && (y_row_stride % 4 || xn_row_stride % 4 || extra_row_stride % 4)) return B200_ERR_SHAPE;
-  const int chunks = (W + 3) / 4;
-  int threads = 64;
-  while (threads < 512 && chunks > threads) threads <<= 1;
-  while (threads < 1024 && chunks > threads * RES_CHUNKS) threads <<= 1;
-  if (chunks > threads * RES_CHUNKS) return B200_ERR_SHAPE;
   ResidualParams p{(float*)x_f32, y, y_row_stride, y_rows, (const int*)scatter_index_i32, topk, extra, extra_row_stride,
                    embed, (const long long*)ids_i64, vocab, (const int*)rows_i32, num_tokens, (const float*)post_f32,
                    (const float*)add_f32, (const float*)norm_w_f32, eps, xn, xn_row_stride, xn_cols, W, write_back};
-  const dim3 g((unsigned)num_rows), b((unsigned)threads);
-  if (dtype == 0) launch_k(residual_step_kernel<__nv_bfloat16>, g, b, 0, (cudaStream_t)stream, p);
-  else launch_k(residual_step_kernel<float>, g, b, 0, (cudaStream_t)stream, p);
-  return launch_status();
+  return dtype == 0 ? residual_launch<__nv_bfloat16>(p, num_rows, (cudaStream_t)stream)
+                    : residual_launch<float>(p, num_rows, (cudaStream_t)stream);
 }

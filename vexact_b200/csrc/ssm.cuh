@@ -470,6 +470,57 @@ __global__ void __launch_bounds__(256) ssm_gate_norm_warp_kernel(const SsmGateNo
   }
 }
 
+// Narrow parts (a multiple of 8 up to 8 LANES columns, heads unpadded, bf16): LANES lanes per (token, part), eight columns each.
+template <int LANES, bool NORM_FIRST>
+__global__ void __launch_bounds__(256) ssm_gate_norm_narrow_kernel(const SsmGateNormParams p, long long pairs) {
+  pdl_trigger();
+  pdl_wait();
+  const long long id = (long long)blockIdx.x * (256 / LANES) + threadIdx.x / LANES;
+  const int n = p.heads * p.P / p.parts, i = (threadIdx.x % LANES) * 8;
+  const bool in = id < pairs && i < n;
+  const long long t = in ? id / p.parts : 0;
+  const int j = in ? (int)(id - t * p.parts) * n + i : 0;
+  uint4 a = make_uint4(0, 0, 0, 0), b = a;
+  float w[8] = {};
+  if (in) {
+    a = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.y) + t * p.y_stride + j);
+    b = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(p.z) + t * p.z_stride + j);
+    load4(p.w + j, *reinterpret_cast<float(*)[4]>(w));
+    load4(p.w + j + 4, *reinterpret_cast<float(*)[4]>(w + 4));
+  }
+  const uint32_t av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+  float g[8], z[8], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    unpack_bf2(av[k], g[2 * k], g[2 * k + 1]);
+    unpack_bf2(bv[k], z[2 * k], z[2 * k + 1]);
+  }
+#pragma unroll
+  for (int k = 0; k < 8; ++k) {
+    z[k] = silu_as<__nv_bfloat16>(z[k]);
+    if (!NORM_FIRST) g[k] *= z[k];
+    ss = fmaf(g[k], g[k], ss);
+  }
+#pragma unroll
+  for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = 1.f / sqrtf(ss / (float)n + p.eps);
+  if (!in) return;
+  uint32_t o[4];
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const float f0 = NORM_FIRST ? z[2 * k] : 1.f, f1 = NORM_FIRST ? z[2 * k + 1] : 1.f;
+    o[k] = pack_bf2(g[2 * k] * inv * w[2 * k] * f0, g[2 * k + 1] * inv * w[2 * k + 1] * f1);
+  }
+  *reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(p.out) + t * p.out_stride + j) = make_uint4(o[0], o[1], o[2], o[3]);
+}
+
+template <int LANES>
+inline int ssm_gate_norm_narrow(const SsmGateNormParams& p, long long pairs, cudaStream_t st) {
+  launch_k(p.norm_first ? ssm_gate_norm_narrow_kernel<LANES, true> : ssm_gate_norm_narrow_kernel<LANES, false>,
+           dim3((unsigned)((pairs * LANES + 255) / 256)), dim3(256), 0, st, p, pairs);
+  return launch_status();
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) ssm_gate_norm_kernel(const SsmGateNormParams p) {
   __shared__ float red[32];
@@ -631,6 +682,9 @@ extern "C" int b200_ssm_gate_norm(const void* y, long long y_row_stride, const v
   auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
   if (dtype == 0 && p_true == P && n % 8 == 0 && n <= 2048 && aligned(y) && aligned(z) && aligned(out) && aligned(w_f32)) {
     const long long pairs = T * parts;
+    if (n <= 64) return ssm_gate_norm_narrow<8>(p, pairs, (cudaStream_t)stream);
+    if (n <= 128) return ssm_gate_norm_narrow<16>(p, pairs, (cudaStream_t)stream);
+    if (n <= 256) return ssm_gate_norm_narrow<32>(p, pairs, (cudaStream_t)stream);
     launch_k(norm_first ? ssm_gate_norm_warp_kernel<true> : ssm_gate_norm_warp_kernel<false>,
              dim3((unsigned)((pairs + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, p, pairs);
     return launch_status();

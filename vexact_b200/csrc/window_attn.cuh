@@ -11,8 +11,8 @@
 //
 // Algorithmic bytes: the keys and values each sequence's window holds, once per KV head: HBM bandwidth.
 #pragma once
-#include "attn_tc.cuh"     // fast_exp2, and through it attn.cuh: ldmatrix, movmatrix, mma, tensor maps
-#include "latent.cuh"      // LatentSeqs
+#include "attn_rows.cuh"       // the exact rows-on-lanes kernel, and through it fast_exp2, ldmatrix, mma, tensor maps
+#include "latent_expand.cuh"   // the mma.sync kernel of long portions; LatentSeqs
 
 namespace b200 {
 
@@ -336,4 +336,89 @@ extern "C" int b200_window_attn_decode(const void* q, long long q_row_stride, co
   if (DK <= 128 && DV <= 128) return window_attn_launch<128, 128, 2, 3>(tk, tv, p, grid, st);
   if (DK <= 192 && DV <= 128) return window_attn_launch<192, 128, 2, 2>(tk, tv, p, grid, st);
   return window_attn_launch<256, 256, 2, 2>(tk, tv, p, grid, st);
+}
+
+// Long portions: the n sequences named, which are those that bring at least min_len tokens.  Heads of 65 .. 128 columns go
+// to the tcgen05 kernel (exact form of attn_rows.cuh) when the query layout suits its copies, others to the mma.sync kernel
+// of latent_expand.cuh; form: 0 = this choice, 1 = mma.sync (cross-checks).
+extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache,
+                                        void* out, long long out_row_stride, const void* query_start_loc,
+                                        const void* context_lens, const void* page_table, long long page_table_stride,
+                                        int max_pages, int page_size, int num_blocks, int num_seqs, const void* seq_ids_i32,
+                                        int n, int max_len, int min_len, int window, long long T, int heads, int kv_heads,
+                                        int DK, int DV, float scale, int form, void* stream) {
+  using namespace b200;
+  LatentExpandParams p{};
+  p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
+            page_size, num_blocks, num_seqs, 0, 0, window};
+  if (!latent_seqs_ok(p.seqs) || !q || !k_cache || !v_cache || !out || !seq_ids_i32 || n <= 0 || max_len <= 0 || T <= 0 ||
+      heads <= 0 || kv_heads <= 0 || heads % kv_heads || DK <= 0 || DV <= 0 || window < 0)
+    return B200_ERR_ARG;
+  if (DK % 8 || DV % 8 || q_row_stride % 8 || out_row_stride % 8 || DK > 256 || DV > 256 || heads > 65535 || n > 65535)
+    return B200_ERR_SHAPE;
+  const cudaStream_t st = (cudaStream_t)stream;
+  const int group = heads / kv_heads, hh = group < 8 ? group : 8;
+  const bool pages_ok = page_size % 8 == 0 && (page_size < ATT_BN ? ATT_BN % page_size == 0 : page_size % ATT_BN == 0);
+  if (form == 0 && DK <= 128 && DV <= 128 && (DK > 64 || DV > 64) && (group <= 8 || group % 8 == 0) && pages_ok &&
+      num_seqs <= 65535) {
+    AttnParams a{};
+    a.q = (const __nv_bfloat16*)q;
+    a.out = (__nv_bfloat16*)out;
+    a.q_tok_stride = q_row_stride;
+    a.q_head_stride = DK;
+    a.o_tok_stride = out_row_stride;
+    a.o_head_stride = DV;
+    a.cu_seqlens_q = p.seqs.query_start_loc;
+    a.seqused_k = p.seqs.context_lens;
+    a.page_table = p.seqs.page_table;
+    a.page_table_stride = page_table_stride;
+    a.max_pages = max_pages;
+    a.page_size = page_size;
+    a.box_tokens = page_size < ATT_BN ? page_size : ATT_BN;
+    a.num_q_heads = heads;
+    a.num_kv_heads = kv_heads;
+    a.group = group;
+    a.head_chunks = (group + 7) / 8;
+    a.pos_per_tile = ATR_ROWS / hh;
+    a.qk_scale = scale * kLog2e;
+    a.num_blocks = num_blocks;
+    a.num_seqs = num_seqs;
+    a.max_seqlen_q = max_len;
+    a.min_q = min_len;
+    a.window = window;
+    a.dv = DV;
+    a.tc_q_tiles = (max_len + a.pos_per_tile - 1) / a.pos_per_tile;
+    a.tc_hy = kv_heads * a.head_chunks;
+    const long long tiles = (long long)a.tc_q_tiles * a.tc_hy * num_seqs;
+    if (tiles > 0x3fffffffLL) return B200_ERR_SHAPE;
+    a.tc_tiles = (int)tiles;
+    const int ctas = a.tc_tiles < sm_count() ? a.tc_tiles : sm_count();
+    a.tc_slots = (a.tc_tiles + ctas - 1) / ctas * ctas;
+    CUtensorMap tk, tv, tq, to;
+    const long long kr = (long long)kv_heads * DK, vr = (long long)kv_heads * DV;
+    int rc = make_tmap_cache(&tk, k_cache, num_blocks, page_size, kv_heads, DK, page_size * kr, kr, DK, a.box_tokens);
+    if (!rc) rc = make_tmap_cache(&tv, v_cache, num_blocks, page_size, kv_heads, DV, page_size * vr, vr, DV, a.box_tokens);
+    if (rc) return rc;
+    to = tk;
+    if (make_tmap_q(&tq, q, T, heads, DK, q_row_stride, DK, hh, a.pos_per_tile) == B200_OK) {
+      a.q_tma = 1;
+      a.o_tma = 32 % hh == 0 && make_tmap_q(&to, out, T, heads, DV, out_row_stride, DV, hh, 32 / hh, true) == B200_OK;
+      return attn_rows_launch<128, true>(tk, tv, tq, to, a, st);
+    }
+  }
+  p.seq_ids = (const int*)seq_ids_i32;
+  p.q = (const __nv_bfloat16*)q;
+  p.k = (const __nv_bfloat16*)k_cache;
+  p.v = (const __nv_bfloat16*)v_cache;
+  p.out = (__nv_bfloat16*)out;
+  p.q_stride = q_row_stride;
+  p.k_stride = (long long)kv_heads * DK;
+  p.v_stride = (long long)kv_heads * DV;
+  p.out_stride = out_row_stride;
+  p.heads = heads;
+  p.group = group;
+  p.DN = DK;
+  p.DV = DV;
+  p.scale_log2 = scale * kLog2e;
+  return latent_expand_dispatch<true>(p, max_len, n, st);
 }

@@ -1,6 +1,7 @@
 """Grouped-query attention without positions in the scores, optionally inside a window, over paged per-head keys and
-values (`csrc/window_attn.cuh` for decoded tokens and short portions, the paged form of `csrc/latent_expand.cuh` for long
-ones, `csrc/latent.cuh` on CUDA cores for fp32 models and for dims the tensor-core kernels do not take)."""
+values (`csrc/window_attn.cuh` for decoded tokens and short portions; for long ones the exact form of
+`csrc/attn_rows.cuh`, or the paged form of `csrc/latent_expand.cuh` by head dims; `csrc/latent.cuh` on CUDA cores for fp32
+models and for dims the tensor-core kernels do not take)."""
 from __future__ import annotations
 
 from dataclasses import dataclass
@@ -57,14 +58,16 @@ def attend_decode(w: AttentionWeights, q: torch.Tensor, k_cache, v_cache, out: t
         "b200_window_attn_decode")
 
 
-def attend_prefill(w: AttentionWeights, q: torch.Tensor, k_cache, v_cache, out: torch.Tensor, step, longs) -> None:
-    """The sequences named by `longs` = (ids, most new tokens)."""
+def attend_prefill(w: AttentionWeights, q: torch.Tensor, k_cache, v_cache, out: torch.Tensor, step, longs,
+                   form: int = 0) -> None:
+    """The sequences named by `longs` = (ids, most new tokens): those beyond the decode kernel.  form 1: the mma.sync
+    kernel whatever the head dims."""
     ids, most = longs
     _lib.check(
         _lib.load().b200_window_attn_prefill(
             q.data_ptr(), q.stride(0), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), out.stride(0),
-            *_pages(step, k_cache), ids.data_ptr(), ids.numel(), most, w.window or 0, w.heads, w.kv_heads, w.DK, w.DV,
-            float(w.scale), _lib.current_stream()),
+            *_pages(step, k_cache), ids.data_ptr(), ids.numel(), most, DECODE_MAX_TOKENS + 1, w.window or 0, q.shape[0],
+            w.heads, w.kv_heads, w.DK, w.DV, float(w.scale), form, _lib.current_stream()),
         "b200_window_attn_prefill")
 
 
