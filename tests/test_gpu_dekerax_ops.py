@@ -53,7 +53,7 @@ def test_residual_step(dtype, W):
 
 
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("top,shared", [(1, False), (3, True)])
+@pytest.mark.parametrize("top,shared", [(1, False), (3, True), (4, True), (6, False), (11, True)])
 def test_residual_step_sums_a_pending_mixture(dtype, top, shared):
     from vexact_b200.fused_moe import PendingMixture
     from vexact_b200.residual import residual_step

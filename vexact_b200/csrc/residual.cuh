@@ -110,8 +110,27 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
         else if (threadIdx.x == 0 && c == 0) report_status(B200_STATUS_BAD_INDEX, row);
       };
 #pragma unroll
-      for (int k = 0; k < 8; ++k)
-        if (k < p.topk) one(pos[k]);
+      for (int k0 = 0; k0 < 8; k0 += 4) {
+        if (vec && k0 + 4 <= p.topk) {      // four rows requested together, added in order
+          float e[4][4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int row = pos[k0 + k];
+            const bool ok = row >= 0 && row < p.y_rows;
+            if (!ok && threadIdx.x == 0 && c == 0) report_status(B200_STATUS_BAD_INDEX, row);
+            load4(reinterpret_cast<const T*>(p.y) + (ok ? row : 0) * p.y_stride + i, e[k]);
+            if (!ok) e[k][0] = e[k][1] = e[k][2] = e[k][3] = 0.f;
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+#pragma unroll
+            for (int q = 0; q < 4; ++q) v[c][q] += e[k][q];
+        } else {
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            if (k0 + k < p.topk) one(pos[k0 + k]);
+        }
+      }
       for (int k = 8; k < p.topk; ++k) one(pick[k]);
     }
     if (extra) add_row(extra, i, v[c]);
