@@ -194,7 +194,8 @@ __global__ void __launch_bounds__(DLC_THREADS) delta_prep_kernel(const DeltaChun
 
 template <int NMAX, int PS>
 struct DlcLayout {
-  static constexpr int STAGES = NMAX <= 128 ? 2 : 1;
+  // one stage where two would leave room for a single CTA on an SM: the other CTA's products cover the copies
+  static constexpr int STAGES = NMAX <= 64 || (NMAX <= 128 && PS <= 16) ? 2 : 1;
   static constexpr int LDN = NMAX + 8, LDP = PS + 8;          // padded pitches: ldmatrix rows in distinct banks
   static constexpr int QK = DLC_L * LDN * 2, X = DLC_L * LDP * 2, ST = NMAX * LDP * 2;
   static constexpr int STAGE = 2 * QK + X + DLC_VECS * DLC_L * 4;    // q, k, v, vectors
