@@ -37,13 +37,13 @@ struct LatentPrepParams {
   int heads, DN, DR, R;
   int r_true;                // columns of c that exist (the rest is padding and zero)
   int rot_dims;
-  int half;                  // 1: pairs (i, i + rot_dims / 2), 0: pairs (2i, 2i + 1)
   float eps;
   long long num_slots;
 };
 
-// Columns of pair i of DR / 2: the rotating pairs first, in either layout, then neighbours that pass.
-__device__ __forceinline__ void rot_pair(int i, int rot_dims, int half, int& a, int& b) {
+// Columns of pair i of DR / 2: the rotating pairs first, as (i, i + rot_dims / 2) with `half` and as (2i, 2i + 1) without,
+// then neighbours that pass.
+__device__ __forceinline__ void rot_pair(int i, int rot_dims, bool half, int& a, int& b) {
   if (half && i < (rot_dims >> 1)) {
     a = i;
     b = i + (rot_dims >> 1);
@@ -53,7 +53,7 @@ __device__ __forceinline__ void rot_pair(int i, int rot_dims, int half, int& a, 
   }
 }
 
-template <typename T>
+template <typename T, bool HALF>
 __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams p) {
   __shared__ float red[32];
   __shared__ float s_cos[128], s_sin[128];
@@ -111,7 +111,7 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
       const T* kr = c + p.R;
       for (int i = tid; i < (p.DR >> 1); i += 128) {
         int a, b;
-        rot_pair(i, p.rot_dims, p.half, a, b);
+        rot_pair(i, p.rot_dims, HALF, a, b);
         float u = to_f32(kr[a]), v = to_f32(kr[b]);
         if (i < half) {
           const float w = u * s_cos[i] - v * s_sin[i];
@@ -130,7 +130,7 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
   for (int e = tid; e < p.heads * pairs; e += 128) {
     const int h = e / pairs, i = e - h * pairs;
     int a, b;
-    rot_pair(i, p.rot_dims, p.half, a, b);
+    rot_pair(i, p.rot_dims, HALF, a, b);
     T* q = reinterpret_cast<T*>(p.q) + t * p.q_stride + h * dq + p.DN;
     float u = to_f32(q[a]), v = to_f32(q[b]);
     if (i < half) {
@@ -310,9 +310,11 @@ extern "C" int b200_latent_prep(void* q, long long q_row_stride, const void* kv,
   if (T == 0) return B200_OK;
   LatentPrepParams p{q, q_row_stride, kv, kv_row_stride, q_latent, q_latent_row_stride, (const float*)q_norm_f32, QL, ql_true,
                      (const long long*)positions_i64, (const int*)slot_mapping_i32, (const float*)inv_freq_f32,
-                     (const float*)c_norm_f32, cache, q_lat, heads, DN, DR, R, r_true, rot_dims, rot_half, eps, num_slots};
-  if (dtype == 0) launch_k(latent_prep_kernel<__nv_bfloat16>, dim3((unsigned)T), dim3(128), 0, (cudaStream_t)stream, p);
-  else launch_k(latent_prep_kernel<float>, dim3((unsigned)T), dim3(128), 0, (cudaStream_t)stream, p);
+                     (const float*)c_norm_f32, cache, q_lat, heads, DN, DR, R, r_true, rot_dims, eps, num_slots};
+  const dim3 g((unsigned)T), b(128);
+  const cudaStream_t st = (cudaStream_t)stream;
+  if (dtype == 0) launch_k(rot_half ? latent_prep_kernel<__nv_bfloat16, true> : latent_prep_kernel<__nv_bfloat16, false>, g, b, 0, st, p);
+  else launch_k(rot_half ? latent_prep_kernel<float, true> : latent_prep_kernel<float, false>, g, b, 0, st, p);
   return launch_status();
 }
 

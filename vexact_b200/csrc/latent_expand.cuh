@@ -58,7 +58,8 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   const int tiles = (len + LEX_BM - 1) / LEX_BM;
   if ((int)blockIdx.x >= tiles) return;
   const int row_base = (tiles - 1 - (int)blockIdx.x) * LEX_BM;
-  const int keys = p.seqs.context_lens[seq], past = keys - len, window = p.seqs.window;
+  const int keys = p.seqs.context_lens[seq], past = keys - len;
+  const int window = p.seqs.window > 0 ? p.seqs.window : 0x3fffffff;
   const int key_base = PAGED ? 0 : p.key_base[i];
   const long long key0 = PAGED ? 0 : p.key_start[i] - key_base;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
@@ -76,24 +77,33 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
                p.q + (long long)(t0 + row_base + (in ? r : 0)) * p.q_stride + (long long)h * (p.DN + p.DR) + (in ? v * 8 : 0),
                in);
   }
+  auto seen = [&](int j) { return (uint32_t)(j - first_key) < (uint32_t)(last_key - first_key); };   // by some row of the tile
+  // source row of key j; a key that is not wanted (or whose page is bad) names some readable row
+  auto row_of = [&](int j, bool& in) -> long long {
+    if constexpr (PAGED) {
+      const long long row = in ? latent_key_row(p.seqs, seq, j) : -1;
+      in = row >= 0;
+      return in ? row : 0;
+    } else {
+      return key0 + (in ? j : first_key);
+    }
+  };
   auto load = [&](int b) {
     const uint32_t k = smem + L::Q + (b & 1) * (L::K + L::V), vt = k + L::K;
     const int base = b * LEX_BN;
     for (int e = tid; e < LEX_BN * (DK / 8); e += LEX_THREADS) {
       const int r = e / (DK / 8), col = (e % (DK / 8)) * 8;
-      const bool seen = base + r >= first_key && base + r < last_key;
-      const long long row = seen ? (PAGED ? latent_key_row(p.seqs, seq, base + r) : key0 + base + r) : -1;
-      const bool in = row >= 0 && col < p.DN + p.DR;
-      const __nv_bfloat16* src = p.k;
-      if (in) src = col < p.DN ? p.k + row * p.k_stride + (long long)kvh * p.DN + col : p.rot + row * p.rot_stride + (col - p.DN);
+      bool in = seen(base + r) && col < p.DN + p.DR;
+      const long long row = row_of(base + r, in);
+      const __nv_bfloat16* src = col < p.DN || !in ? p.k + row * p.k_stride + (long long)kvh * p.DN + (in ? col : 0)
+                                                   : p.rot + row * p.rot_stride + (col - p.DN);
       cp_async16(k + (uint32_t)(r * L::LDK + col) * 2, src, in);
     }
     for (int e = tid; e < LEX_BN * (DV / 8); e += LEX_THREADS) {
       const int r = e / (DV / 8), col = (e % (DV / 8)) * 8;
-      const bool seen = base + r >= first_key && base + r < last_key;
-      const long long row = seen ? (PAGED ? latent_key_row(p.seqs, seq, base + r) : key0 + base + r) : -1;
-      const bool in = row >= 0 && col < p.DV;
-      cp_async16(vt + (uint32_t)(r * L::LDV + col) * 2, in ? p.v + row * p.v_stride + (long long)kvh * p.DV + col : p.v, in);
+      bool in = seen(base + r) && col < p.DV;
+      const long long row = row_of(base + r, in);
+      cp_async16(vt + (uint32_t)(r * L::LDV + col) * 2, p.v + row * p.v_stride + (long long)kvh * p.DV + (in ? col : 0), in);
     }
     cp_async_commit();
   };
@@ -125,7 +135,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
     for (int sub = 0; sub < LEX_BN / LEX_SUB; ++sub) {
       const int base = b * LEX_BN + sub * LEX_SUB;
       if (r0 >= rows || base > first_pos + 16 * MT - 1) break;   // no row of this warp sees these keys
-      if (window > 0 && base + LEX_SUB - 1 <= first_pos - window) continue;   // nor these, before every row's window
+      if (base + LEX_SUB - 1 <= first_pos - window) continue;   // nor these, before every row's window
       float s[MT][NS][4];
 #pragma unroll
       for (int t = 0; t < MT; ++t)
@@ -147,8 +157,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
         }
       }
       // some (row, key) of these is masked
-      const bool edge = base + LEX_SUB - 1 > first_pos || (window > 0 && base <= first_pos + 16 * MT - 1 - window);
-      const uint32_t reach = window > 0 ? (uint32_t)window : 0x80000000u;     // a row sees 0 <= its position - key < reach
+      const bool edge = base + LEX_SUB - 1 > first_pos || base <= first_pos + 16 * MT - 1 - window;
 #pragma unroll
       for (int t = 0; t < MT; ++t) {
         const int pos0 = first_pos + 16 * t + g4;                 // position of row g4 of the tile (and + 8)
@@ -158,7 +167,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             float v = s[t][j][e] * p.scale_log2;
-            if (edge && (uint32_t)(pos0 + 8 * (e >> 1) - (base + 8 * j + 2 * t4 + (e & 1))) >= reach) v = -INFINITY;
+            if (edge && (uint32_t)(pos0 + 8 * (e >> 1) - (base + 8 * j + 2 * t4 + (e & 1))) >= (uint32_t)window) v = -INFINITY;   // a row sees 0 <= its position - key < window
             s[t][j][e] = v;
             mb[e >> 1] = fmaxf(mb[e >> 1], v);
           }

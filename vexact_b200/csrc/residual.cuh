@@ -45,8 +45,8 @@ __device__ __forceinline__ void load4_tail(const T* p, int left, float (&v)[4]) 
   for (int k = 0; k < 4; ++k) v[k] = k < left ? to_f32(p[k]) : 0.f;
 }
 
-// CH: register chunks of four columns per thread (W <= threads * CH * 4); MAXT: threads at most.
-template <typename T, int CH, int MAXT>
+// CH: register chunks of four columns per thread (W <= threads * CH * 4); MAXT: threads at most; PICK: y is expert-sorted.
+template <typename T, int CH, int MAXT, bool PICK>
 __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParams p) {
   __shared__ float red[32];
   pdl_trigger();
@@ -71,14 +71,14 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
       id = 0;
     }
     src = reinterpret_cast<const T*>(p.embed) + id * W;
-  } else if (p.y && !p.scatter_index) {
+  } else if (!PICK && p.y) {
     src = reinterpret_cast<const T*>(p.y) + t * p.y_stride;
   }
   const T* extra = p.extra ? reinterpret_cast<const T*>(p.extra) + t * p.extra_stride : nullptr;
-  const int* pick = p.scatter_index ? p.scatter_index + t * p.topk : nullptr;
+  const int* pick = PICK ? p.scatter_index + t * p.topk : nullptr;
   float* xrow = p.x + t * (long long)W;
   int pos[8];                  // the token's rows of a mixture, looked up once
-  if (pick)
+  if constexpr (PICK)
 #pragma unroll
     for (int k = 0; k < 8; ++k) pos[k] = k < p.topk ? pick[k] : -1;
   float v[CH][4], x[CH][4], w[CH][4], nw[CH][4];
@@ -104,7 +104,7 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
   for (int c = 0; c < CH; ++c) {
     const int i = (c * blockDim.x + threadIdx.x) * 4;
     if (i >= W) continue;
-    if (pick) {
+    if constexpr (PICK) {
       auto one = [&](int row) {
         if (row >= 0 && row < p.y_rows) add_row(reinterpret_cast<const T*>(p.y) + row * p.y_stride, i, v[c]);
         else if (threadIdx.x == 0 && c == 0) report_status(B200_STATUS_BAD_INDEX, row);
@@ -179,16 +179,16 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
   for (int i = W + threadIdx.x; i < p.xn_cols; i += blockDim.x) orow[i] = from_f32<T>(0.f);
 }
 
-template <typename T>
+template <typename T, bool PICK>
 inline int residual_launch(const ResidualParams& p, long long rows, cudaStream_t st) {
   const int chunks = (p.W + 3) / 4;
   const dim3 g((unsigned)rows);
   int threads = 64;
   while (threads < 256 && chunks > threads) threads <<= 1;
-  if (chunks <= threads) launch_k(residual_step_kernel<T, 1, 256>, g, dim3(threads), 0, st, p);
-  else if (chunks <= 512) launch_k(residual_step_kernel<T, 2, 256>, g, dim3(256), 0, st, p);
-  else if (chunks <= 1024) launch_k(residual_step_kernel<T, 2, 512>, g, dim3(512), 0, st, p);
-  else if (chunks <= 4096) launch_k(residual_step_kernel<T, 4, 1024>, g, dim3(1024), 0, st, p);
+  if (chunks <= threads) launch_k(residual_step_kernel<T, 1, 256, PICK>, g, dim3(threads), 0, st, p);
+  else if (chunks <= 512) launch_k(residual_step_kernel<T, 2, 256, PICK>, g, dim3(256), 0, st, p);
+  else if (chunks <= 1024) launch_k(residual_step_kernel<T, 2, 512, PICK>, g, dim3(512), 0, st, p);
+  else if (chunks <= 4096) launch_k(residual_step_kernel<T, 4, 1024, PICK>, g, dim3(1024), 0, st, p);
   else return B200_ERR_SHAPE;
   return launch_status();
 }
@@ -213,6 +213,8 @@ extern "C" int b200_residual_step(void* x_f32, const void* y, long long y_row_st
   ResidualParams p{(float*)x_f32, y, y_row_stride, y_rows, (const int*)scatter_index_i32, topk, extra, extra_row_stride,
                    embed, (const long long*)ids_i64, vocab, (const int*)rows_i32, num_tokens, (const float*)post_f32,
                    (const float*)add_f32, (const float*)norm_w_f32, eps, xn, xn_row_stride, xn_cols, W, write_back};
-  return dtype == 0 ? residual_launch<__nv_bfloat16>(p, num_rows, (cudaStream_t)stream)
-                    : residual_launch<float>(p, num_rows, (cudaStream_t)stream);
+  const cudaStream_t st = (cudaStream_t)stream;
+  if (scatter_index_i32)
+    return dtype == 0 ? residual_launch<__nv_bfloat16, true>(p, num_rows, st) : residual_launch<float, true>(p, num_rows, st);
+  return dtype == 0 ? residual_launch<__nv_bfloat16, false>(p, num_rows, st) : residual_launch<float, false>(p, num_rows, st);
 }
