@@ -386,7 +386,7 @@ int b200_moe_unpermute_add_rmsnorm(const void* y, const void* scatter_index, con
 
 /* b200_gemm_bf16 with an activation in the epilogue, as one product or a batch of them:
  *   out[g][t, n] = act(sum_k x[g][t, k] * w[g][n, k] + bias[n]).
- * act: 0 none, 1 the tanh form of gelu, 2 times sigmoid(gate[g][t, n]).  bias only with batch = 1.  w_batch_stride is
+ * act: 0 none, 1 the tanh form of gelu, 2 times sigmoid(gate[g][t, n]), 3 the square of relu.  bias only with batch = 1.  w_batch_stride is
  * a multiple of w_row_stride (at least N rows); strides of x and w are multiples of 8.  out_dtype 0 = bf16, 1 = f32. */
 int b200_gemm_bf16_ex(const void* x, const void* w, const void* bias, const void* gate, void* out, long long T, int N,
                       int K, int batch, long long x_row_stride, long long x_batch_stride, long long w_row_stride,
@@ -481,27 +481,45 @@ int b200_latent_gather(const void* cache, void* dst, const void* seq_ids_i32, co
                        key_base_i32, int n, long long rows, int row_bytes, const void* page_table, long long
                        page_table_stride, int max_pages, int page_size, int num_blocks, int num_seqs, void* stream);
 
-/* Grouped-query attention over paged per-head keys and values [blocks, page, kv_heads, DK | DV], no positions in the
- * scores, inside a window (0: none), fp32 weights.  _decode: bf16, tensor cores, sequences with min_len .. max_len new
+/* Grouped-query attention over paged per-head keys and values [blocks, page, kv_heads, DK | DV], fp32 weights; a query sees
+ * a window of its last tokens, its own included, and its chunk floor(position / chunk) (0: no limit).  cap: scores become
+ * cap * tanh(score / cap) (0: none); sink_f32 [heads] (or NULL): exp(sink) joins the denominator; gate rows of the model
+ * dtype: the output is times the sigmoid of one number per head (gate_mode 1) or per column (2), 0: none.  _decode: bf16, tensor cores, sequences with min_len .. max_len new
  * tokens (most_new: the most any brings); DK, DV <= 256, page_size a multiple of 8 that divides 32 or is a multiple of it.
  * _prefill: bf16, tensor cores, the n sequences named, which are all those with at least min_len new tokens; form 0, or 1
  * to keep off the tcgen05 kernel.  _simt: any dims, both dtypes.  q and out rows hold the heads. */
 int b200_window_attn_decode(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void*
                             out, long long out_row_stride, const void* query_start_loc, const void* context_lens,
                             const void* page_table, long long page_table_stride, int max_pages, int page_size, int
-                            num_blocks, int num_seqs, int min_len, int max_len, int most_new, int window, int heads,
-                            int kv_heads, int DK, int DV, float scale, void* stream);
+                            num_blocks, int num_seqs, int min_len, int max_len, int most_new, int window, int chunk,
+                            float cap, const void* sink_f32, const void* gate, long long gate_row_stride, int gate_mode,
+                            int heads, int kv_heads, int DK, int DV, float scale, void* stream);
 int b200_window_attn_prefill(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void*
                              out, long long out_row_stride, const void* query_start_loc, const void* context_lens,
                              const void* page_table, long long page_table_stride, int max_pages, int page_size, int
                              num_blocks, int num_seqs, const void* seq_ids_i32, int n, int max_len, int min_len, int
-                             window, long long T, int heads, int kv_heads, int DK, int DV, float scale, int form,
-                             void* stream);
+                             window, int chunk, float cap, const void* sink_f32, const void* gate, long long
+                             gate_row_stride, int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float
+                             scale, int form, void* stream);
 int b200_window_attn_simt(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void* out,
                           const void* query_start_loc, const void* context_lens, const void* page_table, long long
                           page_table_stride, int max_pages, int page_size, int num_blocks, int num_seqs, int min_len,
-                          int max_len, int window, long long T, int heads, int kv_heads, int DK, int DV, float scale,
-                          int dtype, void* stream);
+                          int max_len, int window, int chunk, float cap, const void* sink_f32, const void* gate, long
+                          long gate_row_stride, int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float
+                          scale, int dtype, void* stream);
+
+/* Between the projections [q: heads * DK | k: kv_heads * DK | ..] and that attention: short convolution of q and k
+ * (conv_w_f32 [taps, (heads + kv_heads) * DK] or NULL; conv_state [num_state_slots, taps - 1, channels] is read and moved
+ * on), values (columns from v_off, or with -1 the convolved keys), norm of q and k (0 none, 1 per head, 2 over all heads; dim
+ * true columns of a head), rotation of the first rot_dims columns (rot_half: pairs (i, i + rot_dims / 2), else (2i, 2i + 1);
+ * cosine and sine times rot_mag); q to q_out [T, heads * DK], k and v to their pages.  one_token_each: no sequence brings
+ * more than one token (one launch; otherwise two with a convolution).  DK <= 1024, rot_dims <= 256. */
+int b200_attn_prep(const void* proj, long long proj_row_stride, int v_off, const void* positions_i64, const void*
+                   slot_mapping_i32, const void* conv_w_f32, void* conv_state, int taps, const void* query_start_loc,
+                   const void* context_lens, const void* state_slots, int num_seqs, int num_state_slots, int
+                   one_token_each, int norm, const void* q_norm_f32, const void* k_norm_f32, int dim, float eps, const
+                   void* inv_freq_f32, int rot_dims, int rot_half, float rot_mag, void* q_out, void* k_cache, void* v_cache,
+                   long long T, int heads, int kv_heads, int DK, int DV, long long num_slots, int dtype, void* stream);
 
 /* Gated delta rule over act rows [q: groups * N | k: groups * N | v: heads * P] (convolved, not yet unit vectors):
  *   S = g S; u = beta (v - S^T k); S += k u^T; o = S^T q,   g = exp(-exp(A_log) dt), beta = sigmoid(b), k and q divided by
@@ -522,12 +540,14 @@ int b200_delta_chunk_scan(const void* act, long long act_row_stride, const void*
 /* One boundary of a residual with a norm on both sides of every sublayer (x [num_tokens, W] fp32, in place):
  *   x <- x + rms_norm(y) * post (+ add);  xn = rms_norm(x) * norm_w (NULL = no xn), columns W .. xn_cols zero.
  * y: rows, or with scatter_index the sum of the token's topk rows of y [y_rows]; extra (or NULL) is added to it.  ids given
- * instead of y: the model starts, x = rms_norm(embed[ids]) * post (+ add).  rows_i32 (with write_back = 0): only these. */
+ * instead of y: the model starts, x = rms_norm(embed[ids] * embed_scale) * post (+ add).  rows_i32 (with write_back = 0):
+ * only these.  post_bias_f32 given: both norms are tanh(alpha v) * weight + bias instead. */
 int b200_residual_step(void* x_f32, const void* y, long long y_row_stride, long long y_rows, const void*
                        scatter_index_i32, int topk, const void* extra, long long extra_row_stride, const void* embed,
                        const void* ids_i64, long long vocab, const void* rows_i32, long long num_tokens, long long
                        num_rows, int W, const void* post_f32, const void* add_f32, const void* norm_w_f32, float eps,
-                       void* xn, long long xn_row_stride, int xn_cols, int write_back, int dtype, void* stream);
+                       float embed_scale, const void* post_bias_f32, float post_alpha, const void* norm_bias_f32, float
+                       norm_alpha, void* xn, long long xn_row_stride, int xn_cols, int write_back, int dtype, void* stream);
 
 /* Gated feed-forwards: act(s g) * (s u) * o with fp32 row factors s = scale_in, o = scale_out (NULL: 1); act 1 silu, 2 the
  * tanh form of gelu.  _gemm_glu: one product, w [2 * n_out, K] gate rows first; _moe_grouped_gemm_glu: expert-sorted rows,
@@ -540,9 +560,22 @@ int b200_moe_grouped_gemm_glu(const void* x, const void* w, const void* scale_in
                               void* stream);
 int b200_glu(const void* gu, long long gu_row_stride, const void* scale_in_f32, const void* scale_out_f32, void* out,
              long long rows, int F, int act, int dtype, void* stream);
-/* Expert-sorted rows in true fp32: out[r] = w[group] x[r]; tile table entries of at most 64 rows. */
-int b200_moe_grouped_gemm_f32(const void* x, const void* w, void* out, const void* tile_table, const void* tile_count,
-                              long long x_rows, int num_groups, int n_out, int K, int max_tiles, void* stream);
+/* Expert-sorted rows with an activation: out[r] = max(w[group] x[r], 0)^2 * scale_out[r] (NULL: 1); act 3. */
+int b200_moe_grouped_gemm_act(const void* x, const void* w, const void* scale_out_f32, void* out, const void* tile_table,
+                              const void* tile_count, long long x_rows, int num_groups, int n_out, int K, long long
+                              out_row_stride, int max_tiles, int tile_rows_max, int act, void* stream);
+/* Expert-sorted rows in true fp32: out[r] = w[group] x[r] (act 0) or as above (act 3); tile table entries of at most 64
+ * rows. */
+int b200_moe_grouped_gemm_f32(const void* x, const void* w, const void* scale_out_f32, void* out, const void* tile_table,
+                              const void* tile_count, long long x_rows, int num_groups, int n_out, int K, int max_tiles,
+                              int act, void* stream);
+/* b200_moe_route_plan_softmax_topk for fp32 weights and a choice inside groups: choice score = score + correction (NULL: 0),
+ * score 0 softmax / 1 sigmoid; a group's score is its largest choice score; only experts of the best `keep` of n_group equal
+ * groups; weights = the chosen scores without the correction (renorm: over their sum). */
+int b200_moe_route_plan_group_topk(const void* logits_f32, long long row_stride, int score, const void* correction_f32, int
+                                   n_group, int keep, void* weights_f32, void* experts_i64, void* rank_i32, void*
+                                   counters_i32, void* cu_seqlens, void* tile_table, void* tile_count, long long T, int E,
+                                   int topk, int renorm, int tile_rows, int max_tiles, void* stream);
 /* b200_moe_route_plan_softmax_topk / b200_moe_scatter_ranked for sigmoid scores and fp32 weights: weights = the chosen
  * scores (renorm: over their sum); gate_f32 [T] or NULL = sigmoid of the logit in column E; rows of row_bytes bytes. */
 int b200_moe_route_plan_sigmoid_topk(const void* logits_f32, long long row_stride, void* weights_f32, void* gate_f32,

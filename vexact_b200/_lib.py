@@ -28,18 +28,23 @@ SIGNATURES = {
     "b200_ssm_conv": [P, LL, I, I, I, I, I, P, P, P, P, P, P, P, P, P, I, I, LL, I, I, P],
     "b200_ssm_scan": [P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P],
     "b200_ssm_gate_norm": [P, LL, P, LL, P, P, LL, LL, I, I, I, I, F, I, I, P],
-    "b200_residual_step": [P, P, LL, LL, P, I, P, LL, P, P, LL, P, LL, LL, I, P, P, P, F, P, LL, I, I, I, P],
+    "b200_residual_step": [P, P, LL, LL, P, I, P, LL, P, P, LL, P, LL, LL, I, P, P, P, F, F, P, F, P, F, P, LL, I, I, I, P],
     "b200_delta_scan": [P, LL, P, P, LL, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P],
     "b200_delta_chunk_scan": [P, LL, P, P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P],
     "b200_latent_prep": [P, LL, P, LL, P, LL, P, I, I, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, F, LL, I, P],
     "b200_latent_attn_simt": [P, P, P, P, P, P, LL, I, I, I, I, I, I, I, LL, I, I, I, F, I, P],
-    "b200_window_attn_simt": [P, LL, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, LL, I, I, I, I, F, I, P],
-    "b200_window_attn_decode": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, I, I, I, I, I, I, I, I, F, P],
-    "b200_window_attn_prefill": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, P, I, I, I, I, LL, I, I, I, I, F, I, P],
+    "b200_window_attn_simt": [P, LL, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, I, F, P, P, LL, I, LL, I, I, I, I, F, I, P],
+    "b200_window_attn_decode": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, I, I, I, I, I, F, P, P, LL, I, I, I, I, I, F, P],
+    "b200_window_attn_prefill": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, P, I, I, I, I, I, F, P, P, LL, I, LL, I, I, I,
+                                 I, F, I, P],
+    "b200_attn_prep": [P, LL, I, P, P, P, P, I, P, P, P, I, I, I, I, P, P, I, F, P, I, I, F, P, P, P, LL, I, I, I, I, LL, I,
+                       P],
     "b200_gemm_glu": [P, P, P, P, LL, I, I, LL, LL, I, P],
     "b200_glu": [P, LL, P, P, P, LL, I, I, I, P],
     "b200_moe_grouped_gemm_glu": [P, P, P, P, P, P, P, LL, I, I, I, LL, I, I, I, P],
-    "b200_moe_grouped_gemm_f32": [P, P, P, P, P, LL, I, I, I, I, P],
+    "b200_moe_grouped_gemm_act": [P, P, P, P, P, P, LL, I, I, I, LL, I, I, I, P],
+    "b200_moe_grouped_gemm_f32": [P, P, P, P, P, P, LL, I, I, I, I, I, P],
+    "b200_moe_route_plan_group_topk": [P, LL, I, P, I, I, P, P, P, P, P, P, P, LL, I, I, I, I, I, P],
     "b200_moe_route_plan_sigmoid_topk": [P, LL, P, P, P, P, P, P, P, P, LL, I, I, I, I, I, P],
     "b200_moe_scatter_ranked_f32": [P, LL, P, P, P, P, P, P, P, LL, I, I, I, P],
     "b200_ssm_chunk_scan": [P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
@@ -103,7 +108,7 @@ class B200Error(RuntimeError):
     pass
 
 
-ABI_VERSION = 6
+ABI_VERSION = 7
 
 
 def _check_fresh(lib) -> None:
@@ -155,7 +160,7 @@ def load() -> C.CDLL:
 
 
 # Kernels launched by one successful call of each entry point (for launch accounting).
-_KERNELS_PER_CALL = {"b200_moe_permute": 2, "b200_lm_head_greedy": 2, "b200_rmsnorm_backward": 3, "b200_ssm_conv2": 2, "b200_latent_attn_tc2": 2, "b200_delta_chunk_scan": 2, "b200_status_read": 0, "b200_abi_version": 0}
+_KERNELS_PER_CALL = {"b200_moe_permute": 2, "b200_lm_head_greedy": 2, "b200_rmsnorm_backward": 3, "b200_ssm_conv2": 2, "b200_latent_attn_tc2": 2, "b200_delta_chunk_scan": 2, "b200_attn_prep2": 2, "b200_status_read": 0, "b200_abi_version": 0}
 _launches = 0
 
 

@@ -95,7 +95,7 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = No
     return out.reshape(*x.shape[:-1], N)
 
 
-GEMM_ACTS = {None: 0, "gelu_tanh": 1, "sigmoid_gate": 2}
+GEMM_ACTS = {None: 0, "gelu_tanh": 1, "sigmoid_gate": 2, "relu2": 3}
 
 
 def gemm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = None, act: str | None = None,
@@ -104,8 +104,8 @@ def gemm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = None
     """act(x @ weight^T + bias) for bf16 (tcgen05) or fp32 (true fp32) tensors, one product or a batch.
 
     One product: x [T, K], weight [N, K] -> [T, N].  Batch (3-D weight [B, N, K]): x [T, B, K] -> [T, B, N]; x, `out`
-    and `gate` may be views with any row and batch stride.  act: None, "gelu_tanh", "sigmoid_gate" (times
-    sigmoid(gate), gate shaped like the output)."""
+    and `gate` may be views with any row and batch stride.  act: None, "gelu_tanh", "relu2" (the square of relu),
+    "sigmoid_gate" (times sigmoid(gate), gate shaped like the output)."""
     _require_cuda("x", x)
     _require_cuda("weight", weight)
     assert x.dtype == weight.dtype, "Incompatible dtypes"

@@ -22,8 +22,8 @@
 // A token therefore gets the same bits from a decode step, a chunk and a full prefill.
 //
 // Exact form (EXACT): the weights are not rounded.  P enters its product as a bf16 pair hi + lo in two tiles (two chains of
-// UMMAs into the same O), the row sum adds the fp32 weights, a query may be limited to a window of keys (blocks before it
-// are not walked), and heads may be narrower than 128 columns (the rest arrives as zeros and is not stored).  The second
+// UMMAs into the same O), the row sum adds the fp32 weights, a query may be limited to a window or chunk of keys (blocks
+// before it are not walked), scores may be capped, the row sum may hold a sink and the output a gate, and heads may be narrower than 128 columns (the rest arrives as zeros and is not stored).  The second
 // P tile takes the place of the second Q buffer.
 //
 // Warps (12): 0 K producer, 1 UMMA issuer + TMEM owner, 2 V producer, 3 Q loader, 4-11 compute: a row is
@@ -384,7 +384,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       const int npos = min(t.pos_per_tile, t.q_len - t.tile_pos0);
       const int pi = row / t.heads_here, hd = row - pi * t.heads_here;
       const int cpos = t.q_abs0 + t.tile_pos0 + (pi < npos ? pi : 0);   // padding rows borrow position 0's mask
-      const uint32_t reach = p.window > 0 ? (uint32_t)p.window : 0x80000000u;   // exact form: 0 <= cpos - key < reach
+      const uint32_t reach = EXACT ? visible_keys(p.window, p.chunk, cpos) : 0;   // visible: 0 <= cpos - key < reach
       float m_run = -INFINITY, l_a = 0.f, l_b = 0.f;   // l of my two key groups (2 half, 2 half + 1)
       float o[64];
 #pragma unroll
@@ -417,6 +417,9 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
             v[i] = __uint_as_float(r0[i]) * p.qk_scale;
             v[32 + i] = __uint_as_float(r1[i]) * p.qk_scale;
           }
+        }
+        if constexpr (EXACT) {
+          if (p.extras.cap > 0.f) cap_scores(v, p.extras.cap);
         }
         if (masked) {
 #pragma unroll
@@ -561,7 +564,29 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         // would touch 32 rows' lines with 16 bytes each.  The warp first lays its 32 half rows down in its own
         // 4 KB of the P tile (idle from the tile's last PV product until this warp's next P write; swizzled), then eight
         // lanes store one row's 128 bytes, four rows per instruction.
-        const float inv = 1.0f / (s_lh[0][row] + s_lh[1][row]);
+        float l_row = s_lh[0][row] + s_lh[1][row];
+        const int head = t.kvh * p.group + t.hchunk * 8 + hd;
+        if constexpr (EXACT) l_row += sink_term(p.extras, head, m_run);
+        float inv = 1.0f / l_row;
+        if constexpr (EXACT) {
+          if (p.extras.gate_mode != GATE_NONE && pi < npos) {
+            const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(p.extras.gate) +
+                                        (long long)(t.q_start + t.tile_pos0 + pi) * p.extras.gate_stride;
+            if (p.extras.gate_mode == GATE_HEAD) {
+              inv *= gate_sigmoid(gate[head]);
+            } else {
+              gate += head * p.dv + half * 64;
+#pragma unroll
+              for (int q = 0; q < 8; ++q) {
+                if (half * 64 + q * 8 >= p.dv) break;
+                const uint4 g8 = *reinterpret_cast<const uint4*>(gate + q * 8);
+                const __nv_bfloat16* ge = reinterpret_cast<const __nv_bfloat16*>(&g8);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) o[q * 8 + k] *= gate_sigmoid(ge[k]);
+              }
+            }
+          }
+        }
         const float inv_heads = 1.0f / (float)t.heads_here;
         const bool vec = ((reinterpret_cast<uintptr_t>(p.out) | (uintptr_t)(p.o_tok_stride * 2) |
                            (uintptr_t)(p.o_head_stride * 2)) & 15) == 0;

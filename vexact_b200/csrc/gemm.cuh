@@ -75,7 +75,7 @@ struct GemmParams {
   const __nv_bfloat16* bias;       // [n_w] or null (plain mode)
   const __nv_bfloat16* row_scale;  // [rows] or null (SwiGLU mode: routing weight of each permuted row)
   // SwiGLU mode with GLU_SILU / GLU_GELU_TANH: out = act(s g) * (s u) * o in fp32 with one rounding, s = scale_in[row],
-  // o = scale_out[row] (null: 1).  GLU_REFERENCE: the rounding points of the fused MoE and row_scale.
+  // o = scale_out[row] (null: 1).  Plain mode: scale_out[row] multiplies after the activation.  GLU_REFERENCE: the rounding points of the fused MoE and row_scale.
   int glu;
   const float* scale_in;
   const float* scale_out;
@@ -102,6 +102,7 @@ constexpr float kLog2e = 1.4426950408889634f;
 constexpr int GEMM_ACT_NONE = 0;
 constexpr int GEMM_ACT_GELU_TANH = 1;     // z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3): the tanh form of gelu
 constexpr int GEMM_ACT_SIGMOID_GATE = 2;  // z * sigmoid(gate)
+constexpr int GEMM_ACT_RELU2 = 3;         // max(z, 0)^2
 
 // Activations of the gated forms (SwiGLU mode of the GEMM and glu_kernel).
 constexpr int GLU_REFERENCE = 0;
@@ -509,6 +510,12 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           if (p.act == GEMM_ACT_GELU_TANH) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gelu_tanh_fast(v[j]);
+          } else if (p.act == GEMM_ACT_RELU2) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) {
+              const float s = p.scale_out && c0 + j < t.n ? p.scale_out[t.row0 + c0 + j] : 1.f, z = fmaxf(v[j], 0.f);
+              v[j] = z * z * s;
+            }
           } else if (gate && fvalid) {
             float e[16];
 #pragma unroll
@@ -767,7 +774,8 @@ gemm_f32_tiled_kernel(const float* __restrict__ x, const float* __restrict__ w, 
                       const float* __restrict__ gate, float* __restrict__ out, long long T, int N, int K,
                       long long x_row, long long x_batch, long long w_row, long long w_batch, long long out_row,
                       long long out_batch, long long gate_row, long long gate_batch, int act,
-                      const int4* __restrict__ tile_table = nullptr, const int* __restrict__ tile_count = nullptr) {
+                      const int4* __restrict__ tile_table, const int* __restrict__ tile_count,
+                      const float* __restrict__ scale_out) {
   pdl_trigger();
   pdl_wait();
   __shared__ float sx[16][68], sw[16][68];
@@ -816,6 +824,7 @@ gemm_f32_tiled_kernel(const float* __restrict__ x, const float* __restrict__ w, 
       if (n >= N) continue;
       float v = acc[i][j] + (bias ? bias[n] : 0.f);
       if (act == GEMM_ACT_GELU_TANH) v = gelu_tanh_exact(v);
+      if (act == GEMM_ACT_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f) * (scale_out ? scale_out[t] : 1.f);
       if (act == GEMM_ACT_SIGMOID_GATE)
         v = v / (1.f + expf(-gate[t * gate_row + (long long)blockIdx.z * gate_batch + n]));
       out[t * out_row + (long long)blockIdx.z * out_batch + n] = v;
@@ -832,14 +841,15 @@ extern "C" int b200_gemm_f32_ex(const void* x, const void* w, const void* bias, 
                                 long long gate_batch_stride, int act, void* stream) {
   using namespace b200;
   if (!x || !w || !out || T < 0 || N <= 0 || K <= 0 || batch < 1) return B200_ERR_ARG;
-  if (act < GEMM_ACT_NONE || act > GEMM_ACT_SIGMOID_GATE) return B200_ERR_ARG;
+  if (act < GEMM_ACT_NONE || act > GEMM_ACT_RELU2) return B200_ERR_ARG;
   if ((act == GEMM_ACT_SIGMOID_GATE) != (gate != nullptr) || (batch > 1 && bias)) return B200_ERR_ARG;
   if (T == 0) return B200_OK;
   if ((T + 63) / 64 > 0x7fffffffLL || (N + 63) / 64 > 65535 || batch > 65535) return B200_ERR_SHAPE;
   launch_k(gemm_f32_tiled_kernel, dim3((unsigned)((T + 63) / 64), (unsigned)((N + 63) / 64), (unsigned)batch), dim3(256),
            0, (cudaStream_t)stream, (const float*)x, (const float*)w, (const float*)bias, (const float*)gate,
            (float*)out, T, N, K, x_row_stride, x_batch_stride, w_row_stride, w_batch_stride, out_row_stride,
-           out_batch_stride, gate_row_stride, gate_batch_stride, act, (const int4*)nullptr, (const int*)nullptr);
+           out_batch_stride, gate_row_stride, gate_batch_stride, act, (const int4*)nullptr, (const int*)nullptr,
+           (const float*)nullptr);
   return launch_status();
 }
 
@@ -974,7 +984,7 @@ extern "C" int b200_gemm_bf16_ex(const void* x, const void* w, const void* bias,
                                  long long out_row_stride, long long out_batch_stride, long long gate_row_stride,
                                  long long gate_batch_stride, int act, int out_dtype, void* stream) {
   using namespace b200;
-  if (batch < 1 || act < GEMM_ACT_NONE || act > GEMM_ACT_SIGMOID_GATE) return B200_ERR_ARG;
+  if (batch < 1 || act < GEMM_ACT_NONE || act > GEMM_ACT_RELU2) return B200_ERR_ARG;
   if ((act == GEMM_ACT_SIGMOID_GATE) != (gate != nullptr) || (batch > 1 && bias)) return B200_ERR_ARG;
   GemmExtra ex;
   ex.act = act;
@@ -1106,7 +1116,8 @@ inline int moe_grouped_gemm_impl(const void* x, long long x_rows, long long x_ro
                                  const void* w, const void* row_scale, void* out, const void* tile_table,
                                  const void* tile_count, int num_groups, int n_out, int K, long long out_row_stride,
                                  int max_tiles, int tile_rows_max, int mode, void* stream, int glu = GLU_REFERENCE,
-                                 const void* scale_in = nullptr, const void* scale_out = nullptr) {
+                                 const void* scale_in = nullptr, const void* scale_out = nullptr,
+                                 int act = GEMM_ACT_NONE) {
   if (!x || !w || !out || !tile_table || !tile_count || x_rows < 0 || num_groups <= 0 || n_out <= 0 || K <= 0 ||
       max_tiles < 0 || (mode != 0 && mode != 1))
     return B200_ERR_ARG;
@@ -1137,6 +1148,7 @@ inline int moe_grouped_gemm_impl(const void* x, long long x_rows, long long x_ro
   p.glu = glu;
   p.scale_in = (const float*)scale_in;
   p.scale_out = (const float*)scale_out;
+  p.act = act;
   p.w_policy = ptx::kEvictFirst;
   CUtensorMap tw, tx;
   int rc = make_tmap_2d(&tw, w, (uint64_t)num_groups * p.w_rows_per_group, (uint64_t)K, (uint64_t)K,
@@ -1185,7 +1197,19 @@ extern "C" int b200_moe_grouped_gemm_glu(const void* x, const void* w, const voi
                                      out_row_stride, max_tiles, tile_rows_max, 1, stream, act, scale_in_f32, scale_out_f32);
 }
 
-// One product of the same form over T rows as they lie (no tile table): w [2 * n_out, K].
+// The grouped GEMM with an activation of the plain epilogue: out[r, n] = max(x[r] . w[group, n], 0)^2 * o, o =
+// scale_out[r] (NULL: 1); act: 3.  w [groups, n_out, K].
+extern "C" int b200_moe_grouped_gemm_act(const void* x, const void* w, const void* scale_out_f32, void* out,
+                                         const void* tile_table, const void* tile_count, long long x_rows, int num_groups,
+                                         int n_out, int K, long long out_row_stride, int max_tiles, int tile_rows_max,
+                                         int act, void* stream) {
+  if (act != b200::GEMM_ACT_RELU2) return B200_ERR_ARG;
+  return b200::moe_grouped_gemm_impl(x, x_rows, K, nullptr, w, nullptr, out, tile_table, tile_count, num_groups, n_out, K,
+                                     out_row_stride, max_tiles, tile_rows_max, 0, stream, b200::GLU_REFERENCE, nullptr,
+                                     scale_out_f32, act);
+}
+
+// One product of the gated form over T rows as they lie (no tile table): w [2 * n_out, K].
 extern "C" int b200_gemm_glu(const void* x, const void* w, const void* scale_out_f32, void* out, long long T, int n_out,
                              int K, long long x_row_stride, long long out_row_stride, int act, void* stream) {
   using namespace b200;
@@ -1216,19 +1240,21 @@ extern "C" int b200_gemm_glu(const void* x, const void* w, const void* scale_out
   return gemm_launch<GEMM_SWIGLU>(tw, tx, p, (long long)p.w_tiles * p.dense_t_tiles, (cudaStream_t)stream);
 }
 
-// The grouped GEMM in true fp32: out[r, n] = x[r] . w[group, n]; tile table entries of at most 64 rows.
-extern "C" int b200_moe_grouped_gemm_f32(const void* x, const void* w, void* out, const void* tile_table,
-                                         const void* tile_count, long long x_rows, int num_groups, int n_out, int K,
-                                         int max_tiles, void* stream) {
+// The grouped GEMM in true fp32: out[r, n] = x[r] . w[group, n], with act 3 as b200_moe_grouped_gemm_act; tile table
+// entries of at most 64 rows.
+extern "C" int b200_moe_grouped_gemm_f32(const void* x, const void* w, const void* scale_out_f32, void* out,
+                                         const void* tile_table, const void* tile_count, long long x_rows, int num_groups,
+                                         int n_out, int K, int max_tiles, int act, void* stream) {
   using namespace b200;
-  if (!x || !w || !out || !tile_table || !tile_count || x_rows < 0 || num_groups <= 0 || n_out <= 0 || K <= 0 || max_tiles < 0)
+  if (!x || !w || !out || !tile_table || !tile_count || x_rows < 0 || num_groups <= 0 || n_out <= 0 || K <= 0 || max_tiles < 0 ||
+      (act != GEMM_ACT_NONE && act != GEMM_ACT_RELU2) || (scale_out_f32 && act == GEMM_ACT_NONE))
     return B200_ERR_ARG;
   if (x_rows == 0 || max_tiles == 0) return B200_OK;
   if ((n_out + 63) / 64 > 65535) return B200_ERR_SHAPE;
   launch_k(gemm_f32_tiled_kernel, dim3((unsigned)max_tiles, (unsigned)((n_out + 63) / 64), 1u), dim3(256), 0,
            (cudaStream_t)stream, (const float*)x, (const float*)w, (const float*)nullptr, (const float*)nullptr,
            (float*)out, x_rows, n_out, K, (long long)K, 0LL, (long long)K, (long long)n_out * K, (long long)n_out, 0LL, 0LL,
-           0LL, GEMM_ACT_NONE, (const int4*)tile_table, (const int*)tile_count);
+           0LL, act, (const int4*)tile_table, (const int*)tile_count, (const float*)scale_out_f32);
   return launch_status();
 }
 

@@ -13,8 +13,10 @@
 //   latent_gather_kernel  the latents of a sequence (from the first a window reaches), gathered from their pages into
 //                         packed rows (what the expanded form of long prompts projects up).
 //
-// A window of w tokens (0: none) means that position i sees the keys i - w + 1 .. i.
+// A window of w tokens (0: none) means that position i sees the keys i - w + 1 .. i.  The CUDA-core kernel also takes the
+// chunks, capped scores, sinks and gates of attn_extras.cuh.
 #pragma once
+#include "attn_extras.cuh"
 #include "hyper.cuh"   // load4 / store4 / to_f32 / from_f32
 
 namespace b200 {
@@ -157,6 +159,7 @@ struct LatentSeqs {
   int max_pages, page_size, num_blocks, num_seqs;
   int min_len, max_len;         // only sequences whose step brings min_len .. max_len tokens
   int window;                   // tokens a position sees, its own included; 0: every earlier one
+  int chunk;                    // tokens of a chunk beyond which nothing is seen; 0: none
 };
 
 // First position a query at `pos` sees.
@@ -194,6 +197,7 @@ struct AttnSimtParams {
   int k_row, v_row;
   int heads, group, DK, DV;
   float scale;
+  AttnExtras extras;
 };
 
 constexpr int LATENT_SIMT_THREADS = 128;
@@ -216,7 +220,7 @@ __global__ void __launch_bounds__(LATENT_SIMT_THREADS) attn_simt_kernel(const At
   const int t0 = p.seqs.query_start_loc[s], len = p.seqs.query_start_loc[s + 1] - t0;
   if (t < t0 || t >= t0 + len || len < p.seqs.min_len || len > p.seqs.max_len) return;
   const int pos = p.seqs.context_lens[s] - len + (int)(t - t0);
-  const int keys = pos + 1, kv_head = h / p.group;   // visible keys: positions window_first .. own
+  const int keys = pos + 1, kv_head = h / p.group;   // visible keys: positions first_visible .. own
   const T* q = reinterpret_cast<const T*>(p.q) + t * p.q_row + (long long)h * p.DK;
   for (int i = tid; i < p.DK; i += LATENT_SIMT_THREADS) lat_smem[i] = to_f32(q[i]) * p.scale;
   float acc[LATENT_SIMT_VPT];
@@ -225,7 +229,7 @@ __global__ void __launch_bounds__(LATENT_SIMT_THREADS) attn_simt_kernel(const At
   float m = -INFINITY, l = 0.f;
   const T* kbase = reinterpret_cast<const T*>(p.k) + kv_head * p.DK;
   const T* vbase = reinterpret_cast<const T*>(p.v) + kv_head * p.DV;
-  for (int b = window_first(p.seqs.window, pos); b < keys; b += LATENT_SIMT_THREADS) {
+  for (int b = first_visible(p.seqs.window, p.seqs.chunk, pos); b < keys; b += LATENT_SIMT_THREADS) {
     const int n = min(LATENT_SIMT_THREADS, keys - b);
     __syncthreads();
     long long row = tid < n ? latent_key_row(p.seqs, s, b + tid) : -1;
@@ -240,7 +244,7 @@ __global__ void __launch_bounds__(LATENT_SIMT_THREADS) attn_simt_kernel(const At
 #pragma unroll
         for (int u = 0; u < 4; ++u) a = fmaf(lat_smem[i + u], v[u], a);
       }
-      sc = a;
+      sc = p.extras.cap > 0.f ? p.extras.cap * tanhf(a / p.extras.cap) : a;
     }
     const float bm = fmaxf(m, block_max(sc, red));
     const float e = sc == -INFINITY ? 0.f : expf(sc - bm);
@@ -260,11 +264,16 @@ __global__ void __launch_bounds__(LATENT_SIMT_THREADS) attn_simt_kernel(const At
       }
     }
   }
+  if (p.extras.sink) l += expf(p.extras.sink[h] - m);
+  const T* gate = p.extras.gate ? reinterpret_cast<const T*>(p.extras.gate) + t * p.extras.gate_stride : nullptr;
   T* out = reinterpret_cast<T*>(p.out) + (t * p.heads + h) * (long long)p.DV;
 #pragma unroll
   for (int v = 0; v < LATENT_SIMT_VPT; ++v) {
     const int c = v * LATENT_SIMT_THREADS + tid;
-    if (c < p.DV) out[c] = from_f32<T>(l > 0.f ? acc[v] / l : 0.f);
+    if (c >= p.DV) continue;
+    float o = l > 0.f ? acc[v] / l : 0.f;
+    if (gate) o *= gate_sigmoid<T>(gate[p.extras.gate_mode == GATE_HEAD ? h : h * p.DV + c]);
+    out[c] = from_f32<T>(o);
   }
 }
 
@@ -328,7 +337,7 @@ inline bool latent_seqs_ok(const LatentSeqs& q) {
 namespace b200 {
 inline int attn_simt_launch(AttnSimtParams& p, long long T, int dtype, cudaStream_t st) {
   if (!latent_seqs_ok(p.seqs) || !p.q || !p.k || !p.v || !p.out || T < 0 || p.heads <= 0 || p.group <= 0 || p.DK <= 0 ||
-      p.DV <= 0 || p.seqs.window < 0 || (dtype != 0 && dtype != 1))
+      p.DV <= 0 || p.seqs.window < 0 || p.seqs.chunk < 0 || !attn_extras_ok(p.extras) || (dtype != 0 && dtype != 1))
     return B200_ERR_ARG;
   if (p.heads % p.group || p.DK % 8 || p.DV % 8 || p.k_row % 8 || p.v_row % 8 || p.heads > 65535 ||
       p.DV > LATENT_SIMT_THREADS * LATENT_SIMT_VPT || p.DK > 8192 || T > 0x7fffffffLL)
@@ -359,14 +368,16 @@ extern "C" int b200_latent_attn_simt(const void* q_lat, const void* cache, void*
 extern "C" int b200_window_attn_simt(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache,
                                      void* out, const void* query_start_loc, const void* context_lens,
                                      const void* page_table, long long page_table_stride, int max_pages, int page_size,
-                                     int num_blocks, int num_seqs, int min_len, int max_len, int window, long long T,
-                                     int heads, int kv_heads, int DK, int DV, float scale, int dtype, void* stream) {
+                                     int num_blocks, int num_seqs, int min_len, int max_len, int window, int chunk,
+                                     float cap, const void* sink_f32, const void* gate, long long gate_row_stride,
+                                     int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float scale,
+                                     int dtype, void* stream) {
   using namespace b200;
   if (kv_heads <= 0 || heads % kv_heads) return B200_ERR_ARG;
   AttnSimtParams p{{(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride,
-                    max_pages, page_size, num_blocks, num_seqs, min_len, max_len, window},
+                    max_pages, page_size, num_blocks, num_seqs, min_len, max_len, window, chunk},
                    q, k_cache, v_cache, out, q_row_stride, kv_heads * DK, kv_heads * DV, heads, heads / kv_heads, DK, DV,
-                   scale};
+                   scale, {cap, (const float*)sink_f32, gate, gate_row_stride, gate_mode}};
   return attn_simt_launch(p, T, dtype, (cudaStream_t)stream);
 }
 

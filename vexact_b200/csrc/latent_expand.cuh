@@ -1,5 +1,5 @@
-// Causal attention of long portions of prompts over per-head keys and values (bf16), optionally inside a window.  Two
-// sources of keys:
+// Causal attention of long portions of prompts over per-head keys and values (bf16), optionally inside a window or chunk.
+// Two sources of keys:
 //
 //   expanded latents   the latents of a sequence's context (from the first key the window reaches) have been gathered from
 //                      their pages and projected up: packed kv rows [keys: G * DN | values: G * DV], and lat rows
@@ -7,7 +7,7 @@
 //   paged heads        k and v rows of a paged cache, [G * DN] and [G * DV] (DR = 0)
 //
 //   q         [T, q_stride]: per head DN unrotated, then DR rotated columns; head h uses key / value head h / group
-//   out[t, h] = sum_j softmax(scale q.k_j) v_j, times sigmoid(gate[t, h]) when there is a gate
+//   out[t, h] = sum_j softmax(scale q.k_j) v_j, with the chunks, cap, sink and gate of attn_extras.cuh
 //
 // One CTA per (128 MT queries, head, sequence); warp w of 8 owns query rows 16 MT w .. 16 MT (w + 1) - 1 (MT = 2 for long
 // portions: every key and value fragment read from shared memory then serves two products); 64 keys per block, double
@@ -31,11 +31,11 @@ struct LatentExpandParams {
   const __nv_bfloat16* k;      // rows k_stride apart, head g at column g * DN
   const __nv_bfloat16* v;      // rows v_stride apart, head g at column g * DV
   const __nv_bfloat16* rot;    // rows rot_stride apart: the shared rotated part (DR > 0)
-  const __nv_bfloat16* gate;   // or null
   __nv_bfloat16* out;
-  long long q_stride, k_stride, v_stride, rot_stride, gate_stride, out_stride;
+  long long q_stride, k_stride, v_stride, rot_stride, out_stride;
   int heads, group, DN, DR, DV;
   float scale_log2;
+  AttnExtras extras;
 };
 
 template <int DK, int DV, int MT>
@@ -59,7 +59,6 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   if ((int)blockIdx.x >= tiles) return;
   const int row_base = (tiles - 1 - (int)blockIdx.x) * LEX_BM;
   const int keys = p.seqs.context_lens[seq], past = keys - len;
-  const int window = p.seqs.window > 0 ? p.seqs.window : 0x3fffffff;
   const int key_base = PAGED ? 0 : p.key_base[i];
   const long long key0 = PAGED ? 0 : p.key_start[i] - key_base;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
@@ -67,7 +66,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   const int dk16 = (p.DN + p.DR + 15) / 16;
   const int rows = min(LEX_BM, len - row_base);
   const int last_key = min(keys, past + row_base + rows);       // keys any row of the tile sees
-  const int first_key = window_first(window, past + row_base);
+  const int first_key = first_visible(p.seqs.window, p.seqs.chunk, past + row_base);
   const int block0 = first_key / LEX_BN, blocks = (last_key + LEX_BN - 1) / LEX_BN;
 
   for (int e = tid; e < LEX_BM * (DK / 8); e += LEX_THREADS) {
@@ -122,6 +121,16 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   }
   const int r0 = 16 * MT * warp;
   const int first_pos = past + row_base + r0;                    // position of the warp's first row
+  const int warp_first = first_visible(p.seqs.window, p.seqs.chunk, first_pos);                 // no row sees keys before this
+  const int warp_full = first_visible(p.seqs.window, p.seqs.chunk, first_pos + 16 * MT - 1);    // every row sees from here
+  int row_pos[MT];                                               // position of row g4 of the tile (and + 8)
+  uint32_t reach[MT][2];                                         // a row sees 0 <= its position - key < reach
+#pragma unroll
+  for (int t = 0; t < MT; ++t) {
+    row_pos[t] = first_pos + 16 * t + g4;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) reach[t][e] = visible_keys(p.seqs.window, p.seqs.chunk, row_pos[t] + 8 * e);
+  }
   for (int b = block0; b < blocks; ++b) {
     if (b + 1 < blocks) {
       load(b + 1);
@@ -135,7 +144,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
     for (int sub = 0; sub < LEX_BN / LEX_SUB; ++sub) {
       const int base = b * LEX_BN + sub * LEX_SUB;
       if (r0 >= rows || base > first_pos + 16 * MT - 1) break;   // no row of this warp sees these keys
-      if (base + LEX_SUB - 1 <= first_pos - window) continue;   // nor these, before every row's window
+      if (base + LEX_SUB - 1 < warp_first) continue;             // nor these, before every row's window or chunk
       float s[MT][NS][4];
 #pragma unroll
       for (int t = 0; t < MT; ++t)
@@ -157,17 +166,22 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
         }
       }
       // some (row, key) of these is masked
-      const bool edge = base + LEX_SUB - 1 > first_pos || base <= first_pos + 16 * MT - 1 - window;
+      const bool edge = base + LEX_SUB - 1 > first_pos || base < warp_full;
 #pragma unroll
       for (int t = 0; t < MT; ++t) {
-        const int pos0 = first_pos + 16 * t + g4;                 // position of row g4 of the tile (and + 8)
         float mb[2] = {m[t][0], m[t][1]};
+#pragma unroll
+        for (int j = 0; j < NS; ++j) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[t][j][e] *= p.scale_log2;
+          if (p.extras.cap > 0.f) cap_scores(s[t][j], p.extras.cap);
+        }
 #pragma unroll
         for (int j = 0; j < NS; ++j)
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            float v = s[t][j][e] * p.scale_log2;
-            if (edge && (uint32_t)(pos0 + 8 * (e >> 1) - (base + 8 * j + 2 * t4 + (e & 1))) >= (uint32_t)window) v = -INFINITY;   // a row sees 0 <= its position - key < window
+            float v = s[t][j][e];
+            if (edge && (uint32_t)(row_pos[t] + 8 * (e >> 1) - (base + 8 * j + 2 * t4 + (e & 1))) >= reach[t][e >> 1]) v = -INFINITY;
             s[t][j][e] = v;
             mb[e >> 1] = fmaxf(mb[e >> 1], v);
           }
@@ -234,20 +248,20 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   for (int tt = 0; tt < MT; ++tt)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      const float inv = 1.f / abm_quad_sum(l[tt][e]);
+      float inv = 1.f / (abm_quad_sum(l[tt][e]) + sink_term(p.extras, h, m[tt][e]));
       const int r = r0 + 16 * tt + g4 + 8 * e;
       if (r >= rows) continue;
       const long long t = t0 + row_base + r;
+      const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(p.extras.gate) + t * p.extras.gate_stride;
+      if (p.extras.gate_mode == GATE_HEAD) inv *= gate_sigmoid(gate[h]);
 #pragma unroll
       for (int j = 0; j < DV / 8; ++j) {
         const int c = 8 * j + 2 * t4;
         if (c < p.DV) {
           float a = o[tt][j][2 * e] * inv, b = o[tt][j][2 * e + 1] * inv;
-          if (p.gate) {
-            float ga, gb;
-            unpack_bf2(*reinterpret_cast<const uint32_t*>(p.gate + t * p.gate_stride + (long long)h * p.DV + c), ga, gb);
-            a *= __fdividef(1.f, 1.f + __expf(-ga));
-            b *= __fdividef(1.f, 1.f + __expf(-gb));
+          if (p.extras.gate_mode == GATE_COLUMN) {
+            a *= gate_sigmoid(gate[h * p.DV + c]);
+            b *= gate_sigmoid(gate[h * p.DV + c + 1]);
           }
           *reinterpret_cast<uint32_t*>(p.out + t * p.out_stride + (long long)h * p.DV + c) = pack_bf2(a, b);
         }
@@ -309,12 +323,11 @@ extern "C" int b200_latent_attn_expanded(const void* q, long long q_row_stride, 
   p.k = (const __nv_bfloat16*)kv;
   p.v = (const __nv_bfloat16*)kv + (long long)heads * DN;
   p.rot = (const __nv_bfloat16*)lat + rot_off;
-  p.gate = (const __nv_bfloat16*)gate;
   p.out = (__nv_bfloat16*)out;
   p.q_stride = q_row_stride;
   p.k_stride = p.v_stride = kv_row_stride;
   p.rot_stride = lat_row_stride;
-  p.gate_stride = gate_row_stride;
+  p.extras = {0.f, nullptr, gate, gate_row_stride, gate ? GATE_COLUMN : GATE_NONE};
   p.out_stride = out_row_stride;
   p.heads = heads;
   p.group = 1;

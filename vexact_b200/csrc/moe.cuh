@@ -107,6 +107,106 @@ __device__ __forceinline__ void route_softmax_topk_token(const TIn* __restrict__
   }
 }
 
+// The best of v over the warp's lanes and their entries e = lane, lane + 32, ... < n; the lowest index on ties.
+__device__ __forceinline__ int warp_argmax_shared(const float* v, int n, int lane) {
+  float bv = -INFINITY;
+  int be = 0x7fffffff;
+  for (int e = lane; e < n; e += 32)
+    if (v[e] > bv || be == 0x7fffffff) {
+      bv = v[e];
+      be = e;
+    }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+    const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+    if (ov > bv || (ov == bv && oe < be)) {
+      bv = ov;
+      be = oe;
+    }
+  }
+  return be;
+}
+
+// Scores -> choice scores (score + correction) -> best groups -> top-k of one token by one warp.  Scores: softmax over the
+// experts, or each one's sigmoid.  A group's score is its largest choice score; experts outside the best `keep` of the
+// n_group equal groups cannot be chosen.  Weights are the chosen experts' scores without the correction (renorm: over
+// their sum).  choice, group: scratch of E and n_group floats; score of E.
+__device__ __forceinline__ void route_group_topk_token(const float* __restrict__ row, long long tok, bool sigmoid,
+                                                       const float* __restrict__ correction, int n_group, int keep,
+                                                       float* score, float* choice, float* group,
+                                                       float* __restrict__ w_f32, long long* __restrict__ idx_i64, int E,
+                                                       int topk, int renorm, int lane) {
+  float mx = -INFINITY, sum = 0.f;
+  if (!sigmoid) {
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, row[e]);
+    mx = warp_max(mx);
+    for (int e = lane; e < E; e += 32) sum += score[e] = expf(row[e] - mx);
+    sum = warp_sum(sum);
+  }
+  for (int e = lane; e < E; e += 32) {
+    float s = sigmoid ? 1.f / (1.f + expf(-row[e])) : score[e] / sum;
+    if (!(s == s)) s = 0.f;      // NaN logits of a padded token still have to name experts
+    const float c = s + (correction ? correction[e] : 0.f);
+    score[e] = s;
+    choice[e] = c == c ? c : 0.f;
+  }
+  __syncwarp();
+  const int size = E / n_group;
+  if (keep < n_group) {
+    for (int g = lane; g < n_group; g += 32) {
+      float best = choice[g * size];
+      for (int j = 1; j < size; ++j) best = fmaxf(best, choice[g * size + j]);
+      group[g] = best;
+    }
+    __syncwarp();
+    for (int r = 0; r < n_group - keep; ++r) {
+      // the worst group left goes: highest index on ties, so that the lower ones stay
+      float wv = INFINITY;
+      int wg = -1;
+      for (int g = lane; g < n_group; g += 32)
+        if (group[g] <= wv) {
+          wv = group[g];
+          wg = g;
+        }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, wv, o);
+        const int og = __shfl_xor_sync(0xffffffffu, wg, o);
+        if (ov < wv || (ov == wv && og > wg)) {
+          wv = ov;
+          wg = og;
+        }
+      }
+      if (wg >= 0) {
+        for (int j = lane; j < size; j += 32) choice[wg * size + j] = -INFINITY;
+        if (lane == 0) group[wg] = INFINITY;
+      }
+      __syncwarp();
+    }
+  }
+  float denom = 1.f, w = 0.f;
+  int chosen = 0;
+  if (renorm) denom = 0.f;
+  for (int k = 0; k < topk; ++k) {
+    int e = warp_argmax_shared(choice, E, lane);
+    if (e < 0 || e >= E) e = 0;   // unreachable for topk <= keep * size
+    const float s = score[e];
+    if (renorm) denom += s;
+    if (lane == k) {
+      w = s;
+      chosen = e;
+    }
+    __syncwarp();
+    if (lane == 0) choice[e] = -INFINITY;
+    __syncwarp();
+  }
+  if (lane < topk) {
+    w_f32[tok * topk + lane] = w / denom;
+    idx_i64[tok * topk + lane] = chosen;
+  }
+}
+
 // One warp per token.
 template <typename TIn>
 __global__ void __launch_bounds__(256)
@@ -839,22 +939,34 @@ extern "C" int b200_moe_route_softmax_topk(const void* logits, int logits_dtype 
 // (it is what reproduces the reference's index arrays).
 namespace b200 {
 
+// Choice of experts inside their best groups (route_group_topk_token); n_group 0: the plain top-k.
+struct RouteGroups {
+  const float* correction;
+  int n_group, keep, sigmoid;
+};
+
 // gate_f32: sigmoid of the logit in column E (a gate that shares the router's product), or null.
-template <typename TIn, bool SIGMOID = false>
+template <typename TIn, bool SIGMOID = false, bool GROUPS = false>
 __global__ void __launch_bounds__(256)
 moe_route_plan_kernel(const TIn* __restrict__ logits, long long row_stride, __nv_bfloat16* __restrict__ w_bf16,
                       float* __restrict__ w_f32, float* __restrict__ gate_f32, long long* __restrict__ idx_i64, int* __restrict__ rank_out, int* __restrict__ counters,
                       int* __restrict__ cu_seqlens, int4* __restrict__ tile_table, int* __restrict__ tile_count,
-                      long long T, int E, int topk, int renorm, int tile_rows, int max_tiles) {
+                      long long T, int E, int topk, int renorm, int tile_rows, int max_tiles, const RouteGroups groups) {
   pdl_trigger();
   pdl_wait();
   __shared__ int s_last;
   __shared__ int s_scan[2][8];
+  __shared__ float s_route[GROUPS ? 8 : 1][GROUPS ? 3 * MOE_MAX_EXPERTS : 1];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const long long tok = (long long)blockIdx.x * 8 + warp;
   if (tok < T) {
-    route_softmax_topk_token<TIn, SIGMOID>(logits + tok * row_stride, tok, w_bf16, w_f32, nullptr, idx_i64, E, topk,
-                                           renorm, lane);
+    if constexpr (GROUPS)
+      route_group_topk_token(logits + tok * row_stride, tok, groups.sigmoid != 0, groups.correction, groups.n_group,
+                             groups.keep, s_route[warp], s_route[warp] + MOE_MAX_EXPERTS,
+                             s_route[warp] + 2 * MOE_MAX_EXPERTS, w_f32, idx_i64, E, topk, renorm, lane);
+    else
+      route_softmax_topk_token<TIn, SIGMOID>(logits + tok * row_stride, tok, w_bf16, w_f32, nullptr, idx_i64, E, topk,
+                                             renorm, lane);
     if (gate_f32 && lane == 0) gate_f32[tok] = 1.f / (1.f + expf(-(float)logits[tok * row_stride + E]));
     __syncwarp();
     // the expert ids were just written by lane 0: lane k takes entry k's rank in its expert's group
@@ -969,11 +1081,12 @@ extern "C" int b200_moe_route_plan_softmax_topk(const void* logits, int logits_d
     launch_k(moe_route_plan_kernel<float>, dim3(grid), dim3(256), 0, st, (const float*)logits, row_stride,
              (__nv_bfloat16*)weights_bf16, (float*)nullptr, (float*)nullptr, (long long*)experts_i64, (int*)rank_i32,
              (int*)counters_i32,
-             (int*)cu_seqlens, (int4*)tile_table, (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles);
+             (int*)cu_seqlens, (int4*)tile_table, (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles, RouteGroups{});
   else if (logits_dtype == 1)
     launch_k(moe_route_plan_kernel<__nv_bfloat16>, dim3(grid), dim3(256), 0, st, (const __nv_bfloat16*)logits,
              row_stride, (__nv_bfloat16*)weights_bf16, (float*)nullptr, (float*)nullptr, (long long*)experts_i64,
-             (int*)rank_i32, (int*)counters_i32, (int*)cu_seqlens, (int4*)tile_table, (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles);
+             (int*)rank_i32, (int*)counters_i32, (int*)cu_seqlens, (int4*)tile_table, (int*)tile_count, T, E, topk, renorm,
+             tile_rows, max_tiles, RouteGroups{});
   else
     return B200_ERR_ARG;
   return launch_status();
@@ -1014,7 +1127,31 @@ extern "C" int b200_moe_route_plan_sigmoid_topk(const void* logits_f32, long lon
   launch_k(moe_route_plan_kernel<float, true>, dim3((unsigned)((T + 7) / 8)), dim3(256), 0, (cudaStream_t)stream,
            (const float*)logits_f32, row_stride, (__nv_bfloat16*)nullptr, (float*)weights_f32, (float*)gate_f32,
            (long long*)experts_i64, (int*)rank_i32, (int*)counters_i32, (int*)cu_seqlens, (int4*)tile_table,
-           (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles);
+           (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles, RouteGroups{});
+  return launch_status();
+}
+
+// The same for routers that choose inside groups: choice score = score + correction (or NULL), a group's score its largest
+// choice score, only experts of the best `keep` of n_group equal groups of neighbours; weights are the chosen scores
+// without the correction.  score: 0 softmax over all experts, 1 each one's sigmoid.
+extern "C" int b200_moe_route_plan_group_topk(const void* logits_f32, long long row_stride, int score,
+                                              const void* correction_f32, int n_group, int keep, void* weights_f32,
+                                              void* experts_i64, void* rank_i32, void* counters_i32, void* cu_seqlens,
+                                              void* tile_table, void* tile_count, long long T, int E, int topk, int renorm,
+                                              int tile_rows, int max_tiles, void* stream) {
+  using namespace b200;
+  if (!logits_f32 || !weights_f32 || !experts_i64 || !rank_i32 || !counters_i32 || !cu_seqlens || !tile_table ||
+      !tile_count || T <= 0 || E <= 0 || topk <= 0 || tile_rows <= 0 || max_tiles <= 0 || (score != 0 && score != 1) ||
+      n_group <= 0 || keep <= 0)
+    return B200_ERR_ARG;
+  if (E > MOE_MAX_EXPERTS || topk > MOE_MAX_TOPK || E % n_group || keep > n_group || topk > keep * (E / n_group) ||
+      row_stride < E)
+    return B200_ERR_SHAPE;
+  launch_k(moe_route_plan_kernel<float, false, true>, dim3((unsigned)((T + 7) / 8)), dim3(256), 0, (cudaStream_t)stream,
+           (const float*)logits_f32, row_stride, (__nv_bfloat16*)nullptr, (float*)weights_f32, (float*)nullptr,
+           (long long*)experts_i64, (int*)rank_i32, (int*)counters_i32, (int*)cu_seqlens, (int4*)tile_table,
+           (int*)tile_count, T, E, topk, renorm, tile_rows, max_tiles,
+           RouteGroups{(const float*)correction_f32, n_group, keep, score});
   return launch_status();
 }
 

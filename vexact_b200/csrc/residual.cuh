@@ -9,8 +9,14 @@
 //
 // One CTA per token, everything in registers between the two reductions.  `rows` picks tokens at the end of a model;
 // nothing is written back then.
+//
+// The norms may be dynamic tanh instead, tanh(alpha x) * w + b with one number alpha, which reduces nothing:
+//     x <- x + tanh(post_alpha y) * post + post_bias (+ add),    xn = tanh(norm_alpha x) * norm + norm_bias
+// A thread then owns four columns of a few tokens and keeps the norms' vectors in registers.  At the start of a model y is
+// the embedding row times embed_scale, under either norm.
 // Algorithmic bytes per token: 8 W (x) + b W (topk + shared rows of y) + b W (xn), b = 2 or 4: HBM bandwidth.
 #pragma once
+#include "attn_extras.cuh"   // tanh_as
 #include "hyper.cuh"   // load4 / store4 / to_f32 / from_f32
 
 namespace b200 {
@@ -37,6 +43,12 @@ struct ResidualParams {
   int xn_cols;
   int W;
   int write_back;
+  long long num_rows;
+  float embed_scale;
+  // dynamic tanh (residual_tanh_kernel)
+  const float* post_bias;     // [W]
+  const float* norm_bias;     // [W]
+  float post_alpha, norm_alpha;
 };
 
 template <typename T>
@@ -90,7 +102,12 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
     for (int k = 0; k < 4; ++k) v[c][k] = x[c][k] = w[c][k] = nw[c][k] = 0.f;
     if (i >= W) continue;
     if (src) get(src, i, v[c]);
-    if (!p.ids) get(xrow, i, x[c]);
+    if (p.ids) {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[c][k] *= p.embed_scale;
+    } else {
+      get(xrow, i, x[c]);
+    }
     get(p.post, i, w[c]);
     if (p.norm_w) get(p.norm_w, i, nw[c]);
   }
@@ -179,8 +196,131 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
   for (int i = W + threadIdx.x; i < p.xn_cols; i += blockDim.x) orow[i] = from_f32<T>(0.f);
 }
 
+// The boundary under dynamic tanh.  A thread owns four neighbouring columns of ROWS tokens.
+template <typename T, int ROWS, bool PICK>
+__global__ void __launch_bounds__(128) residual_tanh_kernel(const ResidualParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int W = p.W, i = (blockIdx.y * 128 + threadIdx.x) * 4;
+  const bool vec = W % 4 == 0;
+  auto get = [&](const auto* row, float (&v)[4]) {
+    if (vec) load4(row + i, v);
+    else load4_tail(row + i, W - i, v);
+  };
+  const long long r0 = (long long)blockIdx.x * ROWS;
+  if (i >= W) {                // columns past the width: zeros
+    if (p.norm_w)
+      for (int q = 0; q < ROWS && r0 + q < p.num_rows; ++q)
+        for (int k = i; k < min(i + 4, p.xn_cols); ++k) reinterpret_cast<T*>(p.xn)[(r0 + q) * p.xn_stride + k] = from_f32<T>(0.f);
+    return;
+  }
+  float w[4], wb[4], nw[4] = {}, nb[4] = {}, add[4] = {};
+  get(p.post, w);
+  get(p.post_bias, wb);
+  if (p.norm_w) {
+    get(p.norm_w, nw);
+    get(p.norm_bias, nb);
+  }
+  if (p.add) get(p.add, add);
+  float v[ROWS][4], x[ROWS][4];
+  long long tok[ROWS];
+#pragma unroll
+  for (int q = 0; q < ROWS; ++q) {
+    const long long r = min(r0 + q, p.num_rows - 1);
+    long long t = p.rows ? p.rows[r] : r;
+    if (t < 0 || t >= p.num_tokens) {
+      if (threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, (int)t);
+      t = 0;
+    }
+    tok[q] = t;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) v[q][k] = x[q][k] = 0.f;
+    if (p.ids) {
+      long long id = p.ids[t];
+      if (id < 0 || id >= p.vocab) {
+        if (threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, (int)id);
+        id = 0;
+      }
+      get(reinterpret_cast<const T*>(p.embed) + id * W, v[q]);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[q][k] *= p.embed_scale;
+    } else {
+      get(p.x + t * (long long)W, x[q]);
+      if (!PICK && p.y) get(reinterpret_cast<const T*>(p.y) + t * p.y_stride, v[q]);
+    }
+  }
+  if constexpr (PICK) {        // expert-sorted rows: four of every token requested together, added in order
+    for (int k0 = 0; k0 < p.topk; k0 += 4) {
+      int pos[ROWS][4];
+#pragma unroll
+      for (int q = 0; q < ROWS; ++q)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) pos[q][k] = k0 + k < p.topk ? p.scatter_index[tok[q] * p.topk + k0 + k] : -1;
+#pragma unroll
+      for (int q = 0; q < ROWS; ++q) {
+        float e[4][4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const int row = pos[q][k];
+          const bool ok = row >= 0 && row < p.y_rows;
+          if (!ok && k0 + k < p.topk && threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, row);
+          e[k][0] = e[k][1] = e[k][2] = e[k][3] = 0.f;
+          if (ok) get(reinterpret_cast<const T*>(p.y) + row * p.y_stride, e[k]);
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) v[q][j] += e[k][j];
+      }
+    }
+  }
+  if (p.extra) {
+    float e[ROWS][4];
+#pragma unroll
+    for (int q = 0; q < ROWS; ++q) get(reinterpret_cast<const T*>(p.extra) + tok[q] * p.extra_stride, e[q]);
+#pragma unroll
+    for (int q = 0; q < ROWS; ++q)
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[q][k] += e[q][k];
+  }
+#pragma unroll
+  for (int q = 0; q < ROWS; ++q) {
+    if (r0 + q >= p.num_rows) break;
+    float o[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      x[q][k] += fmaf(tanh_as<T>(p.post_alpha * v[q][k]), w[k], wb[k]) + add[k];
+      o[k] = fmaf(tanh_as<T>(p.norm_alpha * x[q][k]), nw[k], nb[k]);
+    }
+    float* xrow = p.x + tok[q] * (long long)W + i;
+    T* orow = reinterpret_cast<T*>(p.xn) + (r0 + q) * p.xn_stride + i;
+    if (vec) {
+      if (p.write_back) store4(xrow, x[q]);
+      if (p.norm_w) store4(orow, o);
+    } else {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        if (p.write_back && i + k < W) xrow[k] = x[q][k];
+        if (p.norm_w && i + k < p.xn_cols) orow[k] = from_f32<T>(i + k < W ? o[k] : 0.f);
+      }
+    }
+  }
+}
+
+template <typename T, bool PICK>
+inline int residual_tanh_launch(const ResidualParams& p, cudaStream_t st) {
+  constexpr int MANY = 4;
+  const unsigned gy = (unsigned)(((p.norm_w ? p.xn_cols : p.W) + 511) / 512);
+  if (p.num_rows >= 148 * 2 * MANY)
+    launch_k(residual_tanh_kernel<T, MANY, PICK>, dim3((unsigned)((p.num_rows + MANY - 1) / MANY), gy), dim3(128), 0, st, p);
+  else
+    launch_k(residual_tanh_kernel<T, 1, PICK>, dim3((unsigned)p.num_rows, gy), dim3(128), 0, st, p);
+  return launch_status();
+}
+
 template <typename T, bool PICK>
 inline int residual_launch(const ResidualParams& p, long long rows, cudaStream_t st) {
+  if (p.post_bias) return residual_tanh_launch<T, PICK>(p, st);
   const int chunks = (p.W + 3) / 4;
   const dim3 g((unsigned)rows);
   int threads = 64;
@@ -200,19 +340,23 @@ extern "C" int b200_residual_step(void* x_f32, const void* y, long long y_row_st
                                   const void* scatter_index_i32, int topk, const void* extra, long long extra_row_stride,
                                   const void* embed, const void* ids_i64, long long vocab, const void* rows_i32,
                                   long long num_tokens, long long num_rows, int W, const void* post_f32,
-                                  const void* add_f32, const void* norm_w_f32, float eps, void* xn,
-                                  long long xn_row_stride, int xn_cols, int write_back, int dtype, void* stream) {
+                                  const void* add_f32, const void* norm_w_f32, float eps, float embed_scale,
+                                  const void* post_bias_f32, float post_alpha, const void* norm_bias_f32,
+                                  float norm_alpha, void* xn, long long xn_row_stride, int xn_cols, int write_back,
+                                  int dtype, void* stream) {
   using namespace b200;
   if (!x_f32 || !post_f32 || num_tokens < 0 || num_rows < 0 || W <= 0 || (dtype != 0 && dtype != 1)) return B200_ERR_ARG;
   if ((y != nullptr) == (ids_i64 != nullptr) || (ids_i64 && (!embed || extra)) || (scatter_index_i32 && (!y || topk < 1)))
     return B200_ERR_ARG;
+  if (post_bias_f32 && norm_w_f32 && !norm_bias_f32) return B200_ERR_ARG;
   if ((norm_w_f32 && (!xn || xn_cols < W)) || (rows_i32 && write_back)) return B200_ERR_ARG;
   if (num_rows > 0x7fffffffLL) return B200_ERR_SHAPE;
   if (num_rows == 0) return B200_OK;
   if (W % 4 == 0 && (y_row_stride % 4 || xn_row_stride % 4 || extra_row_stride % 4)) return B200_ERR_SHAPE;
   ResidualParams p{(float*)x_f32, y, y_row_stride, y_rows, (const int*)scatter_index_i32, topk, extra, extra_row_stride,
                    embed, (const long long*)ids_i64, vocab, (const int*)rows_i32, num_tokens, (const float*)post_f32,
-                   (const float*)add_f32, (const float*)norm_w_f32, eps, xn, xn_row_stride, xn_cols, W, write_back};
+                   (const float*)add_f32, (const float*)norm_w_f32, eps, xn, xn_row_stride, xn_cols, W, write_back,
+                   num_rows, embed_scale, (const float*)post_bias_f32, (const float*)norm_bias_f32, post_alpha, norm_alpha};
   const cudaStream_t st = (cudaStream_t)stream;
   if (scatter_index_i32)
     return dtype == 0 ? residual_launch<__nv_bfloat16, true>(p, num_rows, st) : residual_launch<float, true>(p, num_rows, st);

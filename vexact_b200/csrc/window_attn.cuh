@@ -1,5 +1,5 @@
 // Grouped-query attention of decoded tokens and short portions over paged per-head keys and values (bf16), optionally
-// inside a window (position i sees the keys i - window + 1 .. i; window 0: every earlier one).  Scores and weights are
+// inside a window or chunk, with capped scores, a sink in the denominator and an output gate (attn_extras.cuh).  Scores and weights are
 // fp32: a weight enters the value product as a bf16 pair hi + lo, whose two products are summed in fp32, and the
 // denominator sums the fp32 weights.  (attn.cuh and its kin round the weights to bf16, as the models they serve do.)
 //
@@ -26,6 +26,7 @@ struct WindowAttnParams {
   int group, head_chunks, pos_per_tile, box_tokens;
   int dk, dv;
   float scale_log2;
+  AttnExtras extras;
 };
 
 template <int DK, int DV, int WARPS, int STAGES>
@@ -67,7 +68,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
   auto col_q = [&](int c) { return pos0 + (col_valid(c) ? c / heads_here : 0); };   // a spare column repeats the first position
   auto col_head = [&](int c) { return kvh * p.group + chunk * 8 + c % heads_here; };
   const int last_pos = q_abs0 + min(pos0 + p.pos_per_tile, q_len) - 1;
-  const int blk0 = window_first(p.seqs.window, q_abs0 + pos0) / WAT_BN, nblk = last_pos / WAT_BN + 1 - blk0;
+  const int blk0 = first_visible(p.seqs.window, p.seqs.chunk, q_abs0 + pos0) / WAT_BN, nblk = last_pos / WAT_BN + 1 - blk0;
   const int mine = (nblk - warp + WARPS - 1) / WARPS;      // blocks of this warp: blk0 + warp + i * WARPS
 
   if (threadIdx.x == 0) {
@@ -120,9 +121,12 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
       }
   }
   int cpos[2];
+  uint32_t reach[2];                // visible: 0 <= cpos - key < reach
 #pragma unroll
-  for (int j = 0; j < 2; ++j) cpos[j] = q_abs0 + col_q(2 * t + j);
-  const uint32_t reach = p.seqs.window > 0 ? (uint32_t)p.seqs.window : 0x80000000u;   // visible: 0 <= cpos - key < reach
+  for (int j = 0; j < 2; ++j) {
+    cpos[j] = q_abs0 + col_q(2 * t + j);
+    reach[j] = visible_keys(p.seqs.window, p.seqs.chunk, cpos[j]);
+  }
 
   float o[DV / 16][4];
 #pragma unroll
@@ -157,6 +161,12 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
         mma_bf16_16816(sc[mt], a0, a1, a2, a3, qb[kk][0], qb[kk][1]);
       }
     }
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sc[mt][e] *= p.scale_log2;
+      if (p.extras.cap > 0.f) cap_scores(sc[mt], p.extras.cap);
+    }
     float alpha[2];
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -166,8 +176,8 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
 #pragma unroll
         for (int hh = 0; hh < 2; ++hh) {
           const int key = key0 + mt * 16 + g + hh * 8;
-          float v = sc[mt][hh * 2 + j] * p.scale_log2;
-          if ((uint32_t)(cpos[j] - key) >= reach) v = -INFINITY;
+          float v = sc[mt][hh * 2 + j];
+          if ((uint32_t)(cpos[j] - key) >= reach[j]) v = -INFINITY;
           sc[mt][hh * 2 + j] = v;
           mx = fmaxf(mx, v);
         }
@@ -269,9 +279,18 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
       a = fmaf(f, q[d * 8 + c], a);
       b = fmaf(f, q[(d + 1) * 8 + c], b);
     }
-    const float inv = 1.f / l;
-    *reinterpret_cast<uint32_t*>(p.out + (long long)(q_start + col_q(c)) * p.out_stride + (long long)col_head(c) * p.dv + d) =
-        pack_bf2(a * inv, b * inv);
+    const int head = col_head(c);
+    const long long row = q_start + col_q(c);
+    const float inv = 1.f / (l + sink_term(p.extras, head, m));
+    a *= inv;
+    b *= inv;
+    if (p.extras.gate_mode != GATE_NONE) {
+      const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(p.extras.gate) + row * p.extras.gate_stride;
+      const bool per_head = p.extras.gate_mode == GATE_HEAD;
+      a *= gate_sigmoid(gate[per_head ? head : head * p.dv + d]);
+      b *= gate_sigmoid(gate[per_head ? head : head * p.dv + d + 1]);
+    }
+    *reinterpret_cast<uint32_t*>(p.out + row * p.out_stride + (long long)head * p.dv + d) = pack_bf2(a, b);
   }
 }
 
@@ -295,14 +314,16 @@ extern "C" int b200_window_attn_decode(const void* q, long long q_row_stride, co
                                        void* out, long long out_row_stride, const void* query_start_loc,
                                        const void* context_lens, const void* page_table, long long page_table_stride,
                                        int max_pages, int page_size, int num_blocks, int num_seqs, int min_len, int max_len,
-                                       int most_new, int window, int heads, int kv_heads, int DK, int DV, float scale,
-                                       void* stream) {
+                                       int most_new, int window, int chunk, float cap, const void* sink_f32,
+                                       const void* gate, long long gate_row_stride, int gate_mode, int heads, int kv_heads,
+                                       int DK, int DV, float scale, void* stream) {
   using namespace b200;
   WindowAttnParams p{};
   p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
-            page_size, num_blocks, num_seqs, min_len < 1 ? 1 : min_len, max_len, window};
+            page_size, num_blocks, num_seqs, min_len < 1 ? 1 : min_len, max_len, window, chunk};
+  p.extras = {cap * kLog2e, (const float*)sink_f32, gate, gate_row_stride, gate_mode};
   if (!latent_seqs_ok(p.seqs) || !q || !k_cache || !v_cache || !out || heads <= 0 || kv_heads <= 0 || heads % kv_heads ||
-      DK <= 0 || DV <= 0 || window < 0 || max_len < 1 || most_new < 0)
+      DK <= 0 || DV <= 0 || window < 0 || chunk < 0 || max_len < 1 || most_new < 0 || !attn_extras_ok(p.extras))
     return B200_ERR_ARG;
   const bool pages_ok = page_size % 8 == 0 && (page_size % WAT_BN == 0 || WAT_BN % page_size == 0);
   if (DK % 8 || DV % 8 || DK > 256 || DV > 256 || !pages_ok || q_row_stride % 2 || out_row_stride % 2 ||
@@ -320,7 +341,7 @@ extern "C" int b200_window_attn_decode(const void* q, long long q_row_stride, co
   p.box_tokens = page_size < WAT_BN ? page_size : WAT_BN;
   p.dk = DK;
   p.dv = DV;
-  p.scale_log2 = scale * kLog2e;
+  p.scale_log2 = cap > 0.f ? scale / cap : scale * kLog2e;
   CUtensorMap tk, tv;
   int rc = make_tmap_cache(&tk, k_cache, num_blocks, page_size, kv_heads, DK, (long long)page_size * kv_heads * DK,
                            (long long)kv_heads * DK, DK, p.box_tokens);
@@ -345,15 +366,21 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
                                         void* out, long long out_row_stride, const void* query_start_loc,
                                         const void* context_lens, const void* page_table, long long page_table_stride,
                                         int max_pages, int page_size, int num_blocks, int num_seqs, const void* seq_ids_i32,
-                                        int n, int max_len, int min_len, int window, long long T, int heads, int kv_heads,
-                                        int DK, int DV, float scale, int form, void* stream) {
+                                        int n, int max_len, int min_len, int window, int chunk, float cap,
+                                        const void* sink_f32, const void* gate, long long gate_row_stride, int gate_mode,
+                                        long long T, int heads, int kv_heads, int DK, int DV, float scale, int form,
+                                        void* stream) {
   using namespace b200;
   LatentExpandParams p{};
   p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
-            page_size, num_blocks, num_seqs, 0, 0, window};
+            page_size, num_blocks, num_seqs, 0, 0, window, chunk};
+  p.extras = {cap * kLog2e, (const float*)sink_f32, gate, gate_row_stride, gate_mode};
   if (!latent_seqs_ok(p.seqs) || !q || !k_cache || !v_cache || !out || !seq_ids_i32 || n <= 0 || max_len <= 0 || T <= 0 ||
-      heads <= 0 || kv_heads <= 0 || heads % kv_heads || DK <= 0 || DV <= 0 || window < 0)
+      heads <= 0 || kv_heads <= 0 || heads % kv_heads || DK <= 0 || DV <= 0 || window < 0 || chunk < 0 ||
+      !attn_extras_ok(p.extras))
     return B200_ERR_ARG;
+  if (gate_mode == GATE_COLUMN && (gate_row_stride % 8 || (reinterpret_cast<uintptr_t>(gate) & 15))) return B200_ERR_SHAPE;
+  const float score_scale = cap > 0.f ? scale / cap : scale * kLog2e;
   if (DK % 8 || DV % 8 || q_row_stride % 8 || out_row_stride % 8 || DK > 256 || DV > 256 || heads > 65535 || n > 65535)
     return B200_ERR_SHAPE;
   const cudaStream_t st = (cudaStream_t)stream;
@@ -380,7 +407,9 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
     a.group = group;
     a.head_chunks = (group + 7) / 8;
     a.pos_per_tile = ATR_ROWS / hh;
-    a.qk_scale = scale * kLog2e;
+    a.qk_scale = score_scale;
+    a.extras = p.extras;
+    a.chunk = chunk;
     a.num_blocks = num_blocks;
     a.num_seqs = num_seqs;
     a.max_seqlen_q = max_len;
@@ -419,6 +448,6 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
   p.group = group;
   p.DN = DK;
   p.DV = DV;
-  p.scale_log2 = scale * kLog2e;
+  p.scale_log2 = score_scale;
   return latent_expand_dispatch<true>(p, max_len, n, st);
 }

@@ -15,12 +15,13 @@ FUSED_MAX_ROWS = 64     # rows (per group) up to which the activation rides on t
 
 @dataclass
 class MLPWeights:
-    """down(gelu(up x + up_b)) + down_b."""
+    """down(act(up x + up_b)) + down_b; the biases may be absent."""
 
     up: torch.Tensor
-    up_b: torch.Tensor
     down: torch.Tensor
-    down_b: torch.Tensor
+    up_b: Optional[torch.Tensor] = None
+    down_b: Optional[torch.Tensor] = None
+    act: str = "gelu_tanh"           # or "relu2": the square of relu
 
 
 @dataclass
@@ -33,7 +34,7 @@ class GLUWeights:
 
 
 def mlp_forward(w: MLPWeights, x: torch.Tensor) -> torch.Tensor:
-    return gemm(gemm(x, w.up, w.up_b, act="gelu_tanh"), w.down, w.down_b)
+    return gemm(gemm(x, w.up, w.up_b, act=w.act), w.down, w.down_b)
 
 
 def glu(gu: torch.Tensor, act: str, scale_in: Optional[torch.Tensor] = None,

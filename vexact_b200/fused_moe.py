@@ -16,13 +16,13 @@ from __future__ import annotations
 
 import os
 from dataclasses import dataclass
-from typing import Optional
+from typing import Optional, Union
 
 import torch
 
 from . import _lib
-from .batch_invariant_ops import gemm
-from .feed_forward import GLU_ACTS, GLUWeights, glu, glu_forward
+from .batch_invariant_ops import GEMM_ACTS, gemm
+from .feed_forward import GLU_ACTS, GLUWeights, MLPWeights, glu, glu_forward, mlp_forward
 
 TILE_ROWS = 64  # largest token tile of the grouped GEMM (rows of one expert per tile)
 FUSED_SWIGLU_MAX_ROWS_PER_EXPERT = 64  # mean rows per expert up to which fc1 keeps its fused SwiGLU epilogue
@@ -391,14 +391,20 @@ def fused_moe_forward(
 # ------------------------------------------------------------------ mixtures of the hybrid decoders
 @dataclass
 class MixtureWeights:
-    """Sigmoid-scored experts whose score multiplies their input, and a gated shared expert."""
+    """Two forms.  act "silu": gated experts, scored by a sigmoid that multiplies their input, and a gated shared expert.
+    act "relu2": plain experts down(relu(up)^2), whose score multiplies their output, chosen inside the best groups, and a
+    shared expert of the same form."""
 
     router: torch.Tensor             # [experts (+ 1: the shared expert's gate), width]
-    gate_up: torch.Tensor            # [experts, 2 * F, width], gate rows first
+    gate_up: torch.Tensor            # [experts, 2 * F, width], gate rows first; plain experts: up alone, [experts, F, width]
     down: torch.Tensor               # [experts, width (padded), F]
     experts: int
     top: int
-    shared: Optional[GLUWeights] = None
+    shared: Union[GLUWeights, MLPWeights, None] = None
+    act: str = "silu"
+    score: str = "sigmoid"
+    correction: Optional[torch.Tensor] = None    # [experts] fp32, added to the scores in the choice
+    groups: tuple = (1, 1)                       # (equal groups of neighbours, groups kept)
 
 
 @dataclass
@@ -418,45 +424,87 @@ def route_plan_sigmoid_topk(router_logits: torch.Tensor, top_k: int, num_experts
     Returns (scores [T, k] fp32, experts [T, k] int64, gate [T] fp32 or None: the sigmoid of column `num_experts`, plan);
     the order of rows inside an expert's group is that of arrival, on which no output depends."""
     T, dev = router_logits.shape[0], router_logits.device
-    n = T * top_k
-    max_tiles = max(1, max_token_tiles(n, num_experts))
-    w = torch.empty((T, top_k), device=dev, dtype=torch.float32)
+    w, idx, plan = _plan_buffers(T, top_k, num_experts, dev)
     g = torch.empty(T, device=dev, dtype=torch.float32) if gate else None
-    idx = torch.empty((T, top_k), device=dev, dtype=torch.int64)
-    ints = torch.empty(n + num_experts + 2, device=dev, dtype=torch.int32)
-    rank, cu_seqlens, tile_count = ints[:n], ints[n:n + num_experts + 1], ints[n + num_experts + 1:]
-    tile_table = torch.empty((max_tiles, 4), device=dev, dtype=torch.int32)
     _lib.check(
         _lib.load().b200_moe_route_plan_sigmoid_topk(
-            router_logits.data_ptr(), router_logits.stride(0), w.data_ptr(), _lib.ptr(g), idx.data_ptr(), rank.data_ptr(),
-            _plan_counters(dev).data_ptr(), cu_seqlens.data_ptr(), tile_table.data_ptr(), tile_count.data_ptr(), T,
-            num_experts, top_k, int(renorm), TILE_ROWS, max_tiles, _lib.current_stream()),
+            router_logits.data_ptr(), router_logits.stride(0), w.data_ptr(), _lib.ptr(g), idx.data_ptr(),
+            plan["rank"].data_ptr(), _plan_counters(dev).data_ptr(), plan["cu_seqlens"].data_ptr(),
+            plan["tile_table"].data_ptr(), plan["tile_count"].data_ptr(), T, num_experts, top_k, int(renorm), TILE_ROWS,
+            plan["max_tiles"], _lib.current_stream()),
         "b200_moe_route_plan_sigmoid_topk",
     )
-    return w, idx, g, dict(rank=rank, cu_seqlens=cu_seqlens, tile_table=tile_table, tile_count=tile_count,
-                           max_tiles=max_tiles)
+    return w, idx, g, plan
 
 
-def _grouped_rows(x: torch.Tensor, w: torch.Tensor, plan: dict) -> torch.Tensor:
-    """Grouped product of expert-sorted rows in the rows' dtype."""
-    if x.dtype == torch.bfloat16:
+def _plan_buffers(T: int, top_k: int, num_experts: int, dev):
+    """(scores, experts, plan) as a routing-plan kernel fills them."""
+    n = T * top_k
+    ints = torch.empty(n + num_experts + 2, device=dev, dtype=torch.int32)
+    max_tiles = max(1, max_token_tiles(n, num_experts))
+    plan = dict(rank=ints[:n], cu_seqlens=ints[n:n + num_experts + 1], tile_count=ints[n + num_experts + 1:],
+                tile_table=torch.empty((max_tiles, 4), device=dev, dtype=torch.int32), max_tiles=max_tiles)
+    return (torch.empty((T, top_k), device=dev, dtype=torch.float32),
+            torch.empty((T, top_k), device=dev, dtype=torch.int64), plan)
+
+
+def route_plan_group_topk(router_logits: torch.Tensor, top_k: int, num_experts: int, *, score: str = "softmax",
+                          correction: Optional[torch.Tensor] = None, groups: tuple = (1, 1), renorm: bool = False):
+    """Top-k by corrected scores inside the best groups, with the permutation planned in the same launch (fp32 logits).
+
+    Choice score: score + correction (fp32 [experts] or None); a group's score is its largest choice score, and only experts
+    of the best groups[1] of groups[0] equal groups can be chosen.  Returns (scores [T, k] fp32 without the correction,
+    experts [T, k] int64, plan)."""
+    T, dev = router_logits.shape[0], router_logits.device
+    w, idx, plan = _plan_buffers(T, top_k, num_experts, dev)
+    _lib.check(
+        _lib.load().b200_moe_route_plan_group_topk(
+            router_logits.data_ptr(), router_logits.stride(0), {"softmax": 0, "sigmoid": 1}[score], _lib.ptr(correction),
+            groups[0], groups[1], w.data_ptr(), idx.data_ptr(), plan["rank"].data_ptr(), _plan_counters(dev).data_ptr(),
+            plan["cu_seqlens"].data_ptr(), plan["tile_table"].data_ptr(), plan["tile_count"].data_ptr(), T, num_experts,
+            top_k, int(renorm), TILE_ROWS, plan["max_tiles"], _lib.current_stream()),
+        "b200_moe_route_plan_group_topk",
+    )
+    return w, idx, plan
+
+
+def _grouped_rows(x: torch.Tensor, w: torch.Tensor, plan: dict, act: Optional[str] = None,
+                  scale_out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Grouped product of expert-sorted rows in the rows' dtype; act "relu2": max(., 0)^2 times scale_out (fp32 per row)."""
+    if x.dtype == torch.bfloat16 and act is None:
         return _grouped_gemm(x, w, None, plan, w.shape[1], mode=0)
     out = torch.empty((x.shape[0], w.shape[1]), device=x.device, dtype=x.dtype)
+    if x.dtype == torch.bfloat16:
+        _lib.check(
+            _lib.load().b200_moe_grouped_gemm_act(
+                x.data_ptr(), w.data_ptr(), _lib.ptr(scale_out), out.data_ptr(), plan["tile_table"].data_ptr(),
+                plan["tile_count"].data_ptr(), x.shape[0], w.shape[0], w.shape[1], x.shape[1], out.stride(0),
+                plan["max_tiles"], TILE_ROWS, GEMM_ACTS[act], _lib.current_stream()),
+            "b200_moe_grouped_gemm_act",
+        )
+        return out
     _lib.check(
-        _lib.load().b200_moe_grouped_gemm_f32(x.data_ptr(), w.data_ptr(), out.data_ptr(), plan["tile_table"].data_ptr(),
-                                              plan["tile_count"].data_ptr(), x.shape[0], w.shape[0], w.shape[1],
-                                              x.shape[1], plan["max_tiles"], _lib.current_stream()),
+        _lib.load().b200_moe_grouped_gemm_f32(
+            x.data_ptr(), w.data_ptr(), _lib.ptr(scale_out), out.data_ptr(), plan["tile_table"].data_ptr(),
+            plan["tile_count"].data_ptr(), x.shape[0], w.shape[0], w.shape[1], x.shape[1], plan["max_tiles"],
+            GEMM_ACTS[act], _lib.current_stream()),
         "b200_moe_grouped_gemm_f32",
     )
     return out
 
 
 def mixture_forward(w: MixtureWeights, x: torch.Tensor) -> PendingMixture:
-    """sum over the top experts e of expert_e(s_e x), s = sigmoid(router x), plus sigmoid(gate x) * shared(x)."""
+    """act "silu": sum over the top experts e of expert_e(s_e x), s = sigmoid(router x), plus sigmoid(gate x) * shared(x).
+    act "relu2": sum of s_e expert_e(x), plus shared(x)."""
     T, K = x.shape
     n, E = T * w.top, w.experts
+    plain = w.act == "relu2"
     logits = gemm(x, w.router, out_dtype=torch.float32)      # exact products, fp32 sums
-    scores, idx, gate, plan = route_plan_sigmoid_topk(logits, w.top, E, w.shared is not None)
+    gate = None
+    if plain:
+        scores, idx, plan = route_plan_group_topk(logits, w.top, E, score=w.score, correction=w.correction, groups=w.groups)
+    else:
+        scores, idx, gate, plan = route_plan_sigmoid_topk(logits, w.top, E, w.shared is not None)
     x_perm = torch.empty((n, K), device=x.device, dtype=x.dtype)
     row_scale = torch.empty(n, device=x.device, dtype=torch.float32)
     scatter_index = torch.empty(n, device=x.device, dtype=torch.int32)
@@ -468,6 +516,10 @@ def mixture_forward(w: MixtureWeights, x: torch.Tensor) -> PendingMixture:
             K * size, _lib.current_stream()),
         "b200_moe_scatter_ranked_f32",
     )
+    if plain:
+        h = _grouped_rows(x_perm, w.gate_up, plan, w.act, row_scale)
+        shared = None if w.shared is None else mlp_forward(w.shared, x)
+        return PendingMixture(_grouped_rows(h, w.down, plan), scatter_index, w.top, shared)
     F = w.gate_up.shape[1] // 2
     if x.dtype == torch.bfloat16 and n <= FUSED_SWIGLU_MAX_ROWS_PER_EXPERT * E:
         h = torch.empty((n, F), device=x.device, dtype=x.dtype)

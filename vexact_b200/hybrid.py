@@ -1,6 +1,6 @@
 """Hybrid decoders: layers that mix recurrent and attention mixers, dense and mixture feed-forwards, hung on
-hyper-connections ("Nurazen") or on one residual with norms on both sides of a sublayer and a looped run of layers
-("Dekerax").
+hyper-connections ("Nurazen") or on one residual with norms on both sides of a sublayer, with a looped run of layers
+("Dekerax") or with layers that share weights ("Tekilix").
 
 `HybridShape.from_config` reads config.json (hybrid_config.py), `HybridWeights` turns checkpoint tensors into what the
 kernels take (hybrid_weights.py), `HybridRunner` runs a packed step, and `HybridModel` is the form the `Inferencer`
@@ -18,7 +18,7 @@ from .delta import DeltaWeights, delta_mixer
 from .fused_moe import MixtureWeights, mixture_forward
 from .feed_forward import GLUWeights, MLPWeights, glu_forward, mlp_forward
 from .hybrid_config import (ARCHITECTURES, AttentionSpec, DeltaSpec, DenseSpec, HybridLayer, HybridShape, LatentSpec,  # noqa: F401
-                            LoopSpec, MixtureSpec, SSMSpec, random_tensors, tensor_shapes)
+                            LoopSpec, MixtureSpec, RotarySpec, SSMSpec, YarnSpec, random_tensors, tensor_shapes)
 from .hybrid_weights import HybridLayerWeights, HybridWeights  # noqa: F401
 from .hyper import hyper_step
 from .kv_cache_context import HybridCacheStore, get_kv_cache_context
@@ -59,7 +59,8 @@ class HybridRunner:
         if isinstance(mixer, DeltaWeights):
             return delta_mixer(mixer, xn, st.conv_state[run], st.ssm_state[run], step, self.shape.eps)
         if isinstance(mixer, AttentionWeights):
-            return attention_mixer(mixer, xn, st.key_cache[run], st.value_cache[run], step)
+            return attention_mixer(mixer, xn, st.key_cache[run], st.value_cache[run], step, self.shape.eps,
+                                   st.conv_state.get(run))
         return latent_mixer(mixer, xn, st.key_cache[run], step, self.shape.eps)
 
     def _feed_forward(self, mlp, xn: torch.Tensor):
@@ -100,7 +101,7 @@ class HybridRunner:
         s, w = self.shape, self.w
         x = torch.empty((step.input_ids.numel(), s.width), device=w.embed.device, dtype=torch.float32)
         common = dict(eps=s.eps, xn_cols=w.xn_cols, dtype=w.dtype)
-        source = dict(embed=w.embed, ids=step.input_ids, post=w.embed_norm)
+        source = dict(embed=w.embed, ids=step.input_ids, post=w.embed_norm, embed_scale=s.embed_scale)
 
         def report(run):          # what the run leaves, before anything that belongs to the next one
             kept = x.clone()
@@ -151,7 +152,8 @@ class HybridModel:
         latent = {r: m.row_width for r, m in mixers.items() if isinstance(m, LatentWeights)}
         heads = {r: (m.kv_heads, m.DK, m.DV) for r, m in mixers.items() if isinstance(m, AttentionWeights)}
         state = {r: m.state_dims() for r, m in mixers.items() if isinstance(m, (SSMWeights, DeltaWeights))}
-        return HybridCacheStore(latent, state, cache_config, num_slots, device, w.dtype, heads)
+        conv = {r: m.conv_dims() for r, m in mixers.items() if isinstance(m, AttentionWeights) and m.conv_w is not None}
+        return HybridCacheStore(latent, state, cache_config, num_slots, device, w.dtype, heads, conv)
 
     def forward(self, input_ids=None, intermediate_tensors=None, position_ids=None, **_unused):
         from .inferencer import StageOutput

@@ -1,13 +1,16 @@
 """Configuration of the hybrid decoders: what config.json says, as specs of mixers, feed-forwards and the residual, and
 the checkpoint tensors that go with them.
 
-Two architectures are read here:
+Three architectures are read here:
   "Nurazen"  state-space (Mamba-2) and latent-attention mixers, dense feed-forwards, hyper-connections, shared weights
   "Dekerax"  windowed attention, windowed latent attention with a query latent, gated delta rule, dense and mixture
              feed-forwards, one residual with a norm on both sides of every sublayer, a run of layers that loops
+  "Tekilix"  chunked attention in two forms (capped scores; convolved keys that are also the values, learned sinks),
+             mixtures chosen inside groups, dynamic tanh on both sides of every sublayer, shared weights, tied embedding
 A mechanism is described by a spec of its own, so that an architecture is a choice of specs."""
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Mapping, Optional, Union
 
@@ -32,13 +35,57 @@ class LatentSpec:
 
 
 @dataclass(frozen=True)
+class YarnSpec:
+    """Rotation frequencies stretched by `factor` for contexts beyond `original` tokens: those that turn fewer than `slow`
+    times in it by all of it, those that turn more than `fast` times not at all."""
+
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
+class RotarySpec:
+    base: float
+    dims: int
+    half: bool                       # pairs (i, i + dims / 2) instead of (2i, 2i + 1)
+    yarn: Optional[YarnSpec] = None
+
+    def frequencies(self) -> tuple:
+        """([dims / 2] float64 turns per position, factor of cosine and sine)."""
+        i = torch.arange(self.dims // 2, dtype=torch.float64)
+        f = self.base ** (-2 * i / max(self.dims, 1))
+        if self.yarn is None:
+            return f, 1.0
+        y = self.yarn
+
+        def pair_that_turns(times):
+            return self.dims * math.log(y.original / (2 * math.pi * times)) / (2 * math.log(self.base))
+
+        lo = max(math.floor(pair_that_turns(y.fast)), 0)
+        hi = min(math.ceil(pair_that_turns(y.slow)), self.dims - 1)
+        ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+        return f / y.factor * ramp + f * (1 - ramp), 0.1 * math.log(y.factor) + 1.0
+
+
+@dataclass(frozen=True)
 class AttentionSpec:
     heads: int
     kv_heads: int
     dim: int
     vdim: int
     scale: float
-    window: Optional[int] = None
+    window: Optional[int] = None             # tokens a query sees, itself included
+    chunk: Optional[int] = None              # a query sees its own chunk only; chunks count from the first token
+    rot: Optional[RotarySpec] = None
+    bias: bool = False                       # of the query, key and value projections
+    qk_norm: Optional[str] = None            # "head": per head, one weight for all; "all": over the whole projection
+    conv: Optional[int] = None               # taps of a convolution of queries and keys, ahead of norm and rotation
+    keys_as_values: bool = False             # values are the keys ahead of norm and rotation
+    softcap: Optional[float] = None          # a score s becomes softcap * tanh(s / softcap)
+    sink: Optional[str] = None               # extra term of the denominator: "unit" (1) or "learned" (exp of one per head)
+    gate: Optional[str] = None               # output times the sigmoid of one number per "head" or per "column"
 
 
 @dataclass(frozen=True)
@@ -73,6 +120,12 @@ class MixtureSpec:
     top: int
     ff: int
     shared_ff: Optional[int] = None
+    act: str = "silu"                        # gated: down(silu(gate) * up); "relu2": down(relu(up)^2)
+    score: str = "sigmoid"                   # or "softmax" over all experts
+    score_on: str = "input"                  # what a chosen expert's score multiplies: its "input" or its "output"
+    shared_gate: bool = True                 # the shared expert is times the sigmoid of one number
+    correction: bool = False                 # a learned number per expert takes part in the choice only
+    groups: tuple = (1, 1)                   # (equal groups of neighbours, groups kept): the rest cannot be chosen
 
 
 MixerSpec = Union[LatentSpec, AttentionSpec, SSMSpec, DeltaSpec]
@@ -106,11 +159,23 @@ class HybridShape:
     eps: float
     architecture: str = "Nurazen"
     loop: Optional[LoopSpec] = None
+    embed_scale: float = 1.0
+    logit_scale: float = 1.0
 
     @property
     def sandwich(self) -> bool:
         """One residual with a norm before and after every sublayer, instead of hyper-connections."""
-        return self.architecture == "Dekerax"
+        return self.architecture in ("Dekerax", "Tekilix")
+
+    @property
+    def tanh_norms(self) -> bool:
+        """The norms are tanh(alpha x) * weight + b instead of a division by the root mean square."""
+        return self.architecture == "Tekilix"
+
+    @property
+    def tied(self) -> bool:
+        """The embedding is the output table too."""
+        return self.architecture == "Tekilix"
 
     @property
     def runs(self) -> tuple:
@@ -135,6 +200,19 @@ class HybridShape:
         return ARCHITECTURES[self.architecture][1](self)
 
 
+def _read_weights_of(i: int, e: Mapping, layers: list, mixer, ff) -> int:
+    """The layer whose tensors layer i uses: an earlier one that equals it, followed to the one that has them."""
+    src = e.get("weights_of")
+    if src is None or src == i:
+        return i
+    if not 0 <= src < i:
+        raise ValueError(f"layer {i}: weights_of {src} is not an earlier layer")
+    src = layers[src].weights_of
+    if layers[src].mixer != mixer or layers[src].ff != ff:
+        raise ValueError(f"layer {i} differs from layer {src}, whose weights it uses")
+    return src
+
+
 # ------------------------------------------------------------------ Nurazen
 def _read_nurazen(cfg: Mapping) -> HybridShape:
     layers = []
@@ -151,15 +229,7 @@ def _read_nurazen(cfg: Mapping) -> HybridShape:
         if mlp is not None and mlp["kind"] != "dense":
             raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']!r}")
         ff = DenseSpec(mlp["ff"]) if mlp else None
-        src = e.get("weights_of")
-        src = i if src is None else src
-        if src != i:
-            if not 0 <= src < i:
-                raise ValueError(f"layer {i}: weights_of {src} is not an earlier layer")
-            src = layers[src].weights_of
-            if layers[src].mixer != mixer or layers[src].ff != ff:
-                raise ValueError(f"layer {i} differs from layer {src}, whose weights it uses")
-        layers.append(HybridLayer(mixer, ff, src))
+        layers.append(HybridLayer(mixer, ff, _read_weights_of(i, e, layers, mixer, ff)))
     return HybridShape(cfg.get("name", "nurazen"), tuple(layers), cfg["width"], cfg["vocab"], cfg["streams"],
                        float(cfg["residual_mult"]), float(cfg["norm"]["eps"]))
 
@@ -264,8 +334,84 @@ def _write_dekerax(s: HybridShape) -> dict:
     return cfg
 
 
+# ------------------------------------------------------------------ Tekilix
+def _read_rotary(i: int, m: Mapping, half: bool) -> RotarySpec:
+    rot, dim = m["rot"], m["dim"]
+    if not 0 <= rot["dims"] <= dim or rot["dims"] % 2:
+        raise ValueError(f"layer {i}: {rot['dims']} of {dim} columns rotate")
+    sc = rot.get("scaling")
+    yarn = YarnSpec(float(sc["factor"]), float(sc["original"]), float(sc["fast"]), float(sc["slow"])) if sc else None
+    return RotarySpec(float(rot["base"]), rot["dims"], half, yarn)
+
+
+def _read_tekilix(cfg: Mapping) -> HybridShape:
+    layers = []
+    for i, e in enumerate(cfg["layers"]):
+        m = e["mixer"]
+        common = dict(heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], scale=float(m["scale"]),
+                      chunk=_read_window(i, m))
+        if e["type"] == "attention":
+            cap = m.get("softcap")
+            mixer = AttentionSpec(**common, rot=_read_rotary(i, m, False), bias=True, qk_norm="all",
+                                  softcap=None if cap is None else float(cap), sink="unit", gate="head")
+        elif e["type"] == "attention_2":
+            mixer = AttentionSpec(**common, rot=_read_rotary(i, m, True), qk_norm="head", conv=m["conv"],
+                                  keys_as_values=True, sink="learned", gate="column")
+            if mixer.vdim != mixer.dim:
+                raise ValueError(f"layer {i}: keys of {mixer.dim} columns as values of {mixer.vdim}")
+        else:
+            raise NotImplementedError(f"layer {i}: mixer {e['type']!r}")
+        if mixer.heads % mixer.kv_heads:
+            raise ValueError(f"layer {i}: {mixer.heads} heads over {mixer.kv_heads} key/value heads")
+        mlp, ff = e.get("mlp"), None
+        if mlp is not None and mlp["kind"] != "moe":
+            raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']!r}")
+        if mlp is not None:
+            r, shared, g = mlp["router"], mlp.get("shared"), mlp["router"].get("groups") or {"count": 1, "keep": 1}
+            ff = MixtureSpec(r["experts"], r["top"], mlp["expert"]["ff"], shared["ff"] if shared else None, act="relu2",
+                             score="softmax", score_on="output", shared_gate=False, correction=True,
+                             groups=(g["count"], g["keep"]))
+            if ff.experts % g["count"] or not 1 <= g["keep"] <= g["count"]:
+                raise ValueError(f"layer {i}: {g['keep']} of {g['count']} groups of {ff.experts} experts")
+            if not 1 <= ff.top <= g["keep"] * (ff.experts // g["count"]):
+                raise ValueError(f"layer {i}: {ff.top} experts out of {g['keep']} groups of {ff.experts // g['count']}")
+        layers.append(HybridLayer(mixer, ff, _read_weights_of(i, e, layers, mixer, ff)))
+    return HybridShape(cfg.get("name", "tekilix"), tuple(layers), cfg["width"], cfg["vocab"], 1, 1.0,
+                       float(cfg["norm"]["eps"]), "Tekilix", embed_scale=float(cfg["embedding"]["scale"]),
+                       logit_scale=float(cfg["logit_scale"]))
+
+
+def _write_tekilix(s: HybridShape) -> dict:
+    out = []
+    for i, layer in enumerate(s.layers):
+        m, ff = layer.mixer, layer.ff
+        mixer = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
+                 "rot": {"base": m.rot.base, "dims": m.rot.dims}}
+        if m.chunk is not None:
+            mixer["mask"] = {"size": m.chunk}
+        if m.rot.yarn is not None:
+            mixer["rot"]["scaling"] = {k: getattr(m.rot.yarn, k) for k in ("factor", "original", "fast", "slow")}
+        if m.conv is not None:
+            mixer["conv"] = m.conv
+        if m.softcap is not None:
+            mixer["softcap"] = m.softcap
+        e = {"type": "attention_2" if m.keys_as_values else "attention", "mixer": mixer, "mlp": None}
+        if ff is not None:
+            e["mlp"] = {"kind": "moe", "expert": {"ff": ff.ff},
+                        "router": {"experts": ff.experts, "top": ff.top,
+                                   "groups": {"count": ff.groups[0], "keep": ff.groups[1]}}}
+            if ff.shared_ff is not None:
+                e["mlp"]["shared"] = {"ff": ff.shared_ff}
+        if layer.weights_of != i:
+            e["weights_of"] = layer.weights_of
+        out.append(e)
+    return {"architecture": "Tekilix", "layers": out, "norm": {"eps": s.eps}, "width": s.width, "vocab": s.vocab,
+            "embedding": {"scale": s.embed_scale}, "logit_scale": s.logit_scale}
+
+
 # config.json "architecture" -> (reader, writer)
-ARCHITECTURES = {"Nurazen": (_read_nurazen, _write_nurazen), "Dekerax": (_read_dekerax, _write_dekerax)}
+ARCHITECTURES = {"Nurazen": (_read_nurazen, _write_nurazen), "Dekerax": (_read_dekerax, _write_dekerax),
+                 "Tekilix": (_read_tekilix, _write_tekilix)}
 
 
 # ------------------------------------------------------------------ checkpoint tensors
@@ -279,8 +425,21 @@ def _mixer_tensors(m: MixerSpec, W: int) -> dict:
             t["g"] = (m.heads * m.vdim, W)
         return dict(t, o=(W, m.heads * m.vdim))
     if isinstance(m, AttentionSpec):
-        return {"q": (m.heads * m.dim, W), "k": (m.kv_heads * m.dim, W), "v": (m.kv_heads * m.vdim, W),
-                "o": (W, m.heads * m.vdim)}
+        rows = {"q": m.heads * m.dim, "k": m.kv_heads * m.dim, "v": m.kv_heads * m.vdim}
+        if m.keys_as_values:
+            del rows["v"]
+        t = {n: (r, W) for n, r in rows.items()}
+        if m.bias:
+            t.update({n + ".b": (r,) for n, r in rows.items()})
+        if m.qk_norm is not None:
+            t.update({n + ".norm": (rows[n] if m.qk_norm == "all" else m.dim,) for n in "qk"})
+        if m.conv is not None:
+            t.update({n + ".conv": (rows[n], m.conv) for n in "qk"})
+        if m.sink == "learned":
+            t["sink"] = (m.heads,)
+        if m.gate is not None:
+            t["g"] = (m.heads * (m.vdim if m.gate == "column" else 1), W)
+        return dict(t, o=(W, m.heads * m.vdim))
     if isinstance(m, DeltaSpec):
         qk, v = m.kv_heads * m.dim, m.heads * m.vdim
         return {"q": (qk, W), "q.conv": (qk, m.conv), "k": (qk, W), "k.conv": (qk, m.conv), "v": (v, W),
@@ -292,16 +451,20 @@ def _mixer_tensors(m: MixerSpec, W: int) -> dict:
 
 
 def _ff_tensors(ff: FFSpec, W: int) -> dict:
-    def gated(p, n):
-        return {p + "gate": (n, W), p + "up": (n, W), p + "down": (W, n)}
+    def expert(p, n, gated):
+        return dict({p + "gate": (n, W)} if gated else {}, **{p + "up": (n, W), p + "down": (W, n)})
 
     if isinstance(ff, DenseSpec):
-        return gated("", ff.ff) if ff.gated else {"up": (ff.ff, W), "up.b": (ff.ff,), "down": (W, ff.ff), "down.b": (W,)}
-    t = {"router": (ff.experts, W)}
+        return expert("", ff.ff, True) if ff.gated else {"up": (ff.ff, W), "up.b": (ff.ff,), "down": (W, ff.ff), "down.b": (W,)}
+    t, gated = {"router": (ff.experts, W)}, ff.act != "relu2"
+    if ff.correction:
+        t["correction"] = (ff.experts,)
     for e in range(ff.experts):
-        t.update(gated(f"e{e}.", ff.ff))
+        t.update(expert(f"e{e}.", ff.ff, gated))
     if ff.shared_ff is not None:
-        t.update(gated("shared.", ff.shared_ff), **{"shared.sg": (1, W)})
+        t.update(expert("shared.", ff.shared_ff, gated))
+        if ff.shared_gate:
+            t["shared.sg"] = (1, W)
     return t
 
 
@@ -309,8 +472,12 @@ def tensor_shapes(shape: HybridShape) -> dict[str, tuple]:
     """Checkpoint tensor names and shapes.  Linear weights are [out, in]."""
     W, n = shape.width, shape.streams
     out = {"embed": (shape.vocab, W)}
+
+    def norm(name):
+        return {name: (W,), name + ".b": (W,), name + ".alpha": ()} if shape.tanh_norms else {name: (W,)}
+
     if shape.sandwich:
-        out["embed.norm"] = (W,)
+        out.update(norm("embed.norm"))
         if shape.loop is not None:
             out["loop.step"] = (shape.loop.times, W)
     for i, layer in enumerate(shape.layers):
@@ -318,15 +485,17 @@ def tensor_shapes(shape: HybridShape) -> dict[str, tuple]:
             continue
         t = {f"mix.{k}": v for k, v in _mixer_tensors(layer.mixer, W).items()}
         for q in ([1] if layer.ff is None else [1, 2]):
-            t[f"norm{q}"] = (W,)
+            t.update(norm(f"norm{q}"))
             if shape.sandwich:
-                t[f"norm{q}b"] = (W,)
+                t.update(norm(f"norm{q}b"))
             else:
                 t.update({f"hc{q}.in": (n,), f"hc{q}.out": (n,), f"hc{q}.mix": (n, n)})
         if layer.ff is not None:
             t.update({f"mlp.{k}": v for k, v in _ff_tensors(layer.ff, W).items()})
         out.update({f"l{i}.{k}": v for k, v in t.items()})
-    out.update({"final.norm": (W,), "head": (shape.vocab, W)})
+    out.update(norm("final.norm"))
+    if not shape.tied:
+        out["head"] = (shape.vocab, W)
     return out
 
 
@@ -341,6 +510,14 @@ def random_tensors(shape: HybridShape, seed: int = 0, device="cpu", dtype=torch.
             pass
         elif name == "loop.step":
             t = 0.3 * t
+        elif name.endswith(".alpha"):
+            t = (0.25 if name == "final.norm.alpha" else 0.7) + 0.1 * t
+        elif name.endswith("norm.b") or leaf.startswith("norm") and leaf.endswith(".b"):
+            t = 0.1 * t
+        elif leaf.endswith(".conv"):
+            t = t / dims[1] ** 0.5
+        elif leaf == "mlp.correction":
+            t = 0.1 * t
         elif leaf.startswith("norm") or name in ("final.norm", "embed.norm"):
             t = 1 + 0.1 * t if shape.sandwich else 0.1 * t
         elif leaf.endswith("norm"):

@@ -15,11 +15,17 @@ from .feed_forward import GLUWeights, MLPWeights
 from .hybrid_config import AttentionSpec, DeltaSpec, DenseSpec, HybridShape, LatentSpec, random_tensors, tensor_shapes
 from .hyper import Connection
 from .latent_attention import LatentWeights
+from .residual import Norm, TanhNorm
 from .ssm import SSMWeights
 from .window_attention import AttentionWeights
 
 MixerWeights = Union[LatentWeights, AttentionWeights, SSMWeights, DeltaWeights]
 FFWeights = Union[MLPWeights, GLUWeights, MixtureWeights]
+
+
+# (activation, score, what the score multiplies, gate of the shared expert) the mixture's kernels take
+MIXTURE_FORMS = {("silu", "sigmoid", "input", True), ("relu2", "softmax", "output", False),
+                 ("relu2", "sigmoid", "output", False)}
 
 
 def _up8(n: int) -> int:
@@ -46,7 +52,7 @@ class HybridLayerWeights:
     mixer: MixerWeights
     mlp: Optional[FFWeights]
     hc: list = field(default_factory=list)      # hyper-connections: Connection of the mixer (and of the feed-forward)
-    norms: list = field(default_factory=list)   # norms on both sides: (before, after) of each, fp32
+    norms: list = field(default_factory=list)   # norms on both sides: (before, after) of each
 
 
 @dataclass
@@ -57,9 +63,9 @@ class HybridWeights:
     dtype: torch.dtype
     embed: torch.Tensor
     layers: list = field(default_factory=list)
-    final_norm: Optional[torch.Tensor] = None
+    final_norm: Optional[Norm] = None
     head: Optional[torch.Tensor] = None
-    embed_norm: Optional[torch.Tensor] = None
+    embed_norm: Optional[Norm] = None
     loop_step: Optional[torch.Tensor] = None     # [times, width] fp32
 
     @property
@@ -75,10 +81,17 @@ class HybridWeights:
             if tuple(tensors[name].shape) != dims:
                 raise ValueError(f"tensor {name} is {tuple(tensors[name].shape)}, the configuration says {dims}")
         b = _Builder(tensors, shape.width, dtype, device)
-        out = HybridWeights(shape, dtype, embed=b.mat(tensors["embed"]), final_norm=b.vec(tensors["final.norm"]),
-                            head=b.mat(_pad_cols(tensors["head"], 1, b.W8)))
+        norm = b.tanh_norm if shape.tanh_norms else lambda name: b.vec(tensors[name])
+        out = HybridWeights(shape, dtype, embed=b.mat(tensors["embed"]), final_norm=norm("final.norm"))
+        if shape.tied and b.W8 == shape.width:
+            out.head = out.embed
+        else:
+            out.head = b.mat(_pad_cols(tensors["embed" if shape.tied else "head"], 1, b.W8))
+        if shape.logit_scale != 1.0:     # the logits' factor rides on the last norm
+            f = out.final_norm
+            out.final_norm = TanhNorm(f.weight * shape.logit_scale, f.bias * shape.logit_scale, f.alpha)
         if shape.sandwich:
-            out.embed_norm = b.vec(tensors["embed.norm"])
+            out.embed_norm = norm("embed.norm")
             if shape.loop is not None:
                 out.loop_step = b.vec(tensors["loop.step"])
         for i, layer in enumerate(shape.layers):
@@ -89,7 +102,7 @@ class HybridWeights:
             lw = HybridLayerWeights(b.mixer(p + "mix.", layer.mixer), None if spec is None else b.ff(p + "mlp.", spec))
             for q in ([1] if spec is None else [1, 2]):
                 if shape.sandwich:
-                    lw.norms.append((b.vec(tensors[f"{p}norm{q}"]), b.vec(tensors[f"{p}norm{q}b"])))
+                    lw.norms.append((norm(f"{p}norm{q}"), norm(f"{p}norm{q}b")))
                 else:
                     hc = f"{p}hc{q}."
                     lw.hc.append(Connection(read=b.vec(tensors[hc + "in"]), mix=b.vec(tensors[hc + "mix"]),
@@ -130,6 +143,10 @@ class _Builder:
 
     def vec(self, t):
         return t.to(device=self.device, dtype=torch.float32).contiguous()
+
+    def tanh_norm(self, name):
+        t = self.tensors
+        return TanhNorm(self.vec(t[name]), self.vec(t[name + ".b"]), float(t[name + ".alpha"]))
 
     def in_proj(self, parts):
         """Row blocks that read the layer's input, stacked; rows up to a multiple of 8."""
@@ -172,10 +189,28 @@ class _Builder:
     def attention(self, p, m):
         H, G, DK, DV = m.heads, m.kv_heads, _up8(m.dim), _up8(m.vdim)
         get = lambda n: self.tensors[p + n]   # noqa: E731
-        return AttentionWeights(w_in=self.in_proj([_pad_rows(get("q"), H, DK), _pad_rows(get("k"), G, DK),
-                                                   _pad_rows(get("v"), G, DV)]),
-                                w_out=self.mat(_pad_cols(get("o"), H, DV)), heads=H, kv_heads=G, DK=DK, DV=DV,
-                                scale=m.scale, window=m.window)
+        wide = {"q": (H, DK), "k": (G, DK), "v": (G, DV)}
+        names = "qk" if m.keys_as_values else "qkv"
+        rows, more = [_pad_rows(get(n), *wide[n]) for n in names], {}
+        if m.gate is not None:
+            rows.append(_pad_rows(get("g"), H, DV if m.gate == "column" else 1))
+        w_in = self.in_proj(rows)
+        if m.bias:
+            b = torch.cat([_pad_rows(get(n + ".b"), *wide[n]) for n in names])
+            more["b_in"] = self.mat(torch.cat([b, b.new_zeros(w_in.shape[0] - b.numel())]))
+        if m.qk_norm is not None:
+            more.update({n + "_norm": self.vec(_pad_rows(get(n + ".norm"), wide[n][0] if m.qk_norm == "all" else 1, DK))
+                         for n in "qk"})
+        if m.conv is not None:
+            more["conv_w"] = self.vec(torch.cat([_pad_rows(get(n + ".conv"), *wide[n]) for n in "qk"]).t())
+        if m.sink is not None:
+            more["sink"] = self.vec(get("sink")) if m.sink == "learned" else torch.zeros(H, device=self.device)
+        if m.rot is not None and m.rot.dims:
+            freq, more["rot_mag"] = m.rot.frequencies()
+            more.update(inv_freq=self.vec(freq), rot_half=m.rot.half)
+        return AttentionWeights(w_in=w_in, w_out=self.mat(_pad_cols(get("o"), H, DV)), heads=H, kv_heads=G, DK=DK, DV=DV,
+                                scale=m.scale, window=m.window, chunk=m.chunk, softcap=m.softcap, gate=m.gate,
+                                keys_as_values=m.keys_as_values, qk_norm=m.qk_norm, dim=m.dim, **more)
 
     def ssm(self, p, m):
         H, P, G, N = m.heads, _up8(m.vdim), m.groups, _up8(m.state)
@@ -213,29 +248,36 @@ class _Builder:
             return self.glu(p, spec.ff, "gelu_tanh") if spec.gated else self.mlp(p, spec.ff)
         return self.mixture(p, spec)
 
-    def mlp(self, p, ff):
+    def mlp(self, p, ff, act="gelu_tanh", bias=True):
         F8, get = _up8(ff), lambda n: self.tensors[p + n]
-        return MLPWeights(up=self.mat(_pad_cols(_pad_rows(get("up"), 1, F8), 1, self.W8)),
-                          up_b=self.mat(_pad_rows(get("up.b"), 1, F8)), down=self.mat(_pad_cols(get("down"), 1, F8)),
-                          down_b=self.mat(get("down.b")))
+        more = dict(up_b=self.mat(_pad_rows(get("up.b"), 1, F8)), down_b=self.mat(get("down.b"))) if bias else {}
+        return MLPWeights(up=self._rows(p, ("up",), ff), down=self.mat(_pad_cols(get("down"), 1, F8)), act=act, **more)
 
-    def _gate_up(self, p, ff):
+    def _rows(self, p, names, ff):
+        """The named [ff, width] tensors, stacked."""
         F8 = _up8(ff)
-        return self.mat(_pad_cols(torch.cat([_pad_rows(self.tensors[p + n], 1, F8) for n in ("gate", "up")]), 1, self.W8))
+        return self.mat(_pad_cols(torch.cat([_pad_rows(self.tensors[p + n], 1, F8) for n in names]), 1, self.W8))
 
     def glu(self, p, ff, act):
-        return GLUWeights(gate_up=self._gate_up(p, ff), down=self.mat(_pad_cols(self.tensors[p + "down"], 1, _up8(ff))),
+        return GLUWeights(gate_up=self._rows(p, ("gate", "up"), ff), down=self.mat(_pad_cols(self.tensors[p + "down"], 1, _up8(ff))),
                           act=act)
 
     def mixture(self, p, spec):
-        rows = [self.tensors[p + "router"]]
-        shared = None
-        if spec.shared_ff is not None:
+        form = (spec.act, spec.score, spec.score_on, spec.shared_gate)
+        if form not in MIXTURE_FORMS or (spec.act == "silu" and (spec.correction or spec.groups != (1, 1))):
+            raise NotImplementedError(f"mixture {spec}")
+        rows, shared, plain = [self.tensors[p + "router"]], None, spec.act == "relu2"
+        if spec.shared_ff is not None and plain:
+            shared = self.mlp(p + "shared.", spec.shared_ff, spec.act, False)
+        elif spec.shared_ff is not None:
             shared = self.glu(p + "shared.", spec.shared_ff, "silu")
             rows.append(self.tensors[p + "shared.sg"])
+        up = ("up",) if plain else ("gate", "up")
         # the output rows of an expert are padded like the layer's input, so that its rows are 16-byte multiples
         down = [self.mat(_pad_rows(_pad_cols(self.tensors[f"{p}e{e}.down"], 1, _up8(spec.ff)), 1, self.W8))
                 for e in range(spec.experts)]
         return MixtureWeights(router=self.mat(_pad_cols(torch.cat(rows), 1, self.W8)),
-                              gate_up=torch.stack([self._gate_up(f"{p}e{e}.", spec.ff) for e in range(spec.experts)]),
-                              down=torch.stack(down), experts=spec.experts, top=spec.top, shared=shared)
+                              gate_up=torch.stack([self._rows(f"{p}e{e}.", up, spec.ff) for e in range(spec.experts)]),
+                              down=torch.stack(down), experts=spec.experts, top=spec.top, shared=shared, act=spec.act,
+                              score=spec.score, groups=spec.groups,
+                              correction=self.vec(self.tensors[p + "correction"]) if spec.correction else None)

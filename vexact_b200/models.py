@@ -297,6 +297,7 @@ def _load_stage(cfg, folder, dtype, device):
 MODEL_LOADERS = {
     "Nurazen": _load_hybrid,
     "Dekerax": _load_hybrid,
+    "Tekilix": _load_hybrid,
     "qwen2": _load_stage,
     "qwen3": _load_stage,
     "qwen3_moe": _load_stage,

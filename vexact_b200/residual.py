@@ -2,6 +2,7 @@
 (`csrc/residual.cuh`): one launch adds the normed output of the sublayer just done and norms the input of the next."""
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional, Union
 
 import torch
@@ -10,16 +11,28 @@ from . import _lib
 from .fused_moe import PendingMixture
 
 
-def residual_step(x: torch.Tensor, *, post: torch.Tensor, y: Union[torch.Tensor, PendingMixture, None] = None,
-                  embed: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
-                  add: Optional[torch.Tensor] = None, norm: Optional[torch.Tensor] = None, eps: float = 0.0,
-                  rows: Optional[torch.Tensor] = None, xn_cols: Optional[int] = None,
-                  dtype=torch.bfloat16) -> Optional[torch.Tensor]:
-    """x [T, W] <- x + rms_norm(y) * post (+ add) in place; returns rms_norm(x) * norm as [R, xn_cols], zero beyond W
-    (None without `norm`).
+@dataclass
+class TanhNorm:
+    """tanh(alpha x) * weight + bias (fp32 vectors): a norm that computes no mean or variance."""
 
-    y: rows of the model dtype, or the pending sum of a mixture; without y the model starts, x = rms_norm(embed[ids]) *
-    post (+ add).  `rows` (int32): only these tokens, and nothing is written back (the end of a model)."""
+    weight: torch.Tensor
+    bias: torch.Tensor
+    alpha: float
+
+
+Norm = Union[torch.Tensor, TanhNorm]     # a tensor: the weight of a division by the root mean square
+
+
+def residual_step(x: torch.Tensor, *, post: Norm, y: Union[torch.Tensor, PendingMixture, None] = None,
+                  embed: Optional[torch.Tensor] = None, ids: Optional[torch.Tensor] = None,
+                  add: Optional[torch.Tensor] = None, norm: Optional[Norm] = None, eps: float = 0.0,
+                  rows: Optional[torch.Tensor] = None, xn_cols: Optional[int] = None, embed_scale: float = 1.0,
+                  dtype=torch.bfloat16) -> Optional[torch.Tensor]:
+    """x [T, W] <- x + post(y) (+ add) in place; returns norm(x) as [R, xn_cols], zero beyond W (None without `norm`).
+    post(v) = rms_norm(v) * post, or both norms are a `TanhNorm`.
+
+    y: rows of the model dtype, or the pending sum of a mixture; without y the model starts, x = post(embed[ids] *
+    embed_scale) (+ add).  `rows` (int32): only these tokens, and nothing is written back (the end of a model)."""
     T, W = x.shape
     R = T if rows is None else rows.numel()
     xn = None
@@ -32,12 +45,20 @@ def residual_step(x: torch.Tensor, *, post: torch.Tensor, y: Union[torch.Tensor,
     for t in (y, extra):
         if t is not None and (t.dtype != dtype or t.stride(-1) != 1):
             raise ValueError("residual_step: y must be rows of the model dtype")
+    pb = nb = None
+    pa = na = 0.0
+    if isinstance(post, TanhNorm):
+        if norm is not None and not isinstance(norm, TanhNorm):
+            raise ValueError("residual_step: both norms are of one kind")
+        post, pb, pa = post.weight, post.bias, post.alpha
+        if norm is not None:
+            norm, nb, na = norm.weight, norm.bias, norm.alpha
     _lib.check(
         _lib.load().b200_residual_step(
             x.data_ptr(), _lib.ptr(y), 0 if y is None else y.stride(0), y_rows, _lib.ptr(scatter), topk, _lib.ptr(extra),
             0 if extra is None else extra.stride(0), _lib.ptr(embed), _lib.ptr(ids),
             0 if embed is None else embed.shape[0], _lib.ptr(rows), T, R, W, post.data_ptr(), _lib.ptr(add),
-            _lib.ptr(norm), float(eps), _lib.ptr(xn), 0 if xn is None else xn.stride(0), 0 if xn is None else xn.shape[1],
+            _lib.ptr(norm), float(eps), float(embed_scale), _lib.ptr(pb), float(pa), _lib.ptr(nb), float(na), _lib.ptr(xn), 0 if xn is None else xn.stride(0), 0 if xn is None else xn.shape[1],
             0 if rows is not None else 1, 0 if dtype == torch.bfloat16 else 1, _lib.current_stream()),
         "b200_residual_step")
     return xn
