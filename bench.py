@@ -81,6 +81,10 @@ def parse_args():
                     help="side measurement: prefill and decode steps of the Dekerax decoders (gated delta rule, windowed "
                          "attention and latent attention, mixtures) beside a grouped-query MoE model and the state-space "
                          "hybrid of equal width, and its kernels beside theirs")
+    ap.add_argument("--tekilix", action="store_true",
+                    help="side measurement: prefill and decode steps of the Tekilix decoders (chunked attention with sinks, "
+                         "capped scores and gates, convolved keys, grouped choice of experts, dynamic tanh) beside the "
+                         "grouped-query MoE model of equal width, and its kernels beside that model's")
     ap.add_argument("--prefill-attention", type=int, default=0, metavar="QLEN",
                     help="side measurement: time one causal prefill attention call of QLEN queries on the "
                          "model's head shape (context --ctx if larger) and print its own JSON line")
@@ -790,8 +794,13 @@ def hybrid_model_case(args, shape, kind, S, new, total, page, device):
                 step.__dict__.pop(k, None)
             return runner.logits(runner.forward(step, rows))
 
-        seen = {run: min(total, (getattr(w.layers[i].mixer, "window", None) or total) + new - 1)
-                for run, (i, _) in enumerate(shape.runs)}
+        def reach(mixer):      # keys that some new token sees
+            chunk = getattr(mixer, "chunk", None)
+            if chunk:
+                return total - (total - new) // chunk * chunk
+            return min(total, (getattr(mixer, "window", None) or total) + new - 1)
+
+        seen = {run: reach(w.layers[i].mixer) for run, (i, _) in enumerate(shape.runs)}
         cache_bytes = sum(S * seen[run] * t[0, 0].numel() * 2 for d in (runner.store.key_cache, runner.store.value_cache)
                           for run, t in d.items())
         cache_bytes += 2 * sum(t.numel() * t.element_size() for d in (runner.store.conv_state, runner.store.ssm_state)
@@ -1223,6 +1232,201 @@ def dekerax_kernels(device):
         torch.cuda.empty_cache()
 
 
+# --------------------------------------------------------------------------- Tekilix decoders
+TK_CHUNK = 1024
+
+
+def tekilix_shapes():
+    """(Tekilix: 8 layers of the two kinds in turn, the grouped-query MoE model), equal width, heads, experts and expert
+    width.  The other model's experts are gated (three matrices), these are not (two) and have a shared one beside them."""
+    from vexact_b200.hybrid import AttentionSpec, HybridLayer, HybridShape, MixtureSpec, RotarySpec, YarnSpec
+    from vexact_b200.inferencer import ModelShape, MoEShape
+
+    W, V, E, TOP, FF = 2048, 32768, 64, 4, 1024
+    common = dict(heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, chunk=TK_CHUNK)
+    first = AttentionSpec(**common, rot=RotarySpec(10000.0, 64, False), bias=True, qk_norm="all", softcap=30.0, sink="unit",
+                          gate="head")
+    second = AttentionSpec(**common, rot=RotarySpec(1e6, 128, True, YarnSpec(8.0, 1024.0, 32.0, 1.0)), qk_norm="head", conv=4,
+                           keys_as_values=True, sink="learned", gate="column")
+    mix = MixtureSpec(E, TOP, FF, FF, "relu2", "softmax", "output", False, True, (8, 4))
+    layers = tuple(HybridLayer((first, second)[i % 2], mix, i) for i in range(8))
+    return (HybridShape("tekilix-8", layers, W, V, 1, 1.0, 1e-6, "Tekilix", embed_scale=W ** 0.5, logit_scale=0.25),
+            ModelShape("gqa-moe", 8, W, 16, 4, 128, V, moe=MoEShape(E, TOP, FF), qk_norm=True, rms_eps=1e-6))
+
+
+def run_tekilix(args):
+    """Side measurement: steps of the Tekilix decoders beside the closest other model (random weights), then its kernels
+    beside the like kernels of that one."""
+    from vexact_b200 import _lib
+
+    device = torch.device("cuda", 0)
+    torch.cuda.set_device(device)
+    cases = [("decode", 64, 1, 4096), ("decode", 256, 1, 1024), ("prefill", 4, 2048, 2048), ("prefill", 1, 2048, 8192)]
+    clocks = ClockSampler(0)
+    clocks.start()
+    clocks.wait_first_sample()
+    for shape in tekilix_shapes():
+        for kind, S, new, total in cases:
+            print(json.dumps(hybrid_model_case(args, shape, kind, S, new, total, DK_PAGE, device)), flush=True)
+            torch.cuda.empty_cache()
+    for line in tekilix_kernels(device):
+        print(json.dumps(line), flush=True)
+    print(json.dumps({"measurement": "tekilix", "clocks": clocks.stop(), "status": list(_lib.read_status())}))
+
+
+def tekilix_kernels(device):
+    """Per kernel of the Tekilix decoders and the like kernel of the grouped-query MoE model (and, for attention, the same
+    kernel without caps, sinks, gates and chunks): device time, achieved bytes or flops over the measured peak.  Several
+    buffers per kernel, together larger than L2."""
+    import vexact_b200 as vb
+    from vexact_b200 import _lib, fused_moe as fm, window_attention as wa
+    from vexact_b200.batch_invariant_ops import gemm
+    from vexact_b200.feed_forward import mlp_forward
+    from vexact_b200.hybrid import HybridLayer, HybridShape, HybridWeights
+    from vexact_b200.residual import residual_step
+
+    peaks = measured_peaks()
+    hbm, tc = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    BF = torch.bfloat16
+    tek, _ = tekilix_shapes()
+    few = HybridShape("few", tuple(HybridLayer(tek.layers[i].mixer, tek.layers[i].ff, i) for i in range(2)), tek.width, 1024, 1,
+                      1.0, 1e-6, "Tekilix")
+    w = HybridWeights.random_init(few, device=device)
+    layer = w.layers[0]
+    mixers = {"attention": layer.mixer, "attention_2": w.layers[1].mixer}
+    mix, (before, after), W = layer.mlp, layer.norms[0], tek.width
+    rn = lambda *s: torch.randn(s, device=device).to(BF)   # noqa: E731
+
+    def line(name, ms, nbytes=None, flops=None, like=None):
+        out = {"measurement": "tekilix_kernel", "kernel": name, "us": round(ms * 1e3, 2)}
+        fr = []
+        if nbytes:
+            out["gb_s"] = round(nbytes / ms / 1e6)
+            fr.append(nbytes / ms / 1e6 / hbm)
+        if flops:
+            out["tflop_s"] = round(flops / ms / 1e9, 1)
+            fr.append(flops / ms / 1e9 / tc)
+        out["of_measured_roofline"] = round(max(fr), 3)
+        if like:
+            out["like"] = like
+        return out
+
+    nw = rn(W)
+    for T in (64, 8192):
+        k = 24 if T == 64 else 3
+        st, blocks = hybrid_step([(1, 100)] * T if T == 64 else [(T // 4, T // 4)] * 4, DK_PAGE, device)
+        S = st.state_slots.numel()
+        sets = [(torch.randn(T, W, device=device), rn(T, W)) for _ in range(k)]
+        ms = graph_ms([lambda x=x, y=y: residual_step(x, y=y, post=after, norm=before) for x, y in sets])
+        yield line(f"residual_step, dynamic tanh T={T}", ms, T * W * 12)
+        ms = graph_ms([lambda x=x, y=y: vb.add_rms_norm(y, rn_y, nw, 1e-6) for (x, y), rn_y in zip(sets, [rn(T, W) for _ in sets])])
+        yield line(f"add_rmsnorm T={T}", ms, T * W * 8, like=f"residual_step, dynamic tanh T={T}")
+        top, E = mix.top, mix.experts
+        scatter = torch.randperm(T * top, device=device).to(torch.int32)
+        pend = [(x, fm.PendingMixture(rn(T * top, W), scatter, top, y)) for x, y in sets]
+        ms = graph_ms([lambda x=x, y=y: residual_step(x, y=y, post=after, norm=before) for x, y in pend])
+        yield line(f"residual_step, dynamic tanh, of a mixture T={T}", ms, T * W * (10 + 2 * (top + 1)))
+        ms = graph_ms([lambda y=y: fm.PendingMoE(y.rows, scatter, None, T, top, W, (T, W)).add_norm(y.shared, nw, 1e-6)
+                       for _, y in pend])
+        yield line(f"moe_unpermute_add_rmsnorm T={T}", ms, T * W * (6 + 2 * top),
+                   like=f"residual_step, dynamic tanh, of a mixture T={T}")
+        del pend
+        # mixture: route + permute + two grouped products, without the sum (in the boundary) and the shared expert
+        xs = [y for _, y in sets]
+        rows, F = T * top, mix.gate_up.shape[1]
+        live = min(E, rows)
+        lone = mix.__class__(**{**vars(mix), "shared": None})
+        ms = graph_ms([lambda x=x: fm.mixture_forward(lone, x) for x in xs])
+        yield line(f"mixture (router to second product) T={T}", ms, 2 * (live * 2 * F * W + rows * (2 * W + 2 * F) + T * W),
+                   4.0 * rows * F * W)
+        gated = torch.cat([mix.gate_up, mix.gate_up], 1)
+
+        def moe(x):
+            rw, sel, plan = fm.route_plan_softmax_topk(vb.linear(x, mix.router), top, True, E)
+            return fm.fused_moe_forward(E, rw, sel, x, fc2_weight=mix.down, fc1_1_2_weight=gated, defer_reduce=True, plan=plan)
+
+        ms = graph_ms([lambda x=x: moe(x) for x in xs])
+        yield line(f"fused_moe (router to second product) T={T}", ms, 2 * (live * 3 * F * W + rows * (2 * W + 2 * F) + T * W),
+                   6.0 * rows * F * W, like=f"mixture (router to second product) T={T}")
+        del gated
+        logits = [torch.randn(T, E, device=device) for _ in range(k)]
+        ms = graph_ms([lambda z=z: fm.route_plan_group_topk(z, top, E, correction=mix.correction, groups=mix.groups) for z in logits])
+        yield line(f"route_plan_group_topk T={T}", ms, T * (E * 4 + top * 16))
+        ms = graph_ms([lambda z=z: fm.route_plan_softmax_topk(z, top, True, E) for z in logits])
+        yield line(f"route_plan_softmax_topk T={T}", ms, T * (E * 4 + top * 14), like=f"route_plan_group_topk T={T}")
+        sh = mix.shared
+        copies = [sh.__class__(up=sh.up.clone(), down=sh.down.clone(), act=sh.act) for _ in range(12)]
+        nbytes, flops = 2 * (2 * sh.up.numel() + 2 * T * W), 4.0 * T * sh.up.numel()
+        ms = graph_ms([lambda x=x, c=c: mlp_forward(c, x) for x, c in zip(xs, copies * 2)])
+        yield line(f"shared expert T={T}", ms, nbytes, flops)
+        ms = graph_ms([lambda x=x, c=c: gemm(gemm(x, c.up), c.down) for x, c in zip(xs, copies * 2)])
+        yield line(f"its two products alone, plain gemm T={T}", ms, nbytes, flops, like=f"shared expert T={T}")
+        del copies, sets, xs, logits
+        torch.cuda.empty_cache()
+        # what lies between the projections and attention
+        kc, vc = (torch.zeros(blocks, DK_PAGE, 4, 128, device=device, dtype=BF) for _ in range(2))
+        for name, m in mixers.items():
+            proj = [rn(T, m.w_in.shape[0]) for _ in range(k)]
+            conv = [torch.zeros(S, 3, m.qk_cols, device=device, dtype=BF) for _ in range(k)] if m.conv_w is not None else [None] * k
+            nbytes = T * 2 * (2 * m.qk_cols + (2 if m.conv_w is None else 1) * 512) + (12 * S * m.qk_cols if m.conv_w is not None else 0)
+            ms = graph_ms([lambda p=p, c=c: wa.attn_prep(m, p, kc, vc, c, st, 1e-6) for p, c in zip(proj, conv)])
+            yield line(f"attn_prep of {name} T={T}", ms, nbytes)
+        qkv, qn = [rn(T, 24 * 128) for _ in range(k)], rn(128)
+        freq, q_out = torch.rand(64, device=device), torch.empty(T, 2048, device=device, dtype=BF)
+        ms = graph_ms([lambda p=p: _lib.check(_lib.load().b200_qknorm_rope_store(
+            p.data_ptr(), p.stride(0), st.positions.data_ptr(), st.slot_mapping.data_ptr(), qn.data_ptr(), qn.data_ptr(),
+            freq.data_ptr(), q_out.data_ptr(), kc.data_ptr(), vc.data_ptr(), T, 16, 4, 128, blocks * DK_PAGE, 1e-6,
+            _lib.current_stream()), "b200_qknorm_rope_store") for p in qkv])
+        yield line(f"qknorm_rope_store T={T}", ms, T * 2 * 2 * 24 * 128, like=f"attn_prep of attention T={T}")
+        del proj, conv, qkv, kc, vc
+        torch.cuda.empty_cache()
+    plain = wa.AttentionWeights(w_in=None, w_out=None, heads=16, kv_heads=4, DK=128, DV=128, scale=128 ** -0.5)
+
+    def gate_of(m, T):
+        return None if m.gate is None else rn(T, m.w_in.shape[0])[:, m.gate_off:]
+
+    # attention of decoded tokens: a chunk of 1024 in 4096 keys, and a context of 1024
+    for S, ctx in ((64, 4096), (256, 1024), (64, 1024)):
+        st, blocks = hybrid_step([(1, ctx)] * S, DK_PAGE, device)
+        n = min(ctx, TK_CHUNK)
+        sets = [(rn(S, 2048), rn(blocks, DK_PAGE, 4, 128), rn(blocks, DK_PAGE, 4, 128),
+                 torch.empty(S, 2048, device=device, dtype=BF)) for _ in range(2 if ctx * S > 200000 else 4)]
+        for name, m in mixers.items():
+            gate = gate_of(m, S)
+            ms = graph_ms([lambda s=s: wa.attend_decode(m, *s, st, gate=gate) for s in sets])
+            yield line(f"{name} decode {S}x{ctx}", ms, S * n * 4 * 256 * 2)
+        if ctx == n:
+            ms = graph_ms([lambda s=s: wa.attend_decode(plain, *s, st) for s in sets])
+            yield line(f"the kernel without extras, decode {S}x{ctx}", ms, S * n * 4 * 256 * 2)
+            ms = graph_ms([lambda s=s: vb.paged_attention(s[0].view(S, 16, 128), s[1], s[2], st.query_start_loc, st.context_lens,
+                                                          st.block_tables, 128 ** -0.5, 1) for s in sets])
+            yield line(f"paged_attn 128/128 decode {S}x{ctx}", ms, S * n * 4 * 256 * 2, like=f"attention decode {S}x{ctx}")
+        del sets
+        torch.cuda.empty_cache()
+    # attention of prompts: chunks of 1024, and one chunk as long as the context
+    for S, new, total in ((4, 2048, 2048), (1, 2048, 8192)):
+        st, blocks = hybrid_step([(new, total)] * S, DK_PAGE, device)
+        T = S * new
+        q, kc, vc = rn(T, 16 * 128), rn(blocks, DK_PAGE, 4, 128), rn(blocks, DK_PAGE, 4, 128)
+        out, longs = torch.empty(T, 16 * 128, device=device, dtype=BF), wa._long_sequences(st, device)[0]
+        pairs = lambda c: S * sum(t % c + 1 for t in range(total - new, total))   # noqa: E731
+        for name, m in mixers.items():
+            gate = gate_of(m, T)
+            ms = graph_ms([lambda: wa.attend_prefill(m, q, kc, vc, out, st, longs, gate=gate)])
+            yield line(f"{name} prefill {S}x{new}/{total}", ms, None, 2.0 * pairs(TK_CHUNK) * 16 * 256)
+            wide = m.__class__(**{**vars(m), "chunk": total})
+            ms = graph_ms([lambda: wa.attend_prefill(wide, q, kc, vc, out, st, longs, gate=gate)])
+            yield line(f"{name} prefill, one chunk {S}x{new}/{total}", ms, None, 2.0 * pairs(total) * 16 * 256)
+        ms = graph_ms([lambda: wa.attend_prefill(plain, q, kc, vc, out, st, longs)])
+        yield line(f"the kernel without extras, prefill {S}x{new}/{total}", ms, None, 2.0 * pairs(total) * 16 * 256)
+        ms = graph_ms([lambda: vb.paged_attention(q.view(T, 16, 128), kc, vc, st.query_start_loc, st.context_lens, st.block_tables,
+                                                  128 ** -0.5, new)])
+        yield line(f"paged_attn 128/128 prefill {S}x{new}/{total}", ms, None, 2.0 * pairs(total) * 16 * 256,
+                   like=f"attention prefill, one chunk {S}x{new}/{total}")
+        del q, kc, vc
+        torch.cuda.empty_cache()
+
+
 def main():
     args = parse_args()
     rank = int(os.environ.get("RANK", "0"))
@@ -1242,6 +1446,9 @@ def main():
         return
     if args.dekerax:
         run_dekerax(args)
+        return
+    if args.tekilix:
+        run_tekilix(args)
         return
     if args.skew:
         run_skew(args, shape)

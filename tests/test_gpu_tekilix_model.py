@@ -1,0 +1,321 @@
+"""Whole Tekilix models through the engine: `Inferencer` steps, pages, convolution state, scheduler, sampling, command line and
+trace replay, against the plain model of oracle/tekilix.py in double precision."""
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+import tekilix_util as tu
+from conftest import ROOT
+from oracle import tekilix as ot
+
+pytestmark = pytest.mark.gpu
+BF, F32 = torch.bfloat16, torch.float32
+# largest relative root mean square error of a position's logits
+TOL = {F32: 3e-5, BF: 5e-2}
+N = 150
+
+
+def _apart(w):
+    """Router weights whose scores lie apart, so that no rounding decides which experts a token takes."""
+    return {k: (v.float() * 3).to(BF) if k.endswith("mlp.router") else v for k, v in w.items()}
+
+
+def _steady(cfg, w, toks, gap=0.01):
+    """The plain model's logits, and the positions up to which none of its routers had a close call."""
+    ok = torch.ones(len(toks), dtype=torch.bool)
+    plain = ot.mixture
+
+    def spy(h, sub, c):
+        r = c["router"]
+        if r["top"] < r["experts"]:
+            s = torch.softmax(h @ sub["router"].T, -1) + sub["correction"]
+            best = s.view(len(h), r["groups"]["count"], -1).max(-1).values.sort(-1, descending=True).values
+            if r["groups"]["keep"] < r["groups"]["count"]:
+                ok.logical_and_(best[:, r["groups"]["keep"] - 1] - best[:, r["groups"]["keep"]] > gap)
+            for t in range(len(h)):
+                chosen = ot.route(torch.softmax(h[t] @ sub["router"].T, -1), sub["correction"], c)
+                floor = best[t, r["groups"]["keep"] - 1]
+                per = r["experts"] // r["groups"]["count"]
+                left = [float(s[t, e]) for e in range(r["experts"])
+                        if e not in chosen and s[t, e // per * per:e // per * per + per].max() >= floor]
+                if left and float(s[t, chosen[-1]]) - max(left) <= gap:
+                    ok[t] = False
+        return plain(h, sub, c)
+
+    ot.mixture = spy
+    try:
+        logits = ot.forward(cfg, tu.as_double(w), toks)
+    finally:
+        ot.mixture = plain
+    return logits, ok.long().cumprod(0).bool()
+
+
+@pytest.fixture(scope="module")
+def ref():
+    """(configuration, tensors, prompt, its logits, positions before a close call) per configuration, computed once."""
+    cache = {}
+
+    def get(name, n=N):
+        if name not in cache:
+            cfg = tu.CONFIGS[name]
+            w = _apart(tu.weights(cfg, seed=len(name)))
+            toks = tu.tokens(n, cfg["vocab"], seed=3)
+            cache[name] = (cfg, w, toks) + _steady(cfg, w, toks)
+        return cache[name]
+
+    return get
+
+
+def _check(got, want, dtype, ok, what):
+    """fp32: every position.  bf16: every position before a router's first close call, and most of the others (a token that
+    takes another expert leaves other keys behind, which later tokens see)."""
+    got, want = got.double().cpu(), want.double()
+    err = ((got - want).pow(2).mean(-1) / want.pow(2).mean(-1)).sqrt()
+    if dtype == F32:
+        assert err.max() < TOL[F32], (what, err.max())
+    else:
+        assert err.median() < TOL[BF], (what, err.median())
+        assert not ok.any() or (err[ok].quantile(0.9) < TOL[BF] and err[ok].max() < 3 * TOL[BF]), (what, err[ok])
+
+
+def _run(eng, toks, cuts, req=None):
+    """Feeds `toks` in portions of the given sizes (the last one repeats); logits of every position."""
+    from vexact_b200.scheduler import Request
+
+    req = req or Request("r", [])
+    out, at, k = [], 0, 0
+    while at < len(toks):
+        n = min(cuts[min(k, len(cuts) - 1)], len(toks) - at)
+        out.append(eng.run_portions([(req, toks[at:at + n], range(n))]).cpu())
+        at += n
+        k += 1
+    return torch.cat(out), req
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+@pytest.mark.parametrize("name", list(tu.CONFIGS))
+def test_whole_prompt_portions_and_token_by_token(ref, name, dtype):
+    cfg, w, toks, want, ok = ref(name)
+    eng = tu.engine(cfg, w, dtype)
+    for cuts in ([N], [1], [2], [17, 2, 16, 33, 1, 64], [100, 1]):
+        got, req = _run(eng, toks, cuts)
+        _check(got, want, dtype, ok, cuts)
+        eng.close_request(req)     # the next run takes the same pages and the same slot again
+    assert eng.scheduler.kv.num_allocated_blocks() == 0 and eng.scheduler.slots.num_free() == 4
+
+
+@pytest.mark.parametrize("name", ["mixed", "odd"])
+def test_every_layer_against_the_plain_model(ref, name):
+    cfg, w, toks, _, _ = ref(name)
+    _, want = ot.forward(cfg, tu.as_double(w), toks, want_layers=True)
+    eng = tu.engine(cfg, w, F32, enforce_eager=True)
+    runner, got = eng.inferencer.model.runner, {}
+    plain = runner.forward
+    runner.forward = lambda step, rows: plain(step, rows, after_layer=lambda i, s: got.__setitem__(i, s.sum(1).cpu()))
+    _run(eng, toks, [N])
+    assert len(got) == len(want) == len(cfg["layers"])
+    for i in range(len(want)):
+        assert tu.rel_rms(got[i], want[i]) < 2e-5, i
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+def test_mixed_batches_equal_each_request_alone(ref, dtype):
+    """Portions of prompts beside decoded tokens, a request that pauses, one that ends and whose pages and slot are used
+    by the next; a pool that is exactly full."""
+    from vexact_b200.scheduler import Request
+
+    cfg, w, _, _, _ = ref("mixed" if dtype == F32 else "every_expert")
+    lens = {"a": 90, "b": 40, "c": 61, "d": 33, "e": 70}
+    toks = {k: tu.tokens(n, cfg["vocab"], seed=ord(k)) for k, n in lens.items()}
+    eng = tu.engine(cfg, w, dtype, max_cache_blocks=6 + 3 + 4 + 3, max_num_batched_tokens=128)
+    plan = [{"a": 50, "b": 2}, {"a": 1, "b": 30, "c": 20}, {"b": 8, "c": 2, "d": 31}, {"a": 1, "c": 1, "d": 1},
+            {"c": 38, "d": 1}, {"e": 40, "a": 20}, {"e": 1, "a": 1}, {"a": 17, "e": 29}]
+    live, at, got = {}, dict.fromkeys(lens, 0), {k: [] for k in lens}
+    for portions in plan:
+        entries = []
+        for k, n in portions.items():
+            req = live.setdefault(k, Request(k, []))
+            entries.append((req, toks[k][at[k]:at[k] + n], range(n)))
+        logits = eng.run_portions(entries).cpu()
+        row = 0
+        for k, n in portions.items():
+            got[k].append(logits[row:row + n])
+            row += n
+            at[k] += n
+            if at[k] == lens[k]:
+                eng.close_request(live.pop(k))
+    assert at == lens
+    for k in lens:
+        want, ok = _steady(cfg, w, toks[k])
+        _check(torch.cat(got[k]), want, dtype, ok, k)
+
+
+def test_logits_of_chosen_places_and_of_none(ref):
+    from vexact_b200.scheduler import Request
+
+    cfg, w, toks, want, _ = ref("mixed")
+    eng = tu.engine(cfg, w, F32)
+    a, b = Request("a", []), Request("b", [])
+    assert eng.run_portions([(a, toks[:60], [])]) is None
+    got = eng.run_portions([(a, toks[60:90], [29, 0, 7]), (b, toks[:5], []), ]).cpu()
+    assert tu.rel_rms(got, want[[89, 60, 67]]) < TOL[F32]
+    got = eng.run_portions([(b, toks[5:6], [0]), (a, toks[90:91], [])]).cpu()     # a decode graph of two
+    assert got.shape[0] == 1 and tu.rel_rms(got, want[[5]]) < TOL[F32]
+
+
+def test_long_decoding_crosses_chunks_pages_and_blocks():
+    """700 positions, the last 250 one by one, over the edges of every layer's chunk."""
+    cfg = tu.CONFIGS["wide"]
+    w = _apart(tu.weights(cfg, 5))
+    toks = tu.tokens(700, cfg["vocab"], seed=9)
+    want, ok = _steady(cfg, w, toks)
+    for dtype in (BF, F32):
+        eng = tu.engine(cfg, w, dtype, max_num_batched_tokens=832, max_model_len=832)
+        got, req = _run(eng, toks, [450, 1])
+        _check(got, want, dtype, ok, dtype)
+        eng.close_request(req)
+
+
+@pytest.mark.parametrize("cuts", [[N], [129, 1], [1], [64, 2, 63, 21]])
+@pytest.mark.parametrize("name", ["every_expert", "mixed"])
+def test_sharp_attention_finds_single_far_keys(ref, name, cuts):
+    """Scores spread so wide that single keys carry a head's weight: a key missed, seen too often or seen from another chunk
+    shows."""
+    cfg, w, toks, _, _ = ref(name)
+    w = {k: (v.float() * 4).to(BF) if k.endswith(".mix.q.norm") else v for k, v in w.items()}
+    want = ot.forward(cfg, tu.as_double(w), toks)
+    got, _ = _run(tu.engine(cfg, w, F32), toks, cuts)
+    assert tu.rel_rms(got, want) < 20 * TOL[F32]
+
+
+def test_faults_would_show(ref):
+    """The comparison is sharp enough: the plain model with one chunk off by one, another sink, no convolution state, swapped
+    groups, another scale or another rotation is far from the framework."""
+    cfg, w, toks, want, _ = ref("mixed")
+    got, _ = _run(tu.engine(cfg, w, F32), toks, [N])
+    assert tu.rel_rms(got, want) < TOL[F32]
+
+    def far(c=cfg, **changed):
+        return tu.rel_rms(got, ot.forward(c, tu.as_double(dict(w, **{k.replace("_", "."): v for k, v in changed.items()})), toks)) > 30 * TOL[F32]
+
+    def other(change):
+        c = json.loads(json.dumps(cfg))
+        change(c)
+        return c
+
+    for i in range(5):
+        assert far(other(lambda c: c["layers"][i]["mixer"]["mask"].__setitem__("size", c["layers"][i]["mixer"]["mask"]["size"] + 1))), i
+    assert far(other(lambda c: c["layers"][1]["mixer"]["rot"].pop("scaling")))
+    assert far(other(lambda c: c["layers"][0]["mixer"].__setitem__("softcap", 2.6)))
+    assert far(other(lambda c: c["layers"][0]["mlp"]["router"]["groups"].__setitem__("keep", 3)))
+    assert far(other(lambda c: c.__setitem__("logit_scale", 0.601))) and far(other(lambda c: c["embedding"].__setitem__("scale", 3.6)))
+    assert far(**{"l1_mix_sink": w["l1.mix.sink"] + 0.1, "l1_mix_q_conv": w["l1.mix.q.conv"]})
+    conv = w["l1.mix.k.conv"].clone()
+    conv[:, 0] = 0
+    assert far(**{"l1_mix_k_conv": conv}) and far(**{"l0_mix_v_b": 0 * w["l0.mix.v.b"]}) and far(**{"l0_norm1b_b": 0 * w["l0.norm1b.b"]})
+
+
+# ------------------------------------------------------------------ the engine's own generation
+def _greedy(cfg, w, prompt, n):
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(ot.forward(cfg, tu.as_double(w), toks)[-1].argmax()))
+    return toks[len(prompt):]
+
+
+def test_greedy_generation_through_the_scheduler(ref):
+    """More requests than slots, prompts cut by a small token budget, decoding beside prompts, with and without graphs."""
+    from vexact_b200.scheduler import GenerationConfig
+
+    cfg, w, _, _, _ = ref("mixed")
+    prompts = [tu.tokens(n, cfg["vocab"], seed=n) for n in (45, 3, 18, 1, 30, 7)]
+    want = [_greedy(cfg, w, p, 5) for p in prompts]
+    for eager in (False, True):
+        eng = tu.engine(cfg, w, F32, max_num_batched_tokens=24, max_model_len=64, enforce_eager=eager)
+        reqs = eng.generate(prompts, GenerationConfig(max_new_tokens=5, output_scores=True))
+        assert [r.generated_tokens for r in reqs] == want
+        assert all(len(r.logprobs) == 5 and max(r.logprobs) <= 0 for r in reqs)
+        assert eng.scheduler.kv.num_allocated_blocks() == 0 and eng.scheduler.slots.num_free() == 4
+
+
+def test_fused_greedy_head_of_a_tied_embedding(ref):
+    """Tokens from the fused output product equal the arg-max of the logits it does not write."""
+    from vexact_b200.engine import Engine
+    from vexact_b200.hybrid import HybridModel, HybridShape, HybridWeights
+    from vexact_b200.scheduler import GenerationConfig
+
+    cfg, w, toks, _, _ = ref("odd")
+    gen = GenerationConfig(max_new_tokens=6, output_scores=True)
+    out = []
+    for fused in (False, True):
+        model = HybridModel(HybridWeights.from_tensors(HybridShape.from_config(cfg), w, BF), fused_greedy=fused)
+        eng = Engine(model, max_num_seqs=4, max_num_batched_tokens=64, max_model_len=64, page_size=16)
+        out.append(eng.generate([toks[:20], toks[:3]], gen))
+    for a, b in zip(*out):
+        assert a.generated_tokens == b.generated_tokens
+        np.testing.assert_allclose(a.logprobs, b.logprobs, atol=0.05)
+
+
+def test_preempted_requests_start_over_and_end_the_same(ref):
+    from vexact_b200.scheduler import GenerationConfig
+
+    cfg, w, _, _, _ = ref("mixed")
+    prompts = [tu.tokens(n, cfg["vocab"], seed=n) for n in (30, 31, 29)]
+    big = tu.engine(cfg, w, F32, max_model_len=64)
+    want = [r.generated_tokens for r in big.generate(prompts, GenerationConfig(max_new_tokens=24))]
+    small = tu.engine(cfg, w, F32, max_model_len=64, max_cache_blocks=7)      # three requests need 4 pages each at the end
+    preempted = []
+    plain = small.scheduler._preempt
+    small.scheduler._preempt = lambda r: (preempted.append(r.request_id), plain(r))
+    got = [r.generated_tokens for r in small.generate(prompts, GenerationConfig(max_new_tokens=24))]
+    assert preempted and got == want
+
+
+def test_sampling_does_not_depend_on_the_batch(ref):
+    from vexact_b200.scheduler import GenerationConfig
+
+    cfg, w, toks, _, _ = ref("odd")
+    eng = tu.engine(cfg, w, BF)
+    cfgs = GenerationConfig(max_new_tokens=8, do_sample=True, temperature=0.8, top_k=20, top_p=0.9, seed=11)
+    first = [r.generated_tokens for r in eng.generate([toks[:9], toks[:4]], cfgs)]
+    assert first == [r.generated_tokens for r in eng.generate([toks[:9], toks[:4]], cfgs)]
+    assert first[0] == eng.generate([toks[:9]], cfgs)[0].generated_tokens
+
+
+def test_command_line_and_trace_replay(ref, tmp_path):
+    from vexact_b200.checkpoint import write_safetensors
+
+    cfg, w, toks, want, ok = ref("mixed")
+    model = tmp_path / "model"
+    model.mkdir()
+    (model / "config.json").write_text(json.dumps(cfg))
+    write_safetensors(model / "model.safetensors", w)
+    out = subprocess.run([sys.executable, "-m", "vexact_b200.generate", "--model", str(model), "--dtype", "float32",
+                          "--prompt", ",".join(map(str, toks[:12])), "--max-new-tokens", "4", "--logprobs",
+                          "--max-num-seqs", "2", "--max-model-len", "128"], cwd=ROOT, capture_output=True, text=True, timeout=120)
+    assert out.returncode == 0, out.stderr[-2000:]
+    line = json.loads(out.stdout.splitlines()[-1])
+    assert line["tokens"] == _greedy(cfg, w, toks[:12], 4) and len(line["logprobs"]) == 4
+
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:70], "want": [0, 69]}], "end": []},
+             {"step": 1, "entries": [{"id": "y", "tokens": toks[:2], "want": []}, {"id": "x", "tokens": toks[70:71], "want": []}],
+              "end": []},
+             {"step": 2, "entries": [{"id": "y", "tokens": toks[2:40], "want": [37, 5]}], "end": ["x"]},
+             {"step": 3, "entries": [{"id": "z", "tokens": toks[:64], "want": [63]}, {"id": "y", "tokens": toks[40:41], "want": [0]}],
+              "end": ["y", "z"]}]
+    rows = {0: [0, 69], 2: [39, 7], 3: [63, 40]}
+    for dtype in ("float32", "bfloat16"):
+        res = tmp_path / dtype
+        out = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", str(model), "--dtype", dtype, "--out",
+                              str(res), "--max-tokens", "192"], input="\n".join(map(json.dumps, steps)) + "\n",
+                             capture_output=True, text=True, timeout=120)
+        assert out.returncode == 0, out.stderr[-2000:]
+        assert [x for x in out.stdout.splitlines() if x.startswith("done")] == [f"done {i}" for i in range(4)]
+        got = torch.cat([torch.from_numpy(np.fromfile(res / f"{n}.f32", dtype="<f4")).view(len(at), -1) for n, at in rows.items()])
+        at = [i for r in rows.values() for i in r]
+        _check(got, want[at], getattr(torch, dtype), ok[at], dtype)

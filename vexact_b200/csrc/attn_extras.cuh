@@ -46,30 +46,35 @@ __device__ __forceinline__ float tanh_series(float x) {
   return fmaf(c * s, x, x);
 }
 __device__ __forceinline__ float tanh_exponential(float x) {
-  float e;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(fminf(fabsf(x), 40.f) * 2.885390081777927f));
-  return copysignf(1.f - __fdividef(2.f, e + 1.f), x);
+  return copysignf(1.f - __fdividef(2.f, __expf(2.f * fabsf(x)) + 1.f), x);
 }
-// tanh of a value that is stored in T afterwards.
+__device__ __forceinline__ float tanh_either(float x) {     // both, and a selection: no branch
+  const float a = tanh_series(x), b = tanh_exponential(x);
+  return fabsf(x) < TANH_SERIES_MAX ? a : b;
+}
+// tanh in a model that stores T.
 template <typename T>
 __device__ __forceinline__ float tanh_as(float x) {
-  if (sizeof(T) == 4) return tanhf(x);
-  return fabsf(x) < TANH_SERIES_MAX ? tanh_series(x) : tanh_exponential(x);
+  return sizeof(T) == 4 ? tanhf(x) : tanh_either(x);
 }
 
-// v[i] <- cap * tanh(v[i]).  Which of the two forms an element takes depends on that element alone.
+// v[i] <- cap * tanh(v[i]), the exponential form only for groups of eight that need it.  Which form an element gets depends
+// on that element alone.
 template <int N>
 __device__ __forceinline__ void cap_scores(float (&v)[N], float cap) {
-  float most = 0.f;
+  constexpr int G = N < 8 ? N : 8;
 #pragma unroll
-  for (int i = 0; i < N; ++i) most = fmaxf(most, fabsf(v[i]));
-  if (most < TANH_SERIES_MAX) {
+  for (int g = 0; g < N; g += G) {
+    float most = 0.f;
 #pragma unroll
-    for (int i = 0; i < N; ++i) v[i] = cap * tanh_series(v[i]);
-  } else {
+    for (int i = 0; i < G; ++i) most = fmaxf(most, fabsf(v[g + i]));
+    if (most < TANH_SERIES_MAX) {
 #pragma unroll
-    for (int i = 0; i < N; ++i)
-      v[i] = cap * (fabsf(v[i]) < TANH_SERIES_MAX ? tanh_series(v[i]) : tanh_exponential(v[i]));
+      for (int i = 0; i < G; ++i) v[g + i] = cap * tanh_series(v[g + i]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < G; ++i) v[g + i] = cap * tanh_either(v[g + i]);
+    }
   }
 }
 
@@ -79,9 +84,10 @@ __device__ __forceinline__ float sink_term(const AttnExtras& x, int head, float 
 }
 
 // Sigmoid of a gate that is stored in T.
+__device__ __forceinline__ float sigmoid_fast(float g) { return __fdividef(1.f, 1.f + __expf(-g)); }
 template <typename T>
 __device__ __forceinline__ float gate_sigmoid(T g) {
-  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-bf2f(g)));
+  if constexpr (sizeof(T) == 2) return sigmoid_fast(bf2f(g));
   else return 1.f / (1.f + expf(-g));
 }
 

@@ -10,8 +10,8 @@
 //                 position * inv_freq[i]; cosine and sine are multiplied by rot_mag
 // q goes to rows of its own, k and v to their pages.  fp32 from the projection's values to the stored ones.
 //
-// A warp owns heads, a lane VEC neighbouring columns of every 32 * VEC; a CTA walks up to PREP_TOKENS tokens with the
-// convolution's weights in registers.  The convolution's state is moved on here in steps that bring one token per sequence,
+// A warp owns heads, a lane VEC neighbouring columns of every 32 * VEC; a CTA walks up to PREP_TOKENS tokens, PREP_BATCH
+// rows requested together, with the convolution's weights and window in registers.  The convolution's state is moved on here in steps that bring one token per sequence,
 // and by ssm_conv_shift_kernel afterwards in others (other CTAs may still need the old inputs).
 // Algorithmic bytes per token: the row once, q, k and v once: HBM bandwidth.
 #pragma once
@@ -20,7 +20,7 @@
 
 namespace b200 {
 
-constexpr int PREP_WARPS = 8, PREP_TOKENS = 4, PREP_MAX_PAIRS = 128;
+constexpr int PREP_WARPS = 8, PREP_TOKENS = 8, PREP_BATCH = 4, PREP_MAX_PAIRS = 128;
 constexpr int PREP_REGISTER_NC = 2;      // heads of up to 256 columns keep four taps in registers
 constexpr int PREP_NORM_NONE = 0, PREP_NORM_HEAD = 1, PREP_NORM_ALL = 2;
 
@@ -69,9 +69,10 @@ __device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
   else *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
 }
 
-// VEC * 32 * NC >= DK.  TAPS: 0 no convolution, 4 up to four taps (weights in registers), -1 any number.
+// VEC * 32 * NC >= DK.  TAPS: 0 no convolution, 4 up to four taps (weights and window in registers), -1 any number.
 template <typename T, int VEC, int NC, int TAPS>
 __global__ void __launch_bounds__(PREP_WARPS * 32) attn_prep_kernel(const AttnPrepParams p) {
+  constexpr int B = PREP_BATCH;
   __shared__ float s_cos[PREP_TOKENS][PREP_MAX_PAIRS], s_sin[PREP_TOKENS][PREP_MAX_PAIRS];
   __shared__ float s_turn[PREP_WARPS][VEC * 32 * NC];     // a head's columns, for pairs that lie in different lanes
   __shared__ float s_red[PREP_TOKENS][2][PREP_WARPS];
@@ -82,6 +83,30 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) attn_prep_kernel(const AttnPr
   const long long t0 = (long long)blockIdx.x * p.per_cta;
   const int tokens = (int)min((long long)p.per_cta, p.num_tokens - t0);
   const int half = p.rot_dims >> 1, channels = (p.heads + p.kv_heads) * p.DK;
+  const int qk_heads = p.heads + p.kv_heads, stride = PREP_WARPS * gridDim.y, h0 = blockIdx.y * PREP_WARPS + warp;
+  const T* proj = reinterpret_cast<const T*>(p.proj);
+  const T* state = reinterpret_cast<const T*>(p.conv_state);
+  int cols[NC];                // this lane's columns of a head, clamped
+  bool mine[NC];
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    mine[c] = (c * 32 + lane) * VEC < p.DK;
+    cols[c] = mine[c] ? (c * 32 + lane) * VEC : 0;
+  }
+  // projection rows of the batch q0 .. q0 + B - 1, all requested together
+  auto rows = [&](int q0, int h, float (&x)[B][NC][VEC]) {
+#pragma unroll
+    for (int b = 0; b < B; ++b)
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        load_vec<T, VEC>(proj + (t0 + min(q0 + b, tokens - 1)) * p.proj_stride + h * p.DK + cols[c], x[b][c]);
+        if (!mine[c])
+#pragma unroll
+          for (int k = 0; k < VEC; ++k) x[b][c][k] = 0.f;
+      }
+  };
+  float x[B][NC][VEC];
+  if (h0 < qk_heads) rows(0, h0, x);         // on their way while the tables are made
   for (int e = threadIdx.x; e < tokens * half; e += PREP_WARPS * 32) {
     const int q = e / half, i = e - q * half;
     float s, c;
@@ -96,75 +121,74 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) attn_prep_kernel(const AttnPr
     bool fresh;
     const bool live = ssm_seq(p.seqs, s, first, len, fresh, slot) && t < first + len;
     s_j[threadIdx.x] = live ? (int)(t - first) : 0;
-    // a padding token convolves zeros; -2: a fresh sequence, whose state is written but not read
+    // a padding token convolves zeros; below -1: a fresh sequence, whose state is written but not read
     s_slot[threadIdx.x] = !live || slot < 0 ? -1 : fresh ? -2 - slot : slot;
   }
   __syncthreads();
-  const T* proj = reinterpret_cast<const T*>(p.proj);
-  const T* state = reinterpret_cast<const T*>(p.conv_state);
 
-  // the projection's (or convolution's) values of token q, head h in fp32
-  float win[TAPS == 4 ? 4 : 1][NC][VEC];
-  auto fetch = [&](int q, int h, const float (&w)[TAPS == 4 ? 4 : 1][NC][VEC], float (&x)[NC][VEC]) {
-    const long long t = t0 + q;
-#pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      const int col = (c * 32 + lane) * VEC;
-#pragma unroll
-      for (int k = 0; k < VEC; ++k) x[c][k] = 0.f;
-      if (col >= p.DK) continue;
-      const int ch = h * p.DK + col;
-      if constexpr (TAPS == 0) {
-        load_vec<T, VEC>(proj + t * p.proj_stride + ch, x[c]);
-      } else {
-        const int j = s_j[q], slot = s_slot[q];
-        auto input = [&](int i, float (&u)[VEC]) {        // input of the step's token i (negative: before the step)
-#pragma unroll
-          for (int k = 0; k < VEC; ++k) u[k] = 0.f;
-          if (i >= 0) load_vec<T, VEC>(proj + (t - j + i) * p.proj_stride + ch, u);
-          else if (slot >= 0) load_vec<T, VEC>(state + ((long long)slot * (p.taps - 1) + i + p.taps - 1) * channels + ch, u);
-        };
-        if constexpr (TAPS == 4) {
-#pragma unroll
-          for (int k = 0; k < 4; ++k) {
-            if (k >= 4 - p.taps) {
-              input(j - 3 + k, win[k][c]);
-            } else {
-#pragma unroll
-              for (int e = 0; e < VEC; ++e) win[k][c][e] = 0.f;
-            }
-          }
-#pragma unroll
-          for (int k = 0; k < 4; ++k)
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) x[c][e] = fmaf(w[k][c][e], win[k][c][e], x[c][e]);
-        } else {
-          for (int k = 0; k < p.taps; ++k) {
-            float u[VEC], wk[VEC];
-            input(j - (p.taps - 1) + k, u);
-            load_vec<float, VEC>(p.conv_w + (long long)k * channels + ch, wk);
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) x[c][e] = fmaf(wk[e], u[e], x[c][e]);
-          }
-        }
-        if constexpr (sizeof(T) == 2) {      // a convolved value is a value of the model dtype, like a projected one
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) x[c][e] = round_bf(x[c][e]);
-        }
-      }
-    }
-  };
-  auto weights = [&](int h, float (&w)[TAPS == 4 ? 4 : 1][NC][VEC]) {
+  constexpr int WT = TAPS == 4 ? 4 : 1, PAST = TAPS == 4 ? 3 : 1;
+  float w[WT][NC][VEC], past[PAST][NC][VEC];     // the convolution's weights of a head, the inputs before the current one
+  auto weights = [&](int h) {
     if constexpr (TAPS == 4) {
 #pragma unroll
       for (int k = 0; k < 4; ++k)
 #pragma unroll
         for (int c = 0; c < NC; ++c) {
-          const int col = (c * 32 + lane) * VEC, kk = k - (4 - p.taps);
+          const int kk = k - (4 - p.taps);
 #pragma unroll
           for (int e = 0; e < VEC; ++e) w[k][c][e] = 0.f;
-          if (kk >= 0 && col < p.DK) load_vec<float, VEC>(p.conv_w + (long long)kk * channels + h * p.DK + col, w[k][c]);
+          if (kk >= 0 && mine[c]) load_vec<float, VEC>(p.conv_w + (long long)kk * channels + h * p.DK + cols[c], w[k][c]);
         }
+    }
+  };
+  // input i of the step of token q's sequence (negative: before the step, from its state), columns of group c
+  auto input = [&](int q, int h, int i, int c, float (&u)[VEC]) {
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) u[k] = 0.f;
+    if (!mine[c]) return;
+    const int ch = h * p.DK + cols[c], slot = s_slot[q];
+    if (i >= 0) load_vec<T, VEC>(proj + (t0 + q - s_j[q] + i) * p.proj_stride + ch, u);
+    else if (slot >= 0 && i + p.taps - 1 >= 0) load_vec<T, VEC>(state + ((long long)slot * (p.taps - 1) + i + p.taps - 1) * channels + ch, u);
+  };
+  // x: the inputs of token q -> the convolution's values
+  auto convolve = [&](int q, int h, float (&x)[NC][VEC]) {
+    if constexpr (TAPS == 4) {
+      if (q == 0 || s_j[q] == 0 || s_slot[q] == -1) {      // the window does not go on from the token before
+#pragma unroll
+        for (int k = 0; k < 3; ++k)
+#pragma unroll
+          for (int c = 0; c < NC; ++c) input(q, h, s_j[q] - 3 + k, c, past[k][c]);
+      }
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) {
+          const float u = x[c][e];
+          x[c][e] = fmaf(w[3][c][e], u, fmaf(w[2][c][e], past[2][c][e], fmaf(w[1][c][e], past[1][c][e], w[0][c][e] * past[0][c][e])));
+          past[0][c][e] = past[1][c][e];
+          past[1][c][e] = past[2][c][e];
+          past[2][c][e] = u;
+        }
+    } else if constexpr (TAPS == -1) {
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        float a[VEC] = {};
+        for (int k = 0; k < p.taps; ++k) {
+          float u[VEC], wk[VEC];
+          input(q, h, s_j[q] - (p.taps - 1) + k, c, u);
+          load_vec<float, VEC>(p.conv_w + (long long)k * channels + h * p.DK + cols[c], wk);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) a[e] = fmaf(wk[e], u[e], a[e]);
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[c][e] = a[e];
+      }
+    }
+    if constexpr (TAPS != 0 && sizeof(T) == 2) {     // a convolved value is a value of the model dtype, like a projected one
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[c][e] = round_bf(x[c][e]);
     }
   };
   auto squares = [&](const float (&x)[NC][VEC]) {
@@ -176,136 +200,140 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) attn_prep_kernel(const AttnPr
     return ss;
   };
 
-  const int qk_heads = p.heads + p.kv_heads, stride = PREP_WARPS * gridDim.y, h0 = blockIdx.y * PREP_WARPS + warp;
   if (p.norm == PREP_NORM_ALL) {       // one CTA holds every head of its tokens (gridDim.y is 1)
-    float ss[PREP_TOKENS][2] = {};
-    for (int h = h0; h < qk_heads; h += stride) {
-      float w[TAPS == 4 ? 4 : 1][NC][VEC];
-      weights(h, w);
+    for (int q0 = 0; q0 < tokens; q0 += B) {
+      float ss[B][2] = {};
+      for (int h = h0; h < qk_heads; h += stride) {
+        if (h != h0 || q0 != 0) rows(q0, h, x);
+        weights(h);
 #pragma unroll
-      for (int q = 0; q < PREP_TOKENS; ++q) {
-        if (q >= tokens) break;
-        float x[NC][VEC];
-        fetch(q, h, w, x);
-        if (h < p.heads) ss[q][0] += squares(x);
-        else ss[q][1] += squares(x);
+        for (int b = 0; b < B; ++b) {
+          if (q0 + b >= tokens) break;
+          if (TAPS == 4 && b == 0 && q0 != 0)        // the window of another batch's head has gone
+#pragma unroll
+            for (int k = 0; k < PAST; ++k)
+#pragma unroll
+              for (int c = 0; c < NC; ++c) input(q0, h, s_j[q0] - 3 + k, c, past[k][c]);
+          convolve(q0 + b, h, x[b]);
+          ss[b][h < p.heads ? 0 : 1] += squares(x[b]);
+        }
       }
+#pragma unroll
+      for (int b = 0; b < B; ++b)
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+          const float s = warp_sum(ss[b][k]);
+          if (lane == 0 && q0 + b < tokens) s_red[q0 + b][k][warp] = s;
+        }
     }
-#pragma unroll
-    for (int q = 0; q < PREP_TOKENS; ++q)
-#pragma unroll
-      for (int k = 0; k < 2; ++k) {
-        const float s = warp_sum(ss[q][k]);
-        if (lane == 0) s_red[q][k][warp] = s;
-      }
     __syncthreads();
   }
   for (int h = h0; h < qk_heads; h += stride) {
     const bool is_q = h < p.heads;
     const int kvh = h - p.heads;
-    float w[TAPS == 4 ? 4 : 1][NC][VEC], nw[NC][VEC];
-    weights(h, w);
+    float nw[NC][VEC];
+    weights(h);
     if (p.norm != PREP_NORM_NONE) {
       const float* src = is_q ? p.q_norm : p.k_norm;
       if (p.norm == PREP_NORM_ALL) src += (is_q ? h : kvh) * p.DK;
 #pragma unroll
-      for (int c = 0; c < NC; ++c) {
-        const int col = (c * 32 + lane) * VEC;
-#pragma unroll
-        for (int k = 0; k < VEC; ++k) nw[c][k] = 0.f;
-        if (col < p.DK) load_vec<float, VEC>(src + col, nw[c]);
-      }
+      for (int c = 0; c < NC; ++c) load_vec<float, VEC>(src + cols[c], nw[c]);
     }
-    for (int q = 0; q < tokens; ++q) {
-      const long long t = t0 + q;
-      float x[NC][VEC];
-      fetch(q, h, w, x);
-      if constexpr (TAPS == 4) {
-        if (p.shift && p.taps > 1 && s_slot[q] != -1) {
-          const int slot = s_slot[q] < -1 ? -2 - s_slot[q] : s_slot[q];
-          T* st = reinterpret_cast<T*>(p.conv_state) + (long long)slot * (p.taps - 1) * channels + h * p.DK;
+    for (int q0 = 0; q0 < tokens; q0 += B) {
+      if (h != h0 || q0 != 0 || p.norm == PREP_NORM_ALL) rows(q0, h, x);
 #pragma unroll
-          for (int k = 1; k < 4; ++k)
-            if (k > 4 - p.taps)
+      for (int b = 0; b < B; ++b) {
+        const int q = q0 + b;
+        if (q >= tokens) break;
+        float (&v)[NC][VEC] = x[b];
+        convolve(q, h, v);
+        if constexpr (TAPS == 4) {
+          if (p.shift && p.taps > 1 && s_slot[q] != -1) {      // past: the last three inputs, this token's included
+            const int slot = s_slot[q] < -1 ? -2 - s_slot[q] : s_slot[q];
+            T* st = reinterpret_cast<T*>(p.conv_state) + (long long)slot * (p.taps - 1) * channels + h * p.DK;
 #pragma unroll
-              for (int c = 0; c < NC; ++c)
-                if ((c * 32 + lane) * VEC < p.DK)
-                  store_vec<T, VEC>(st + (long long)(k - 1 - (4 - p.taps)) * channels + (c * 32 + lane) * VEC, win[k][c]);
-        }
-      }
-      long long slot = p.slot_mapping[t];
-      if (slot >= p.num_slots) {
-        if (lane == 0 && h == h0) report_status(B200_STATUS_BAD_INDEX, (int)slot);
-        slot = -1;
-      }
-      if (!is_q && slot < 0) continue;
-      if (!is_q && p.v_off < 0) {
-        T* v = reinterpret_cast<T*>(p.v_cache) + (slot * p.kv_heads + kvh) * p.DV;
+            for (int k = 0; k < 3; ++k)
+              if (k + 1 > 4 - p.taps)
 #pragma unroll
-        for (int c = 0; c < NC; ++c)
-          if ((c * 32 + lane) * VEC < p.DK) store_vec<T, VEC>(v + (c * 32 + lane) * VEC, x[c]);
-      }
-      if (p.norm != PREP_NORM_NONE) {
-        float ss = 0.f, n = (float)p.dim;
-        if (p.norm == PREP_NORM_HEAD) {
-          ss = warp_sum(squares(x));
-        } else {
-#pragma unroll
-          for (int k = 0; k < PREP_WARPS; ++k) ss += s_red[q][is_q ? 0 : 1][k];
-          n *= (float)(is_q ? p.heads : p.kv_heads);
-        }
-        const float inv = 1.f / sqrtf(ss / n + p.eps);
-#pragma unroll
-        for (int c = 0; c < NC; ++c)
-#pragma unroll
-          for (int k = 0; k < VEC; ++k) x[c][k] = x[c][k] * inv * nw[c][k];
-      }
-      if (half > 0 && p.rot_half) {
-        __syncwarp();
-#pragma unroll
-        for (int c = 0; c < NC; ++c)
-          if ((c * 32 + lane) * VEC < p.rot_dims) {
-#pragma unroll
-            for (int k = 0; k < VEC; ++k) s_turn[warp][(c * 32 + lane) * VEC + k] = x[c][k];
+                for (int c = 0; c < NC; ++c)
+                  if (mine[c]) store_vec<T, VEC>(st + (long long)(k - (4 - p.taps)) * channels + cols[c], past[k][c]);
           }
-        __syncwarp();
+        }
+        const long long t = t0 + q;
+        long long slot = p.slot_mapping[t];
+        if (slot >= p.num_slots) {
+          if (lane == 0 && h == h0) report_status(B200_STATUS_BAD_INDEX, (int)slot);
+          slot = -1;
+        }
+        if (!is_q && slot < 0) continue;
+        if (!is_q && p.v_off < 0) {
+          T* dst = reinterpret_cast<T*>(p.v_cache) + (slot * p.kv_heads + kvh) * p.DV;
 #pragma unroll
-        for (int c = 0; c < NC; ++c)
+          for (int c = 0; c < NC; ++c)
+            if (mine[c]) store_vec<T, VEC>(dst + cols[c], v[c]);
+        }
+        if (p.norm != PREP_NORM_NONE) {
+          float ss = 0.f, n = (float)p.dim;
+          if (p.norm == PREP_NORM_HEAD) {
+            ss = warp_sum(squares(v));
+          } else {
 #pragma unroll
-          for (int k = 0; k < VEC; ++k) {
-            const int col = (c * 32 + lane) * VEC + k;
-            if (col < half) x[c][k] = x[c][k] * s_cos[q][col] - s_turn[warp][col + half] * s_sin[q][col];
-            else if (col < p.rot_dims) x[c][k] = x[c][k] * s_cos[q][col - half] + s_turn[warp][col - half] * s_sin[q][col - half];
+            for (int k = 0; k < PREP_WARPS; ++k) ss += s_red[q][is_q ? 0 : 1][k];
+            n *= (float)(is_q ? p.heads : p.kv_heads);
           }
-      } else if (half > 0) {
+          const float inv = 1.f / sqrtf(ss / n + p.eps);
 #pragma unroll
-        for (int c = 0; c < NC; ++c)
+          for (int c = 0; c < NC; ++c)
 #pragma unroll
-          for (int k = 0; k < VEC; k += 2) {
-            const int col = (c * 32 + lane) * VEC + k;
-            if (col < p.rot_dims) {
-              const float u = x[c][k], v = x[c][k + 1], co = s_cos[q][col >> 1], si = s_sin[q][col >> 1];
-              x[c][k] = u * co - v * si;
-              x[c][k + 1] = v * co + u * si;
+            for (int k = 0; k < VEC; ++k) v[c][k] = v[c][k] * inv * nw[c][k];
+        }
+        if (half > 0 && p.rot_half) {
+          __syncwarp();
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+            if (mine[c] && cols[c] < p.rot_dims) {
+#pragma unroll
+              for (int k = 0; k < VEC; ++k) s_turn[warp][cols[c] + k] = v[c][k];
             }
-          }
-      }
-      T* dst = is_q ? reinterpret_cast<T*>(p.q_out) + (t * p.heads + h) * p.DK
-                    : reinterpret_cast<T*>(p.k_cache) + (slot * p.kv_heads + kvh) * p.DK;
+          __syncwarp();
 #pragma unroll
-      for (int c = 0; c < NC; ++c)
-        if ((c * 32 + lane) * VEC < p.DK) store_vec<T, VEC>(dst + (c * 32 + lane) * VEC, x[c]);
+          for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) {
+              const int col = cols[c] + k;
+              if (col < half) v[c][k] = v[c][k] * s_cos[q][col] - s_turn[warp][col + half] * s_sin[q][col];
+              else if (col < p.rot_dims) v[c][k] = v[c][k] * s_cos[q][col - half] + s_turn[warp][col - half] * s_sin[q][col - half];
+            }
+        } else if (half > 0) {
+#pragma unroll
+          for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int k = 0; k < VEC; k += 2) {
+              const int col = cols[c] + k;
+              if (col < p.rot_dims) {
+                const float u = v[c][k], z = v[c][k + 1], co = s_cos[q][col >> 1], si = s_sin[q][col >> 1];
+                v[c][k] = u * co - z * si;
+                v[c][k + 1] = z * co + u * si;
+              }
+            }
+        }
+        T* dst = is_q ? reinterpret_cast<T*>(p.q_out) + (t * p.heads + h) * p.DK
+                      : reinterpret_cast<T*>(p.k_cache) + (slot * p.kv_heads + kvh) * p.DK;
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+          if (mine[c]) store_vec<T, VEC>(dst + cols[c], v[c]);
+      }
     }
   }
   if (p.v_off < 0) return;
-  const int cols = p.kv_heads * p.DV;       // a multiple of 8
-  for (int e = (int)(blockIdx.y * PREP_WARPS * 32 + threadIdx.x) * 4; e < cols * tokens; e += (int)gridDim.y * PREP_WARPS * 32 * 4) {
-    const int q = e / cols, col = e - q * cols;
+  const int width = p.kv_heads * p.DV;       // a multiple of 8
+  for (int e = (int)(blockIdx.y * PREP_WARPS * 32 + threadIdx.x) * 4; e < width * tokens; e += (int)gridDim.y * PREP_WARPS * 32 * 4) {
+    const int q = e / width, col = e - q * width;
     const long long slot = p.slot_mapping[t0 + q];
     if (slot < 0 || slot >= p.num_slots) continue;
     float v[4];
     load4(proj + (t0 + q) * p.proj_stride + p.v_off + col, v);
-    store4(reinterpret_cast<T*>(p.v_cache) + slot * cols + col, v);
+    store4(reinterpret_cast<T*>(p.v_cache) + slot * width + col, v);
   }
 }
 

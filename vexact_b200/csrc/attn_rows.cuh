@@ -575,14 +575,27 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
             if (p.extras.gate_mode == GATE_HEAD) {
               inv *= gate_sigmoid(gate[head]);
             } else {
-              gate += head * p.dv + half * 64;
+              gate += head * p.dv;
 #pragma unroll
-              for (int q = 0; q < 8; ++q) {
-                if (half * 64 + q * 8 >= p.dv) break;
-                const uint4 g8 = *reinterpret_cast<const uint4*>(gate + q * 8);
-                const __nv_bfloat16* ge = reinterpret_cast<const __nv_bfloat16*>(&g8);
+              for (int part = 0; part < 2; ++part) {      // four loads ahead of their first use
+                uint4 g8[4];
 #pragma unroll
-                for (int k = 0; k < 8; ++k) o[q * 8 + k] *= gate_sigmoid(ge[k]);
+                for (int q = 0; q < 4; ++q) {   // columns past the head's are not stored: any will do
+                  const int col = half * 64 + part * 32 + q * 8;
+                  g8[q] = *reinterpret_cast<const uint4*>(gate + (col < p.dv ? col : 0));
+                }
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                  const uint32_t pair[4] = {g8[q].x, g8[q].y, g8[q].z, g8[q].w};
+#pragma unroll
+                  for (int k = 0; k < 4; ++k) {
+                    float a, b;
+                    unpack_bf2(pair[k], a, b);
+                    o[part * 32 + q * 8 + 2 * k] *= sigmoid_fast(a);
+                    o[part * 32 + q * 8 + 2 * k + 1] *= sigmoid_fast(b);
+                  }
+                }
+                asm volatile("" ::: "memory");
               }
             }
           }

@@ -153,10 +153,20 @@ __device__ __forceinline__ AtcRaw atc_raw(const AttnParams& p, int lin) {
   return r;
 }
 
+// Query tile of rank r, most expensive first: the last tile first, or where chunks of `per` tiles start over, the last tile of
+// every chunk, then those before them, and so on (a portion that does not start with a chunk is dealt a little less evenly).
+__device__ __forceinline__ int atc_query_tile(int tiles, int per, int r) {
+  if (per < 1 || per >= tiles) return tiles - 1 - r;
+  const int full = tiles / per, rem = tiles - full * per, head = (per - rem) * full;   // the first phases have `full` tiles
+  if (r < head) return r % full * per + per - 1 - r / full;
+  r -= head;
+  return r % (full + 1) * per + rem - 1 - r / (full + 1);
+}
+
 template <int NC>
 __device__ __forceinline__ void atc_make(const AttnParams& p, int lin, const AtcRaw& r, AtcTile& t) {
   const int eff = r.eff < 0 ? 0 : r.eff;
-  const int x = p.tc_q_tiles - 1 - eff / (p.tc_hy * p.num_seqs);
+  const int x = atc_query_tile(p.tc_q_tiles, p.chunk / max(1, NC / min(8, p.group)), eff / (p.tc_hy * p.num_seqs));
   const int y = eff % p.tc_hy;
   t.seq = r.seq;
   t.kvh = y / p.head_chunks;

@@ -12,7 +12,7 @@
 //
 // The norms may be dynamic tanh instead, tanh(alpha x) * w + b with one number alpha, which reduces nothing:
 //     x <- x + tanh(post_alpha y) * post + post_bias (+ add),    xn = tanh(norm_alpha x) * norm + norm_bias
-// A thread then owns four columns of a few tokens and keeps the norms' vectors in registers.  At the start of a model y is
+// A thread then owns four columns, keeps the norms' vectors in registers and walks tokens, ROWS at a time.  At the start of a model y is
 // the embedding row times embed_scale, under either norm.
 // Algorithmic bytes per token: 8 W (x) + b W (topk + shared rows of y) + b W (xn), b = 2 or 4: HBM bandwidth.
 #pragma once
@@ -196,7 +196,7 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
   for (int i = W + threadIdx.x; i < p.xn_cols; i += blockDim.x) orow[i] = from_f32<T>(0.f);
 }
 
-// The boundary under dynamic tanh.  A thread owns four neighbouring columns of ROWS tokens.
+// The boundary under dynamic tanh.  A thread owns four neighbouring columns; a CTA takes batches of ROWS tokens.
 template <typename T, int ROWS, bool PICK>
 __global__ void __launch_bounds__(128) residual_tanh_kernel(const ResidualParams p) {
   pdl_trigger();
@@ -207,11 +207,11 @@ __global__ void __launch_bounds__(128) residual_tanh_kernel(const ResidualParams
     if (vec) load4(row + i, v);
     else load4_tail(row + i, W - i, v);
   };
-  const long long r0 = (long long)blockIdx.x * ROWS;
   if (i >= W) {                // columns past the width: zeros
     if (p.norm_w)
-      for (int q = 0; q < ROWS && r0 + q < p.num_rows; ++q)
-        for (int k = i; k < min(i + 4, p.xn_cols); ++k) reinterpret_cast<T*>(p.xn)[(r0 + q) * p.xn_stride + k] = from_f32<T>(0.f);
+      for (long long r0 = (long long)blockIdx.x * ROWS; r0 < p.num_rows; r0 += (long long)gridDim.x * ROWS)
+        for (int q = 0; q < ROWS && r0 + q < p.num_rows; ++q)
+          for (int k = i; k < min(i + 4, p.xn_cols); ++k) reinterpret_cast<T*>(p.xn)[(r0 + q) * p.xn_stride + k] = from_f32<T>(0.f);
     return;
   }
   float w[4], wb[4], nw[4] = {}, nb[4] = {}, add[4] = {};
@@ -222,6 +222,7 @@ __global__ void __launch_bounds__(128) residual_tanh_kernel(const ResidualParams
     get(p.norm_bias, nb);
   }
   if (p.add) get(p.add, add);
+  for (long long r0 = (long long)blockIdx.x * ROWS; r0 < p.num_rows; r0 += (long long)gridDim.x * ROWS) {
   float v[ROWS][4], x[ROWS][4];
   long long tok[ROWS];
 #pragma unroll
@@ -305,14 +306,16 @@ __global__ void __launch_bounds__(128) residual_tanh_kernel(const ResidualParams
       }
     }
   }
+  }
 }
 
 template <typename T, bool PICK>
 inline int residual_tanh_launch(const ResidualParams& p, cudaStream_t st) {
-  constexpr int MANY = 4;
+  constexpr int MANY = 4, BATCHES = 4;
   const unsigned gy = (unsigned)(((p.norm_w ? p.xn_cols : p.W) + 511) / 512);
-  if (p.num_rows >= 148 * 2 * MANY)
-    launch_k(residual_tanh_kernel<T, MANY, PICK>, dim3((unsigned)((p.num_rows + MANY - 1) / MANY), gy), dim3(128), 0, st, p);
+  const long long many = (p.num_rows + MANY * BATCHES - 1) / (MANY * BATCHES);
+  if (many * gy >= 148 * 2)
+    launch_k(residual_tanh_kernel<T, MANY, PICK>, dim3((unsigned)many, gy), dim3(128), 0, st, p);
   else
     launch_k(residual_tanh_kernel<T, 1, PICK>, dim3((unsigned)p.num_rows, gy), dim3(128), 0, st, p);
   return launch_status();
