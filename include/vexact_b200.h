@@ -513,7 +513,7 @@ int b200_window_attn_simt(const void* q, long long q_row_stride, const void* k_c
  * on), values (columns from v_off, or with -1 the convolved keys), norm of q and k (0 none, 1 per head, 2 over all heads; dim
  * true columns of a head), rotation of the first rot_dims columns (rot_half: pairs (i, i + rot_dims / 2), else (2i, 2i + 1);
  * cosine and sine times rot_mag); q to q_out [T, heads * DK], k and v to their pages.  one_token_each: no sequence brings
- * more than one token (one launch; otherwise two with a convolution).  DK <= 1024, rot_dims <= 256. */
+ * more than one token (one launch; otherwise two with a convolution).  DK <= 512, rot_dims <= 256. */
 int b200_attn_prep(const void* proj, long long proj_row_stride, int v_off, const void* positions_i64, const void*
                    slot_mapping_i32, const void* conv_w_f32, void* conv_state, int taps, const void* query_start_loc,
                    const void* context_lens, const void* state_slots, int num_seqs, int num_state_slots, int

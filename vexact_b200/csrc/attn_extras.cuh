@@ -6,8 +6,7 @@
 //   sink      exp(sink[head]) is added to the denominator: a key without a value
 //   gate      the head's output is multiplied by the sigmoid of one number per head, or of one per column
 //
-// All of it is fp32.  In the kernels that keep scores in units of log2, the caller passes scale / cap as the score's factor
-// and cap * log2(e) as `cap` (without a cap scale * log2(e) and 0).
+// All of it is fp32.  Kernels that keep scores in units of log2 get the cap in those units, cap * log2(e).
 #pragma once
 #include "common.cuh"
 
@@ -15,8 +14,19 @@ namespace b200 {
 
 constexpr int GATE_NONE = 0, GATE_HEAD = 1, GATE_COLUMN = 2;
 
-struct AttnExtras {
+// A cap and the coefficients of cap * tanh(s / cap) = s + c3 s^3 + c5 s^5 + c7 s^7 .. in the scores' units.
+struct ScoreCap {
   float cap;               // 0: none
+  float inv, small, c3, c5, c7;
+};
+inline ScoreCap score_cap(float cap) {
+  if (!(cap > 0.f)) return {};
+  const double q = 1.0 / ((double)cap * cap);
+  return {cap, 1.f / cap, 0.2f * cap, (float)(-q / 3), (float)(2 * q * q / 15), (float)(-17 * q * q * q / 315)};
+}
+
+struct AttnExtras {
+  ScoreCap cap;
   const float* sink;       // [heads] or null
   const void* gate;        // rows of the model dtype, gate_stride apart: [heads] or [heads * DV]; null with GATE_NONE
   long long gate_stride;
@@ -34,46 +44,40 @@ __device__ __forceinline__ int first_visible(int window, int chunk, int pos) {
   return chunk > 0 ? max(a, pos - pos % chunk) : a;
 }
 
-// tanh in fp32.  Below 1/4 the odd Taylor polynomial through x^9 (the next term is below 3e-9), above it
+// tanh in fp32.  Below 0.2 the odd Taylor polynomial through x^7 (the next term is below 1.2e-8), above it
 // 1 - 2 / (e^(2 |x|) + 1) on the special-function unit (absolute error below 4e-7).
-constexpr float TANH_SERIES_MAX = 0.25f;
-__device__ __forceinline__ float tanh_series(float x) {
+constexpr float TANH_SERIES_MAX = 0.2f;
+__device__ __forceinline__ float tanh_series(float x, float c3 = -1.f / 3.f, float c5 = 2.f / 15.f, float c7 = -17.f / 315.f) {
   const float s = x * x;
-  float c = 62.f / 2835.f;
-  c = fmaf(c, s, -17.f / 315.f);
-  c = fmaf(c, s, 2.f / 15.f);
-  c = fmaf(c, s, -1.f / 3.f);
-  return fmaf(c * s, x, x);
+  return fmaf(fmaf(fmaf(c7, s, c5), s, c3) * s, x, x);
 }
 __device__ __forceinline__ float tanh_exponential(float x) {
   return copysignf(1.f - __fdividef(2.f, __expf(2.f * fabsf(x)) + 1.f), x);
 }
-__device__ __forceinline__ float tanh_either(float x) {     // both, and a selection: no branch
+// tanh in a model that stores T (both forms and a selection: no branch).
+template <typename T>
+__device__ __forceinline__ float tanh_as(float x) {
+  if (sizeof(T) == 4) return tanhf(x);
   const float a = tanh_series(x), b = tanh_exponential(x);
   return fabsf(x) < TANH_SERIES_MAX ? a : b;
 }
-// tanh in a model that stores T.
-template <typename T>
-__device__ __forceinline__ float tanh_as(float x) {
-  return sizeof(T) == 4 ? tanhf(x) : tanh_either(x);
-}
 
-// v[i] <- cap * tanh(v[i]), the exponential form only for groups of eight that need it.  Which form an element gets depends
-// on that element alone.
+// v[i] <- cap * tanh(v[i] / cap).  Which form an element gets depends on that element alone; rows of small scores, the usual
+// case, pay for the polynomial only.
 template <int N>
-__device__ __forceinline__ void cap_scores(float (&v)[N], float cap) {
-  constexpr int G = N < 8 ? N : 8;
+__device__ __forceinline__ void cap_scores(float (&v)[N], const ScoreCap& c) {
+  float most[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-  for (int g = 0; g < N; g += G) {
-    float most = 0.f;
+  for (int i = 0; i < N; ++i) most[i & 3] = fmaxf(most[i & 3], fabsf(v[i]));
+  if (fmaxf(fmaxf(most[0], most[1]), fmaxf(most[2], most[3])) < c.small) {
 #pragma unroll
-    for (int i = 0; i < G; ++i) most = fmaxf(most, fabsf(v[g + i]));
-    if (most < TANH_SERIES_MAX) {
+    for (int i = 0; i < N; ++i) v[i] = tanh_series(v[i], c.c3, c.c5, c.c7);
+  } else {
 #pragma unroll
-      for (int i = 0; i < G; ++i) v[g + i] = cap * tanh_series(v[g + i]);
-    } else {
-#pragma unroll
-      for (int i = 0; i < G; ++i) v[g + i] = cap * tanh_either(v[g + i]);
+    for (int i = 0; i < N; ++i) {
+      if (fabsf(v[i]) < c.small) v[i] = tanh_series(v[i], c.c3, c.c5, c.c7);
+      else v[i] = c.cap * tanh_exponential(v[i] * c.inv);
+      if (i % 4 == 3) asm volatile("" : "+f"(v[i]), "+f"(v[i - 1]), "+f"(v[i - 2]), "+f"(v[i - 3]));   // few at a time
     }
   }
 }
@@ -92,7 +96,7 @@ __device__ __forceinline__ float gate_sigmoid(T g) {
 }
 
 inline bool attn_extras_ok(const AttnExtras& x) {
-  return x.cap >= 0.f && x.gate_mode >= GATE_NONE && x.gate_mode <= GATE_COLUMN && (x.gate != nullptr) == (x.gate_mode != GATE_NONE);
+  return x.gate_mode >= GATE_NONE && x.gate_mode <= GATE_COLUMN && (x.gate != nullptr) == (x.gate_mode != GATE_NONE);
 }
 
 }  // namespace b200

@@ -87,7 +87,7 @@ template <int DK, bool EXACT>
 __global__ void __launch_bounds__(ATR_THREADS, 1)
 paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                        const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_out,
-                       const AttnParams p) {
+                       const __grid_constant__ CUtensorMap tm_gate, const AttnParams p) {
   constexpr int DV = 128, NC = ATR_ROWS, KST = 2, VST = 2;
   constexpr int KH = DK / 64, VH = DV / 64;
   constexpr int K_BYTES = ATC_BN * DK * 2, V_BYTES = ATC_BN * DV * 2;
@@ -123,7 +123,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       return;
     }
   }
-  uint64_t* bars = reinterpret_cast<uint64_t*>(small);                       // 2*KST + 2*VST + 15 barriers (< 256 bytes)
+  uint64_t* bars = reinterpret_cast<uint64_t*>(small);                       // 2*KST + 2*VST + 23 barriers (< 256 bytes)
   float (*s_hmax)[2][NC] = reinterpret_cast<float (*)[2][NC]>(small + 256);   // [block parity][half][row] half-row maxima
   uint32_t* tmem_slot_p = reinterpret_cast<uint32_t*>(small + 256 + 4 * NC * 4);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(small + 256 + 4 * NC * 4 + 8);
@@ -140,6 +140,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   auto qfull_bar = [&](int b) { return bar(NB + 7 + b); };
   auto qfree_bar = [&](int b) { return bar(NB + 9 + b); };
   auto pair_bar = [&](int q) { return bar(NB + 11 + q); };   // the two compute warps of lane quadrant q meet here
+  auto gate_bar = [&](int w) { return bar(NB + 15 + w); };   // exact form: compute warp w's gate columns have arrived
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
@@ -160,6 +161,8 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       ptx::mbar_init(qfree_bar(b), 1);
     }
     for (int q = 0; q < 4; ++q) ptx::mbar_init(pair_bar(q), 2);
+    if (EXACT)
+      for (int w = 0; w < 8; ++w) ptx::mbar_init(gate_bar(w), 1);
     ptx::mbar_init(pready_bar, 8);       // compute warps
     ptx::mbar_init(ofull_bar, 1);
     ptx::mbar_init(ofree_bar, 8);
@@ -168,6 +171,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
     ptx::prefetch_tensormap(&tm_v);
     if (p.q_tma) ptx::prefetch_tensormap(&tm_q);
     if (p.o_tma) ptx::prefetch_tensormap(&tm_out);
+    if (EXACT && p.g_tma) ptx::prefetch_tensormap(&tm_gate);
   }
   if (warp == 1) {
     ptx::tmem_alloc(ptx::smem_u32(tmem_slot_p), TMEM_COLS);
@@ -361,7 +365,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
     const uint32_t lane_addr = (uint32_t)(q4 * 32) << 16;
     const uint32_t o_addr = tm_o + lane_addr + half * 64;
     uint8_t* p_half = p_ptr + half * (NC * 128);   // my 64 keys are one 64-key half of the P tile
-    uint32_t g0 = 0, pair_phase = 0;
+    uint32_t g0 = 0, pair_phase = 0, gate_phase = 0;
     // Meeting point of a row's two threads: a bounded mbarrier wait like every other wait here (a bar.sync
     // would strand one warp if its partner left on an abort).
     auto pair_sync = [&]() {
@@ -419,7 +423,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
           }
         }
         if constexpr (EXACT) {
-          if (p.extras.cap > 0.f) cap_scores(v, p.extras.cap);
+          if (p.extras.cap.cap > 0.f) cap_scores(v, p.extras.cap);
         }
         if (masked) {
 #pragma unroll
@@ -535,8 +539,28 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       }
       if (!alive) break;
       // tile end: the last block's O, the row sum, the store
+      const int head = t.kvh * p.group + t.hchunk * 8 + hd;
+      const long long gate_row = EXACT ? (long long)(t.q_start + t.tile_pos0 + (pi < npos ? pi : 0)) * p.extras.gate_stride : 0;
+      float head_gate = 1.f;
+      if constexpr (EXACT) {
+        if (p.extras.gate_mode == GATE_HEAD)
+          head_gate = gate_sigmoid(reinterpret_cast<const __nv_bfloat16*>(p.extras.gate)[gate_row + head]);
+      }
       if (!ptx::mbar_wait_warp(ofull_bar, (g0 + t.nblk - 1) & 1, abort_flag, 751)) break;
       ptx::tc_fence_after();
+      if constexpr (EXACT) {
+        // The last product has read the P tiles: this warp's 4 KB of the second one receive its rows' gate columns (the box
+        // its output rows leave by), while O and the row sums are read.
+        if (p.extras.gate_mode == GATE_COLUMN && p.g_tma && half * 64 < p.dv) {
+          ptx::fence_proxy_async_smem();
+          __syncwarp();
+          if (lane == 0) {
+            ptx::mbar_expect_tx(gate_bar(warp - 4), 32 * 128);
+            ptx::tma_load_3d(ptx::smem_u32(p_half + P_TILE + q4 * 32 * 128), &tm_gate, gate_bar(warp - 4), half * 64,
+                             t.kvh * p.group + t.hchunk * 8, t.q_start + t.tile_pos0 + q4 * (32 / t.heads_here), ptx::kEvictFirst);
+          }
+        }
+      }
       if (warp == 4) ATR_STAMP(2, g0 + t.nblk - 1, 0);   // last O complete
       {
         uint32_t r0[32], r1[32];
@@ -565,37 +589,28 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         // 4 KB of the P tile (idle from the tile's last PV product until this warp's next P write; swizzled), then eight
         // lanes store one row's 128 bytes, four rows per instruction.
         float l_row = s_lh[0][row] + s_lh[1][row];
-        const int head = t.kvh * p.group + t.hchunk * 8 + hd;
         if constexpr (EXACT) l_row += sink_term(p.extras, head, m_run);
         float inv = 1.0f / l_row;
         if constexpr (EXACT) {
-          if (p.extras.gate_mode != GATE_NONE && pi < npos) {
-            const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(p.extras.gate) +
-                                        (long long)(t.q_start + t.tile_pos0 + pi) * p.extras.gate_stride;
-            if (p.extras.gate_mode == GATE_HEAD) {
-              inv *= gate_sigmoid(gate[head]);
-            } else {
-              gate += head * p.dv;
+          inv *= head_gate;
+          if (p.extras.gate_mode == GATE_COLUMN && half * 64 < p.dv) {
+            if (p.g_tma) {
+              if (!ptx::mbar_wait_warp(gate_bar(warp - 4), gate_phase & 1, abort_flag, 790 + warp)) break;
+              ++gate_phase;
+            }
+            const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(p.extras.gate) + gate_row + head * p.dv + half * 64;
 #pragma unroll
-              for (int part = 0; part < 2; ++part) {      // four loads ahead of their first use
-                uint4 g8[4];
+            for (int q = 0; q < 8; ++q) {
+              if (half * 64 + q * 8 >= p.dv) break;
+              const uint4 g = p.g_tma ? *reinterpret_cast<const uint4*>(p_half + P_TILE + sw128(row, q))
+                                      : *reinterpret_cast<const uint4*>(gate + q * 8);
+              const uint32_t pair[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
-                for (int q = 0; q < 4; ++q) {   // columns past the head's are not stored: any will do
-                  const int col = half * 64 + part * 32 + q * 8;
-                  g8[q] = *reinterpret_cast<const uint4*>(gate + (col < p.dv ? col : 0));
-                }
-#pragma unroll
-                for (int q = 0; q < 4; ++q) {
-                  const uint32_t pair[4] = {g8[q].x, g8[q].y, g8[q].z, g8[q].w};
-#pragma unroll
-                  for (int k = 0; k < 4; ++k) {
-                    float a, b;
-                    unpack_bf2(pair[k], a, b);
-                    o[part * 32 + q * 8 + 2 * k] *= sigmoid_fast(a);
-                    o[part * 32 + q * 8 + 2 * k + 1] *= sigmoid_fast(b);
-                  }
-                }
-                asm volatile("" ::: "memory");
+              for (int k = 0; k < 4; ++k) {
+                float a, b;
+                unpack_bf2(pair[k], a, b);
+                o[q * 8 + 2 * k] *= sigmoid_fast(a);
+                o[q * 8 + 2 * k + 1] *= sigmoid_fast(b);
               }
             }
           }
@@ -670,7 +685,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
 
 template <int DK, bool EXACT>
 inline int attn_rows_launch(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq, const CUtensorMap& to,
-                            const AttnParams& p, cudaStream_t st) {
+                            const CUtensorMap& tg, const AttnParams& p, cudaStream_t st) {
   // tiles (K ring, V ring, Q buffers, P) + small arrays (barriers, alpha, l, TMEM slot, abort flag) + alignment
   constexpr int tiles = ATC_BN * (2 * DK + 2 * 128) * 2 + (EXACT ? 1 : 2) * (DK / 64) * ATR_ROWS * 128 +
                         (EXACT ? 4 : 2) * ATR_ROWS * 128;
@@ -680,13 +695,13 @@ inline int attn_rows_launch(const CUtensorMap& tk, const CUtensorMap& tv, const 
   static PerDeviceFlags attr_set;
   if (int rc = set_max_dyn_smem_once(attr_set, paged_attn_rows_kernel<DK, EXACT>, smem)) return rc;
   const int nctas = p.tc_tiles < sm_count() ? p.tc_tiles : sm_count();
-  launch_k(paged_attn_rows_kernel<DK, EXACT>, dim3((unsigned)nctas), dim3(ATR_THREADS), (size_t)smem, st, tk, tv, tq, to, p);
+  launch_k(paged_attn_rows_kernel<DK, EXACT>, dim3((unsigned)nctas), dim3(ATR_THREADS), (size_t)smem, st, tk, tv, tq, to, tg, p);
   return launch_status();
 }
 
 inline int attn_rows_dispatch(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq, const CUtensorMap& to,
                               const AttnParams& p, cudaStream_t st) {
-  return attn_rows_launch<128, false>(tk, tv, tq, to, p, st);
+  return attn_rows_launch<128, false>(tk, tv, tq, to, tk, p, st);
 }
 
 }  // namespace b200

@@ -244,7 +244,7 @@ __global__ void __launch_bounds__(LATENT_SIMT_THREADS) attn_simt_kernel(const At
 #pragma unroll
         for (int u = 0; u < 4; ++u) a = fmaf(lat_smem[i + u], v[u], a);
       }
-      sc = p.extras.cap > 0.f ? p.extras.cap * tanhf(a / p.extras.cap) : a;
+      sc = p.extras.cap.cap > 0.f ? p.extras.cap.cap * tanhf(a / p.extras.cap.cap) : a;
     }
     const float bm = fmaxf(m, block_max(sc, red));
     const float e = sc == -INFINITY ? 0.f : expf(sc - bm);
@@ -377,7 +377,7 @@ extern "C" int b200_window_attn_simt(const void* q, long long q_row_stride, cons
   AttnSimtParams p{{(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride,
                     max_pages, page_size, num_blocks, num_seqs, min_len, max_len, window, chunk},
                    q, k_cache, v_cache, out, q_row_stride, kv_heads * DK, kv_heads * DV, heads, heads / kv_heads, DK, DV,
-                   scale, {cap, (const float*)sink_f32, gate, gate_row_stride, gate_mode}};
+                   scale, {score_cap(cap), (const float*)sink_f32, gate, gate_row_stride, gate_mode}};
   return attn_simt_launch(p, T, dtype, (cudaStream_t)stream);
 }
 

@@ -174,7 +174,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
         for (int j = 0; j < NS; ++j) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[t][j][e] *= p.scale_log2;
-          if (p.extras.cap > 0.f) cap_scores(s[t][j], p.extras.cap);
+          if (p.extras.cap.cap > 0.f) cap_scores(s[t][j], p.extras.cap);
         }
 #pragma unroll
         for (int j = 0; j < NS; ++j)
@@ -327,7 +327,7 @@ extern "C" int b200_latent_attn_expanded(const void* q, long long q_row_stride, 
   p.q_stride = q_row_stride;
   p.k_stride = p.v_stride = kv_row_stride;
   p.rot_stride = lat_row_stride;
-  p.extras = {0.f, nullptr, gate, gate_row_stride, gate ? GATE_COLUMN : GATE_NONE};
+  p.extras = {{}, nullptr, gate, gate_row_stride, gate ? GATE_COLUMN : GATE_NONE};
   p.out_stride = out_row_stride;
   p.heads = heads;
   p.group = 1;

@@ -196,9 +196,11 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
   for (int i = W + threadIdx.x; i < p.xn_cols; i += blockDim.x) orow[i] = from_f32<T>(0.f);
 }
 
-// The boundary under dynamic tanh.  A thread owns four neighbouring columns; a CTA takes batches of ROWS tokens.
+// The boundary under dynamic tanh.  A thread owns four neighbouring columns; a CTA takes batches of ROWS tokens and, where y
+// comes as rows, has the next batch on its way while it works on one.
 template <typename T, int ROWS, bool PICK>
 __global__ void __launch_bounds__(128) residual_tanh_kernel(const ResidualParams p) {
+  constexpr bool AHEAD = ROWS > 1 && !PICK;
   pdl_trigger();
   pdl_wait();
   const int W = p.W, i = (blockIdx.y * 128 + threadIdx.x) * 4;
@@ -207,13 +209,81 @@ __global__ void __launch_bounds__(128) residual_tanh_kernel(const ResidualParams
     if (vec) load4(row + i, v);
     else load4_tail(row + i, W - i, v);
   };
+  const long long first = (long long)blockIdx.x * ROWS, stride = (long long)gridDim.x * ROWS;
   if (i >= W) {                // columns past the width: zeros
     if (p.norm_w)
-      for (long long r0 = (long long)blockIdx.x * ROWS; r0 < p.num_rows; r0 += (long long)gridDim.x * ROWS)
+      for (long long r0 = first; r0 < p.num_rows; r0 += stride)
         for (int q = 0; q < ROWS && r0 + q < p.num_rows; ++q)
           for (int k = i; k < min(i + 4, p.xn_cols); ++k) reinterpret_cast<T*>(p.xn)[(r0 + q) * p.xn_stride + k] = from_f32<T>(0.f);
     return;
   }
+  auto token = [&](long long r) {
+    r = min(r, p.num_rows - 1);
+    if (!p.rows) return r;
+    const long long t = p.rows[r];
+    if (t >= 0 && t < p.num_tokens) return t;
+    if (threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, (int)t);
+    return 0ll;
+  };
+  // what the sublayer left (v) and the residual (x) of the batch that starts at r0
+  auto fetch = [&](long long r0, float (&v)[ROWS][4], float (&x)[ROWS][4]) {
+    long long tok[ROWS];
+#pragma unroll
+    for (int q = 0; q < ROWS; ++q) {
+      const long long t = tok[q] = token(r0 + q);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[q][k] = x[q][k] = 0.f;
+      if (p.ids) {
+        long long id = p.ids[t];
+        if (id < 0 || id >= p.vocab) {
+          if (threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, (int)id);
+          id = 0;
+        }
+        get(reinterpret_cast<const T*>(p.embed) + id * W, v[q]);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[q][k] *= p.embed_scale;
+      } else {
+        get(p.x + t * (long long)W, x[q]);
+        if (!PICK && p.y) get(reinterpret_cast<const T*>(p.y) + t * p.y_stride, v[q]);
+      }
+    }
+    if constexpr (PICK) {        // expert-sorted rows: four of every token requested together, added in order
+      for (int k0 = 0; k0 < p.topk; k0 += 4) {
+        int pos[ROWS][4];
+#pragma unroll
+        for (int q = 0; q < ROWS; ++q)
+#pragma unroll
+          for (int k = 0; k < 4; ++k) pos[q][k] = k0 + k < p.topk ? p.scatter_index[tok[q] * p.topk + k0 + k] : -1;
+#pragma unroll
+        for (int q = 0; q < ROWS; ++q) {
+          float e[4][4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int row = pos[q][k];
+            const bool ok = row >= 0 && row < p.y_rows;
+            if (!ok && k0 + k < p.topk && threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, row);
+            e[k][0] = e[k][1] = e[k][2] = e[k][3] = 0.f;
+            if (ok) get(reinterpret_cast<const T*>(p.y) + row * p.y_stride, e[k]);
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[q][j] += e[k][j];
+        }
+      }
+    }
+    if (p.extra) {
+      float e[ROWS][4];
+#pragma unroll
+      for (int q = 0; q < ROWS; ++q) get(reinterpret_cast<const T*>(p.extra) + tok[q] * p.extra_stride, e[q]);
+#pragma unroll
+      for (int q = 0; q < ROWS; ++q)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) v[q][k] += e[q][k];
+    }
+  };
+  float v[ROWS][4], x[ROWS][4];
+  if (first < p.num_rows) fetch(first, v, x);
   float w[4], wb[4], nw[4] = {}, nb[4] = {}, add[4] = {};
   get(p.post, w);
   get(p.post_bias, wb);
@@ -222,96 +292,52 @@ __global__ void __launch_bounds__(128) residual_tanh_kernel(const ResidualParams
     get(p.norm_bias, nb);
   }
   if (p.add) get(p.add, add);
-  for (long long r0 = (long long)blockIdx.x * ROWS; r0 < p.num_rows; r0 += (long long)gridDim.x * ROWS) {
-  float v[ROWS][4], x[ROWS][4];
-  long long tok[ROWS];
 #pragma unroll
-  for (int q = 0; q < ROWS; ++q) {
-    const long long r = min(r0 + q, p.num_rows - 1);
-    long long t = p.rows ? p.rows[r] : r;
-    if (t < 0 || t >= p.num_tokens) {
-      if (threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, (int)t);
-      t = 0;
-    }
-    tok[q] = t;
+  for (int k = 0; k < 4; ++k) wb[k] += add[k];
+  for (long long r0 = first; r0 < p.num_rows; r0 += stride) {
+    float v2[ROWS][4], x2[ROWS][4];
+    const bool more = r0 + stride < p.num_rows;
+    if (AHEAD && more) fetch(r0 + stride, v2, x2);
 #pragma unroll
-    for (int k = 0; k < 4; ++k) v[q][k] = x[q][k] = 0.f;
-    if (p.ids) {
-      long long id = p.ids[t];
-      if (id < 0 || id >= p.vocab) {
-        if (threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, (int)id);
-        id = 0;
+    for (int q = 0; q < ROWS; ++q) {
+      if (r0 + q >= p.num_rows) break;
+      float o[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        x[q][k] += fmaf(tanh_as<T>(p.post_alpha * v[q][k]), w[k], wb[k]);
+        o[k] = fmaf(tanh_as<T>(p.norm_alpha * x[q][k]), nw[k], nb[k]);
       }
-      get(reinterpret_cast<const T*>(p.embed) + id * W, v[q]);
+      float* xrow = p.x + token(r0 + q) * (long long)W + i;
+      T* orow = reinterpret_cast<T*>(p.xn) + (r0 + q) * p.xn_stride + i;
+      if (vec) {
+        if (p.write_back) store4(xrow, x[q]);
+        if (p.norm_w) store4(orow, o);
+      } else {
 #pragma unroll
-      for (int k = 0; k < 4; ++k) v[q][k] *= p.embed_scale;
-    } else {
-      get(p.x + t * (long long)W, x[q]);
-      if (!PICK && p.y) get(reinterpret_cast<const T*>(p.y) + t * p.y_stride, v[q]);
+        for (int k = 0; k < 4; ++k) {
+          if (p.write_back && i + k < W) xrow[k] = x[q][k];
+          if (p.norm_w && i + k < p.xn_cols) orow[k] = from_f32<T>(i + k < W ? o[k] : 0.f);
+        }
+      }
     }
-  }
-  if constexpr (PICK) {        // expert-sorted rows: four of every token requested together, added in order
-    for (int k0 = 0; k0 < p.topk; k0 += 4) {
-      int pos[ROWS][4];
+    if (!more) break;
+    if constexpr (AHEAD) {
 #pragma unroll
       for (int q = 0; q < ROWS; ++q)
 #pragma unroll
-        for (int k = 0; k < 4; ++k) pos[q][k] = k0 + k < p.topk ? p.scatter_index[tok[q] * p.topk + k0 + k] : -1;
-#pragma unroll
-      for (int q = 0; q < ROWS; ++q) {
-        float e[4][4];
-#pragma unroll
         for (int k = 0; k < 4; ++k) {
-          const int row = pos[q][k];
-          const bool ok = row >= 0 && row < p.y_rows;
-          if (!ok && k0 + k < p.topk && threadIdx.x == 0) report_status(B200_STATUS_BAD_INDEX, row);
-          e[k][0] = e[k][1] = e[k][2] = e[k][3] = 0.f;
-          if (ok) get(reinterpret_cast<const T*>(p.y) + row * p.y_stride, e[k]);
+          v[q][k] = v2[q][k];
+          x[q][k] = x2[q][k];
         }
-#pragma unroll
-        for (int k = 0; k < 4; ++k)
-#pragma unroll
-          for (int j = 0; j < 4; ++j) v[q][j] += e[k][j];
-      }
-    }
-  }
-  if (p.extra) {
-    float e[ROWS][4];
-#pragma unroll
-    for (int q = 0; q < ROWS; ++q) get(reinterpret_cast<const T*>(p.extra) + tok[q] * p.extra_stride, e[q]);
-#pragma unroll
-    for (int q = 0; q < ROWS; ++q)
-#pragma unroll
-      for (int k = 0; k < 4; ++k) v[q][k] += e[q][k];
-  }
-#pragma unroll
-  for (int q = 0; q < ROWS; ++q) {
-    if (r0 + q >= p.num_rows) break;
-    float o[4];
-#pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      x[q][k] += fmaf(tanh_as<T>(p.post_alpha * v[q][k]), w[k], wb[k]) + add[k];
-      o[k] = fmaf(tanh_as<T>(p.norm_alpha * x[q][k]), nw[k], nb[k]);
-    }
-    float* xrow = p.x + tok[q] * (long long)W + i;
-    T* orow = reinterpret_cast<T*>(p.xn) + (r0 + q) * p.xn_stride + i;
-    if (vec) {
-      if (p.write_back) store4(xrow, x[q]);
-      if (p.norm_w) store4(orow, o);
     } else {
-#pragma unroll
-      for (int k = 0; k < 4; ++k) {
-        if (p.write_back && i + k < W) xrow[k] = x[q][k];
-        if (p.norm_w && i + k < p.xn_cols) orow[k] = from_f32<T>(i + k < W ? o[k] : 0.f);
-      }
+      fetch(r0 + stride, v, x);
     }
-  }
   }
 }
 
 template <typename T, bool PICK>
 inline int residual_tanh_launch(const ResidualParams& p, cudaStream_t st) {
-  constexpr int MANY = 4, BATCHES = 4;
+  constexpr int MANY = PICK ? 4 : 2, BATCHES = 8;
   const unsigned gy = (unsigned)(((p.norm_w ? p.xn_cols : p.W) + 511) / 512);
   const long long many = (p.num_rows + MANY * BATCHES - 1) / (MANY * BATCHES);
   if (many * gy >= 148 * 2)

@@ -1,6 +1,6 @@
 // Grouped-query attention of decoded tokens and short portions over paged per-head keys and values (bf16), optionally
-// inside a window or chunk, with capped scores, a sink in the denominator and an output gate (attn_extras.cuh).  Scores and weights are
-// fp32: a weight enters the value product as a bf16 pair hi + lo, whose two products are summed in fp32, and the
+// inside a window or chunk, with capped scores, a sink in the denominator and an output gate (attn_extras.cuh).  Scores and
+// weights are fp32: a weight enters the value product as a bf16 pair hi + lo, whose two products are summed in fp32, and the
 // denominator sums the fp32 weights.  (attn.cuh and its kin round the weights to bf16, as the models they serve do.)
 //
 // One CTA of WARPS warps owns up to 8 columns of one KV head of one sequence, a column being one (token, query head)
@@ -165,7 +165,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
     for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) sc[mt][e] *= p.scale_log2;
-      if (p.extras.cap > 0.f) cap_scores(sc[mt], p.extras.cap);
+      if (p.extras.cap.cap > 0.f) cap_scores(sc[mt], p.extras.cap);
     }
     float alpha[2];
 #pragma unroll
@@ -321,7 +321,7 @@ extern "C" int b200_window_attn_decode(const void* q, long long q_row_stride, co
   WindowAttnParams p{};
   p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
             page_size, num_blocks, num_seqs, min_len < 1 ? 1 : min_len, max_len, window, chunk};
-  p.extras = {cap * kLog2e, (const float*)sink_f32, gate, gate_row_stride, gate_mode};
+  p.extras = {score_cap(cap * kLog2e), (const float*)sink_f32, gate, gate_row_stride, gate_mode};
   if (!latent_seqs_ok(p.seqs) || !q || !k_cache || !v_cache || !out || heads <= 0 || kv_heads <= 0 || heads % kv_heads ||
       DK <= 0 || DV <= 0 || window < 0 || chunk < 0 || max_len < 1 || most_new < 0 || !attn_extras_ok(p.extras))
     return B200_ERR_ARG;
@@ -341,7 +341,7 @@ extern "C" int b200_window_attn_decode(const void* q, long long q_row_stride, co
   p.box_tokens = page_size < WAT_BN ? page_size : WAT_BN;
   p.dk = DK;
   p.dv = DV;
-  p.scale_log2 = cap > 0.f ? scale / cap : scale * kLog2e;
+  p.scale_log2 = scale * kLog2e;
   CUtensorMap tk, tv;
   int rc = make_tmap_cache(&tk, k_cache, num_blocks, page_size, kv_heads, DK, (long long)page_size * kv_heads * DK,
                            (long long)kv_heads * DK, DK, p.box_tokens);
@@ -374,13 +374,12 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
   LatentExpandParams p{};
   p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
             page_size, num_blocks, num_seqs, 0, 0, window, chunk};
-  p.extras = {cap * kLog2e, (const float*)sink_f32, gate, gate_row_stride, gate_mode};
+  p.extras = {score_cap(cap * kLog2e), (const float*)sink_f32, gate, gate_row_stride, gate_mode};
   if (!latent_seqs_ok(p.seqs) || !q || !k_cache || !v_cache || !out || !seq_ids_i32 || n <= 0 || max_len <= 0 || T <= 0 ||
       heads <= 0 || kv_heads <= 0 || heads % kv_heads || DK <= 0 || DV <= 0 || window < 0 || chunk < 0 ||
       !attn_extras_ok(p.extras))
     return B200_ERR_ARG;
   if (gate_mode == GATE_COLUMN && (gate_row_stride % 8 || (reinterpret_cast<uintptr_t>(gate) & 15))) return B200_ERR_SHAPE;
-  const float score_scale = cap > 0.f ? scale / cap : scale * kLog2e;
   if (DK % 8 || DV % 8 || q_row_stride % 8 || out_row_stride % 8 || DK > 256 || DV > 256 || heads > 65535 || n > 65535)
     return B200_ERR_SHAPE;
   const cudaStream_t st = (cudaStream_t)stream;
@@ -407,7 +406,7 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
     a.group = group;
     a.head_chunks = (group + 7) / 8;
     a.pos_per_tile = ATR_ROWS / hh;
-    a.qk_scale = score_scale;
+    a.qk_scale = scale * kLog2e;
     a.extras = p.extras;
     a.chunk = chunk;
     a.num_blocks = num_blocks;
@@ -432,7 +431,10 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
     if (make_tmap_q(&tq, q, T, heads, DK, q_row_stride, DK, hh, a.pos_per_tile) == B200_OK) {
       a.q_tma = 1;
       a.o_tma = 32 % hh == 0 && make_tmap_q(&to, out, T, heads, DV, out_row_stride, DV, hh, 32 / hh, true) == B200_OK;
-      return attn_rows_launch<128, true>(tk, tv, tq, to, a, st);
+      CUtensorMap tg = tk;
+      a.g_tma = gate_mode == GATE_COLUMN && 32 % hh == 0 &&
+                make_tmap_q(&tg, gate, T, heads, DV, gate_row_stride, DV, hh, 32 / hh, true) == B200_OK;
+      return attn_rows_launch<128, true>(tk, tv, tq, to, tg, a, st);
     }
   }
   p.seq_ids = (const int*)seq_ids_i32;
@@ -448,6 +450,6 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
   p.group = group;
   p.DN = DK;
   p.DV = DV;
-  p.scale_log2 = score_scale;
+  p.scale_log2 = scale * kLog2e;
   return latent_expand_dispatch<true>(p, max_len, n, st);
 }
