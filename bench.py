@@ -1334,19 +1334,21 @@ def tekilix_kernels(device):
         # mixture: route + permute + two grouped products, without the sum (in the boundary) and the shared expert
         xs = [y for _, y in sets]
         rows, F = T * top, mix.gate_up.shape[1]
-        live = min(E, rows)
+        live = fm.route_plan_group_topk(gemm(xs[0], mix.router, out_dtype=torch.float32), top, E, score=mix.score,
+                                        correction=mix.correction, groups=mix.groups)[1].unique().numel()
         lone = mix.__class__(**{**vars(mix), "shared": None})
         ms = graph_ms([lambda x=x: fm.mixture_forward(lone, x) for x in xs])
         yield line(f"mixture (router to second product) T={T}", ms, 2 * (live * 2 * F * W + rows * (2 * W + 2 * F) + T * W),
                    4.0 * rows * F * W)
         gated = torch.cat([mix.gate_up, mix.gate_up], 1)
+        live_plain = vb.linear(xs[0], mix.router).topk(top).indices.unique().numel()
 
         def moe(x):
             rw, sel, plan = fm.route_plan_softmax_topk(vb.linear(x, mix.router), top, True, E)
             return fm.fused_moe_forward(E, rw, sel, x, fc2_weight=mix.down, fc1_1_2_weight=gated, defer_reduce=True, plan=plan)
 
         ms = graph_ms([lambda x=x: moe(x) for x in xs])
-        yield line(f"fused_moe (router to second product) T={T}", ms, 2 * (live * 3 * F * W + rows * (2 * W + 2 * F) + T * W),
+        yield line(f"fused_moe (router to second product) T={T}", ms, 2 * (live_plain * 3 * F * W + rows * (2 * W + 2 * F) + T * W),
                    6.0 * rows * F * W, like=f"mixture (router to second product) T={T}")
         del gated
         logits = [torch.randn(T, E, device=device) for _ in range(k)]

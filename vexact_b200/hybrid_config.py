@@ -517,7 +517,7 @@ def random_tensors(shape: HybridShape, seed: int = 0, device="cpu", dtype=torch.
         elif leaf.endswith(".conv"):
             t = t / dims[1] ** 0.5
         elif leaf == "mlp.correction":
-            t = 0.1 * t
+            t = 0.3 * t / dims[0]        # of the order of the scores
         elif leaf.startswith("norm") or name in ("final.norm", "embed.norm"):
             t = 1 + 0.1 * t if shape.sandwich else 0.1 * t
         elif leaf.endswith("norm"):
