@@ -132,6 +132,7 @@ def test_mixture_of_squared_relu_experts(dtype, E, top, ff, shared, W, count, ke
     cfg = tu.config([tu.layer(tu.attention(), tu.moe(E, top, ff, shared, count, keep))], width=W)
     w = tu.weights(cfg, seed=E)
     w["l0.mlp.router"] = _rand(E, W, seed=1, std=2 * W ** -0.5).to(BF)
+    w["l0.mlp.correction"] = _rand(E, seed=3, std=0.1).to(BF)
     lw = HybridWeights.from_tensors(HybridShape.from_config(cfg), w, dtype).layers[0].mlp
     x = _rand(T, W, seed=2).to(BF)
     sub = {k[len("l0.mlp."):]: v.double() for k, v in w.items() if k.startswith("l0.mlp.")}

@@ -95,6 +95,11 @@ __device__ __forceinline__ float gate_sigmoid(T g) {
   else return 1.f / (1.f + expf(-g));
 }
 
+// Whether a layer needs the kernels' form with extras (EXTRAS); without it they know a window and nothing else.
+inline bool attn_has_extras(const AttnExtras& x, int chunk) {
+  return chunk > 0 || x.cap.cap > 0.f || x.sink || x.gate_mode != GATE_NONE;
+}
+
 inline bool attn_extras_ok(const AttnExtras& x) {
   return x.gate_mode >= GATE_NONE && x.gate_mode <= GATE_COLUMN && (x.gate != nullptr) == (x.gate_mode != GATE_NONE);
 }

@@ -22,9 +22,10 @@
 // A token therefore gets the same bits from a decode step, a chunk and a full prefill.
 //
 // Exact form (EXACT): the weights are not rounded.  P enters its product as a bf16 pair hi + lo in two tiles (two chains of
-// UMMAs into the same O), the row sum adds the fp32 weights, a query may be limited to a window or chunk of keys (blocks
-// before it are not walked), scores may be capped, the row sum may hold a sink and the output a gate, and heads may be narrower than 128 columns (the rest arrives as zeros and is not stored).  The second
-// P tile takes the place of the second Q buffer.
+// UMMAs into the same O), the row sum adds the fp32 weights, a query may be limited to a window of keys (blocks before it
+// are not walked), and heads may be narrower than 128 columns (the rest arrives as zeros and is not stored).  The second
+// P tile takes the place of the second Q buffer.  EXTRAS: chunks of keys, capped scores, a sink in the row sum and an output
+// gate besides (attn_extras.cuh).
 //
 // Warps (12): 0 K producer, 1 UMMA issuer + TMEM owner, 2 V producer, 3 Q loader, 4-11 compute: a row is
 // shared by two threads (warps w and w + 4 of a lane quadrant), each taking 64 of the block's 128 keys for
@@ -83,7 +84,7 @@ __device__ __forceinline__ float butterfly_order_sum32(const float (&p)[32]) {
   return (c[0] + c[2]) + (c[1] + c[3]);
 }
 
-template <int DK, bool EXACT>
+template <int DK, bool EXACT, bool EXTRAS>
 __global__ void __launch_bounds__(ATR_THREADS, 1)
 paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                        const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_out,
@@ -140,7 +141,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   auto qfull_bar = [&](int b) { return bar(NB + 7 + b); };
   auto qfree_bar = [&](int b) { return bar(NB + 9 + b); };
   auto pair_bar = [&](int q) { return bar(NB + 11 + q); };   // the two compute warps of lane quadrant q meet here
-  auto gate_bar = [&](int w) { return bar(NB + 15 + w); };   // exact form: compute warp w's gate columns have arrived
+  auto gate_bar = [&](int w) { return bar(NB + 15 + w); };   // EXTRAS: compute warp w's gate columns have arrived
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
@@ -161,7 +162,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       ptx::mbar_init(qfree_bar(b), 1);
     }
     for (int q = 0; q < 4; ++q) ptx::mbar_init(pair_bar(q), 2);
-    if (EXACT)
+    if (EXTRAS)
       for (int w = 0; w < 8; ++w) ptx::mbar_init(gate_bar(w), 1);
     ptx::mbar_init(pready_bar, 8);       // compute warps
     ptx::mbar_init(ofull_bar, 1);
@@ -171,7 +172,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
     ptx::prefetch_tensormap(&tm_v);
     if (p.q_tma) ptx::prefetch_tensormap(&tm_q);
     if (p.o_tma) ptx::prefetch_tensormap(&tm_out);
-    if (EXACT && p.g_tma) ptx::prefetch_tensormap(&tm_gate);
+    if (EXTRAS && p.g_tma) ptx::prefetch_tensormap(&tm_gate);
   }
   if (warp == 1) {
     ptx::tmem_alloc(ptx::smem_u32(tmem_slot_p), TMEM_COLS);
@@ -388,7 +389,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       const int npos = min(t.pos_per_tile, t.q_len - t.tile_pos0);
       const int pi = row / t.heads_here, hd = row - pi * t.heads_here;
       const int cpos = t.q_abs0 + t.tile_pos0 + (pi < npos ? pi : 0);   // padding rows borrow position 0's mask
-      const uint32_t reach = EXACT ? visible_keys(p.window, p.chunk, cpos) : 0;   // visible: 0 <= cpos - key < reach
+      const uint32_t reach = EXACT ? visible_keys(p.window, EXTRAS ? p.chunk : 0, cpos) : 0;   // visible: 0 <= cpos - key < reach
       float m_run = -INFINITY, l_a = 0.f, l_b = 0.f;   // l of my two key groups (2 half, 2 half + 1)
       float o[64];
 #pragma unroll
@@ -422,7 +423,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
             v[32 + i] = __uint_as_float(r1[i]) * p.qk_scale;
           }
         }
-        if constexpr (EXACT) {
+        if constexpr (EXTRAS) {
           if (p.extras.cap.cap > 0.f) cap_scores(v, p.extras.cap);
         }
         if (masked) {
@@ -539,16 +540,16 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       }
       if (!alive) break;
       // tile end: the last block's O, the row sum, the store
-      const int head = t.kvh * p.group + t.hchunk * 8 + hd;
-      const long long gate_row = EXACT ? (long long)(t.q_start + t.tile_pos0 + (pi < npos ? pi : 0)) * p.extras.gate_stride : 0;
+      const int head = EXTRAS ? t.kvh * p.group + t.hchunk * 8 + hd : 0;
+      const long long gate_row = EXTRAS ? (long long)(t.q_start + t.tile_pos0 + (pi < npos ? pi : 0)) * p.extras.gate_stride : 0;
       float head_gate = 1.f;
-      if constexpr (EXACT) {
+      if constexpr (EXTRAS) {
         if (p.extras.gate_mode == GATE_HEAD)
           head_gate = gate_sigmoid(reinterpret_cast<const __nv_bfloat16*>(p.extras.gate)[gate_row + head]);
       }
       if (!ptx::mbar_wait_warp(ofull_bar, (g0 + t.nblk - 1) & 1, abort_flag, 751)) break;
       ptx::tc_fence_after();
-      if constexpr (EXACT) {
+      if constexpr (EXTRAS) {
         // The last product has read the P tiles: this warp's 4 KB of the second one receive its rows' gate columns (the box
         // its output rows leave by), while O and the row sums are read.
         if (p.extras.gate_mode == GATE_COLUMN && p.g_tma && half * 64 < p.dv) {
@@ -589,9 +590,9 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         // 4 KB of the P tile (idle from the tile's last PV product until this warp's next P write; swizzled), then eight
         // lanes store one row's 128 bytes, four rows per instruction.
         float l_row = s_lh[0][row] + s_lh[1][row];
-        if constexpr (EXACT) l_row += sink_term(p.extras, head, m_run);
+        if constexpr (EXTRAS) l_row += sink_term(p.extras, head, m_run);
         float inv = 1.0f / l_row;
-        if constexpr (EXACT) {
+        if constexpr (EXTRAS) {
           inv *= head_gate;
           if (p.extras.gate_mode == GATE_COLUMN && half * 64 < p.dv) {
             if (p.g_tma) {
@@ -683,7 +684,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   }
 }
 
-template <int DK, bool EXACT>
+template <int DK, bool EXACT, bool EXTRAS>
 inline int attn_rows_launch(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq, const CUtensorMap& to,
                             const CUtensorMap& tg, const AttnParams& p, cudaStream_t st) {
   // tiles (K ring, V ring, Q buffers, P) + small arrays (barriers, alpha, l, TMEM slot, abort flag) + alignment
@@ -693,15 +694,15 @@ inline int attn_rows_launch(const CUtensorMap& tk, const CUtensorMap& tv, const 
   constexpr int smem = (tiles + small + 1023 <= 227 * 1024) ? tiles + small + 1023 : 227 * 1024;
   static_assert(tiles + small <= 227 * 1024, "shared memory budget");
   static PerDeviceFlags attr_set;
-  if (int rc = set_max_dyn_smem_once(attr_set, paged_attn_rows_kernel<DK, EXACT>, smem)) return rc;
+  if (int rc = set_max_dyn_smem_once(attr_set, paged_attn_rows_kernel<DK, EXACT, EXTRAS>, smem)) return rc;
   const int nctas = p.tc_tiles < sm_count() ? p.tc_tiles : sm_count();
-  launch_k(paged_attn_rows_kernel<DK, EXACT>, dim3((unsigned)nctas), dim3(ATR_THREADS), (size_t)smem, st, tk, tv, tq, to, tg, p);
+  launch_k(paged_attn_rows_kernel<DK, EXACT, EXTRAS>, dim3((unsigned)nctas), dim3(ATR_THREADS), (size_t)smem, st, tk, tv, tq, to, tg, p);
   return launch_status();
 }
 
 inline int attn_rows_dispatch(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq, const CUtensorMap& to,
                               const AttnParams& p, cudaStream_t st) {
-  return attn_rows_launch<128, false>(tk, tv, tq, to, tk, p, st);
+  return attn_rows_launch<128, false, false>(tk, tv, tq, to, tk, p, st);
 }
 
 }  // namespace b200

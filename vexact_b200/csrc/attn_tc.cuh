@@ -166,7 +166,8 @@ __device__ __forceinline__ int atc_query_tile(int tiles, int per, int r) {
 template <int NC>
 __device__ __forceinline__ void atc_make(const AttnParams& p, int lin, const AtcRaw& r, AtcTile& t) {
   const int eff = r.eff < 0 ? 0 : r.eff;
-  const int x = atc_query_tile(p.tc_q_tiles, p.chunk / max(1, NC / min(8, p.group)), eff / (p.tc_hy * p.num_seqs));
+  const int rank = eff / (p.tc_hy * p.num_seqs);
+  const int x = p.chunk > 0 ? atc_query_tile(p.tc_q_tiles, p.chunk / max(1, NC / min(8, p.group)), rank) : p.tc_q_tiles - 1 - rank;
   const int y = eff % p.tc_hy;
   t.seq = r.seq;
   t.kvh = y / p.head_chunks;

@@ -7,7 +7,8 @@
 //   paged heads        k and v rows of a paged cache, [G * DN] and [G * DV] (DR = 0)
 //
 //   q         [T, q_stride]: per head DN unrotated, then DR rotated columns; head h uses key / value head h / group
-//   out[t, h] = sum_j softmax(scale q.k_j) v_j, with the chunks, cap, sink and gate of attn_extras.cuh
+//   out[t, h] = sum_j softmax(scale q.k_j) v_j, times the sigmoid of a gate per column, if any; EXTRAS: with the chunks, cap,
+//               sink and gate of attn_extras.cuh
 //
 // One CTA per (128 MT queries, head, sequence); warp w of 8 owns query rows 16 MT w .. 16 MT (w + 1) - 1 (MT = 2 for long
 // portions: every key and value fragment read from shared memory then serves two products); 64 keys per block, double
@@ -46,7 +47,7 @@ struct LexLayout {
   static constexpr int BYTES = Q + 2 * (K + V);
 };
 
-template <int DK, int DV, int MT, bool PAGED>
+template <int DK, int DV, int MT, bool PAGED, bool EXTRAS>
 __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const LatentExpandParams p) {
   using L = LexLayout<DK, DV, MT>;
   constexpr int LEX_BM = L::BM, NS = LEX_SUB / 8;
@@ -59,6 +60,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   if ((int)blockIdx.x >= tiles) return;
   const int row_base = (tiles - 1 - (int)blockIdx.x) * LEX_BM;
   const int keys = p.seqs.context_lens[seq], past = keys - len;
+  const int window = p.seqs.window > 0 ? p.seqs.window : 0x3fffffff, chunk = EXTRAS ? p.seqs.chunk : 0;
   const int key_base = PAGED ? 0 : p.key_base[i];
   const long long key0 = PAGED ? 0 : p.key_start[i] - key_base;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
@@ -66,7 +68,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   const int dk16 = (p.DN + p.DR + 15) / 16;
   const int rows = min(LEX_BM, len - row_base);
   const int last_key = min(keys, past + row_base + rows);       // keys any row of the tile sees
-  const int first_key = first_visible(p.seqs.window, p.seqs.chunk, past + row_base);
+  const int first_key = first_visible(window, chunk, past + row_base);
   const int block0 = first_key / LEX_BN, blocks = (last_key + LEX_BN - 1) / LEX_BN;
 
   for (int e = tid; e < LEX_BM * (DK / 8); e += LEX_THREADS) {
@@ -121,15 +123,15 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   }
   const int r0 = 16 * MT * warp;
   const int first_pos = past + row_base + r0;                    // position of the warp's first row
-  const int warp_first = first_visible(p.seqs.window, p.seqs.chunk, first_pos);                 // no row sees keys before this
-  const int warp_full = first_visible(p.seqs.window, p.seqs.chunk, first_pos + 16 * MT - 1);    // every row sees from here
-  int row_pos[MT];                                               // position of row g4 of the tile (and + 8)
-  uint32_t reach[MT][2];                                         // a row sees 0 <= its position - key < reach
+  // no row of the warp sees keys before the first of these, every row sees from the second (up to itself)
+  const int warp_first = EXTRAS ? first_visible(window, chunk, first_pos) : first_pos - window + 1;
+  const int warp_full = EXTRAS ? first_visible(window, chunk, first_pos + 16 * MT - 1) : first_pos + 16 * MT - window;
+  uint32_t reach[EXTRAS ? MT : 1][2];                            // a row sees 0 <= its position - key < reach
+  if constexpr (EXTRAS) {
 #pragma unroll
-  for (int t = 0; t < MT; ++t) {
-    row_pos[t] = first_pos + 16 * t + g4;
+    for (int t = 0; t < MT; ++t)
 #pragma unroll
-    for (int e = 0; e < 2; ++e) reach[t][e] = visible_keys(p.seqs.window, p.seqs.chunk, row_pos[t] + 8 * e);
+      for (int e = 0; e < 2; ++e) reach[t][e] = visible_keys(window, chunk, first_pos + 16 * t + g4 + 8 * e);
   }
   for (int b = block0; b < blocks; ++b) {
     if (b + 1 < blocks) {
@@ -169,19 +171,23 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
       const bool edge = base + LEX_SUB - 1 > first_pos || base < warp_full;
 #pragma unroll
       for (int t = 0; t < MT; ++t) {
+        const int pos0 = first_pos + 16 * t + g4;                 // position of row g4 of the tile (and + 8)
         float mb[2] = {m[t][0], m[t][1]};
 #pragma unroll
         for (int j = 0; j < NS; ++j) {
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[t][j][e] *= p.scale_log2;
-          if (p.extras.cap.cap > 0.f) cap_scores(s[t][j], p.extras.cap);
+          if constexpr (EXTRAS) {
+            if (p.extras.cap.cap > 0.f) cap_scores(s[t][j], p.extras.cap);
+          }
         }
 #pragma unroll
         for (int j = 0; j < NS; ++j)
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             float v = s[t][j][e];
-            if (edge && (uint32_t)(row_pos[t] + 8 * (e >> 1) - (base + 8 * j + 2 * t4 + (e & 1))) >= reach[t][e >> 1]) v = -INFINITY;
+            const uint32_t seen = EXTRAS ? reach[EXTRAS ? t : 0][e >> 1] : (uint32_t)window;   // 0 <= position - key < seen
+            if (edge && (uint32_t)(pos0 + 8 * (e >> 1) - (base + 8 * j + 2 * t4 + (e & 1))) >= seen) v = -INFINITY;
             s[t][j][e] = v;
             mb[e >> 1] = fmaxf(mb[e >> 1], v);
           }
@@ -248,20 +254,24 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   for (int tt = 0; tt < MT; ++tt)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      float inv = 1.f / (abm_quad_sum(l[tt][e]) + sink_term(p.extras, h, m[tt][e]));
+      float sum = abm_quad_sum(l[tt][e]);
+      if (EXTRAS) sum += sink_term(p.extras, h, m[tt][e]);
+      float inv = 1.f / sum;
       const int r = r0 + 16 * tt + g4 + 8 * e;
       if (r >= rows) continue;
       const long long t = t0 + row_base + r;
       const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(p.extras.gate) + t * p.extras.gate_stride;
-      if (p.extras.gate_mode == GATE_HEAD) inv *= gate_sigmoid(gate[h]);
+      if (EXTRAS && p.extras.gate_mode == GATE_HEAD) inv *= gate_sigmoid(gate[h]);
 #pragma unroll
       for (int j = 0; j < DV / 8; ++j) {
         const int c = 8 * j + 2 * t4;
         if (c < p.DV) {
           float a = o[tt][j][2 * e] * inv, b = o[tt][j][2 * e + 1] * inv;
           if (p.extras.gate_mode == GATE_COLUMN) {
-            a *= gate_sigmoid(gate[h * p.DV + c]);
-            b *= gate_sigmoid(gate[h * p.DV + c + 1]);
+            float ga, gb;
+            unpack_bf2(*reinterpret_cast<const uint32_t*>(gate + h * p.DV + c), ga, gb);
+            a *= sigmoid_fast(ga);
+            b *= sigmoid_fast(gb);
           }
           *reinterpret_cast<uint32_t*>(p.out + t * p.out_stride + (long long)h * p.DV + c) = pack_bf2(a, b);
         }
@@ -269,29 +279,29 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
     }
 }
 
-template <int DK, int DV, int MT, bool PAGED>
+template <int DK, int DV, int MT, bool PAGED, bool EXTRAS>
 inline int latent_expand_launch(const LatentExpandParams& p, int max_len, int n, cudaStream_t st) {
   constexpr int smem = LexLayout<DK, DV, MT>::BYTES, LEX_BM = LexLayout<DK, DV, MT>::BM;
   static_assert(smem <= 227 * 1024, "shared memory budget");
   static PerDeviceFlags attr_set;
-  if (int rc = set_max_dyn_smem_once(attr_set, latent_expand_kernel<DK, DV, MT, PAGED>, smem)) return rc;
-  launch_k(latent_expand_kernel<DK, DV, MT, PAGED>,
+  if (int rc = set_max_dyn_smem_once(attr_set, latent_expand_kernel<DK, DV, MT, PAGED, EXTRAS>, smem)) return rc;
+  launch_k(latent_expand_kernel<DK, DV, MT, PAGED, EXTRAS>,
            dim3((unsigned)((max_len + LEX_BM - 1) / LEX_BM), (unsigned)p.heads, (unsigned)n), dim3(LEX_THREADS), (size_t)smem,
            st, p);
   return launch_status();
 }
 
-template <bool PAGED>
+template <bool PAGED, bool EXTRAS>
 inline int latent_expand_dispatch(const LatentExpandParams& p, int max_len, int n, cudaStream_t st) {
   const int dk = p.DN + p.DR;
   const bool two = max_len > 128;
   if (dk <= 64 && p.DV <= 64)
-    return two ? latent_expand_launch<64, 64, 2, PAGED>(p, max_len, n, st) : latent_expand_launch<64, 64, 1, PAGED>(p, max_len, n, st);
+    return two ? latent_expand_launch<64, 64, 2, PAGED, EXTRAS>(p, max_len, n, st) : latent_expand_launch<64, 64, 1, PAGED, EXTRAS>(p, max_len, n, st);
   if (dk <= 128 && p.DV <= 128)
-    return two ? latent_expand_launch<128, 128, 2, PAGED>(p, max_len, n, st) : latent_expand_launch<128, 128, 1, PAGED>(p, max_len, n, st);
+    return two ? latent_expand_launch<128, 128, 2, PAGED, EXTRAS>(p, max_len, n, st) : latent_expand_launch<128, 128, 1, PAGED, EXTRAS>(p, max_len, n, st);
   if (dk <= 192 && p.DV <= 128)
-    return two ? latent_expand_launch<192, 128, 2, PAGED>(p, max_len, n, st) : latent_expand_launch<192, 128, 1, PAGED>(p, max_len, n, st);
-  return latent_expand_launch<256, 256, 1, PAGED>(p, max_len, n, st);
+    return two ? latent_expand_launch<192, 128, 2, PAGED, EXTRAS>(p, max_len, n, st) : latent_expand_launch<192, 128, 1, PAGED, EXTRAS>(p, max_len, n, st);
+  return latent_expand_launch<256, 256, 1, PAGED, EXTRAS>(p, max_len, n, st);
 }
 
 }  // namespace b200
@@ -335,5 +345,5 @@ extern "C" int b200_latent_attn_expanded(const void* q, long long q_row_stride, 
   p.DR = DR;
   p.DV = DV;
   p.scale_log2 = scale * kLog2e;
-  return latent_expand_dispatch<false>(p, max_len, n, (cudaStream_t)stream);
+  return latent_expand_dispatch<false, false>(p, max_len, n, (cudaStream_t)stream);
 }

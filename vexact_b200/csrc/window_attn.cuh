@@ -36,7 +36,7 @@ struct WatLayout {
   static_assert(STAGES * STAGE >= DV * 8 * 4 + 64, "a warp's ring holds its partial result");
 };
 
-template <int DK, int DV, int WARPS, int STAGES>
+template <int DK, int DV, int WARPS, int STAGES, bool EXTRAS>
 __global__ void __launch_bounds__(WARPS * 32)
 window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                    const WindowAttnParams p) {
@@ -51,8 +51,8 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
   pdl_trigger();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-  const int seq = blockIdx.z, kvh = blockIdx.y / p.head_chunks, chunk = blockIdx.y % p.head_chunks;
-  const int heads_here = min(8, p.group - chunk * 8);
+  const int seq = blockIdx.z, kvh = blockIdx.y / p.head_chunks, hchunk = blockIdx.y % p.head_chunks;
+  const int heads_here = min(8, p.group - hchunk * 8);
   const int q_start = p.seqs.query_start_loc[seq], q_len = p.seqs.query_start_loc[seq + 1] - q_start;
   const int kv_len = p.seqs.context_lens[seq], pos0 = blockIdx.x * p.pos_per_tile;
   if (q_len < p.seqs.min_len || q_len > p.seqs.max_len || pos0 >= q_len) return;
@@ -66,9 +66,10 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
     return pi < p.pos_per_tile && pos0 + pi < q_len;
   };
   auto col_q = [&](int c) { return pos0 + (col_valid(c) ? c / heads_here : 0); };   // a spare column repeats the first position
-  auto col_head = [&](int c) { return kvh * p.group + chunk * 8 + c % heads_here; };
+  auto col_head = [&](int c) { return kvh * p.group + hchunk * 8 + c % heads_here; };
   const int last_pos = q_abs0 + min(pos0 + p.pos_per_tile, q_len) - 1;
-  const int blk0 = first_visible(p.seqs.window, p.seqs.chunk, q_abs0 + pos0) / WAT_BN, nblk = last_pos / WAT_BN + 1 - blk0;
+  const int chunk = EXTRAS ? p.seqs.chunk : 0;
+  const int blk0 = first_visible(p.seqs.window, chunk, q_abs0 + pos0) / WAT_BN, nblk = last_pos / WAT_BN + 1 - blk0;
   const int mine = (nblk - warp + WARPS - 1) / WARPS;      // blocks of this warp: blk0 + warp + i * WARPS
 
   if (threadIdx.x == 0) {
@@ -125,7 +126,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
 #pragma unroll
   for (int j = 0; j < 2; ++j) {
     cpos[j] = q_abs0 + col_q(2 * t + j);
-    reach[j] = visible_keys(p.seqs.window, p.seqs.chunk, cpos[j]);
+    reach[j] = visible_keys(p.seqs.window, chunk, cpos[j]);
   }
 
   float o[DV / 16][4];
@@ -165,7 +166,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
     for (int mt = 0; mt < MT; ++mt) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) sc[mt][e] *= p.scale_log2;
-      if (p.extras.cap.cap > 0.f) cap_scores(sc[mt], p.extras.cap);
+      if (EXTRAS && p.extras.cap.cap > 0.f) cap_scores(sc[mt], p.extras.cap);
     }
     float alpha[2];
 #pragma unroll
@@ -281,10 +282,11 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
     }
     const int head = col_head(c);
     const long long row = q_start + col_q(c);
-    const float inv = 1.f / (l + sink_term(p.extras, head, m));
+    if (EXTRAS) l += sink_term(p.extras, head, m);
+    const float inv = 1.f / l;
     a *= inv;
     b *= inv;
-    if (p.extras.gate_mode != GATE_NONE) {
+    if (EXTRAS && p.extras.gate_mode != GATE_NONE) {
       const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(p.extras.gate) + row * p.extras.gate_stride;
       const bool per_head = p.extras.gate_mode == GATE_HEAD;
       a *= gate_sigmoid(gate[per_head ? head : head * p.dv + d]);
@@ -294,15 +296,24 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
   }
 }
 
-template <int DK, int DV, int WARPS, int STAGES>
+template <int DK, int DV, int WARPS, int STAGES, bool EXTRAS>
 inline int window_attn_launch(const CUtensorMap& tk, const CUtensorMap& tv, const WindowAttnParams& p, dim3 grid,
                               cudaStream_t st) {
   constexpr int smem = WatLayout<DK, DV, WARPS, STAGES>::BYTES;
   static_assert(smem <= 226 * 1024, "shared memory budget");
   static PerDeviceFlags attr_set;
-  if (int rc = set_max_dyn_smem_once(attr_set, window_attn_kernel<DK, DV, WARPS, STAGES>, smem)) return rc;
-  launch_k(window_attn_kernel<DK, DV, WARPS, STAGES>, grid, dim3(WARPS * 32), (size_t)smem, st, tk, tv, p);
+  if (int rc = set_max_dyn_smem_once(attr_set, window_attn_kernel<DK, DV, WARPS, STAGES, EXTRAS>, smem)) return rc;
+  launch_k(window_attn_kernel<DK, DV, WARPS, STAGES, EXTRAS>, grid, dim3(WARPS * 32), (size_t)smem, st, tk, tv, p);
   return launch_status();
+}
+
+template <bool EXTRAS>
+inline int window_attn_dispatch(const CUtensorMap& tk, const CUtensorMap& tv, const WindowAttnParams& p, dim3 grid,
+                                cudaStream_t st) {
+  if (p.dk <= 64 && p.dv <= 64) return window_attn_launch<64, 64, 2, 4, EXTRAS>(tk, tv, p, grid, st);
+  if (p.dk <= 128 && p.dv <= 128) return window_attn_launch<128, 128, 2, 3, EXTRAS>(tk, tv, p, grid, st);
+  if (p.dk <= 192 && p.dv <= 128) return window_attn_launch<192, 128, 2, 2, EXTRAS>(tk, tv, p, grid, st);
+  return window_attn_launch<256, 256, 2, 2, EXTRAS>(tk, tv, p, grid, st);
 }
 
 }  // namespace b200
@@ -353,10 +364,8 @@ extern "C" int b200_window_attn_decode(const void* q, long long q_row_stride, co
   const dim3 grid((unsigned)((most + p.pos_per_tile - 1) / p.pos_per_tile), (unsigned)(kv_heads * p.head_chunks),
                   (unsigned)num_seqs);
   const cudaStream_t st = (cudaStream_t)stream;
-  if (DK <= 64 && DV <= 64) return window_attn_launch<64, 64, 2, 4>(tk, tv, p, grid, st);
-  if (DK <= 128 && DV <= 128) return window_attn_launch<128, 128, 2, 3>(tk, tv, p, grid, st);
-  if (DK <= 192 && DV <= 128) return window_attn_launch<192, 128, 2, 2>(tk, tv, p, grid, st);
-  return window_attn_launch<256, 256, 2, 2>(tk, tv, p, grid, st);
+  return attn_has_extras(p.extras, chunk) ? window_attn_dispatch<true>(tk, tv, p, grid, st)
+                                          : window_attn_dispatch<false>(tk, tv, p, grid, st);
 }
 
 // Long portions: the n sequences named, which are those that bring at least min_len tokens.  Heads of 65 .. 128 columns go
@@ -434,7 +443,8 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
       CUtensorMap tg = tk;
       a.g_tma = gate_mode == GATE_COLUMN && 32 % hh == 0 &&
                 make_tmap_q(&tg, gate, T, heads, DV, gate_row_stride, DV, hh, 32 / hh, true) == B200_OK;
-      return attn_rows_launch<128, true>(tk, tv, tq, to, tg, a, st);
+      return attn_has_extras(a.extras, chunk) ? attn_rows_launch<128, true, true>(tk, tv, tq, to, tg, a, st)
+                                              : attn_rows_launch<128, true, false>(tk, tv, tq, to, tg, a, st);
     }
   }
   p.seq_ids = (const int*)seq_ids_i32;
@@ -451,5 +461,6 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
   p.DN = DK;
   p.DV = DV;
   p.scale_log2 = scale * kLog2e;
-  return latent_expand_dispatch<true>(p, max_len, n, st);
+  return attn_has_extras(p.extras, chunk) ? latent_expand_dispatch<true, true>(p, max_len, n, st)
+                                          : latent_expand_dispatch<true, false>(p, max_len, n, st);
 }
