@@ -66,9 +66,9 @@ struct AttnParams {
   int o_tma;             // rows-on-lanes kernel: a warp's 32 output rows leave by one asynchronous TMA store
   int min_q;             // tcgen05 kernels: sequences with fewer queries are skipped (another kernel's)
   int window;            // rows-on-lanes kernel, exact form: keys a query sees, its own included (0: every earlier one)
-  int chunk;             // .. : tokens of a chunk beyond which nothing is seen (0: none)
-  AttnExtras extras;     // .. : capped scores, sink, output gate
-  int g_tma;             // .. : a warp's gate columns arrive by one TMA box
+  int chunk;             // the same with extras: tokens of a chunk beyond which nothing is seen (0: none)
+  AttnExtras extras;     // the same with extras: capped scores, sink, output gate
+  int g_tma;             // the same with extras: a warp's gate columns arrive by one TMA box
   int dv;                // rows-on-lanes kernel, exact form: value columns of a head (at most 128)
   int scalar_out;        // development knob B200_ATTN_OUT_SCALAR=1: 2-byte output stores in the keys-on-lanes kernel
 };

@@ -67,7 +67,8 @@ struct Eight<__nv_bfloat16> {
     unpack_bf2(v.w, f[6], f[7]);
   }
   static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&f)[8]) {
-    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf2(f[0], f[1]), pack_bf2(f[2], f[3]), pack_bf2(f[4], f[5]), pack_bf2(f[6], f[7]));
+    *reinterpret_cast<uint4*>(p) =
+        make_uint4(pack_bf2(f[0], f[1]), pack_bf2(f[2], f[3]), pack_bf2(f[4], f[5]), pack_bf2(f[6], f[7]));
   }
 };
 template <>
@@ -200,7 +201,8 @@ __global__ void __launch_bounds__(PREP_MAX_WARPS * 32, 2) attn_prep_kernel(const
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           const float u = x[c][e];
-          x[c][e] = fmaf(w[3][c][e], u, fmaf(w[2][c][e], past[2][c][e], fmaf(w[1][c][e], past[1][c][e], w[0][c][e] * past[0][c][e])));
+          const float a = fmaf(w[1][c][e], past[1][c][e], w[0][c][e] * past[0][c][e]);
+          x[c][e] = fmaf(w[3][c][e], u, fmaf(w[2][c][e], past[2][c][e], a));
           past[0][c][e] = past[1][c][e];
           past[1][c][e] = past[2][c][e];
           past[2][c][e] = u;
@@ -453,13 +455,14 @@ extern "C" int b200_attn_prep(const void* proj, long long proj_row_stride, int v
                      num_seqs <= 0 || num_seqs > 65535))
     return B200_ERR_ARG;
   if (DK % 8 || DV % 8 || proj_row_stride % 8 || rot_dims % 2 || rot_dims > 2 * PREP_MAX_PAIRS || DK > 512 || v_off < -1 ||
-      v_off % 8 > 0 || (v_off < 0 && DV != DK) || T > 0x7fffffffLL)
+      v_off % 8 > 0 || (v_off < 0 && DV != DK) || T > 0x7fffffffLL ||
+      ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_out)) & 15))
     return B200_ERR_SHAPE;
   if (T == 0) return B200_OK;
   AttnPrepParams p{{(const int*)query_start_loc, (const int*)context_lens, (const int*)state_slots, num_seqs, num_state_slots},
                    proj, proj_row_stride, v_off, (const long long*)positions_i64, (const int*)slot_mapping_i32,
-                   (const float*)conv_w_f32, conv_state, taps, one_token_each, 0, norm, (const float*)q_norm_f32, (const float*)k_norm_f32,
-                   dim, eps, (const float*)inv_freq_f32, rot_dims, rot_half, rot_mag, q_out, k_cache, v_cache, heads,
+                   (const float*)conv_w_f32, conv_state, taps, one_token_each, 0, norm, (const float*)q_norm_f32,
+                   (const float*)k_norm_f32, dim, eps, (const float*)inv_freq_f32, rot_dims, rot_half, rot_mag, q_out, k_cache, v_cache, heads,
                    kv_heads, DK, DV, T, num_slots, 1};
   const cudaStream_t st = (cudaStream_t)stream;
   return dtype == 0 ? attn_prep_dispatch<__nv_bfloat16>(p, st) : attn_prep_dispatch<float>(p, st);
