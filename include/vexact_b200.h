@@ -385,18 +385,19 @@ int b200_moe_unpermute_add_rmsnorm(const void* y, const void* scatter_index, con
  *      Sequences: query_start_loc [S + 1], context_lens [S] (tokens after the step), state_slots [S] (-1 = none), i32. */
 
 /* b200_gemm_bf16 with an activation in the epilogue, as one product or a batch of them:
- *   out[g][t, n] = act(sum_k x[g][t, k] * w[g][n, k] + bias[n]).
+ *   out[g][t, n] = act(sum_k x[g][t, k] * w[g][n, k] + bias[n])      (n >= N - act_skip: without act).
  * act: 0 none, 1 the tanh form of gelu, 2 times sigmoid(gate[g][t, n]), 3 the square of relu.  bias only with batch = 1.  w_batch_stride is
  * a multiple of w_row_stride (at least N rows); strides of x and w are multiples of 8.  out_dtype 0 = bf16, 1 = f32. */
 int b200_gemm_bf16_ex(const void* x, const void* w, const void* bias, const void* gate, void* out, long long T, int N,
                       int K, int batch, long long x_row_stride, long long x_batch_stride, long long w_row_stride,
                       long long w_batch_stride, long long out_row_stride, long long out_batch_stride,
-                      long long gate_row_stride, long long gate_batch_stride, int act, int out_dtype, void* stream);
+                      long long gate_row_stride, long long gate_batch_stride, int act, int act_skip, int out_dtype,
+                      void* stream);
 /* The same in true fp32, every tensor fp32, any strides. */
 int b200_gemm_f32_ex(const void* x, const void* w, const void* bias, const void* gate, void* out, long long T, int N,
                      int K, int batch, long long x_row_stride, long long x_batch_stride, long long w_row_stride,
                      long long w_batch_stride, long long out_row_stride, long long out_batch_stride,
-                     long long gate_row_stride, long long gate_batch_stride, int act, void* stream);
+                     long long gate_row_stride, long long gate_batch_stride, int act, int act_skip, void* stream);
 
 /* One sublayer boundary of a hyper-connected residual (streams [num_tokens, num_streams, W] fp32, in place):
  *   x_t <- sum_s mix[s, t] x_s + m * out[t] * y   (y given), or the streams start as copies of embed[ids] (ids given);
@@ -482,7 +483,9 @@ int b200_latent_gather(const void* cache, void* dst, const void* seq_ids_i32, co
                        page_table_stride, int max_pages, int page_size, int num_blocks, int num_seqs, void* stream);
 
 /* Grouped-query attention over paged per-head keys and values [blocks, page, kv_heads, DK | DV], fp32 weights; a query sees
- * a window of its last tokens, its own included, and its chunk floor(position / chunk) (0: no limit).  cap: scores become
+ * a window of its last tokens, its own included, and its chunk floor(position / chunk) (0: no limit); `keep` first tokens are seen
+ * besides.  sigmoid_bias_f32 [heads] (or NULL): weights are sigmoid(score + bias) and not normalized; the output is times
+ * out_scale.  cap: scores become
  * cap * tanh(score / cap) (0: none); sink_f32 [heads] (or NULL): exp(sink) joins the denominator; gate rows of the model
  * dtype: the output is times the sigmoid of one number per head (gate_mode 1) or per column (2), 0: none.  _decode: bf16, tensor cores, sequences with min_len .. max_len new
  * tokens (most_new: the most any brings); DK, DV <= 256, page_size a multiple of 8 that divides 32 or is a multiple of it.
@@ -492,34 +495,49 @@ int b200_window_attn_decode(const void* q, long long q_row_stride, const void* k
                             out, long long out_row_stride, const void* query_start_loc, const void* context_lens,
                             const void* page_table, long long page_table_stride, int max_pages, int page_size, int
                             num_blocks, int num_seqs, int min_len, int max_len, int most_new, int window, int chunk,
-                            float cap, const void* sink_f32, const void* gate, long long gate_row_stride, int gate_mode,
-                            int heads, int kv_heads, int DK, int DV, float scale, void* stream);
+                            int keep, float cap, const void* sink_f32, const void* sigmoid_bias_f32, float out_scale,
+                            const void* gate, long long gate_row_stride, int gate_mode, int heads, int kv_heads, int DK, int DV, float scale, void* stream);
 int b200_window_attn_prefill(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void*
                              out, long long out_row_stride, const void* query_start_loc, const void* context_lens,
                              const void* page_table, long long page_table_stride, int max_pages, int page_size, int
                              num_blocks, int num_seqs, const void* seq_ids_i32, int n, int max_len, int min_len, int
-                             window, int chunk, float cap, const void* sink_f32, const void* gate, long long
-                             gate_row_stride, int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float
+                             window, int chunk, int keep, float cap, const void* sink_f32, const void*
+                             sigmoid_bias_f32, float out_scale, const void* gate, long long gate_row_stride, int
+                             gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float
                              scale, int form, void* stream);
 int b200_window_attn_simt(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache, void* out,
-                          const void* query_start_loc, const void* context_lens, const void* page_table, long long
+                          long long out_row_stride, const void* query_start_loc, const void* context_lens, const void* page_table, long long
                           page_table_stride, int max_pages, int page_size, int num_blocks, int num_seqs, int min_len,
-                          int max_len, int window, int chunk, float cap, const void* sink_f32, const void* gate, long
-                          long gate_row_stride, int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float
+                          int max_len, int window, int chunk, int keep, float cap, const void* sink_f32, const void*
+                          sigmoid_bias_f32, float out_scale, const void* gate, long long gate_row_stride, int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float
                           scale, int dtype, void* stream);
 
 /* Between the projections [q: heads * DK | k: kv_heads * DK | ..] and that attention: short convolution of q and k
  * (conv_w_f32 [taps, (heads + kv_heads) * DK] or NULL; conv_state [num_state_slots, taps - 1, channels] is read and moved
- * on), values (columns from v_off, or with -1 the convolved keys), norm of q and k (0 none, 1 per head, 2 over all heads; dim
+ * on), values (columns from v_off, or with -1 the convolved keys), norm of q and k (0 none, 1 per head, weights NULL: ones, 2 over all heads; dim
  * true columns of a head), rotation of the first rot_dims columns (rot_half: pairs (i, i + rot_dims / 2), else (2i, 2i + 1);
- * cosine and sine times rot_mag); q to q_out [T, heads * DK], k and v to their pages.  one_token_each: no sequence brings
+ * cosine and sine times rot_mag), values mixed with the rows v_first, (1 - v_mix) v + v_mix first (NULL: not); q to q_out [T, heads * DK], k and v to their pages.  one_token_each: no sequence brings
  * more than one token (one launch; otherwise two with a convolution).  DK <= 512, rot_dims <= 256. */
 int b200_attn_prep(const void* proj, long long proj_row_stride, int v_off, const void* positions_i64, const void*
                    slot_mapping_i32, const void* conv_w_f32, void* conv_state, int taps, const void* query_start_loc,
                    const void* context_lens, const void* state_slots, int num_seqs, int num_state_slots, int
                    one_token_each, int norm, const void* q_norm_f32, const void* k_norm_f32, int dim, float eps, const
-                   void* inv_freq_f32, int rot_dims, int rot_half, float rot_mag, void* q_out, void* k_cache, void* v_cache,
+                   void* inv_freq_f32, int rot_dims, int rot_half, float rot_mag, const void* v_first, long long
+                   v_first_row_stride, float v_mix, void* q_out, void* k_cache, void* v_cache,
                    long long T, int heads, int kv_heads, int DK, int DV, long long num_slots, int dtype, void* stream);
+
+/* minGRU over projection rows, `width` columns each from z_off, x_off and g_off: z = sigmoid(z + z_bias), u = x + x_bias,
+ *   S = (1 - z) S + z (u >= 0 ? u + 1/2 : sigmoid(u)),  out = S * silu(g) * out_scale;  state [num_slots, width] fp32.
+ * _scan: token by token, sequences with min_len .. max_len new tokens.  _chunk_scan: bf16, tiles of tokens, sequences with at
+ * least min_len; channels of a CTA, 16 or 32 (speed only).  width, offsets and strides multiples of 8. */
+int b200_gru_scan(const void* proj, long long proj_row_stride, int z_off, int x_off, int g_off, const void* z_bias_f32,
+                  const void* x_bias_f32, void* state_f32, void* out, long long out_row_stride, const void* query_start_loc,
+                  const void* context_lens, const void* state_slots, int num_seqs, int num_slots, int width, float out_scale,
+                  int min_len, int max_len, int dtype, void* stream);
+int b200_gru_chunk_scan(const void* proj, long long proj_row_stride, int z_off, int x_off, int g_off, const void* z_bias_f32,
+                        const void* x_bias_f32, void* state_f32, void* out, long long out_row_stride, const void*
+                        query_start_loc, const void* context_lens, const void* state_slots, int num_seqs, int num_slots, int
+                        width, float out_scale, int min_len, int channels, void* stream);
 
 /* Gated delta rule over act rows [q: groups * N | k: groups * N | v: heads * P] (convolved, not yet unit vectors):
  *   S = g S; u = beta (v - S^T k); S += k u^T; o = S^T q,   g = exp(-exp(A_log) dt), beta = sigmoid(b), k and q divided by
@@ -541,13 +559,15 @@ int b200_delta_chunk_scan(const void* act, long long act_row_stride, const void*
  *   x <- x + rms_norm(y) * post (+ add);  xn = rms_norm(x) * norm_w (NULL = no xn), columns W .. xn_cols zero.
  * y: rows, or with scatter_index the sum of the token's topk rows of y [y_rows]; extra (or NULL) is added to it.  ids given
  * instead of y: the model starts, x = rms_norm(embed[ids] * embed_scale) * post (+ add).  rows_i32 (with write_back = 0):
- * only these.  post_bias_f32 given: both norms are tanh(alpha v) * weight + bias instead. */
+ * only these.  post_bias_f32 given: both norms are tanh(alpha v) * weight + bias instead.  post_f32 NULL: y is not normed, and
+ * is times sigmoid(gate + gate_bias) where gate (rows of the model dtype) is given. */
 int b200_residual_step(void* x_f32, const void* y, long long y_row_stride, long long y_rows, const void*
                        scatter_index_i32, int topk, const void* extra, long long extra_row_stride, const void* embed,
                        const void* ids_i64, long long vocab, const void* rows_i32, long long num_tokens, long long
                        num_rows, int W, const void* post_f32, const void* add_f32, const void* norm_w_f32, float eps,
                        float embed_scale, const void* post_bias_f32, float post_alpha, const void* norm_bias_f32, float
-                       norm_alpha, void* xn, long long xn_row_stride, int xn_cols, int write_back, int dtype, void* stream);
+                       norm_alpha, const void* gate, long long gate_row_stride, const void* gate_bias_f32, void* xn, long
+                       long xn_row_stride, int xn_cols, int write_back, int dtype, void* stream);
 
 /* Gated feed-forwards: act(s g) * (s u) * o with fp32 row factors s = scale_in, o = scale_out (NULL: 1); act 1 silu, 2 the
  * tanh form of gelu.  _gemm_glu: one product, w [2 * n_out, K] gate rows first; _moe_grouped_gemm_glu: expert-sorted rows,

@@ -22,23 +22,28 @@ SIGNATURES = {
     "b200_status_read": [C.POINTER(C.c_int), P],
     "b200_gemm_bf16": [P, P, P, P, LL, I, I, LL, LL, LL, I, P],
     "b200_gemm_f16": [P, P, P, P, LL, I, I, LL, LL, LL, I, P],
-    "b200_gemm_bf16_ex": [P, P, P, P, P, LL, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, I, I, P],
-    "b200_gemm_f32_ex": [P, P, P, P, P, LL, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, I, P],
+    "b200_gemm_bf16_ex": [P, P, P, P, P, LL, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, I, I, I, P],
+    "b200_gemm_f32_ex": [P, P, P, P, P, LL, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, I, I, P],
     "b200_hyper_step": [P, P, LL, P, P, LL, P, LL, LL, I, I, P, P, F, P, P, F, P, LL, I, I, I, P],
     "b200_ssm_conv": [P, LL, I, I, I, I, I, P, P, P, P, P, P, P, P, P, I, I, LL, I, I, P],
     "b200_ssm_scan": [P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P],
     "b200_ssm_gate_norm": [P, LL, P, LL, P, P, LL, LL, I, I, I, I, F, I, I, P],
-    "b200_residual_step": [P, P, LL, LL, P, I, P, LL, P, P, LL, P, LL, LL, I, P, P, P, F, F, P, F, P, F, P, LL, I, I, I, P],
+    "b200_residual_step": [P, P, LL, LL, P, I, P, LL, P, P, LL, P, LL, LL, I, P, P, P, F, F, P, F, P, F, P, LL, P, P, LL, I, I, I,
+                           P],
+    "b200_gru_scan": [P, LL, I, I, I, P, P, P, P, LL, P, P, P, I, I, I, F, I, I, I, P],
+    "b200_gru_chunk_scan": [P, LL, I, I, I, P, P, P, P, LL, P, P, P, I, I, I, F, I, I, P],
     "b200_delta_scan": [P, LL, P, P, LL, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P],
     "b200_delta_chunk_scan": [P, LL, P, P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P],
     "b200_latent_prep": [P, LL, P, LL, P, LL, P, I, I, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, F, LL, I, P],
     "b200_latent_attn_simt": [P, P, P, P, P, P, LL, I, I, I, I, I, I, I, LL, I, I, I, F, I, P],
-    "b200_window_attn_simt": [P, LL, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, I, F, P, P, LL, I, LL, I, I, I, I, F, I, P],
-    "b200_window_attn_decode": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, I, I, I, I, I, F, P, P, LL, I, I, I, I, I, F, P],
-    "b200_window_attn_prefill": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, P, I, I, I, I, I, F, P, P, LL, I, LL, I, I, I,
-                                 I, F, I, P],
-    "b200_attn_prep": [P, LL, I, P, P, P, P, I, P, P, P, I, I, I, I, P, P, I, F, P, I, I, F, P, P, P, LL, I, I, I, I, LL, I,
-                       P],
+    "b200_window_attn_simt": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, I, I, I, I, I, F, P, P, F, P, LL, I, LL, I, I, I, I,
+                              F, I, P],
+    "b200_window_attn_decode": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, I, I, I, I, I, I, F, P, P, F, P, LL, I, I, I, I, I,
+                                F, P],
+    "b200_window_attn_prefill": [P, LL, P, P, P, LL, P, P, P, LL, I, I, I, I, P, I, I, I, I, I, I, F, P, P, F, P, LL, I, LL, I,
+                                 I, I, I, F, I, P],
+    "b200_attn_prep": [P, LL, I, P, P, P, P, I, P, P, P, I, I, I, I, P, P, I, F, P, I, I, F, P, LL, F, P, P, P, LL, I, I, I, I,
+                       LL, I, P],
     "b200_gemm_glu": [P, P, P, P, LL, I, I, LL, LL, I, P],
     "b200_glu": [P, LL, P, P, P, LL, I, I, I, P],
     "b200_moe_grouped_gemm_glu": [P, P, P, P, P, P, P, LL, I, I, I, LL, I, I, I, P],
@@ -108,7 +113,7 @@ class B200Error(RuntimeError):
     pass
 
 
-ABI_VERSION = 7
+ABI_VERSION = 8
 
 
 def _check_fresh(lib) -> None:

@@ -100,12 +100,12 @@ GEMM_ACTS = {None: 0, "gelu_tanh": 1, "sigmoid_gate": 2, "relu2": 3}
 
 def gemm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = None, act: str | None = None,
          gate: torch.Tensor | None = None, out: torch.Tensor | None = None,
-         out_dtype: torch.dtype | None = None) -> torch.Tensor:
+         out_dtype: torch.dtype | None = None, act_skip: int = 0) -> torch.Tensor:
     """act(x @ weight^T + bias) for bf16 (tcgen05) or fp32 (true fp32) tensors, one product or a batch.
 
     One product: x [T, K], weight [N, K] -> [T, N].  Batch (3-D weight [B, N, K]): x [T, B, K] -> [T, B, N]; x, `out`
     and `gate` may be views with any row and batch stride.  act: None, "gelu_tanh", "relu2" (the square of relu),
-    "sigmoid_gate" (times sigmoid(gate), gate shaped like the output)."""
+    "sigmoid_gate" (times sigmoid(gate), gate shaped like the output); the last `act_skip` of the N columns pass without."""
     _require_cuda("x", x)
     _require_cuda("weight", weight)
     assert x.dtype == weight.dtype, "Incompatible dtypes"
@@ -132,7 +132,7 @@ def gemm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None = None
     xs, os_, gs = strides(x), strides(out), strides(gate)
     ws = (weight.stride(-2), weight.stride(0) if batched else 0)
     args = [x.data_ptr(), weight.data_ptr(), _lib.ptr(bias), _lib.ptr(gate), out.data_ptr(), T, N, K, B, *xs, *ws, *os_,
-            *gs, GEMM_ACTS[act]]
+            *gs, GEMM_ACTS[act], act_skip]
     if x.dtype == torch.bfloat16:
         if out.dtype not in (torch.bfloat16, torch.float32):
             raise ValueError(f"unsupported output dtype {out.dtype}")

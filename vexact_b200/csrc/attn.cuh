@@ -67,7 +67,8 @@ struct AttnParams {
   int min_q;             // tcgen05 kernels: sequences with fewer queries are skipped (another kernel's)
   int window;            // rows-on-lanes kernel, exact form: keys a query sees, its own included (0: every earlier one)
   int chunk;             // the same with extras: tokens of a chunk beyond which nothing is seen (0: none)
-  AttnExtras extras;     // the same with extras: capped scores, sink, output gate
+  int keep;              // the same with extras: first tokens seen whatever the window or chunk
+  AttnExtras extras;     // the same with extras: capped scores, sink, output gate, sigmoid weights
   int g_tma;             // the same with extras: a warp's gate columns arrive by one TMA box
   int dv;                // rows-on-lanes kernel, exact form: value columns of a head (at most 128)
   int scalar_out;        // development knob B200_ATTN_OUT_SCALAR=1: 2-byte output stores in the keys-on-lanes kernel

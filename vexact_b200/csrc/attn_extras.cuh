@@ -1,9 +1,12 @@
 // What an attention layer may add around softmax(q k^T) v, as every kernel that offers it reads it:
 //
 //   mask      window of w tokens: position i sees the keys i - w + 1 .. i;  chunks of c tokens: position i sees the keys
-//             j <= i of its own chunk, floor(j / c) = floor(i / c), counted from the sequence's first token (0: no limit)
+//             j <= i of its own chunk, floor(j / c) = floor(i / c), counted from the sequence's first token (0: no limit);
+//             beside either, the sequence's first `keep` tokens are seen from everywhere behind them
 //   cap       a score s becomes cap * tanh(s / cap)
 //   sink      exp(sink[head]) is added to the denominator: a key without a value
+//   sigmoid   a key's weight is sigmoid(score + bias[head]) and nothing is divided by a sum of weights
+//   scale     the head's output times a constant
 //   gate      the head's output is multiplied by the sigmoid of one number per head, or of one per column
 //
 // All of it is fp32.  Kernels that keep scores in units of log2 get the cap in those units, cap * log2(e).
@@ -13,6 +16,8 @@
 namespace b200 {
 
 constexpr int GATE_NONE = 0, GATE_HEAD = 1, GATE_COLUMN = 2;
+// Forms of an attention kernel: softmax inside a window and nothing else, softmax with all of the above, sigmoid weights.
+constexpr int ATTN_PLAIN = 0, ATTN_EXTRAS = 1, ATTN_SIGMOID = 2;
 
 // A cap and the coefficients of cap * tanh(s / cap) = s + c3 s^3 + c5 s^5 + c7 s^7 .. in the scores' units.
 struct ScoreCap {
@@ -31,6 +36,8 @@ struct AttnExtras {
   const void* gate;        // rows of the model dtype, gate_stride apart: [heads] or [heads * DV]; null with GATE_NONE
   long long gate_stride;
   int gate_mode;
+  const float* sigmoid_bias;   // [heads]: sigmoid weights; null: softmax
+  float out_scale;
 };
 
 // Keys that the query at `pos` sees, its own included, and the first of them.
@@ -42,6 +49,40 @@ __device__ __forceinline__ uint32_t visible_keys(int window, int chunk, int pos)
 __device__ __forceinline__ int first_visible(int window, int chunk, int pos) {
   const int a = window > 0 ? max(0, pos - window + 1) : 0;
   return chunk > 0 ? max(a, pos - pos % chunk) : a;
+}
+
+// Key j (of a causal walk) is seen from `pos`: n = visible_keys(window, chunk, pos).
+__device__ __forceinline__ bool key_visible(uint32_t n, int keep, int pos, int j) {
+  return (uint32_t)(pos - j) < (keep > 0 && j < keep ? 0x80000000u : n);
+}
+
+// Blocks of BN keys that some query of first .. last sees: `head` blocks from key 0 that hold kept tokens and lie before
+// the window, then those from block `from`.
+struct KeyBlocks {
+  int head, from, count;
+  __device__ __forceinline__ int at(int i) const { return i < head ? i : from + (i - head); }
+};
+template <int BN>
+__device__ __forceinline__ KeyBlocks key_blocks(int window, int chunk, int keep, int first, int last) {
+  KeyBlocks k;
+  k.from = first_visible(window, chunk, first) / BN;
+  k.head = keep > 0 ? min((keep + BN - 1) / BN, k.from) : 0;
+  k.count = last / BN + 1 - k.from + k.head;
+  return k;
+}
+
+// Sigmoid weights of scores in units of log2 (bias included), w[i] = 1 / (1 + 2^-v[i]); two share a reciprocal.  2^-v is
+// kept below 2^60, so that a product of two stays in range; weights below 2^-60 come out as 2^-60.  Keys that are not seen
+// (va, vb) weigh nothing, and what their scores hold does not reach the other key's rounding.
+__device__ __forceinline__ void sigmoid_pair(float& a, float& b, bool va = true, bool vb = true) {
+  a = va ? a : -INFINITY;
+  b = vb ? b : -INFINITY;
+  float ea, eb;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(ea) : "f"(fminf(-a, 60.f)));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(eb) : "f"(fminf(-b, 60.f)));
+  const float da = 1.f + ea, db = 1.f + eb, inv = __fdividef(1.f, da * db);
+  a = va ? db * inv : 0.f;
+  b = vb ? da * inv : 0.f;
 }
 
 // tanh in fp32.  Below 0.2 the odd Taylor polynomial through x^7 (the next term is below 1.2e-8), above it
@@ -95,13 +136,16 @@ __device__ __forceinline__ float gate_sigmoid(T g) {
   else return 1.f / (1.f + expf(-g));
 }
 
-// Whether a layer needs the kernels' form with extras (EXTRAS); without it they know a window and nothing else.
-inline bool attn_has_extras(const AttnExtras& x, int chunk) {
-  return chunk > 0 || x.cap.cap > 0.f || x.sink || x.gate_mode != GATE_NONE;
+// The form of the kernels that a layer needs.
+inline int attn_form(const AttnExtras& x, int chunk, int keep) {
+  if (x.sigmoid_bias) return ATTN_SIGMOID;
+  return chunk > 0 || keep > 0 || x.cap.cap > 0.f || x.sink || x.gate_mode != GATE_NONE || x.out_scale != 1.f ? ATTN_EXTRAS
+                                                                                                       : ATTN_PLAIN;
 }
 
 inline bool attn_extras_ok(const AttnExtras& x) {
-  return x.gate_mode >= GATE_NONE && x.gate_mode <= GATE_COLUMN && (x.gate != nullptr) == (x.gate_mode != GATE_NONE);
+  return x.gate_mode >= GATE_NONE && x.gate_mode <= GATE_COLUMN && (x.gate != nullptr) == (x.gate_mode != GATE_NONE) &&
+         !(x.sink && x.sigmoid_bias);
 }
 
 }  // namespace b200

@@ -3,9 +3,11 @@
 // Projection row of a token: [q: H * DK | k: G * DK | ...], the values anywhere in it or none.  Every part is optional:
 //   convolution   y_t = sum_j w[j] u_(t - taps + 1 + j) per channel of q and k, no bias, no activation, zeros before the
 //                 sequence's first token; the last taps - 1 inputs of a sequence are its state (slots as in ssm.cuh)
-//   values        columns of the row, or (keys as values) the convolved keys before norm and rotation
-//   norm          x / sqrt(mean(x^2) + eps) * w per head (w [DK]), or over all heads of q, and of k, at once (w [H * DK],
-//                 [G * DK])
+//   values        columns of the row, or (keys as values) the convolved keys before norm and rotation; columns of the row may be
+//                 mixed with another row of the same token, (1 - mix) v + mix first
+//   norm          x / sqrt(mean(x^2) + eps) * w per head (w [DK], or none), or over all heads of q, and of k, at once
+//                 (w [H * DK], [G * DK]).  The rotation that follows keeps lengths as long as rot_mag is 1, so a norm without
+//                 a weight may as well be meant behind it
 //   rotation      the first rot_dims columns of a head turn in pairs (2i, 2i + 1) or (i, i + rot_dims / 2) by
 //                 position * inv_freq[i]; cosine and sine are multiplied by rot_mag
 // q goes to rows of its own, k and v to their pages.  fp32 from the projection's values to the stored ones.
@@ -50,6 +52,9 @@ struct AttnPrepParams {
   int heads, kv_heads, DK, DV;
   long long num_tokens, num_slots;
   int per_cta;                 // tokens of a CTA
+  const void* v_first;         // [T, v_first_stride]: values mixed in, or null
+  long long v_first_stride;
+  float v_mix;
 };
 
 // Eight neighbouring values.
@@ -278,7 +283,11 @@ __global__ void __launch_bounds__(PREP_MAX_WARPS * 32, 2) attn_prep_kernel(const
       const float* src = is_q ? p.q_norm : p.k_norm;
       if (p.norm == PREP_NORM_ALL) src += (is_q ? h : kvh) * p.DK;
 #pragma unroll
-      for (int c = 0; c < NC; ++c) load8(src + col[c], nw[c]);
+      for (int c = 0; c < NC; ++c) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) nw[c][e] = 1.f;
+        if (src) load8(src + col[c], nw[c]);
+      }
     }
     T* qk_out = is_q ? reinterpret_cast<T*>(p.q_out) + (t0 * p.heads + h) * p.DK : reinterpret_cast<T*>(p.k_cache) + kvh * p.DK;
     T* v_out = reinterpret_cast<T*>(p.v_cache) + kvh * p.DV;
@@ -389,6 +398,13 @@ __global__ void __launch_bounds__(PREP_MAX_WARPS * 32, 2) attn_prep_kernel(const
       float f[8];
       v.load(proj + q * p.proj_stride + p.v_off + e);
       v.get(f);
+      if (p.v_first) {
+        float first[8];
+        v.load(reinterpret_cast<const T*>(p.v_first) + (t0 + q) * p.v_first_stride + e);
+        v.get(first);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) f[k] = fmaf(p.v_mix, first[k], (1.f - p.v_mix) * f[k]);
+      }
       Eight<T>::store(reinterpret_cast<T*>(p.v_cache) + (long long)s_store[q] * width + e, f);
     }
   }
@@ -437,25 +453,27 @@ inline int attn_prep_dispatch(AttnPrepParams& p, cudaStream_t st) {
 
 // See the head of this file.  proj rows [q: heads * DK | k: kv_heads * DK | ..]; v_off -1: keys as values (DV = DK).
 // conv_w_f32 [taps, (heads + kv_heads) * DK] or NULL; conv_state [num_state_slots, taps - 1, the same] (unused with one
-// tap); one_token_each: no sequence brings more than one token.  norm: 0 none, 1 per head, 2 over all heads.
+// tap); one_token_each: no sequence brings more than one token.  norm: 0 none, 1 per head (weights NULL: ones), 2 over all
+// heads.  v_first NULL: values as they are projected.
 extern "C" int b200_attn_prep(const void* proj, long long proj_row_stride, int v_off, const void* positions_i64,
                               const void* slot_mapping_i32, const void* conv_w_f32, void* conv_state, int taps,
                               const void* query_start_loc, const void* context_lens, const void* state_slots, int num_seqs,
                               int num_state_slots, int one_token_each, int norm, const void* q_norm_f32,
                               const void* k_norm_f32, int dim, float eps, const void* inv_freq_f32, int rot_dims,
-                              int rot_half, float rot_mag, void* q_out, void* k_cache, void* v_cache, long long T, int heads,
-                              int kv_heads, int DK, int DV, long long num_slots, int dtype, void* stream) {
+                              int rot_half, float rot_mag, const void* v_first, long long v_first_row_stride, float v_mix,
+                              void* q_out, void* k_cache, void* v_cache, long long T, int heads, int kv_heads, int DK, int DV,
+                              long long num_slots, int dtype, void* stream) {
   using namespace b200;
   if (!proj || !positions_i64 || !slot_mapping_i32 || !q_out || !k_cache || !v_cache || T < 0 || heads <= 0 || kv_heads <= 0 ||
       DK <= 0 || DV <= 0 || dim <= 0 || dim > DK || (dtype != 0 && dtype != 1) || norm < PREP_NORM_NONE ||
-      norm > PREP_NORM_ALL || (norm && (!q_norm_f32 || !k_norm_f32)) || rot_dims < 0 || rot_dims > dim ||
+      norm > PREP_NORM_ALL || (norm == PREP_NORM_ALL && (!q_norm_f32 || !k_norm_f32)) || (!q_norm_f32 != !k_norm_f32) || (v_first && v_off < 0) || rot_dims < 0 || rot_dims > dim ||
       (rot_dims && !inv_freq_f32))
     return B200_ERR_ARG;
   if (conv_w_f32 && (taps < 1 || (taps > 1 && !conv_state) || !query_start_loc || !context_lens || !state_slots ||
                      num_seqs <= 0 || num_seqs > 65535))
     return B200_ERR_ARG;
   if (DK % 8 || DV % 8 || proj_row_stride % 8 || rot_dims % 2 || rot_dims > 2 * PREP_MAX_PAIRS || DK > 512 || v_off < -1 ||
-      v_off % 8 > 0 || (v_off < 0 && DV != DK) || T > 0x7fffffffLL ||
+      v_off % 8 > 0 || v_first_row_stride % 8 || (reinterpret_cast<uintptr_t>(v_first) & 15) || (v_off < 0 && DV != DK) || T > 0x7fffffffLL ||
       ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_out)) & 15))
     return B200_ERR_SHAPE;
   if (T == 0) return B200_OK;
@@ -463,7 +481,7 @@ extern "C" int b200_attn_prep(const void* proj, long long proj_row_stride, int v
                    proj, proj_row_stride, v_off, (const long long*)positions_i64, (const int*)slot_mapping_i32,
                    (const float*)conv_w_f32, conv_state, taps, one_token_each, 0, norm, (const float*)q_norm_f32,
                    (const float*)k_norm_f32, dim, eps, (const float*)inv_freq_f32, rot_dims, rot_half, rot_mag, q_out, k_cache, v_cache, heads,
-                   kv_heads, DK, DV, T, num_slots, 1};
+                   kv_heads, DK, DV, T, num_slots, 1, v_first, v_first_row_stride, v_mix};
   const cudaStream_t st = (cudaStream_t)stream;
   return dtype == 0 ? attn_prep_dispatch<__nv_bfloat16>(p, st) : attn_prep_dispatch<float>(p, st);
 }

@@ -24,8 +24,9 @@
 // Exact form (EXACT): the weights are not rounded.  P enters its product as a bf16 pair hi + lo in two tiles (two chains of
 // UMMAs into the same O), the row sum adds the fp32 weights, a query may be limited to a window of keys (blocks before it
 // are not walked), and heads may be narrower than 128 columns (the rest arrives as zeros and is not stored).  The second
-// P tile takes the place of the second Q buffer.  EXTRAS: chunks of keys, capped scores, a sink in the row sum and an output
-// gate besides (attn_extras.cuh).
+// P tile takes the place of the second Q buffer.  FORM ATTN_EXTRAS: kept first tokens, chunks of keys, capped scores, a sink
+// in the row sum and an output gate besides (attn_extras.cuh).  ATTN_SIGMOID: all but the sink with sigmoid weights; no
+// maximum and no sum then, and O stays in TMEM from a tile's first block to its last.
 //
 // Warps (12): 0 K producer, 1 UMMA issuer + TMEM owner, 2 V producer, 3 Q loader, 4-11 compute: a row is
 // shared by two threads (warps w and w + 4 of a lane quadrant), each taking 64 of the block's 128 keys for
@@ -84,12 +85,13 @@ __device__ __forceinline__ float butterfly_order_sum32(const float (&p)[32]) {
   return (c[0] + c[2]) + (c[1] + c[3]);
 }
 
-template <int DK, bool EXACT, bool EXTRAS>
+template <int DK, bool EXACT, int FORM>
 __global__ void __launch_bounds__(ATR_THREADS, 1)
 paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                        const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_out,
                        const __grid_constant__ CUtensorMap tm_gate, const AttnParams p) {
   constexpr int DV = 128, NC = ATR_ROWS, KST = 2, VST = 2;
+  constexpr bool EXTRAS = FORM != ATTN_PLAIN, SIGMOID = FORM == ATTN_SIGMOID;
   constexpr int KH = DK / 64, VH = DV / 64;
   constexpr int K_BYTES = ATC_BN * DK * 2, V_BYTES = ATC_BN * DV * 2;
   constexpr int KV_BYTES = KST * K_BYTES + VST * V_BYTES;
@@ -100,6 +102,11 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   // Q buffer of a tile, and the parity of its use
   auto q_buf = [](uint32_t it) { return EXACT ? 0u : it & 1u; };
   auto q_par = [](uint32_t it) { return EXACT ? it & 1u : (it >> 1) & 1u; };
+  // key block j of a tile's walk
+  auto block_of = [](const AtcTile& t, int j) {
+    if constexpr (EXTRAS) return j < t.head ? j : t.blk0 + j - t.head;
+    else return EXACT ? t.blk0 + j : j;
+  };
   constexpr int TMEM_COLS = 512;           // S0, S1 (128 each), O (128)
 
   // All shared memory is dynamic (the tiles take 224 of the 227 KB): the 1024-byte aligned tiles first,
@@ -205,7 +212,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       const int* ptab = p.page_table + (long long)t.seq * p.page_table_stride;
       const int valid_pages = (t.kv_len + p.page_size - 1) / p.page_size;
       auto page_of = [&](int j, int b, int& in_page) {
-        const int tok = (EXACT ? t.blk0 + j : j) * ATC_BN + b * p.box_tokens;
+        const int tok = block_of(t, j) * ATC_BN + b * p.box_tokens;
         const int lpage = tok / p.page_size;
         in_page = tok - lpage * p.page_size;
         int phys = -1;
@@ -248,6 +255,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       AtcTile t;
       int lin = atc_next_tile<NC>(p, blockIdx.x, t);   // tile of the next QK^T to issue
       uint32_t gs = 0, gp = 0, tile_it = 0;             // next QK^T block, next PV block, tile counter
+      uint32_t starts = 0;                              // SIGMOID: bit g & 31, block g is the first of its tile
       int j = 0;
       auto issue_next_s = [&]() {   // S of global block gs into S buffer gs & 1
         const int qb = q_buf(tile_it);
@@ -266,6 +274,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         ptx::umma_commit(sfull_bar(b));
         ptx::umma_commit(kempty_bar(s));
         ATR_STAMP(0, gs, 0);   // QK issued
+        if constexpr (SIGMOID) starts = (starts & ~(1u << (gs & 31))) | ((j == 0 ? 1u : 0u) << (gs & 31));
         ++gs;
         if (++j == t.nblk) {
           ptx::umma_commit(qfree_bar(qb));
@@ -293,7 +302,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
           const uint64_t da = kdesc(p_smem + (kk >> 2) * (NC * 128) + (kk & 3) * 32);    // A = P rows, K = keys
           // B = V as it lies: 16 keys per step are 16 rows of 128 B; the other 64-wide d half is ATC_BN*128 B on
           const uint64_t db = umma_desc_mn_sw128(sv + kk * 16 * 128, ATC_BN * 128);
-          ptx::umma_bf16(tm_o, da, db, idesc_o, kk != 0 ? 1u : 0u);
+          ptx::umma_bf16(tm_o, da, db, idesc_o, kk != 0 || (SIGMOID && !(starts >> (g & 31) & 1u)) ? 1u : 0u);
         }
         if constexpr (EXACT) {
 #pragma unroll
@@ -390,6 +399,9 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       const int pi = row / t.heads_here, hd = row - pi * t.heads_here;
       const int cpos = t.q_abs0 + t.tile_pos0 + (pi < npos ? pi : 0);   // padding rows borrow position 0's mask
       const uint32_t reach = EXACT ? visible_keys(p.window, EXTRAS ? p.chunk : 0, cpos) : 0;   // visible: 0 <= cpos - key < reach
+      const int keep = EXTRAS ? p.keep : 0;
+      float bias = 0.f;                                // of sigmoid weights, in units of log2
+      if constexpr (SIGMOID) bias = p.extras.sigmoid_bias[t.kvh * p.group + t.hchunk * 8 + hd] * kLog2e;
       float m_run = -INFINITY, l_a = 0.f, l_b = 0.f;   // l of my two key groups (2 half, 2 half + 1)
       float o[64];
 #pragma unroll
@@ -397,7 +409,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       for (int j = 0; j < t.nblk; ++j) {
         const uint32_t g = g0 + j;
         const int b = g & 1, s = g % VST;
-        const int blk = EXACT ? t.blk0 + j : j;
+        const int blk = block_of(t, j);
         const int key0 = blk * ATC_BN + half * 64;        // first key of my half of the block
         const bool masked = key0 + 63 > cpos || (EXACT && (uint32_t)(cpos - key0) >= reach);
         if (!ptx::mbar_wait_warp(sfull_bar(b), (g >> 1) & 1, abort_flag, 740 + b)) {
@@ -411,7 +423,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
           __syncwarp();
           store_pending = false;
         }
-        float v[64];
+        float v[64], alpha = 1.f;
         {
           uint32_t r0[32], r1[32];
           tmem_ld32(tm_s0 + b * ATC_BN + lane_addr + half * 64, r0);
@@ -426,10 +438,36 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         if constexpr (EXTRAS) {
           if (p.extras.cap.cap > 0.f) cap_scores(v, p.extras.cap);
         }
+        if constexpr (SIGMOID) {
+          if (masked) {
+#pragma unroll
+            for (int i = 0; i < 64; i += 2) {
+              v[i] += bias;
+              v[i + 1] += bias;
+              sigmoid_pair(v[i], v[i + 1], key_visible(reach, keep, cpos, key0 + i), key_visible(reach, keep, cpos, key0 + i + 1));
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 64; i += 2) {
+              v[i] += bias;
+              v[i + 1] += bias;
+              sigmoid_pair(v[i], v[i + 1]);
+            }
+          }
+          // the block before has been multiplied: its P tile may be overwritten (O stays where it is)
+          if (j > 0) {
+            if (!ptx::mbar_wait_warp(ofull_bar, (g - 1) & 1, abort_flag, 750)) {
+              alive = false;
+              break;
+            }
+            __syncwarp();
+            if (lane == 0) ptx::mbar_arrive(ofree_bar);
+          }
+        } else {
         if (masked) {
 #pragma unroll
           for (int i = 0; i < 64; ++i)
-            if (EXACT ? (uint32_t)(cpos - key0 - i) >= reach : key0 + i > cpos) v[i] = -INFINITY;
+            if (EXACT ? !key_visible(reach, keep, cpos, key0 + i) : key0 + i > cpos) v[i] = -INFINITY;
         }
         float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -441,7 +479,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
           break;
         }
         const float m_new = fmaxf(fmaxf(m_run, kMinMax), fmaxf(mx, s_hmax[b][half ^ 1][row]));
-        const float alpha = fast_exp2(m_run - m_new);
+        alpha = fast_exp2(m_run - m_new);
         m_run = m_new;
         if (warp == 4) ATR_STAMP(1, g, 1);   // maxima joined
         // fold the previous block's O (its PV product has also finished reading the P tile by then)
@@ -467,6 +505,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
           __syncwarp();
           if (lane == 0) ptx::mbar_arrive(ofree_bar);
         }
+        }
         if (warp == 4) ATR_STAMP(1, g, 2);   // folded
         // p = bf16(2^(v - m)), group sums in butterfly order, P half row -> shared memory
         float sa, sb;
@@ -477,7 +516,8 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
             uint32_t hi[4], lo[4];
 #pragma unroll
             for (int k = 0; k < 4; ++k) {
-              const float a = fast_exp2(v[q * 8 + 2 * k] - m_new), c = fast_exp2(v[q * 8 + 2 * k + 1] - m_new);
+              const float a = SIGMOID ? v[q * 8 + 2 * k] : fast_exp2(v[q * 8 + 2 * k] - m_run);
+              const float c = SIGMOID ? v[q * 8 + 2 * k + 1] : fast_exp2(v[q * 8 + 2 * k + 1] - m_run);
               s4[k] += a + c;
               hi[k] = pack_bf2(a, c);
               float ha, hc;
@@ -494,7 +534,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
           uint32_t pk[16];
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
-            const __nv_bfloat162 b2 = __floats2bfloat162_rn(fast_exp2(v[i] - m_new), fast_exp2(v[i + 1] - m_new));
+            const __nv_bfloat162 b2 = __floats2bfloat162_rn(fast_exp2(v[i] - m_run), fast_exp2(v[i + 1] - m_run));
             pf[i] = __low2float(b2);
             pf[i + 1] = __high2float(b2);
             pk[i >> 1] = *reinterpret_cast<const uint32_t*>(&b2);
@@ -506,7 +546,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
 #pragma unroll
           for (int i = 0; i < 32; i += 2) {
             const __nv_bfloat162 b2 =
-                __floats2bfloat162_rn(fast_exp2(v[32 + i] - m_new), fast_exp2(v[32 + i + 1] - m_new));
+                __floats2bfloat162_rn(fast_exp2(v[32 + i] - m_run), fast_exp2(v[32 + i + 1] - m_run));
             pf[i] = __low2float(b2);
             pf[i + 1] = __high2float(b2);
             pk[i >> 1] = *reinterpret_cast<const uint32_t*>(&b2);
@@ -581,19 +621,24 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
       // The half-row sums meet in the maxima buffer of the tile's last block: both threads of every row read
       // it before that block's P was published, and the next tile's first block uses the other buffer.
       float (*s_lh)[NC] = s_hmax[(g0 + t.nblk - 1) & 1];
-      s_lh[half][row] = l_a + l_b;             // (l_0 + l_1) from half 0, (l_2 + l_3) from half 1
-      if (!pair_sync()) break;
+      if constexpr (!SIGMOID) {
+        s_lh[half][row] = l_a + l_b;           // (l_0 + l_1) from half 0, (l_2 + l_3) from half 1
+        if (!pair_sync()) break;
+      }
       if (warp == 4) ATR_STAMP(2, g0 + t.nblk - 1, 2);   // row sums joined
       {
         // Output.  A thread holds 64 value dims of one row (128 bytes); stored from there, one warp instruction
         // would touch 32 rows' lines with 16 bytes each.  The warp first lays its 32 half rows down in its own
         // 4 KB of the P tile (idle from the tile's last PV product until this warp's next P write; swizzled), then eight
         // lanes store one row's 128 bytes, four rows per instruction.
-        float l_row = s_lh[0][row] + s_lh[1][row];
-        if constexpr (EXTRAS) l_row += sink_term(p.extras, head, m_run);
-        float inv = 1.0f / l_row;
+        float inv = 1.f;
+        if constexpr (!SIGMOID) {
+          float l_row = s_lh[0][row] + s_lh[1][row];
+          if constexpr (EXTRAS) l_row += sink_term(p.extras, head, m_run);
+          inv = 1.0f / l_row;
+        }
         if constexpr (EXTRAS) {
-          inv *= head_gate;
+          inv *= p.extras.out_scale * head_gate;
           if (p.extras.gate_mode == GATE_COLUMN && half * 64 < p.dv) {
             if (p.g_tma) {
               if (!ptx::mbar_wait_warp(gate_bar(warp - 4), gate_phase & 1, abort_flag, 790 + warp)) break;
@@ -684,7 +729,7 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   }
 }
 
-template <int DK, bool EXACT, bool EXTRAS>
+template <int DK, bool EXACT, int FORM>
 inline int attn_rows_launch(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq, const CUtensorMap& to,
                             const CUtensorMap& tg, const AttnParams& p, cudaStream_t st) {
   // tiles (K ring, V ring, Q buffers, P) + small arrays (barriers, alpha, l, TMEM slot, abort flag) + alignment
@@ -694,15 +739,15 @@ inline int attn_rows_launch(const CUtensorMap& tk, const CUtensorMap& tv, const 
   constexpr int smem = (tiles + small + 1023 <= 227 * 1024) ? tiles + small + 1023 : 227 * 1024;
   static_assert(tiles + small <= 227 * 1024, "shared memory budget");
   static PerDeviceFlags attr_set;
-  if (int rc = set_max_dyn_smem_once(attr_set, paged_attn_rows_kernel<DK, EXACT, EXTRAS>, smem)) return rc;
+  if (int rc = set_max_dyn_smem_once(attr_set, paged_attn_rows_kernel<DK, EXACT, FORM>, smem)) return rc;
   const int nctas = p.tc_tiles < sm_count() ? p.tc_tiles : sm_count();
-  launch_k(paged_attn_rows_kernel<DK, EXACT, EXTRAS>, dim3((unsigned)nctas), dim3(ATR_THREADS), (size_t)smem, st, tk, tv, tq, to, tg, p);
+  launch_k(paged_attn_rows_kernel<DK, EXACT, FORM>, dim3((unsigned)nctas), dim3(ATR_THREADS), (size_t)smem, st, tk, tv, tq, to, tg, p);
   return launch_status();
 }
 
 inline int attn_rows_dispatch(const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& tq, const CUtensorMap& to,
                               const AttnParams& p, cudaStream_t st) {
-  return attn_rows_launch<128, false, false>(tk, tv, tq, to, tk, p, st);
+  return attn_rows_launch<128, false, ATTN_PLAIN>(tk, tv, tq, to, tk, p, st);
 }
 
 }  // namespace b200

@@ -105,7 +105,8 @@ __device__ __forceinline__ void halving_warp_sum(float (&e)[N], int lane) {
 // One unit of work: NC columns of one (sequence, KV head[, head chunk]) pair.
 struct AtcTile {
   int seq, kvh, hchunk, heads_here, pos_per_tile, q_start, q_len, kv_len, tile_pos0, q_abs0;
-  int blk0, nblk;   // key blocks blk0 .. blk0 + nblk - 1 (blk0 is 0 without a window or chunk)
+  int blk0, nblk;   // nblk key blocks: `head` from key 0 (kept tokens before the window), the others from block blk0
+  int head;         // (head and blk0 are 0 without a window or chunk)
   bool valid;
 };
 
@@ -182,8 +183,10 @@ __device__ __forceinline__ void atc_make(const AttnParams& p, int lin, const Atc
   t.q_abs0 = t.kv_len - t.q_len;
   int last_q = t.tile_pos0 + t.pos_per_tile - 1;
   if (last_q > t.q_len - 1) last_q = t.q_len - 1;
-  t.blk0 = first_visible(p.window, p.chunk, max(0, t.q_abs0 + t.tile_pos0)) / ATC_BN;
-  t.nblk = t.valid ? (t.q_abs0 + last_q) / ATC_BN + 1 - t.blk0 : 0;
+  const KeyBlocks walk = key_blocks<ATC_BN>(p.window, p.chunk, p.keep, max(0, t.q_abs0 + t.tile_pos0), t.q_abs0 + last_q);
+  t.blk0 = walk.from;
+  t.head = walk.head;
+  t.nblk = t.valid ? walk.count : 0;
 }
 
 template <int NC>

@@ -86,6 +86,7 @@ struct GemmParams {
   long long out_batch_stride;
   // Plain-mode activation of the fp32 accumulator (after the bias), see GEMM_ACT_*.
   int act;
+  int act_skip;                    // last features that pass without it
   const __nv_bfloat16* gate;       // GEMM_ACT_SIGMOID_GATE: gate[row * gate_stride + g * gate_batch_stride + feature]
   long long gate_stride, gate_batch_stride;
   uint64_t w_policy;
@@ -500,17 +501,18 @@ gemm_ws_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__
           return __bfloat16_as_ushort(f2bf(v));
         };
         // activation of one accumulator element of tile column c (row t.row0 + c of the product)
+        const int act = f < p.n_w - p.act_skip ? p.act : GEMM_ACT_NONE;
         const __nv_bfloat16* gate =
-            p.act == GEMM_ACT_SIGMOID_GATE ? p.gate + (long long)t.group * p.gate_batch_stride + f : nullptr;
+            act == GEMM_ACT_SIGMOID_GATE ? p.gate + (long long)t.group * p.gate_batch_stride + f : nullptr;
         const long long out_base = (long long)t.group * p.out_batch_stride;
         // one branch around sixteen independent chains, not one inside each: the chains then overlap
         auto finish = [&](const uint32_t (&r)[16], float (&v)[16], int c0) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]) + bias;
-          if (p.act == GEMM_ACT_GELU_TANH) {
+          if (act == GEMM_ACT_GELU_TANH) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) v[j] = gelu_tanh_fast(v[j]);
-          } else if (p.act == GEMM_ACT_RELU2) {
+          } else if (act == GEMM_ACT_RELU2) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const float s = p.scale_out && c0 + j < t.n ? p.scale_out[t.row0 + c0 + j] : 1.f, z = fmaxf(v[j], 0.f);
@@ -773,7 +775,7 @@ __global__ void __launch_bounds__(256)
 gemm_f32_tiled_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias,
                       const float* __restrict__ gate, float* __restrict__ out, long long T, int N, int K,
                       long long x_row, long long x_batch, long long w_row, long long w_batch, long long out_row,
-                      long long out_batch, long long gate_row, long long gate_batch, int act,
+                      long long out_batch, long long gate_row, long long gate_batch, int act, int act_skip,
                       const int4* __restrict__ tile_table, const int* __restrict__ tile_count,
                       const float* __restrict__ scale_out) {
   pdl_trigger();
@@ -823,9 +825,10 @@ gemm_f32_tiled_kernel(const float* __restrict__ x, const float* __restrict__ w, 
       const int n = n0 + tx + 16 * j;
       if (n >= N) continue;
       float v = acc[i][j] + (bias ? bias[n] : 0.f);
-      if (act == GEMM_ACT_GELU_TANH) v = gelu_tanh_exact(v);
-      if (act == GEMM_ACT_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f) * (scale_out ? scale_out[t] : 1.f);
-      if (act == GEMM_ACT_SIGMOID_GATE)
+      const int act_n = n < N - act_skip ? act : GEMM_ACT_NONE;
+      if (act_n == GEMM_ACT_GELU_TANH) v = gelu_tanh_exact(v);
+      if (act_n == GEMM_ACT_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f) * (scale_out ? scale_out[t] : 1.f);
+      if (act_n == GEMM_ACT_SIGMOID_GATE)
         v = v / (1.f + expf(-gate[t * gate_row + (long long)blockIdx.z * gate_batch + n]));
       out[t * out_row + (long long)blockIdx.z * out_batch + n] = v;
     }
@@ -838,17 +841,17 @@ extern "C" int b200_gemm_f32_ex(const void* x, const void* w, const void* bias, 
                                 long long T, int N, int K, int batch, long long x_row_stride,
                                 long long x_batch_stride, long long w_row_stride, long long w_batch_stride,
                                 long long out_row_stride, long long out_batch_stride, long long gate_row_stride,
-                                long long gate_batch_stride, int act, void* stream) {
+                                long long gate_batch_stride, int act, int act_skip, void* stream) {
   using namespace b200;
   if (!x || !w || !out || T < 0 || N <= 0 || K <= 0 || batch < 1) return B200_ERR_ARG;
-  if (act < GEMM_ACT_NONE || act > GEMM_ACT_RELU2) return B200_ERR_ARG;
+  if (act < GEMM_ACT_NONE || act > GEMM_ACT_RELU2 || act_skip < 0 || act_skip > N) return B200_ERR_ARG;
   if ((act == GEMM_ACT_SIGMOID_GATE) != (gate != nullptr) || (batch > 1 && bias)) return B200_ERR_ARG;
   if (T == 0) return B200_OK;
   if ((T + 63) / 64 > 0x7fffffffLL || (N + 63) / 64 > 65535 || batch > 65535) return B200_ERR_SHAPE;
   launch_k(gemm_f32_tiled_kernel, dim3((unsigned)((T + 63) / 64), (unsigned)((N + 63) / 64), (unsigned)batch), dim3(256),
            0, (cudaStream_t)stream, (const float*)x, (const float*)w, (const float*)bias, (const float*)gate,
            (float*)out, T, N, K, x_row_stride, x_batch_stride, w_row_stride, w_batch_stride, out_row_stride,
-           out_batch_stride, gate_row_stride, gate_batch_stride, act, (const int4*)nullptr, (const int*)nullptr,
+           out_batch_stride, gate_row_stride, gate_batch_stride, act, act_skip, (const int4*)nullptr, (const int*)nullptr,
            (const float*)nullptr);
   return launch_status();
 }
@@ -887,7 +890,7 @@ extern "C" int b200_gemm_f32_from_bf16(const void* x, const void* w, void* out, 
 namespace b200 {
 // What the plain dense form can do beyond one product: an activation, a batch of products.
 struct GemmExtra {
-  int act = GEMM_ACT_NONE;
+  int act = GEMM_ACT_NONE, act_skip = 0;
   const void* gate = nullptr;
   long long gate_row_stride = 0, gate_batch_stride = 0;
   int batch = 1;
@@ -941,6 +944,7 @@ inline int gemm_dense_16bit(const void* x, const void* w, const void* bias, void
   p.w_policy = p.dense_t_tiles == 1 ? ptx::kEvictFirst : ptx::kEvictNormal;
   p.fp16 = fp16 ? 1 : 0;
   p.act = ex.act;
+  p.act_skip = ex.act_skip;
   p.gate = (const __nv_bfloat16*)ex.gate;
   p.gate_stride = ex.gate_row_stride;
   p.gate_batch_stride = ex.gate_batch_stride;
@@ -976,18 +980,19 @@ extern "C" int b200_gemm_bf16(const void* x, const void* w, const void* bias, vo
 }
 
 // The bf16 GEMM with an activation in its epilogue and / or as a batch of products (no bias then):
-//   out[g][t, n] = act(sum_k x[g][t, k] * w[g][n, k] + bias[n]),  g < batch
+//   out[g][t, n] = act(sum_k x[g][t, k] * w[g][n, k] + bias[n]),  g < batch       (n >= N - act_skip: without act)
 // A product's arithmetic is that of b200_gemm_bf16 on its slices.
 extern "C" int b200_gemm_bf16_ex(const void* x, const void* w, const void* bias, const void* gate, void* out,
                                  long long T, int N, int K, int batch, long long x_row_stride,
                                  long long x_batch_stride, long long w_row_stride, long long w_batch_stride,
                                  long long out_row_stride, long long out_batch_stride, long long gate_row_stride,
-                                 long long gate_batch_stride, int act, int out_dtype, void* stream) {
+                                 long long gate_batch_stride, int act, int act_skip, int out_dtype, void* stream) {
   using namespace b200;
-  if (batch < 1 || act < GEMM_ACT_NONE || act > GEMM_ACT_RELU2) return B200_ERR_ARG;
+  if (batch < 1 || act < GEMM_ACT_NONE || act > GEMM_ACT_RELU2 || act_skip < 0 || act_skip > N) return B200_ERR_ARG;
   if ((act == GEMM_ACT_SIGMOID_GATE) != (gate != nullptr) || (batch > 1 && bias)) return B200_ERR_ARG;
   GemmExtra ex;
   ex.act = act;
+  ex.act_skip = act_skip;
   ex.gate = gate;
   ex.gate_row_stride = gate_row_stride;
   ex.gate_batch_stride = gate_batch_stride;
@@ -1254,7 +1259,7 @@ extern "C" int b200_moe_grouped_gemm_f32(const void* x, const void* w, const voi
   launch_k(gemm_f32_tiled_kernel, dim3((unsigned)max_tiles, (unsigned)((n_out + 63) / 64), 1u), dim3(256), 0,
            (cudaStream_t)stream, (const float*)x, (const float*)w, (const float*)nullptr, (const float*)nullptr,
            (float*)out, x_rows, n_out, K, (long long)K, 0LL, (long long)K, (long long)n_out * K, (long long)n_out, 0LL, 0LL,
-           0LL, act, (const int4*)tile_table, (const int*)tile_count, (const float*)scale_out_f32);
+           0LL, act, 0, (const int4*)tile_table, (const int*)tile_count, (const float*)scale_out_f32);
   return launch_status();
 }
 

@@ -14,7 +14,7 @@
 //                         packed rows (what the expanded form of long prompts projects up).
 //
 // A window of w tokens (0: none) means that position i sees the keys i - w + 1 .. i.  The CUDA-core kernel also takes the
-// chunks, capped scores, sinks and gates of attn_extras.cuh.
+// kept tokens, chunks, capped scores, sinks, gates and sigmoid weights of attn_extras.cuh.
 #pragma once
 #include "attn_extras.cuh"
 #include "hyper.cuh"   // load4 / store4 / to_f32 / from_f32
@@ -160,6 +160,7 @@ struct LatentSeqs {
   int min_len, max_len;         // only sequences whose step brings min_len .. max_len tokens
   int window;                   // tokens a position sees, its own included; 0: every earlier one
   int chunk;                    // tokens of a chunk beyond which nothing is seen; 0: none
+  int keep;                     // first tokens seen from everywhere behind them, whatever the window or chunk
 };
 
 // First position a query at `pos` sees.
@@ -192,8 +193,8 @@ struct AttnSimtParams {
   const void* q;       // [T, H, DK]
   const void* k;       // [num_blocks * page_size, k_row]; a head's key starts at (h / group) * DK
   const void* v;       // [num_blocks * page_size, v_row]; a head's value starts at (h / group) * DV
-  void* out;           // [T, H, DV]
-  long long q_row;     // elements between tokens of q
+  void* out;           // rows of [H, DV]
+  long long q_row, out_row;   // elements between tokens of q, of out
   int k_row, v_row;
   int heads, group, DK, DV;
   float scale;
@@ -220,7 +221,10 @@ __global__ void __launch_bounds__(LATENT_SIMT_THREADS) attn_simt_kernel(const At
   const int t0 = p.seqs.query_start_loc[s], len = p.seqs.query_start_loc[s + 1] - t0;
   if (t < t0 || t >= t0 + len || len < p.seqs.min_len || len > p.seqs.max_len) return;
   const int pos = p.seqs.context_lens[s] - len + (int)(t - t0);
-  const int keys = pos + 1, kv_head = h / p.group;   // visible keys: positions first_visible .. own
+  const int keys = pos + 1, kv_head = h / p.group;   // visible keys: the kept ones, and positions first .. own
+  const int first = first_visible(p.seqs.window, p.seqs.chunk, pos), kept = min(p.seqs.keep, first);
+  const bool sigmoid = p.extras.sigmoid_bias != nullptr;
+  const float bias = sigmoid ? p.extras.sigmoid_bias[h] : 0.f;
   const T* q = reinterpret_cast<const T*>(p.q) + t * p.q_row + (long long)h * p.DK;
   for (int i = tid; i < p.DK; i += LATENT_SIMT_THREADS) lat_smem[i] = to_f32(q[i]) * p.scale;
   float acc[LATENT_SIMT_VPT];
@@ -229,8 +233,8 @@ __global__ void __launch_bounds__(LATENT_SIMT_THREADS) attn_simt_kernel(const At
   float m = -INFINITY, l = 0.f;
   const T* kbase = reinterpret_cast<const T*>(p.k) + kv_head * p.DK;
   const T* vbase = reinterpret_cast<const T*>(p.v) + kv_head * p.DV;
-  for (int b = first_visible(p.seqs.window, p.seqs.chunk, pos); b < keys; b += LATENT_SIMT_THREADS) {
-    const int n = min(LATENT_SIMT_THREADS, keys - b);
+  for (int b = kept > 0 ? 0 : first, n; b < keys; b = b < kept && b + n == kept ? first : b + n) {
+    n = min(LATENT_SIMT_THREADS, (b < kept ? kept : keys) - b);
     __syncthreads();
     long long row = tid < n ? latent_key_row(p.seqs, s, b + tid) : -1;
     s_row[tid] = row;
@@ -246,12 +250,17 @@ __global__ void __launch_bounds__(LATENT_SIMT_THREADS) attn_simt_kernel(const At
       }
       sc = p.extras.cap.cap > 0.f ? p.extras.cap.cap * tanhf(a / p.extras.cap.cap) : a;
     }
-    const float bm = fmaxf(m, block_max(sc, red));
-    const float e = sc == -INFINITY ? 0.f : expf(sc - bm);
-    s_p[tid] = e;
-    const float alpha = m == -INFINITY ? 0.f : expf(m - bm);
-    l = l * alpha + block_sum(e, red);
-    m = bm;
+    float alpha = 1.f;
+    if (sigmoid) {
+      s_p[tid] = sc == -INFINITY ? 0.f : 1.f / (1.f + expf(-(sc + bias)));
+    } else {
+      const float bm = fmaxf(m, block_max(sc, red));
+      const float e = sc == -INFINITY ? 0.f : expf(sc - bm);
+      s_p[tid] = e;
+      alpha = m == -INFINITY ? 0.f : expf(m - bm);
+      l = l * alpha + block_sum(e, red);
+      m = bm;
+    }
     __syncthreads();
 #pragma unroll
     for (int v = 0; v < LATENT_SIMT_VPT; ++v) {
@@ -266,12 +275,13 @@ __global__ void __launch_bounds__(LATENT_SIMT_THREADS) attn_simt_kernel(const At
   }
   if (p.extras.sink) l += expf(p.extras.sink[h] - m);
   const T* gate = p.extras.gate ? reinterpret_cast<const T*>(p.extras.gate) + t * p.extras.gate_stride : nullptr;
-  T* out = reinterpret_cast<T*>(p.out) + (t * p.heads + h) * (long long)p.DV;
+  T* out = reinterpret_cast<T*>(p.out) + t * p.out_row + (long long)h * p.DV;
 #pragma unroll
   for (int v = 0; v < LATENT_SIMT_VPT; ++v) {
     const int c = v * LATENT_SIMT_THREADS + tid;
     if (c >= p.DV) continue;
-    float o = l > 0.f ? acc[v] / l : 0.f;
+    float o = sigmoid ? acc[v] : l > 0.f ? acc[v] / l : 0.f;
+    o *= p.extras.out_scale;
     if (gate) o *= gate_sigmoid<T>(gate[p.extras.gate_mode == GATE_HEAD ? h : h * p.DV + c]);
     out[c] = from_f32<T>(o);
   }
@@ -309,7 +319,7 @@ extern "C" int b200_latent_prep(void* q, long long q_row_stride, const void* kv,
                                 int R, int r_true, int rot_dims, int rot_half, float eps, long long num_slots, int dtype,
                                 void* stream) {
   using namespace b200;
-  if ((!q && !kv && !q_latent) || !positions_i64 || !slot_mapping_i32 || !inv_freq_f32 || (kv && (!c_norm_f32 || !cache)) ||
+  if ((!q && !kv && !q_latent) || !positions_i64 || !slot_mapping_i32 || (rot_dims > 0 && !inv_freq_f32) || (kv && (!c_norm_f32 || !cache)) ||
       (q_latent && (!q_norm_f32 || QL <= 0 || ql_true <= 0 || ql_true > QL)) || (q_lat && !q) || T < 0 || heads <= 0 ||
       DN < 0 || DR < 0 || R <= 0 || r_true <= 0 || r_true > R || rot_dims < 0 || rot_dims > DR || (dtype != 0 && dtype != 1))
     return B200_ERR_ARG;
@@ -337,7 +347,7 @@ inline bool latent_seqs_ok(const LatentSeqs& q) {
 namespace b200 {
 inline int attn_simt_launch(AttnSimtParams& p, long long T, int dtype, cudaStream_t st) {
   if (!latent_seqs_ok(p.seqs) || !p.q || !p.k || !p.v || !p.out || T < 0 || p.heads <= 0 || p.group <= 0 || p.DK <= 0 ||
-      p.DV <= 0 || p.seqs.window < 0 || p.seqs.chunk < 0 || !attn_extras_ok(p.extras) || (dtype != 0 && dtype != 1))
+      p.DV <= 0 || p.seqs.window < 0 || p.seqs.chunk < 0 || p.seqs.keep < 0 || !attn_extras_ok(p.extras) || (dtype != 0 && dtype != 1))
     return B200_ERR_ARG;
   if (p.heads % p.group || p.DK % 8 || p.DV % 8 || p.k_row % 8 || p.v_row % 8 || p.heads > 65535 ||
       p.DV > LATENT_SIMT_THREADS * LATENT_SIMT_VPT || p.DK > 8192 || T > 0x7fffffffLL)
@@ -360,24 +370,28 @@ extern "C" int b200_latent_attn_simt(const void* q_lat, const void* cache, void*
   if (R <= 0 || DR < 0 || R % 8 || DR % 8) return B200_ERR_ARG;
   AttnSimtParams p{{(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride,
                     max_pages, page_size, num_blocks, num_seqs, min_len, max_len, window},
-                   q_lat, cache, cache, out, (long long)heads * (R + DR), R + DR, R + DR, heads, heads, R + DR, R, scale};
+                   q_lat, cache, cache, out, (long long)heads * (R + DR), (long long)heads * R, R + DR, R + DR, heads, heads,
+                   R + DR, R, scale, {{}, nullptr, nullptr, 0, GATE_NONE, nullptr, 1.f}};
   return attn_simt_launch(p, T, dtype, (cudaStream_t)stream);
 }
 
 // Grouped-query attention over paged per-head keys and values (the window_attn kernels' cross-check and fp32 form).
 extern "C" int b200_window_attn_simt(const void* q, long long q_row_stride, const void* k_cache, const void* v_cache,
-                                     void* out, const void* query_start_loc, const void* context_lens,
-                                     const void* page_table, long long page_table_stride, int max_pages, int page_size,
-                                     int num_blocks, int num_seqs, int min_len, int max_len, int window, int chunk,
-                                     float cap, const void* sink_f32, const void* gate, long long gate_row_stride,
-                                     int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float scale,
+                                     void* out, long long out_row_stride, const void* query_start_loc,
+                                     const void* context_lens, const void* page_table, long long page_table_stride,
+                                     int max_pages, int page_size, int num_blocks, int num_seqs, int min_len, int max_len,
+                                     int window, int chunk, int keep, float cap, const void* sink_f32,
+                                     const void* sigmoid_bias_f32, float out_scale, const void* gate,
+                                     long long gate_row_stride, int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float scale,
                                      int dtype, void* stream) {
   using namespace b200;
   if (kv_heads <= 0 || heads % kv_heads) return B200_ERR_ARG;
   AttnSimtParams p{{(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride,
-                    max_pages, page_size, num_blocks, num_seqs, min_len, max_len, window, chunk},
-                   q, k_cache, v_cache, out, q_row_stride, kv_heads * DK, kv_heads * DV, heads, heads / kv_heads, DK, DV,
-                   scale, {score_cap(cap), (const float*)sink_f32, gate, gate_row_stride, gate_mode}};
+                    max_pages, page_size, num_blocks, num_seqs, min_len, max_len, window, chunk, keep},
+                   q, k_cache, v_cache, out, q_row_stride, out_row_stride, kv_heads * DK, kv_heads * DV, heads, heads / kv_heads, DK, DV,
+                   scale,
+                   {score_cap(cap), (const float*)sink_f32, gate, gate_row_stride, gate_mode, (const float*)sigmoid_bias_f32,
+                    out_scale}};
   return attn_simt_launch(p, T, dtype, (cudaStream_t)stream);
 }
 

@@ -7,8 +7,8 @@
 //   paged heads        k and v rows of a paged cache, [G * DN] and [G * DV] (DR = 0)
 //
 //   q         [T, q_stride]: per head DN unrotated, then DR rotated columns; head h uses key / value head h / group
-//   out[t, h] = sum_j softmax(scale q.k_j) v_j, times the sigmoid of a gate per column, if any; EXTRAS: with the chunks, cap,
-//               sink and gate of attn_extras.cuh
+//   out[t, h] = sum_j softmax(scale q.k_j) v_j, times the sigmoid of a gate per column, if any; FORM: with
+//               the kept tokens, chunks, cap, sink, gate or sigmoid weights of attn_extras.cuh
 //
 // One CTA per (128 MT queries, head, sequence); warp w of 8 owns query rows 16 MT w .. 16 MT (w + 1) - 1 (MT = 2 for long
 // portions: every key and value fragment read from shared memory then serves two products); 64 keys per block, double
@@ -47,10 +47,11 @@ struct LexLayout {
   static constexpr int BYTES = Q + 2 * (K + V);
 };
 
-template <int DK, int DV, int MT, bool PAGED, bool EXTRAS>
+template <int DK, int DV, int MT, bool PAGED, int FORM>
 __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const LatentExpandParams p) {
   using L = LexLayout<DK, DV, MT>;
   constexpr int LEX_BM = L::BM, NS = LEX_SUB / 8;
+  constexpr bool EXTRAS = FORM != ATTN_PLAIN, SIGMOID = FORM == ATTN_SIGMOID;
   extern __shared__ __align__(16) uint8_t lex_smem[];
   pdl_trigger();
   pdl_wait();
@@ -61,6 +62,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   const int row_base = (tiles - 1 - (int)blockIdx.x) * LEX_BM;
   const int keys = p.seqs.context_lens[seq], past = keys - len;
   const int window = p.seqs.window > 0 ? p.seqs.window : 0x3fffffff, chunk = EXTRAS ? p.seqs.chunk : 0;
+  const int keep = EXTRAS ? p.seqs.keep : 0;
   const int key_base = PAGED ? 0 : p.key_base[i];
   const long long key0 = PAGED ? 0 : p.key_start[i] - key_base;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
@@ -69,7 +71,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   const int rows = min(LEX_BM, len - row_base);
   const int last_key = min(keys, past + row_base + rows);       // keys any row of the tile sees
   const int first_key = first_visible(window, chunk, past + row_base);
-  const int block0 = first_key / LEX_BN, blocks = (last_key + LEX_BN - 1) / LEX_BN;
+  const KeyBlocks walk = key_blocks<LEX_BN>(window, chunk, keep, past + row_base, last_key - 1);
 
   for (int e = tid; e < LEX_BM * (DK / 8); e += LEX_THREADS) {
     const int r = e / (DK / 8), v = e % (DK / 8);
@@ -78,7 +80,9 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
                p.q + (long long)(t0 + row_base + (in ? r : 0)) * p.q_stride + (long long)h * (p.DN + p.DR) + (in ? v * 8 : 0),
                in);
   }
-  auto seen = [&](int j) { return (uint32_t)(j - first_key) < (uint32_t)(last_key - first_key); };   // by some row of the tile
+  auto seen = [&](int j) {      // by some row of the tile
+    return (uint32_t)(j - first_key) < (uint32_t)(last_key - first_key) || (EXTRAS && j < min(keep, last_key));
+  };
   // source row of key j; a key that is not wanted (or whose page is bad) names some readable row
   auto row_of = [&](int j, bool& in) -> long long {
     if constexpr (PAGED) {
@@ -89,9 +93,9 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
       return key0 + (in ? j : first_key);
     }
   };
-  auto load = [&](int b) {
+  auto load = [&](int b) {      // block b of the walk
     const uint32_t k = smem + L::Q + (b & 1) * (L::K + L::V), vt = k + L::K;
-    const int base = b * LEX_BN;
+    const int base = walk.at(b) * LEX_BN;
     for (int e = tid; e < LEX_BN * (DK / 8); e += LEX_THREADS) {
       const int r = e / (DK / 8), col = (e % (DK / 8)) * 8;
       bool in = seen(base + r) && col < p.DN + p.DR;
@@ -108,7 +112,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
     }
     cp_async_commit();
   };
-  load(block0);
+  load(0);
 
   float o[MT][DV / 8][4];
 #pragma unroll
@@ -133,8 +137,10 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
 #pragma unroll
       for (int e = 0; e < 2; ++e) reach[t][e] = visible_keys(window, chunk, first_pos + 16 * t + g4 + 8 * e);
   }
-  for (int b = block0; b < blocks; ++b) {
-    if (b + 1 < blocks) {
+  float bias = 0.f;                                              // of sigmoid weights, in units of log2
+  if constexpr (SIGMOID) bias = p.extras.sigmoid_bias[h] * kLog2e;
+  for (int b = 0; b < walk.count; ++b) {
+    if (b + 1 < walk.count) {
       load(b + 1);
       cp_async_wait<1>();
     } else {
@@ -144,9 +150,9 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
     const uint32_t sk = smem + L::Q + (b & 1) * (L::K + L::V), sv = sk + L::K;
 #pragma unroll 1
     for (int sub = 0; sub < LEX_BN / LEX_SUB; ++sub) {
-      const int base = b * LEX_BN + sub * LEX_SUB;
+      const int base = walk.at(b) * LEX_BN + sub * LEX_SUB;
       if (r0 >= rows || base > first_pos + 16 * MT - 1) break;   // no row of this warp sees these keys
-      if (base + LEX_SUB - 1 < warp_first) continue;             // nor these, before every row's window or chunk
+      if (base + LEX_SUB - 1 < warp_first && base >= keep) continue;   // nor these, before every row's window or chunk
       float s[MT][NS][4];
 #pragma unroll
       for (int t = 0; t < MT; ++t)
@@ -181,13 +187,27 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
             if (p.extras.cap.cap > 0.f) cap_scores(s[t][j], p.extras.cap);
           }
         }
+        if constexpr (SIGMOID) {
+#pragma unroll
+          for (int j = 0; j < NS; ++j) {
+#pragma unroll
+            for (int e = 0; e < 4; e += 2) {
+              const int key = base + 8 * j + 2 * t4, pos = pos0 + 4 * e;
+              float a = s[t][j][e] + bias, b = s[t][j][e + 1] + bias;
+              sigmoid_pair(a, b, !edge || key_visible(reach[t][e >> 1], keep, pos, key),
+                           !edge || key_visible(reach[t][e >> 1], keep, pos, key + 1));
+              s[t][j][e] = a;
+              s[t][j][e + 1] = b;
+            }
+          }
+        } else {
 #pragma unroll
         for (int j = 0; j < NS; ++j)
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             float v = s[t][j][e];
             const uint32_t seen = EXTRAS ? reach[EXTRAS ? t : 0][e >> 1] : (uint32_t)window;   // 0 <= position - key < seen
-            if (edge && (uint32_t)(pos0 + 8 * (e >> 1) - (base + 8 * j + 2 * t4 + (e & 1))) >= seen) v = -INFINITY;
+            if (edge && !key_visible(seen, keep, pos0 + 8 * (e >> 1), base + 8 * j + 2 * t4 + (e & 1))) v = -INFINITY;
             s[t][j][e] = v;
             mb[e >> 1] = fmaxf(mb[e >> 1], v);
           }
@@ -217,6 +237,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
             o[t][j][2] *= alpha[1];
             o[t][j][3] *= alpha[1];
           }
+        }
         }
       }
 #pragma unroll
@@ -254,9 +275,12 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
   for (int tt = 0; tt < MT; ++tt)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      float sum = abm_quad_sum(l[tt][e]);
-      if (EXTRAS) sum += sink_term(p.extras, h, m[tt][e]);
-      float inv = 1.f / sum;
+      float inv = EXTRAS ? p.extras.out_scale : 1.f;
+      if constexpr (!SIGMOID) {
+        float sum = abm_quad_sum(l[tt][e]);
+        if (EXTRAS) sum += sink_term(p.extras, h, m[tt][e]);
+        inv /= sum;
+      }
       const int r = r0 + 16 * tt + g4 + 8 * e;
       if (r >= rows) continue;
       const long long t = t0 + row_base + r;
@@ -279,29 +303,29 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
     }
 }
 
-template <int DK, int DV, int MT, bool PAGED, bool EXTRAS>
+template <int DK, int DV, int MT, bool PAGED, int FORM>
 inline int latent_expand_launch(const LatentExpandParams& p, int max_len, int n, cudaStream_t st) {
   constexpr int smem = LexLayout<DK, DV, MT>::BYTES, LEX_BM = LexLayout<DK, DV, MT>::BM;
   static_assert(smem <= 227 * 1024, "shared memory budget");
   static PerDeviceFlags attr_set;
-  if (int rc = set_max_dyn_smem_once(attr_set, latent_expand_kernel<DK, DV, MT, PAGED, EXTRAS>, smem)) return rc;
-  launch_k(latent_expand_kernel<DK, DV, MT, PAGED, EXTRAS>,
+  if (int rc = set_max_dyn_smem_once(attr_set, latent_expand_kernel<DK, DV, MT, PAGED, FORM>, smem)) return rc;
+  launch_k(latent_expand_kernel<DK, DV, MT, PAGED, FORM>,
            dim3((unsigned)((max_len + LEX_BM - 1) / LEX_BM), (unsigned)p.heads, (unsigned)n), dim3(LEX_THREADS), (size_t)smem,
            st, p);
   return launch_status();
 }
 
-template <bool PAGED, bool EXTRAS>
+template <bool PAGED, int FORM>
 inline int latent_expand_dispatch(const LatentExpandParams& p, int max_len, int n, cudaStream_t st) {
   const int dk = p.DN + p.DR;
   const bool two = max_len > 128;
   if (dk <= 64 && p.DV <= 64)
-    return two ? latent_expand_launch<64, 64, 2, PAGED, EXTRAS>(p, max_len, n, st) : latent_expand_launch<64, 64, 1, PAGED, EXTRAS>(p, max_len, n, st);
+    return two ? latent_expand_launch<64, 64, 2, PAGED, FORM>(p, max_len, n, st) : latent_expand_launch<64, 64, 1, PAGED, FORM>(p, max_len, n, st);
   if (dk <= 128 && p.DV <= 128)
-    return two ? latent_expand_launch<128, 128, 2, PAGED, EXTRAS>(p, max_len, n, st) : latent_expand_launch<128, 128, 1, PAGED, EXTRAS>(p, max_len, n, st);
+    return two ? latent_expand_launch<128, 128, 2, PAGED, FORM>(p, max_len, n, st) : latent_expand_launch<128, 128, 1, PAGED, FORM>(p, max_len, n, st);
   if (dk <= 192 && p.DV <= 128)
-    return two ? latent_expand_launch<192, 128, 2, PAGED, EXTRAS>(p, max_len, n, st) : latent_expand_launch<192, 128, 1, PAGED, EXTRAS>(p, max_len, n, st);
-  return latent_expand_launch<256, 256, 1, PAGED, EXTRAS>(p, max_len, n, st);
+    return two ? latent_expand_launch<192, 128, 2, PAGED, FORM>(p, max_len, n, st) : latent_expand_launch<192, 128, 1, PAGED, FORM>(p, max_len, n, st);
+  return latent_expand_launch<256, 256, 1, PAGED, FORM>(p, max_len, n, st);
 }
 
 }  // namespace b200
@@ -337,7 +361,7 @@ extern "C" int b200_latent_attn_expanded(const void* q, long long q_row_stride, 
   p.q_stride = q_row_stride;
   p.k_stride = p.v_stride = kv_row_stride;
   p.rot_stride = lat_row_stride;
-  p.extras = {{}, nullptr, gate, gate_row_stride, gate ? GATE_COLUMN : GATE_NONE};
+  p.extras = {{}, nullptr, gate, gate_row_stride, gate ? GATE_COLUMN : GATE_NONE, nullptr, 1.f};
   p.out_stride = out_row_stride;
   p.heads = heads;
   p.group = 1;
@@ -345,5 +369,5 @@ extern "C" int b200_latent_attn_expanded(const void* q, long long q_row_stride, 
   p.DR = DR;
   p.DV = DV;
   p.scale_log2 = scale * kLog2e;
-  return latent_expand_dispatch<false, false>(p, max_len, n, (cudaStream_t)stream);
+  return latent_expand_dispatch<false, ATTN_PLAIN>(p, max_len, n, (cudaStream_t)stream);
 }

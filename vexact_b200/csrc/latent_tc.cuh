@@ -305,7 +305,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
           t = ltc_item(p, raw_next);
           row_next = row_of(t, 0);
         }
-        {
+        if (RB > 0) {
           const int s = rc % NR;
           ok = ptx::mbar_wait_warp(rempty(s), ((rc / NR) & 1) ^ 1, abort_flag, 700 + s);
           if (!ok) break;
@@ -349,7 +349,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
         const int qb = it & 1, b = gs & 1, rs = NR == 2 ? gs & 1 : 0;
         if (j == 0 && !ptx::mbar_wait(qfull(qb), (it >> 1) & 1, abort_flag, 720 + qb)) return false;
         if (!ptx::mbar_wait(sfree(b), ((gs >> 1) & 1) ^ 1, abort_flag, 722 + b)) return false;
-        if (!ptx::mbar_wait(rfull(rs), (NR == 2 ? gs >> 1 : gs) & 1, abort_flag, 724 + rs)) return false;
+        if (RB > 0 && !ptx::mbar_wait(rfull(rs), (NR == 2 ? gs >> 1 : gs) & 1, abort_flag, 724 + rs)) return false;
         ptx::tc_fence_after();
         const uint32_t q0 = base + q_off + qb * q_bytes, d = tm_s + b * NC;
         // one 64-column box of the contraction; descriptors step by 32 bytes (2 units) per 16 columns
@@ -367,13 +367,13 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tm, const LatentTcParams p)
         };
         for (int r = 0; r < RB; ++r)
           box(base + rot_off + (uint32_t)(rs * RB + r) * LTC_BOX, r, min(64, DR - 64 * r), r != 0 ? 1u : 0u);
-        ptx::umma_commit(rempty(rs));
+        if (RB > 0) ptx::umma_commit(rempty(rs));
 #pragma unroll
         for (int i = 0; i < CP; ++i) {
           if (!ptx::mbar_wait(pfull(ss), sph, abort_flag, 730 + ss)) return false;
           ptx::tc_fence_after();
           const uint32_t a = base + (uint32_t)(2 * ss) * LTC_BOX;
-          box(a, RB + 2 * i, min(64, R - 128 * i), 1u);
+          box(a, RB + 2 * i, min(64, R - 128 * i), i != 0 || RB > 0 ? 1u : 0u);
           if (2 * i + 1 < CB) box(a + LTC_BOX, RB + 2 * i + 1, min(64, R - 128 * i - 64), 1u);
           if (++ss == NP) {
             ss = 0;
@@ -640,7 +640,7 @@ extern "C" int b200_latent_plan(const void* query_start_loc, const void* context
 }
 
 // b200_latent_attn_simt on tensor cores (bf16) for the sequences of a plan; min_len / max_len as the plan was made with.
-// R <= 512, DR <= 128, multiples of 8; page_size a power of two of at least 8, or a multiple of 128.
+// R <= 512, DR <= 128 (0: no rotated part), multiples of 8; page_size a power of two of at least 8, or a multiple of 128.
 // part_o [max_items, 16, R] and part_ml [max_items, 16, 2] fp32: scratch, NULL when no sequence has several splits (of 512
 // keys, at multiples of 512).
 extern "C" int b200_latent_attn_tc(const void* q_lat, const void* cache, void* out, const void* query_start_loc,
@@ -654,7 +654,7 @@ extern "C" int b200_latent_attn_tc(const void* q_lat, const void* cache, void* o
   p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
             page_size, num_blocks, num_seqs, min_len, max_len, window};
   if (!latent_seqs_ok(p.seqs) || window < 0 || !q_lat || !cache || !out || !items || !item_count || !first_item || T < 0 || heads <= 0 ||
-      R <= 0 || DR <= 0 || max_items <= 0 || (part_o != nullptr) != (part_ml != nullptr))
+      R <= 0 || DR < 0 || max_items <= 0 || (part_o != nullptr) != (part_ml != nullptr))
     return B200_ERR_ARG;
   const bool pages_ok = page_size % LTC_BN == 0 || (page_size >= 8 && LTC_BN % page_size == 0);
   if (R % 8 || DR % 8 || R > 512 || DR > 128 || !pages_ok || T > 0x7fffffffLL || heads > 65535) return B200_ERR_SHAPE;

@@ -22,6 +22,7 @@
 #include "latent_expand.cuh"
 #include "latent_tc.cuh"
 #include "window_attn.cuh"
+#include "gru.cuh"
 #include "attn_prep.cuh"
 
 // Self-test of the bounded wait every kernel here relies on: one CTA waits, with a limit of
@@ -69,7 +70,7 @@ extern "C" int b200_status_read(int* host_out4, void* stream) {
 }
 
 // Bumped whenever an exported signature changes.
-extern "C" int b200_abi_version(void) { return 7; }
+extern "C" int b200_abi_version(void) { return 8; }
 
 // Hash of the sources and compiler flags this binary was built from (set by the build script);
 // the loader compares it with the sources beside it and refuses a stale library.

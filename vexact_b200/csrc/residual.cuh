@@ -10,6 +10,9 @@
 // One CTA per token, everything in registers between the two reductions.  `rows` picks tokens at the end of a model;
 // nothing is written back then.
 //
+// Without `post` (PRE) the sublayer's result is not normed, and may be multiplied column by column by a gate of the token:
+//     x  <- x + y * sigmoid(gate + gate_bias) (+ add)       (start of the model: x = the embedding row)
+//
 // The norms may be dynamic tanh instead, tanh(alpha x) * w + b with one number alpha, which reduces nothing:
 //     x <- x + tanh(post_alpha y) * post + post_bias (+ add),    xn = tanh(norm_alpha x) * norm + norm_bias
 // A thread then owns four columns, keeps the norms' vectors in registers and walks tokens, ROWS at a time.  At the start of a model y is
@@ -49,6 +52,10 @@ struct ResidualParams {
   const float* post_bias;     // [W]
   const float* norm_bias;     // [W]
   float post_alpha, norm_alpha;
+  // gate of the sublayer's result (PRE)
+  const void* gate;           // [T, gate_stride] or null
+  long long gate_stride;
+  const float* gate_bias;     // [W] or null
 };
 
 template <typename T>
@@ -57,8 +64,9 @@ __device__ __forceinline__ void load4_tail(const T* p, int left, float (&v)[4]) 
   for (int k = 0; k < 4; ++k) v[k] = k < left ? to_f32(p[k]) : 0.f;
 }
 
-// CH: register chunks of four columns per thread (W <= threads * CH * 4); MAXT: threads at most; PICK: y is expert-sorted.
-template <typename T, int CH, int MAXT, bool PICK>
+// CH: register chunks of four columns per thread (W <= threads * CH * 4); MAXT: threads at most; PICK: y is expert-sorted;
+// PRE: no norm of y.
+template <typename T, int CH, int MAXT, bool PICK, bool PRE>
 __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParams p) {
   __shared__ float red[32];
   pdl_trigger();
@@ -108,7 +116,15 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
     } else {
       get(xrow, i, x[c]);
     }
-    get(p.post, i, w[c]);
+    if constexpr (!PRE) {
+      get(p.post, i, w[c]);
+    } else if (p.gate) {          // w: the gate ahead of its sigmoid
+      get(reinterpret_cast<const T*>(p.gate) + t * p.gate_stride, i, w[c]);
+      float b[4] = {0.f, 0.f, 0.f, 0.f};
+      if (p.gate_bias) get(p.gate_bias, i, b);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) w[c][k] += b[k];
+    }
     if (p.norm_w) get(p.norm_w, i, nw[c]);
   }
   auto add_row = [&](const T* row, int i, float (&a)[4]) {
@@ -151,12 +167,17 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
       for (int k = 8; k < p.topk; ++k) one(pick[k]);
     }
     if (extra) add_row(extra, i, v[c]);
+    if constexpr (!PRE) {
 #pragma unroll
-    for (int k = 0; k < 4; ++k) ss = fmaf(v[c][k], v[c][k], ss);
+      for (int k = 0; k < 4; ++k) ss = fmaf(v[c][k], v[c][k], ss);
+    }
   }
-  ss = block_sum(ss, red);
-  const float inv_y = 1.f / sqrtf(ss / (float)W + p.eps);
-  ss = 0.f;
+  float inv_y = 1.f;
+  if constexpr (!PRE) {
+    ss = block_sum(ss, red);
+    inv_y = 1.f / sqrtf(ss / (float)W + p.eps);
+    ss = 0.f;
+  }
 #pragma unroll
   for (int c = 0; c < CH; ++c) {
     const int i = (c * blockDim.x + threadIdx.x) * 4;
@@ -165,7 +186,12 @@ __global__ void __launch_bounds__(MAXT) residual_step_kernel(const ResidualParam
     if (p.add) get(p.add, i, a);
 #pragma unroll
     for (int k = 0; k < 4; ++k) {
-      x[c][k] = x[c][k] + v[c][k] * inv_y * w[c][k] + a[k];
+      if constexpr (PRE) {
+        const float s = !p.gate ? 1.f : sizeof(T) == 2 ? sigmoid_fast(w[c][k]) : 1.f / (1.f + expf(-w[c][k]));
+        x[c][k] = x[c][k] + v[c][k] * s + a[k];
+      } else {
+        x[c][k] = x[c][k] + v[c][k] * inv_y * w[c][k] + a[k];
+      }
       ss = fmaf(x[c][k], x[c][k], ss);      // columns past W are zero in every term
     }
     if (p.write_back) {
@@ -347,17 +373,20 @@ inline int residual_tanh_launch(const ResidualParams& p, cudaStream_t st) {
   return launch_status();
 }
 
-template <typename T, bool PICK>
+template <typename T, bool PICK, bool PRE = false>
 inline int residual_launch(const ResidualParams& p, long long rows, cudaStream_t st) {
-  if (p.post_bias) return residual_tanh_launch<T, PICK>(p, st);
+  if constexpr (!PRE) {
+    if (!p.post) return residual_launch<T, PICK, true>(p, rows, st);
+    if (p.post_bias) return residual_tanh_launch<T, PICK>(p, st);
+  }
   const int chunks = (p.W + 3) / 4;
   const dim3 g((unsigned)rows);
   int threads = 64;
   while (threads < 256 && chunks > threads) threads <<= 1;
-  if (chunks <= threads) launch_k(residual_step_kernel<T, 1, 256, PICK>, g, dim3(threads), 0, st, p);
-  else if (chunks <= 512) launch_k(residual_step_kernel<T, 2, 256, PICK>, g, dim3(256), 0, st, p);
-  else if (chunks <= 1024) launch_k(residual_step_kernel<T, 2, 512, PICK>, g, dim3(512), 0, st, p);
-  else if (chunks <= 4096) launch_k(residual_step_kernel<T, 4, 1024, PICK>, g, dim3(1024), 0, st, p);
+  if (chunks <= threads) launch_k(residual_step_kernel<T, 1, 256, PICK, PRE>, g, dim3(threads), 0, st, p);
+  else if (chunks <= 512) launch_k(residual_step_kernel<T, 2, 256, PICK, PRE>, g, dim3(256), 0, st, p);
+  else if (chunks <= 1024) launch_k(residual_step_kernel<T, 2, 512, PICK, PRE>, g, dim3(512), 0, st, p);
+  else if (chunks <= 4096) launch_k(residual_step_kernel<T, 4, 1024, PICK, PRE>, g, dim3(1024), 0, st, p);
   else return B200_ERR_SHAPE;
   return launch_status();
 }
@@ -371,21 +400,24 @@ extern "C" int b200_residual_step(void* x_f32, const void* y, long long y_row_st
                                   long long num_tokens, long long num_rows, int W, const void* post_f32,
                                   const void* add_f32, const void* norm_w_f32, float eps, float embed_scale,
                                   const void* post_bias_f32, float post_alpha, const void* norm_bias_f32,
-                                  float norm_alpha, void* xn, long long xn_row_stride, int xn_cols, int write_back,
-                                  int dtype, void* stream) {
+                                  float norm_alpha, const void* gate, long long gate_row_stride,
+                                  const void* gate_bias_f32, void* xn, long long xn_row_stride, int xn_cols,
+                                  int write_back, int dtype, void* stream) {
   using namespace b200;
-  if (!x_f32 || !post_f32 || num_tokens < 0 || num_rows < 0 || W <= 0 || (dtype != 0 && dtype != 1)) return B200_ERR_ARG;
+  if (!x_f32 || num_tokens < 0 || num_rows < 0 || W <= 0 || (dtype != 0 && dtype != 1)) return B200_ERR_ARG;
   if ((y != nullptr) == (ids_i64 != nullptr) || (ids_i64 && (!embed || extra)) || (scatter_index_i32 && (!y || topk < 1)))
     return B200_ERR_ARG;
-  if (post_bias_f32 && norm_w_f32 && !norm_bias_f32) return B200_ERR_ARG;
+  if (post_bias_f32 && (!post_f32 || (norm_w_f32 && !norm_bias_f32))) return B200_ERR_ARG;
+  if ((gate && (post_f32 || !y)) || (gate_bias_f32 && !gate)) return B200_ERR_ARG;
   if ((norm_w_f32 && (!xn || xn_cols < W)) || (rows_i32 && write_back)) return B200_ERR_ARG;
   if (num_rows > 0x7fffffffLL) return B200_ERR_SHAPE;
   if (num_rows == 0) return B200_OK;
-  if (W % 4 == 0 && (y_row_stride % 4 || xn_row_stride % 4 || extra_row_stride % 4)) return B200_ERR_SHAPE;
+  if (W % 4 == 0 && (y_row_stride % 4 || xn_row_stride % 4 || extra_row_stride % 4 || gate_row_stride % 4)) return B200_ERR_SHAPE;
   ResidualParams p{(float*)x_f32, y, y_row_stride, y_rows, (const int*)scatter_index_i32, topk, extra, extra_row_stride,
                    embed, (const long long*)ids_i64, vocab, (const int*)rows_i32, num_tokens, (const float*)post_f32,
                    (const float*)add_f32, (const float*)norm_w_f32, eps, xn, xn_row_stride, xn_cols, W, write_back,
-                   num_rows, embed_scale, (const float*)post_bias_f32, (const float*)norm_bias_f32, post_alpha, norm_alpha};
+                   num_rows, embed_scale, (const float*)post_bias_f32, (const float*)norm_bias_f32, post_alpha, norm_alpha, gate,
+                   gate_row_stride, (const float*)gate_bias_f32};
   const cudaStream_t st = (cudaStream_t)stream;
   if (scatter_index_i32)
     return dtype == 0 ? residual_launch<__nv_bfloat16, true>(p, num_rows, st) : residual_launch<float, true>(p, num_rows, st);

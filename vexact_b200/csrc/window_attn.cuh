@@ -1,6 +1,6 @@
 // Grouped-query attention of decoded tokens and short portions over paged per-head keys and values (bf16), optionally
-// inside a window or chunk, with capped scores, a sink in the denominator and an output gate (attn_extras.cuh).  Scores and
-// weights are fp32: a weight enters the value product as a bf16 pair hi + lo, whose two products are summed in fp32, and the
+// inside a window or chunk, with capped scores, a sink in the denominator, an output gate or sigmoid weights
+// (attn_extras.cuh).  Scores and weights are fp32: a weight enters the value product as a bf16 pair hi + lo, whose two products are summed in fp32, and the
 // denominator sums the fp32 weights.  (attn.cuh and its kin round the weights to bf16, as the models they serve do.)
 //
 // One CTA of WARPS warps owns up to 8 columns of one KV head of one sequence, a column being one (token, query head)
@@ -36,12 +36,13 @@ struct WatLayout {
   static_assert(STAGES * STAGE >= DV * 8 * 4 + 64, "a warp's ring holds its partial result");
 };
 
-template <int DK, int DV, int WARPS, int STAGES, bool EXTRAS>
+template <int DK, int DV, int WARPS, int STAGES, int FORM>
 __global__ void __launch_bounds__(WARPS * 32)
 window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                    const WindowAttnParams p) {
   using L = WatLayout<DK, DV, WARPS, STAGES>;
   constexpr int KH = DK / 64, VH = DV / 64, MT = WAT_BN / 16;
+  constexpr bool EXTRAS = FORM != ATTN_PLAIN, SIGMOID = FORM == ATTN_SIGMOID;
   extern __shared__ uint8_t smem_raw[];
   __shared__ uint64_t full_bar[WARPS][STAGES];
   __shared__ int abort_mem;
@@ -68,9 +69,9 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
   auto col_q = [&](int c) { return pos0 + (col_valid(c) ? c / heads_here : 0); };   // a spare column repeats the first position
   auto col_head = [&](int c) { return kvh * p.group + hchunk * 8 + c % heads_here; };
   const int last_pos = q_abs0 + min(pos0 + p.pos_per_tile, q_len) - 1;
-  const int chunk = EXTRAS ? p.seqs.chunk : 0;
-  const int blk0 = first_visible(p.seqs.window, chunk, q_abs0 + pos0) / WAT_BN, nblk = last_pos / WAT_BN + 1 - blk0;
-  const int mine = (nblk - warp + WARPS - 1) / WARPS;      // blocks of this warp: blk0 + warp + i * WARPS
+  const int chunk = EXTRAS ? p.seqs.chunk : 0, keep = EXTRAS ? p.seqs.keep : 0;
+  const KeyBlocks walk = key_blocks<WAT_BN>(p.seqs.window, chunk, keep, q_abs0 + pos0, last_pos);
+  const int mine = (walk.count - warp + WARPS - 1) / WARPS;      // blocks of this warp: number warp + i * WARPS of the walk
 
   if (threadIdx.x == 0) {
     *abort_flag = 0;
@@ -93,7 +94,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
     if (lane == 0) ptx::mbar_expect_tx(bar, L::STAGE);
     __syncwarp();
     if (lane < boxes) {
-      const int tok = (blk0 + warp + i * WARPS) * WAT_BN + lane * p.box_tokens;
+      const int tok = walk.at(warp + i * WARPS) * WAT_BN + lane * p.box_tokens;
       const int page = tok / p.seqs.page_size, in_page = tok - page * p.seqs.page_size;
       int phys = -1;                // out of range: zeros arrive
       if (tok < kv_len && page < p.seqs.max_pages) phys = p.seqs.page_table[(long long)seq * p.seqs.page_table_stride + page];
@@ -123,10 +124,12 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
   }
   int cpos[2];
   uint32_t reach[2];                // visible: 0 <= cpos - key < reach
+  float bias[2];                    // of sigmoid weights, in units of log2
 #pragma unroll
   for (int j = 0; j < 2; ++j) {
     cpos[j] = q_abs0 + col_q(2 * t + j);
     reach[j] = visible_keys(p.seqs.window, chunk, cpos[j]);
+    bias[j] = SIGMOID ? p.extras.sigmoid_bias[col_head(2 * t + j)] * kLog2e : 0.f;
   }
 
   float o[DV / 16][4];
@@ -141,7 +144,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
     ok = __all_sync(0xffffffffu, ok);
     if (!ok) break;
     const uint32_t sk = ring + (uint32_t)s * L::STAGE, sv = sk + L::K;
-    const int key0 = (blk0 + warp + i * WARPS) * WAT_BN;
+    const int key0 = walk.at(warp + i * WARPS) * WAT_BN;
     if (key0 + WAT_BN > kv_len) {   // rows past the context may hold anything: 0 * value has to stay 0
       uint8_t* vt = ring_ptr + (size_t)s * L::STAGE + L::K;
       for (int r = kv_len - key0; r < WAT_BN; ++r)
@@ -168,6 +171,18 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
       for (int e = 0; e < 4; ++e) sc[mt][e] *= p.scale_log2;
       if (EXTRAS && p.extras.cap.cap > 0.f) cap_scores(sc[mt], p.extras.cap);
     }
+    if constexpr (SIGMOID) {
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const int key = key0 + mt * 16 + g;
+          float a = sc[mt][j] + bias[j], b = sc[mt][2 + j] + bias[j];
+          sigmoid_pair(a, b, key_visible(reach[j], keep, cpos[j], key), key_visible(reach[j], keep, cpos[j], key + 8));
+          sc[mt][j] = a;
+          sc[mt][2 + j] = b;
+        }
+    } else {
     float alpha[2];
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
@@ -178,7 +193,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
         for (int hh = 0; hh < 2; ++hh) {
           const int key = key0 + mt * 16 + g + hh * 8;
           float v = sc[mt][hh * 2 + j];
-          if ((uint32_t)(cpos[j] - key) >= reach[j]) v = -INFINITY;
+          if (!key_visible(reach[j], keep, cpos[j], key)) v = -INFINITY;
           sc[mt][hh * 2 + j] = v;
           mx = fmaxf(mx, v);
         }
@@ -206,6 +221,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
         o[d][2] *= alpha[0];
         o[d][3] *= alpha[1];
       }
+    }
     }
     uint32_t hi[MT][2], lo[MT][2];
 #pragma unroll
@@ -275,7 +291,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
 #pragma unroll
     for (int w = 0; w < WARPS; ++w) {
       const float* q = parts + w * PITCH;
-      const float f = fast_exp2(q[DV * 8 + c] - m);
+      const float f = SIGMOID ? 1.f : fast_exp2(q[DV * 8 + c] - m);
       l = fmaf(f, q[DV * 8 + 8 + c], l);
       a = fmaf(f, q[d * 8 + c], a);
       b = fmaf(f, q[(d + 1) * 8 + c], b);
@@ -283,7 +299,7 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
     const int head = col_head(c);
     const long long row = q_start + col_q(c);
     if (EXTRAS) l += sink_term(p.extras, head, m);
-    const float inv = 1.f / l;
+    const float inv = SIGMOID ? p.extras.out_scale : EXTRAS ? p.extras.out_scale / l : 1.f / l;
     a *= inv;
     b *= inv;
     if (EXTRAS && p.extras.gate_mode != GATE_NONE) {
@@ -296,24 +312,24 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
   }
 }
 
-template <int DK, int DV, int WARPS, int STAGES, bool EXTRAS>
+template <int DK, int DV, int WARPS, int STAGES, int FORM>
 inline int window_attn_launch(const CUtensorMap& tk, const CUtensorMap& tv, const WindowAttnParams& p, dim3 grid,
                               cudaStream_t st) {
   constexpr int smem = WatLayout<DK, DV, WARPS, STAGES>::BYTES;
   static_assert(smem <= 226 * 1024, "shared memory budget");
   static PerDeviceFlags attr_set;
-  if (int rc = set_max_dyn_smem_once(attr_set, window_attn_kernel<DK, DV, WARPS, STAGES, EXTRAS>, smem)) return rc;
-  launch_k(window_attn_kernel<DK, DV, WARPS, STAGES, EXTRAS>, grid, dim3(WARPS * 32), (size_t)smem, st, tk, tv, p);
+  if (int rc = set_max_dyn_smem_once(attr_set, window_attn_kernel<DK, DV, WARPS, STAGES, FORM>, smem)) return rc;
+  launch_k(window_attn_kernel<DK, DV, WARPS, STAGES, FORM>, grid, dim3(WARPS * 32), (size_t)smem, st, tk, tv, p);
   return launch_status();
 }
 
-template <bool EXTRAS>
+template <int FORM>
 inline int window_attn_dispatch(const CUtensorMap& tk, const CUtensorMap& tv, const WindowAttnParams& p, dim3 grid,
                                 cudaStream_t st) {
-  if (p.dk <= 64 && p.dv <= 64) return window_attn_launch<64, 64, 2, 4, EXTRAS>(tk, tv, p, grid, st);
-  if (p.dk <= 128 && p.dv <= 128) return window_attn_launch<128, 128, 2, 3, EXTRAS>(tk, tv, p, grid, st);
-  if (p.dk <= 192 && p.dv <= 128) return window_attn_launch<192, 128, 2, 2, EXTRAS>(tk, tv, p, grid, st);
-  return window_attn_launch<256, 256, 2, 2, EXTRAS>(tk, tv, p, grid, st);
+  if (p.dk <= 64 && p.dv <= 64) return window_attn_launch<64, 64, 2, 4, FORM>(tk, tv, p, grid, st);
+  if (p.dk <= 128 && p.dv <= 128) return window_attn_launch<128, 128, 2, 3, FORM>(tk, tv, p, grid, st);
+  if (p.dk <= 192 && p.dv <= 128) return window_attn_launch<192, 128, 2, 2, FORM>(tk, tv, p, grid, st);
+  return window_attn_launch<256, 256, 2, 2, FORM>(tk, tv, p, grid, st);
 }
 
 }  // namespace b200
@@ -325,16 +341,18 @@ extern "C" int b200_window_attn_decode(const void* q, long long q_row_stride, co
                                        void* out, long long out_row_stride, const void* query_start_loc,
                                        const void* context_lens, const void* page_table, long long page_table_stride,
                                        int max_pages, int page_size, int num_blocks, int num_seqs, int min_len, int max_len,
-                                       int most_new, int window, int chunk, float cap, const void* sink_f32,
-                                       const void* gate, long long gate_row_stride, int gate_mode, int heads, int kv_heads,
-                                       int DK, int DV, float scale, void* stream) {
+                                       int most_new, int window, int chunk, int keep, float cap, const void* sink_f32,
+                                       const void* sigmoid_bias_f32, float out_scale, const void* gate,
+                                       long long gate_row_stride, int gate_mode, int heads, int kv_heads, int DK, int DV,
+                                       float scale, void* stream) {
   using namespace b200;
   WindowAttnParams p{};
   p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
-            page_size, num_blocks, num_seqs, min_len < 1 ? 1 : min_len, max_len, window, chunk};
-  p.extras = {score_cap(cap * kLog2e), (const float*)sink_f32, gate, gate_row_stride, gate_mode};
+            page_size, num_blocks, num_seqs, min_len < 1 ? 1 : min_len, max_len, window, chunk, keep};
+  p.extras = {score_cap(cap * kLog2e), (const float*)sink_f32, gate, gate_row_stride, gate_mode,
+              (const float*)sigmoid_bias_f32, out_scale};
   if (!latent_seqs_ok(p.seqs) || !q || !k_cache || !v_cache || !out || heads <= 0 || kv_heads <= 0 || heads % kv_heads ||
-      DK <= 0 || DV <= 0 || window < 0 || chunk < 0 || max_len < 1 || most_new < 0 || !attn_extras_ok(p.extras))
+      DK <= 0 || DV <= 0 || window < 0 || chunk < 0 || keep < 0 || max_len < 1 || most_new < 0 || !attn_extras_ok(p.extras))
     return B200_ERR_ARG;
   const bool pages_ok = page_size % 8 == 0 && (page_size % WAT_BN == 0 || WAT_BN % page_size == 0);
   if (DK % 8 || DV % 8 || DK > 256 || DV > 256 || !pages_ok || q_row_stride % 2 || out_row_stride % 2 ||
@@ -364,8 +382,11 @@ extern "C" int b200_window_attn_decode(const void* q, long long q_row_stride, co
   const dim3 grid((unsigned)((most + p.pos_per_tile - 1) / p.pos_per_tile), (unsigned)(kv_heads * p.head_chunks),
                   (unsigned)num_seqs);
   const cudaStream_t st = (cudaStream_t)stream;
-  return attn_has_extras(p.extras, chunk) ? window_attn_dispatch<true>(tk, tv, p, grid, st)
-                                          : window_attn_dispatch<false>(tk, tv, p, grid, st);
+  switch (attn_form(p.extras, chunk, keep)) {
+    case ATTN_PLAIN: return window_attn_dispatch<ATTN_PLAIN>(tk, tv, p, grid, st);
+    case ATTN_EXTRAS: return window_attn_dispatch<ATTN_EXTRAS>(tk, tv, p, grid, st);
+    default: return window_attn_dispatch<ATTN_SIGMOID>(tk, tv, p, grid, st);
+  }
 }
 
 // Long portions: the n sequences named, which are those that bring at least min_len tokens.  Heads of 65 .. 128 columns go
@@ -375,17 +396,18 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
                                         void* out, long long out_row_stride, const void* query_start_loc,
                                         const void* context_lens, const void* page_table, long long page_table_stride,
                                         int max_pages, int page_size, int num_blocks, int num_seqs, const void* seq_ids_i32,
-                                        int n, int max_len, int min_len, int window, int chunk, float cap,
-                                        const void* sink_f32, const void* gate, long long gate_row_stride, int gate_mode,
-                                        long long T, int heads, int kv_heads, int DK, int DV, float scale, int form,
+                                        int n, int max_len, int min_len, int window, int chunk, int keep,
+                                        float cap, const void* sink_f32, const void* sigmoid_bias_f32, float out_scale,
+                                        const void* gate, long long gate_row_stride, int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float scale, int form,
                                         void* stream) {
   using namespace b200;
   LatentExpandParams p{};
   p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,
-            page_size, num_blocks, num_seqs, 0, 0, window, chunk};
-  p.extras = {score_cap(cap * kLog2e), (const float*)sink_f32, gate, gate_row_stride, gate_mode};
+            page_size, num_blocks, num_seqs, 0, 0, window, chunk, keep};
+  p.extras = {score_cap(cap * kLog2e), (const float*)sink_f32, gate, gate_row_stride, gate_mode,
+              (const float*)sigmoid_bias_f32, out_scale};
   if (!latent_seqs_ok(p.seqs) || !q || !k_cache || !v_cache || !out || !seq_ids_i32 || n <= 0 || max_len <= 0 || T <= 0 ||
-      heads <= 0 || kv_heads <= 0 || heads % kv_heads || DK <= 0 || DV <= 0 || window < 0 || chunk < 0 ||
+      heads <= 0 || kv_heads <= 0 || heads % kv_heads || DK <= 0 || DV <= 0 || window < 0 || chunk < 0 || keep < 0 ||
       !attn_extras_ok(p.extras))
     return B200_ERR_ARG;
   if (gate_mode == GATE_COLUMN && (gate_row_stride % 8 || (reinterpret_cast<uintptr_t>(gate) & 15))) return B200_ERR_SHAPE;
@@ -418,6 +440,7 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
     a.qk_scale = scale * kLog2e;
     a.extras = p.extras;
     a.chunk = chunk;
+    a.keep = keep;
     a.num_blocks = num_blocks;
     a.num_seqs = num_seqs;
     a.max_seqlen_q = max_len;
@@ -443,8 +466,11 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
       CUtensorMap tg = tk;
       a.g_tma = gate_mode == GATE_COLUMN && 32 % hh == 0 &&
                 make_tmap_q(&tg, gate, T, heads, DV, gate_row_stride, DV, hh, 32 / hh, true) == B200_OK;
-      return attn_has_extras(a.extras, chunk) ? attn_rows_launch<128, true, true>(tk, tv, tq, to, tg, a, st)
-                                              : attn_rows_launch<128, true, false>(tk, tv, tq, to, tg, a, st);
+      switch (attn_form(a.extras, chunk, keep)) {
+        case ATTN_PLAIN: return attn_rows_launch<128, true, ATTN_PLAIN>(tk, tv, tq, to, tg, a, st);
+        case ATTN_EXTRAS: return attn_rows_launch<128, true, ATTN_EXTRAS>(tk, tv, tq, to, tg, a, st);
+        default: return attn_rows_launch<128, true, ATTN_SIGMOID>(tk, tv, tq, to, tg, a, st);
+      }
     }
   }
   p.seq_ids = (const int*)seq_ids_i32;
@@ -461,6 +487,9 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
   p.DN = DK;
   p.DV = DV;
   p.scale_log2 = scale * kLog2e;
-  return attn_has_extras(p.extras, chunk) ? latent_expand_dispatch<true, true>(p, max_len, n, st)
-                                          : latent_expand_dispatch<true, false>(p, max_len, n, st);
+  switch (attn_form(p.extras, chunk, keep)) {
+    case ATTN_PLAIN: return latent_expand_dispatch<true, ATTN_PLAIN>(p, max_len, n, st);
+    case ATTN_EXTRAS: return latent_expand_dispatch<true, ATTN_EXTRAS>(p, max_len, n, st);
+    default: return latent_expand_dispatch<true, ATTN_SIGMOID>(p, max_len, n, st);
+  }
 }

@@ -3,6 +3,7 @@ norm-then-gate between two projections."""
 from __future__ import annotations
 
 from dataclasses import dataclass
+from typing import Optional
 
 import torch
 
@@ -88,8 +89,10 @@ def delta_chunk_scan(w: DeltaWeights, act: torch.Tensor, dt: torch.Tensor, b: to
 
 
 def delta_mixer(w: DeltaWeights, xn: torch.Tensor, conv_state: torch.Tensor, state: torch.Tensor, step,
-                eps: float) -> torch.Tensor:
-    proj = gemm(xn, w.w_in)
+                eps: float, proj: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """proj: the projection rows of xn, where the caller has them already."""
+    if proj is None:
+        proj = gemm(xn, w.w_in)
     act, dt = short_conv(w, proj, conv_state, step)
     b = proj[:, w.dt_off + w.heads:w.dt_off + 2 * w.heads]
     o = torch.empty((xn.shape[0], w.inner), device=xn.device, dtype=xn.dtype)

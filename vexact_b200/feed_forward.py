@@ -15,13 +15,15 @@ FUSED_MAX_ROWS = 64     # rows (per group) up to which the activation rides on t
 
 @dataclass
 class MLPWeights:
-    """down(act(up x + up_b)) + down_b; the biases may be absent."""
+    """down(act(up x + up_b)) + down_b; the biases may be absent.  The last `tail` rows of `up` are no part of it: their products
+    are for whoever reads the same input."""
 
     up: torch.Tensor
     down: torch.Tensor
     up_b: Optional[torch.Tensor] = None
     down_b: Optional[torch.Tensor] = None
     act: str = "gelu_tanh"           # or "relu2": the square of relu
+    tail: int = 0
 
 
 @dataclass
@@ -33,8 +35,13 @@ class GLUWeights:
     act: str
 
 
-def mlp_forward(w: MLPWeights, x: torch.Tensor) -> torch.Tensor:
-    return gemm(gemm(x, w.up, w.up_b, act=w.act), w.down, w.down_b)
+def mlp_forward(w: MLPWeights, x: torch.Tensor):
+    """The feed-forward of rows x; with a tail, its columns as well: (rows, tail columns)."""
+    h = gemm(x, w.up, w.up_b, act=w.act, act_skip=w.tail)
+    if not w.tail:
+        return gemm(h, w.down, w.down_b)
+    F = h.shape[1] - w.tail
+    return gemm(h[:, :F], w.down, w.down_b), h[:, F:]
 
 
 def glu(gu: torch.Tensor, act: str, scale_in: Optional[torch.Tensor] = None,

@@ -1,6 +1,6 @@
 """Hybrid decoders: layers that mix recurrent and attention mixers, dense and mixture feed-forwards, hung on
 hyper-connections ("Nurazen") or on one residual with norms on both sides of a sublayer, with a looped run of layers
-("Dekerax") or with layers that share weights ("Tekilix").
+("Dekerax") or with layers that share weights ("Tekilix"), or with a norm ahead of it and a gate behind it ("Purozen").
 
 `HybridShape.from_config` reads config.json (hybrid_config.py), `HybridWeights` turns checkpoint tensors into what the
 kernels take (hybrid_weights.py), `HybridRunner` runs a packed step, and `HybridModel` is the form the `Inferencer`
@@ -18,11 +18,13 @@ from .delta import DeltaWeights, delta_mixer
 from .fused_moe import MixtureWeights, mixture_forward
 from .feed_forward import GLUWeights, MLPWeights, glu_forward, mlp_forward
 from .hybrid_config import (ARCHITECTURES, AttentionSpec, DeltaSpec, DenseSpec, HybridLayer, HybridShape, LatentSpec,  # noqa: F401
-                            LoopSpec, MixtureSpec, RotarySpec, SSMSpec, YarnSpec, random_tensors, tensor_shapes)
+                            LoopSpec, MinGRUSpec, MixtureSpec, ParallelSpec, RotarySpec, SSMSpec, YarnSpec, random_tensors,
+                            tensor_shapes)
 from .hybrid_weights import HybridLayerWeights, HybridWeights  # noqa: F401
 from .hyper import hyper_step
 from .kv_cache_context import HybridCacheStore, get_kv_cache_context
 from .latent_attention import LatentWeights, latent_mixer
+from .parallel import ParallelWeights, parallel_mixer
 from .residual import residual_step
 from .ssm import SSMWeights, ssm_mixer
 from .standalone_logprobs import lm_head_greedy
@@ -44,6 +46,7 @@ class HybridStep:
     state_slots: torch.Tensor
     page_size: int = 64
     seq_lens: Optional[list] = None      # host (new, total) tokens per sequence; None inside a captured graph
+    source_values: Optional[torch.Tensor] = None   # values of the layer that others mix into theirs, once it has run
 
 
 class HybridRunner:
@@ -52,27 +55,39 @@ class HybridRunner:
         self.shape = weights.shape
         self.store = store
 
-    def _mixer(self, run: int, mixer, xn: torch.Tensor, step: HybridStep) -> torch.Tensor:
-        st = self.store
+    def _mixer(self, run: int, mixer, xn: torch.Tensor, step: HybridStep, proj: Optional[torch.Tensor] = None) -> torch.Tensor:
+        st, eps = self.store, self.shape.eps
         if isinstance(mixer, SSMWeights):
-            return ssm_mixer(mixer, xn, st.conv_state[run], st.ssm_state[run], step, self.shape.eps)
+            return ssm_mixer(mixer, xn, st.conv_state[run], st.ssm_state[run], step, eps, proj)
         if isinstance(mixer, DeltaWeights):
-            return delta_mixer(mixer, xn, st.conv_state[run], st.ssm_state[run], step, self.shape.eps)
+            return delta_mixer(mixer, xn, st.conv_state[run], st.ssm_state[run], step, eps, proj)
         if isinstance(mixer, AttentionWeights):
-            return attention_mixer(mixer, xn, st.key_cache[run], st.value_cache[run], step, self.shape.eps,
-                                   st.conv_state.get(run))
-        return latent_mixer(mixer, xn, st.key_cache[run], step, self.shape.eps)
+            return attention_mixer(mixer, xn, st.key_cache[run], st.value_cache[run], step, eps, st.conv_state.get(run), proj)
+        if isinstance(mixer, ParallelWeights):
+            return parallel_mixer(mixer, xn, st.key_cache[run], st.value_cache[run], st.ssm_state[run], step, eps, proj)
+        return latent_mixer(mixer, xn, st.key_cache[run], step, eps, proj)
 
     def _feed_forward(self, mlp, xn: torch.Tensor):
-        """Rows, or the pending sum of a mixture (what `residual_step` takes)."""
+        """Rows, or the pending sum of a mixture (what `residual_step` takes), or rows and the gate's columns behind `up`."""
         if isinstance(mlp, MixtureWeights):
             return mixture_forward(mlp, xn)
         return glu_forward(mlp, xn) if isinstance(mlp, GLUWeights) else mlp_forward(mlp, xn)
 
+    def _sublayer(self, q: int, run: int, layer, xn: torch.Tensor, step: HybridStep) -> dict:
+        """Mixer (q = 0) or feed-forward of a layer; its result and gate as `residual_step` takes them."""
+        if not layer.gates:
+            return dict(y=self._mixer(run, layer.mixer, xn, step) if q == 0 else self._feed_forward(layer.mlp, xn))
+        if q == 0:      # the gate's rows are the last of the in-projection
+            proj = gemm(xn, layer.mixer.w_in, getattr(layer.mixer, "b_in", None))
+            y, gate = self._mixer(run, layer.mixer, xn, step, proj), proj[:, -self.w.xn_cols:]
+        else:
+            y, gate = self._feed_forward(layer.mlp, xn)
+        return dict(y=y, gate=gate, gate_bias=layer.gates[q])
+
     def forward(self, step: HybridStep, rows: torch.Tensor, after_layer=None) -> torch.Tensor:
         """Final-normed hidden states [R, width] of the packed token `rows` (int32).  `after_layer(run, streams)`: called
         with the residual streams [T, streams, width] a layer leaves (development and tests)."""
-        return (self._forward_sandwich if self.shape.sandwich else self._forward_hyper)(step, rows, after_layer)
+        return (self._forward_residual if self.shape.sandwich or self.shape.pre_norm else self._forward_hyper)(step, rows, after_layer)
 
     def _forward_hyper(self, step, rows, after_layer):
         s, w = self.shape, self.w
@@ -97,7 +112,7 @@ class HybridRunner:
             return streams.new_empty((0, w.xn_cols), dtype=w.dtype)
         return hyper_step(streams, norm=w.final_norm, rows=rows, **source, **common)
 
-    def _forward_sandwich(self, step, rows, after_layer):
+    def _forward_residual(self, step, rows, after_layer):
         s, w = self.shape, self.w
         x = torch.empty((step.input_ids.numel(), s.width), device=w.embed.device, dtype=torch.float32)
         common = dict(eps=s.eps, xn_cols=w.xn_cols, dtype=w.dtype)
@@ -115,8 +130,7 @@ class HybridRunner:
             for q, (before, after) in enumerate(layer.norms):
                 add = w.loop_step[loop_pass] if q == 0 and loop_pass is not None else None
                 xn = residual_step(x, norm=before, add=add, **source, **common)
-                y = self._mixer(run, layer.mixer, xn, step) if q == 0 else self._feed_forward(layer.mlp, xn)
-                source = dict(y=y, post=after)
+                source = dict(self._sublayer(q, run, layer, xn, step), post=after)
         if after_layer is not None:
             report(len(s.runs) - 1)
         if rows.numel() == 0:
@@ -150,10 +164,12 @@ class HybridModel:
         w = self.runner.w
         mixers = {run: w.layers[i].mixer for run, (i, _) in enumerate(w.shape.runs)}
         latent = {r: m.row_width for r, m in mixers.items() if isinstance(m, LatentWeights)}
+        gru = {r: m.right.width for r, m in mixers.items() if isinstance(m, ParallelWeights)}
+        mixers = {r: m.left if isinstance(m, ParallelWeights) else m for r, m in mixers.items()}
         heads = {r: (m.kv_heads, m.DK, m.DV) for r, m in mixers.items() if isinstance(m, AttentionWeights)}
         state = {r: m.state_dims() for r, m in mixers.items() if isinstance(m, (SSMWeights, DeltaWeights))}
         conv = {r: m.conv_dims() for r, m in mixers.items() if isinstance(m, AttentionWeights) and m.conv_w is not None}
-        return HybridCacheStore(latent, state, cache_config, num_slots, device, w.dtype, heads, conv)
+        return HybridCacheStore(latent, state, cache_config, num_slots, device, w.dtype, heads, conv, gru)
 
     def forward(self, input_ids=None, intermediate_tensors=None, position_ids=None, **_unused):
         from .inferencer import StageOutput

@@ -1,12 +1,15 @@
 """Configuration of the hybrid decoders: what config.json says, as specs of mixers, feed-forwards and the residual, and
 the checkpoint tensors that go with them.
 
-Three architectures are read here:
+Four architectures are read here:
   "Nurazen"  state-space (Mamba-2) and latent-attention mixers, dense feed-forwards, hyper-connections, shared weights
   "Dekerax"  windowed attention, windowed latent attention with a query latent, gated delta rule, dense and mixture
              feed-forwards, one residual with a norm on both sides of every sublayer, a run of layers that loops
   "Tekilix"  chunked attention in two forms (capped scores; convolved keys that are also the values, learned sinks),
              mixtures chosen inside groups, dynamic tanh on both sides of every sublayer, shared weights, tied embedding
+  "Purozen"  sigmoid attention beside a minGRU, windowed attention that keeps the first tokens (unit-length queries and keys,
+             values mixed with an earlier layer's), latent attention without positions, dense feed-forwards, a norm ahead of
+             every sublayer and a gate per column behind it, tied embedding
 A mechanism is described by a spec of its own, so that an architecture is a choice of specs."""
 from __future__ import annotations
 
@@ -51,11 +54,12 @@ class RotarySpec:
     dims: int
     half: bool                       # pairs (i, i + dims / 2) instead of (2i, 2i + 1)
     yarn: Optional[YarnSpec] = None
+    factor: float = 1.0              # every frequency is divided by it
 
     def frequencies(self) -> tuple:
         """([dims / 2] float64 turns per position, factor of cosine and sine)."""
         i = torch.arange(self.dims // 2, dtype=torch.float64)
-        f = self.base ** (-2 * i / max(self.dims, 1))
+        f = self.base ** (-2 * i / max(self.dims, 1)) / self.factor
         if self.yarn is None:
             return f, 1.0
         y = self.yarn
@@ -78,14 +82,18 @@ class AttentionSpec:
     scale: float
     window: Optional[int] = None             # tokens a query sees, itself included
     chunk: Optional[int] = None              # a query sees its own chunk only; chunks count from the first token
+    keep: int = 0                            # first tokens that are seen from beyond a window or chunk as well
     rot: Optional[RotarySpec] = None
     bias: bool = False                       # of the query, key and value projections
-    qk_norm: Optional[str] = None            # "head": per head, one weight for all; "all": over the whole projection
+    qk_norm: Optional[str] = None            # "head": per head, one weight for all; "unit": per head, no weight; "all": over
+                                             # the whole projection
     conv: Optional[int] = None               # taps of a convolution of queries and keys, ahead of norm and rotation
     keys_as_values: bool = False             # values are the keys ahead of norm and rotation
     softcap: Optional[float] = None          # a score s becomes softcap * tanh(s / softcap)
     sink: Optional[str] = None               # extra term of the denominator: "unit" (1) or "learned" (exp of one per head)
     gate: Optional[str] = None               # output times the sigmoid of one number per "head" or per "column"
+    sigmoid: bool = False                    # a key weighs sigmoid(score + a number per head), no softmax
+    value_mix: Optional[str] = None          # "source": its values are mixed into those of the layers that "mix"
 
 
 @dataclass(frozen=True)
@@ -107,11 +115,27 @@ class DeltaSpec:
     conv: int
 
 
+@dataclass(frozen=True)
+class MinGRUSpec:
+    width: int
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Two mixers that read the same input; the result is left_scale * left + right_scale * right."""
+
+    left: AttentionSpec
+    right: MinGRUSpec
+    left_scale: float
+    right_scale: float
+
+
 # ------------------------------------------------------------------ feed-forwards
 @dataclass(frozen=True)
 class DenseSpec:
     ff: int
     gated: bool = False              # down(gelu(gate) * up), no biases; otherwise down(gelu(up + b)) + b
+    bias: bool = True
 
 
 @dataclass(frozen=True)
@@ -128,7 +152,7 @@ class MixtureSpec:
     groups: tuple = (1, 1)                   # (equal groups of neighbours, groups kept): the rest cannot be chosen
 
 
-MixerSpec = Union[LatentSpec, AttentionSpec, SSMSpec, DeltaSpec]
+MixerSpec = Union[LatentSpec, AttentionSpec, SSMSpec, DeltaSpec, ParallelSpec]
 FFSpec = Union[DenseSpec, MixtureSpec]
 
 
@@ -154,7 +178,7 @@ class HybridShape:
     layers: tuple
     width: int
     vocab: int
-    streams: int             # residual streams (1 for the residual with norms on both sides)
+    streams: int             # residual streams (1 without hyper-connections)
     residual_mult: float
     eps: float
     architecture: str = "Nurazen"
@@ -168,6 +192,17 @@ class HybridShape:
         return self.architecture in ("Dekerax", "Tekilix")
 
     @property
+    def pre_norm(self) -> bool:
+        """One residual with a norm ahead of every sublayer only; a sublayer's result is times the sigmoid of a projection of
+        its input."""
+        return self.architecture == "Purozen"
+
+    @property
+    def norms_around_one(self) -> bool:
+        """Norm weights are stored as their distance from one."""
+        return self.architecture in ("Nurazen", "Purozen")
+
+    @property
     def tanh_norms(self) -> bool:
         """The norms are tanh(alpha x) * weight + b instead of a division by the root mean square."""
         return self.architecture == "Tekilix"
@@ -175,7 +210,7 @@ class HybridShape:
     @property
     def tied(self) -> bool:
         """The embedding is the output table too."""
-        return self.architecture == "Tekilix"
+        return self.architecture in ("Tekilix", "Purozen")
 
     @property
     def runs(self) -> tuple:
@@ -409,9 +444,90 @@ def _write_tekilix(s: HybridShape) -> dict:
             "embedding": {"scale": s.embed_scale}, "logit_scale": s.logit_scale}
 
 
+# ------------------------------------------------------------------ Purozen
+def _read_keeping_window(i: int, m: Mapping) -> tuple:
+    """(window, kept first tokens)."""
+    mask = m.get("mask")
+    if mask is None:
+        return None, 0
+    keep = int(mask.get("keep_first", 0))
+    if keep < 0:
+        raise ValueError(f"layer {i}: {keep} kept tokens")
+    return _read_window(i, {"mask": {k: v for k, v in mask.items() if k != "keep_first"}}), keep
+
+
+def _read_linear_rotary(i: int, m: Mapping) -> Optional[RotarySpec]:
+    rot, dim = m.get("rot"), m["dim"]
+    if rot is None:
+        return None
+    if not 0 <= rot["dims"] <= dim or rot["dims"] % 2:
+        raise ValueError(f"layer {i}: {rot['dims']} of {dim} columns rotate")
+    factor = float((rot.get("scaling") or {"factor": 1.0})["factor"])
+    if factor <= 0:
+        raise ValueError(f"layer {i}: frequencies divided by {factor}")
+    return RotarySpec(float(rot["base"]), rot["dims"], True, factor=factor)
+
+
+def _read_purozen(cfg: Mapping) -> HybridShape:
+    layers, source = [], None
+    for i, e in enumerate(cfg["layers"]):
+        m = e["mixer"]
+        if e["type"] == "parallel":
+            a = m["left"]
+            mixer = ParallelSpec(AttentionSpec(a["heads"], a["kv_heads"], a["dim"], a["vdim"], float(a["scale"]), sigmoid=True),
+                                 MinGRUSpec(m["right"]["width"]), float(m["left_scale"]), float(m["right_scale"]))
+        elif e["type"] == "attention":
+            window, keep = _read_keeping_window(i, m)
+            mix = None
+            if m.get("v_mix"):
+                mix, values = "source" if source is None else "mix", (m["kv_heads"], m["vdim"])
+                source = source or (i, values)
+                if values != source[1]:
+                    raise ValueError(f"layer {i}: values of {values} heads and columns mixed with layer {source[0]}'s of {source[1]}")
+            mixer = AttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), window=window, keep=keep,
+                                  rot=_read_linear_rotary(i, m), qk_norm="unit", value_mix=mix)
+        elif e["type"] == "latent_attention":
+            mixer = LatentSpec(m["heads"], m["dim"], 0, m["vdim"], m["kv_rank"], float(m["scale"]), 1.0, 0, gated=False)
+        else:
+            raise NotImplementedError(f"layer {i}: mixer {e['type']!r}")
+        heads = mixer.left if isinstance(mixer, ParallelSpec) else mixer
+        if heads.heads % getattr(heads, "kv_heads", 1):
+            raise ValueError(f"layer {i}: {heads.heads} heads over {heads.kv_heads} key/value heads")
+        mlp = e.get("mlp")
+        if mlp is not None and mlp["kind"] != "dense":
+            raise NotImplementedError(f"layer {i}: feed-forward {mlp['kind']!r}")
+        layers.append(HybridLayer(mixer, DenseSpec(mlp["ff"], bias=False) if mlp else None, i))
+    return HybridShape(cfg.get("name", "purozen"), tuple(layers), cfg["width"], cfg["vocab"], 1, 1.0,
+                       float(cfg["norm"]["eps"]), "Purozen")
+
+
+def _write_purozen(s: HybridShape) -> dict:
+    def sizes(m):
+        return {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale}
+
+    out = []
+    for layer in s.layers:
+        m = layer.mixer
+        if isinstance(m, ParallelSpec):
+            e = {"type": "parallel", "mixer": {"left": sizes(m.left), "left_scale": m.left_scale,
+                                               "right": {"width": m.right.width}, "right_scale": m.right_scale}}
+        elif isinstance(m, AttentionSpec):
+            e = {"type": "attention", "mixer": dict(sizes(m), v_mix=m.value_mix is not None)}
+            if m.window is not None:
+                e["mixer"]["mask"] = {"size": m.window, "keep_first": m.keep}
+            if m.rot is not None:
+                e["mixer"]["rot"] = {"base": m.rot.base, "dims": m.rot.dims, "scaling": {"factor": m.rot.factor}}
+        else:
+            e = {"type": "latent_attention", "mixer": {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "kv_rank": m.kv_rank,
+                                                       "scale": m.scale}}
+        e["mlp"] = None if layer.ff is None else {"kind": "dense", "ff": layer.ff.ff}
+        out.append(e)
+    return {"architecture": "Purozen", "layers": out, "norm": {"eps": s.eps}, "width": s.width, "vocab": s.vocab}
+
+
 # config.json "architecture" -> (reader, writer)
 ARCHITECTURES = {"Nurazen": (_read_nurazen, _write_nurazen), "Dekerax": (_read_dekerax, _write_dekerax),
-                 "Tekilix": (_read_tekilix, _write_tekilix)}
+                 "Tekilix": (_read_tekilix, _write_tekilix), "Purozen": (_read_purozen, _write_purozen)}
 
 
 # ------------------------------------------------------------------ checkpoint tensors
@@ -431,7 +547,11 @@ def _mixer_tensors(m: MixerSpec, W: int) -> dict:
         t = {n: (r, W) for n, r in rows.items()}
         if m.bias:
             t.update({n + ".b": (r,) for n, r in rows.items()})
-        if m.qk_norm is not None:
+        if m.sigmoid:
+            t["pb"] = (m.heads,)
+        if m.value_mix is not None:
+            t["vmix"] = ()
+        if m.qk_norm in ("head", "all"):
             t.update({n + ".norm": (rows[n] if m.qk_norm == "all" else m.dim,) for n in "qk"})
         if m.conv is not None:
             t.update({n + ".conv": (rows[n], m.conv) for n in "qk"})
@@ -440,6 +560,11 @@ def _mixer_tensors(m: MixerSpec, W: int) -> dict:
         if m.gate is not None:
             t["g"] = (m.heads * (m.vdim if m.gate == "column" else 1), W)
         return dict(t, o=(W, m.heads * m.vdim))
+    if isinstance(m, ParallelSpec):
+        return {f"{side}.{k}": v for side, part in (("left", m.left), ("right", m.right)) for k, v in _mixer_tensors(part, W).items()}
+    if isinstance(m, MinGRUSpec):
+        n = m.width
+        return {"z": (n, W), "z.b": (n,), "x": (n, W), "x.b": (n,), "g": (n, W), "o": (W, n)}
     if isinstance(m, DeltaSpec):
         qk, v = m.kv_heads * m.dim, m.heads * m.vdim
         return {"q": (qk, W), "q.conv": (qk, m.conv), "k": (qk, W), "k.conv": (qk, m.conv), "v": (v, W),
@@ -455,7 +580,8 @@ def _ff_tensors(ff: FFSpec, W: int) -> dict:
         return dict({p + "gate": (n, W)} if gated else {}, **{p + "up": (n, W), p + "down": (W, n)})
 
     if isinstance(ff, DenseSpec):
-        return expert("", ff.ff, True) if ff.gated else {"up": (ff.ff, W), "up.b": (ff.ff,), "down": (W, ff.ff), "down.b": (W,)}
+        t = expert("", ff.ff, ff.gated)
+        return dict(t, **{"up.b": (ff.ff,), "down.b": (W,)}) if ff.bias and not ff.gated else t
     t, gated = {"router": (ff.experts, W)}, ff.act != "relu2"
     if ff.correction:
         t["correction"] = (ff.experts,)
@@ -488,6 +614,8 @@ def tensor_shapes(shape: HybridShape) -> dict[str, tuple]:
             t.update(norm(f"norm{q}"))
             if shape.sandwich:
                 t.update(norm(f"norm{q}b"))
+            elif shape.pre_norm:
+                t.update({f"rg{q}": (W, W), f"rg{q}.b": (W,)})
             else:
                 t.update({f"hc{q}.in": (n,), f"hc{q}.out": (n,), f"hc{q}.mix": (n, n)})
         if layer.ff is not None:
@@ -519,13 +647,17 @@ def random_tensors(shape: HybridShape, seed: int = 0, device="cpu", dtype=torch.
         elif leaf == "mlp.correction":
             t = 0.3 * t / dims[0]        # of the order of the scores
         elif leaf.startswith("norm") or name in ("final.norm", "embed.norm"):
-            t = 1 + 0.1 * t if shape.sandwich else 0.1 * t
+            t = 0.1 * t if shape.norms_around_one else 1 + 0.1 * t
         elif leaf.endswith("norm"):
             t = 1 + 0.1 * t
         elif leaf.endswith((".in", ".out")) and leaf.startswith("hc"):
             t = 1.0 / shape.streams + 0.2 * t
         elif leaf.startswith("hc"):
             t = torch.eye(shape.streams, device=device) * 0.8 + 0.2 / shape.streams + 0.05 * t
+        elif leaf.endswith(".vmix"):
+            t = 0.4 + 0.1 * t
+        elif leaf.endswith(".pb"):
+            t = t - 2.0
         elif leaf == "mix.A_log":
             t = 0.5 * t
         elif leaf == "mix.dt_bias":

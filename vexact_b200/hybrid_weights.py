@@ -12,14 +12,17 @@ import torch
 from .delta import DeltaWeights
 from .fused_moe import MixtureWeights
 from .feed_forward import GLUWeights, MLPWeights
-from .hybrid_config import AttentionSpec, DeltaSpec, DenseSpec, HybridShape, LatentSpec, random_tensors, tensor_shapes
+from .gru import MinGRUWeights
+from .hybrid_config import (AttentionSpec, DeltaSpec, DenseSpec, HybridShape, LatentSpec, ParallelSpec, random_tensors,
+                            tensor_shapes)
 from .hyper import Connection
 from .latent_attention import LatentWeights
+from .parallel import ParallelWeights
 from .residual import Norm, TanhNorm
 from .ssm import SSMWeights
 from .window_attention import AttentionWeights
 
-MixerWeights = Union[LatentWeights, AttentionWeights, SSMWeights, DeltaWeights]
+MixerWeights = Union[LatentWeights, AttentionWeights, SSMWeights, DeltaWeights, ParallelWeights]
 FFWeights = Union[MLPWeights, GLUWeights, MixtureWeights]
 
 
@@ -52,7 +55,8 @@ class HybridLayerWeights:
     mixer: MixerWeights
     mlp: Optional[FFWeights]
     hc: list = field(default_factory=list)      # hyper-connections: Connection of the mixer (and of the feed-forward)
-    norms: list = field(default_factory=list)   # norms on both sides: (before, after) of each
+    norms: list = field(default_factory=list)   # one residual: (before, after or None) of each sublayer
+    gates: list = field(default_factory=list)   # bias of each sublayer's residual gate, whose rows end w_in and up; or none
 
 
 @dataclass
@@ -81,7 +85,7 @@ class HybridWeights:
             if tuple(tensors[name].shape) != dims:
                 raise ValueError(f"tensor {name} is {tuple(tensors[name].shape)}, the configuration says {dims}")
         b = _Builder(tensors, shape.width, dtype, device)
-        norm = b.tanh_norm if shape.tanh_norms else lambda name: b.vec(tensors[name])
+        norm = b.tanh_norm if shape.tanh_norms else b.norm_around_one if shape.pre_norm else lambda name: b.vec(tensors[name])
         out = HybridWeights(shape, dtype, embed=b.mat(tensors["embed"]), final_norm=norm("final.norm"))
         if shape.tied and b.W8 == shape.width:
             out.head = out.embed
@@ -99,10 +103,15 @@ class HybridWeights:
                 out.layers.append(out.layers[layer.weights_of])
                 continue
             p, spec = f"l{i}.", layer.ff
-            lw = HybridLayerWeights(b.mixer(p + "mix.", layer.mixer), None if spec is None else b.ff(p + "mlp.", spec))
+            tail = lambda q: [tensors[f"{p}rg{q}"]] if shape.pre_norm else []   # noqa: E731
+            lw = HybridLayerWeights(b.mixer(p + "mix.", layer.mixer, tail(1)),
+                                    None if spec is None else b.ff(p + "mlp.", spec, tail(2)))
             for q in ([1] if spec is None else [1, 2]):
                 if shape.sandwich:
                     lw.norms.append((norm(f"{p}norm{q}"), norm(f"{p}norm{q}b")))
+                elif shape.pre_norm:
+                    lw.norms.append((norm(f"{p}norm{q}"), None))
+                    lw.gates.append(b.vec(tensors[f"{p}rg{q}.b"]))
                 else:
                     hc = f"{p}hc{q}."
                     lw.hc.append(Connection(read=b.vec(tensors[hc + "in"]), mix=b.vec(tensors[hc + "mix"]),
@@ -148,25 +157,52 @@ class _Builder:
         t = self.tensors
         return TanhNorm(self.vec(t[name]), self.vec(t[name + ".b"]), float(t[name + ".alpha"]))
 
+    def norm_around_one(self, name):
+        return 1 + self.vec(self.tensors[name])
+
     def in_proj(self, parts):
         """Row blocks that read the layer's input, stacked; rows up to a multiple of 8."""
         t = torch.cat(parts)
         return self.mat(_pad_cols(_pad_rows(t, 1, _up8(t.shape[0])), 1, self.W8))
 
+    def stack(self, mat, tail):
+        """mat with the rows `tail` (of width x width tensors, padded) under it."""
+        return torch.cat([mat] + [self.in_proj([t]) for t in tail]) if tail else mat
+
     # ------------------------------------------------------------------ mixers
-    def mixer(self, p, m):
+    def mixer(self, p, m, tail=()):
         if isinstance(m, LatentSpec):
-            return self.latent(p, m)
-        if isinstance(m, AttentionSpec):
-            return self.attention(p, m)
-        return self.delta(p, m) if isinstance(m, DeltaSpec) else self.ssm(p, m)
+            w = self.latent(p, m)
+        elif isinstance(m, AttentionSpec):
+            w = self.attention(p, m)
+        elif isinstance(m, ParallelSpec):
+            w = self.parallel(p, m)
+        else:
+            w = self.delta(p, m) if isinstance(m, DeltaSpec) else self.ssm(p, m)
+        rows, w.w_in = w.w_in.shape[0], self.stack(w.w_in, tail)
+        if getattr(w, "b_in", None) is not None:
+            w.b_in = torch.cat([w.b_in, w.b_in.new_zeros(w.w_in.shape[0] - rows)])
+        return w
+
+    def parallel(self, p, m):
+        left, n = self.attention(p + "left.", m.left), _up8(m.right.width)
+        get = lambda name: self.tensors[p + "right." + name]   # noqa: E731
+        right = MinGRUWeights(z_bias=self.vec(_pad_rows(get("z.b"), 1, n)), x_bias=self.vec(_pad_rows(get("x.b"), 1, n)),
+                              width=n, out_scale=m.right_scale)
+        w = ParallelWeights(w_in=torch.cat([left.w_in, self.in_proj([_pad_rows(get(k), 1, n) for k in "zxg"])]),
+                            w_out=torch.cat([left.w_out, self.mat(_pad_cols(get("o"), 1, n))], 1), left=left, right=right)
+        left.w_in = left.w_out = None
+        left.out_scale = m.left_scale
+        return w
 
     def latent(self, p, m):
         H, DN, DR, R, V = m.heads, _up8(m.dim), _up8(m.rot_dim), _up8(m.kv_rank), _up8(m.vdim)
         get = lambda n: self.tensors[p + n]   # noqa: E731
-        q = get("q" if m.q_rank is None else "uq").view(H, m.dim + m.rot_dim, -1)
-        qn, qr = _pad_rows(q[:, :m.dim].reshape(H * m.dim, -1), H, DN), _pad_rows(q[:, m.dim:].reshape(H * m.rot_dim, -1), H, DR)
-        q = torch.cat([qn.view(H, DN, -1), qr.view(H, DR, -1)], 1).reshape(H * (DN + DR), -1)
+        q = get("q" if m.q_rank is None else "uq")
+        K = q.shape[1]
+        q = q.view(H, m.dim + m.rot_dim, K)
+        qn, qr = _pad_rows(q[:, :m.dim].reshape(H * m.dim, K), H, DN), _pad_rows(q[:, m.dim:].reshape(H * m.rot_dim, K), H, DR)
+        q = torch.cat([qn.view(H, DN, K), qr.view(H, DR, K)], 1).reshape(H * (DN + DR), K)
         dkv, query = get("dkv"), {}
         head = q
         if m.q_rank is not None:
@@ -198,7 +234,11 @@ class _Builder:
         if m.bias:
             b = torch.cat([_pad_rows(get(n + ".b"), *wide[n]) for n in names])
             more["b_in"] = self.mat(torch.cat([b, b.new_zeros(w_in.shape[0] - b.numel())]))
-        if m.qk_norm is not None:
+        if m.sigmoid:
+            more["sigmoid_bias"] = self.vec(get("pb"))
+        if m.value_mix == "mix":
+            more["v_mix"] = float(get("vmix"))
+        if m.qk_norm in ("head", "all"):
             more.update({n + "_norm": self.vec(_pad_rows(get(n + ".norm"), wide[n][0] if m.qk_norm == "all" else 1, DK))
                          for n in "qk"})
         if m.conv is not None:
@@ -210,7 +250,8 @@ class _Builder:
             more.update(inv_freq=self.vec(freq), rot_half=m.rot.half)
         return AttentionWeights(w_in=w_in, w_out=self.mat(_pad_cols(get("o"), H, DV)), heads=H, kv_heads=G, DK=DK, DV=DV,
                                 scale=m.scale, window=m.window, chunk=m.chunk, softcap=m.softcap, gate=m.gate,
-                                keys_as_values=m.keys_as_values, qk_norm=m.qk_norm, dim=m.dim, **more)
+                                keys_as_values=m.keys_as_values, qk_norm=m.qk_norm, dim=m.dim, keep=m.keep,
+                                value_mix=m.value_mix, **more)
 
     def ssm(self, p, m):
         H, P, G, N = m.heads, _up8(m.vdim), m.groups, _up8(m.state)
@@ -243,15 +284,20 @@ class _Builder:
                             vdim=m.vdim, dim=m.dim)
 
     # ------------------------------------------------------------------ feed-forwards
-    def ff(self, p, spec):
-        if isinstance(spec, DenseSpec):
-            return self.glu(p, spec.ff, "gelu_tanh") if spec.gated else self.mlp(p, spec.ff)
-        return self.mixture(p, spec)
+    def ff(self, p, spec, tail=()):
+        if isinstance(spec, DenseSpec) and not spec.gated:
+            return self.mlp(p, spec.ff, bias=spec.bias, tail=tail)
+        if tail:
+            raise NotImplementedError(f"a residual gate behind {spec}")
+        return self.glu(p, spec.ff, "gelu_tanh") if isinstance(spec, DenseSpec) else self.mixture(p, spec)
 
-    def mlp(self, p, ff, act="gelu_tanh", bias=True):
+    def mlp(self, p, ff, act="gelu_tanh", bias=True, tail=()):
         F8, get = _up8(ff), lambda n: self.tensors[p + n]
         more = dict(up_b=self.mat(_pad_rows(get("up.b"), 1, F8)), down_b=self.mat(get("down.b"))) if bias else {}
-        return MLPWeights(up=self._rows(p, ("up",), ff), down=self.mat(_pad_cols(get("down"), 1, F8)), act=act, **more)
+        up = self.stack(self._rows(p, ("up",), ff), tail)
+        if bias and tail:
+            more["up_b"] = torch.cat([more["up_b"], more["up_b"].new_zeros(up.shape[0] - F8)])
+        return MLPWeights(up=up, down=self.mat(_pad_cols(get("down"), 1, F8)), act=act, tail=up.shape[0] - F8, **more)
 
     def _rows(self, p, names, ff):
         """The named [ff, width] tensors, stacked."""

@@ -179,10 +179,13 @@ class HybridCacheStore:
     attention layer: `key_cache[layer]` [blocks, page, kv_heads, DK] and `value_cache[layer]` [blocks, page, kv_heads, DV].
     recurrent layer: `conv_state[layer]` [slots, taps - 1, channels] in the model dtype and `ssm_state[layer]`
     [slots, heads, N, P] fp32.
-    attention layer with a convolution: `conv_state[layer]` beside its pages."""
+    attention layer with a convolution: `conv_state[layer]` beside its pages.
+    layer with an element-by-element recurrence: `ssm_state[layer]` [slots, width] fp32, beside pages where it runs at an
+    attention's side."""
 
     def __init__(self, latent_widths: dict, ssm_dims: dict, cache_config, num_slots: int, device,
-                 dtype=torch.bfloat16, head_dims: Optional[dict] = None, conv_dims: Optional[dict] = None):
+                 dtype=torch.bfloat16, head_dims: Optional[dict] = None, conv_dims: Optional[dict] = None,
+                 gru_widths: Optional[dict] = None):
         self.cache_config = cache_config
         self.device = torch.device(device)
         self.page_size = cache_config.page_size
@@ -200,6 +203,8 @@ class HybridCacheStore:
             self.ssm_state[li] = torch.zeros((num_slots, heads, n, p), device=self.device, dtype=torch.float32)
         for li, (channels, taps) in (conv_dims or {}).items():
             self.conv_state[li] = torch.zeros((num_slots, taps - 1, channels), device=self.device, dtype=dtype)
+        for li, width in (gru_widths or {}).items():
+            self.ssm_state[li] = torch.zeros((num_slots, width), device=self.device, dtype=torch.float32)
 
     def num_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for d in (self.key_cache, self.value_cache, self.conv_state,

@@ -1,6 +1,6 @@
 """Latent attention over the paged latent cache (`csrc/latent.cuh`).
 
-The cache holds the normed latent and the shared rotated key part of every token.  Attention runs in the absorbed
+The cache holds the normed latent and the shared rotated key part, if there is one, of every token.  Attention runs in the absorbed
 form: the query's unrotated part goes through W_uk (one small product per head), attention is one KV head of width
 R + DR whose value is the latent, and W_uv turns a head's latent output into its value (the output gate, where a model
 has one, rides on that product's epilogue).
@@ -72,7 +72,7 @@ def latent_prep(w: LatentWeights, cache: torch.Tensor, step, eps: float, *, q: O
         _lib.load().b200_latent_prep(
             _lib.ptr(q), stride(q), _lib.ptr(kv), stride(kv), _lib.ptr(q_latent), stride(q_latent), _lib.ptr(w.q_norm),
             0 if w.q_norm is None else w.q_norm.numel(), w.q_true, step.positions.data_ptr(), step.slot_mapping.data_ptr(),
-            w.inv_freq.data_ptr(), w.c_norm.data_ptr(), cache.data_ptr(), _lib.ptr(q_lat), some.shape[0], w.heads,
+            _lib.ptr(w.inv_freq), w.c_norm.data_ptr(), cache.data_ptr(), _lib.ptr(q_lat), some.shape[0], w.heads,
             w.DN, w.DR, w.R, w.r_true, w.rot_dims, int(w.rot_half), float(eps), cache.shape[0] * cache.shape[1],
             _dt(some.dtype), _lib.current_stream()),
         "b200_latent_prep")
@@ -97,7 +97,7 @@ TC_BLOCK, TC_SPLIT, TC_COLUMNS = 128, 512, 16     # keys of a block and of a spl
 def tc_supported(w: LatentWeights, dtype, page_size: int) -> bool:
     """Whether the tensor-core kernel takes these dims (the CUDA-core kernel takes every one)."""
     pages = page_size % 128 == 0 or (page_size >= 8 and 128 % page_size == 0)
-    return dtype == torch.bfloat16 and pages and w.R <= 512 and 0 < w.DR <= 128
+    return dtype == torch.bfloat16 and pages and w.R <= 512 and w.DR <= 128
 
 
 def _tc_splits(new: int, total: int, window: Optional[int]) -> int:
@@ -211,9 +211,12 @@ def latent_expanded(w: LatentWeights, q: torch.Tensor, gate: Optional[torch.Tens
         "b200_latent_attn_expanded")
 
 
-def latent_mixer(w: LatentWeights, xn: torch.Tensor, cache: torch.Tensor, step, eps: float) -> torch.Tensor:
+def latent_mixer(w: LatentWeights, xn: torch.Tensor, cache: torch.Tensor, step, eps: float,
+                 proj: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """proj: the projection rows of xn, where the caller has them already."""
     T, H = xn.shape[0], w.heads
-    proj = gemm(xn, w.w_in)
+    if proj is None:
+        proj = gemm(xn, w.w_in)
     dq, q_cols = w.DN + w.DR, w.q_cols
     kv = proj[:, q_cols:q_cols + w.row_width]
     gate = proj[:, q_cols + w.row_width:q_cols + w.row_width + H * w.V].view(T, H, w.V) if w.gated else None

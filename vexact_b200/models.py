@@ -298,6 +298,7 @@ MODEL_LOADERS = {
     "Nurazen": _load_hybrid,
     "Dekerax": _load_hybrid,
     "Tekilix": _load_hybrid,
+    "Purozen": _load_hybrid,
     "qwen2": _load_stage,
     "qwen3": _load_stage,
     "qwen3_moe": _load_stage,

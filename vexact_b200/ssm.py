@@ -2,6 +2,7 @@
 from __future__ import annotations
 
 from dataclasses import dataclass
+from typing import Optional
 
 import torch
 
@@ -127,9 +128,11 @@ def ssm_gate_norm(w: SSMWeights, y: torch.Tensor, proj: torch.Tensor, eps: float
     return head_gate_norm(y, proj[:, :w.inner], w.norm, w.heads, w.P, w.vdim, w.parts, eps)
 
 
-def ssm_mixer(w: SSMWeights, xn: torch.Tensor, conv_state: torch.Tensor, state: torch.Tensor, step,
-              eps: float) -> torch.Tensor:
-    proj = gemm(xn, w.w_in)
+def ssm_mixer(w: SSMWeights, xn: torch.Tensor, conv_state: torch.Tensor, state: torch.Tensor, step, eps: float,
+              proj: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """proj: the projection rows of xn, where the caller has them already."""
+    if proj is None:
+        proj = gemm(xn, w.w_in)
     act, dt = short_conv(w, proj, conv_state, step)
     y = torch.empty((xn.shape[0], w.inner), device=xn.device, dtype=xn.dtype)
     if step.max_seqlen_q <= SCAN_MAX_TOKENS or xn.dtype != torch.bfloat16 or w.N > CHUNK_MAX_STATE:
