@@ -85,6 +85,10 @@ def parse_args():
                     help="side measurement: prefill and decode steps of the Tekilix decoders (chunked attention with sinks, "
                          "capped scores and gates, convolved keys, grouped choice of experts, dynamic tanh) beside the "
                          "grouped-query MoE model of equal width, and its kernels beside that model's")
+    ap.add_argument("--purozen", action="store_true",
+                    help="side measurement: prefill and decode steps of the Purozen decoders (sigmoid attention beside a "
+                         "minGRU, windows that keep the first tokens, latent attention without positions, gated residual) "
+                         "beside a grouped-query dense model of equal width, and its kernels beside that model's")
     ap.add_argument("--prefill-attention", type=int, default=0, metavar="QLEN",
                     help="side measurement: time one causal prefill attention call of QLEN queries on the "
                          "model's head shape (context --ctx if larger) and print its own JSON line")
@@ -795,10 +799,11 @@ def hybrid_model_case(args, shape, kind, S, new, total, page, device):
             return runner.logits(runner.forward(step, rows))
 
         def reach(mixer):      # keys that some new token sees
+            mixer = getattr(mixer, "left", mixer)
             chunk = getattr(mixer, "chunk", None)
             if chunk:
                 return total - (total - new) // chunk * chunk
-            return min(total, (getattr(mixer, "window", None) or total) + new - 1)
+            return min(total, (getattr(mixer, "window", None) or total) + new - 1 + getattr(mixer, "keep", 0))
 
         seen = {run: reach(w.layers[i].mixer) for run, (i, _) in enumerate(shape.runs)}
         cache_bytes = sum(S * seen[run] * t[0, 0].numel() * 2 for d in (runner.store.key_cache, runner.store.value_cache)
@@ -1429,6 +1434,218 @@ def tekilix_kernels(device):
         torch.cuda.empty_cache()
 
 
+# --------------------------------------------------------------------------- Purozen decoders
+PZ_WINDOW, PZ_KEEP = 1024, 128
+
+
+def purozen_shapes():
+    """(Purozen: 2 parallel + 4 windowed attention + 2 latent layers, the grouped-query dense model), equal width, heads and
+    parameters per feed-forward.  The other model's feed-forward is gated (three matrices), these are not (two)."""
+    from vexact_b200.hybrid import (AttentionSpec, DenseSpec, HybridLayer, HybridShape, LatentSpec, MinGRUSpec, ParallelSpec,
+                                    RotarySpec)
+    from vexact_b200.inferencer import ModelShape
+
+    W, V, scale = 2048, 32768, 128 ** -0.5
+    par = ParallelSpec(AttentionSpec(16, 4, 128, 128, scale, sigmoid=True), MinGRUSpec(2048), 0.6, 0.9)
+    lat = LatentSpec(16, 128, 0, 128, 512, scale, 1.0, 0, gated=False)
+
+    def att(mix):
+        return AttentionSpec(16, 4, 128, 128, scale, window=PZ_WINDOW, keep=PZ_KEEP, rot=RotarySpec(50000.0, 64, True, factor=8.0),
+                             qk_norm="unit", value_mix=mix)
+
+    kinds = [par, att("source"), lat, att("mix"), par, att("mix"), lat, att("mix")]
+    return (HybridShape("purozen-2parallel-4attention-2latent", tuple(HybridLayer(m, DenseSpec(8192, bias=False), i)
+                                                                      for i, m in enumerate(kinds)), W, V, 1, 1.0, 1e-6, "Purozen"),
+            ModelShape("gqa-dense", 8, W, 16, 4, 128, V, ffn=5504, qk_norm=True, rms_eps=1e-6))
+
+
+def run_purozen(args):
+    """Side measurement: steps of the Purozen decoders beside the closest other model (random weights), then its kernels
+    beside the like kernels of that one."""
+    from vexact_b200 import _lib
+
+    device = torch.device("cuda", 0)
+    torch.cuda.set_device(device)
+    cases = [("decode", 64, 1, 4096), ("decode", 256, 1, 1024), ("prefill", 4, 2048, 2048), ("prefill", 1, 2048, 8192)]
+    clocks = ClockSampler(0)
+    clocks.start()
+    clocks.wait_first_sample()
+    for shape in purozen_shapes():
+        for kind, S, new, total in cases:
+            print(json.dumps(hybrid_model_case(args, shape, kind, S, new, total, DK_PAGE, device)), flush=True)
+            torch.cuda.empty_cache()
+    for line in purozen_kernels(device):
+        print(json.dumps(line), flush=True)
+    print(json.dumps({"measurement": "purozen", "clocks": clocks.stop(), "status": list(_lib.read_status())}))
+
+
+def purozen_kernels(device):
+    """Per kernel of the Purozen decoders and the like kernel of the grouped-query dense model (for what that model does not
+    have, of the other hybrids): device time, achieved bytes or flops over the measured peak.  Several buffers per kernel,
+    together larger than L2."""
+    import vexact_b200 as vb
+    from vexact_b200 import _lib, gru, latent_attention as la, ssm, window_attention as wa
+    from vexact_b200.batch_invariant_ops import gemm
+    from vexact_b200.feed_forward import mlp_forward
+    from vexact_b200.hybrid import HybridLayer, HybridShape, HybridWeights
+    from vexact_b200.residual import residual_step
+
+    peaks = measured_peaks()
+    hbm, tc = float(peaks.get("hbm_gbs", 6650.0)), float(peaks.get("bf16_tflops", 1590.0))
+    BF = torch.bfloat16
+    pz, _ = purozen_shapes()
+    W = pz.width
+    few = HybridShape("few", tuple(HybridLayer(pz.layers[i].mixer, pz.layers[i].ff, n) for n, i in enumerate((0, 1, 2, 3))), W, 1024, 1,
+                      1.0, 1e-6, "Purozen")
+    w = HybridWeights.random_init(few, device=device)
+    par, _, lw, aw = (layer.mixer for layer in w.layers)
+    one = HybridShape("one", tuple(HybridLayer(hybrid_shapes()[0].layers[i].mixer, None, n) for n, i in enumerate((0, 2))), W, 1024, 4,
+                      0.3, 1e-5)
+    sw, olw = (layer.mixer for layer in HybridWeights.random_init(one, device=device).layers)
+    left, right, mlp, norm, gb = par.left, par.right, w.layers[0].mlp, w.layers[0].norms[0][0], w.layers[0].gates[0]
+    rn = lambda *s: torch.randn(s, device=device).to(BF)   # noqa: E731
+
+    def line(name, ms, nbytes=None, flops=None, like=None):
+        out = {"measurement": "purozen_kernel", "kernel": name, "us": round(ms * 1e3, 2)}
+        fr = []
+        if nbytes:
+            out["gb_s"] = round(nbytes / ms / 1e6)
+            fr.append(nbytes / ms / 1e6 / hbm)
+        if flops:
+            out["tflop_s"] = round(flops / ms / 1e9, 1)
+            fr.append(flops / ms / 1e9 / tc)
+        out["of_measured_roofline"] = round(max(fr), 3)
+        if like:
+            out["like"] = like
+        return out
+
+    nw = rn(W)
+    for T in (64, 8192):
+        k = 24 if T == 64 else 3
+        st, blocks = hybrid_step([(1, 100)] * T if T == 64 else [(T // 4, T // 4)] * 4, DK_PAGE, device)
+        S = st.state_slots.numel()
+        # boundaries of sublayers
+        sets = [(torch.randn(T, W, device=device), rn(T, W), rn(T, 4 * W)[:, 3 * W:]) for _ in range(k)]
+        ms = graph_ms([lambda x=x, y=y, g=g: residual_step(x, y=y, gate=g, gate_bias=gb, norm=norm, eps=1e-6) for x, y, g in sets])
+        yield line(f"residual_step, gated T={T}", ms, T * W * 14)
+        pairs = [(y, rn(T, W)) for _, y, _ in sets]
+        ms = graph_ms([lambda y=y, r=r: vb.add_rms_norm(y, r, nw, 1e-6) for y, r in pairs])
+        yield line(f"add_rmsnorm T={T}", ms, T * W * 8, like=f"residual_step, gated T={T}")
+        xs = [y for _, y, _ in sets]
+        # feed-forward; the weights of several copies rotate at the small size, so that they come from HBM
+        copies = [mlp] + [mlp.__class__(up=mlp.up.clone(), down=mlp.down.clone(), act=mlp.act, tail=mlp.tail) for _ in range(3)]
+        n, F = mlp.up.numel() + mlp.down.numel(), mlp.down.shape[1]
+        nbytes, flops = 2 * (n + 2 * T * W + T * W), 2.0 * T * n
+        ms = graph_ms([lambda x=x, c=c: mlp_forward(c, x) for x, c in zip(xs, copies * 6)])
+        yield line(f"feed-forward and gate T={T}", ms, nbytes, flops)
+        ms = graph_ms([lambda x=x, c=c: gemm(gemm(x, c.up)[:, :F], c.down) for x, c in zip(xs, copies * 6)])
+        yield line(f"its two products, plain gemm T={T}", ms, nbytes, flops, like=f"feed-forward and gate T={T}")
+        del copies, sets, pairs, xs
+        torch.cuda.empty_cache()
+        # minGRU beside the state-space scan
+        cols = left.in_rows
+        proj = [rn(T, par.w_in.shape[0])[:, cols:] for _ in range(k)]
+        outs = [torch.empty(T, left.heads * left.DV + right.width, device=device, dtype=BF)[:, left.heads * left.DV:] for _ in range(k)]
+        states = [torch.zeros(S, right.width, device=device) for _ in range(k)]
+        nbytes = T * right.width * 8 + S * right.width * 8
+        if T == 64:
+            ms = graph_ms([lambda p=p, s=s, o=o: gru.gru_scan(right, p, s, o, st) for p, s, o in zip(proj, states, outs)])
+            yield line("gru_scan (decode) S=64", ms, nbytes)
+            act = [(rn(T, sw.channels), torch.rand(T, sw.heads, device=device) * 0.1,
+                    torch.zeros(S, sw.heads, sw.N, sw.P, device=device), rn(T, sw.inner)) for _ in range(4)]
+            ms = graph_ms([lambda a=a: ssm.ssm_scan(sw, *a, st) for a in act])
+            yield line("ssm_scan (decode) S=64", ms, T * (sw.channels + sw.inner) * 2 + T * sw.heads * 4 + 8 * S * sw.heads * sw.N * sw.P,
+                       like="gru_scan (decode) S=64")
+            del act
+        else:
+            for channels in (16, 32):
+                ms = graph_ms([lambda p=p, s=s, o=o: gru.gru_chunk_scan(right, p, s, o, st, 17, 4, channels)
+                               for p, s, o in zip(proj, states, outs)])
+                yield line(f"gru_chunk T={T}, {channels} channels", ms, nbytes)
+            lone, _ = hybrid_step([(2048, 8192)], DK_PAGE, device)
+            for channels in (16, 32):
+                ms = graph_ms([lambda p=p, s=s, o=o: gru.gru_chunk_scan(right, p[:2048], s, o[:2048], lone, 17, 1, channels)
+                               for p, s, o in zip(proj, states, outs)])
+                yield line(f"gru_chunk T=2048, one sequence, {channels} channels", ms, 2048 * right.width * 8)
+        del proj, outs, states
+        torch.cuda.empty_cache()
+        # what lies between the projections and attention
+        kc, vc = (torch.zeros(blocks, DK_PAGE, 4, 128, device=device, dtype=BF) for _ in range(2))
+        proj, first = [rn(T, aw.w_in.shape[0]) for _ in range(k)], rn(T, 5120)[:, 2560:3072]
+        ms = graph_ms([lambda p=p: wa.attn_prep(aw, p, kc, vc, None, st, 1e-6, first) for p in proj])
+        yield line(f"attn_prep, unit length and mixed values T={T}", ms, T * 2 * (2 * 24 * 128 + 512))
+        qkv, qn = [rn(T, 24 * 128) for _ in range(k)], rn(128)
+        freq, q_out = torch.rand(64, device=device), torch.empty(T, 2048, device=device, dtype=BF)
+        ms = graph_ms([lambda p=p: _lib.check(_lib.load().b200_qknorm_rope_store(
+            p.data_ptr(), p.stride(0), st.positions.data_ptr(), st.slot_mapping.data_ptr(), qn.data_ptr(), qn.data_ptr(),
+            freq.data_ptr(), q_out.data_ptr(), kc.data_ptr(), vc.data_ptr(), T, 16, 4, 128, blocks * DK_PAGE, 1e-6,
+            _lib.current_stream()), "b200_qknorm_rope_store") for p in qkv])
+        yield line(f"qknorm_rope_store T={T}", ms, T * 2 * 2 * 24 * 128, like=f"attn_prep, unit length and mixed values T={T}")
+        keys, values = ([p[:, a:a + 512].unflatten(1, (4, 128)) for p in proj] for a in (2048, 2560))
+        ms = graph_ms([lambda a=a, b=b: wa.store_kvcache(a, b, kc, vc, st.slot_mapping) for a, b in zip(keys, values)])
+        yield line(f"kv_store T={T}", ms, T * 4 * 1024)
+        del proj, qkv, keys, values, kc, vc
+        cache, rows = torch.zeros(blocks, DK_PAGE, lw.row_width, device=device, dtype=BF), [rn(T, lw.w_in.shape[0]) for _ in range(k)]
+        ms = graph_ms([lambda p=p: la.latent_prep(lw, cache, st, 1e-6, kv=p[:, lw.q_cols:lw.q_cols + lw.R]) for p in rows])
+        yield line(f"latent_prep without rotation T={T}", ms, T * lw.R * 4)
+        cache, rows = torch.zeros(blocks, DK_PAGE, olw.row_width, device=device, dtype=BF), [rn(T, olw.w_in.shape[0]) for _ in range(k)]
+        ms = graph_ms([lambda p=p: la.latent_prep(olw, cache, st, 1e-6, kv=p[:, olw.q_cols:olw.q_cols + olw.row_width]) for p in rows])
+        yield line(f"latent_prep with a rotated part T={T}", ms, T * olw.row_width * 4, like=f"latent_prep without rotation T={T}")
+        del cache, rows
+        torch.cuda.empty_cache()
+    plain = wa.AttentionWeights(w_in=None, w_out=None, heads=16, kv_heads=4, DK=128, DV=128, scale=128 ** -0.5)
+    kinds = {"sigmoid attention": left, "windowed attention": aw}
+    # attention of decoded tokens
+    for S, ctx in ((64, 4096), (256, 1024), (64, 1024)):
+        st, blocks = hybrid_step([(1, ctx)] * S, DK_PAGE, device)
+        sets = [(rn(S, 2048), rn(blocks, DK_PAGE, 4, 128), rn(blocks, DK_PAGE, 4, 128),
+                 torch.empty(S, 2048, device=device, dtype=BF)) for _ in range(2 if ctx * S > 200000 else 4)]
+        for name, m in kinds.items():
+            n = min(ctx, PZ_WINDOW + PZ_KEEP) if m.window else ctx
+            ms = graph_ms([lambda s=s: wa.attend_decode(m, *s, st) for s in sets])
+            yield line(f"{name} decode {S}x{ctx}", ms, S * n * 4 * 256 * 2)
+        ms = graph_ms([lambda s=s: wa.attend_decode(plain, *s, st) for s in sets])
+        yield line(f"the kernel without extras, decode {S}x{ctx}", ms, S * ctx * 4 * 256 * 2)
+        ms = graph_ms([lambda s=s: vb.paged_attention(s[0].view(S, 16, 128), s[1], s[2], st.query_start_loc, st.context_lens,
+                                                      st.block_tables, 128 ** -0.5, 1) for s in sets])
+        yield line(f"paged_attn 128/128 decode {S}x{ctx}", ms, S * ctx * 4 * 256 * 2, like=f"sigmoid attention decode {S}x{ctx}")
+        del sets
+        torch.cuda.empty_cache()
+        for name, m in (("latent_tc without a rotated part", lw), ("latent_tc with one", olw)):
+            sets = [(rn(S, 16, m.row_width), rn(blocks, DK_PAGE, m.row_width), torch.empty(S, 16, m.R, device=device, dtype=BF))
+                    for _ in range(4)]
+            ms = graph_ms([lambda s=s: la.latent_attn_tc(m, *s, st) for s in sets])
+            yield line(f"{name} {S}x{ctx}", ms, S * ctx * m.row_width * 2,
+                       like=None if m is lw else f"latent_tc without a rotated part {S}x{ctx}")
+            del sets
+            torch.cuda.empty_cache()
+    # attention of prompts
+    for S, new, total in ((4, 2048, 2048), (1, 2048, 8192)):
+        st, blocks = hybrid_step([(new, total)] * S, DK_PAGE, device)
+        T = S * new
+        q, kc, vc = rn(T, 16 * 128), rn(blocks, DK_PAGE, 4, 128), rn(blocks, DK_PAGE, 4, 128)
+        out, longs = torch.empty(T, 16 * 128, device=device, dtype=BF), wa._long_sequences(st, device)[0]
+        pairs = lambda win, keep=0: S * sum(min(t + 1, win + min(keep, max(0, t + 1 - win))) for t in range(total - new, total))   # noqa: E731
+        every = 1 << 30
+        for name, m, win, keep in (("sigmoid attention", left, every, 0), ("windowed attention", aw, PZ_WINDOW, PZ_KEEP),
+                                   ("the kernel with a window alone", plain.__class__(**{**vars(plain), "window": PZ_WINDOW}), PZ_WINDOW, 0),
+                                   ("the kernel without extras", plain, every, 0)):
+            ms = graph_ms([lambda: wa.attend_prefill(m, q, kc, vc, out, st, longs)])
+            yield line(f"{name} prefill {S}x{new}/{total}", ms, None, 2.0 * pairs(win, keep) * 16 * 256)
+        ms = graph_ms([lambda: vb.paged_attention(q.view(T, 16, 128), kc, vc, st.query_start_loc, st.context_lens, st.block_tables,
+                                                  128 ** -0.5, new)])
+        yield line(f"paged_attn 128/128 prefill {S}x{new}/{total}", ms, None, 2.0 * pairs(every) * 16 * 256,
+                   like=f"sigmoid attention prefill {S}x{new}/{total}")
+        for name, m, rot in (("latent gather + up-projection + attention", lw, 0), ("the same with a rotated part", olw, 64)):
+            q, cache, heads = rn(T, 16, 128 + rot), rn(blocks, DK_PAGE, m.row_width), torch.empty(T, 16, 128, device=device, dtype=BF)
+            plan = la._split_plan(st, None, device)[1]
+            ms = graph_ms([lambda: la.latent_expanded(m, q, None, cache, heads, st, plan)])
+            yield line(f"{name} {S}x{new}/{total}", ms, None, 2.0 * pairs(every) * 16 * (256 + rot) + 2.0 * plan[4] * m.w_kv.numel(),
+                       like=f"latent gather + up-projection + attention {S}x{new}/{total}" if rot else None)
+        del q, kc, vc, cache, heads
+        torch.cuda.empty_cache()
+
+
 def main():
     args = parse_args()
     rank = int(os.environ.get("RANK", "0"))
@@ -1451,6 +1668,9 @@ def main():
         return
     if args.tekilix:
         run_tekilix(args)
+        return
+    if args.purozen:
+        run_purozen(args)
         return
     if args.skew:
         run_skew(args, shape)
