@@ -1558,15 +1558,12 @@ def purozen_kernels(device):
                        like="gru_scan (decode) S=64")
             del act
         else:
-            for channels in (16, 32):
-                ms = graph_ms([lambda p=p, s=s, o=o: gru.gru_chunk_scan(right, p, s, o, st, 17, 4, channels)
-                               for p, s, o in zip(proj, states, outs)])
-                yield line(f"gru_chunk T={T}, {channels} channels", ms, nbytes)
+            ms = graph_ms([lambda p=p, s=s, o=o: gru.gru_chunk_scan(right, p, s, o, st, 17) for p, s, o in zip(proj, states, outs)])
+            yield line(f"gru maps + walk T={T}", ms, nbytes)
             lone, _ = hybrid_step([(2048, 8192)], DK_PAGE, device)
-            for channels in (16, 32):
-                ms = graph_ms([lambda p=p, s=s, o=o: gru.gru_chunk_scan(right, p[:2048], s, o[:2048], lone, 17, 1, channels)
-                               for p, s, o in zip(proj, states, outs)])
-                yield line(f"gru_chunk T=2048, one sequence, {channels} channels", ms, 2048 * right.width * 8)
+            ms = graph_ms([lambda p=p, s=s, o=o: gru.gru_chunk_scan(right, p[:2048], s, o[:2048], lone, 17)
+                           for p, s, o in zip(proj, states, outs)])
+            yield line("gru maps + walk T=2048, one sequence", ms, 2048 * right.width * 8)
         del proj, outs, states
         torch.cuda.empty_cache()
         # what lies between the projections and attention

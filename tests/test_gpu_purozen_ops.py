@@ -451,14 +451,13 @@ def _gru_reference(w, proj, start=None):
 def _gru_forms():
     from vexact_b200 import gru
 
-    return {"scan": gru.gru_scan, "rows": gru.gru_rows, "chunk16": lambda *a: gru.gru_chunk_scan(*a, 1, 1, 16),
-            "chunk32": lambda *a: gru.gru_chunk_scan(*a, 1, 1, 32)}
+    return {"scan": gru.gru_scan, "rows": gru.gru_rows, "chunk": lambda *a: gru.gru_chunk_scan(*a, 1)}
 
 
-@pytest.mark.parametrize("form,dtype", [("scan", F32), ("scan", BF), ("rows", F32), ("rows", BF), ("chunk16", BF), ("chunk32", BF)])
+@pytest.mark.parametrize("form,dtype", [("scan", F32), ("scan", BF), ("rows", F32), ("rows", BF), ("chunk", BF)])
 @pytest.mark.parametrize("width", [8, 24, 72, 320, 1032])
 def test_gru_in_portions(form, dtype, width):
-    """Sequences that start, go on in portions of every length (runs and tiles of tokens begin and end anywhere) and sit beside
+    """Sequences that start, go on in portions of every length (runs of tokens begin and end anywhere) and sit beside
     each other; slots that nobody uses keep what they hold."""
     w, run = _gru(width, width), _gru_forms()[form]
     lens, slot_of, done = [700, 90, 33], [3, 0, 4], [0, 0, 0]
@@ -482,9 +481,9 @@ def test_gru_in_portions(form, dtype, width):
     assert done == lens and state[[1, 2, 5]].isnan().all()
 
 
-@pytest.mark.parametrize("form,dtype", [("scan", F32), ("scan", BF), ("chunk16", BF), ("chunk32", BF)])
+@pytest.mark.parametrize("form,dtype", [("scan", F32), ("scan", BF), ("chunk", BF)])
 def test_gru_keeps_a_far_token_and_forgets_at_an_open_gate(form, dtype):
-    """Gates shut but at two tokens: the state of the first lives on over every run and tile until the second replaces it; a
+    """Gates shut but at two tokens: the state of the first lives on over every run until the second replaces it; a
     gate that is wide open keeps nothing, one that is shut takes nothing."""
     from vexact_b200.gru import MinGRUWeights
 
@@ -508,11 +507,11 @@ def test_gru_keeps_a_far_token_and_forgets_at_an_open_gate(form, dtype):
 
 def test_gru_of_a_batch_equals_each_alone_bitwise():
     w, forms = _gru(40, 7), _gru_forms()
-    lens = [(20, 20), (300, 420), (17, 90), (1, 8), (3, 3)]
+    lens = [(20, 20), (700, 820), (17, 90), (1, 8), (3, 3)]
     T = sum(n for n, _ in lens)
     proj, start = _rand(T, 128, seed=1, dtype=BF).cuda(), _rand(7, 40, seed=2).cuda()
     slots = [5, 2, 0, 6, 1]
-    for name in ("rows", "scan", "chunk16"):
+    for name in ("rows", "scan", "chunk"):
         state, out = start.clone(), torch.empty(T, 40, dtype=BF, device=DEV)
         forms[name](w, proj, state, out, hu.step(lens, page=16, slots=slots))
         at = 0

@@ -31,7 +31,7 @@ SIGNATURES = {
     "b200_residual_step": [P, P, LL, LL, P, I, P, LL, P, P, LL, P, LL, LL, I, P, P, P, F, F, P, F, P, F, P, LL, P, P, LL, I, I, I,
                            P],
     "b200_gru_scan": [P, LL, I, I, I, P, P, P, P, LL, P, P, P, I, I, I, F, I, I, I, P],
-    "b200_gru_chunk_scan": [P, LL, I, I, I, P, P, P, P, LL, P, P, P, I, I, I, F, I, I, P],
+    "b200_gru_chunk_scan": [P, LL, I, I, I, P, P, P, P, LL, P, P, P, I, I, I, F, I, I, LL, P, P],
     "b200_delta_scan": [P, LL, P, P, LL, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P],
     "b200_delta_chunk_scan": [P, LL, P, P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P],
     "b200_latent_prep": [P, LL, P, LL, P, LL, P, I, I, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, F, LL, I, P],
@@ -165,7 +165,7 @@ def load() -> C.CDLL:
 
 
 # Kernels launched by one successful call of each entry point (for launch accounting).
-_KERNELS_PER_CALL = {"b200_moe_permute": 2, "b200_lm_head_greedy": 2, "b200_rmsnorm_backward": 3, "b200_ssm_conv2": 2, "b200_latent_attn_tc2": 2, "b200_delta_chunk_scan": 2, "b200_attn_prep2": 2, "b200_status_read": 0, "b200_abi_version": 0}
+_KERNELS_PER_CALL = {"b200_moe_permute": 2, "b200_lm_head_greedy": 2, "b200_rmsnorm_backward": 3, "b200_ssm_conv2": 2, "b200_latent_attn_tc2": 2, "b200_delta_chunk_scan": 2, "b200_gru_chunk_scan": 2, "b200_attn_prep2": 2, "b200_status_read": 0, "b200_abi_version": 0}
 _launches = 0
 
 

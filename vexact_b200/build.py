@@ -23,7 +23,6 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "-shared",
     "-cudart", "static",
     "--expt-relaxed-constexpr",
-    "--split-compile=0",      # functions optimised on every core
 ]
 
 

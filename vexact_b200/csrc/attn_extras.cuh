@@ -80,7 +80,9 @@ __device__ __forceinline__ void sigmoid_pair(float& a, float& b, bool va = true,
   float ea, eb;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(ea) : "f"(fminf(-a, 60.f)));
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(eb) : "f"(fminf(-b, 60.f)));
-  const float da = 1.f + ea, db = 1.f + eb, inv = __fdividef(1.f, da * db);
+  const float da = 1.f + ea, db = 1.f + eb;
+  float inv;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(inv) : "f"(da * db));
   a = va ? db * inv : 0.f;
   b = vb ? da * inv : 0.f;
 }

@@ -411,7 +411,8 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
         const int b = g & 1, s = g % VST;
         const int blk = block_of(t, j);
         const int key0 = blk * ATC_BN + half * 64;        // first key of my half of the block
-        const bool masked = key0 + 63 > cpos || (EXACT && (uint32_t)(cpos - key0) >= reach);
+        // some key of mine is not seen (a half block of kept tokens is, whatever the window)
+        const bool masked = key0 + 63 > cpos || (EXACT && (uint32_t)(cpos - key0) >= reach && !(EXTRAS && key0 + 64 <= keep));
         if (!ptx::mbar_wait_warp(sfull_bar(b), (g >> 1) & 1, abort_flag, 740 + b)) {
           alive = false;
           break;
@@ -429,30 +430,31 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
           tmem_ld32(tm_s0 + b * ATC_BN + lane_addr + half * 64, r0);
           tmem_ld32(tm_s0 + b * ATC_BN + lane_addr + half * 64 + 32, r1);
           ptx::tmem_ld_wait();
+          const float shift = SIGMOID && !(p.extras.cap.cap > 0.f) ? bias : 0.f;
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            v[i] = __uint_as_float(r0[i]) * p.qk_scale;
-            v[32 + i] = __uint_as_float(r1[i]) * p.qk_scale;
+            v[i] = SIGMOID ? fmaf(__uint_as_float(r0[i]), p.qk_scale, shift) : __uint_as_float(r0[i]) * p.qk_scale;
+            v[32 + i] = SIGMOID ? fmaf(__uint_as_float(r1[i]), p.qk_scale, shift) : __uint_as_float(r1[i]) * p.qk_scale;
           }
         }
         if constexpr (EXTRAS) {
-          if (p.extras.cap.cap > 0.f) cap_scores(v, p.extras.cap);
+          if (p.extras.cap.cap > 0.f) {
+            cap_scores(v, p.extras.cap);
+            if constexpr (SIGMOID) {
+#pragma unroll
+              for (int i = 0; i < 64; ++i) v[i] += bias;
+            }
+          }
         }
         if constexpr (SIGMOID) {
           if (masked) {
 #pragma unroll
             for (int i = 0; i < 64; i += 2) {
-              v[i] += bias;
-              v[i + 1] += bias;
               sigmoid_pair(v[i], v[i + 1], key_visible(reach, keep, cpos, key0 + i), key_visible(reach, keep, cpos, key0 + i + 1));
             }
           } else {
 #pragma unroll
-            for (int i = 0; i < 64; i += 2) {
-              v[i] += bias;
-              v[i + 1] += bias;
-              sigmoid_pair(v[i], v[i + 1]);
-            }
+            for (int i = 0; i < 64; i += 2) sigmoid_pair(v[i], v[i + 1]);
           }
           // the block before has been multiplied: its P tile may be overwritten (O stays where it is)
           if (j > 0) {
@@ -464,10 +466,14 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
             if (lane == 0) ptx::mbar_arrive(ofree_bar);
           }
         } else {
-        if (masked) {
+        if (masked && EXTRAS && key0 < keep) {
 #pragma unroll
           for (int i = 0; i < 64; ++i)
-            if (EXACT ? !key_visible(reach, keep, cpos, key0 + i) : key0 + i > cpos) v[i] = -INFINITY;
+            if (!key_visible(reach, keep, cpos, key0 + i)) v[i] = -INFINITY;
+        } else if (masked) {
+#pragma unroll
+          for (int i = 0; i < 64; ++i)
+            if (EXACT ? (uint32_t)(cpos - key0 - i) >= reach : key0 + i > cpos) v[i] = -INFINITY;
         }
         float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll

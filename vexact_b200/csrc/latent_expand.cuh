@@ -174,7 +174,7 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
         }
       }
       // some (row, key) of these is masked
-      const bool edge = base + LEX_SUB - 1 > first_pos || base < warp_full;
+      const bool edge = base + LEX_SUB - 1 > first_pos || (base < warp_full && !(EXTRAS && base + LEX_SUB <= keep));
 #pragma unroll
       for (int t = 0; t < MT; ++t) {
         const int pos0 = first_pos + 16 * t + g4;                 // position of row g4 of the tile (and + 8)

@@ -2,12 +2,13 @@
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Optional
 
 import torch
 
 from . import _lib
 from .ssm import SCAN_MAX_TOKENS
+
+RUN, GROUP = 16, 128     # tokens of a run, and of the runs of a CTA
 
 
 @dataclass
@@ -35,14 +36,13 @@ def gru_scan(w: MinGRUWeights, proj: torch.Tensor, state: torch.Tensor, out: tor
         "b200_gru_scan")
 
 
-def gru_chunk_scan(w: MinGRUWeights, proj: torch.Tensor, state: torch.Tensor, out: torch.Tensor, step, min_len: int,
-                   num_long: int, channels: Optional[int] = None) -> None:
-    """The same in tiles of tokens (bf16), the sequences that bring at least min_len tokens.  `num_long`: how many those are;
-    with few of them a CTA takes fewer channels, so that every SM has some."""
-    if channels is None:
-        channels = 32 if num_long * ((w.width + 31) // 32) >= 148 else 16
+def gru_chunk_scan(w: MinGRUWeights, proj: torch.Tensor, state: torch.Tensor, out: torch.Tensor, step, min_len: int) -> None:
+    """The same in runs of tokens (bf16), the sequences that bring at least min_len tokens."""
+    T, S = proj.shape[0], step.state_slots.numel()
+    maps = torch.empty((T // RUN + T // GROUP + 3 * S, w.width, 2), device=proj.device, dtype=torch.float32)
     _lib.check(
-        _lib.load().b200_gru_chunk_scan(*_where(proj, state, out, step, w), min_len, channels, _lib.current_stream()),
+        _lib.load().b200_gru_chunk_scan(*_where(proj, state, out, step, w), min_len, step.max_seqlen_q, T, maps.data_ptr(),
+                                        _lib.current_stream()),
         "b200_gru_chunk_scan")
 
 
@@ -51,7 +51,6 @@ def gru_rows(w: MinGRUWeights, proj: torch.Tensor, state: torch.Tensor, out: tor
     if step.max_seqlen_q <= SCAN_MAX_TOKENS or proj.dtype != torch.bfloat16:
         gru_scan(w, proj, state, out, step)
         return
-    num_long = sum(n > SCAN_MAX_TOKENS for n, _ in step.seq_lens)
-    gru_chunk_scan(w, proj, state, out, step, SCAN_MAX_TOKENS + 1, num_long)
-    if num_long < len(step.seq_lens):
+    gru_chunk_scan(w, proj, state, out, step, SCAN_MAX_TOKENS + 1)
+    if any(n <= SCAN_MAX_TOKENS for n, _ in step.seq_lens):
         gru_scan(w, proj, state, out, step, 1, SCAN_MAX_TOKENS)
