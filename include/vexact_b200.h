@@ -530,7 +530,7 @@ int b200_attn_prep(const void* proj, long long proj_row_stride, int v_off, const
  *   S = (1 - z) S + z (u >= 0 ? u + 1/2 : sigmoid(u)),  out = S * silu(g) * out_scale;  state [num_slots, width] fp32.
  * _scan: token by token, sequences with min_len .. max_len new tokens.  _chunk_scan: bf16, runs of 16 tokens, sequences with at
  * least min_len (max_new: the most any brings); maps: scratch, num_tokens / 16 + num_tokens /
- * 128 + 3 num_seqs rows of 2 width floats, num_tokens those of the step.  width, offsets and strides multiples of 8. */
+ * 64 + 3 num_seqs rows of 2 width floats, num_tokens those of the step.  width, offsets and strides multiples of 8. */
 int b200_gru_scan(const void* proj, long long proj_row_stride, int z_off, int x_off, int g_off, const void* z_bias_f32,
                   const void* x_bias_f32, void* state_f32, void* out, long long out_row_stride, const void* query_start_loc,
                   const void* context_lens, const void* state_slots, int num_seqs, int num_slots, int width, float out_scale,

@@ -191,7 +191,7 @@ __global__ void __launch_bounds__(GRU_THREADS) gru_scan_kernel(const GruParams p
 
 // ------------------------------------------------------------------ runs of tokens
 // A warp has GRU_CH neighbouring channels (a lane four of them) of a run of GRU_RUN tokens, whose columns it has copied into
-// shared memory, all requested at once. gru_maps_kernel composes the maps S -> a S + b of every run and of
+// shared memory, all requested at once.  gru_maps_kernel composes the maps S -> a S + b of every run and of
 // every group, the GRU_WARPS runs of a CTA; gru_walk_kernel finds the state ahead of its run by applying the maps of the groups
 // before (a CTA's warps share the work) and of the runs between, and walks the tokens.  Runs and groups lie at multiples of
 // their length in a sequence's step and are applied in an order that depends on their number alone.
@@ -199,7 +199,7 @@ __global__ void __launch_bounds__(GRU_THREADS) gru_scan_kernel(const GruParams p
 // maps: rows of [width] (a, b), first those of groups, then those of runs.  Sequence s, t0 its first token of the step, has the
 // group rows from t0 / GRU_GROUP + 2 s, its state at the step's start as the map to a constant and then its groups, and the run
 // rows from t0 / GRU_RUN + s.
-constexpr int GRU_RUN = 16, GRU_WARPS = 8, GRU_CH = 128, GRU_GROUP = GRU_WARPS * GRU_RUN;
+constexpr int GRU_RUN = 16, GRU_WARPS = 4, GRU_CH = 128, GRU_GROUP = GRU_WARPS * GRU_RUN;
 // shared memory of a CTA that copies COLS of the columns z, x, g
 constexpr int gru_smem(int cols) { return GRU_WARPS * GRU_RUN * cols * GRU_CH * 2; }
 
@@ -275,7 +275,7 @@ struct GruMap {
   }
 };
 
-__global__ void __launch_bounds__(GRU_WARPS * 32, 3) gru_maps_kernel(const GruParams p, float2* maps) {
+__global__ void __launch_bounds__(GRU_WARPS * 32, 6) gru_maps_kernel(const GruParams p, float2* maps) {
   extern __shared__ __align__(16) uint8_t gru_raw[];
   pdl_trigger();
   pdl_wait();
@@ -324,7 +324,7 @@ __global__ void __launch_bounds__(GRU_WARPS * 32, 3) gru_maps_kernel(const GruPa
   }
 }
 
-__global__ void __launch_bounds__(GRU_WARPS * 32, 2) gru_walk_kernel(const GruParams p, const float2* maps) {
+__global__ void __launch_bounds__(GRU_WARPS * 32, 4) gru_walk_kernel(const GruParams p, const float2* maps) {
   extern __shared__ __align__(16) uint8_t gru_raw[];
   __shared__ __align__(16) float2 s_map[GRU_WARPS][GRU_CH];      // what the rows of a warp's share of the past compose to
   __shared__ __align__(16) float2 s_own[GRU_WARPS][GRU_CH];      // the maps of this CTA's runs
@@ -339,7 +339,7 @@ __global__ void __launch_bounds__(GRU_WARPS * 32, 2) gru_walk_kernel(const GruPa
   GruBias bias;
   bias.load(p, r.cc);
   const float2* row = maps + r.start * p.width + r.cc;
-  // the start and the groups before this one, an eighth for each warp
+  // the start and the groups before this one, a share for each warp
   const int past = 1 + (int)blockIdx.y, share = (past + GRU_WARPS - 1) / GRU_WARPS;
   GruMap m, one;
   m.same();
@@ -429,7 +429,7 @@ extern "C" int b200_gru_scan(const void* proj, long long proj_row_stride, int z_
 }
 
 // The same recurrence in runs of 16 tokens (bf16), for the sequences that bring at least min_len tokens (max_new: the most any
-// brings).  maps: scratch, rows of 2 width floats, num_tokens / 128 + 2 num_seqs of them and then num_tokens / 16 + num_seqs,
+// brings).  maps: scratch, rows of 2 width floats, num_tokens / 64 + 2 num_seqs of them and then num_tokens / 16 + num_seqs,
 // num_tokens those of the step.
 extern "C" int b200_gru_chunk_scan(const void* proj, long long proj_row_stride, int z_off, int x_off, int g_off,
                                    const void* z_bias_f32, const void* x_bias_f32, void* state_f32, void* out,

@@ -8,7 +8,7 @@ import torch
 from . import _lib
 from .ssm import SCAN_MAX_TOKENS
 
-RUN, GROUP = 16, 128     # tokens of a run, and of the runs of a CTA
+RUN, GROUP = 16, 64     # tokens of a run, and of the runs of a CTA
 
 
 @dataclass
