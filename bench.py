@@ -1446,11 +1446,11 @@ def purozen_shapes():
     from vexact_b200.inferencer import ModelShape
 
     W, V, scale = 2048, 32768, 128 ** -0.5
-    par = ParallelSpec(AttentionSpec(16, 4, 128, 128, scale, sigmoid=True), MinGRUSpec(2048), 0.6, 0.9)
+    par = ParallelSpec(AttentionSpec(16, 4, 128, 128, scale, sigmoid=True), MinGRUSpec(2048), 0.7, 0.8)
     lat = LatentSpec(16, 128, 0, 128, 512, scale, 1.0, 0, gated=False)
 
     def att(mix):
-        return AttentionSpec(16, 4, 128, 128, scale, window=PZ_WINDOW, keep=PZ_KEEP, rot=RotarySpec(50000.0, 64, True, factor=8.0),
+        return AttentionSpec(16, 4, 128, 128, scale, window=PZ_WINDOW, keep=PZ_KEEP, rot=RotarySpec(50000.0, 64, True, factor=4.0),
                              qk_norm="unit", value_mix=mix)
 
     kinds = [par, att("source"), lat, att("mix"), par, att("mix"), lat, att("mix")]

@@ -46,7 +46,7 @@ CONFIGS = {
     "wide_groups": config([layer(attention(heads=12, kv_heads=1, dim=16, vdim=8, size=1, keep=1, dims=16, v_mix=False), 16),
                            layer(parallel(heads=10, kv_heads=1, dim=72, vdim=80, width=136, left_scale=0.0), 40),
                            layer(attention(heads=9, kv_heads=1, dim=72, vdim=72, size=18, keep=300, dims=20, v_mix=False))], width=64),
-    "wide": config([layer(parallel(heads=4, kv_heads=2, dim=64, vdim=128, width=264), 48),
+    "wide": config([layer(parallel(heads=6, kv_heads=3, dim=72, vdim=112, width=264), 48),
                     layer(attention(heads=4, kv_heads=1, dim=88, vdim=88, size=210, keep=130, dims=44)),
                     layer(latent(heads=3, dim=72, vdim=64, kv_rank=136), 40),
                     layer(attention(heads=2, kv_heads=1, dim=200, vdim=88, size=300, keep=33, dims=200)),

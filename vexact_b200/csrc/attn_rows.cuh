@@ -466,51 +466,51 @@ paged_attn_rows_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
             if (lane == 0) ptx::mbar_arrive(ofree_bar);
           }
         } else {
-        if (masked && EXTRAS && key0 < keep) {
+          if (masked && EXTRAS && key0 < keep) {
 #pragma unroll
-          for (int i = 0; i < 64; ++i)
-            if (!key_visible(reach, keep, cpos, key0 + i)) v[i] = -INFINITY;
-        } else if (masked) {
+            for (int i = 0; i < 64; ++i)
+              if (!key_visible(reach, keep, cpos, key0 + i)) v[i] = -INFINITY;
+          } else if (masked) {
 #pragma unroll
-          for (int i = 0; i < 64; ++i)
-            if (EXACT ? (uint32_t)(cpos - key0 - i) >= reach : key0 + i > cpos) v[i] = -INFINITY;
-        }
-        float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+            for (int i = 0; i < 64; ++i)
+              if (EXACT ? (uint32_t)(cpos - key0 - i) >= reach : key0 + i > cpos) v[i] = -INFINITY;
+          }
+          float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-        for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], v[i]);
-        const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-        s_hmax[b][half][row] = mx;
-        if (!pair_sync()) {
-          alive = false;
-          break;
-        }
-        const float m_new = fmaxf(fmaxf(m_run, kMinMax), fmaxf(mx, s_hmax[b][half ^ 1][row]));
-        alpha = fast_exp2(m_run - m_new);
-        m_run = m_new;
-        if (warp == 4) ATR_STAMP(1, g, 1);   // maxima joined
-        // fold the previous block's O (its PV product has also finished reading the P tile by then)
-        if (j > 0) {
-          if (!ptx::mbar_wait_warp(ofull_bar, (g - 1) & 1, abort_flag, 750)) {
+          for (int i = 0; i < 64; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], v[i]);
+          const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+          s_hmax[b][half][row] = mx;
+          if (!pair_sync()) {
             alive = false;
             break;
           }
-          ptx::tc_fence_after();
-#pragma unroll
-          for (int c = 0; c < 2; ++c) {   // two 16-column loads in flight per wait
-            uint32_t r0[16], r1[16];
-            ptx::tmem_ld16(o_addr + c * 32, r0);
-            ptx::tmem_ld16(o_addr + c * 32 + 16, r1);
-            ptx::tmem_ld_wait();
-#pragma unroll
-            for (int i = 0; i < 16; ++i) {
-              o[c * 32 + i] = (o[c * 32 + i] + __uint_as_float(r0[i])) * alpha;
-              o[c * 32 + 16 + i] = (o[c * 32 + 16 + i] + __uint_as_float(r1[i])) * alpha;
+          const float m_new = fmaxf(fmaxf(m_run, kMinMax), fmaxf(mx, s_hmax[b][half ^ 1][row]));
+          alpha = fast_exp2(m_run - m_new);
+          m_run = m_new;
+          if (warp == 4) ATR_STAMP(1, g, 1);   // maxima joined
+          // fold the previous block's O (its PV product has also finished reading the P tile by then)
+          if (j > 0) {
+            if (!ptx::mbar_wait_warp(ofull_bar, (g - 1) & 1, abort_flag, 750)) {
+              alive = false;
+              break;
             }
+            ptx::tc_fence_after();
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {   // two 16-column loads in flight per wait
+              uint32_t r0[16], r1[16];
+              ptx::tmem_ld16(o_addr + c * 32, r0);
+              ptx::tmem_ld16(o_addr + c * 32 + 16, r1);
+              ptx::tmem_ld_wait();
+#pragma unroll
+              for (int i = 0; i < 16; ++i) {
+                o[c * 32 + i] = (o[c * 32 + i] + __uint_as_float(r0[i])) * alpha;
+                o[c * 32 + 16 + i] = (o[c * 32 + 16 + i] + __uint_as_float(r1[i])) * alpha;
+              }
+            }
+            ptx::tc_fence_before();
+            __syncwarp();
+            if (lane == 0) ptx::mbar_arrive(ofree_bar);
           }
-          ptx::tc_fence_before();
-          __syncwarp();
-          if (lane == 0) ptx::mbar_arrive(ofree_bar);
-        }
         }
         if (warp == 4) ATR_STAMP(1, g, 2);   // folded
         // p = bf16(2^(v - m)), group sums in butterfly order, P half row -> shared memory

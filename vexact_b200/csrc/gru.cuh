@@ -191,10 +191,10 @@ __global__ void __launch_bounds__(GRU_THREADS) gru_scan_kernel(const GruParams p
 
 // ------------------------------------------------------------------ runs of tokens
 // A warp has GRU_CH neighbouring channels (a lane four of them) of a run of GRU_RUN tokens, whose columns it has copied into
-// shared memory, all requested at once.  gru_maps_kernel composes the maps S -> a S + b of every run and of
-// every group, the GRU_WARPS runs of a CTA; gru_walk_kernel finds the state ahead of its run by applying the maps of the groups
-// before (a CTA's warps share the work) and of the runs between, and walks the tokens.  Runs and groups lie at multiples of
-// their length in a sequence's step and are applied in an order that depends on their number alone.
+// shared memory, all requested at once.  gru_maps_kernel composes the maps S -> a S + b of every run and of every group, the
+// GRU_WARPS runs of a CTA; gru_walk_kernel finds the state ahead of its run by applying the maps of the groups before (a CTA's
+// warps share the work) and of the runs between, and walks the tokens.  Runs and groups lie at multiples of their length in a
+// sequence's step and are applied in an order that depends on their number alone.
 //
 // maps: rows of [width] (a, b), first those of groups, then those of runs.  Sequence s, t0 its first token of the step, has the
 // group rows from t0 / GRU_GROUP + 2 s, its state at the step's start as the map to a constant and then its groups, and the run
@@ -228,7 +228,8 @@ template <int COLS>
 __device__ __forceinline__ void gru_fetch(const GruParams& p, const GruRun& r, int n, uint32_t smem) {
   const int lane = threadIdx.x & 31, c = blockIdx.x * GRU_CH + (lane & 15) * 8;
   const bool in = c < p.width;
-  const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(p.proj) + (long long)(r.t0 + r.first) * p.proj_stride + (in ? c : 0);
+  const __nv_bfloat16* src =
+      reinterpret_cast<const __nv_bfloat16*>(p.proj) + (long long)(r.t0 + r.first) * p.proj_stride + (in ? c : 0);
 #pragma unroll
   for (int i = 0; i < GRU_RUN * COLS / 2; ++i) {
     const int row = 2 * i + (lane >> 4), token = row / COLS, col = row - token * COLS;

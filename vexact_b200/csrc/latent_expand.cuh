@@ -202,42 +202,42 @@ __global__ void __launch_bounds__(LEX_THREADS, 1) latent_expand_kernel(const Lat
           }
         } else {
 #pragma unroll
-        for (int j = 0; j < NS; ++j)
+          for (int j = 0; j < NS; ++j)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            float v = s[t][j][e];
-            const uint32_t seen = EXTRAS ? reach[EXTRAS ? t : 0][e >> 1] : (uint32_t)window;   // 0 <= position - key < seen
-            if (edge && !key_visible(seen, keep, pos0 + 8 * (e >> 1), base + 8 * j + 2 * t4 + (e & 1))) v = -INFINITY;
-            s[t][j][e] = v;
-            mb[e >> 1] = fmaxf(mb[e >> 1], v);
+            for (int e = 0; e < 4; ++e) {
+              float v = s[t][j][e];
+              const uint32_t seen = EXTRAS ? reach[EXTRAS ? t : 0][e >> 1] : (uint32_t)window;   // 0 <= position - key < seen
+              if (edge && !key_visible(seen, keep, pos0 + 8 * (e >> 1), base + 8 * j + 2 * t4 + (e & 1))) v = -INFINITY;
+              s[t][j][e] = v;
+              mb[e >> 1] = fmaxf(mb[e >> 1], v);
+            }
+          float alpha[2], sum[2] = {0.f, 0.f};
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            mb[e] = abm_quad_max(mb[e]);
+            alpha[e] = fast_exp2(m[t][e] - mb[e]);
           }
-        float alpha[2], sum[2] = {0.f, 0.f};
+          const bool moved = mb[0] > m[t][0] || mb[1] > m[t][1];
+          m[t][0] = mb[0];
+          m[t][1] = mb[1];
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          mb[e] = abm_quad_max(mb[e]);
-          alpha[e] = fast_exp2(m[t][e] - mb[e]);
-        }
-        const bool moved = mb[0] > m[t][0] || mb[1] > m[t][1];
-        m[t][0] = mb[0];
-        m[t][1] = mb[1];
+          for (int j = 0; j < NS; ++j)
 #pragma unroll
-        for (int j = 0; j < NS; ++j)
+            for (int e = 0; e < 4; ++e) {
+              s[t][j][e] = fast_exp2(s[t][j][e] - m[t][e >> 1]);
+              sum[e >> 1] += s[t][j][e];
+            }
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            s[t][j][e] = fast_exp2(s[t][j][e] - m[t][e >> 1]);
-            sum[e >> 1] += s[t][j][e];
+          for (int e = 0; e < 2; ++e) l[t][e] = l[t][e] * alpha[e] + sum[e];   // the quad's four shares meet at the end
+          if (__any_sync(0xffffffffu, moved)) {                     // otherwise every factor is exactly 1
+#pragma unroll
+            for (int j = 0; j < DV / 8; ++j) {
+              o[t][j][0] *= alpha[0];
+              o[t][j][1] *= alpha[0];
+              o[t][j][2] *= alpha[1];
+              o[t][j][3] *= alpha[1];
+            }
           }
-#pragma unroll
-        for (int e = 0; e < 2; ++e) l[t][e] = l[t][e] * alpha[e] + sum[e];   // the quad's four shares meet at the end
-        if (__any_sync(0xffffffffu, moved)) {                     // otherwise every factor is exactly 1
-#pragma unroll
-          for (int j = 0; j < DV / 8; ++j) {
-            o[t][j][0] *= alpha[0];
-            o[t][j][1] *= alpha[0];
-            o[t][j][2] *= alpha[1];
-            o[t][j][3] *= alpha[1];
-          }
-        }
         }
       }
 #pragma unroll

@@ -1,10 +1,11 @@
 // Grouped-query attention of decoded tokens and short portions over paged per-head keys and values (bf16), optionally
 // inside a window or chunk, with capped scores, a sink in the denominator, an output gate or sigmoid weights
-// (attn_extras.cuh).  Scores and weights are fp32: a weight enters the value product as a bf16 pair hi + lo, whose two products are summed in fp32, and the
-// denominator sums the fp32 weights.  (attn.cuh and its kin round the weights to bf16, as the models they serve do.)
+// (attn_extras.cuh).  Scores and weights are fp32: a weight enters the value product as a bf16 pair hi + lo, whose two
+// products are summed in fp32, and the denominator sums the fp32 weights.  (attn.cuh and its kin round the weights to bf16, as
+// the models they serve do.)
 //
 // One CTA of WARPS warps owns up to 8 columns of one KV head of one sequence, a column being one (token, query head)
-// pair.  Warp w walks every WARPS-th block of 32 keys, from the block that holds the first key any column sees, through a
+// pair.  Warp w walks every WARPS-th block of 32 keys that some column sees (key_blocks), through a
 // ring of stages of its own (TMA boxes of 64 columns, 128-byte swizzle; columns past the head dim arrive as zeros), with
 //     S^T[key, col] = K[key, :] . Q[col, :],      O^T[d, col] += V[key, d]^T . P^T[key, col]          (mma.sync)
 // so no MMA row is padding in decode.  The warps' results meet in shared memory in a fixed order.
@@ -183,45 +184,45 @@ window_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_consta
           sc[mt][2 + j] = b;
         }
     } else {
-    float alpha[2];
+      float alpha[2];
 #pragma unroll
-    for (int j = 0; j < 2; ++j) {
-      float mx = m_run[j];
+      for (int j = 0; j < 2; ++j) {
+        float mx = m_run[j];
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
+        for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-        for (int hh = 0; hh < 2; ++hh) {
-          const int key = key0 + mt * 16 + g + hh * 8;
-          float v = sc[mt][hh * 2 + j];
-          if (!key_visible(reach[j], keep, cpos[j], key)) v = -INFINITY;
-          sc[mt][hh * 2 + j] = v;
-          mx = fmaxf(mx, v);
-        }
-      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
-      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
-      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));
-      alpha[j] = fast_exp2(m_run[j] - mx);
-      m_run[j] = mx;
-      float sum = 0.f;
+          for (int hh = 0; hh < 2; ++hh) {
+            const int key = key0 + mt * 16 + g + hh * 8;
+            float v = sc[mt][hh * 2 + j];
+            if (!key_visible(reach[j], keep, cpos[j], key)) v = -INFINITY;
+            sc[mt][hh * 2 + j] = v;
+            mx = fmaxf(mx, v);
+          }
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));
+        alpha[j] = fast_exp2(m_run[j] - mx);
+        m_run[j] = mx;
+        float sum = 0.f;
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt)
+        for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-        for (int hh = 0; hh < 2; ++hh) {
-          const float e = fast_exp2(sc[mt][hh * 2 + j] - mx);
-          sc[mt][hh * 2 + j] = e;
-          sum += e;
-        }
-      l_run[j] = l_run[j] * alpha[j] + sum;      // this lane's keys; the lanes' shares meet at the end
-    }
-    if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
-#pragma unroll
-      for (int d = 0; d < DV / 16; ++d) {
-        o[d][0] *= alpha[0];
-        o[d][1] *= alpha[1];
-        o[d][2] *= alpha[0];
-        o[d][3] *= alpha[1];
+          for (int hh = 0; hh < 2; ++hh) {
+            const float e = fast_exp2(sc[mt][hh * 2 + j] - mx);
+            sc[mt][hh * 2 + j] = e;
+            sum += e;
+          }
+        l_run[j] = l_run[j] * alpha[j] + sum;      // this lane's keys; the lanes' shares meet at the end
       }
-    }
+      if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+        for (int d = 0; d < DV / 16; ++d) {
+          o[d][0] *= alpha[0];
+          o[d][1] *= alpha[1];
+          o[d][2] *= alpha[0];
+          o[d][3] *= alpha[1];
+        }
+      }
     }
     uint32_t hi[MT][2], lo[MT][2];
 #pragma unroll
@@ -398,8 +399,8 @@ extern "C" int b200_window_attn_prefill(const void* q, long long q_row_stride, c
                                         int max_pages, int page_size, int num_blocks, int num_seqs, const void* seq_ids_i32,
                                         int n, int max_len, int min_len, int window, int chunk, int keep,
                                         float cap, const void* sink_f32, const void* sigmoid_bias_f32, float out_scale,
-                                        const void* gate, long long gate_row_stride, int gate_mode, long long T, int heads, int kv_heads, int DK, int DV, float scale, int form,
-                                        void* stream) {
+                                        const void* gate, long long gate_row_stride, int gate_mode, long long T,
+                                        int heads, int kv_heads, int DK, int DV, float scale, int form, void* stream) {
   using namespace b200;
   LatentExpandParams p{};
   p.seqs = {(const int*)query_start_loc, (const int*)context_lens, (const int*)page_table, page_table_stride, max_pages,

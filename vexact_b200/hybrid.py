@@ -87,7 +87,8 @@ class HybridRunner:
     def forward(self, step: HybridStep, rows: torch.Tensor, after_layer=None) -> torch.Tensor:
         """Final-normed hidden states [R, width] of the packed token `rows` (int32).  `after_layer(run, streams)`: called
         with the residual streams [T, streams, width] a layer leaves (development and tests)."""
-        return (self._forward_residual if self.shape.sandwich or self.shape.pre_norm else self._forward_hyper)(step, rows, after_layer)
+        one_residual = self.shape.sandwich or self.shape.pre_norm
+        return (self._forward_residual if one_residual else self._forward_hyper)(step, rows, after_layer)
 
     def _forward_hyper(self, step, rows, after_layer):
         s, w = self.shape, self.w

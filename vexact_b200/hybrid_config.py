@@ -483,7 +483,7 @@ def _read_purozen(cfg: Mapping) -> HybridShape:
                 mix, values = "source" if source is None else "mix", (m["kv_heads"], m["vdim"])
                 source = source or (i, values)
                 if values != source[1]:
-                    raise ValueError(f"layer {i}: values of {values} heads and columns mixed with layer {source[0]}'s of {source[1]}")
+                    raise ValueError(f"layer {i}: values of {values} heads and columns mixed with {source[1]} of layer {source[0]}")
             mixer = AttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), window=window, keep=keep,
                                   rot=_read_linear_rotary(i, m), qk_norm="unit", value_mix=mix)
         elif e["type"] == "latent_attention":
@@ -561,7 +561,7 @@ def _mixer_tensors(m: MixerSpec, W: int) -> dict:
             t["g"] = (m.heads * (m.vdim if m.gate == "column" else 1), W)
         return dict(t, o=(W, m.heads * m.vdim))
     if isinstance(m, ParallelSpec):
-        return {f"{side}.{k}": v for side, part in (("left", m.left), ("right", m.right)) for k, v in _mixer_tensors(part, W).items()}
+        return {f"{side}.{k}": v for side in ("left", "right") for k, v in _mixer_tensors(getattr(m, side), W).items()}
     if isinstance(m, MinGRUSpec):
         n = m.width
         return {"z": (n, W), "z.b": (n,), "x": (n, W), "x.b": (n,), "g": (n, W), "o": (W, n)}

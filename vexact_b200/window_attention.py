@@ -1,7 +1,7 @@
 """Grouped-query attention over paged per-head keys and values, optionally inside a window (beside the sequence's first tokens)
-or chunk, with capped scores, a sink in the denominator, an output gate or sigmoid weights (`csrc/window_attn.cuh` for decoded tokens and short portions; for long ones the
-exact form of `csrc/attn_rows.cuh`, or the paged form of `csrc/latent_expand.cuh` by head dims; `csrc/latent.cuh` on CUDA
-cores for fp32 models and for dims the tensor-core kernels do not take).
+or chunk, with capped scores, a sink in the denominator, an output gate or sigmoid weights (`csrc/window_attn.cuh` for decoded
+tokens and short portions; for long ones the exact form of `csrc/attn_rows.cuh`, or the paged form of `csrc/latent_expand.cuh`
+by head dims; `csrc/latent.cuh` on CUDA cores for fp32 models and for dims the tensor-core kernels do not take).
 
 Between the projections and attention queries and keys may be convolved, normed and rotated and values mixed with those of
 an earlier layer (`csrc/attn_prep.cuh`); a model that does none of it stores keys and values as they are projected."""
@@ -85,7 +85,8 @@ def _pages(step, cache):
 
 
 def _extras(w: AttentionWeights, gate: Optional[torch.Tensor]):
-    """window, chunk, kept tokens, cap, sink, sigmoid bias, output scale and gate as the kernels take them; gate: rows of the model dtype (w.gate says which kind)."""
+    """window, chunk, kept tokens, cap, sink, sigmoid bias, output scale and gate as the kernels take them; gate: rows of the model
+    dtype (w.gate says which kind)."""
     mode = GATES[w.gate]
     if (gate is None) != (mode == 0):
         raise ValueError(f"attention with gate {w.gate!r}: gate rows {'are' if gate is None else 'are not'} wanted")
